@@ -26,8 +26,11 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
               "-Xcompiler", "-fPIC,-fvisibility=hidden", "--expt-relaxed-constexpr", "-Xptxas", "-v"]
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-Wextra", "-Wno-unused-parameter"]
 
-BACKEND_CU = ["src/backends/b200/efm_b200.cu", "src/layers/qwen_text.cu", "src/backends/b200/vit_b200.cu", "src/backends/b200/vla_b200.cu",
-              "src/backends/b200/nccl_glue.cpp"]
+# model-independent part of the backend, then one group per model family
+CORE_CU = ["src/backends/b200/efm_b200.cu", "src/layers/gemm_launch.cu", "src/layers/attention_launch.cu", "src/backends/b200/nccl_glue.cpp"]
+QWEN_CU = ["src/backends/b200/qwen_b200.cu", "src/layers/qwen_text.cu", "src/backends/b200/ops_b200.cu", "src/backends/b200/vit_b200.cu"]
+VLA_CU = ["src/backends/b200/vla_b200.cu"]
+BACKEND_CU = CORE_CU + QWEN_CU + VLA_CU
 ENGINE_CPP = sorted(glob.glob(os.path.join(HERE, "src", "engine", "*.cpp"))) + \
     [os.path.join(HERE, "src", "edge-fm.cpp"), os.path.join(HERE, "src", "tensor.cpp")]
 
@@ -84,7 +87,7 @@ def build_backend(force=False) -> str:
         _run([NVCC, *NVCC_FLAGS, "-I", os.path.join(ROOT, "include"), "-c", os.path.join(HERE, rel), "-o", obj],
              log=obj + ".log")
         return obj
-    with ThreadPoolExecutor(max_workers=4) as ex:
+    with ThreadPoolExecutor(max_workers=8) as ex:
         objs = list(ex.map(compile_one, BACKEND_CU))
     _run([NVCC, "-shared", "-o", out, *objs, "-gencode", "arch=compute_100a,code=sm_100a", "-lcudart", "-ldl"])
     return out

@@ -90,7 +90,31 @@ struct PrefillGraph {
 };
 }  // namespace efm
 
+namespace efm {
+struct Launcher;
+struct DecoderModel;
+// What a model family plugs into the model-independent C ABI (efm_b200.cu).  Null members: not supported by the family.
+struct ModelOps {
+    efm_status (*set_weight)(efm_b200_ctx* c, const char* name, const void* data, const int64_t* shape, int32_t ndim, int32_t dtype,
+                             int32_t mem_kind);
+    efm_status (*set_decode_weight)(efm_b200_ctx* c, const char* name, const void* data, const int64_t* shape, int32_t ndim, int32_t dtype,
+                                    int32_t mem_kind);
+    efm_status (*finalize)(efm_b200_ctx* c);
+    efm_status (*alloc_slot)(efm_b200_ctx* c, int32_t slot, int32_t max_tokens);
+    // before the launches of a prefill / decode pass (host checks, per-request device copies); may be null
+    efm_status (*prefill_begin)(efm_b200_ctx* c, int32_t slot_id, KvSlot& slot, int n_tokens, int kv_offset, int n_embeds);
+    efm_status (*decode_begin)(efm_b200_ctx* c, KvSlot& slot, int kv_len);
+    void (*prefill_chunk)(efm_b200_ctx& c, KvSlot& slot, int S, int kv_offset, int n_custom, int embed_token_id, bool sample_last, Launcher& L);
+    void (*decode_step)(efm_b200_ctx& c, KvSlot& slot, Launcher& L);
+    void (*gather_logits)(efm_b200_ctx& c, Launcher& L);          // before a read-back, when the logits are spread over ranks
+    int64_t (*step_bytes)(const efm_b200_ctx& c, int32_t kv_len);
+    void (*destroy)(efm_b200_ctx* c);
+};
+}  // namespace efm
+
 struct efm_b200_ctx {
+    const efm::ModelOps* ops = nullptr;
+    efm::DecoderModel* decoder = nullptr; // layered-decoder family (decoder_b200.cu); null for the Qwen text tower
     efm_model_desc d{};                   // geometry as THIS RANK sees it (heads / MLP columns already sharded)
     efm_model_desc full{};                // geometry of the whole model (weight slicing)
     // tensor parallel layout: attention is sharded att_shards ways (each shard held by att_rep ranks,

@@ -12,9 +12,12 @@
 #include "../operators/sage_attention.cuh"
 #include "../operators/gemm_tc.cuh"
 #include "../operators/prefill.cuh"
+#define EFM_DECLARATIONS_ONLY
 #include "../operators/sample.cuh"
+#undef EFM_DECLARATIONS_ONLY
 #include "../backends/b200/nccl_glue.h"
 #include "launch.cuh"
+#include "tensor_map.h"
 
 namespace efm {
 
@@ -48,45 +51,6 @@ static void tp_all_reduce(efm_b200_ctx& c, Launcher& L, const float* send, float
 static void tp_all_gather(efm_b200_ctx& c, Launcher& L, const float* send, float* recv, size_t count);
 static void launch_sample_only(efm_b200_ctx& c, Launcher& L, int n_part, int advance);
 bool tp_greedy_exchange(const efm_b200_ctx& c);
-
-// Widest cluster the sampler can run with on this device: 16, 8, ... or 1 (single block; also with
-// EFM_B200_SAMPLER_CLUSTER=1).  Found once, outside any stream capture.
-static int g_sampler_cluster = -1;
-
-cudaError_t configure_sampler() {
-    if (g_sampler_cluster >= 0) return cudaSuccess;
-    int best = 1;
-    const bool wide = cudaFuncSetAttribute(sample_kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess;
-    for (int cs = wide ? 16 : 8; cs >= 2; cs >>= 1) {
-        cudaLaunchConfig_t cfg = {};
-        cfg.gridDim = dim3(cs, 1, 1);
-        cfg.blockDim = dim3(1024);
-        cudaLaunchAttribute at;
-        at.id = cudaLaunchAttributeClusterDimension;
-        at.val.clusterDim.x = (unsigned)cs;
-        at.val.clusterDim.y = at.val.clusterDim.z = 1;
-        cfg.attrs = &at;
-        cfg.numAttrs = 1;
-        int n = 0;
-        if (cudaOccupancyMaxActiveClusters(&n, sample_kernel, &cfg) == cudaSuccess && n >= 1) { best = cs; break; }
-    }
-    (void)cudaGetLastError();
-    if (const char* env = std::getenv("EFM_B200_SAMPLER_CLUSTER")) {
-        const int v = std::atoi(env);
-        if (v >= 1) { int cs = 1; while (cs * 2 <= v && cs * 2 <= best) cs *= 2; best = cs; }
-    }
-    g_sampler_cluster = best;
-    return cudaSuccess;
-}
-
-// Greedy decoding needs one block (the arg-max of the logits pass's partial maxima); top-p sampling
-// spreads its passes over the vocabulary across one cluster.
-void launch_sample(Launcher& L, const SampleParams& p) {
-    if (g_sampler_cluster < 0) (void)configure_sampler();
-    const int cs = (p.temperature >= 1e-6f && p.xchg != nullptr) ? g_sampler_cluster : 1;
-    L.cluster_x = cs;
-    L.launch(sample_kernel, dim3(cs), dim3(1024), 0, p);
-}
 
 void launch_lm_head_and_sample(efm_b200_ctx& c, Launcher& L, const float* resid_row, int advance, bool decode_pass) {
     const efm_model_desc& d = c.d;
@@ -416,270 +380,6 @@ void qwen_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L) {
     launch_lm_head_and_sample(c, L, c.resid_d, /*advance=*/1, /*decode_pass=*/true);
 }
 
-// ---- tensor maps for the TMA-fed GEMM --------------------------------------------------------
-typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                                  const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                  CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-static EncodeTiledFn encode_tiled_fn() {
-    static EncodeTiledFn fn = [] {
-        void* f = nullptr;
-        cudaDriverEntryPointQueryResult st;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &f, cudaEnableDefault, &st) != cudaSuccess ||
-            st != cudaDriverEntryPointSuccess)
-            f = nullptr;
-        return reinterpret_cast<EncodeTiledFn>(f);
-    }();
-    return fn;
-}
-
-// bf16 row-major [rows, cols] tensor, box = 64 columns x box_rows rows, 128-byte swizzle, zero fill
-// outside the tensor.
-static bool make_tile_map(CUtensorMap* map, const void* ptr, int rows, int cols, int row_stride, int box_rows) {
-    EncodeTiledFn fn = encode_tiled_fn();
-    if (fn == nullptr) return false;
-    const cuuint64_t gdim[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
-    const cuuint64_t gstride[1] = {(cuuint64_t)row_stride * 2};
-    const cuuint32_t box[2] = {(cuuint32_t)tc::BK, (cuuint32_t)box_rows};
-    const cuuint32_t estride[2] = {1, 1};
-    return fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), gdim, gstride, box, estride,
-              CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
-}
-
-// fewest 64-wide k-blocks a split may get (EFM_B200_GEMM_MIN_KB overrides, for measurements)
-static int min_kb_per_split() {
-    static int v = [] { const char* e = std::getenv("EFM_B200_GEMM_MIN_KB"); const int x = e != nullptr ? std::atoi(e) : 0; return x >= 1 ? x : 4; }();
-    return v;
-}
-
-// EFM_B200_GEMM_TAIL=0 switches the tail split off (for A/B timing)
-static bool tail_split_enabled() {
-    static const bool on = [] { const char* e = std::getenv("EFM_B200_GEMM_TAIL"); return e == nullptr || e[0] != '0'; }();
-    return on;
-}
-
-template <GemmEpi EPI>
-static void launch_gemm(Launcher& L, const GemmParams& p, int* error_word = nullptr) {
-    static bool attr_set = false;
-    if (!attr_set) {
-        cudaFuncSetAttribute(gemm_tc_kernel<EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)tc::SMEM_BYTES);
-        attr_set = true;
-    }
-    CUtensorMap ma, mb;
-    if (!make_tile_map(&ma, p.A, p.M, p.K, p.lda > 0 ? p.lda : p.K, tc::BM) || !make_tile_map(&mb, p.B, p.N, p.K, p.K, tc::BN)) {
-        if (L.err == cudaSuccess) L.err = cudaErrorInvalidValue;
-        return;
-    }
-    const int tiles = ((p.N + tc::BN - 1) / tc::BN) * ((p.M + tc::BM - 1) / tc::BM);
-    const dim3 block(tc::kThreads);
-    const bool pdl = L.pdl;
-    L.pdl = false;     // prefill kernels do not use the dependent-launch protocol
-    // Few output tiles and a long K: split K so that the whole GPU works, fp32 partials to the workspace, then
-    // a fixed-order sum with the epilogue.
-    if constexpr (EPI == GemmEpi::Bf16Bias || EPI == GemmEpi::Residual || EPI == GemmEpi::F32 || EPI == GemmEpi::SwiGlu) {
-        const int KB = (p.K + tc::BK - 1) / tc::BK;
-        int splits = std::min(L.num_sms / std::max(1, tiles), KB / min_kb_per_split());
-        if (L.gemm_ws != nullptr && splits >= 2 && (p.N & 3) == 0 && (EPI != GemmEpi::SwiGlu || (p.N & 127) == 0) &&
-            (size_t)splits * p.M * p.N <= L.gemm_ws_floats) {
-            const int per = (KB + splits - 1) / splits;
-            splits = (KB + per - 1) / per;                 // no empty split
-            GemmParams q = p;
-            q.kb_per_split = per;
-            q.Cf = L.gemm_ws;
-            q.bias = nullptr;
-            static bool attr_f32 = false;
-            if (!attr_f32) {
-                cudaFuncSetAttribute(gemm_tc_kernel<GemmEpi::F32>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)tc::SMEM_BYTES);
-                attr_f32 = true;
-            }
-            L.launch(gemm_tc_kernel<GemmEpi::F32>, dim3(std::min(L.num_sms, tiles * splits)), block, tc::SMEM_BYTES, ma, mb, q, error_word);
-            const size_t total4 = (size_t)p.M * p.N / (EPI == GemmEpi::SwiGlu ? 8 : 4);
-            const int fin = (int)std::min<size_t>((total4 + 255) / 256, (size_t)L.num_sms * 4);
-            L.launch(gemm_splitk_finish_kernel<EPI>, dim3(fin), dim3(256), 0, (const float*)L.gemm_ws, splits, p);
-            L.pdl = pdl;
-            return;
-        }
-    }
-    // Tail split: a few tiles more than a multiple of the SM count would cost a whole extra round in which most SMs
-    // idle (1324 x 3584 outputs = 154 tiles on 148 SMs: two rounds for 1.04 rounds of work).  The full rounds run as
-    // they are; the remaining tiles are cut along K into as many slices as fill the GPU once (compact fp32 slots in
-    // the workspace) and a small kernel sums the slices in order with the epilogue.  Worth it only when a tile's K
-    // loop is long against the two extra launches (about 12 us).
-    if constexpr (EPI == GemmEpi::Bf16Bias || EPI == GemmEpi::Residual || EPI == GemmEpi::F32) {
-        const int P = L.num_sms, rounds = tiles / P, rem = tiles % P;
-        const int KB = (p.K + tc::BK - 1) / tc::BK;
-        if (tail_split_enabled() && L.gemm_ws != nullptr && rounds >= 1 && rem > 0 && rem * 2 <= P && (p.N & 3) == 0 && p.kb_per_split == 0 &&
-            p.tile_count == 0) {
-            int splits = std::min(P / rem, KB / min_kb_per_split());
-            const int per = splits >= 2 ? (KB + splits - 1) / splits : KB;
-            splits = (KB + per - 1) / per;
-            const double tile_us = KB * 0.45, gain_us = tile_us * (1.0 - 1.0 / std::max(1, splits)) - 12.0;
-            if (splits >= 2 && gain_us > 5.0 && (size_t)splits * rem * tc::BM * tc::BN <= L.gemm_ws_floats) {
-                GemmParams full = p;
-                full.tile_begin = 0;
-                full.tile_count = rounds * P;
-                L.launch(gemm_tc_kernel<EPI>, dim3(P), block, tc::SMEM_BYTES, ma, mb, full, error_word);
-                GemmParams q = p;
-                q.tile_begin = rounds * P;
-                q.tile_count = rem;
-                q.kb_per_split = per;
-                q.Cf = L.gemm_ws;
-                q.bias = nullptr;
-                static bool attr_f32 = false;
-                if (!attr_f32) {
-                    cudaFuncSetAttribute(gemm_tc_kernel<GemmEpi::F32>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)tc::SMEM_BYTES);
-                    attr_f32 = true;
-                }
-                L.launch(gemm_tc_kernel<GemmEpi::F32>, dim3(std::min(P, rem * splits)), block, tc::SMEM_BYTES, ma, mb, q, error_word);
-                const int per_tile = std::max(1, std::min(32, (P * 4) / rem));
-                L.launch(gemm_tail_finish_kernel<EPI>, dim3(per_tile, rem), dim3(256), 0, (const float*)L.gemm_ws, splits, rounds * P, rem, p);
-                L.pdl = pdl;
-                return;
-            }
-        }
-    }
-    L.launch(gemm_tc_kernel<EPI>, dim3(std::min(L.num_sms, tiles)), block, tc::SMEM_BYTES, ma, mb, p, error_word);
-    L.pdl = pdl;
-}
-
-void launch_gemm_bf16(Launcher& L, const GemmParams& p) { launch_gemm<GemmEpi::Bf16Bias>(L, p); }
-
-void launch_rmsnorm_rows(Launcher& L, const float* x, const __nv_bfloat16* w, __nv_bfloat16* y, int rows, int hidden, float eps) {
-    const bool pdl = L.pdl;
-    L.pdl = pdl && L.pdl_rows;
-    // many short rows (vision tower, action model): one warp per row; otherwise one block per row
-    if (hidden <= 2048 && (hidden & 3) == 0 && rows >= 256)
-        L.launch(rmsnorm_rows_warp_kernel, dim3((rows + 7) / 8), dim3(256), 0, x, w, y, rows, hidden, eps);
-    else
-        L.launch(rmsnorm_rows_kernel, dim3(rows), dim3(256), 0, x, w, y, hidden, eps);
-    L.pdl = pdl;
-}
-
-void launch_gemm_epi(Launcher& L, GemmEpi epi, const GemmParams& p, int* error_word) {
-    switch (epi) {
-        case GemmEpi::Bf16Bias: launch_gemm<GemmEpi::Bf16Bias>(L, p, error_word); break;
-        case GemmEpi::Residual: launch_gemm<GemmEpi::Residual>(L, p, error_word); break;
-        case GemmEpi::F32: launch_gemm<GemmEpi::F32>(L, p, error_word); break;
-        case GemmEpi::Bf16Gelu: launch_gemm<GemmEpi::Bf16Gelu>(L, p, error_word); break;
-        case GemmEpi::Bf16GeluTanh: launch_gemm<GemmEpi::Bf16GeluTanh>(L, p, error_word); break;
-        case GemmEpi::SwiGlu: launch_gemm<GemmEpi::SwiGlu>(L, p, error_word); break;
-    }
-}
-
-template <int D, int NW>
-static void launch_seg_attention_dn(Launcher& L, const SegAttnParams& p) {
-    static bool attr_set = false;
-    if (!attr_set) {
-        cudaFuncSetAttribute(seg_attention_kernel<D, NW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sa::smem_bytes<D, NW>());
-        attr_set = true;
-    }
-    const dim3 grid((p.S + 16 * NW - 1) / (16 * NW), p.q_heads), block(32 * NW);
-    const bool pdl = L.pdl;
-    L.pdl = pdl && L.pdl_rows;
-    L.launch(seg_attention_kernel<D, NW>, grid, block, sa::smem_bytes<D, NW>(), p);
-    L.pdl = pdl;
-}
-
-template <int D>
-static void launch_seg_attention_d(Launcher& L, const SegAttnParams& p) {
-    // 64-query blocks: 128-query blocks (NW 8) measured 1-2 % slower on B200 at 1324 and 4784 rows (register-bound
-    // occupancy does not improve with them)
-    launch_seg_attention_dn<D, 4>(L, p);
-}
-
-void launch_seg_attention(Launcher& L, const SegAttnParams& p, int D);
-// Head dim 64, at most 64 queries and at most 320 keys per block (the action expert's attention): every key of the
-// block is requested at once.  Anything else goes to the streaming kernel.
-void launch_seg_attention_short(Launcher& L, const SegAttnParams& p, int D, int max_keys) {
-    constexpr int PRE = 5;
-    if (D != 64 || p.S <= 0 || p.S > 64 || max_keys > PRE * sa::BKV) { launch_seg_attention(L, p, D); return; }
-    static bool attr_set = false;
-    if (!attr_set) {
-        cudaFuncSetAttribute(seg_attention_kernel<64, 4, PRE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sa::smem_bytes<64, 4, PRE>());
-        attr_set = true;
-    }
-    const bool pdl = L.pdl;
-    L.pdl = pdl && L.pdl_rows;
-    L.launch(seg_attention_kernel<64, 4, PRE>, dim3(1, p.q_heads), dim3(128), sa::smem_bytes<64, 4, PRE>(), p);
-    L.pdl = pdl;
-}
-
-// bf16 tensor of up to three dimensions for TMA: dims / box innermost first, byte strides of dimensions 1 and 2.
-static bool make_map_nd(CUtensorMap* map, const void* ptr, int rank, const uint64_t* dims, const uint64_t* strides_bytes,
-                        const uint32_t* box, CUtensorMapDataType dtype = CU_TENSOR_MAP_DATA_TYPE_BFLOAT16) {
-    EncodeTiledFn fn = encode_tiled_fn();
-    if (fn == nullptr) return false;
-    cuuint64_t gdim[3], gstride[2];
-    cuuint32_t bx[3], estride[3] = {1, 1, 1};
-    for (int i = 0; i < rank; ++i) { gdim[i] = dims[i]; bx[i] = box[i]; }
-    for (int i = 0; i + 1 < rank; ++i) gstride[i] = strides_bytes[i];
-    return fn(map, dtype, (cuuint32_t)rank, const_cast<void*>(ptr), gdim, gstride, bx, estride,
-              CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
-}
-
-static bool attention_tc_enabled() {
-    static const bool on = [] { const char* e = std::getenv("EFM_B200_ATTN_TC"); return e == nullptr || e[0] != '0'; }();
-    return on;
-}
-
-// tcgen05 / TMEM form (attention_tc.cuh).
-template <int D>
-static bool launch_seg_attention_tc_d(Launcher& L, const SegAttnParams& p0) {
-    using C = at::Cfg<D>;
-    static bool attr_set = false;
-    if (!attr_set) {
-        cudaFuncSetAttribute(seg_attention_tc_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)C::SMEM);
-        attr_set = true;
-    }
-    const SegAttnParams& p = p0;
-    CUtensorMap mq, mk, mv;
-    const uint64_t qd[3] = {(uint64_t)D, (uint64_t)p.q_heads, (uint64_t)p.S}, qs[2] = {(uint64_t)D * 2, (uint64_t)p.q_stride * 2};
-    const uint64_t kd[3] = {(uint64_t)D, (uint64_t)p.kv_heads, (uint64_t)p.kv_rows}, ks[2] = {(uint64_t)D * 2, (uint64_t)p.kv_stride * 2};
-    const uint32_t qb[3] = {64, 1, (uint32_t)at::BM}, kb[3] = {64, 1, (uint32_t)at::BN};
-    if (!make_map_nd(&mq, p.q, 3, qd, qs, qb) || !make_map_nd(&mk, p.k, 3, kd, ks, kb) || !make_map_nd(&mv, p.v, 3, kd, ks, kb)) return false;
-    const bool pdl = L.pdl;
-    L.pdl = false;
-    L.launch(seg_attention_tc_kernel<D>, dim3((p.S + at::BM - 1) / at::BM, p.q_heads), dim3(at::kThreads), C::SMEM, mq, mk, mv, p, p.error);
-    L.pdl = pdl;
-    return true;
-}
-
-static bool launch_seg_attention_tc(Launcher& L, const SegAttnParams& p, int D) {
-    // TMA needs 16-byte aligned bases and strides; anything else stays on the mma.sync kernel
-    if (p.kv_rows <= 0 || (p.q_stride & 7) || (p.kv_stride & 7) || (reinterpret_cast<uintptr_t>(p.q) & 15) ||
-        (reinterpret_cast<uintptr_t>(p.k) & 15) || (reinterpret_cast<uintptr_t>(p.v) & 15) || (p.out_stride & 7) ||
-        (reinterpret_cast<uintptr_t>(p.out) & 15) || !attention_tc_enabled())
-        return false;
-    if (D == 128) return launch_seg_attention_tc_d<128>(L, p);
-    if (D == 80) return launch_seg_attention_tc_d<80>(L, p);
-    if (D == 64) return launch_seg_attention_tc_d<64>(L, p);
-    return false;
-}
-
-void launch_seg_attention(Launcher& L, const SegAttnParams& p, int D) {
-    if (p.S <= 0) return;
-    if (launch_seg_attention_tc(L, p, D)) return;
-    if (D == 128) launch_seg_attention_d<128>(L, p);
-    else if (D == 80) launch_seg_attention_d<80>(L, p);
-    else if (D == 64) launch_seg_attention_d<64>(L, p);
-    else if (L.err == cudaSuccess) L.err = cudaErrorInvalidValue;
-}
-
-// Causal GQA attention of a prefill chunk: queries at cache rows [kv_offset, kv_offset + S).
-void launch_prefill_attention(Launcher& L, const __nv_bfloat16* q, const __nv_bfloat16* k, const __nv_bfloat16* v,
-                              __nv_bfloat16* out, int S, int kv_offset, int q_heads, int kv_heads, int D, int* error) {
-    SegAttnParams p{};
-    p.q = q; p.k = k; p.v = v; p.out = out;
-    p.q_stride = q_heads * D; p.kv_stride = kv_heads * D; p.out_stride = q_heads * D;
-    p.S = S; p.kv_offset = kv_offset; p.q_heads = q_heads; p.kv_heads = kv_heads;
-    p.scale = 1.0f / sqrtf((float)D);
-    p.kv_rows = kv_offset + S;
-    p.error = error;
-    launch_seg_attention(L, p, D);
-}
-
 template <int D>
 static void launch_sage_d(Launcher& L, const SageAttnParams& p) {
     static bool attr_set = false;
@@ -753,14 +453,13 @@ void qwen_prefill_chunk(efm_b200_ctx& c, KvSlot& slot, int S, int kv_offset, int
     const int H = d.hidden, D = d.head_dim, QD = d.q_heads * D, KVD = d.kv_heads * D, I = d.intermediate;
     const bool pdl = L.pdl;
     L.pdl = false;
-    L.launch(embed_rows_kernel, dim3(S), dim3(128), 0, (const int32_t*)c.ids, (const __nv_bfloat16*)c.embed,
-             (const __nv_bfloat16*)(n_custom > 0 ? c.custom_embeds : nullptr), c.resid, d.vocab, H, embed_token_id, n_custom);
+    launch_embed_rows(L, c.ids, c.embed, n_custom > 0 ? c.custom_embeds : nullptr, c.resid, S, d.vocab, H, embed_token_id, n_custom);
     for (int l = 0; l < d.num_layers; ++l) {
         const LayerWeights& w = c.layers[l];
         launch_rmsnorm_rows(L, c.resid, w.in_norm, c.norm, S, H, d.rms_eps);
         {
             GemmParams g{c.norm, w.qkv, w.qkv_bias, c.qkv, nullptr, S, QD + 2 * KVD, H};
-            launch_gemm<GemmEpi::Bf16Bias>(L, g, &c.state->error);
+            launch_gemm_epi(L, GemmEpi::Bf16Bias, g, &c.state->error);
         }
         L.launch(rope_scatter_kernel, dim3(S), dim3(256), 0,
                  (const __nv_bfloat16*)c.qkv, c.qbuf, slot.k[l], slot.v[l], (const float*)c.inv_freq,
@@ -772,23 +471,23 @@ void qwen_prefill_chunk(efm_b200_ctx& c, KvSlot& slot, int S, int kv_offset, int
             launch_prefill_attention(L, c.qbuf, slot.k[l], slot.v[l], c.attn, S, kv_offset, d.q_heads, d.kv_heads, D, &c.state->error);
         if (c.tp_size == 1) {
             GemmParams g{c.attn, w.o, nullptr, nullptr, c.resid, S, H, QD};
-            launch_gemm<GemmEpi::Residual>(L, g, &c.state->error);
+            launch_gemm_epi(L, GemmEpi::Residual, g, &c.state->error);
         } else {      // row-parallel: this rank's input columns, fp32 partial, all-reduce, then the residual add
             GemmParams g{c.attn + (size_t)c.att_rep_idx * c.o_k, w.o, nullptr, nullptr, c.ybuf, S, H, c.o_k, QD};
-            launch_gemm<GemmEpi::F32>(L, g, &c.state->error);
+            launch_gemm_epi(L, GemmEpi::F32, g, &c.state->error);
             tp_prefill_sum(c, L, S, 0);
         }
         launch_rmsnorm_rows(L, c.resid, w.post_norm, c.norm, S, H, d.rms_eps);
         {     // gate|up with silu(gate) * up in the epilogue
             GemmParams g{c.norm, w.gate_up, nullptr, c.act, nullptr, S, 2 * I, H};
-            launch_gemm<GemmEpi::SwiGlu>(L, g, &c.state->error);
+            launch_gemm_epi(L, GemmEpi::SwiGlu, g, &c.state->error);
         }
         if (c.tp_size == 1) {
             GemmParams g{c.act, w.down, nullptr, nullptr, c.resid, S, H, I};
-            launch_gemm<GemmEpi::Residual>(L, g, &c.state->error);
+            launch_gemm_epi(L, GemmEpi::Residual, g, &c.state->error);
         } else {
             GemmParams g{c.act, w.down, nullptr, nullptr, c.ybuf, S, H, I};
-            launch_gemm<GemmEpi::F32>(L, g, &c.state->error);
+            launch_gemm_epi(L, GemmEpi::F32, g, &c.state->error);
             tp_prefill_sum(c, L, S, 1);
         }
     }
@@ -797,3 +496,4 @@ void qwen_prefill_chunk(efm_b200_ctx& c, KvSlot& slot, int S, int kv_offset, int
 }
 
 }  // namespace efm
+

@@ -3,6 +3,7 @@ module.  No CMake, no network; every output lands in-tree under lib/ and python/
 
     python edge-fm-x_b200/build.py            # build what is out of date
     python edge-fm-x_b200/build.py --force    # rebuild everything
+    python edge-fm-x_b200/build.py --trace-run    # only what bin/trace_run needs
 """
 from __future__ import annotations
 
@@ -27,12 +28,19 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-Wextra", "-Wno-unused-parameter"]
 
 # model-independent part of the backend, then one group per model family
-CORE_CU = ["src/backends/b200/efm_b200.cu", "src/layers/gemm_launch.cu", "src/layers/attention_launch.cu", "src/backends/b200/nccl_glue.cpp"]
-QWEN_CU = ["src/backends/b200/qwen_b200.cu", "src/layers/qwen_text.cu", "src/backends/b200/ops_b200.cu", "src/backends/b200/vit_b200.cu"]
+CORE_CU = ["src/backends/b200/efm_b200.cu", "src/layers/gemm_launch.cu", "src/backends/b200/nccl_glue.cpp"]
+QWEN_CU = ["src/backends/b200/qwen_b200.cu", "src/layers/attention_launch.cu", "src/layers/qwen_text.cu", "src/backends/b200/ops_b200.cu", "src/backends/b200/vit_b200.cu"]
 VLA_CU = ["src/backends/b200/vla_b200.cu"]
-BACKEND_CU = CORE_CU + QWEN_CU + VLA_CU
+DECODER_CU = ["src/backends/b200/decoder_b200.cu", "src/layers/decoder.cu"]
+BACKEND_CU = CORE_CU + DECODER_CU + QWEN_CU + VLA_CU
 ENGINE_CPP = sorted(glob.glob(os.path.join(HERE, "src", "engine", "*.cpp"))) + \
     [os.path.join(HERE, "src", "edge-fm.cpp"), os.path.join(HERE, "src", "tensor.cpp")]
+
+
+# host sources of the trace runner
+TRACE_CPP = ["trace_run.cpp", "tensor.cpp"] + ["engine/" + n + ".cpp" for n in (
+    "compact_vocab", "config", "kv_manager", "model_decoder", "model_registry", "paged_cache", "safetensors", "scheduler", "standard_engine",
+    "step_scheduler")]
 
 
 def _newer(target: str, deps) -> bool:
@@ -73,24 +81,40 @@ def dlpack_include() -> str:
     raise RuntimeError("dlpack/dlpack.h not found in the image")
 
 
-def build_backend(force=False) -> str:
-    os.makedirs(LIB_DIR, exist_ok=True)
-    os.makedirs(OBJ_DIR, exist_ok=True)
-    out = os.path.join(LIB_DIR, "libefm_b200.so")
-    deps = _all_sources()
-    if not force and not _newer(out, deps):
-        return out
-    objs = []
+def _headers():
+    out = []
+    for pat in ("src/**/*.cuh", "src/**/*.h", "include/**/*.h"):
+        out += glob.glob(os.path.join(HERE, pat), recursive=True)
+    return out + glob.glob(os.path.join(ROOT, "include", "*.h"))
 
-    def compile_one(rel):
-        obj = os.path.join(OBJ_DIR, os.path.basename(rel) + ".o")
-        _run([NVCC, *NVCC_FLAGS, "-I", os.path.join(ROOT, "include"), "-c", os.path.join(HERE, rel), "-o", obj],
-             log=obj + ".log")
+
+def _compile_backend(sources, force=False):
+    """Objects of backend sources that are out of date against their own text or any header."""
+    os.makedirs(OBJ_DIR, exist_ok=True)
+    headers = _headers()
+
+    def one(rel):
+        src, obj = os.path.join(HERE, rel), os.path.join(OBJ_DIR, os.path.basename(rel) + ".o")
+        if force or _newer(obj, [src] + headers):
+            tmp = obj + f".{os.getpid()}.tmp"
+            _run([NVCC, *NVCC_FLAGS, "-I", os.path.join(ROOT, "include"), "-c", src, "-o", tmp], log=obj + ".log")
+            os.replace(tmp, obj)
         return obj
     with ThreadPoolExecutor(max_workers=8) as ex:
-        objs = list(ex.map(compile_one, BACKEND_CU))
-    _run([NVCC, "-shared", "-o", out, *objs, "-gencode", "arch=compute_100a,code=sm_100a", "-lcudart", "-ldl"])
+        return list(ex.map(one, sources))
+
+
+def build_backend(force=False) -> str:
+    os.makedirs(LIB_DIR, exist_ok=True)
+    out = os.path.join(LIB_DIR, "libefm_b200.so")
+    objs = _compile_backend(BACKEND_CU, force)
+    if force or _newer(out, objs):
+        _run([NVCC, "-shared", "-o", out, *objs, "-gencode", "arch=compute_100a,code=sm_100a", "-lcudart", "-ldl"])
     return out
+
+
+def _engine_includes():
+    return ["-I", os.path.join(HERE, "include"), "-I", os.path.join(ROOT, "include"), "-I", dlpack_include(), "-I", CUDA_INC]
 
 
 def build_engine(force=False):
@@ -98,8 +122,7 @@ def build_engine(force=False):
     import pybind11
     os.makedirs(PY_DIR, exist_ok=True)
     backend = build_backend(force)
-    inc = ["-I", os.path.join(HERE, "include"), "-I", os.path.join(ROOT, "include"), "-I", dlpack_include(),
-           "-I", CUDA_INC]
+    inc = _engine_includes()
     lib = os.path.join(LIB_DIR, "libedge_fm.so")
     deps = _all_sources()
     if force or _newer(lib, deps):
@@ -114,6 +137,28 @@ def build_engine(force=False):
     return backend, lib, mod
 
 
+def build_trace_run(force=False) -> str:
+    """The trace runner as one executable: the engine and the model families with batched steps, nothing else."""
+    out = os.path.join(OBJ_DIR, "trace_run")
+    cpp = [os.path.join(HERE, "src", r) for r in TRACE_CPP]
+    with ThreadPoolExecutor(max_workers=8) as ex:
+        objs = ex.submit(_compile_backend, CORE_CU + DECODER_CU, force)
+
+        def host(src):
+            obj = os.path.join(OBJ_DIR, "trace_" + os.path.basename(src) + ".o")
+            os.makedirs(OBJ_DIR, exist_ok=True)
+            if force or _newer(obj, [src] + _headers()):
+                _run(["g++", *CXX_FLAGS, "-c", src, "-o", obj, *_engine_includes()])
+            return obj
+        hosts = list(ex.map(host, cpp))
+        objs = objs.result()
+    if force or _newer(out, objs + hosts):
+        tmp = out + f".{os.getpid()}.tmp"
+        _run([NVCC, "-o", tmp, *hosts, *objs, "-gencode", "arch=compute_100a,code=sm_100a", "-ldl", "-lpthread"])
+        os.replace(tmp, out)
+    return out
+
+
 def ptxas_report() -> str:
     out = []
     for f in sorted(glob.glob(os.path.join(OBJ_DIR, "*.log"))):
@@ -123,7 +168,9 @@ def ptxas_report() -> str:
 
 if __name__ == "__main__":
     force = "--force" in sys.argv
-    if "--backend-only" in sys.argv:
+    if "--trace-run" in sys.argv:
+        print(build_trace_run(force))
+    elif "--backend-only" in sys.argv:
         print(build_backend(force))
     else:
         print(build_engine(force))

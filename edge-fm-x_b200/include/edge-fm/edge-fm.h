@@ -9,8 +9,16 @@
 #include <memory>
 #include <string>
 #include <unordered_map>
+#include <vector>
 
 namespace edge_fm {
+
+// One request's share of a batched step: its next tokens, and the places among them whose logits are wanted.
+struct StepEntry {
+    std::string id;
+    std::vector<int32_t> tokens;
+    std::vector<int32_t> want;
+};
 
 class EdgeFM {
 public:
@@ -22,6 +30,15 @@ public:
     // Prefill the non-prefix part of the request, then decode until max_new_tokens or the
     // slot's capacity; stop tokens cut the returned ids on the host afterwards.
     Response generate(const Request& request) const;
+
+    // Batched steps (models on the paged cache; not part of the reference's API).  All entries run as one batch, portions
+    // of prompts beside single decoded tokens; a request is admitted at its first entry and holds its cache pages and
+    // state until finish().  Returns the wanted logits, [wanted, vocab] fp32 in the order of the entries and of `want`.
+    std::vector<float> step(const std::vector<StepEntry>& entries) const;
+    void finish(const std::string& id) const;
+    int32_t vocab_size() const;
+    // Many requests at once with continuous batching over the same steps (request ids need no declared slot).
+    std::vector<Response> generate_batch(const std::vector<const Request*>& requests) const;
 
     // task = trajectory_planning: host tensors "images" f32 [n, 3, S, S], "lang_tokens" i32, "state" f32 and optionally
     // the planner's state tensor (default "current_actions", f32 [chunk, action_dim]) -> {"trajectory": f32 [chunk, action_dim]}.

@@ -57,6 +57,11 @@ struct KvSlot {
     cudaGraphExec_t graph = nullptr;      // decode step captured against this slot's pointers
     int graph_nodes = 0;
     int n_splits = 1, chunk_cap = 1, attn_cluster = 0;
+    // layered decoders: pages come from the context's pool
+    int table = -1, n_pages = 0;          // row of the page table, pages mapped
+    int state_slot = -1;                  // recurrent state of the sequence
+    int len = 0;                          // tokens the cache and state hold
+    int pin_state = -1, pin_len = 0;      // fixed prefix: state after it, its length
 };
 
 // Scratch of the INT8 prefill attention (operators/sage_attention.cuh).

@@ -373,6 +373,7 @@ efm_status efm_b200_decode_steps(efm_b200_ctx* c, int32_t n_steps, int32_t use_g
         Launcher L = make_launcher(c);
         for (int i = 0; i < n_steps; ++i) c->ops->decode_step(*c, s, L);
         if (L.err != cudaSuccess) return cuda_fail(c, L.err, "decode launch");
+        s.len += n_steps;
         return EFM_OK;
     }
     const efm_status st = ensure_graph(c, s);
@@ -384,6 +385,7 @@ efm_status efm_b200_decode_steps(efm_b200_ctx* c, int32_t n_steps, int32_t use_g
                                                     std::to_string(i) + " queued steps");
         EFM_CK(c, cudaGraphLaunch(s.graph, c->stream));
         c->launches += s.graph_nodes;
+        ++s.len;
     }
     return EFM_OK;
 }

@@ -33,6 +33,20 @@ Response EdgeFM::generate(const Request& request) const {
     return impl_->engine->generate(request);
 }
 
+std::vector<float> EdgeFM::step(const std::vector<StepEntry>& entries) const {
+    if (!impl_->engine) throw ConfigurationError("step() is not supported by the active engine (task=trajectory_planning)");
+    return impl_->engine->step(entries);
+}
+void EdgeFM::finish(const std::string& id) const {
+    if (!impl_->engine) throw ConfigurationError("finish() is not supported by the active engine (task=trajectory_planning)");
+    impl_->engine->finish(id);
+}
+int32_t EdgeFM::vocab_size() const { return impl_->engine ? impl_->engine->vocab() : 0; }
+std::vector<Response> EdgeFM::generate_batch(const std::vector<const Request*>& requests) const {
+    if (!impl_->engine) throw ConfigurationError("generate_batch() is not supported by the active engine (task=trajectory_planning)");
+    return impl_->engine->generate_batch(requests);
+}
+
 TensorMap EdgeFM::plan(int32_t request_id, const TensorRefMap& inputs) const {
     if (!impl_->planner) throw ConfigurationError("plan() is not supported by the active engine (task=token_generation)");
     return impl_->planner->plan(request_id, inputs);

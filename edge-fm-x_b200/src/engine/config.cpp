@@ -76,7 +76,15 @@ EngineConfig::EngineConfig(const std::string& config_path) {
         const size_t slash = config_path.find_last_of('/');
         config_dir_ = slash == std::string::npos ? std::string(".") : (slash == 0 ? std::string("/") : config_path.substr(0, slash));
     }
-    const json::Value user = load_json(config_path, "configuration file");
+    apply(load_json(config_path, "configuration file"));
+}
+
+EngineConfig::EngineConfig(const json::Value& user, const std::string& dir) : config_dir_(dir) {
+    config_ = json::parse(kDefaults);
+    apply(user);
+}
+
+void EngineConfig::apply(const json::Value& user) {
     if (!user.is_object()) throw ConfigurationError("configuration file must hold a JSON object");
     for (const auto& kv : user.obj) config_.set(kv.first, kv.second);     // shallow: sections replace wholesale
 
@@ -118,12 +126,8 @@ std::string EngineConfig::model_name() const { return config_.get_string("model_
 std::string EngineConfig::prefill_model_path() const { return config_.get_string("prefill_model_path", ""); }
 std::string EngineConfig::decode_model_path() const { return config_.get_string("decode_model_path", ""); }
 
-std::string EngineConfig::resolved_model_name() const {
-    const std::string n = normalize_model_name(model_name());
-    if (n == "qwen2_5" || n == "qwen2_5_vl") return n;
-    throw ConfigurationError(
-        "Unsupported or missing model_name in engine config. Supported values include: Qwen2.5, qwen2_5, "
-        "Qwen2.5-VL, qwen2_5_vl");
+std::string EngineConfig::checkpoint_architecture() const {
+    return load_json(prefill_model_path() + "/config.json", "config.json file").get_string("architecture", "");
 }
 
 json::Value EngineConfig::prefill_model_config() const {
@@ -150,6 +154,9 @@ int32_t EngineConfig::tp_rank() const {
     return 0;
 }
 std::string EngineConfig::prefill_attention() const { return section("runtime").get_string("prefill_attention", "bf16"); }
+std::string EngineConfig::compute_dtype() const { return section("runtime").get_string("compute_dtype", "bf16"); }
+int32_t EngineConfig::kv_pool_tokens() const { return (int32_t)section("kvcache").get_int("pool_tokens", 0); }
+int32_t EngineConfig::kv_max_live_requests() const { return (int32_t)section("kvcache").get_int("max_live_requests", 4); }
 int32_t EngineConfig::tensor_parallel() const { return (int32_t)section("runtime").get_int("tensor_parallel", 1); }
 bool EngineConfig::lm_head_top1_enabled() const {
     const json::Value rt = section("runtime");

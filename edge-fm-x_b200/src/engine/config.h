@@ -20,13 +20,15 @@ struct KvRequestConfig {
 class EngineConfig {
 public:
     explicit EngineConfig(const std::string& config_path);
+    // The same from a parsed engine JSON; relative names inside are resolved against `dir`.
+    EngineConfig(const json::Value& user, const std::string& dir);
 
     const json::Value& root() const { return config_; }
     const std::string& config_dir() const { return config_dir_; }   // directory of the engine JSON
     json::Value compact_vocab() const { return section("compact_vocab"); }
     std::string task() const;                     // "token_generation" (default) | "trajectory_planning"
     std::string model_name() const;               // as written
-    std::string resolved_model_name() const;      // "qwen2_5" | "qwen2_5_vl" (throws otherwise)
+    std::string checkpoint_architecture() const;  // config.json "architecture" ("" when absent)
     std::string prefill_model_path() const;
     std::string decode_model_path() const;
     json::Value prefill_model_config() const;     // text_config unwrapped for VLM checkpoints
@@ -38,6 +40,9 @@ public:
     std::string tp_rendezvous() const;            // runtime.tp_rendezvous (new key) or $EFM_TP_RENDEZVOUS: fresh shared directory
     int32_t tp_rank() const;                      // $EFM_TP_RANK, else $RANK, else 0
     std::string prefill_attention() const;        // runtime.prefill_attention (new key): "bf16" (default) | "int8"
+    std::string compute_dtype() const;            // runtime.compute_dtype (new key): "bf16" (default) | "fp32"
+    int32_t kv_pool_tokens() const;               // kvcache.pool_tokens (new key): paged-cache tokens for batched steps, default 0
+    int32_t kv_max_live_requests() const;         // kvcache.max_live_requests (new key), default 4
     bool lm_head_top1_enabled() const;            // accepted; the fused argmax is always on here
     std::string kvcache_dtype() const;
     std::string kvcache_attention_type() const;
@@ -54,6 +59,7 @@ public:
     static std::string normalize_model_name(const std::string& raw);
 
 private:
+    void apply(const json::Value& user);
     json::Value section(const std::string& name) const;
     json::Value config_;
     std::string config_dir_;

@@ -27,9 +27,10 @@ AttentionType attention_type_from_string(const std::string& s) {
 KVManager::KVManager(const std::vector<KvRequestConfig>& requests, const KVGeometry& geometry, AttentionType type,
                      int32_t device_id, std::shared_ptr<KVBufferAllocator> allocator)
     : geo_(geometry), type_(type), device_id_(device_id), allocator_(std::move(allocator)) {
-    if (geo_.num_layers <= 0 || geo_.kv_heads <= 0 || geo_.head_dim <= 0)
+    if (geo_.paged) geo_.num_layers = 0;
+    if (!geo_.paged && (geo_.num_layers <= 0 || geo_.kv_heads <= 0 || geo_.head_dim <= 0))
         throw ConfigurationError("KV geometry must be positive");
-    if (requests.empty()) throw ConfigurationError("kvcache.requests must declare at least one slot");
+    if (requests.empty() && !geo_.paged) throw ConfigurationError("kvcache.requests must declare at least one slot");
     const size_t k_stride = (size_t)geo_.kv_heads * geo_.head_dim * get_dtype_size(geo_.dtype);
     for (const KvRequestConfig& r : requests) {
         if (slots_.count(r.request_id)) throw ConfigurationError("duplicate request_id in kvcache.requests: " + std::to_string(r.request_id));
@@ -42,7 +43,7 @@ KVManager::KVManager(const std::vector<KvRequestConfig>& requests, const KVGeome
         s.status.prefix_size = r.prefix_token_ids.size();
         s.status.max_tokens = r.max_tokens;
         const size_t layer_bytes = 2 * (size_t)r.max_tokens * k_stride;
-        s.status.allocated_size = layer_bytes * (size_t)geo_.num_layers;
+        s.status.allocated_size = geo_.paged ? (size_t)r.max_tokens * geo_.token_bytes : layer_bytes * (size_t)geo_.num_layers;
         s.read_ptrs = allocator_->allocate_slot(r.request_id, r.max_tokens, layer_bytes, geo_.num_layers);
         if ((int32_t)s.read_ptrs.size() != geo_.num_layers) throw InternalError("KV allocator returned a wrong layer count");
         for (void* p : s.read_ptrs)
@@ -53,6 +54,7 @@ KVManager::KVManager(const std::vector<KvRequestConfig>& requests, const KVGeome
 }
 
 size_t KVManager::get_token_stride() const {
+    if (geo_.paged) return geo_.token_bytes;
     return 2 * (size_t)geo_.kv_heads * geo_.head_dim * get_dtype_size(geo_.dtype);
 }
 

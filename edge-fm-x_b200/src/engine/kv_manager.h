@@ -35,6 +35,10 @@ enum class AttentionType { MHA, GQA, MQA };
 struct KVGeometry {
     int32_t num_layers = 0, kv_heads = 0, head_dim = 0;
     DType dtype = DType::BFloat16;
+    // Paged models: a slot is a list of pages instead of per-layer buffers (the allocator returns no pointers), layers may
+    // differ; token_bytes is what one token takes over all layers.
+    bool paged = false;
+    size_t token_bytes = 0;
 };
 
 // Where the per-layer buffers come from.  The engine plugs in the device backend; tests plug
@@ -43,7 +47,7 @@ class KVBufferAllocator {
 public:
     virtual ~KVBufferAllocator() = default;
     virtual Device device() const = 0;
-    // Returns num_layers base pointers, each to layer_bytes of zeroed memory.
+    // Returns num_layers base pointers, each to layer_bytes of zeroed memory (paged: none).
     virtual std::vector<void*> allocate_slot(int32_t request_id, int32_t max_tokens, size_t layer_bytes,
                                              int32_t num_layers) = 0;
 };

@@ -1,0 +1,205 @@
+// Layered decoders: config.json -> efm_decoder_desc, checkpoint tensors, paged cache.  A family is a reader of its
+// config.json; everything behind it (mixers, cache, steps) is shared.
+//
+// Folizen: "layers" lists {type, mixer, mlp}; type "attention" {heads, kv_heads, dim, vdim, scale, mask.size} or
+// "general_delta" {heads, dim}; mlp null or {kind: "dense", ff}; "norm.eps", "token_side.dim", "vocab", "width".  Sizes
+// the JSON does not give (rank of the decay projection) are read from the tensors' shapes.
+#include <efm_b200.h>
+
+#include <algorithm>
+#include <cstring>
+#include <map>
+
+#include "model_registry.h"
+#include "safetensors.h"
+
+namespace edge_fm {
+
+namespace {
+
+struct DecoderConfig {
+    efm_decoder_desc desc{};
+    std::vector<efm_decoder_layer> layers;
+};
+using Shapes = std::map<std::string, std::vector<int64_t>>;
+
+const json::Value& member(const json::Value& v, const char* key, const std::string& where) {
+    const json::Value* m = v.find(key);
+    if (m == nullptr) throw ConfigurationError("config.json: " + where + " lacks \"" + key + "\"");
+    return *m;
+}
+int32_t positive(const json::Value& v, const char* key, const std::string& where) {
+    const json::Value& m = member(v, key, where);
+    if (!m.is_number() || m.num <= 0) throw ConfigurationError("config.json: " + where + "." + key + " must be a positive number");
+    return (int32_t)(m.is_int ? m.inum : (int64_t)m.num);
+}
+
+DecoderConfig folizen_config(const json::Value& cfg, const Shapes& shapes) {
+    DecoderConfig out;
+    efm_decoder_desc& d = out.desc;
+    d.struct_size = (int32_t)sizeof(d);
+    d.vocab = positive(cfg, "vocab", "model");
+    d.width = positive(cfg, "width", "model");
+    d.norm_eps = (float)member(member(cfg, "norm", "model"), "eps", "norm").num;
+    const json::Value* side = cfg.find("token_side");
+    if (side != nullptr && side->is_object()) d.side_dim = positive(*side, "dim", "token_side");
+    const json::Value& layers = member(cfg, "layers", "model");
+    if (!layers.is_array() || layers.arr.empty()) throw ConfigurationError("config.json: \"layers\" must be a non-empty list");
+    for (size_t i = 0; i < layers.arr.size(); ++i) {
+        const json::Value& l = layers.arr[i];
+        const std::string where = "layers[" + std::to_string(i) + "]";
+        const json::Value& mix = member(l, "mixer", where);
+        const std::string type = l.get_string("type", "");
+        efm_decoder_layer e{};
+        e.heads = positive(mix, "heads", where + ".mixer");
+        e.dim = positive(mix, "dim", where + ".mixer");
+        if (type == "attention") {
+            e.mixer = EFM_MIXER_ATTENTION;
+            e.kv_heads = positive(mix, "kv_heads", where + ".mixer");
+            e.vdim = positive(mix, "vdim", where + ".mixer");
+            e.scale = (float)member(mix, "scale", where + ".mixer").num;
+            e.distance_bias = 1;
+            const json::Value* mask = mix.find("mask");
+            if (mask != nullptr && mask->is_object()) e.window = positive(*mask, "size", where + ".mixer.mask");
+        } else if (type == "general_delta") {
+            e.mixer = EFM_MIXER_GENERAL_DELTA;
+            const auto it = shapes.find("l" + std::to_string(i) + ".mix.w1");
+            if (it == shapes.end() || it->second.size() != 2) throw ModelNotLoadedError("checkpoint lacks l" + std::to_string(i) + ".mix.w1");
+            e.decay_rank = (int32_t)it->second[0];
+        } else {
+            throw ConfigurationError("config.json: " + where + " has an unknown type \"" + type + "\"");
+        }
+        const json::Value* mlp = l.find("mlp");
+        if (mlp != nullptr && mlp->is_object()) {
+            const std::string kind = mlp->get_string("kind", "");
+            if (kind != "dense") throw ConfigurationError("config.json: " + where + ".mlp has an unknown kind \"" + kind + "\"");
+            e.ff = positive(*mlp, "ff", where + ".mlp");
+        }
+        out.layers.push_back(e);
+    }
+    d.num_layers = (int32_t)out.layers.size();
+    return out;
+}
+
+// Page lists go to the device context; declared slots get their pages once, for good.
+class DevicePageMapper : public PageMapper {
+public:
+    explicit DevicePageMapper(efm_b200_ctx* ctx) : ctx_(ctx) {}
+    void map(int32_t slot, const std::vector<int32_t>& pages, int32_t state_slot) override {
+        check_backend(efm_b200_decoder_map_slot(ctx_, slot, pages.data(), (int32_t)pages.size(), state_slot), ctx_, "mapping cache pages");
+    }
+    void unmap(int32_t slot) override { check_backend(efm_b200_decoder_unmap_slot(ctx_, slot), ctx_, "unmapping cache pages"); }
+
+private:
+    efm_b200_ctx* ctx_;
+};
+
+// Keeps the mapper alive next to the cache that uses it.
+class OwningPagedCache : public PagedCache {
+public:
+    OwningPagedCache(int32_t pages, int32_t states, std::unique_ptr<PageMapper> mapper)
+        : PagedCache(pages, states, mapper.get()), mapper_own_(std::move(mapper)) {}
+
+private:
+    std::unique_ptr<PageMapper> mapper_own_;
+};
+
+class PagedKVAllocator : public KVBufferAllocator {
+public:
+    explicit PagedKVAllocator(std::shared_ptr<PagedCache> cache) : cache_(std::move(cache)) {}
+    Device device() const override { return Device::GPU; }
+    std::vector<void*> allocate_slot(int32_t request_id, int32_t max_tokens, size_t, int32_t) override {
+        if (!cache_->reserve(request_id, max_tokens)) throw OutOfMemoryError("the cache pool has no room for request_id " + std::to_string(request_id));
+        return {};
+    }
+
+private:
+    std::shared_ptr<PagedCache> cache_;
+};
+
+ModelSetup build_decoder(const EngineConfig& config, DecoderConfig (*read)(const json::Value&, const Shapes&)) {
+    const std::vector<std::string> files = collect_safetensors_files(config.prefill_model_path());
+    if (files.empty())
+        throw ConfigurationError("No model.safetensors or model-*-of-*.safetensors found in: " + config.prefill_model_path());
+    std::vector<std::unique_ptr<SafeTensorsFile>> maps;
+    Shapes shapes;
+    for (const std::string& f : files) {
+        maps.emplace_back(new SafeTensorsFile(f));
+        for (const SafeTensorEntry& e : maps.back()->entries()) shapes[e.name] = e.shape;
+    }
+    DecoderConfig dc = read(config.prefill_model_config(), shapes);
+    efm_decoder_desc& d = dc.desc;
+
+    const std::string compute = config.compute_dtype();
+    if (compute != "bf16" && compute != "fp32") throw ConfigurationError("runtime.compute_dtype must be \"bf16\" or \"fp32\", got " + compute);
+    d.compute_dtype = compute == "fp32" ? EFM_F32 : EFM_BF16;
+    const DType cache_dtype = dtype_from_string(config.kvcache_dtype());
+    if (cache_dtype != (compute == "fp32" ? DType::Float32 : DType::BFloat16))
+        throw ConfigurationError("kvcache.dtype must be " + compute + " with runtime.compute_dtype " + compute);
+    if (config.tensor_parallel() != 1) throw ConfigurationError("runtime.tensor_parallel: this model runs on one GPU");
+    if (config.prefill_attention() != "bf16") throw ConfigurationError("runtime.prefill_attention: this model has one form only");
+    const std::string decode_path = config.decode_model_path();
+    if (!decode_path.empty() && decode_path != config.prefill_model_path()) throw ConfigurationError("decode_model_path: this model takes no second checkpoint");
+
+    const std::vector<KvRequestConfig> reqs = config.kv_requests();
+    const int32_t pool = std::max(0, config.kv_pool_tokens()), live = pool > 0 ? std::max(1, config.kv_max_live_requests()) : 0;
+    int64_t pages = PagedCache::pages_for(pool);
+    int32_t longest = pool, states = live;
+    for (const KvRequestConfig& r : reqs) {
+        pages += PagedCache::pages_for(std::max(1, r.max_tokens));
+        longest = std::max(longest, r.max_tokens);
+        states += 1 + (r.prefix_token_ids.empty() ? 0 : 1);
+    }
+    if (pages <= 0) throw ConfigurationError("kvcache declares neither requests nor pool_tokens");
+    const bool recurrent = std::any_of(dc.layers.begin(), dc.layers.end(), [](const efm_decoder_layer& l) { return l.mixer != EFM_MIXER_ATTENTION; });
+    d.cache_pages = (int32_t)pages;
+    d.state_slots = recurrent ? states : 0;
+    d.max_slots = (int32_t)reqs.size() + live;
+    d.max_step_tokens = std::min(PagedCache::pages_for(longest) * kCachePageTokens, 2048);
+    d.max_response_tokens = config.sampling_max_new_tokens() + 1;
+
+    ModelSetup setup;
+    setup.device_id = config.runtime_device_id();
+    setup.hidden = d.width;
+    setup.vocab = d.vocab;
+    setup.max_live_requests = live;
+    setup.max_step_tokens = d.max_step_tokens;
+    const efm_status st = efm_b200_decoder_create(&d, dc.layers.data(), setup.device_id, &setup.ctx);
+    if (st != EFM_OK) {
+        const std::string msg = std::string("backend creation failed: ") + efm_b200_last_error(nullptr);
+        if (st == EFM_ERR_OUT_OF_MEMORY) throw OutOfMemoryError(msg);
+        if (st == EFM_ERR_UNSUPPORTED || st == EFM_ERR_INVALID_ARGUMENT) throw ConfigurationError(msg);
+        throw DeviceError(msg);
+    }
+    try {
+        for (const auto& m : maps)
+            for (const SafeTensorEntry& e : m->entries()) {
+                const int32_t code = backend_dtype_code(e.dtype);
+                if (code < 0) continue;
+                if (efm_b200_set_weight(setup.ctx, e.name.c_str(), e.data, e.shape.data(), (int32_t)e.shape.size(), code, EFM_MEM_HOST) != EFM_OK)
+                    throw ModelNotLoadedError("loading " + e.name + ": " + efm_b200_last_error(setup.ctx));
+            }
+        if (efm_b200_finalize_weights(setup.ctx) != EFM_OK)
+            throw ModelNotLoadedError(std::string("checkpoint incomplete: ") + efm_b200_last_error(setup.ctx));
+        setup.paged_cache = std::make_shared<OwningPagedCache>(d.cache_pages, d.state_slots, std::unique_ptr<PageMapper>(new DevicePageMapper(setup.ctx)));
+        KVGeometry geo;
+        geo.paged = true;
+        geo.dtype = cache_dtype;
+        for (const efm_decoder_layer& l : dc.layers)
+            if (l.mixer == EFM_MIXER_ATTENTION) geo.token_bytes += (size_t)l.kv_heads * (l.dim + l.vdim) * get_dtype_size(cache_dtype);
+        setup.kv_manager = std::make_shared<KVManager>(reqs, geo, attention_type_from_string(config.kvcache_attention_type()), setup.device_id,
+                                                       std::make_shared<PagedKVAllocator>(setup.paged_cache));
+    } catch (...) {
+        efm_b200_destroy(setup.ctx);
+        throw;
+    }
+    return setup;
+}
+
+ModelSetup build_folizen(const EngineConfig& config) { return build_decoder(config, folizen_config); }
+
+const ModelRegistrar kFolizen({"folizen", {"Folizen"}, build_folizen});
+
+}  // namespace
+
+}  // namespace edge_fm

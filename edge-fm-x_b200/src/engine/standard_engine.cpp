@@ -1,7 +1,5 @@
 #include "standard_engine.h"
 
-#include "tp_rendezvous.h"
-
 #include <cuda_runtime.h>
 #include <efm_b200.h>
 
@@ -11,7 +9,7 @@
 #include <cstring>
 #include <unordered_set>
 
-#include "safetensors.h"
+#include "model_registry.h"
 
 namespace edge_fm {
 
@@ -22,199 +20,27 @@ double now_ms() {
     return duration<double, std::milli>(steady_clock::now().time_since_epoch()).count();
 }
 
-// KV buffers live in the backend; the manager only keeps the bookkeeping and the pointers.
-class BackendKVAllocator : public KVBufferAllocator {
-public:
-    explicit BackendKVAllocator(efm_b200_ctx* ctx) : ctx_(ctx) {}
-    Device device() const override { return Device::GPU; }
-    std::vector<void*> allocate_slot(int32_t request_id, int32_t max_tokens, size_t, int32_t num_layers) override {
-        efm_status st = efm_b200_alloc_kv_slot(ctx_, request_id, max_tokens);
-        if (st == EFM_ERR_OUT_OF_MEMORY) throw OutOfMemoryError(efm_b200_last_error(ctx_));
-        if (st != EFM_OK) throw DeviceError(efm_b200_last_error(ctx_));
-        std::vector<void*> out;
-        for (int32_t l = 0; l < num_layers; ++l) {
-            void* p = nullptr;
-            if (efm_b200_kv_layer_ptr(ctx_, request_id, l, &p, nullptr) != EFM_OK) throw InternalError(efm_b200_last_error(ctx_));
-            out.push_back(p);
-        }
-        return out;
-    }
-
-private:
-    efm_b200_ctx* ctx_;
-};
-
-int32_t dtype_code(const std::string& st) {
-    if (st == "BF16") return EFM_BF16;
-    if (st == "F16") return EFM_F16;
-    if (st == "F32") return EFM_F32;
-    if (st == "I32") return EFM_I32;
-    if (st == "I64") return EFM_I64;
-    if (st == "U8") return EFM_U8;
-    if (st == "I8") return EFM_I8;
-    return -1;
-}
-
 }  // namespace
 
-void StandardEngine::check(int32_t st, const char* what) const {
-    if (st == EFM_OK) return;
-    const std::string msg = std::string(what) + ": " + efm_b200_last_error(ctx_);
-    switch (st) {
-        case EFM_ERR_OUT_OF_MEMORY: throw OutOfMemoryError(msg);
-        case EFM_ERR_INVALID_ARGUMENT: throw InvalidRequestError(msg);
-        case EFM_ERR_UNSUPPORTED: throw ConfigurationError(msg);
-        case EFM_ERR_STATE: throw InternalError(msg);
-        default: throw DeviceError(msg);
-    }
-}
+void StandardEngine::check(int32_t st, const char* what) const { check_backend(st, ctx_, what); }
 
 StandardEngine::StandardEngine(const EngineConfig& config) : config_(config) {
     if (device_from_string(config_.runtime_device()) != Device::GPU)
         throw ConfigurationError("token generation needs runtime.device = cuda (there is no CPU path)");
-    const std::string model = config_.resolved_model_name();
-    const json::Value mc = config_.prefill_model_config();
-    device_id_ = config_.runtime_device_id();
+    const ModelFamily& family = ModelRegistry::resolve(config_);
     use_graph_ = config_.use_cuda_graph();
-    if (dtype_from_string(config_.kvcache_dtype()) != DType::BFloat16)
-        throw ConfigurationError("kvcache.dtype must be bf16 for this backend");
-    const AttentionType attn = attention_type_from_string(config_.kvcache_attention_type());
-
-    efm_model_desc d;
-    std::memset(&d, 0, sizeof(d));
-    d.struct_size = (int32_t)sizeof(d);
-    d.num_layers = (int32_t)mc.get_int("num_hidden_layers", 0);
-    d.hidden = (int32_t)mc.get_int("hidden_size", 0);
-    d.q_heads = (int32_t)mc.get_int("num_attention_heads", 0);
-    d.kv_heads = (int32_t)mc.get_int("num_key_value_heads", d.q_heads);
-    d.intermediate = (int32_t)mc.get_int("intermediate_size", 0);
-    d.vocab = (int32_t)mc.get_int("vocab_size", 0);
-    if (d.num_layers <= 0 || d.hidden <= 0 || d.q_heads <= 0 || d.vocab <= 0 || d.intermediate <= 0)
-        throw ConfigurationError("config.json lacks num_hidden_layers / hidden_size / num_attention_heads / vocab_size / intermediate_size");
-    d.head_dim = d.hidden / d.q_heads;      // as the reference derives it (kv_manager.cpp:80)
-    d.rms_eps = (float)mc.get_double("rms_norm_eps", 1e-6);
-    d.rope_theta = (float)mc.get_double("rope_theta", 10000.0);
-    const std::string act = mc.get_string("hidden_act", "silu");
-    if (act != "silu") throw ConfigurationError("hidden_act must be silu, got " + act);
-    const std::string torch_dtype = mc.get_string("torch_dtype", mc.get_string("dtype", "bfloat16"));
-    if (torch_dtype != "bfloat16") throw ConfigurationError("checkpoint dtype must be bfloat16, got " + torch_dtype);
-    const json::Value* rs = mc.find("rope_scaling");
-    if (rs != nullptr && rs->is_object()) {
-        const json::Value* sec = rs->find("mrope_section");
-        if (sec != nullptr && sec->is_array() && sec->arr.size() == 3) {
-            d.use_mrope = 1;
-            for (int i = 0; i < 3; ++i) d.mrope_section[i] = (int32_t)sec->arr[i].inum;
-        }
-    }
-    use_mrope_ = d.use_mrope != 0;
-    hidden_ = d.hidden;
-    vocab_ = d.vocab;
-    if (model == "qwen2_5" && use_mrope_) throw ConfigurationError("model_name Qwen2.5 with an mrope checkpoint: use Qwen2.5-VL");
-
-    // tied lm_head <=> the checkpoint carries no lm_head.weight (reference: src/layers/linear.cu:2244-2248)
-    const std::vector<std::string> files = collect_safetensors_files(config_.prefill_model_path());
-    if (files.empty())
-        throw ConfigurationError("No model.safetensors or model-*-of-*.safetensors found in: " + config_.prefill_model_path());
-    std::vector<std::unique_ptr<SafeTensorsFile>> maps;
-    bool has_lm_head = false;
-    const bool vlm = model == "qwen2_5_vl";
-    for (const std::string& f : files) {
-        maps.emplace_back(new SafeTensorsFile(f));
-        for (const SafeTensorEntry& e : maps.back()->entries()) {
-            std::string name = e.name;
-            if (vlm && !map_vlm_weight_name(e.name, &name)) continue;
-            if (name == "lm_head.weight") has_lm_head = true;
-        }
-    }
-    d.tied_lm_head = has_lm_head ? 0 : 1;
-
-    const std::vector<KvRequestConfig> reqs = config_.kv_requests();
-    int32_t max_tokens = 1;
-    for (const KvRequestConfig& r : reqs) max_tokens = std::max(max_tokens, r.max_tokens);
-    d.max_prefill_tokens = std::min(max_tokens, 2048);
-    d.max_response_tokens = config_.sampling_max_new_tokens() + 1;
-
-    // Tensor parallel: one process per GPU, every process builds the same engine and issues the same requests.
-    // Rank from the environment, device = $LOCAL_RANK (else runtime.device_id + rank), host exchange through files.
-    const int32_t tp = config_.tensor_parallel();
-    if (tp < 1 || tp > 8) throw ConfigurationError("runtime.tensor_parallel must be between 1 and 8");
-    const int32_t tp_rank = tp > 1 ? config_.tp_rank() : 0;
-    std::unique_ptr<TpRendezvous> meet;
-    if (tp > 1) {
-        if (tp_rank < 0 || tp_rank >= tp) throw ConfigurationError("tensor parallel rank (EFM_TP_RANK / RANK) must be in [0, runtime.tensor_parallel)");
-        const char* local = std::getenv("LOCAL_RANK");
-        device_id_ = local != nullptr && local[0] != 0 ? std::atoi(local) : device_id_ + tp_rank;
-        meet.reset(new TpRendezvous(config_.tp_rendezvous(), tp_rank, tp));
-    }
-    efm_status st = efm_b200_create(&d, device_id_, tp_rank, tp, &ctx_);
-    if (st != EFM_OK) {
-        const std::string msg = std::string("backend creation failed: ") + efm_b200_last_error(nullptr);
-        if (st == EFM_ERR_OUT_OF_MEMORY) throw OutOfMemoryError(msg);
-        if (st == EFM_ERR_UNSUPPORTED || st == EFM_ERR_INVALID_ARGUMENT) throw ConfigurationError(msg);
-        throw DeviceError(msg);
-    }
+    ModelSetup m = family.build(config_);
+    ctx_ = m.ctx;
+    device_id_ = m.device_id;
+    hidden_ = m.hidden;
+    vocab_ = m.vocab;
+    use_mrope_ = m.use_mrope;
+    kv_manager_ = m.kv_manager;
+    paged_cache_ = m.paged_cache;
+    max_step_tokens_ = m.max_step_tokens;
     try {
-        if (tp > 1) {
-            std::vector<char> id(128, 0);
-            if (tp_rank == 0) check(efm_b200_tp_unique_id(id.data()), "communicator id");
-            id = meet->broadcast_from_root("nccl_id", id);
-            if (id.size() != 128) throw ConfigurationError("tensor parallel rendezvous: malformed communicator id");
-            check(efm_b200_tp_init(ctx_, id.data()), "communicator initialisation");
-        }
-        for (const auto& m : maps) {
-            for (const SafeTensorEntry& e : m->entries()) {
-                std::string name = e.name;
-                if (vlm && !map_vlm_weight_name(e.name, &name)) continue;
-                const int32_t code = dtype_code(e.dtype);
-                if (code < 0) continue;
-                st = efm_b200_set_weight(ctx_, name.c_str(), e.data, e.shape.data(), (int32_t)e.shape.size(), code, EFM_MEM_HOST);
-                if (st != EFM_OK) throw ModelNotLoadedError(std::string("loading ") + name + ": " + efm_b200_last_error(ctx_));
-            }
-        }
-        // Two checkpoints (reference: engine_factory.cpp:64-72): when decode_model_path names another directory, its
-        // group-wise INT4 tensors (<linear>.qweight / .scaling_factors) become the decode pass's weights; prefill keeps
-        // the bf16 ones.  Tensors of other kinds in that directory are ignored.
-        const std::string decode_path = config_.decode_model_path();
-        if (!decode_path.empty() && decode_path != config_.prefill_model_path()) {
-            const std::vector<std::string> dfiles = collect_safetensors_files(decode_path);
-            if (dfiles.empty()) throw ConfigurationError("No model.safetensors or model-*-of-*.safetensors found in decode path");
-            for (const std::string& f : dfiles) {
-                SafeTensorsFile dm(f);
-                for (const SafeTensorEntry& e : dm.entries()) {
-                    std::string name = e.name;
-                    if (vlm && !map_vlm_weight_name(e.name, &name)) continue;
-                    const int32_t code = dtype_code(e.dtype);
-                    if (code < 0) continue;
-                    st = efm_b200_set_decode_weight(ctx_, name.c_str(), e.data, e.shape.data(), (int32_t)e.shape.size(), code, EFM_MEM_HOST);
-                    if (st == EFM_ERR_UNSUPPORTED) throw ConfigurationError(std::string("decode checkpoint, ") + name + ": " + efm_b200_last_error(ctx_));
-                    if (st != EFM_OK) throw ModelNotLoadedError(std::string("loading decode weight ") + name + ": " + efm_b200_last_error(ctx_));
-                }
-            }
-        }
-        st = efm_b200_finalize_weights(ctx_);
-        if (st != EFM_OK) throw ModelNotLoadedError(std::string("checkpoint incomplete: ") + efm_b200_last_error(ctx_));
-        maps.clear();
-
-        KVGeometry geo;
-        geo.num_layers = d.num_layers;
-        geo.kv_heads = d.kv_heads;
-        geo.head_dim = d.head_dim;
-        geo.dtype = DType::BFloat16;
-        kv_manager_ = std::make_shared<KVManager>(reqs, geo, attn, device_id_, std::make_shared<BackendKVAllocator>(ctx_));
         scheduler_.reset(new Scheduler(kv_manager_, config_.sampling_max_new_tokens()));
-        if (tp > 1) {      // decode all-reduces inside the GEMVs over peer memory: exchange the buffer handles, then a barrier
-            std::vector<char> mine(64, 0);
-            check(efm_b200_tp_peer_export(ctx_, mine.data()), "peer buffer export");
-            const std::vector<std::vector<char>> all = meet->all_gather("peer", mine);
-            std::vector<char> flat;
-            for (const auto& h : all) {
-                if (h.size() != 64) throw ConfigurationError("tensor parallel rendezvous: malformed peer handle");
-                flat.insert(flat.end(), h.begin(), h.end());
-            }
-            check(efm_b200_tp_peer_import(ctx_, flat.data(), tp), "peer buffer import");
-            meet->barrier("ready");
-        }
-
+        if (m.max_live_requests > 0) steps_.reset(new StepScheduler(paged_cache_, kFirstStepSlot, m.max_live_requests));
         efm_sampling s;
         std::memset(&s, 0, sizeof(s));
         s.temperature = config_.sampling_temperature();
@@ -226,9 +52,6 @@ StandardEngine::StandardEngine(const EngineConfig& config) : config_(config) {
         // (standard_engine.cpp:568-770)
         check(efm_b200_set_prefill_graph(ctx_, use_graph_ ? 1 : 0), "prefill graph selection");
         compact_ = CompactVocab(config_);
-        const std::string pa = config_.prefill_attention();
-        if (pa == "int8") check(efm_b200_set_prefill_attention(ctx_, 1), "prefill attention selection");
-        else if (pa != "bf16") throw ConfigurationError("runtime.prefill_attention must be \"bf16\" or \"int8\", got " + pa);
     } catch (...) {
         efm_b200_destroy(ctx_);
         ctx_ = nullptr;
@@ -237,6 +60,9 @@ StandardEngine::StandardEngine(const EngineConfig& config) : config_(config) {
 }
 
 StandardEngine::~StandardEngine() {
+    steps_.reset();
+    kv_manager_.reset();
+    paged_cache_.reset();
     if (ctx_ != nullptr) efm_b200_destroy(ctx_);
 }
 
@@ -255,6 +81,9 @@ void StandardEngine::warmup() {
             check(efm_b200_prefill(ctx_, slot.request_id, prefix_ids.data(), n, 0, nullptr, 0, -1, EFM_MEM_HOST,
                                    use_mrope_ ? pos.data() : nullptr, 0),
                   "prefix prefill");
+            if (paged_cache_ != nullptr) {      // a recurrent state moves on with every token: keep the one after the prefix
+                check(efm_b200_decoder_pin_prefix(ctx_, slot.request_id, paged_cache_->take_state()), "prefix state");
+            }
         }
         if (use_graph_) check(efm_b200_capture_decode(ctx_, slot.request_id), "decode graph capture");
     }
@@ -530,6 +359,133 @@ Response StandardEngine::generate(const Request& request) {
         {"response_tokens_capacity", (double)ctx.max_generated_tokens},
     };
     return response;
+}
+
+// ---- batched steps ---------------------------------------------------------------------------------------------
+void StandardEngine::run_entries(const std::vector<StepEntry>& entries, std::vector<float>* logits, std::vector<int32_t>* sampled,
+                                 const std::vector<uint32_t>& rng_steps) {
+    if (steps_ == nullptr) throw ConfigurationError("batched steps are not supported by this model");
+    const std::vector<PlannedEntry> plan = steps_->plan(entries);
+    std::vector<efm_step_entry> dev(entries.size());
+    size_t n_want = 0;
+    for (size_t i = 0; i < entries.size(); ++i) {
+        dev[i].slot = plan[i].slot;
+        dev[i].n_tokens = (int32_t)entries[i].tokens.size();
+        dev[i].kv_offset = plan[i].kv_offset;
+        dev[i].n_want = (int32_t)entries[i].want.size();
+        dev[i].tokens = entries[i].tokens.data();
+        dev[i].want = entries[i].want.data();
+        dev[i].rng_step = i < rng_steps.size() ? rng_steps[i] : 0;
+        dev[i].reserved = 0;
+        n_want += entries[i].want.size();
+    }
+    if (logits != nullptr) logits->assign(n_want * (size_t)vocab_, 0.f);
+    if (sampled != nullptr) sampled->assign(n_want, 0);
+    check(efm_b200_decoder_step(ctx_, dev.data(), (int32_t)dev.size(), logits != nullptr ? logits->data() : nullptr,
+                                sampled != nullptr ? sampled->data() : nullptr),
+          "step");
+    steps_->commit(entries);
+}
+
+std::vector<float> StandardEngine::step(const std::vector<StepEntry>& entries) {
+    std::vector<float> logits;
+    run_entries(entries, &logits, nullptr, {});
+    return logits;
+}
+
+void StandardEngine::finish(const std::string& id) {
+    if (steps_ == nullptr) throw ConfigurationError("batched steps are not supported by this model");
+    steps_->finish(id);
+}
+
+// Continuous batching: prompts enter in portions beside the single tokens of the requests that already decode; a request
+// is admitted when a slot and the pages for its whole length are free.
+std::vector<Response> StandardEngine::generate_batch(const std::vector<const Request*>& requests) {
+    if (steps_ == nullptr) throw ConfigurationError("batched generation is not supported by this model");
+    struct Job {
+        std::string id;
+        std::vector<int32_t> prompt;
+        size_t fed = 0;
+        std::vector<int32_t> out;
+        std::unordered_set<int32_t> stop;
+        bool live = false, done = false;
+    };
+    const int32_t max_new = config_.sampling_max_new_tokens();
+    std::vector<Job> jobs(requests.size());
+    for (size_t i = 0; i < requests.size(); ++i) {
+        const Request& r = *requests[i];
+        Job& j = jobs[i];
+        j.id = "batch:" + std::to_string(i);
+        if (r.has_embedding()) throw InvalidRequestError("batched generation takes token ids only");
+        if (r.token_ids().empty()) throw InvalidRequestError("Request token_ids is empty for request_id: " + std::to_string(r.request_id()));
+        j.prompt = compact_.remap_token_ids(r.token_ids(), "request token_ids");
+        if (!r.ignore_stop_tokens()) {
+            for (int32_t id : config_.eos_token_ids()) j.stop.insert(id);
+            for (int32_t id : config_.stop_token_ids()) j.stop.insert(id);
+            for (int32_t id : r.stop_token_ids()) j.stop.insert(id);
+        }
+    }
+    auto end_live = [&]() {
+        for (Job& j : jobs)
+            if (j.live) { steps_->finish(j.id); j.live = false; }
+    };
+    try {
+        for (;;) {
+            std::vector<StepEntry> entries;
+            std::vector<Job*> who;
+            int32_t budget = max_step_tokens_;
+            for (Job& j : jobs)                                   // decoding requests first: one token each
+                if (j.live && j.fed == j.prompt.size() && budget > 0) {
+                    entries.push_back(StepEntry{j.id, {j.out.back()}, {0}});
+                    who.push_back(&j);
+                    --budget;
+                }
+            for (Job& j : jobs) {
+                if (j.done || j.fed == j.prompt.size() || budget <= 0) continue;
+                if (!j.live) {
+                    if (!steps_->try_admit(j.id, (int32_t)j.prompt.size() + max_new - 1)) {
+                        if (steps_->live() == 0) throw InvalidRequestError("a request needs more cache than the pool holds");
+                        continue;
+                    }
+                    j.live = true;
+                }
+                const size_t n = std::min((size_t)budget, j.prompt.size() - j.fed);
+                StepEntry e{j.id, std::vector<int32_t>(j.prompt.begin() + (long)j.fed, j.prompt.begin() + (long)(j.fed + n)), {}};
+                j.fed += n;
+                if (j.fed == j.prompt.size()) e.want.push_back((int32_t)n - 1);
+                entries.push_back(std::move(e));
+                who.push_back(&j);
+                budget -= (int32_t)n;
+            }
+            if (entries.empty()) break;
+            std::vector<int32_t> sampled;
+            std::vector<uint32_t> counters;                       // as generate() counts: a request's n-th sample uses counter n
+            for (const Job* j : who) counters.push_back((uint32_t)j->out.size());
+            run_entries(entries, nullptr, &sampled, counters);
+            size_t at = 0;
+            for (size_t i = 0; i < entries.size(); ++i) {
+                if (entries[i].want.empty()) continue;
+                Job& j = *who[i];
+                j.out.push_back(sampled[at++]);
+                int32_t shown = j.out.back();
+                if (compact_.enabled()) shown = compact_.restore_token_ids({shown}, "response token_ids")[0];
+                if (j.stop.count(shown) || (int32_t)j.out.size() >= max_new) {
+                    steps_->finish(j.id);
+                    j.live = false;
+                    j.done = true;
+                }
+            }
+        }
+    } catch (...) {
+        end_live();
+        throw;
+    }
+    std::vector<Response> out(requests.size());
+    for (size_t i = 0; i < jobs.size(); ++i) {
+        std::vector<int32_t> ids = compact_.enabled() ? compact_.restore_token_ids(jobs[i].out, "response token_ids") : jobs[i].out;
+        out[i].token_ids().swap(ids);
+    }
+    return out;
 }
 
 }  // namespace edge_fm

@@ -4,6 +4,7 @@
 // through the C ABI in include/efm_b200.h.
 #pragma once
 #include <edge-fm/core.h>
+#include <edge-fm/edge-fm.h>
 
 #include <memory>
 #include <string>
@@ -13,7 +14,9 @@
 #include "compact_vocab.h"
 #include "config.h"
 #include "kv_manager.h"
+#include "paged_cache.h"
 #include "scheduler.h"
+#include "step_scheduler.h"
 
 struct efm_b200_ctx;
 
@@ -40,10 +43,17 @@ public:
     // in the engine's own slot between calls.
     TensorMap run_stage(int32_t request_id, const std::string& stage_name, const TensorRefMap& inputs);
     std::unordered_map<std::string, double> last_stage_metrics() const { return stage_metrics_; }
+    // Batched steps and batched generation (models on the paged cache; edge-fm.h).
+    std::vector<float> step(const std::vector<StepEntry>& entries);
+    void finish(const std::string& id);
+    std::vector<Response> generate_batch(const std::vector<const Request*>& requests);
+    int32_t vocab() const { return vocab_; }
     void* backend_handle() const { return ctx_; }
 
 private:
-    void load_weights();
+    static constexpr int32_t kFirstStepSlot = 1 << 24;     // slot numbers of batched requests, away from declared ids
+    void run_entries(const std::vector<StepEntry>& entries, std::vector<float>* logits, std::vector<int32_t>* sampled,
+                     const std::vector<uint32_t>& rng_steps);
     void check(int32_t status, const char* what) const;    // backend status -> edge_fm exception
     // M-RoPE prefill positions [3, prefill_tokens] and the last position per axis (text models: untouched)
     void build_positions(const Request& request, const Context& ctx, std::vector<int32_t>* pos, int32_t last_pos[3]) const;
@@ -62,6 +72,9 @@ private:
     bool use_graph_ = false;
     std::shared_ptr<KVManager> kv_manager_;
     std::unique_ptr<Scheduler> scheduler_;
+    std::shared_ptr<PagedCache> paged_cache_;
+    std::unique_ptr<StepScheduler> steps_;
+    int32_t max_step_tokens_ = 0;
     CompactVocab compact_;                // identity unless compact_vocab.enabled
     std::unordered_map<std::string, double> metrics_;
 };

@@ -1,0 +1,419 @@
+// Launch sequences of the layered decoders.
+//
+// Decode (one row), per layer:  [pending output norm + residual add] + input projections | mixer (norms, cache / state
+// update, attention or recurrence) | W_o | [norm1 + add] + W_up | [PolyNorm] + W_down | [norm2 + add] + token gate |
+// token projection; what stands in brackets is the prologue of the GEMV that follows it.  The recurrent mixers launch
+// five kernels per layer, attention with a feed-forward seven.
+// Many rows: tensor-core GEMMs (bf16 operands) or fp32 FMAs (32-bit mode) between row kernels.
+#include "decoder.h"
+
+#include <cstdlib>
+
+#include "../operators/decoder_rows.cuh"
+#include "../operators/delta_rule.cuh"
+#include "../operators/gemm_tc.cuh"
+#include "../operators/window_attention.cuh"
+#define EFM_DECLARATIONS_ONLY
+#include "../operators/sample.cuh"
+#undef EFM_DECLARATIONS_ONLY
+#include "gemv_plan.h"
+#include "launcher.h"
+#include "shared_launch.h"
+
+namespace efm {
+
+// ---- one row -----------------------------------------------------------------------------------------------------
+namespace {
+
+// The sublayer output that has not been added to the residual stream yet.
+struct Pending {
+    const float* y = nullptr;
+    const __nv_bfloat16* norm = nullptr;
+    int flip = 0;                        // which residual buffer holds the stream
+};
+
+template <Epi EPI>
+void gemv_ext(efm_b200_ctx& c, Launcher& L, const DecLinear& w, GemvParams& p) {
+    p.W = w.w;
+    p.N = w.N;
+    p.K = w.Kp;
+    p.n_items = w.Np / 2;
+    p.eps = c.decoder->d.norm_eps;
+    p.state = c.state;
+    p.vocab = c.d.vocab;
+    const int ks = plan_gemv_ksplit(p.n_items, p.K, c.num_sms);
+    // Logits publishes one maximum per block of a full grid; the others launch no idle blocks
+    const int per = kGemvWarps / ks, need = (p.n_items + per - 1) / per;
+    const int grid = EPI == Epi::Logits ? c.num_sms : std::min(c.num_sms, need);
+    const size_t smem = p.prologue == kProAddNorm ? gemv_ext_smem_bytes(p.K) : gemv_smem_bytes(p.K);
+    L.launch(gemv_kernel<EPI, true>, dim3(grid), dim3(kGemvThreads), smem, p, ks);
+}
+
+// Input of a product that reads the residual stream: embedding row (first layer) or stream + pending output.
+void stream_input(efm_b200_ctx& c, GemvParams& p, Pending& pend, bool first) {
+    float* bufs[2] = {c.resid_d, c.resid_d2};
+    p.k_true = c.decoder->W;
+    if (first) {
+        p.prologue = kProEmbed;
+        p.embed_table = c.embed;
+        p.resid_out = bufs[pend.flip];
+        return;
+    }
+    if (pend.y == nullptr) { p.prologue = kProPlain; p.xf = bufs[pend.flip]; return; }
+    p.prologue = kProAddNorm;
+    p.xr = bufs[pend.flip];
+    p.addend = pend.y;
+    p.norm_w = pend.norm;
+    pend.flip ^= 1;                      // other blocks still read the old row: the new one goes to the other buffer
+    p.resid_out = bufs[pend.flip];
+    pend.y = nullptr;
+}
+
+WindowAttnShape attn_shape(const DecoderModel& m, const DecoderLayer& l) {
+    WindowAttnShape s{};
+    s.H = l.d.heads; s.G = l.d.kv_heads; s.D = l.d.dim; s.Dv = l.d.vdim; s.Dp = l.Dp; s.Vp = l.Vp;
+    s.window = l.d.window; s.bias = l.d.distance_bias; s.scale = l.d.scale; s.eps = m.d.norm_eps;
+    s.q_norm = l.q_norm; s.k_norm = l.k_norm; s.temp = l.temp;
+    return s;
+}
+DeltaShape delta_shape(const DecoderModel& m, const DecoderLayer& l) {
+    DeltaShape s{};
+    s.heads = l.d.heads; s.D = l.d.dim; s.Dp = round_up(l.d.dim, 32); s.rank = l.d.decay_rank; s.ld = l.in.Np;
+    s.eps = m.d.norm_eps; s.w0 = l.w0; s.a_bias = l.a_bias; s.norm = l.mix_norm;
+    return s;
+}
+
+template <typename TC, int VM>
+void launch_attn_decode_v(Launcher& L, const WindowDecodeParams<TC>& p, int cluster) {
+    const int hb = (p.s.H / p.s.G + wd::kHeads - 1) / wd::kHeads;
+    L.cluster_x = cluster;
+    L.launch(window_attention_decode_kernel<TC, VM>, dim3(cluster, p.s.G * hb), dim3(wd::kThreads), sizeof(wd::Smem<VM>), p);
+}
+template <typename TC>
+void launch_attn_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const KvSlot& slot, bool early) {
+    DecoderModel& m = *c.decoder;
+    WindowDecodeParams<TC> p{};
+    p.s = attn_shape(m, l);
+    p.qkv = m.d_in;
+    p.k_pool = static_cast<TC*>(l.k_pool);
+    p.v_pool = static_cast<TC*>(l.v_pool);
+    p.pages = m.page_table + (size_t)slot.table * m.d.cache_pages;
+    p.max_pages = slot.n_pages;
+    p.state = c.state;
+    p.out = m.d_mix;
+    p.early = early ? 1 : 0;
+    // one block per page of the visible range, up to the cluster width (a power of two)
+    int pages = slot.n_pages;
+    if (l.d.window > 0) pages = std::min(pages, (l.d.window + kPageTokens - 2) / kPageTokens + 1);
+    int cluster = 1;
+    while (cluster < pages && cluster < m.attn_cluster) cluster *= 2;
+    const int v = std::max(l.Dp, l.Vp);
+    if (v <= 64) launch_attn_decode_v<TC, 64>(L, p, cluster);
+    else if (v <= 128) launch_attn_decode_v<TC, 128>(L, p, cluster);
+    else launch_attn_decode_v<TC, 256>(L, p, cluster);
+}
+
+void launch_delta_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const KvSlot& slot, bool early) {
+    DecoderModel& m = *c.decoder;
+    DeltaDecodeParams p{};
+    p.s = delta_shape(m, l);
+    p.proj = m.d_in;
+    p.w2 = l.w2.w;
+    p.ld_w2 = l.w2.Kp;
+    p.pool = m.state_pool + (size_t)slot.state_slot * m.state_stride + l.state_off;
+    p.state = c.state;
+    p.out = m.d_mix;
+    p.early = early ? 1 : 0;
+    const int D = l.d.dim, rpt = (D + 512 / D - 1) / (512 / D);
+    const dim3 grid(l.d.heads), block(512);
+    if (rpt <= 8) L.launch(delta_decode_kernel<8>, grid, block, 0, p);
+    else if (rpt <= 32) L.launch(delta_decode_kernel<32>, grid, block, 0, p);
+    else L.launch(delta_decode_kernel<0>, grid, block, 0, p);
+}
+
+}  // namespace
+
+void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample, bool want_logits) {
+    DecoderModel& m = *c.decoder;
+    Pending pend;
+    auto tap = [&](int layer) {
+        if (m.tap == nullptr || m.tap_row0 >= m.tap_rows) return;
+        const float* src = pend.flip ? c.resid_d2 : c.resid_d;
+        if (L.err == cudaSuccess)
+            L.err = cudaMemcpyAsync(m.tap + ((size_t)layer * m.tap_rows + m.tap_row0) * m.Wp, src, (size_t)m.Wp * 4, cudaMemcpyDeviceToDevice, L.stream);
+    };
+    for (size_t i = 0; i < m.layers.size(); ++i) {
+        const DecoderLayer& l = m.layers[i];
+        // From the second layer on a mixer may read the device state and what earlier steps left in its cache before its
+        // dependency wait: the mixer one layer up releases its dependents only after its own wait, so nothing of an
+        // earlier step is still running.
+        const bool early = i > 0;
+        {
+            GemvParams p{};
+            stream_input(c, p, pend, i == 0);
+            p.out_f = m.d_in;
+            gemv_ext<Epi::Store32>(c, L, l.in, p);
+            if (i > 0) tap((int)i - 1);
+        }
+        if (l.d.mixer == EFM_MIXER_ATTENTION) {
+            if (m.f32) launch_attn_decode<float>(c, L, l, slot, early);
+            else launch_attn_decode<__nv_bfloat16>(c, L, l, slot, early);
+        } else {
+            launch_delta_decode(c, L, l, slot, early);
+        }
+        {
+            GemvParams p{};
+            p.prologue = kProPlain;
+            p.xf = m.d_mix;
+            p.out_f = m.d_y;
+            gemv_ext<Epi::Store32>(c, L, l.out, p);
+            pend.y = m.d_y;
+            pend.norm = l.norm1;
+        }
+        if (l.d.ff > 0) {
+            GemvParams p{};
+            stream_input(c, p, pend, false);
+            p.out_f = m.d_ff;
+            gemv_ext<Epi::Store32>(c, L, l.up, p);
+            GemvParams q{};
+            q.prologue = kProPolyNorm;
+            q.xf = m.d_ff;
+            q.k_true = l.d.ff;
+            q.poly = l.act;
+            q.out_f = m.d_y;
+            gemv_ext<Epi::Store32>(c, L, l.down, q);
+            pend.y = m.d_y;
+            pend.norm = l.norm2;
+        }
+        if (m.d.side_dim > 0) {
+            GemvParams p{};
+            stream_input(c, p, pend, false);
+            p.out_f = m.d_gate;
+            p.gate_table = m.side_embed;
+            p.gate_ld = m.d.side_dim * m.d.num_layers;
+            p.gate_off = (int)i * m.d.side_dim;
+            gemv_ext<Epi::TokenGate>(c, L, l.gate, p);
+            GemvParams q{};
+            q.prologue = kProPlain;
+            q.xf = m.d_gate;
+            q.out_f = m.d_y;
+            gemv_ext<Epi::Store32>(c, L, l.proj, q);
+            pend.y = m.d_y;
+            pend.norm = l.side_norm;
+        }
+    }
+    if (!want_logits && !sample && m.tap == nullptr) return;
+    {
+        GemvParams p{};
+        stream_input(c, p, pend, false);
+        p.norm2_w = m.final_norm;
+        p.logits = c.logits;
+        p.part_val = c.part_val;
+        p.part_idx = c.part_idx;
+        gemv_ext<Epi::Logits>(c, L, m.head, p);
+        tap((int)m.layers.size() - 1);
+    }
+    if (!sample) return;
+    SampleParams s{};
+    s.logits = c.logits;
+    s.vocab = c.d.vocab;
+    s.part_val = c.part_val;
+    s.part_idx = c.part_idx;
+    s.n_part = c.num_sms;
+    s.temperature = c.sampling.temperature;
+    s.top_p = c.sampling.top_p;
+    s.seed = c.sampling.seed;
+    s.state = c.state;
+    s.tokens_out = c.tokens_out;
+    s.max_response = c.d.max_response_tokens;
+    s.advance = 1;
+    s.wbuf = c.wbuf;
+    s.xchg = sample_xchg(c.wbuf, c.d.vocab);
+    launch_sample(L, s);
+}
+
+// ---- many rows ---------------------------------------------------------------------------------------------------
+int decoder_tc_tile_rows() { return 128; }
+int decoder_simt_tile_rows() { return wa::QT; }
+bool decoder_layer_tc(const DecoderModel&, const DecoderLayer&) { return false; }
+
+namespace {
+
+// out[rows, w.Np] = a[rows, w.Kp] . w^T.  bf16 activations run on the tensor cores, fp32 ones in fp32 FMAs.
+void linear_f32(efm_b200_ctx& c, Launcher& L, const DecLinear& w, const void* a, float* out, int rows) {
+    if (c.decoder->f32) {
+        L.launch(gemm_f32_kernel, dim3((w.Np + 63) / 64, (rows + 63) / 64), dim3(256), 0, static_cast<const float*>(a), w.Kp,
+                 (const __nv_bfloat16*)w.w, w.Kp, out, w.Np, rows, w.Np, w.Kp);
+        return;
+    }
+    GemmParams g{static_cast<const __nv_bfloat16*>(a), w.w, nullptr, nullptr, out, rows, w.Np, w.Kp};
+    launch_gemm_epi(L, GemmEpi::F32, g, &c.state->error);
+}
+// the same with the activation type of the pass as output
+void linear_act(efm_b200_ctx& c, Launcher& L, const DecLinear& w, const void* a, void* out, int rows) {
+    if (c.decoder->f32) { linear_f32(c, L, w, a, static_cast<float*>(out), rows); return; }
+    GemmParams g{static_cast<const __nv_bfloat16*>(a), w.w, nullptr, static_cast<__nv_bfloat16*>(out), nullptr, rows, w.Np, w.Kp};
+    launch_gemm_epi(L, GemmEpi::Bf16Bias, g, &c.state->error);
+}
+
+template <int NC>
+void launch_delta_scan(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const RowPlan& plan) {
+    DecoderModel& m = *c.decoder;
+    const DeltaShape s = delta_shape(m, l);
+    const int groups = (s.Dp + ds::kCols - 1) / ds::kCols;
+    L.launch(delta_scan_kernel<NC>, dim3(l.d.heads * groups, plan.n_entries), dim3(ds::kThreads), ds::smem_bytes(s.Dp), (const float*)m.pack, m.o, l.mix_wp,
+             m.state_pool, m.state_stride, l.state_off, s, plan);
+}
+
+// TA: activation type of the pass, TC: cache type (the same)
+template <typename TA>
+void attention_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const RowPlan& plan, const RowTiles& tiles) {
+    DecoderModel& m = *c.decoder;
+    const WindowAttnShape s = attn_shape(m, l);
+    linear_act(c, L, l.in, m.f32 ? (void*)c.resid : m.xa, m.proj_a, plan.rows);
+    TA* kp = static_cast<TA*>(l.k_pool);
+    TA* vp = static_cast<TA*>(l.v_pool);
+    L.launch(qk_scatter_rows_kernel<TA, TA, TA>, dim3(plan.rows), dim3(256), 0, static_cast<const TA*>(m.proj_a), l.in.Np, static_cast<TA*>(m.q), kp, vp, s, plan);
+    const RowTile* list = tiles.all;
+    const int n = tiles.listed ? tiles.n_all : (plan.rows + wa::QT - 1) / wa::QT;
+    L.launch(window_attention_rows_kernel<TA, TA, TA>, dim3(n, s.H), dim3(256), wa::rows_smem_bytes(s.Dp, s.Vp), static_cast<const TA*>(m.q), (const TA*)kp,
+             (const TA*)vp, static_cast<TA*>(m.mix), l.mix_wp, s, plan, list);
+}
+
+template <typename TA>
+void delta_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const RowPlan& plan) {
+    DecoderModel& m = *c.decoder;
+    const DeltaShape s = delta_shape(m, l);
+    linear_f32(c, L, l.in, m.f32 ? (void*)c.resid : m.xa, m.proj_f, plan.rows);
+    L.launch(delta_tanh_rows_kernel, dim3(plan.rows), dim3(128), 0, (const float*)m.proj_f, m.tanh_w, l.w2.Kp, s);
+    L.launch(gemm_f32_kernel, dim3((l.w2.Np + 63) / 64, (plan.rows + 63) / 64), dim3(256), 0, (const float*)m.tanh_w, l.w2.Kp, (const __nv_bfloat16*)l.w2.w,
+             l.w2.Kp, m.decay, l.w2.Np, plan.rows, l.w2.Np, l.w2.Kp);
+    L.launch(delta_inputs_rows_kernel, dim3(plan.rows), dim3(256), 0, (const float*)m.proj_f, (const float*)m.decay, l.w2.Np, m.pack, s);
+    switch (s.Dp / 32) {
+        case 1: launch_delta_scan<1>(c, L, l, plan); break;
+        case 2: launch_delta_scan<2>(c, L, l, plan); break;
+        case 3: launch_delta_scan<3>(c, L, l, plan); break;
+        case 4: launch_delta_scan<4>(c, L, l, plan); break;
+        case 5: launch_delta_scan<5>(c, L, l, plan); break;
+        case 6: launch_delta_scan<6>(c, L, l, plan); break;
+        case 7: launch_delta_scan<7>(c, L, l, plan); break;
+        default: launch_delta_scan<8>(c, L, l, plan); break;
+    }
+    L.launch(delta_output_rows_kernel<TA>, dim3(plan.rows), dim3(256), 0, (const float*)m.o, l.mix_wp, (const float*)m.proj_f, static_cast<TA*>(m.mix), l.mix_wp, s);
+}
+
+template <typename TA>
+void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const RowTiles& tiles, Launcher& L) {
+    DecoderModel& m = *c.decoder;
+    const int T = plan.rows;
+    TA* xa = m.f32 ? nullptr : static_cast<TA*>(m.xa);          // 32-bit mode reads the stream itself
+    const void* xin = m.f32 ? (const void*)c.resid : m.xa;
+    auto add_norm = [&](const float* y, const __nv_bfloat16* w) {
+        L.launch(add_norm_rows_kernel<TA>, dim3(T), dim3(256), 0, c.resid, y, w, xa, m.W, m.Wp, m.d.norm_eps);
+    };
+    launch_embed_rows(L, ids, c.embed, nullptr, c.resid, T, c.d.vocab, m.Wp, -1, 0);
+    if (xa != nullptr) add_norm(nullptr, nullptr);
+    for (size_t i = 0; i < m.layers.size(); ++i) {
+        const DecoderLayer& l = m.layers[i];
+        if (l.d.mixer == EFM_MIXER_ATTENTION) attention_rows<TA>(c, L, l, plan, tiles);
+        else delta_rows<TA>(c, L, l, plan);
+        linear_f32(c, L, l.out, m.mix, m.y, T);
+        add_norm(m.y, l.norm1);
+        if (l.d.ff > 0) {
+            linear_act(c, L, l.up, xin, m.ff, T);
+            L.launch(poly_norm_rows_kernel<TA>, dim3(T), dim3(256), 0, static_cast<const TA*>(m.ff), static_cast<TA*>(m.ff2), (const __nv_bfloat16*)l.act, l.d.ff,
+                     l.down.Kp, m.d.norm_eps);
+            linear_f32(c, L, l.down, m.ff2, m.y, T);
+            add_norm(m.y, l.norm2);
+        }
+        if (m.d.side_dim > 0) {
+            linear_f32(c, L, l.gate, xin, m.side_f, T);
+            L.launch(token_gate_rows_kernel<TA>, dim3(T), dim3(128), 0, (const float*)m.side_f, ids, (const __nv_bfloat16*)m.side_embed,
+                     m.d.side_dim * m.d.num_layers, (int)i * m.d.side_dim, c.d.vocab, static_cast<TA*>(m.side_a), m.d.side_dim, m.side_p);
+            linear_f32(c, L, l.proj, m.side_a, m.y, T);
+            add_norm(m.y, l.side_norm);
+        }
+        if (m.tap != nullptr && m.tap_row0 + T <= m.tap_rows && L.err == cudaSuccess)
+            L.err = cudaMemcpyAsync(m.tap + ((size_t)i * m.tap_rows + m.tap_row0) * m.Wp, c.resid, (size_t)T * m.Wp * 4, cudaMemcpyDeviceToDevice, L.stream);
+    }
+}
+
+}  // namespace
+
+void decoder_rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const RowTiles& tiles, Launcher& L) {
+    const bool pdl = L.pdl;
+    L.pdl = false;
+    if (c.decoder->f32) rows_pass<float>(c, plan, ids, tiles, L);
+    else rows_pass<__nv_bfloat16>(c, plan, ids, tiles, L);
+    L.pdl = pdl;
+}
+
+void decoder_rows_logits(efm_b200_ctx& c, const int32_t* rows, int n, Launcher& L) {
+    DecoderModel& m = *c.decoder;
+    const bool pdl = L.pdl;
+    L.pdl = false;
+    if (m.f32)
+        L.launch(gather_norm_rows_kernel<float>, dim3(n), dim3(256), 0, (const float*)c.resid, rows, (const __nv_bfloat16*)m.final_norm,
+                 static_cast<float*>(m.head_a), m.W, m.Wp, m.d.norm_eps);
+    else
+        L.launch(gather_norm_rows_kernel<__nv_bfloat16>, dim3(n), dim3(256), 0, (const float*)c.resid, rows, (const __nv_bfloat16*)m.final_norm,
+                 static_cast<__nv_bfloat16*>(m.head_a), m.W, m.Wp, m.d.norm_eps);
+    linear_f32(c, L, m.head, m.head_a, m.logits_rows, n);
+    L.pdl = pdl;
+}
+
+// ---- set-up ------------------------------------------------------------------------------------------------------
+namespace {
+template <typename K>
+cudaError_t smem_attr(K kernel, size_t bytes) { return cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes); }
+
+// widest cluster the decode attention kernel can be placed with
+template <typename TC, int VM>
+cudaError_t fit_cluster(int& width) {
+    cudaError_t e = smem_attr(window_attention_decode_kernel<TC, VM>, sizeof(wd::Smem<VM>));
+    if (e != cudaSuccess) return e;
+    const bool wide = cudaFuncSetAttribute(window_attention_decode_kernel<TC, VM>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess;
+    int cs = wide ? 16 : 8;
+    for (; cs > 1; cs >>= 1) {
+        cudaLaunchConfig_t cfg = {};
+        cfg.gridDim = dim3(cs, 1, 1);
+        cfg.blockDim = dim3(wd::kThreads);
+        cfg.dynamicSmemBytes = sizeof(wd::Smem<VM>);
+        cudaLaunchAttribute at;
+        at.id = cudaLaunchAttributeClusterDimension;
+        at.val.clusterDim.x = (unsigned)cs;
+        at.val.clusterDim.y = at.val.clusterDim.z = 1;
+        cfg.attrs = &at;
+        cfg.numAttrs = 1;
+        int n = 0;
+        if (cudaOccupancyMaxActiveClusters(&n, window_attention_decode_kernel<TC, VM>, &cfg) == cudaSuccess && n >= 1) break;
+    }
+    (void)cudaGetLastError();
+    width = std::min(width, cs);
+    return cudaSuccess;
+}
+}  // namespace
+
+cudaError_t configure_decoder(DecoderModel& m) {
+    int dev = 0, optin = 0;
+    cudaError_t e = cudaGetDevice(&dev);
+    if (e == cudaSuccess) e = cudaDeviceGetAttribute(&optin, cudaDevAttrMaxSharedMemoryPerBlockOptin, dev);
+    const size_t gv = (size_t)optin - 2048;
+    if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::Store32, true>, gv);
+    if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::TokenGate, true>, gv);
+    if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::Logits, true>, gv);
+    const size_t rows = wa::rows_smem_bytes(256, 256);
+    if (e == cudaSuccess) e = smem_attr(window_attention_rows_kernel<float, float, float>, rows);
+    if (e == cudaSuccess) e = smem_attr(window_attention_rows_kernel<__nv_bfloat16, __nv_bfloat16, __nv_bfloat16>, rows);
+    if (e == cudaSuccess) e = smem_attr(delta_scan_kernel<5>, ds::smem_bytes(160));
+    if (e == cudaSuccess) e = smem_attr(delta_scan_kernel<6>, ds::smem_bytes(192));
+    if (e == cudaSuccess) e = smem_attr(delta_scan_kernel<7>, ds::smem_bytes(224));
+    if (e == cudaSuccess) e = smem_attr(delta_scan_kernel<8>, ds::smem_bytes(256));
+    m.attn_cluster = 16;
+    if (e == cudaSuccess) e = m.f32 ? fit_cluster<float, 64>(m.attn_cluster) : fit_cluster<__nv_bfloat16, 64>(m.attn_cluster);
+    if (e == cudaSuccess) e = m.f32 ? fit_cluster<float, 128>(m.attn_cluster) : fit_cluster<__nv_bfloat16, 128>(m.attn_cluster);
+    if (e == cudaSuccess) e = m.f32 ? fit_cluster<float, 256>(m.attn_cluster) : fit_cluster<__nv_bfloat16, 256>(m.attn_cluster);
+    return e;
+}
+
+}  // namespace efm

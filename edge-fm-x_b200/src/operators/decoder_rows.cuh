@@ -1,0 +1,156 @@
+// Row kernels of the layered decoders' many-row pass: output norms with the residual add, PolyNorm, the per-layer token
+// input, gathered final norms, and the all-32-bit matrix product.  T = bf16 (tensor-core operands) or fp32.
+#pragma once
+#include "common.cuh"
+#include "gemv.cuh"
+#include "window_attention.cuh"
+
+namespace efm {
+
+__device__ __forceinline__ float block_sum_256(float v, float* part) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    v = warp_sum(v);
+    if (lane == 0) part[warp] = v;
+    __syncthreads();
+    float t = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) t += part[i];
+    return t;
+}
+__device__ __forceinline__ void store4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float4& v) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+}
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    return make_float4(bf16lo(v.x), bf16hi(v.x), bf16lo(v.y), bf16hi(v.y));
+}
+
+// x += y / sqrt(mean(y^2) + eps) * w (y null: x unchanged); copy of x as T (null: none).  One block per row.
+template <typename T>
+__global__ void __launch_bounds__(256) add_norm_rows_kernel(float* __restrict__ x, const float* __restrict__ y, const __nv_bfloat16* __restrict__ w,
+                                                            T* __restrict__ copy, int n, int ld, float eps) {
+    __shared__ float part[8];
+    const size_t base = (size_t)blockIdx.x * ld;
+    const int nv = ld / 4;
+    if (y != nullptr) {
+        float ss = 0.f;
+        for (int c = threadIdx.x; c < nv; c += 256) {
+            const float4 v = load4(y + base + 4 * c);
+            ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
+        }
+        const float inv = 1.0f / sqrtf(block_sum_256(ss, part) / (float)n + eps);
+        for (int c = threadIdx.x; c < nv; c += 256) {
+            const float4 v = load4(y + base + 4 * c), g = load4(w + 4 * c);
+            float4 r = load4(x + base + 4 * c);
+            r.x += v.x * inv * g.x; r.y += v.y * inv * g.y; r.z += v.z * inv * g.z; r.w += v.w * inv * g.w;
+            store4(x + base + 4 * c, r);
+            if (copy != nullptr) store4(copy + base + 4 * c, r);
+        }
+    } else {
+        for (int c = threadIdx.x; c < nv; c += 256) store4(copy + base + 4 * c, load4(x + base + 4 * c));
+    }
+}
+
+// out = c0 rms(z) + c1 rms(z^2) + c2 rms(z^3) + c3 over n channels; pads [n, ld) become zero.  One block per row.
+template <typename T>
+__global__ void __launch_bounds__(256) poly_norm_rows_kernel(const T* __restrict__ z, T* __restrict__ out, const __nv_bfloat16* __restrict__ coef, int n,
+                                                             int ld, float eps) {
+    __shared__ float part[3][8];
+    const size_t base = (size_t)blockIdx.x * ld;
+    const int nv = ld / 4;
+    float s0 = 0.f, s1 = 0.f, s2 = 0.f;
+    auto add = [&](float v) { const float v2 = v * v, v4 = v2 * v2; s0 += v2; s1 += v4; s2 = fmaf(v4, v2, s2); };
+    for (int c = threadIdx.x; c < nv; c += 256) {
+        const float4 v = load4(z + base + 4 * c);                       // pads are zero
+        add(v.x); add(v.y); add(v.z); add(v.w);
+    }
+    s0 = block_sum_256(s0, part[0]);
+    s1 = block_sum_256(s1, part[1]);
+    s2 = block_sum_256(s2, part[2]);
+    const float c0 = __bfloat162float(coef[0]) / sqrtf(s0 / (float)n + eps), c1 = __bfloat162float(coef[1]) / sqrtf(s1 / (float)n + eps),
+                c2 = __bfloat162float(coef[2]) / sqrtf(s2 / (float)n + eps), c3 = __bfloat162float(coef[3]);
+    for (int c = threadIdx.x; c < nv; c += 256) {
+        const float4 v = load4(z + base + 4 * c);
+        float f[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int j = 0; j < 4; ++j) f[j] = 4 * c + j < n ? fmaf(f[j], fmaf(f[j], fmaf(f[j], c2, c1), c0), c3) : 0.f;
+        store4(out + base + 4 * c, make_float4(f[0], f[1], f[2], f[3]));
+    }
+}
+
+// out[row][c] = gelu_tanh(s[row][c]) * table[id(row)][off + c] for c < n, zero in the pads.
+template <typename T>
+__global__ void __launch_bounds__(128) token_gate_rows_kernel(const float* __restrict__ s, const int32_t* __restrict__ ids,
+                                                              const __nv_bfloat16* __restrict__ table, int table_ld, int off, int vocab,
+                                                              T* __restrict__ out, int n, int ld) {
+    const int row = blockIdx.x, id = ids[row];
+    const bool ok = id >= 0 && id < vocab;
+    const __nv_bfloat16* e = table + (size_t)(ok ? id : 0) * table_ld + off;
+    for (int c = threadIdx.x; c < ld; c += 128)
+        store_f32(out + (size_t)row * ld + c, ok && c < n ? gelu_tanh(s[(size_t)row * ld + c]) * __bfloat162float(e[c]) : 0.f);
+}
+
+// out[i] = rms(x[rows[i]]) * w
+template <typename T>
+__global__ void __launch_bounds__(256) gather_norm_rows_kernel(const float* __restrict__ x, const int32_t* __restrict__ rows,
+                                                               const __nv_bfloat16* __restrict__ w, T* __restrict__ out, int n, int ld, float eps) {
+    __shared__ float part[8];
+    const float* src = x + (size_t)rows[blockIdx.x] * ld;
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < ld / 4; c += 256) {
+        const float4 v = load4(src + 4 * c);
+        ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
+    }
+    const float inv = 1.0f / sqrtf(block_sum_256(ss, part) / (float)n + eps);
+    for (int c = threadIdx.x; c < ld / 4; c += 256) {
+        const float4 v = load4(src + 4 * c), g = load4(w + 4 * c);
+        store4(out + (size_t)blockIdx.x * ld + 4 * c, make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w));
+    }
+}
+
+// C[M, N] = A[M, K] . W[N, K]^T in fp32 FMAs (fp32 activations, bf16 weights): the products of the all-32-bit mode and
+// the small ones that feed a recurrence.  64 x 64 tiles, 256 threads, 4 x 4 outputs per thread.
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ W, int ldw,
+                                                       float* __restrict__ C, int ldc, int M, int N, int K) {
+    __shared__ float as[16][64 + 4], ws[16][64 + 4];
+    const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+    const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+    float acc[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+    const int lr = tid >> 2, lk = (tid & 3) * 4;
+    for (int k0 = 0; k0 < K; k0 += 16) {                                // K % 4 == 0
+        const bool kin = k0 + lk < K;
+        const float4 a = kin && m0 + lr < M ? load4(A + (size_t)(m0 + lr) * lda + k0 + lk) : make_float4(0.f, 0.f, 0.f, 0.f);
+        const float4 w = kin && n0 + lr < N ? load4(W + (size_t)(n0 + lr) * ldw + k0 + lk) : make_float4(0.f, 0.f, 0.f, 0.f);
+        __syncthreads();
+        as[lk][lr] = a.x; as[lk + 1][lr] = a.y; as[lk + 2][lr] = a.z; as[lk + 3][lr] = a.w;
+        ws[lk][lr] = w.x; ws[lk + 1][lr] = w.y; ws[lk + 2][lr] = w.z; ws[lk + 3][lr] = w.w;
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < 16; ++k) {
+            const float4 x = *reinterpret_cast<const float4*>(&as[k][ty * 4]), y = *reinterpret_cast<const float4*>(&ws[k][tx * 4]);
+            const float xa[4] = {x.x, x.y, x.z, x.w}, ya[4] = {y.x, y.y, y.z, y.w};
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(xa[i], ya[j], acc[i][j]);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int m = m0 + ty * 4 + i;
+        if (m >= M) continue;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int n = n0 + tx * 4 + j;
+            if (n < N) C[(size_t)m * ldc + n] = acc[i][j];
+        }
+    }
+}
+
+}  // namespace efm

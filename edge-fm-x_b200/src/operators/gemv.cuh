@@ -30,9 +30,14 @@
 
 namespace efm {
 
-enum class Epi : int { Plain = 0, Residual = 1, QkvRope = 2, SwiGlu = 3, Logits = 4, Peers = 5 };
+enum class Epi : int { Plain = 0, Residual = 1, QkvRope = 2, SwiGlu = 3, Logits = 4, Peers = 5, Store32 = 6, TokenGate = 7 };
 constexpr int kMaxPeers = 8;
-enum : int { kProPlain = 0, kProRmsNorm = 1, kProEmbedRmsNorm = 2 };
+// The last three (and the epilogues Store32, TokenGate) exist in the EXT instantiations only (layered decoders):
+//   Embed    x = embed_table[token], no norm
+//   AddNorm  x = xr + rmsnorm(addend) * norm_w: a sublayer whose OUTPUT is normalised, folded into the next product;
+//            with norm2_w the product reads rmsnorm(x) * norm2_w instead of x
+//   PolyNorm x = c0 rms(z) + c1 rms(z^2) + c2 rms(z^3) + c3 with z = xf and the four numbers of `poly`
+enum : int { kProPlain = 0, kProRmsNorm = 1, kProEmbedRmsNorm = 2, kProEmbed = 3, kProAddNorm = 4, kProPolyNorm = 5 };
 
 struct GemvParams {
     const __nv_bfloat16* W;   // [N, K] row-major
@@ -80,7 +85,19 @@ struct GemvParams {
     volatile int* error_host; // optional mirror of `error` in mapped host memory (the host stops queueing steps)
     unsigned long long wait_ns;   // total wait budget of one kernel; 0 = kPeerWaitDefaultNs
     unsigned int want_override;   // != 0: wait for this count instead of *epoch (single-GPU test of the wait)
+    // EXT instantiations.  Rows are padded to K (a multiple of 8) with zeros; means divide by k_true.
+    int k_true;
+    const __nv_bfloat16* norm2_w;
+    const __nv_bfloat16* poly;
+    float* out_f;             // Store32, TokenGate: [2 * n_items]
+    // TokenGate: out[n] = gelu_tanh(W x)[n] * gate_table[token][gate_off + n] for n < N, 0 beyond
+    const __nv_bfloat16* gate_table;
+    int gate_ld, gate_off;
 };
+
+__device__ __forceinline__ float gelu_tanh(float z) {
+    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
 
 // One {value, count} word is ONE 64-bit element (value in the low half), so that value and count are read and
 // written together by the memory model's own rule (a 64-bit access is single-copy atomic), not by the accident
@@ -138,8 +155,18 @@ __device__ __forceinline__ void item_epilogue(const GemvParams& p, int item, flo
             if (r < p.n_peers) st_peer_words(p.peer_out[r] + item * 2, w0, w1);
     } else if constexpr (EPI == Epi::Logits) {
         *reinterpret_cast<float2*>(p.logits + item * 2) = make_float2(a0, a1);
+        if (item * 2 >= p.N) a0 = -INFINITY;                          // padding rows
+        if (item * 2 + 1 >= p.N) a1 = -INFINITY;
         if (a0 > best_v) { best_v = a0; best_i = item * 2; }          // ascending ids: strict > keeps
         if (a1 > best_v) { best_v = a1; best_i = item * 2 + 1; }      // the lowest id on ties
+    } else if constexpr (EPI == Epi::Store32) {
+        *reinterpret_cast<float2*>(p.out_f + item * 2) = make_float2(a0, a1);
+    } else if constexpr (EPI == Epi::TokenGate) {
+        const int n = item * 2, tok = p.state->token;
+        const bool ok = tok >= 0 && tok < p.vocab;
+        const __nv_bfloat16* e = p.gate_table + (size_t)(ok ? tok : 0) * p.gate_ld + p.gate_off + n;
+        p.out_f[n] = ok && n < p.N ? gelu_tanh(a0) * __bfloat162float(e[0]) : 0.f;
+        p.out_f[n + 1] = ok && n + 1 < p.N ? gelu_tanh(a1) * __bfloat162float(e[1]) : 0.f;
     } else {  // QkvRope
         const int D = p.head_dim, half = D >> 1;
         const int head = item / half, d = item - head * half;
@@ -240,14 +267,131 @@ __host__ __device__ inline unsigned int gemv_xbytes(int K) { return ((unsigned i
 __host__ __device__ inline unsigned int gemv_wbytes(int K) { return ((unsigned int)K * 2u + 15u) & ~15u; }
 
 // Weights only: the first two units into registers, the norm weight into shared memory.
-template <Epi EPI>
+template <Epi EPI, bool EXT>
 __device__ __forceinline__ void gemv_prefetch(const GemvParams& p, const GemvSched& sc, GemvRegs& r, unsigned char* smem,
                                               const unsigned int xbytes) {
     gemv_load_unit<EPI>(p, sc, 0, r.a);
-    if (p.prologue != kProPlain) {
+    if (EXT ? p.prologue == kProAddNorm : p.prologue != kProPlain) {
         uint4* gs = reinterpret_cast<uint4*>(smem + xbytes);        // xbytes = gemv_xbytes(K)
         for (int c = threadIdx.x; c < sc.nch; c += kGemvThreads) gs[c] = ld_cached(p.norm_w + (size_t)c * 8);
     }
+}
+
+// Sums of N per-thread values over the block (all threads get them); red: N x kGemvWarps floats, free on return only after
+// the next block barrier.
+template <int N>
+__device__ __forceinline__ void gemv_block_sums(float (&v)[N], float* red) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+        v[i] = warp_sum(v[i]);
+        if (lane == 0) red[i * kGemvWarps + warp] = v[i];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+        v[i] = 0.f;
+#pragma unroll
+        for (int w = 0; w < kGemvWarps; ++w) v[i] += red[i * kGemvWarps + w];
+    }
+}
+__device__ __forceinline__ void ld8f(const float* p, float (&f)[8]) {
+    const float4 lo = __ldcg(reinterpret_cast<const float4*>(p)), hi = __ldcg(reinterpret_cast<const float4*>(p) + 1);
+    f[0] = lo.x; f[1] = lo.y; f[2] = lo.z; f[3] = lo.w; f[4] = hi.x; f[5] = hi.y; f[6] = hi.z; f[7] = hi.w;
+}
+__device__ __forceinline__ void st8f(float* p, const float (&f)[8]) {
+    reinterpret_cast<float4*>(p)[0] = make_float4(f[0], f[1], f[2], f[3]);
+    reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
+}
+
+// Offset of the second staged vector of the AddNorm prologue (behind red + misc).
+__host__ __device__ inline unsigned int gemv_ext_off(int K) { return gemv_xbytes(K) + gemv_wbytes(K) + (2 * 16 * 2 + 16) * 4u; }
+
+// EXT prologues; false: not one of them.  Ends with a block barrier.
+__device__ __forceinline__ bool gemv_stage_ext(const GemvParams& p, const int nch, unsigned char* smem, const unsigned int xbytes) {
+    __shared__ float red3[3 * kGemvWarps];
+    float* xs = reinterpret_cast<float*>(smem);
+    const int tid = threadIdx.x;
+    if (p.prologue == kProEmbed) {
+        const int tok = p.state->token;
+        const bool zero = tok < 0 || tok >= p.vocab;
+        const __nv_bfloat16* row = p.embed_table + (size_t)(zero ? 0 : tok) * p.K;
+        for (int c = tid; c < nch; c += kGemvThreads) {
+            float f[8];
+            unpack8(zero ? make_uint4(0, 0, 0, 0) : ld_cached(row + (size_t)c * 8), f);
+            st8f(xs + 8 * c, f);
+            if (blockIdx.x == 0) st8f(p.resid_out + 8 * c, f);
+        }
+    } else if (p.prologue == kProAddNorm) {
+        const uint4* gs = reinterpret_cast<const uint4*>(smem + xbytes);
+        float* xs2 = reinterpret_cast<float*>(smem + gemv_ext_off(p.K));
+        float ss[1] = {0.f};
+        for (int c = tid; c < nch; c += kGemvThreads) {
+            float y[8], x[8];
+            ld8f(p.addend + 8 * c, y);
+            ld8f(p.xr + 8 * c, x);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) ss[0] = fmaf(y[j], y[j], ss[0]);
+            st8f(xs + 8 * c, y);
+            st8f(xs2 + 8 * c, x);
+        }
+        gemv_block_sums<1>(ss, red3);
+        const float inv = 1.0f / sqrtf(ss[0] / (float)p.k_true + p.eps);
+        float s2[1] = {0.f};
+        for (int c = tid; c < nch; c += kGemvThreads) {       // same thread, same chunks as above
+            float w[8], x[8];
+            unpack8(gs[c], w);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                x[j] = xs2[8 * c + j] + xs[8 * c + j] * inv * w[j];
+                s2[0] = fmaf(x[j], x[j], s2[0]);
+            }
+            st8f(xs + 8 * c, x);
+            if (blockIdx.x == 0) st8f(p.resid_out + 8 * c, x);
+        }
+        if (p.norm2_w != nullptr) {
+            gemv_block_sums<1>(s2, red3 + kGemvWarps);
+            const float inv2 = 1.0f / sqrtf(s2[0] / (float)p.k_true + p.eps);
+            for (int c = tid; c < nch; c += kGemvThreads) {
+                float w[8], x[8];
+                unpack8(ld_cached(p.norm2_w + (size_t)c * 8), w);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) x[j] = xs[8 * c + j] * inv2 * w[j];
+                st8f(xs + 8 * c, x);
+            }
+        }
+    } else if (p.prologue == kProPolyNorm) {
+        float s[3] = {0.f, 0.f, 0.f};
+        for (int c = tid; c < nch; c += kGemvThreads) {
+            float z[8];
+            ld8f(p.xf + 8 * c, z);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                const float z2 = z[j] * z[j], z4 = z2 * z2;
+                s[0] += z2;
+                s[1] += z4;
+                s[2] = fmaf(z4, z2, s[2]);
+            }
+            st8f(xs + 8 * c, z);
+        }
+        gemv_block_sums<3>(s, red3);
+        const float n = (float)p.k_true;
+        const float c0 = __bfloat162float(p.poly[0]) / sqrtf(s[0] / n + p.eps), c1 = __bfloat162float(p.poly[1]) / sqrtf(s[1] / n + p.eps),
+                    c2 = __bfloat162float(p.poly[2]) / sqrtf(s[2] / n + p.eps), c3 = __bfloat162float(p.poly[3]);
+        for (int c = tid; c < nch; c += kGemvThreads) {
+            float z[8];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                z[j] = xs[8 * c + j];
+                z[j] = fmaf(z[j], fmaf(z[j], fmaf(z[j], c2, c1), c0), c3);
+            }
+            st8f(xs + 8 * c, z);
+        }
+    } else {
+        return false;
+    }
+    __syncthreads();
+    return true;
 }
 
 // Activations of one GEMV phase into shared memory as fp32 [K], with the fused prologue (embedding row / residual
@@ -352,7 +496,7 @@ __device__ __forceinline__ void gemv_stage(const GemvParams& p, const int nch, u
 }
 
 // Stage activations (with the fused norm), stream the rows, reduce, epilogue.
-template <Epi EPI>
+template <Epi EPI, bool EXT>
 __device__ __forceinline__ void gemv_run(const GemvParams& p, const GemvSched& sc, GemvRegs& r, unsigned char* smem,
                                          const unsigned int xbytes, float& best_v, int& best_i) {
     const float* xs = reinterpret_cast<const float*>(smem);
@@ -366,7 +510,11 @@ __device__ __forceinline__ void gemv_run(const GemvParams& p, const GemvSched& s
         if (sc.wk == 0 && lane == 0 && sc.total > 0)
             old_first = __ldcg(reinterpret_cast<const float2*>(p.residual + sc.ig0 * 2));
     }
-    gemv_stage(p, nch, smem, xbytes);
+    if constexpr (EXT) {
+        if (!gemv_stage_ext(p, nch, smem, xbytes)) gemv_stage(p, nch, smem, xbytes);
+    } else {
+        gemv_stage(p, nch, smem, xbytes);
+    }
     (void)tid;
 
     // ---- rows ------------------------------------------------------------------------------------
@@ -438,7 +586,7 @@ __device__ __forceinline__ void gemv_publish_best(const GemvParams& p, float bes
 }
 
 // One GEMV phase as its own launch (phase-per-launch decode form, prefill lm_head, operator API).
-template <Epi EPI>
+template <Epi EPI, bool EXT = false>
 __global__ void __launch_bounds__(kGemvThreads, 1) gemv_kernel(const GemvParams p, const int ks) {
     extern __shared__ __align__(16) unsigned char gemv_smem[];
     __shared__ float bv[kGemvWarps];
@@ -451,10 +599,10 @@ __global__ void __launch_bounds__(kGemvThreads, 1) gemv_kernel(const GemvParams 
     // one is resident, then prefetch (independent of every earlier kernel), then wait.
     pdl_launch_dependents();
     const GemvSched sc = gemv_sched(p, ks, blockIdx.x, gridDim.x);
-    gemv_prefetch<EPI>(p, sc, regs, gemv_smem, xbytes);
+    gemv_prefetch<EPI, EXT>(p, sc, regs, gemv_smem, xbytes);
     pdl_wait();
     if constexpr (EPI == Epi::Peers) best_i = (int)(__ldcg(p.epoch) + 1u);      // this launch's exchange count rides in best_i
-    gemv_run<EPI>(p, sc, regs, gemv_smem, xbytes, best_v, best_i);
+    gemv_run<EPI, EXT>(p, sc, regs, gemv_smem, xbytes, best_v, best_i);
     if constexpr (EPI == Epi::Logits) gemv_publish_best(p, best_v, best_i, bv, bi);
     if constexpr (EPI == Epi::Peers) {
         // every block has read the count by now; the one that draws the last ticket advances it for the consumer
@@ -472,5 +620,8 @@ __global__ void __launch_bounds__(kGemvThreads, 1) gemv_kernel(const GemvParams 
 __host__ __device__ inline size_t gemv_smem_bytes(int K) {      // xs (fp32) | norm weight | red + misc
     return (size_t)gemv_xbytes(K) + gemv_wbytes(K) + (size_t)(2 * kGemvWarps * 2 + 16) * sizeof(float);
 }
+
+// EXT instantiations: room for the second vector of the AddNorm prologue.
+__host__ __device__ inline size_t gemv_ext_smem_bytes(int K) { return (size_t)gemv_ext_off(K) + (size_t)K * 4; }
 
 }  // namespace efm

@@ -1,0 +1,426 @@
+// Causal softmax attention over a paged cache with a sliding window and per-head score modification:
+//   score(i, j) = (q_i . k_j) * scale * temp[h] - slope_h * (i - j),   0 <= i - j < window   (window 0: no lower bound)
+// with slope_h = 2^(-8 (h + 1) / H), q and k RMS-normalised per head before they are used / cached, value width free.
+// Cache: per layer a K pool [pages * 64][kv_heads][Dp] and a V pool [pages * 64][kv_heads][Vp], channels zero-padded to
+// Dp / Vp (multiples of 64); a sequence's pages are listed in a page table.  TC = bf16 or fp32 (the all-32-bit mode).
+//
+//   qk_scatter_rows      many rows: per-head norms, q -> [T][H][Dp], k and v -> cache rows
+//   window_attention_rows many rows on the CUDA cores, fp32 throughout (32-bit mode, short portions, head sizes the
+//                        tensor-core form does not take)
+//   window_attention_decode one row: norms of q and k, cache append and split-key attention in one launch; the splits of
+//                        a kv head are the blocks of one cluster and merge through distributed shared memory
+#pragma once
+#include <cooperative_groups.h>
+
+#include "common.cuh"
+#include "row_plan.cuh"
+
+namespace efm {
+
+struct WindowAttnShape {
+    int H, G, D, Dv, Dp, Vp;          // query heads, kv heads, channels and padded channels
+    int window;                       // 0: full causal
+    int bias;                         // 1: distance bias
+    float scale, eps;
+    const __nv_bfloat16* q_norm;      // [D]
+    const __nv_bfloat16* k_norm;      // [D]
+    const __nv_bfloat16* temp;        // [H]
+};
+
+__device__ __forceinline__ float to_f32(float v) { return v; }
+__device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ void store_f32(float* p, float v) { *p = v; }
+__device__ __forceinline__ void store_f32(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ float distance_slope(int h, int H) { return exp2f(-8.0f * (float)(h + 1) / (float)H); }
+template <typename T> __device__ __forceinline__ float round_as(float v);
+template <> __device__ __forceinline__ float round_as<float>(float v) { return v; }
+template <> __device__ __forceinline__ float round_as<__nv_bfloat16>(float v) { return round_bf16(v); }
+
+// ---- many rows: norms and scatter --------------------------------------------------------------------------------
+// One block per row, one warp per head at a time.  TI: projections, TQ: q operand, TC: cache.
+template <typename TI, typename TQ, typename TC>
+__global__ void __launch_bounds__(256) qk_scatter_rows_kernel(const TI* __restrict__ qkv, int ld, TQ* __restrict__ q_out, TC* __restrict__ k_pool,
+                                                              TC* __restrict__ v_pool, const WindowAttnShape s, const RowPlan plan) {
+    const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const RowEntry e = plan.of_row(row);
+    const size_t cr = plan.cache_row(e, e.pos0 + row - e.row0);
+    const TI* src = qkv + (size_t)row * ld;
+    for (int u = warp; u < s.H + 2 * s.G; u += 8) {
+        if (u < s.H + s.G) {
+            const bool is_q = u < s.H;
+            const TI* x = src + (size_t)u * s.D;                       // q heads, then k heads
+            const __nv_bfloat16* w = is_q ? s.q_norm : s.k_norm;
+            float ss = 0.f;
+            for (int d = lane; d < s.D; d += 32) { const float v = to_f32(x[d]); ss = fmaf(v, v, ss); }
+            const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)s.D + s.eps);
+            TQ* qd = q_out + ((size_t)row * s.H + u) * s.Dp;
+            TC* kd = k_pool + (cr * s.G + (u - s.H)) * s.Dp;
+            for (int d = lane; d < s.Dp; d += 32) {
+                const float v = d < s.D ? to_f32(x[d]) * inv * __bfloat162float(w[d]) : 0.f;
+                if (is_q) store_f32(qd + d, v); else store_f32(kd + d, v);
+            }
+        } else {
+            const int g = u - s.H - s.G;
+            const TI* x = src + (size_t)(s.H + s.G) * s.D + (size_t)g * s.Dv;
+            TC* vd = v_pool + (cr * s.G + g) * s.Vp;
+            for (int d = lane; d < s.Vp; d += 32) store_f32(vd + d, d < s.Dv ? to_f32(x[d]) : 0.f);
+        }
+    }
+}
+
+// ---- many rows on the CUDA cores ---------------------------------------------------------------------------------
+namespace wa {
+constexpr int QT = 16, KT = 32;
+inline size_t rows_smem_bytes(int Dp, int Vp) { return (size_t)(QT * (Dp + 4) + KT * (Dp + 4) + KT * (Vp + 4) + QT * (KT + 1)) * sizeof(float); }
+}  // namespace wa
+
+// Block = 16 rows of one entry x one head; keys in tiles of 32 staged as fp32.  tiles: [gridDim.x] (null: the single
+// entry's rows in order).  out: [T][H * Dv].
+template <typename TQ, typename TC, typename TO>
+__global__ void __launch_bounds__(256) window_attention_rows_kernel(const TQ* __restrict__ q, const TC* __restrict__ k_pool, const TC* __restrict__ v_pool,
+                                                                    TO* __restrict__ out, int ld_out, const WindowAttnShape s, const RowPlan plan,
+                                                                    const RowTile* __restrict__ tiles) {
+    using namespace wa;
+    extern __shared__ __align__(16) float wa_smem[];
+    const int tid = threadIdx.x, h = blockIdx.y, g = h / (s.H / s.G);
+    const int DS = s.Dp + 4, VS = s.Vp + 4;
+    float* qs = wa_smem;
+    float* ks = qs + QT * DS;
+    float* vs = ks + KT * DS;
+    float* ps = vs + KT * VS;
+    RowEntry e;
+    int r0;                                                            // first row inside the entry
+    if (tiles != nullptr) { const RowTile t = tiles[blockIdx.x]; e = plan.entry(t.entry); r0 = t.row; }
+    else { e = plan.one; r0 = blockIdx.x * QT; }
+    const int nq = min(QT, e.n - r0);
+    for (int i = tid; i < QT * s.Dp; i += 256) {
+        const int r = i / s.Dp, d = i - r * s.Dp;
+        qs[r * DS + d] = r < nq ? to_f32(q[((size_t)(e.row0 + r0 + r) * s.H + h) * s.Dp + d]) : 0.f;
+    }
+    const int r = tid >> 4, c = tid & 15;
+    const int i_pos = e.pos0 + r0 + r;                                 // this row's position
+    const int lo = s.window > 0 ? max(0, i_pos - s.window + 1) : 0;
+    const int first = s.window > 0 ? max(0, e.pos0 + r0 - s.window + 1) : 0;
+    const int end = e.pos0 + r0 + nq;                                  // one past the last visible key of the block
+    const float mul = s.scale * __bfloat162float(s.temp[h]);
+    const float slope = s.bias ? distance_slope(h, s.H) : 0.f;
+    float acc[4][4];
+#pragma unroll
+    for (int n = 0; n < 4; ++n)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[n][j] = 0.f;
+    float m = -INFINITY, l = 0.f;
+    for (int k0 = first & ~(KT - 1); k0 < end; k0 += KT) {
+        __syncthreads();
+        for (int i = tid; i < KT * s.Dp; i += 256) {
+            const int kr = i / s.Dp, d = i - kr * s.Dp;
+            ks[kr * DS + d] = k0 + kr < end ? to_f32(k_pool[(plan.cache_row(e, k0 + kr) * s.G + g) * s.Dp + d]) : 0.f;
+        }
+        for (int i = tid; i < KT * s.Vp; i += 256) {
+            const int kr = i / s.Vp, d = i - kr * s.Vp;
+            vs[kr * VS + d] = k0 + kr < end ? to_f32(v_pool[(plan.cache_row(e, k0 + kr) * s.G + g) * s.Vp + d]) : 0.f;
+        }
+        __syncthreads();
+        float sc[2];
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+            const int j = k0 + c + 16 * u;
+            float d0 = 0.f, d1 = 0.f;
+            const float4* a = reinterpret_cast<const float4*>(qs + r * DS);
+            const float4* b = reinterpret_cast<const float4*>(ks + (c + 16 * u) * DS);
+            for (int t = 0; t < s.Dp / 4; ++t) {
+                const float4 x = a[t], y = b[t];
+                d0 = fmaf(x.x, y.x, d0); d1 = fmaf(x.y, y.y, d1); d0 = fmaf(x.z, y.z, d0); d1 = fmaf(x.w, y.w, d1);
+            }
+            sc[u] = (j >= lo && j <= i_pos) ? (d0 + d1) * mul - slope * (float)(i_pos - j) : -INFINITY;
+        }
+        float mx = fmaxf(sc[0], sc[1]);
+#pragma unroll
+        for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        const float mn = fmaxf(m, mx), mb = mn == -INFINITY ? 0.f : mn;
+        const float alpha = m == -INFINITY ? 0.f : expf(m - mb);
+        m = mn;
+        float rs = 0.f;
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+            const float p = sc[u] == -INFINITY ? 0.f : expf(sc[u] - mb);
+            rs += p;
+            ps[r * (KT + 1) + c + 16 * u] = p;
+        }
+#pragma unroll
+        for (int o = 8; o > 0; o >>= 1) rs += __shfl_xor_sync(0xffffffffu, rs, o);
+        l = l * alpha + rs;
+#pragma unroll
+        for (int n = 0; n < 4; ++n)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) acc[n][j] *= alpha;
+        __syncwarp();                                                  // the 16 lanes of a row share a warp
+        for (int kr = 0; kr < KT; ++kr) {
+            const float p = ps[r * (KT + 1) + kr];
+#pragma unroll
+            for (int n = 0; n < 4; ++n)
+                if (n * 64 < s.Vp) {
+                    const float4 v = *reinterpret_cast<const float4*>(vs + kr * VS + n * 64 + c * 4);
+                    acc[n][0] = fmaf(p, v.x, acc[n][0]); acc[n][1] = fmaf(p, v.y, acc[n][1]);
+                    acc[n][2] = fmaf(p, v.z, acc[n][2]); acc[n][3] = fmaf(p, v.w, acc[n][3]);
+                }
+        }
+    }
+    if (r >= nq) return;
+    const float inv = l > 0.f ? 1.0f / l : 0.f;
+    TO* dst = out + (size_t)(e.row0 + r0 + r) * ld_out + (size_t)h * s.Dv;
+#pragma unroll
+    for (int n = 0; n < 4; ++n)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int d = n * 64 + c * 4 + j;
+            if (d < s.Dv) store_f32(dst + d, acc[n][j] * inv);
+        }
+}
+
+// ---- one row -----------------------------------------------------------------------------------------------------
+namespace wd {
+constexpr int kThreads = 256, kHeads = 8;      // query heads per block (of one kv head)
+template <int VM>
+struct Smem {
+    static constexpr int MAXP = VM;            // padded channels at most
+    float q[kHeads][MAXP + 8];
+    float knew[MAXP], vnew[MAXP];
+    float p[kHeads][kPageTokens];
+    float alpha[kHeads], m[kHeads], l[kHeads];
+    float out[kHeads][MAXP];                   // this block's un-normalised output
+    float red[8192];                           // [key groups][kHeads][Vp]: at most 256 / (Vp / 4) * 8 * Vp = 8192
+};
+}  // namespace wd
+
+template <typename TC>
+struct WindowDecodeParams {
+    WindowAttnShape s;
+    const float* qkv;                 // [H * D | G * D | G * Dv]
+    TC* k_pool;
+    TC* v_pool;
+    const int32_t* pages;             // page table row of the sequence
+    int max_pages;
+    DecodeState* state;
+    float* out;                       // [H * Dv]
+    int early;                        // 1: state and the older cache rows may be read before the dependency wait
+};
+
+// 8 channels of a cache row as fp32
+template <typename TC> struct Row8;
+template <> struct Row8<__nv_bfloat16> {
+    uint4 v;
+    __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = ld_cg(p); }
+    __device__ __forceinline__ void get(float (&f)[8]) const { unpack8(v, f); }
+};
+template <> struct Row8<float> {
+    float4 a, b;
+    __device__ __forceinline__ void load(const float* p) { a = __ldcg(reinterpret_cast<const float4*>(p)); b = __ldcg(reinterpret_cast<const float4*>(p) + 1); }
+    __device__ __forceinline__ void get(float (&f)[8]) const { f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w; }
+};
+template <typename TC> struct Row4;
+template <> struct Row4<__nv_bfloat16> {
+    uint2 v;
+    __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = __ldcg(reinterpret_cast<const uint2*>(p)); }
+    __device__ __forceinline__ void get(float (&f)[4]) const { f[0] = bf16lo(v.x); f[1] = bf16hi(v.x); f[2] = bf16lo(v.y); f[3] = bf16hi(v.y); }
+};
+template <> struct Row4<float> {
+    float4 v;
+    __device__ __forceinline__ void load(const float* p) { v = __ldcg(reinterpret_cast<const float4*>(p)); }
+    __device__ __forceinline__ void get(float (&f)[4]) const { f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w; }
+};
+
+// grid (splits = cluster size, kv_heads * head blocks); block `split` walks every splits-th page of the visible range.
+// VM: upper bound of Dp and Vp.
+template <typename TC, int VM>
+__global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(const WindowDecodeParams<TC> p) {
+    using namespace wd;
+    constexpr int KC = VM / 32;                                        // 8-channel chunks per thread and key (4 threads per key)
+    constexpr int VK = VM <= 64 ? 4 : (VM <= 128 ? 8 : 16);            // keys per thread in the P.V phase
+    extern __shared__ __align__(16) unsigned char wd_smem[];
+    Smem<VM>& sm = *reinterpret_cast<Smem<VM>*>(wd_smem);
+    const WindowAttnShape& s = p.s;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int split = blockIdx.x, n_splits = gridDim.x;
+    const int group = s.H / s.G, hb = (group + kHeads - 1) / kHeads;
+    const int g = blockIdx.y / hb, h0 = g * group + (blockIdx.y % hb) * kHeads, nh = min(kHeads, (g + 1) * group - h0);
+    const int key = tid >> 2, part = tid & 3;                          // score phase
+    const int tpr = s.Vp / 4, kg = kThreads / tpr, dpart = tid % tpr, tg = tid / tpr;     // P.V phase: 4 channels per thread
+    const bool pv = tg < kg;
+
+    if (!p.early) { pdl_wait(); pdl_launch_dependents(); }
+    const int kv_len = (int)p.state->kv_len, pos = kv_len - 1;
+    const bool ok = kv_len > 0 && kv_len <= p.max_pages * kPageTokens;
+    const int lo = s.window > 0 ? max(0, kv_len - s.window) : 0;
+    const int pg0 = lo / kPageTokens, pg1 = ok ? pos / kPageTokens : pg0 - 1;
+
+    Row8<TC> kr[KC];
+    Row4<TC> vr[VK];
+    // rows of page `pg` except the one this launch appends
+    auto load_page = [&](int pg) {
+        const size_t base = (size_t)p.pages[pg] * kPageTokens;
+        const int j = pg * kPageTokens + key;
+        if (j >= lo && j < pos) {
+#pragma unroll
+            for (int c = 0; c < KC; ++c)
+                if ((c * 4 + part) * 8 < s.Dp) kr[c].load(p.k_pool + ((base + key) * s.G + g) * s.Dp + (c * 4 + part) * 8);
+        }
+        if (pv) {
+#pragma unroll
+            for (int i = 0; i < VK; ++i) {
+                const int kk = tg + i * kg, jj = pg * kPageTokens + kk;
+                if (kk < kPageTokens && jj >= lo && jj < pos) vr[i].load(p.v_pool + ((base + kk) * s.G + g) * s.Vp + dpart * 4);
+            }
+        }
+    };
+    int pg = pg0 + split;
+    if (pg <= pg1) load_page(pg);
+    if (p.early) { pdl_wait(); pdl_launch_dependents(); }
+
+    // ---- norms of this token's q heads and k, v ------------------------------------------------------------------
+    for (int u = warp; u < nh + 1; u += 8) {
+        const bool is_q = u < nh;
+        const float* x = is_q ? p.qkv + (size_t)(h0 + u) * s.D : p.qkv + (size_t)(s.H + g) * s.D;
+        const __nv_bfloat16* w = is_q ? s.q_norm : s.k_norm;
+        float ss = 0.f;
+        for (int d = lane; d < s.D; d += 32) { const float v = __ldcg(x + d); ss = fmaf(v, v, ss); }
+        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)s.D + s.eps);
+        for (int d = lane; d < s.Dp; d += 32) {
+            const float v = d < s.D ? __ldcg(x + d) * inv * __bfloat162float(w[d]) : 0.f;
+            if (is_q) sm.q[u][d] = v; else sm.knew[d] = round_as<TC>(v);
+        }
+    }
+    for (int d = tid; d < s.Vp; d += kThreads)
+        sm.vnew[d] = d < s.Dv ? round_as<TC>(__ldcg(p.qkv + (size_t)(s.H + s.G) * s.D + (size_t)g * s.Dv + d)) : 0.f;
+    if (tid < kHeads) { sm.m[tid] = -INFINITY; sm.l[tid] = 0.f; }
+    __syncthreads();
+    if (ok && pg1 % n_splits == (split + pg0) % n_splits && pg1 >= pg0 + split && blockIdx.y % hb == 0) {     // the block that walks the last page appends
+        const size_t cr = (size_t)p.pages[pg1] * kPageTokens + pos % kPageTokens;
+        for (int d = tid; d < s.Dp; d += kThreads) store_f32(p.k_pool + (cr * s.G + g) * s.Dp + d, sm.knew[d]);
+        for (int d = tid; d < s.Vp; d += kThreads) store_f32(p.v_pool + (cr * s.G + g) * s.Vp + d, sm.vnew[d]);
+    }
+    if (!ok && tid == 0) p.state->error = 2;
+
+    float acc[kHeads][4];
+#pragma unroll
+    for (int h = 0; h < kHeads; ++h)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[h][j] = 0.f;
+
+    for (; pg <= pg1; pg += n_splits) {
+        const int j = pg * kPageTokens + key;
+        const bool vis = j >= lo && j <= pos;
+        // ---- scores: 4 threads per key ----------------------------------------------------------------------------
+        float kf[KC][8];
+#pragma unroll
+        for (int c = 0; c < KC; ++c) {
+            const int d0 = (c * 4 + part) * 8;
+            if (d0 < s.Dp && j == pos) {
+#pragma unroll
+                for (int i = 0; i < 8; ++i) kf[c][i] = sm.knew[d0 + i];
+            } else {
+                kr[c].get(kf[c]);
+            }
+        }
+        for (int h = 0; h < nh; ++h) {
+            float d = 0.f;
+            if (vis) {
+#pragma unroll
+                for (int c = 0; c < KC; ++c) {
+                    const int d0 = (c * 4 + part) * 8;
+                    if (d0 < s.Dp) {
+                        const float4 a = *reinterpret_cast<const float4*>(&sm.q[h][d0]), b = *reinterpret_cast<const float4*>(&sm.q[h][d0 + 4]);
+                        d = fmaf(a.x, kf[c][0], d); d = fmaf(a.y, kf[c][1], d); d = fmaf(a.z, kf[c][2], d); d = fmaf(a.w, kf[c][3], d);
+                        d = fmaf(b.x, kf[c][4], d); d = fmaf(b.y, kf[c][5], d); d = fmaf(b.z, kf[c][6], d); d = fmaf(b.w, kf[c][7], d);
+                    }
+                }
+            }
+            d += __shfl_xor_sync(0xffffffffu, d, 1);
+            d += __shfl_xor_sync(0xffffffffu, d, 2);
+            if (part == 0) {
+                const float slope = s.bias ? distance_slope(h0 + h, s.H) : 0.f;
+                sm.p[h][key] = vis ? d * (s.scale * __bfloat162float(s.temp[h0 + h])) - slope * (float)(pos - j) : -INFINITY;
+            }
+        }
+        __syncthreads();
+        // ---- online softmax: one warp per head --------------------------------------------------------------------
+        if (warp < nh) {
+            const float s0 = sm.p[warp][lane], s1 = sm.p[warp][lane + 32];
+            const float m_old = sm.m[warp], mn = fmaxf(m_old, warp_max(fmaxf(s0, s1)));       // the page holds a visible key
+            const float p0 = expf(s0 - mn), p1 = expf(s1 - mn);
+            sm.p[warp][lane] = p0;
+            sm.p[warp][lane + 32] = p1;
+            const float sum = warp_sum(p0 + p1);
+            if (lane == 0) {
+                const float al = expf(m_old - mn);
+                sm.alpha[warp] = al;
+                sm.m[warp] = mn;
+                sm.l[warp] = sm.l[warp] * al + sum;
+            }
+        }
+        __syncthreads();
+        if (pv) {
+#pragma unroll
+            for (int h = 0; h < kHeads; ++h)
+                if (h < nh) {
+                    const float al = sm.alpha[h];
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) acc[h][c] *= al;
+                }
+#pragma unroll
+            for (int i = 0; i < VK; ++i) {
+                const int kk = tg + i * kg, jj = pg * kPageTokens + kk;
+                if (kk < kPageTokens && jj >= lo && jj <= pos) {
+                    float v[4];
+                    if (jj == pos) {
+#pragma unroll
+                        for (int c = 0; c < 4; ++c) v[c] = sm.vnew[dpart * 4 + c];
+                    } else {
+                        vr[i].get(v);
+                    }
+#pragma unroll
+                    for (int h = 0; h < kHeads; ++h)
+                        if (h < nh) {
+                            const float w = sm.p[h][kk];
+#pragma unroll
+                            for (int c = 0; c < 4; ++c) acc[h][c] = fmaf(w, v[c], acc[h][c]);
+                        }
+                }
+            }
+        }
+        if (pg + n_splits <= pg1) load_page(pg + n_splits);
+        __syncthreads();
+    }
+    // ---- sum over the key groups, then over the splits -------------------------------------------------------------
+    if (pv) {
+#pragma unroll
+        for (int h = 0; h < kHeads; ++h)
+            if (h < nh) *reinterpret_cast<float4*>(sm.red + ((size_t)tg * kHeads + h) * s.Vp + dpart * 4) = make_float4(acc[h][0], acc[h][1], acc[h][2], acc[h][3]);
+    }
+    __syncthreads();
+    for (int i = tid; i < nh * s.Vp; i += kThreads) {
+        const int h = i / s.Vp, d = i - h * s.Vp;
+        float v = 0.f;
+        for (int t = 0; t < kg; ++t) v += sm.red[((size_t)t * kHeads + h) * s.Vp + d];
+        sm.out[h][d] = v;
+    }
+    namespace cg = cooperative_groups;
+    cg::cluster_group cl = cg::this_cluster();
+    cl.sync();
+    for (int i = split * kThreads + tid; i < nh * s.Dv; i += n_splits * kThreads) {
+        const int h = i / s.Dv, d = i - h * s.Dv;
+        float m = -INFINITY;
+        for (int r = 0; r < n_splits; ++r) m = fmaxf(m, *cl.map_shared_rank(&sm.m[h], r));
+        float num = 0.f, den = 0.f;
+        for (int r = 0; r < n_splits; ++r) {
+            const float mr = *cl.map_shared_rank(&sm.m[h], r);
+            const float w = mr == -INFINITY ? 0.f : expf(mr - m);
+            num = fmaf(w, *cl.map_shared_rank(&sm.out[h][d], r), num);
+            den = fmaf(w, *cl.map_shared_rank(&sm.l[h], r), den);
+        }
+        p.out[(size_t)(h0 + h) * s.Dv + d] = den > 0.f ? num / den : 0.f;
+    }
+    cl.sync();
+}
+
+}  // namespace efm

@@ -151,6 +151,39 @@ PYBIND11_MODULE(edge_fm, m) {
     py::class_<EdgeFM>(m, "EdgeFM")
         .def(py::init<const std::string&>(), py::arg("config_path"))
         .def("generate", &EdgeFM::generate, py::arg("request"), py::call_guard<py::gil_scoped_release>())
+        .def("generate_batch",
+             [](const EdgeFM& self, const py::list& requests) {
+                 std::vector<const Request*> in;
+                 for (const py::handle& h : requests) in.push_back(py::cast<const Request*>(h));
+                 py::gil_scoped_release release;
+                 return self.generate_batch(in);
+             },
+             py::arg("requests"))
+        .def("step",
+             [](const EdgeFM& self, const py::list& entries) {
+                 std::vector<StepEntry> in;
+                 size_t n_want = 0;
+                 for (const py::handle& h : entries) {
+                     const py::tuple t = py::cast<py::tuple>(h);
+                     StepEntry e{py::cast<std::string>(t[0]), py::cast<std::vector<int32_t>>(t[1]), {}};
+                     if (t.size() > 2) e.want = py::cast<std::vector<int32_t>>(t[2]);
+                     n_want += e.want.size();
+                     in.push_back(std::move(e));
+                 }
+                 std::vector<float> logits;
+                 {
+                     py::gil_scoped_release release;
+                     logits = self.step(in);
+                 }
+                 const size_t vocab = (size_t)self.vocab_size();
+                 py::list rows;
+                 for (size_t i = 0; i < n_want; ++i)
+                     rows.append(py::bytes(reinterpret_cast<const char*>(logits.data() + i * vocab), vocab * sizeof(float)));
+                 return rows;
+             },
+             py::arg("entries"), "entries: (id, tokens, want) tuples -> one fp32 byte row [vocab] per wanted place")
+        .def("finish", &EdgeFM::finish, py::arg("id"))
+        .def("vocab_size", &EdgeFM::vocab_size)
         .def("plan",
              [](const EdgeFM& self, int32_t request_id, const py::dict& inputs) {
                  TensorRefMap refs = tensor_ref_map_from_py_dict(inputs);

@@ -359,6 +359,81 @@ EFM_API efm_status efm_b200_vit_encode(efm_b200_vit* vit, const void* pixels, in
                                        const int32_t* grid_thw, int32_t n_grids, void* out,
                                        int32_t out_mem);
 
+/* ---- layered decoders ---------------------------------------------------------------------
+ * A decoder described layer by layer: every layer names its mixer (softmax attention or the generalised delta rule), the
+ * mixer's sizes and an optional dense feed-forward; sublayer outputs are RMS-normalised before the residual add; an
+ * optional per-layer token input follows.  (No counterpart in the reference.)  Such a context serves the same calls as
+ * the text tower (set_weight, finalize_weights, prefill, decode_begin, decode_steps, read_tokens, read_logits, ...) and,
+ * in addition, batched steps over a paged cache: one pool of 64-token pages per attention layer and one pool of recurrent
+ * state slots, handed out by the caller (who maps page numbers to sequences).
+ *
+ * Tensor names: embed, side.embed, final.norm, head and, for layer i, l<i>.norm1 / norm2, l<i>.mix.{q,k,v,o,q.norm,k.norm,
+ * temp} (attention) or l<i>.mix.{r,k,v,g,a,a.b,w1,w2,w0,norm,o} (delta rule), l<i>.mlp.{up,down,act},
+ * l<i>.side.{gate,proj,norm}; bf16. */
+enum { EFM_MIXER_ATTENTION = 0, EFM_MIXER_GENERAL_DELTA = 1 };
+enum { EFM_PAGE_TOKENS = 64 };
+
+typedef struct efm_decoder_layer {
+    int32_t mixer;                /* EFM_MIXER_* */
+    int32_t heads;
+    int32_t kv_heads;             /* attention only */
+    int32_t dim;                  /* per-head key channels (delta rule: value channels too), <= 256 */
+    int32_t vdim;                 /* attention: per-head value channels, <= 256 */
+    int32_t window;               /* attention: position i sees j with 0 <= i - j < window; 0: all j <= i */
+    int32_t distance_bias;        /* attention: 1 = subtract 2^(-8 (h+1) / heads) * (i - j) from the score of head h */
+    float scale;                  /* attention: score multiplier */
+    int32_t decay_rank;           /* delta rule: rows of w1, <= 512 */
+    int32_t ff;                   /* feed-forward width, 0: none */
+} efm_decoder_layer;
+
+typedef struct efm_decoder_desc {
+    int32_t struct_size;          /* = sizeof(efm_decoder_desc) */
+    int32_t num_layers, vocab, width;
+    int32_t side_dim;             /* per-layer token input width, 0: none */
+    float norm_eps;
+    int32_t compute_dtype;        /* EFM_BF16: matrix products on bf16 operands; EFM_F32: everything in 32-bit */
+    int32_t max_step_tokens;      /* rows one pass computes; longer steps run in several passes */
+    int32_t max_response_tokens;
+    int32_t cache_pages;          /* pages of each attention layer's pool */
+    int32_t state_slots;          /* recurrent state slots */
+    int32_t max_slots;            /* sequences mapped at a time */
+} efm_decoder_desc;
+
+EFM_API efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decoder_layer* layers, int32_t device_id,
+                                           efm_b200_ctx** out);
+/* Maps sequence `slot` (any number) to pool pages pages[0..n_pages) (page k holds positions [64 k, 64 k + 64)) and to a
+ * state slot (-1 when the model keeps no recurrent state).  A new slot starts empty; mapping an existing one again
+ * changes its pages (those that hold tokens must keep their contents) and keeps its length. */
+EFM_API efm_status efm_b200_decoder_map_slot(efm_b200_ctx* ctx, int32_t slot, const int32_t* pages, int32_t n_pages,
+                                             int32_t state_slot);
+EFM_API efm_status efm_b200_decoder_unmap_slot(efm_b200_ctx* ctx, int32_t slot);
+/* The tokens `slot` holds now become a fixed prefix: its recurrent state is copied to `pin_state`, and a later prefill or
+ * step at kv_offset = that length starts from the copy (the cache pages of the prefix are never rewritten). */
+EFM_API efm_status efm_b200_decoder_pin_prefix(efm_b200_ctx* ctx, int32_t slot, int32_t pin_state);
+
+/* One entry of a batched step: n_tokens new tokens of `slot` at positions kv_offset ... (kv_offset must be what the slot
+ * holds, its pinned prefix, or 0: start over); the logits at want[0..n_want) (indices into tokens) are returned. */
+typedef struct efm_step_entry {
+    int32_t slot;
+    int32_t n_tokens;
+    int32_t kv_offset;
+    int32_t n_want;
+    uint32_t rng_step;            /* random counter of the entry's samples */
+    uint32_t reserved;
+    const int32_t* tokens;        /* host */
+    const int32_t* want;          /* host, ascending order not required */
+} efm_step_entry;
+
+/* All entries run as one batch.  logits: host fp32 [sum of n_want, vocab] in entry order (may be NULL when nothing is
+ * wanted); sampled: host int32 [sum of n_want] or NULL: the wanted rows sampled with the context's sampling parameters
+ * and the entry's random counter.  Synchronises when something is returned. */
+EFM_API efm_status efm_b200_decoder_step(efm_b200_ctx* ctx, const efm_step_entry* entries, int32_t n_entries,
+                                         float* logits, int32_t* sampled);
+/* Residual stream after every layer of the steps that follow: copied to host_out [num_layers, rows, width] by
+ * efm_b200_decoder_read_taps.  rows = 0 switches it off. */
+EFM_API efm_status efm_b200_decoder_set_taps(efm_b200_ctx* ctx, int32_t rows);
+EFM_API efm_status efm_b200_decoder_read_taps(efm_b200_ctx* ctx, float* host_out);
+
 /* ---- SmolVLA-shaped action chunk ----------------------------------------------------------
  * The reference describes this model (doc/smolvla_architecture.md) but ships no code for it; its
  * closest entry point is the trajectory planner's Euler loop

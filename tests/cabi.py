@@ -42,6 +42,22 @@ class VlaDesc(C.Structure):
         "action_dim", "chunk", "steps")] + [("rope_theta", C.c_float), ("rms_eps", C.c_float), ("ln_eps", C.c_float)]
 
 
+class DecoderLayer(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "kv_heads", "dim", "vdim", "window", "distance_bias")] + \
+        [("scale", C.c_float), ("decay_rank", C.c_int32), ("ff", C.c_int32)]
+
+
+class DecoderDesc(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("struct_size", "num_layers", "vocab", "width", "side_dim")] + \
+        [("norm_eps", C.c_float)] + [(n, C.c_int32) for n in (
+            "compute_dtype", "max_step_tokens", "max_response_tokens", "cache_pages", "state_slots", "max_slots")]
+
+
+class StepEntry(C.Structure):
+    _fields_ = [("slot", C.c_int32), ("n_tokens", C.c_int32), ("kv_offset", C.c_int32), ("n_want", C.c_int32),
+                ("rng_step", C.c_uint32), ("reserved", C.c_uint32), ("tokens", C.POINTER(C.c_int32)), ("want", C.POINTER(C.c_int32))]
+
+
 class Sampling(C.Structure):
     _fields_ = [("temperature", C.c_float), ("top_p", C.c_float), ("top_k", C.c_int32),
                 ("reserved", C.c_uint32), ("seed", C.c_uint64)]
@@ -97,6 +113,13 @@ SIGNATURES = {
     "efm_b200_vit_finalize_weights": (I32, [P]),
     "efm_b200_vit_plan": (I32, [C.POINTER(VitDesc), C.POINTER(I32), I32] + [C.POINTER(I32)] * 7),
     "efm_b200_vit_encode": (I32, [P, P, I32, C.POINTER(I32), I32, P, I32]),
+    "efm_b200_decoder_create": (I32, [C.POINTER(DecoderDesc), C.POINTER(DecoderLayer), I32, C.POINTER(P)]),
+    "efm_b200_decoder_map_slot": (I32, [P, I32, C.POINTER(I32), I32, I32]),
+    "efm_b200_decoder_unmap_slot": (I32, [P, I32]),
+    "efm_b200_decoder_pin_prefix": (I32, [P, I32, I32]),
+    "efm_b200_decoder_step": (I32, [P, C.POINTER(StepEntry), I32, C.POINTER(C.c_float), C.POINTER(I32)]),
+    "efm_b200_decoder_set_taps": (I32, [P, I32]),
+    "efm_b200_decoder_read_taps": (I32, [P, C.POINTER(C.c_float)]),
     "efm_b200_vla_create": (I32, [C.POINTER(VlaDesc), I32, C.POINTER(P)]),
     "efm_b200_vla_destroy": (I32, [P]),
     "efm_b200_vla_last_error": (C.c_char_p, [P]),

@@ -8,17 +8,20 @@
 #include "decoder.h"
 
 #include <cstdlib>
+#include <type_traits>
 
 #include "../operators/decoder_rows.cuh"
 #include "../operators/delta_rule.cuh"
 #include "../operators/gemm_tc.cuh"
 #include "../operators/window_attention.cuh"
+#include "../operators/window_attention_tc.cuh"
 #define EFM_DECLARATIONS_ONLY
 #include "../operators/sample.cuh"
 #undef EFM_DECLARATIONS_ONLY
 #include "gemv_plan.h"
 #include "launcher.h"
 #include "shared_launch.h"
+#include "tensor_map.h"
 
 namespace efm {
 
@@ -233,9 +236,15 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
 }
 
 // ---- many rows ---------------------------------------------------------------------------------------------------
-int decoder_tc_tile_rows() { return 128; }
+int decoder_tc_tile_rows() { return wt::BM; }
 int decoder_simt_tile_rows() { return wa::QT; }
-bool decoder_layer_tc(const DecoderModel&, const DecoderLayer&) { return false; }
+// bf16 heads of at most 128 channels whose visible pages fit the kernel's page list
+bool decoder_layer_tc(const DecoderModel& m, const DecoderLayer& l) {
+    static const bool off = [] { const char* e = std::getenv("EFM_B200_ATTN_TC"); return e != nullptr && e[0] == '0'; }();
+    int pages = m.d.cache_pages;
+    if (l.d.window > 0) pages = std::min(pages, (l.d.window + wt::BM) / kPageTokens + 2);
+    return !off && !m.f32 && l.Dp <= 128 && l.Vp <= 128 && pages <= wt::kMaxTiles;
+}
 
 namespace {
 
@@ -265,7 +274,31 @@ void launch_delta_scan(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, cons
              m.state_pool, m.state_stride, l.state_off, s, plan);
 }
 
-// TA: activation type of the pass, TC: cache type (the same)
+template <int DP, int VP>
+void launch_attention_tc_v(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const WindowAttnShape& s, const RowPlan& plan, const RowTile* list, int n) {
+    DecoderModel& m = *c.decoder;
+    CUtensorMap mq, mk, mv;
+    const uint64_t rows = (uint64_t)m.d.cache_pages * kPageTokens;
+    const uint64_t qd[3] = {(uint64_t)DP, (uint64_t)s.H, (uint64_t)plan.rows}, qs[2] = {(uint64_t)DP * 2, (uint64_t)s.H * DP * 2};
+    const uint64_t kd[3] = {(uint64_t)DP, (uint64_t)s.G, rows}, ks[2] = {(uint64_t)DP * 2, (uint64_t)s.G * DP * 2};
+    const uint64_t vd[3] = {(uint64_t)VP, (uint64_t)s.G, rows}, vs[2] = {(uint64_t)VP * 2, (uint64_t)s.G * VP * 2};
+    const uint32_t qb[3] = {64, 1, (uint32_t)wt::BM}, kb[3] = {64, 1, (uint32_t)wt::BN};
+    if (!make_map_nd(&mq, m.q, 3, qd, qs, qb) || !make_map_nd(&mk, l.k_pool, 3, kd, ks, kb) || !make_map_nd(&mv, l.v_pool, 3, vd, vs, kb)) {
+        if (L.err == cudaSuccess) L.err = cudaErrorInvalidValue;
+        return;
+    }
+    L.launch(window_attention_tc_kernel<DP, VP>, dim3(n, s.H), dim3(wt::kThreads), wt::Cfg<DP, VP>::SMEM, mq, mk, mv, static_cast<__nv_bfloat16*>(m.mix), l.mix_wp,
+             s, plan, list, &c.state->error);
+}
+void launch_attention_tc(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const WindowAttnShape& s, const RowPlan& plan, const RowTile* list, int n) {
+    if (n <= 0) return;
+    if (l.Dp == 64 && l.Vp == 64) launch_attention_tc_v<64, 64>(c, L, l, s, plan, list, n);
+    else if (l.Dp == 64) launch_attention_tc_v<64, 128>(c, L, l, s, plan, list, n);
+    else if (l.Vp == 64) launch_attention_tc_v<128, 64>(c, L, l, s, plan, list, n);
+    else launch_attention_tc_v<128, 128>(c, L, l, s, plan, list, n);
+}
+
+// TA: activation and cache type of the pass
 template <typename TA>
 void attention_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const RowPlan& plan, const RowTiles& tiles) {
     DecoderModel& m = *c.decoder;
@@ -274,10 +307,25 @@ void attention_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const R
     TA* kp = static_cast<TA*>(l.k_pool);
     TA* vp = static_cast<TA*>(l.v_pool);
     L.launch(qk_scatter_rows_kernel<TA, TA, TA>, dim3(plan.rows), dim3(256), 0, static_cast<const TA*>(m.proj_a), l.in.Np, static_cast<TA*>(m.q), kp, vp, s, plan);
-    const RowTile* list = tiles.all;
-    const int n = tiles.listed ? tiles.n_all : (plan.rows + wa::QT - 1) / wa::QT;
-    L.launch(window_attention_rows_kernel<TA, TA, TA>, dim3(n, s.H), dim3(256), wa::rows_smem_bytes(s.Dp, s.Vp), static_cast<const TA*>(m.q), (const TA*)kp,
-             (const TA*)vp, static_cast<TA*>(m.mix), l.mix_wp, s, plan, list);
+    auto cuda_cores = [&](const RowTile* list, int n) {
+        if (n > 0)
+            L.launch(window_attention_rows_kernel<TA, TA, TA>, dim3(n, s.H), dim3(256), wa::rows_smem_bytes(s.Dp, s.Vp), static_cast<const TA*>(m.q),
+                     (const TA*)kp, (const TA*)vp, static_cast<TA*>(m.mix), l.mix_wp, s, plan, list);
+    };
+    if constexpr (std::is_same<TA, __nv_bfloat16>::value) {
+        if (decoder_layer_tc(m, l)) {
+            if (tiles.listed) {
+                launch_attention_tc(c, L, l, s, plan, tiles.tc, tiles.n_tc);
+                cuda_cores(tiles.simt, tiles.n_simt);
+                return;
+            }
+            if (plan.rows >= kTcMinRows) {
+                launch_attention_tc(c, L, l, s, plan, nullptr, (plan.rows + wt::BM - 1) / wt::BM);
+                return;
+            }
+        }
+    }
+    cuda_cores(tiles.all, tiles.listed ? tiles.n_all : (plan.rows + wa::QT - 1) / wa::QT);
 }
 
 template <typename TA>
@@ -409,6 +457,10 @@ cudaError_t configure_decoder(DecoderModel& m) {
     if (e == cudaSuccess) e = smem_attr(delta_scan_kernel<6>, ds::smem_bytes(192));
     if (e == cudaSuccess) e = smem_attr(delta_scan_kernel<7>, ds::smem_bytes(224));
     if (e == cudaSuccess) e = smem_attr(delta_scan_kernel<8>, ds::smem_bytes(256));
+    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<64, 64>, wt::Cfg<64, 64>::SMEM);
+    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<64, 128>, wt::Cfg<64, 128>::SMEM);
+    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<128, 64>, wt::Cfg<128, 64>::SMEM);
+    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<128, 128>, wt::Cfg<128, 128>::SMEM);
     m.attn_cluster = 16;
     if (e == cudaSuccess) e = m.f32 ? fit_cluster<float, 64>(m.attn_cluster) : fit_cluster<__nv_bfloat16, 64>(m.attn_cluster);
     if (e == cudaSuccess) e = m.f32 ? fit_cluster<float, 128>(m.attn_cluster) : fit_cluster<__nv_bfloat16, 128>(m.attn_cluster);

@@ -1,0 +1,231 @@
+// Many-row form of the windowed attention (window_attention.cuh) on the 5th-generation tensor cores: the structure of
+// attention_tc.cuh (S = Q K^T and O_tile = P V as tcgen05.mma with TMEM accumulators, operands by TMA, online softmax with
+// two threads per query row) over a paged cache, with the per-head multiplier and the distance bias applied to the scores
+// in fp32.  A key tile is exactly one 64-token page: its TMA coordinate is the page number of the sequence's table.
+// Block = 128 rows of one entry x one head, 256 threads.  Rows of the tile that belong to the next entry are computed and
+// not stored.  Every mbarrier wait is bounded and raises *error.
+#pragma once
+#include "attention_tc.cuh"
+#include "window_attention.cuh"
+
+namespace efm {
+
+namespace wt {
+
+constexpr int BM = 128, BN = kPageTokens, kThreads = 256, kMaxTiles = 1024;
+
+template <int DP, int VP>
+struct Cfg {
+    static constexpr int QB = DP / 64, VB = VP / 64;         // 64-channel boxes per row
+    static constexpr int Q_BYTES = BM * 128 * QB, K_BYTES = BN * 128 * QB, V_BYTES = BN * 128 * VB, P_BYTES = BM * 128;
+    static constexpr int O_COL = 64;
+    static constexpr int TMEM_COLS = VP == 64 ? 128 : 256;   // S (64 columns) + O tile, power of two
+    static constexpr int HALF = VP / 2;
+    static constexpr size_t SMEM = (size_t)Q_BYTES + 2 * K_BYTES + V_BYTES + P_BYTES + 2 * BM * 4 + 128 + kMaxTiles * 4 + 1024;
+};
+
+}  // namespace wt
+
+template <int DP, int VP>
+__global__ void __launch_bounds__(wt::kThreads) window_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
+                                                                           const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out,
+                                                                           int ld_out, const WindowAttnShape s, const RowPlan plan,
+                                                                           const RowTile* __restrict__ tiles, int* error) {
+    using namespace wt;
+    using at::instr_desc;
+    using at::tma_load_3d;
+    using at::umma_d;
+    using tc::mbar_expect_tx;
+    using tc::mbar_init;
+    using tc::mbar_wait;
+    using tc::smem_u32;
+    using tc::umma_commit;
+    using tc::umma_desc;
+    using C = Cfg<DP, VP>;
+    extern __shared__ unsigned char wt_smem[];
+    const uint32_t raw = smem_u32(wt_smem);
+    const uint32_t base = (raw + 1023u) & ~1023u;
+    unsigned char* base_ptr = wt_smem + (base - raw);
+    const uint32_t sQ = base, sK = sQ + C::Q_BYTES, sV = sK + 2 * C::K_BYTES, sP = sV + C::V_BYTES;
+    constexpr int XCH = C::Q_BYTES + 2 * C::K_BYTES + C::V_BYTES + C::P_BYTES;
+    float* xch = reinterpret_cast<float*>(base_ptr + XCH);                       // [2][BM]
+    const uint32_t bars = sP + C::P_BYTES + 2 * BM * 4;
+    const uint32_t qfull = bars, kfull0 = bars + 8, vfull = bars + 24, sbar = bars + 32, obar = bars + 40;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(base_ptr + XCH + 2 * BM * 4 + 48);
+    volatile int* abort_s = reinterpret_cast<volatile int*>(tmem_slot + 1);
+    int* pages = reinterpret_cast<int*>(base_ptr + XCH + 2 * BM * 4 + 128);
+
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int row = (warp & 3) * 32 + lane, hf = warp >> 2;       // TMEM lane = query row; which half of the columns
+    const int bx = (int)gridDim.x - 1 - (int)blockIdx.x, h = blockIdx.y, g = h / (s.H / s.G);     // late rows first: they see most keys
+    RowEntry e;
+    int r0;
+    if (tiles != nullptr) { const RowTile t = tiles[bx]; e = plan.entry(t.entry); r0 = t.row; }
+    else { e = plan.one; r0 = bx * BM; }
+    const int nq = min(BM, e.n - r0), p0 = e.pos0 + r0;           // rows of the tile, position of the first
+    const int i_pos = p0 + row;
+    const bool valid = row < nq;
+    const int lo = s.window > 0 ? max(0, i_pos - s.window + 1) : 0, hi = i_pos + 1;
+    const int first = s.window > 0 ? max(0, p0 - s.window + 1) : 0, lo_max = s.window > 0 ? max(0, p0 + nq - s.window) : 0, hi_min = p0 + 1;
+    const int pg0 = first / BN, ntiles = min((p0 + nq - 1) / BN - pg0 + 1, kMaxTiles), kb0 = pg0 * BN;
+
+    if (tid == 0) {
+        mbar_init(qfull, 1); mbar_init(kfull0, 1); mbar_init(kfull0 + 8, 1); mbar_init(vfull, 1); mbar_init(sbar, 1); mbar_init(obar, 1);
+        *abort_s = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == 0) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_slot)), "r"(C::TMEM_COLS) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    for (int i = tid; i < ntiles; i += kThreads) pages[i] = plan.page_table[(size_t)e.table * plan.max_pages + pg0 + i] * BN;
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    const uint32_t tmem = *tmem_slot;
+
+    constexpr uint32_t kDescS = instr_desc(BM, BN);
+    constexpr uint32_t kDescO = instr_desc(BM, VP) | (1u << 16);
+    const uint64_t vdesc = at::umma_desc_mn(sV, (uint32_t)(BN * 128), 1024u);
+    constexpr float kLog2e = 1.4426950408889634f;
+    const float f2 = s.scale * __bfloat162float(s.temp[h]) * kLog2e;
+    const float b2 = (s.bias ? distance_slope(h, s.H) : 0.f) * kLog2e;
+    float o[C::HALF];
+#pragma unroll
+    for (int i = 0; i < C::HALF; ++i) o[i] = 0.f;
+    float m = -INFINITY, l = 0.f;
+
+    auto load_k = [&](int tile, int buf) {
+        mbar_expect_tx(kfull0 + 8 * buf, C::K_BYTES);
+#pragma unroll
+        for (int b = 0; b < C::QB; ++b) tma_load_3d(sK + buf * C::K_BYTES + b * (BN * 128), &map_k, b * 64, g, pages[tile], kfull0 + 8 * buf);
+    };
+    auto load_v = [&](int tile) {
+        mbar_expect_tx(vfull, C::V_BYTES);
+#pragma unroll
+        for (int b = 0; b < C::VB; ++b) tma_load_3d(sV + b * (BN * 128), &map_v, b * 64, g, pages[tile], vfull);
+    };
+    auto issue_s = [&](int buf) {
+#pragma unroll
+        for (int k = 0; k < DP / 16; ++k) {
+            const uint64_t da = umma_desc(sQ + (k >> 2) * (BM * 128)) + (uint64_t)((k & 3) * 2);
+            const uint64_t db = umma_desc(sK + buf * C::K_BYTES + (k >> 2) * (BN * 128)) + (uint64_t)((k & 3) * 2);
+            umma_d(tmem, da, db, kDescS, k != 0 ? 1u : 0u);
+        }
+        umma_commit(sbar);
+    };
+    if (tid == 0) {
+        mbar_expect_tx(qfull, C::Q_BYTES);
+#pragma unroll
+        for (int b = 0; b < C::QB; ++b) tma_load_3d(sQ + b * (BM * 128), &map_q, b * 64, h, e.row0 + r0, qfull);
+        load_k(0, 0);
+        if (ntiles > 1) load_k(1, 1);
+        load_v(0);
+        const bool ok = mbar_wait(qfull, 0, abort_s) && mbar_wait(kfull0, 0, abort_s);
+        if (!ok) *abort_s = 1;
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        if (ok) issue_s(0);
+    }
+
+    for (int j = 0; j < ntiles; ++j) {
+        if (!mbar_wait(sbar, (uint32_t)j & 1u, abort_s)) *abort_s = 1;
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        if (tid == 0 && j + 2 < ntiles && *abort_s == 0) load_k(j + 2, j & 1);      // S_j has read K buffer j % 2
+        uint32_t sr[32];
+        tc::tmem_ld32(tmem + ((uint32_t)((warp & 3) * 32) << 16) + (uint32_t)(hf * 32), sr);
+        const int key0 = kb0 + j * BN + hf * 32;
+        float sc[32];                                            // scores in units of log2
+        float mx = -INFINITY;
+        const float bias0 = b2 * (float)(key0 - i_pos);
+        const bool interior = kb0 + j * BN >= lo_max && kb0 + (j + 1) * BN <= hi_min;
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+            const float v = fmaf(__uint_as_float(sr[i]), f2, fmaf(b2, (float)i, bias0));
+            sc[i] = interior || (key0 + i >= lo && key0 + i < hi) ? v : -INFINITY;
+            mx = fmaxf(mx, sc[i]);
+        }
+        xch[hf * BM + row] = mx;
+        if (__syncthreads_or(*abort_s != 0)) break;             // every thread takes the same decision
+        const float m_new = fmaxf(m, fmaxf(xch[row], xch[BM + row]));
+        const float mb = m_new == -INFINITY ? 0.f : m_new;
+        const float alpha = m == -INFINITY ? 0.f : at::ex2(m - mb);
+        m = m_new;
+        float rs = 0.f;
+        uint32_t pk[16];
+#pragma unroll
+        for (int i = 0; i < 32; i += 2) {
+            const float a = at::ex2(sc[i] - mb), b = at::ex2(sc[i + 1] - mb);      // exp2(-inf) = 0 for masked keys
+            rs += a + b;
+            pk[i >> 1] = pack_bf16(a, b);
+        }
+        l = l * alpha + rs;
+        {   // P row into the K-major, 128-byte-swizzled operand layout: chunk c of row r lives at chunk c ^ (r % 8)
+            const uint32_t prow = sP + (uint32_t)(row >> 3) * 1024u + (uint32_t)(row & 7) * 128u;
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                const uint32_t addr = prow + (uint32_t)(((hf * 4 + c) ^ (row & 7)) << 4);
+                asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(addr), "r"(pk[4 * c]), "r"(pk[4 * c + 1]), "r"(pk[4 * c + 2]),
+                             "r"(pk[4 * c + 3]) : "memory");
+            }
+        }
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+        asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+        __syncthreads();
+        if (tid == 0) {
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            bool ok = mbar_wait(vfull, (uint32_t)j & 1u, abort_s);
+            if (ok) {
+#pragma unroll
+                for (int k = 0; k < BN / 16; ++k)
+                    umma_d(tmem + C::O_COL, umma_desc(sP) + (uint64_t)(k * 2), vdesc + (uint64_t)(k * (2048 >> 4)), kDescO, k != 0 ? 1u : 0u);
+                umma_commit(obar);
+                if (j + 1 < ntiles) {
+                    ok = mbar_wait(kfull0 + 8 * ((j + 1) & 1), (uint32_t)((j + 1) >> 1) & 1u, abort_s);
+                    if (ok) issue_s((j + 1) & 1);
+                }
+            }
+            if (!ok) *abort_s = 1;
+        }
+        if (!mbar_wait(obar, (uint32_t)j & 1u, abort_s)) *abort_s = 1;
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        if (tid == 0 && j + 1 < ntiles && *abort_s == 0) load_v(j + 1);             // P V of tile j has read the V buffer
+        const uint32_t orow = tmem + ((uint32_t)((warp & 3) * 32) << 16) + (uint32_t)(C::O_COL + hf * C::HALF);
+#pragma unroll
+        for (int c0 = 0; c0 < C::HALF; c0 += 32) {
+            uint32_t r[32];
+            tc::tmem_ld32(orow + (uint32_t)c0, r);
+#pragma unroll
+            for (int i = 0; i < 32; ++i) o[c0 + i] = fmaf(o[c0 + i], alpha, __uint_as_float(r[i]));
+        }
+    }
+
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    xch[hf * BM + row] = l;
+    __syncthreads();
+    const float L = xch[row] + xch[BM + row];
+    const float inv = L > 0.f ? 1.0f / L : 0.f;
+    if (valid && *abort_s == 0) {
+        __nv_bfloat16* dst = out + (size_t)(e.row0 + r0 + row) * ld_out + (size_t)h * s.Dv;
+        const bool vec = (s.Dv & 7) == 0;                        // ld_out is a multiple of 8
+#pragma unroll
+        for (int i = 0; i < C::HALF; i += 8) {
+            const int d = hf * C::HALF + i;
+            if (vec && d + 8 <= s.Dv)
+                *reinterpret_cast<uint4*>(dst + d) = make_uint4(pack_bf16(o[i] * inv, o[i + 1] * inv), pack_bf16(o[i + 2] * inv, o[i + 3] * inv),
+                                                                pack_bf16(o[i + 4] * inv, o[i + 5] * inv), pack_bf16(o[i + 6] * inv, o[i + 7] * inv));
+            else {
+#pragma unroll
+                for (int c = 0; c < 8; ++c)
+                    if (d + c < s.Dv) dst[d + c] = __float2bfloat16_rn(o[i + c] * inv);
+            }
+        }
+    }
+    if (*abort_s != 0 && tid == 0 && error != nullptr) atomicExch(error, 1);
+    if (warp == 0) {
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(C::TMEM_COLS) : "memory");
+    }
+}
+
+}  // namespace efm

@@ -919,6 +919,120 @@ def summarise(line):
     return out
 
 
+# ---- layered decoder (Folizen) beside the text tower at equal size -----------------------------------------------------
+DESIGN_SIZES = {        # width, heads, kv heads (head dim 128), attention feed-forward, vocabulary
+    "1024": (1024, 8, 2, 4096, 32768),
+    "2048": (2048, 16, 4, 8192, 32768),
+    "4096": (4096, 32, 8, 16384, 32768),
+}
+DESIGN_LAYERS, DESIGN_WINDOW, DESIGN_PROMPT, DESIGN_DECODE, DESIGN_RANK = 8, 1024, 2048, 64, 64
+
+
+def design_config(size):
+    W, H, G, ff, V = DESIGN_SIZES[size]
+    att = {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": DESIGN_WINDOW}},
+           "mlp": {"kind": "dense", "ff": ff}}
+    delta = {"type": "general_delta", "mixer": {"heads": W // 64, "dim": 64}, "mlp": None}
+    return {"architecture": "Folizen", "width": W, "vocab": V, "norm": {"eps": 1e-5}, "token_side": {"dim": 64},
+            "layers": [att if i % 2 == 0 else delta for i in range(DESIGN_LAYERS)]}
+
+
+def design_flops(cfg, n):
+    """Matrix products plus visible attention pairs plus the recurrence (7 D^2 multiply-adds per token and head), 2 per multiply-add."""
+    W, side, out = cfg["width"], cfg["token_side"]["dim"], 0
+    for l in cfg["layers"]:
+        m = l["mixer"]
+        if l["type"] == "attention":
+            qd, kd = m["heads"] * m["dim"], m["kv_heads"] * (m["dim"] + m["vdim"])
+            w = m["mask"]["size"]
+            seen = sum(min(i + 1, w) for i in range(n))
+            out += 2 * n * W * (2 * qd + kd) + 4 * m["heads"] * m["dim"] * seen
+        else:
+            hd = m["heads"] * m["dim"]
+            out += 2 * n * (W * (6 * hd + DESIGN_RANK) + DESIGN_RANK * hd) + 14 * n * m["heads"] * m["dim"] ** 2
+        if l["mlp"]:
+            out += 4 * n * W * l["mlp"]["ff"]
+        out += 4 * n * W * side
+    return out
+
+
+def time_model(be, slot, prompt, steps, warmup):
+    """Median device times: prefill of the whole prompt (no sample), decode per token at that context (captured graph)."""
+    pre, dec = [], []
+    be.set_prefill_graph(True)
+    for it in range(warmup + steps):
+        be.event_record(0)
+        be.prefill(slot, prompt, sample=False)
+        be.event_record(1)
+        be.synchronize()
+        if it >= warmup:
+            pre.append(be.elapsed_ms(0, 1))
+    for it in range(warmup + steps):
+        be.prefill(slot, prompt, sample=True)
+        be.decode_begin(slot, len(prompt))
+        be.synchronize()
+        be.event_record(2)
+        be.decode_steps(DESIGN_DECODE, True)
+        be.event_record(3)
+        be.read_tokens(0, 1)
+        if it >= warmup:
+            dec.append(be.elapsed_ms(2, 3) / DESIGN_DECODE)
+    return sorted(pre)[len(pre) // 2], sorted(dec)[len(dec) // 2]
+
+
+def run_design(args):
+    """Prefill and decode throughput of the Folizen design at sizes that resemble real layers (random weights), and of the
+    text tower with the same width, heads, depth and number of weights."""
+    import torch
+    import cabi
+    import folizen_util as fu
+    from oracle import qwen_text, synth
+    hbm, _ = peaks()
+    tf, _ = tensor_peak()
+    clocks = ClockSampler(0)
+    out = {"metric": "Folizen prefill / decode throughput beside the text tower at equal size", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic",
+           "config": {"layers": DESIGN_LAYERS, "prompt": DESIGN_PROMPT, "decode_steps": DESIGN_DECODE, "window": DESIGN_WINDOW}, "sizes": {}}
+    clocks.start()
+    for size in args.design_sizes.split(","):
+        cfg = design_config(size)
+        pages = (DESIGN_PROMPT + DESIGN_DECODE + 64) // 64
+        g = torch.Generator(device="cuda").manual_seed(0)
+        be = cabi.Decoder(cfg, decay_rank=DESIGN_RANK, cache_pages=pages, state_slots=1, max_slots=1)
+        n_weights = 0
+        for name, shape in fu.shapes(cfg, DESIGN_RANK).items():
+            t = torch.randn(shape, generator=g, device="cuda") * (shape[-1] ** -0.5 if len(shape) == 2 else 0.1)
+            if "norm" in name or name.endswith("temp"):
+                t += 1.0
+            n_weights += t.numel() if len(shape) == 2 and "embed" not in name else 0
+            be.load_weights_partial({name: t.to(torch.bfloat16)})
+        be.finalize()
+        be.map_slot(0, list(range(pages)), 0)
+        be.set_sampling()
+        prompt = synth.make_token_ids(DESIGN_PROMPT, vocab=cfg["vocab"])
+        pre, dec = time_model(be, 0, prompt, args.steps, args.warmup)
+        nbytes = be.decode_step_bytes(DESIGN_PROMPT)
+        be.close()
+        W, H, G, _, V = DESIGN_SIZES[size]
+        rest = (n_weights - V * W) // DESIGN_LAYERS - W * (2 * H + 2 * G) * 128
+        q = qwen_text.QwenConfig(DESIGN_LAYERS, W, H, G, max(64, rest // (3 * W) // 64 * 64), V, tied=True)
+        qb = cabi.Backend(q, max_prefill_tokens=2048)
+        draw_weights_on_device(q, qb, False)
+        qb.alloc_slot(0, DESIGN_PROMPT + DESIGN_DECODE + 64)
+        qb.set_sampling()
+        qpre, qdec = time_model(qb, 0, prompt, args.steps, args.warmup)
+        qbytes = qb.decode_step_bytes(DESIGN_PROMPT)
+        qb.close()
+        fl, qfl = design_flops(cfg, DESIGN_PROMPT), prefill_flops(q, DESIGN_PROMPT, 0) - 2 * V * W
+
+        def report(p, d, f, b):
+            return {"prefill_ms": p, "prefill_tokens_per_s": DESIGN_PROMPT / p * 1e3, "prefill_frac_of_bf16_peak": f / p / 1e9 / tf,
+                    "decode_ms": d, "decode_tokens_per_s": 1e3 / d, "bytes_per_step": b, "decode_frac_of_hbm": b / d / 1e6 / hbm}
+        out["sizes"][size] = {"folizen": report(pre, dec, fl, nbytes), "text_tower": dict(report(qpre, qdec, qfl, qbytes), intermediate=q.intermediate)}
+    out["clocks"] = clocks.stop()
+    out["value"] = out["sizes"][args.design_sizes.split(",")[-1]]["folizen"]["decode_tokens_per_s"]
+    print(json.dumps(out), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -928,6 +1042,8 @@ def main():
     ap.add_argument("--config", type=int, default=None, choices=[0, 1, 2, 3, 4],
                     help="run one configuration alone; default: configuration 3 (tensor parallel over the ranks) plus, on one GPU, "
                          "a short pass over the other four")
+    ap.add_argument("--design", choices=["folizen"], default=None, help="layered decoder beside the text tower at equal size (one GPU)")
+    ap.add_argument("--design-sizes", default="1024,2048,4096", help="comma-separated widths for --design")
     ap.add_argument("--tokens", type=int, default=0, help="override the number of generated tokens")
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
     ap.add_argument("--no-e2e", action="store_true", help="skip the public-API end-to-end leg (profiling runs)")
@@ -947,6 +1063,9 @@ def main():
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))
+    if args.design is not None:
+        run_design(args)
+        return
     if args.impl == "reference":
         if args.config == 4:
             run_vla_reference(args, rank)

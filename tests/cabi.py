@@ -468,6 +468,34 @@ class VlaPolicy:
         return a.value, b.value
 
 
+class Decoder(Backend):
+    """A layered-decoder context described by a Folizen configuration dict; one mapped slot per call of map_slot."""
+
+    def __init__(self, config, *, decay_rank=64, cache_pages=64, state_slots=4, max_slots=4, max_step_tokens=2048,
+                 max_response_tokens=512, dtype=EFM_BF16, device_id=0):
+        self.L = lib()
+        layers = (DecoderLayer * len(config["layers"]))()
+        for e, l in zip(layers, config["layers"]):
+            m = l["mixer"]
+            e.heads, e.dim, e.ff = m["heads"], m["dim"], l["mlp"]["ff"] if l["mlp"] else 0
+            if l["type"] == "attention":
+                e.mixer, e.kv_heads, e.vdim, e.scale, e.distance_bias = 0, m["kv_heads"], m["vdim"], m["scale"], 1
+                e.window = m["mask"]["size"] if m.get("mask") else 0
+            else:
+                e.mixer, e.decay_rank = 1, decay_rank
+        d = DecoderDesc(C.sizeof(DecoderDesc), len(layers), config["vocab"], config["width"],
+                        (config.get("token_side") or {}).get("dim", 0), config["norm"]["eps"], dtype, max_step_tokens,
+                        max_response_tokens, cache_pages, state_slots, max_slots)
+        self.cfg = type("Cfg", (), {"vocab": config["vocab"], "mrope_section": None})()
+        self.ctx = P()
+        st = self.L.efm_b200_decoder_create(C.byref(d), layers, device_id, C.byref(self.ctx))
+        if st != EFM_OK:
+            raise BackendError(f"decoder_create failed ({st}): {self.L.efm_b200_last_error(None).decode()}")
+
+    def map_slot(self, slot, pages, state_slot):
+        self.check(self.L.efm_b200_decoder_map_slot(self.ctx, slot, _i32_array(pages), len(pages), state_slot), "decoder_map_slot")
+
+
 def generate(be: Backend, slot, prompt, max_new_tokens, *, prefix_len=0, embeds=None, embed_token_id=-1, pos3=None,
              mrope_last_pos=None, use_graph=True, forced=None, collect_logits=False):
     """generate() through the C ABI: prefill of prompt[prefix_len:], then decode steps.

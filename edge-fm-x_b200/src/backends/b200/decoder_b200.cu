@@ -99,7 +99,7 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
     EFM_TRY(configure_sampler());
 
     const size_t rows = (size_t)std::max(desc->cache_pages, 1) * EFM_PAGE_TOKENS, es = act_bytes(*m);
-    size_t w_in = 8, w_mix = 8, w_ff = 8, w_q = 8, w_delta_in = 8, w_pack = 8, w_rank = 8, k_max = Wp;
+    size_t w_in = 8, w_mix = 8, w_ff = 8, w_q = 8, w_delta_in = 8, n_pack = 8, w_rank = 8, k_max = Wp;
     bool any_delta = false;
     m->layers.resize(desc->num_layers);
     for (int i = 0; i < desc->num_layers; ++i) {
@@ -134,7 +134,7 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
             l.state_off = m->state_stride;
             m->state_stride += (size_t)HD * d.dim;
             w_delta_in = std::max(w_delta_in, (size_t)l.in.Np);
-            w_pack = std::max(w_pack, (size_t)d.heads * 6 * round_up(d.dim, 32));
+            n_pack = std::max(n_pack, decoder_delta_pack_floats(d.heads, d.dim, S, std::min(desc->max_slots, S)));
             w_rank = std::max(w_rank, (size_t)l.w2.Kp);
         }
         l.mix_wp = round_up(l.mix_w, 8);
@@ -193,7 +193,7 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
     EFM_TRY(dev_alloc(c, &m->y, (size_t)S * Wp));
     if (any_delta) {
         EFM_TRY(dev_alloc(c, &m->proj_f, S * w_delta_in));
-        EFM_TRY(dev_alloc(c, &m->pack, S * w_pack));
+        EFM_TRY(dev_alloc(c, &m->pack, n_pack));
         EFM_TRY(dev_alloc(c, &m->tanh_w, S * w_rank));
         EFM_TRY(dev_alloc(c, &m->decay, S * w_mix));
         EFM_TRY(dev_alloc(c, &m->o, S * w_mix));

@@ -11,6 +11,7 @@
 #include <type_traits>
 
 #include "../operators/decoder_rows.cuh"
+#include "../operators/delta_chunk.cuh"
 #include "../operators/delta_rule.cuh"
 #include "../operators/gemm_tc.cuh"
 #include "../operators/window_attention.cuh"
@@ -298,6 +299,18 @@ void launch_attention_tc(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, co
     else launch_attention_tc_v<128, 128>(c, L, l, s, plan, list, n);
 }
 
+// Chunked recurrence: every chunk's state-independent part at once, then the chunks in sequence.
+template <int DP>
+void launch_delta_chunks(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const RowPlan& plan) {
+    DecoderModel& m = *c.decoder;
+    const DeltaShape s = delta_shape(m, l);
+    const int chunks = plan.n_entries == 1 ? (plan.rows + dc::C - 1) / dc::C : plan.rows / dc::C + plan.n_entries;     // at most
+    L.launch(delta_prepare_kernel<DP>, dim3(chunks, l.d.heads), dim3(dc::kThreads), sizeof(dc::PrepSmem<DP>), (const float*)m.proj_f, (const float*)m.decay,
+             l.w2.Np, m.pack, s, plan);
+    L.launch(delta_chunk_scan_kernel<DP>, dim3(l.d.heads * (DP / dc::kCols), plan.n_entries), dim3(dc::kThreads), sizeof(dc::ScanSmem<DP>), (const float*)m.pack,
+             m.o, l.mix_wp, m.state_pool, m.state_stride, l.state_off, s, plan);
+}
+
 // TA: activation and cache type of the pass
 template <typename TA>
 void attention_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const RowPlan& plan, const RowTiles& tiles) {
@@ -336,18 +349,31 @@ void delta_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const RowPl
     L.launch(delta_tanh_rows_kernel, dim3(plan.rows), dim3(128), 0, (const float*)m.proj_f, m.tanh_w, l.w2.Kp, s);
     L.launch(gemm_f32_kernel, dim3((l.w2.Np + 63) / 64, (plan.rows + 63) / 64), dim3(256), 0, (const float*)m.tanh_w, l.w2.Kp, (const __nv_bfloat16*)l.w2.w,
              l.w2.Kp, m.decay, l.w2.Np, plan.rows, l.w2.Np, l.w2.Kp);
-    L.launch(delta_inputs_rows_kernel, dim3(plan.rows), dim3(256), 0, (const float*)m.proj_f, (const float*)m.decay, l.w2.Np, m.pack, s);
-    switch (s.Dp / 32) {
-        case 1: launch_delta_scan<1>(c, L, l, plan); break;
-        case 2: launch_delta_scan<2>(c, L, l, plan); break;
-        case 3: launch_delta_scan<3>(c, L, l, plan); break;
-        case 4: launch_delta_scan<4>(c, L, l, plan); break;
-        case 5: launch_delta_scan<5>(c, L, l, plan); break;
-        case 6: launch_delta_scan<6>(c, L, l, plan); break;
-        case 7: launch_delta_scan<7>(c, L, l, plan); break;
-        default: launch_delta_scan<8>(c, L, l, plan); break;
+    const bool chunked = plan.rows >= dc::C && s.Dp <= 128;         // short passes and larger heads: token by token
+    if (chunked) {
+        switch (s.Dp / 32) {
+            case 1: launch_delta_chunks<32>(c, L, l, plan); break;
+            case 2: launch_delta_chunks<64>(c, L, l, plan); break;
+            case 3: launch_delta_chunks<96>(c, L, l, plan); break;
+            default: launch_delta_chunks<128>(c, L, l, plan); break;
+        }
+    } else {
+        L.launch(delta_inputs_rows_kernel, dim3(plan.rows), dim3(256), 0, (const float*)m.proj_f, (const float*)m.decay, l.w2.Np, m.pack, s);
+        switch (s.Dp / 32) {
+            case 1: launch_delta_scan<1>(c, L, l, plan); break;
+            case 2: launch_delta_scan<2>(c, L, l, plan); break;
+            case 3: launch_delta_scan<3>(c, L, l, plan); break;
+            case 4: launch_delta_scan<4>(c, L, l, plan); break;
+            case 5: launch_delta_scan<5>(c, L, l, plan); break;
+            case 6: launch_delta_scan<6>(c, L, l, plan); break;
+            case 7: launch_delta_scan<7>(c, L, l, plan); break;
+            default: launch_delta_scan<8>(c, L, l, plan); break;
+        }
     }
-    L.launch(delta_output_rows_kernel<TA>, dim3(plan.rows), dim3(256), 0, (const float*)m.o, l.mix_wp, (const float*)m.proj_f, static_cast<TA*>(m.mix), l.mix_wp, s);
+    int lanes = 1;
+    while (lanes * 4 < s.D && lanes < 32) lanes *= 2;
+    L.launch(delta_output_rows_kernel<TA>, dim3(plan.rows), dim3(256), 0, (const float*)m.o, l.mix_wp, (const float*)m.proj_f, static_cast<TA*>(m.mix), l.mix_wp,
+             s, lanes);
 }
 
 template <typename TA>
@@ -442,6 +468,14 @@ cudaError_t fit_cluster(int& width) {
 }
 }  // namespace
 
+// token-by-token form: 6 vectors a row; chunked form: one packed block a chunk, the last chunk of every entry short
+size_t decoder_delta_pack_floats(int heads, int dim, int rows, int entries) {
+    const int Dp = round_up(dim, 32);
+    size_t n = (size_t)rows * heads * kDeltaParts * Dp;
+    if (Dp <= 128) n = std::max(n, (size_t)(rows / dc::C + 1 + entries) * heads * dc::pack_floats(Dp));
+    return n;
+}
+
 cudaError_t configure_decoder(DecoderModel& m) {
     int dev = 0, optin = 0;
     cudaError_t e = cudaGetDevice(&dev);
@@ -461,6 +495,11 @@ cudaError_t configure_decoder(DecoderModel& m) {
     if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<64, 128>, wt::Cfg<64, 128>::SMEM);
     if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<128, 64>, wt::Cfg<128, 64>::SMEM);
     if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<128, 128>, wt::Cfg<128, 128>::SMEM);
+    if (e == cudaSuccess) e = smem_attr(delta_prepare_kernel<96>, sizeof(dc::PrepSmem<96>));
+    if (e == cudaSuccess) e = smem_attr(delta_prepare_kernel<128>, sizeof(dc::PrepSmem<128>));
+    if (e == cudaSuccess) e = smem_attr(delta_chunk_scan_kernel<64>, sizeof(dc::ScanSmem<64>));
+    if (e == cudaSuccess) e = smem_attr(delta_chunk_scan_kernel<96>, sizeof(dc::ScanSmem<96>));
+    if (e == cudaSuccess) e = smem_attr(delta_chunk_scan_kernel<128>, sizeof(dc::ScanSmem<128>));
     m.attn_cluster = 16;
     if (e == cudaSuccess) e = m.f32 ? fit_cluster<float, 64>(m.attn_cluster) : fit_cluster<__nv_bfloat16, 64>(m.attn_cluster);
     if (e == cudaSuccess) e = m.f32 ? fit_cluster<float, 128>(m.attn_cluster) : fit_cluster<__nv_bfloat16, 128>(m.attn_cluster);

@@ -81,6 +81,8 @@ constexpr int kTcMinRows = 16;
 int decoder_tc_tile_rows();
 int decoder_simt_tile_rows();
 bool decoder_layer_tc(const DecoderModel& m, const DecoderLayer& l);
+// scratch of one recurrent layer for `rows` rows of at most `entries` sequences
+size_t decoder_delta_pack_floats(int heads, int dim, int rows, int entries);
 cudaError_t configure_decoder(DecoderModel& m);
 
 }  // namespace efm

@@ -27,6 +27,8 @@ struct DeltaShape {
     const __nv_bfloat16* norm;        // [heads * D]
 };
 
+__device__ __forceinline__ void store_vec4(float* p, const float (&r)[4]) { *reinterpret_cast<float4*>(p) = make_float4(r[0], r[1], r[2], r[3]); }
+__device__ __forceinline__ void store_vec4(__nv_bfloat16* p, const float (&r)[4]) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(r[0], r[1]), pack_bf16(r[2], r[3])); }
 constexpr float kDecayRate = 0.6065306597126334f;      // e^{-1/2}
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
 
@@ -168,19 +170,43 @@ __global__ void __launch_bounds__(ds::kThreads) delta_scan_kernel(const float* _
         }
 }
 
-// out[row] = rms(o per head) * norm * sigmoid(g), row length ld_out (pads untouched)
+// out[row] = rms(o per head) * norm * sigmoid(g), row length ld_out (pads untouched).  One block per row; `lanes` (a power
+// of two, at least D / 4 where possible) threads share a head, four channels at a time.
 template <typename TO>
 __global__ void __launch_bounds__(256) delta_output_rows_kernel(const float* __restrict__ o, int ld_o, const float* __restrict__ proj, TO* __restrict__ out,
-                                                                int ld_out, const DeltaShape s) {
-    const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, HD = s.heads * s.D;
-    for (int h = warp; h < s.heads; h += 8) {
-        const float* x = o + (size_t)row * ld_o + h * s.D;
+                                                                int ld_out, const DeltaShape s, int lanes) {
+    const int row = blockIdx.x, HD = s.heads * s.D, l = threadIdx.x & (lanes - 1), per = 256 / lanes;
+    const float* orow = o + (size_t)row * ld_o;
+    const float* grow = proj + (size_t)row * s.ld + 3 * HD;
+    TO* dst = out + (size_t)row * ld_out;
+    const bool vec = (s.D & 3) == 0;
+    for (int h0 = 0; h0 < s.heads; h0 += per) {                    // every thread takes part in the shuffles
+        const int h = h0 + threadIdx.x / lanes, c0 = h * s.D;
+        const bool in = h < s.heads;
         float ss = 0.f;
-        for (int d = lane; d < s.D; d += 32) ss = fmaf(x[d], x[d], ss);
-        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)s.D + s.eps);
-        for (int d = lane; d < s.D; d += 32) {
-            const int c = h * s.D + d;
-            store_f32(out + (size_t)row * ld_out + c, x[d] * inv * __bfloat162float(s.norm[c]) * sigmoid_f(proj[(size_t)row * s.ld + 3 * HD + c]));
+        if (in)
+            for (int d = 4 * l; d < s.D; d += 4 * lanes) {
+                if (vec) {
+                    const float4 v = *reinterpret_cast<const float4*>(orow + c0 + d);
+                    ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
+                } else {
+                    for (int j = d; j < min(d + 4, s.D); ++j) ss = fmaf(orow[c0 + j], orow[c0 + j], ss);
+                }
+            }
+        for (int x = lanes / 2; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+        if (!in) continue;
+        const float inv = 1.0f / sqrtf(ss / (float)s.D + s.eps);
+        for (int d = 4 * l; d < s.D; d += 4 * lanes) {
+            if (vec) {
+                const float4 v = *reinterpret_cast<const float4*>(orow + c0 + d), g = *reinterpret_cast<const float4*>(grow + c0 + d);
+                const uint2 w = *reinterpret_cast<const uint2*>(s.norm + c0 + d);
+                const float r[4] = {v.x * inv * bf16lo(w.x) * sigmoid_f(g.x), v.y * inv * bf16hi(w.x) * sigmoid_f(g.y),
+                                    v.z * inv * bf16lo(w.y) * sigmoid_f(g.z), v.w * inv * bf16hi(w.y) * sigmoid_f(g.w)};
+                store_vec4(dst + c0 + d, r);
+            } else {
+                for (int j = d; j < min(d + 4, s.D); ++j)
+                    store_f32(dst + c0 + j, orow[c0 + j] * inv * __bfloat162float(s.norm[c0 + j]) * sigmoid_f(grow[c0 + j]));
+            }
         }
     }
 }

@@ -307,7 +307,7 @@ void launch_delta_chunks(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, co
     const int chunks = plan.n_entries == 1 ? (plan.rows + dc::C - 1) / dc::C : plan.rows / dc::C + plan.n_entries;     // at most
     L.launch(delta_prepare_kernel<DP>, dim3(chunks, l.d.heads), dim3(dc::kThreads), sizeof(dc::PrepSmem<DP>), (const float*)m.proj_f, (const float*)m.decay,
              l.w2.Np, m.pack, s, plan);
-    L.launch(delta_chunk_scan_kernel<DP>, dim3(l.d.heads * (DP / dc::kCols), plan.n_entries), dim3(dc::kThreads), sizeof(dc::ScanSmem<DP>), (const float*)m.pack,
+    L.launch(delta_chunk_scan_kernel<DP>, dim3(l.d.heads * (DP / dc::kCols), plan.n_entries), dim3(dc::kScanThreads), sizeof(dc::ScanSmem<DP>), (const float*)m.pack,
              m.o, l.mix_wp, m.state_pool, m.state_stride, l.state_off, s, plan);
 }
 

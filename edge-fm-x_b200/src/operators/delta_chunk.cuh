@@ -9,14 +9,14 @@
 //   Y = X' S + V1,   O = Q' S + O1,   S <- P_16 (S + C^T V - B^T Y).
 // Decays are at least e^{-0.61}, so P_16^{-1} stays below 2e4 and every factor of the dot products is of moderate size.
 // A chunk that is cut short is filled with tokens that change nothing (w = 1, the rest 0).
-// Packed chunk (floats, D padded to DP): XQ [DP][32] = X'^T | Q'^T, CB [32][DP] = C | -B, V, V1, O1 [16][DP], P [DP].
+// Packed chunk (floats, D padded to DP): XQ [32][DP] = X' | Q', CB [32][DP] = C | -B, V, V1, O1 [16][DP], P [DP].
 #pragma once
 #include "delta_rule.cuh"
 
 namespace efm {
 
 namespace dc {
-constexpr int C = 16, kThreads = 128, kCols = 16;
+constexpr int C = 16, kThreads = 128, kScanThreads = 256, kCols = 16;
 __host__ __device__ constexpr int pack_floats(int DP) { return 113 * DP; }
 
 // Chunk `idx` of the pass -> entry, first token; false past the last chunk.  first: index of the entry's first chunk.
@@ -37,15 +37,15 @@ struct PrepSmem {
     float bc[32][DP + 4];             // B rows, then C rows
     float w[C][DP];
     float v[C][DP];
-    float g[32][36];                  // masked products: rows x / q, columns b | c
+    float g[32][36];                  // masked products, transposed: [b | c of token s][x | q of token t]
 };
 template <int DP>
 struct ScanSmem {
-    float xq[2][DP][40];
+    float xq[2][32][DP + 4];
     float cb[2][32][DP];
     float vin[2][3][C][kCols];        // V | V1 | O1
     float p[2][DP];
-    float s[DP][kCols];
+    float st[kCols][DP + 4];          // the state, transposed
     float y[C][kCols];
 };
 }  // namespace dc
@@ -63,51 +63,74 @@ __global__ void __launch_bounds__(dc::kThreads) delta_prepare_kernel(const float
     if (!locate(plan, blockIdx.x, e, t0)) return;
     const int nv = min(C, e.n - t0);
     // ---- step inputs: a warp per token ----------------------------------------------------------------------------
-    for (int t = warp; t < C; t += 4) {
+    constexpr int NT = C / 4, NI = DP / 32;
+    float k[NT][NI], r[NT][NI], v[NT][NI], a[NT][NI], dec[NT][NI];
+#pragma unroll
+    for (int q = 0; q < NT; ++q) {
+        const int t = warp + 4 * q;
         const size_t row = (size_t)(e.row0 + t0 + t);
         const float* x = proj + row * s.ld + c0;
-        const float* dec = decay_in + row * ld_decay + c0;
-        float k[DP / 32], ss = 0.f;
 #pragma unroll
-        for (int i = 0; i < DP / 32; ++i) {
-            const int d = lane + 32 * i;
-            k[i] = t < nv && d < s.D ? x[HD + d] : 0.f;
-            ss = fmaf(k[i], k[i], ss);
-        }
-        const float inv = 1.0f / sqrtf(warp_sum(ss) + 1e-6f);
-#pragma unroll
-        for (int i = 0; i < DP / 32; ++i) {
+        for (int i = 0; i < NI; ++i) {
             const int d = lane + 32 * i;
             const bool in = t < nv && d < s.D;
-            const float u = k[i] * inv;
+            r[q][i] = in ? x[d] : 0.f;
+            k[q][i] = in ? x[HD + d] : 0.f;
+            v[q][i] = in ? x[2 * HD + d] : 0.f;
+            a[q][i] = in ? x[4 * HD + d] : 0.f;
+            dec[q][i] = in ? decay_in[row * ld_decay + c0 + d] : 0.f;
+        }
+    }
+#pragma unroll
+    for (int q = 0; q < NT; ++q) {
+        const int t = warp + 4 * q;
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) ss = fmaf(k[q][i], k[q][i], ss);
+        const float inv = 1.0f / sqrtf(warp_sum(ss) + 1e-6f);
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const int d = lane + 32 * i;
+            const bool in = t < nv && d < s.D;
+            const float u = k[q][i] * inv;
             sm.xq[t][d] = u;
-            sm.xq[C + t][d] = in ? x[d] : 0.f;
-            sm.bc[t][d] = in ? sigmoid_f(x[4 * HD + d] + __bfloat162float(s.a_bias[c0 + d])) * u : 0.f;
-            sm.bc[C + t][d] = k[i];
-            sm.w[t][d] = in ? expf(-kDecayRate * sigmoid_f(dec[d] + __bfloat162float(s.w0[c0 + d]))) : 1.f;
-            sm.v[t][d] = in ? x[2 * HD + d] : 0.f;
+            sm.xq[C + t][d] = r[q][i];
+            sm.bc[t][d] = in ? sigmoid_f(a[q][i] + __bfloat162float(s.a_bias[c0 + d])) * u : 0.f;
+            sm.bc[C + t][d] = k[q][i];
+            sm.w[t][d] = in ? expf(-kDecayRate * sigmoid_f(dec[q][i] + __bfloat162float(s.w0[c0 + d]))) : 1.f;
+            sm.v[t][d] = v[q][i];
         }
     }
     __syncthreads();
     float* out = pack + ((size_t)blockIdx.x * s.heads + h) * pack_floats(DP);
     float* o_cb = out + 32 * DP;
     float* o_v = out + 64 * DP;
-    // ---- decay products, a thread per channel ----------------------------------------------------------------------
-    if (tid < DP) {
-        float P = 1.f;
+    // ---- decay products: two threads per channel, half of the tokens each -------------------------------------------
+    for (int r = tid; r < 2 * DP; r += kThreads) {
+        const int ch = r % DP, half = (r / DP) * (C / 2);
+        float w[C], P = 1.f;
+#pragma unroll
+        for (int t = 0; t < C; ++t) w[t] = sm.w[t][ch];
+        float before[C / 2], after[C / 2];
 #pragma unroll
         for (int t = 0; t < C; ++t) {
-            sm.xq[t][tid] *= P;
-            P *= sm.w[t][tid];
-            const float inv = 1.0f / P;
-            sm.xq[C + t][tid] *= P;
-            const float b = sm.bc[t][tid] * inv, c = sm.bc[C + t][tid] * inv;
-            sm.bc[t][tid] = b;
-            sm.bc[C + t][tid] = c;
-            o_cb[t * DP + tid] = c;
-            o_cb[(C + t) * DP + tid] = -b;
+            const float prev = P;
+            P *= w[t];
+            if (t < C / 2 ? half == 0 : half != 0) { before[t % (C / 2)] = prev; after[t % (C / 2)] = P; }
         }
-        out[112 * DP + tid] = P;
+#pragma unroll
+        for (int q = 0; q < C / 2; ++q) {
+            const int t = half + q;
+            const float inv = 1.0f / after[q];
+            sm.xq[t][ch] *= before[q];
+            sm.xq[C + t][ch] *= after[q];
+            const float b = sm.bc[t][ch] * inv, c = sm.bc[C + t][ch] * inv;
+            sm.bc[t][ch] = b;
+            sm.bc[C + t][ch] = c;
+            o_cb[t * DP + ch] = c;
+            o_cb[(C + t) * DP + ch] = -b;
+        }
+        if (half != 0) out[112 * DP + ch] = P;
     }
     __syncthreads();
     // ---- 32 x 32 products, 2 x 4 per thread ------------------------------------------------------------------------
@@ -138,65 +161,57 @@ __global__ void __launch_bounds__(dc::kThreads) delta_prepare_kernel(const float
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const int col = j * 8 + ct, src = col & 15;
-                sm.g[i * 16 + rt][col] = (i == 0 ? src < rt : src <= rt) ? acc[i][j] : 0.f;
+sm.g[col][i * 16 + rt] = (i == 0 ? src < rt : src <= rt) ? acc[i][j] : 0.f;
             }
     }
     __syncthreads();
-    // ---- triangular solves: a thread per channel of X' / Q' or of V1 / O1 ------------------------------------------
+    // ---- triangular solves, a thread per channel of X' / Q' or of V1 / O1: once token q is solved, its share leaves every
+    // later row (independent multiply-adds, coefficients of one q are consecutive)
     for (int role = tid; role < 2 * DP; role += kThreads) {
-        if (role < DP) {
-            float x[C], y[C];
+        const bool is_x = role < DP;
+        const int ch = is_x ? role : role - DP;
+        float x[C], y[C];
+        auto subtract = [&](int q, float v, int col, float sign) {
 #pragma unroll
-            for (int t = 0; t < C; ++t) {
-                float a = sm.xq[t][role];
+            for (int t4 = 0; t4 < C; t4 += 4) {
+                const float4 gx = *reinterpret_cast<const float4*>(&sm.g[col][t4]), gq = *reinterpret_cast<const float4*>(&sm.g[col][C + t4]);
+                const float ax[4] = {gx.x, gx.y, gx.z, gx.w}, aq[4] = {gq.x, gq.y, gq.z, gq.w};
 #pragma unroll
-                for (int q = 0; q < t; ++q) a = fmaf(-sm.g[t][q], x[q], a);
-                x[t] = a;
+                for (int t = 0; t < 4; ++t) {
+                    if (t4 + t > q) x[t4 + t] = fmaf(sign * ax[t], v, x[t4 + t]);
+                    if (t4 + t >= q) y[t4 + t] = fmaf(sign * aq[t], v, y[t4 + t]);
+                }
             }
-            float4* dst = reinterpret_cast<float4*>(out + role * 32);
+        };
+        float* o_x = is_x ? out + ch : o_v + C * DP + ch;              // X' and Q' rows, or V1 and O1 rows
+        if (is_x) {
 #pragma unroll
-            for (int t = 0; t < C; t += 4) dst[t / 4] = make_float4(x[t], x[t + 1], x[t + 2], x[t + 3]);
-#pragma unroll
-            for (int t = 0; t < C; ++t) {
-                float a = sm.xq[C + t][role];
-#pragma unroll
-                for (int q = 0; q <= t; ++q) a = fmaf(-sm.g[C + t][q], x[q], a);
-                y[t] = a;
-            }
-#pragma unroll
-            for (int t = 0; t < C; t += 4) dst[4 + t / 4] = make_float4(y[t], y[t + 1], y[t + 2], y[t + 3]);
+            for (int t = 0; t < C; ++t) { x[t] = sm.xq[t][ch]; y[t] = sm.xq[C + t][ch]; }
         } else {
-            const int ch = role - DP;
-            float v[C], v1[C];
 #pragma unroll
-            for (int t = 0; t < C; ++t) { v[t] = sm.v[t][ch]; o_v[t * DP + ch] = v[t]; }
+            for (int t = 0; t < C; ++t) { x[t] = 0.f; y[t] = 0.f; }
 #pragma unroll
             for (int t = 0; t < C; ++t) {
-                float a = 0.f;
-#pragma unroll
-                for (int q = 0; q < t; ++q) a = fmaf(sm.g[t][C + q], v[q], fmaf(-sm.g[t][q], v1[q], a));
-                v1[t] = a;
-                o_v[(C + t) * DP + ch] = a;
-            }
-#pragma unroll
-            for (int t = 0; t < C; ++t) {
-                float a = 0.f;
-#pragma unroll
-                for (int q = 0; q <= t; ++q) a = fmaf(sm.g[C + t][C + q], v[q], fmaf(-sm.g[C + t][q], v1[q], a));
-                o_v[(2 * C + t) * DP + ch] = a;
+                const float v = sm.v[t][ch];
+                o_v[t * DP + ch] = v;
+                subtract(t, v, C + t, 1.f);
             }
         }
+#pragma unroll
+        for (int t = 0; t < C; ++t) subtract(t, x[t], t, -1.f);
+#pragma unroll
+        for (int t = 0; t < C; ++t) { o_x[t * DP] = x[t]; o_x[(C + t) * DP] = y[t]; }
     }
 }
 
 // grid (heads * ceil(DP / 16), entries): the sequential part for 16 value channels of one head.
 template <int DP>
-__global__ void __launch_bounds__(dc::kThreads) delta_chunk_scan_kernel(const float* __restrict__ pack, float* __restrict__ o, int ld_o,
+__global__ void __launch_bounds__(dc::kScanThreads) delta_chunk_scan_kernel(const float* __restrict__ pack, float* __restrict__ o, int ld_o,
                                                                         float* __restrict__ pool, size_t slot_stride, size_t offset, const DeltaShape s,
                                                                         const RowPlan plan) {
     using namespace dc;
     using ds::cp16;
-    constexpr int CT = DP == 32 ? 1 : (DP == 64 ? 2 : 4);          // state columns per thread (4 rows each)
+    constexpr int CT = DP <= 64 ? 1 : 2;                           // state columns per thread (4 rows each)
     constexpr int RT = DP / 4;                                     // row tiles of the state
     constexpr int GROUPS = DP / kCols;
     extern __shared__ __align__(16) unsigned char dc_smem[];
@@ -210,9 +225,9 @@ __global__ void __launch_bounds__(dc::kThreads) delta_chunk_scan_kernel(const fl
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     auto stage = [&](int c, int b) {
         const float* src = pack + ((size_t)(chunk0 + c) * s.heads + h) * pack_floats(DP);
-        for (int i = tid; i < DP * 8; i += kThreads) cp16(&sm.xq[b][i >> 3][(i & 7) * 4], src + i * 4);
-        for (int i = tid; i < DP * 8; i += kThreads) cp16(&sm.cb[b][0][0] + i * 4, src + 32 * DP + i * 4);
-        for (int i = tid; i < 3 * C * 4; i += kThreads) cp16(&sm.vin[b][0][i >> 2][(i & 3) * 4], src + 64 * DP + (i >> 2) * DP + c0 + (i & 3) * 4);
+        for (int i = tid; i < DP * 8; i += kScanThreads) cp16(&sm.xq[b][i / RT][(i % RT) * 4], src + i * 4);
+        for (int i = tid; i < DP * 8; i += kScanThreads) cp16(&sm.cb[b][0][0] + i * 4, src + 32 * DP + i * 4);
+        for (int i = tid; i < 3 * C * 4; i += kScanThreads) cp16(&sm.vin[b][0][i >> 2][(i & 3) * 4], src + 64 * DP + (i >> 2) * DP + c0 + (i & 3) * 4);
         if (tid < DP / 4) cp16(&sm.p[b][tid * 4], src + 112 * DP + tid * 4);
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -229,11 +244,11 @@ __global__ void __launch_bounds__(dc::kThreads) delta_chunk_scan_kernel(const fl
             for (int j = 0; j < CT; ++j) {
                 const int r = 4 * it + i;
                 S[i][j] = e.pos0 > 0 && r < s.D && c0 + CT * jt + j < s.D ? st[(size_t)r * s.D + j] : 0.f;
-                sm.s[r][CT * jt + j] = S[i][j];
+                sm.st[CT * jt + j][r] = S[i][j];
             }
     }
-    // first product: 4 x 4 outputs per thread, k split over the four lanes of a quad
-    const int ks = lane & 3, ct = (lane >> 2) & 3, rt = (lane >> 4) | (warp << 1);
+    // first product: 4 x 4 outputs per thread, k split over eight lanes
+    const int ks = lane & 7, ct = lane >> 3, rt = warp;
     for (int c = 0; c < n_chunks; ++c) {
         const int b = c & 1;
         asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -244,18 +259,24 @@ __global__ void __launch_bounds__(dc::kThreads) delta_chunk_scan_kernel(const fl
         for (int i = 0; i < 4; ++i)
 #pragma unroll
             for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
-#pragma unroll 8
-        for (int k = 0; k < DP / 4; ++k) {
-            const float4 a = *reinterpret_cast<const float4*>(&sm.xq[b][4 * k + ks][rt * 4]);
-            const float4 y = *reinterpret_cast<const float4*>(&sm.s[4 * k + ks][ct * 4]);
-            const float av[4] = {a.x, a.y, a.z, a.w}, yv[4] = {y.x, y.y, y.z, y.w};
+#pragma unroll
+        for (int k4 = 0; k4 < DP / 32; ++k4) {
+            const int k = (k4 * 8 + ks) * 4;
+            float4 a[4], y[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) a[i] = *reinterpret_cast<const float4*>(&sm.xq[b][rt * 4 + i][k]);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) y[j] = *reinterpret_cast<const float4*>(&sm.st[ct * 4 + j][k]);
 #pragma unroll
             for (int i = 0; i < 4; ++i)
 #pragma unroll
-                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], yv[j], acc[i][j]);
+                for (int j = 0; j < 4; ++j) {
+                    acc[i][j] = fmaf(a[i].x, y[j].x, acc[i][j]); acc[i][j] = fmaf(a[i].y, y[j].y, acc[i][j]);
+                    acc[i][j] = fmaf(a[i].z, y[j].z, acc[i][j]); acc[i][j] = fmaf(a[i].w, y[j].w, acc[i][j]);
+                }
         }
-        // sum over the quad; lane ks keeps row ks of the tile
-        float half[2][4], rowv[4];
+        // sum over the eight lanes; lane ks keeps row ks & 3 and one pair of columns
+        float half[2][4], rowv[4], v2[2];
 #pragma unroll
         for (int i = 0; i < 2; ++i)
 #pragma unroll
@@ -268,20 +289,23 @@ __global__ void __launch_bounds__(dc::kThreads) delta_chunk_scan_kernel(const fl
             const float mine = ks & 2 ? half[1][j] : half[0][j], other = ks & 2 ? half[0][j] : half[1][j];
             rowv[j] = mine + __shfl_xor_sync(0xffffffffu, other, 2);
         }
-        const int row = rt * 4 + ks;
-        if (row < C) {
-            const float4 v1 = *reinterpret_cast<const float4*>(&sm.vin[b][1][row][ct * 4]);
-            *reinterpret_cast<float4*>(&sm.y[row][ct * 4]) = make_float4(rowv[0] + v1.x, rowv[1] + v1.y, rowv[2] + v1.z, rowv[3] + v1.w);
-        } else if (c * C + row - C < e.n) {
-            const float4 o1 = *reinterpret_cast<const float4*>(&sm.vin[b][2][row - C][ct * 4]);
-            float* dst = o + (size_t)(e.row0 + c * C + row - C) * ld_o + h * s.D + c0 + ct * 4;
-            const float r[4] = {rowv[0] + o1.x, rowv[1] + o1.y, rowv[2] + o1.z, rowv[3] + o1.w};
-            if ((s.D & 3) == 0) {
-                if (c0 + ct * 4 < s.D) *reinterpret_cast<float4*>(dst) = make_float4(r[0], r[1], r[2], r[3]);
-            } else {
 #pragma unroll
-                for (int j = 0; j < 4; ++j)
-                    if (c0 + ct * 4 + j < s.D) dst[j] = r[j];
+        for (int j = 0; j < 2; ++j) {
+            const float mine = ks & 4 ? rowv[2 + j] : rowv[j], other = ks & 4 ? rowv[j] : rowv[2 + j];
+            v2[j] = mine + __shfl_xor_sync(0xffffffffu, other, 4);
+        }
+        const int row = rt * 4 + (ks & 3), col = ct * 4 + (ks >> 2) * 2;
+        if (row < C) {
+            const float2 v1 = *reinterpret_cast<const float2*>(&sm.vin[b][1][row][col]);
+            *reinterpret_cast<float2*>(&sm.y[row][col]) = make_float2(v2[0] + v1.x, v2[1] + v1.y);
+        } else if (c * C + row - C < e.n) {
+            const float2 o1 = *reinterpret_cast<const float2*>(&sm.vin[b][2][row - C][col]);
+            float* dst = o + (size_t)(e.row0 + c * C + row - C) * ld_o + h * s.D + c0 + col;
+            if ((s.D & 1) == 0) {
+                if (c0 + col < s.D) *reinterpret_cast<float2*>(dst) = make_float2(v2[0] + o1.x, v2[1] + o1.y);
+            } else {
+                if (c0 + col < s.D) dst[0] = v2[0] + o1.x;
+                if (c0 + col + 1 < s.D) dst[1] = v2[1] + o1.y;
             }
         }
         __syncthreads();
@@ -304,13 +328,12 @@ __global__ void __launch_bounds__(dc::kThreads) delta_chunk_scan_kernel(const fl
 #pragma unroll
                     for (int j = 0; j < CT; ++j) u[i][j] = fmaf(av[i], yv[j], u[i][j]);
             }
+            const float4 pd = *reinterpret_cast<const float4*>(&sm.p[b][4 * it]);
 #pragma unroll
-            for (int i = 0; i < 4; ++i)
-#pragma unroll
-                for (int j = 0; j < CT; ++j) {
-                    S[i][j] = u[i][j] * sm.p[b][4 * it + i];
-                    sm.s[4 * it + i][CT * jt + j] = S[i][j];
-                }
+            for (int j = 0; j < CT; ++j) {
+                S[0][j] = u[0][j] * pd.x; S[1][j] = u[1][j] * pd.y; S[2][j] = u[2][j] * pd.z; S[3][j] = u[3][j] * pd.w;
+                *reinterpret_cast<float4*>(&sm.st[CT * jt + j][4 * it]) = make_float4(S[0][j], S[1][j], S[2][j], S[3][j]);
+            }
         }
     }
     if (own) {

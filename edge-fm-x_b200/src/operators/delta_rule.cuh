@@ -227,7 +227,7 @@ struct DeltaDecodeParams {
 template <int RPT>
 __global__ void __launch_bounds__(512) delta_decode_kernel(const DeltaDecodeParams p) {
     constexpr int NT = 512;
-    __shared__ float sw[256], sau[256], su[256], sk[256], sr[256], sv[256], tw[512], red[NT], dot[256], part[16];
+    __shared__ float sa[256], sw[256], sau[256], su[256], sk[256], sr[256], sv[256], tw[512], red[NT], dot[256], part[16];
     const DeltaShape& s = p.s;
     const int D = s.D, HD = s.heads * D, h = blockIdx.x, c0 = h * D;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -236,6 +236,8 @@ __global__ void __launch_bounds__(512) delta_decode_kernel(const DeltaDecodePara
     float* S = p.pool + (size_t)h * D * D + col;
     constexpr int R = RPT > 0 ? RPT : 1;
     float reg[R];
+    uint4 w2_first = make_uint4(0u, 0u, 0u, 0u);                       // weights: independent of earlier launches
+    if ((tid >> 3) < D && (tid & 7) * 8 < p.ld_w2) w2_first = ld_cached(p.w2 + (size_t)(c0 + (tid >> 3)) * p.ld_w2 + (tid & 7) * 8);
     if (!p.early) { pdl_wait(); pdl_launch_dependents(); }
     const bool fresh = p.state->kv_len <= 1u;                          // first token: the state is zero
     if (RPT > 0 && act) {
@@ -246,13 +248,14 @@ __global__ void __launch_bounds__(512) delta_decode_kernel(const DeltaDecodePara
         }
     }
     if (p.early) { pdl_wait(); pdl_launch_dependents(); }
-    for (int i = tid; i < s.rank; i += NT) tw[i] = tanhf(__ldcg(p.proj + 5 * HD + i));
+    for (int i = tid; i < p.ld_w2; i += NT) tw[i] = i < s.rank ? tanhf(__ldcg(p.proj + 5 * HD + i)) : 0.f;
     float ss = 0.f;
     for (int d = tid; d < D; d += NT) {
         const float k = __ldcg(p.proj + HD + c0 + d);
         sk[d] = k;
         sr[d] = __ldcg(p.proj + c0 + d);
         sv[d] = __ldcg(p.proj + 2 * HD + c0 + d);
+        sa[d] = __ldcg(p.proj + 4 * HD + c0 + d);
         ss = fmaf(k, k, ss);
     }
     ss = warp_sum(ss);
@@ -262,16 +265,21 @@ __global__ void __launch_bounds__(512) delta_decode_kernel(const DeltaDecodePara
 #pragma unroll
     for (int w = 0; w < 16; ++w) tot += part[w];
     const float inv = 1.0f / sqrtf(tot + 1e-6f);
-    for (int d = warp; d < D; d += 16) {                               // decay: one warp per channel
-        const __nv_bfloat16* w2 = p.w2 + (size_t)(c0 + d) * p.ld_w2;
+    for (int d = tid >> 3; d < D; d += NT / 8) {                       // decay: eight lanes per channel
         float a = 0.f;
-        for (int i = lane; i < s.rank; i += 32) a = fmaf(__bfloat162float(w2[i]), tw[i], a);
-        a = warp_sum(a);
-        if (lane == 0) {
+        for (int i = (tid & 7) * 8; i < p.ld_w2; i += 64) {
+            float f[8];
+            unpack8(d == (tid >> 3) && i == (tid & 7) * 8 ? w2_first : ld_cached(p.w2 + (size_t)(c0 + d) * p.ld_w2 + i), f);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) a = fmaf(f[j], tw[i + j], a);
+        }
+#pragma unroll
+        for (int x = 4; x > 0; x >>= 1) a += __shfl_xor_sync(0xffffffffu, a, x);
+        if ((tid & 7) == 0) {
             sw[d] = expf(-kDecayRate * sigmoid_f(a + __bfloat162float(s.w0[c0 + d])));
             const float u = sk[d] * inv;
             su[d] = u;
-            sau[d] = sigmoid_f(__ldcg(p.proj + 4 * HD + c0 + d) + __bfloat162float(s.a_bias[c0 + d])) * u;
+            sau[d] = sigmoid_f(sa[d] + __bfloat162float(s.a_bias[c0 + d])) * u;
         }
     }
     __syncthreads();

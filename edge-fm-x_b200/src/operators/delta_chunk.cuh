@@ -211,8 +211,8 @@ __global__ void __launch_bounds__(dc::kScanThreads) delta_chunk_scan_kernel(cons
                                                                         const RowPlan plan) {
     using namespace dc;
     using ds::cp16;
-    constexpr int CT = DP <= 64 ? 1 : 2;                           // state columns per thread (4 rows each)
-    constexpr int RT = DP / 4;                                     // row tiles of the state
+    constexpr int RT = DP / 4;                                     // row tiles of the state (4 x 4 each)
+    constexpr int TI = (RT * 4 + 63) / 64;                         // tiles per group of four lanes
     constexpr int GROUPS = DP / kCols;
     extern __shared__ __align__(16) unsigned char dc_smem[];
     ScanSmem<DP>& sm = *reinterpret_cast<ScanSmem<DP>*>(dc_smem);
@@ -232,20 +232,26 @@ __global__ void __launch_bounds__(dc::kScanThreads) delta_chunk_scan_kernel(cons
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     stage(0, 0);
-    // this thread's tile of the state: rows 4 it .. 4 it + 3, columns CT jt ..
-    const int it = tid % RT, jt = tid / RT;
-    const bool own = jt < kCols / CT;
-    float* st = pool + (size_t)e.state * slot_stride + offset + (size_t)h * s.D * s.D + c0 + CT * jt;
-    float S[4][CT];
-    if (own) {
+    // Second product: a 4 x 4 tile of the state per four lanes (8 apart), each with a quarter of k; a lane then keeps one
+    // column of its tiles: rows 4 it .., column 4 jt + lane / 8.
+    const int kq = lane >> 3;
+    int it[TI], jc[TI];
+    bool own[TI];
+    float S[TI][4];
+    float* st = pool + (size_t)e.state * slot_stride + offset + (size_t)h * s.D * s.D + c0;
 #pragma unroll
-        for (int i = 0; i < 4; ++i)
+    for (int n = 0; n < TI; ++n) {
+        const int tile = warp * 8 + (lane & 7) + 64 * n;
+        own[n] = tile < RT * 4;
+        it[n] = tile % RT;
+        jc[n] = tile / RT * 4;
+        if (!own[n]) continue;                                     // whole groups of eight tiles: a warp's lanes agree
 #pragma unroll
-            for (int j = 0; j < CT; ++j) {
-                const int r = 4 * it + i;
-                S[i][j] = e.pos0 > 0 && r < s.D && c0 + CT * jt + j < s.D ? st[(size_t)r * s.D + j] : 0.f;
-                sm.st[CT * jt + j][r] = S[i][j];
-            }
+        for (int i = 0; i < 4; ++i) {
+            const int r = 4 * it[n] + i, j = jc[n] + kq;
+            S[n][i] = e.pos0 > 0 && r < s.D && c0 + j < s.D ? st[(size_t)r * s.D + j] : 0.f;
+            sm.st[j][r] = S[n][i];
+        }
     }
     // first product: 4 x 4 outputs per thread, k split over eight lanes
     const int ks = lane & 7, ct = lane >> 3, rt = warp;
@@ -309,41 +315,51 @@ __global__ void __launch_bounds__(dc::kScanThreads) delta_chunk_scan_kernel(cons
             }
         }
         __syncthreads();
-        if (own) {
-            float u[4][CT];
+#pragma unroll
+        for (int n = 0; n < TI; ++n) {
+            if (!own[n]) continue;
+            float u[4][4];
 #pragma unroll
             for (int i = 0; i < 4; ++i)
 #pragma unroll
-                for (int j = 0; j < CT; ++j) u[i][j] = S[i][j];
-#pragma unroll 8
-            for (int k = 0; k < 32; ++k) {
-                const float4 a = *reinterpret_cast<const float4*>(&sm.cb[b][k][4 * it]);
-                const float* vy = k < C ? &sm.vin[b][0][k][CT * jt] : &sm.y[k - C][CT * jt];
-                const float av[4] = {a.x, a.y, a.z, a.w};
-                float yv[CT];
+                for (int j = 0; j < 4; ++j) u[i][j] = 0.f;
 #pragma unroll
-                for (int j = 0; j < CT; ++j) yv[j] = vy[j];
+            for (int kk = 0; kk < 8; ++kk) {
+                const int k = kk * 4 + kq;
+                const float4 a = *reinterpret_cast<const float4*>(&sm.cb[b][k][4 * it[n]]);
+                const float4 y = *reinterpret_cast<const float4*>(kk < 4 ? &sm.vin[b][0][k][jc[n]] : &sm.y[k - C][jc[n]]);
+                const float av[4] = {a.x, a.y, a.z, a.w}, yv[4] = {y.x, y.y, y.z, y.w};
 #pragma unroll
                 for (int i = 0; i < 4; ++i)
 #pragma unroll
-                    for (int j = 0; j < CT; ++j) u[i][j] = fmaf(av[i], yv[j], u[i][j]);
+                    for (int j = 0; j < 4; ++j) u[i][j] = fmaf(av[i], yv[j], u[i][j]);
             }
-            const float4 pd = *reinterpret_cast<const float4*>(&sm.p[b][4 * it]);
+            float r[4];
 #pragma unroll
-            for (int j = 0; j < CT; ++j) {
-                S[0][j] = u[0][j] * pd.x; S[1][j] = u[1][j] * pd.y; S[2][j] = u[2][j] * pd.z; S[3][j] = u[3][j] * pd.w;
-                *reinterpret_cast<float4*>(&sm.st[CT * jt + j][4 * it]) = make_float4(S[0][j], S[1][j], S[2][j], S[3][j]);
+            for (int i = 0; i < 4; ++i) {
+                float p2[2];
+#pragma unroll
+                for (int j = 0; j < 2; ++j) {
+                    const float mine = kq & 2 ? u[i][2 + j] : u[i][j], other = kq & 2 ? u[i][j] : u[i][2 + j];
+                    p2[j] = mine + __shfl_xor_sync(0xffffffffu, other, 16);
+                }
+                const float mine = kq & 1 ? p2[1] : p2[0], other = kq & 1 ? p2[0] : p2[1];
+                r[i] = mine + __shfl_xor_sync(0xffffffffu, other, 8);
             }
+            const float4 pd = *reinterpret_cast<const float4*>(&sm.p[b][4 * it[n]]);
+            S[n][0] = (S[n][0] + r[0]) * pd.x; S[n][1] = (S[n][1] + r[1]) * pd.y;
+            S[n][2] = (S[n][2] + r[2]) * pd.z; S[n][3] = (S[n][3] + r[3]) * pd.w;
+            *reinterpret_cast<float4*>(&sm.st[jc[n] + kq][4 * it[n]]) = make_float4(S[n][0], S[n][1], S[n][2], S[n][3]);
         }
     }
-    if (own) {
 #pragma unroll
-        for (int i = 0; i < 4; ++i)
+    for (int n = 0; n < TI; ++n) {
+        if (!own[n]) continue;
 #pragma unroll
-            for (int j = 0; j < CT; ++j) {
-                const int r = 4 * it + i;
-                if (r < s.D && c0 + CT * jt + j < s.D) st[(size_t)r * s.D + j] = S[i][j];
-            }
+        for (int i = 0; i < 4; ++i) {
+            const int r = 4 * it[n] + i, j = jc[n] + kq;
+            if (r < s.D && c0 + j < s.D) st[(size_t)r * s.D + j] = S[n][i];
+        }
     }
 }
 

@@ -210,6 +210,7 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
     EFM_TRY(dev_alloc(c, &m->d_in, std::max(w_in, w_delta_in)));
     EFM_TRY(dev_alloc(c, &m->d_mix, w_mix));
     EFM_TRY(dev_alloc(c, &m->d_y, Wp));
+    EFM_TRY(dev_alloc(c, &m->d_y2, Wp));
     EFM_TRY(dev_alloc(c, &m->d_ff, w_ff));
     EFM_TRY(dev_alloc(c, &m->d_gate, m->side_p));
     EFM_TRY(dev_alloc(c, &c->logits, m->head.Np));

@@ -1,9 +1,9 @@
 // Launch sequences of the layered decoders.
 //
 // Decode (one row), per layer:  [pending output norm + residual add] + input projections | mixer (norms, cache / state
-// update, attention or recurrence) | W_o | [norm1 + add] + W_up | [PolyNorm] + W_down | [norm2 + add] + token gate |
-// token projection; what stands in brackets is the prologue of the GEMV that follows it.  The recurrent mixers launch
-// five kernels per layer, attention with a feed-forward seven.
+// update, attention or recurrence) | W_o | [norm1 + add] + W_up | [PolyNorm] + W_down | [norm2 + add] + token
+// input; what stands in brackets is the prologue of the kernel that follows it: four launches for a layer without a
+// feed-forward, six with one.
 // Many rows: tensor-core GEMMs (bf16 operands) or fp32 FMAs (32-bit mode) between row kernels.
 #include "decoder.h"
 
@@ -14,6 +14,7 @@
 #include "../operators/delta_chunk.cuh"
 #include "../operators/delta_rule.cuh"
 #include "../operators/gemm_tc.cuh"
+#include "../operators/token_side.cuh"
 #include "../operators/window_attention.cuh"
 #include "../operators/window_attention_tc.cuh"
 #define EFM_DECLARATIONS_ONLY
@@ -196,13 +197,31 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
             p.gate_table = m.side_embed;
             p.gate_ld = m.d.side_dim * m.d.num_layers;
             p.gate_off = (int)i * m.d.side_dim;
-            gemv_ext<Epi::TokenGate>(c, L, l.gate, p);
-            GemvParams q{};
-            q.prologue = kProPlain;
-            q.xf = m.d_gate;
-            q.out_f = m.d_y;
-            gemv_ext<Epi::Store32>(c, L, l.proj, q);
-            pend.y = m.d_y;
+            if (m.side_cluster > 1 && p.prologue == kProAddNorm) {
+                TokenSideParams q{};
+                p.W = l.gate.w;
+                p.N = l.gate.N;
+                p.K = l.gate.Kp;
+                p.eps = m.d.norm_eps;
+                p.state = c.state;
+                p.vocab = c.d.vocab;
+                q.p = p;
+                q.proj = l.proj.w;
+                q.side_p = l.proj.Kp;
+                q.n_out = l.proj.Np;
+                q.y = m.d_y2;
+                L.cluster_x = m.side_cluster;
+                L.launch(token_side_kernel, dim3(m.side_cluster), dim3(kGemvThreads), ts::layout(p.K, q.side_p, q.n_out, m.side_cluster).bytes, q);
+                pend.y = m.d_y2;
+            } else {
+                gemv_ext<Epi::TokenGate>(c, L, l.gate, p);
+                GemvParams q{};
+                q.prologue = kProPlain;
+                q.xf = m.d_gate;
+                q.out_f = m.d_y;
+                gemv_ext<Epi::Store32>(c, L, l.proj, q);
+                pend.y = m.d_y;
+            }
             pend.norm = l.side_norm;
         }
     }
@@ -319,7 +338,10 @@ void attention_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const R
     linear_act(c, L, l.in, m.f32 ? (void*)c.resid : m.xa, m.proj_a, plan.rows);
     TA* kp = static_cast<TA*>(l.k_pool);
     TA* vp = static_cast<TA*>(l.v_pool);
-    L.launch(qk_scatter_rows_kernel<TA, TA, TA>, dim3(plan.rows), dim3(256), 0, static_cast<const TA*>(m.proj_a), l.in.Np, static_cast<TA*>(m.q), kp, vp, s, plan);
+    int lanes = 8;                                                  // 8 channels each: at most 256 (padded) channels a head
+    while (lanes * 8 < std::max(s.Dp, s.Vp)) lanes *= 2;
+    L.launch(qk_scatter_rows_kernel<TA, TA, TA>, dim3(plan.rows), dim3(256), 0, static_cast<const TA*>(m.proj_a), l.in.Np, static_cast<TA*>(m.q), kp, vp, s, plan,
+             lanes);
     auto cuda_cores = [&](const RowTile* list, int n) {
         if (n > 0)
             L.launch(window_attention_rows_kernel<TA, TA, TA>, dim3(n, s.H), dim3(256), wa::rows_smem_bytes(s.Dp, s.Vp), static_cast<const TA*>(m.q),
@@ -476,6 +498,32 @@ size_t decoder_delta_pack_floats(int heads, int dim, int rows, int entries) {
     return n;
 }
 
+// Widest cluster the one-launch token input fits; 1: two products instead.
+static cudaError_t fit_side_cluster(DecoderModel& m, int optin) {
+    m.side_cluster = 1;
+    if (m.d.side_dim <= 0) return cudaSuccess;
+    const bool wide = cudaFuncSetAttribute(token_side_kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess;
+    for (int cs = wide ? 16 : 8; cs > 1; cs >>= 1) {
+        const size_t bytes = ts::layout(m.Wp, m.side_p, m.Wp, cs).bytes;
+        if (bytes + 2048 > (size_t)optin) break;                   // narrower clusters need more per block
+        if (smem_attr(token_side_kernel, bytes) != cudaSuccess) continue;
+        cudaLaunchConfig_t cfg = {};
+        cfg.gridDim = dim3(cs, 1, 1);
+        cfg.blockDim = dim3(kGemvThreads);
+        cfg.dynamicSmemBytes = bytes;
+        cudaLaunchAttribute at;
+        at.id = cudaLaunchAttributeClusterDimension;
+        at.val.clusterDim.x = (unsigned)cs;
+        at.val.clusterDim.y = at.val.clusterDim.z = 1;
+        cfg.attrs = &at;
+        cfg.numAttrs = 1;
+        int n = 0;
+        if (cudaOccupancyMaxActiveClusters(&n, token_side_kernel, &cfg) == cudaSuccess && n >= 1) { m.side_cluster = cs; break; }
+    }
+    (void)cudaGetLastError();
+    return m.side_cluster > 1 ? smem_attr(token_side_kernel, (size_t)optin - 2048) : cudaSuccess;
+}
+
 cudaError_t configure_decoder(DecoderModel& m) {
     int dev = 0, optin = 0;
     cudaError_t e = cudaGetDevice(&dev);
@@ -500,6 +548,7 @@ cudaError_t configure_decoder(DecoderModel& m) {
     if (e == cudaSuccess) e = smem_attr(delta_chunk_scan_kernel<64>, sizeof(dc::ScanSmem<64>));
     if (e == cudaSuccess) e = smem_attr(delta_chunk_scan_kernel<96>, sizeof(dc::ScanSmem<96>));
     if (e == cudaSuccess) e = smem_attr(delta_chunk_scan_kernel<128>, sizeof(dc::ScanSmem<128>));
+    if (e == cudaSuccess) e = fit_side_cluster(m, optin);
     m.attn_cluster = 16;
     if (e == cudaSuccess) e = m.f32 ? fit_cluster<float, 64>(m.attn_cluster) : fit_cluster<__nv_bfloat16, 64>(m.attn_cluster);
     if (e == cudaSuccess) e = m.f32 ? fit_cluster<float, 128>(m.attn_cluster) : fit_cluster<__nv_bfloat16, 128>(m.attn_cluster);

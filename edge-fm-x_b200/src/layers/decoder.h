@@ -59,8 +59,8 @@ struct DecoderModel {
     float* tap = nullptr;                 // debugging / tests: residual stream after every layer [layers][rows][Wp]
     int tap_rows = 0, tap_row0 = 0;
     // one-row buffers
-    float *d_in = nullptr, *d_mix = nullptr, *d_y = nullptr, *d_ff = nullptr, *d_gate = nullptr;
-    int attn_cluster = 8;
+    float *d_in = nullptr, *d_mix = nullptr, *d_y = nullptr, *d_y2 = nullptr, *d_ff = nullptr, *d_gate = nullptr;
+    int attn_cluster = 8, side_cluster = 1;
 };
 
 // One decode step of the bound slot (reads the device state); sample: run the sampler and advance the state.

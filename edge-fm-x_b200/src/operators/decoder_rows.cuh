@@ -53,31 +53,56 @@ __global__ void __launch_bounds__(256) add_norm_rows_kernel(float* __restrict__ 
     }
 }
 
-// out = c0 rms(z) + c1 rms(z^2) + c2 rms(z^3) + c3 over n channels; pads [n, ld) become zero.  One block per row.
+__device__ __forceinline__ void load8(const float* p, float (&f)[8]) {
+    const float4 a = load4(p), b = load4(p + 4);
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&f)[8]) { unpack8(ld_cached(p), f); }
+__device__ __forceinline__ void store8(float* p, const float (&f)[8]) {
+    store4(p, make_float4(f[0], f[1], f[2], f[3]));
+    store4(p + 4, make_float4(f[4], f[5], f[6], f[7]));
+}
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&f)[8]) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
+}
+
+// out = c0 rms(z) + c1 rms(z^2) + c2 rms(z^3) + c3 over n channels; pads [n, ld) become zero.  One block per row; the first
+// 8 * 256 * KEEP channels of the row stay in registers between the sums and the polynomial.
 template <typename T>
 __global__ void __launch_bounds__(256) poly_norm_rows_kernel(const T* __restrict__ z, T* __restrict__ out, const __nv_bfloat16* __restrict__ coef, int n,
                                                              int ld, float eps) {
+    constexpr int KEEP = 4;
     __shared__ float part[3][8];
     const size_t base = (size_t)blockIdx.x * ld;
-    const int nv = ld / 4;
+    const int nv = ld / 8;                                              // ld % 8 == 0, pads of z are zero
+    float keep[KEEP][8];
     float s0 = 0.f, s1 = 0.f, s2 = 0.f;
-    auto add = [&](float v) { const float v2 = v * v, v4 = v2 * v2; s0 += v2; s1 += v4; s2 = fmaf(v4, v2, s2); };
-    for (int c = threadIdx.x; c < nv; c += 256) {
-        const float4 v = load4(z + base + 4 * c);                       // pads are zero
-        add(v.x); add(v.y); add(v.z); add(v.w);
-    }
+    auto add = [&](const float (&f)[8]) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) { const float v2 = f[j] * f[j], v4 = v2 * v2; s0 += v2; s1 += v4; s2 = fmaf(v4, v2, s2); }
+    };
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+        if ((int)threadIdx.x + 256 * i < nv) load8(z + base + 8 * (threadIdx.x + 256 * i), keep[i]);
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+        if ((int)threadIdx.x + 256 * i < nv) add(keep[i]);
+    for (int c = threadIdx.x + 256 * KEEP; c < nv; c += 256) { float f[8]; load8(z + base + 8 * c, f); add(f); }
     s0 = block_sum_256(s0, part[0]);
     s1 = block_sum_256(s1, part[1]);
     s2 = block_sum_256(s2, part[2]);
     const float c0 = __bfloat162float(coef[0]) / sqrtf(s0 / (float)n + eps), c1 = __bfloat162float(coef[1]) / sqrtf(s1 / (float)n + eps),
                 c2 = __bfloat162float(coef[2]) / sqrtf(s2 / (float)n + eps), c3 = __bfloat162float(coef[3]);
-    for (int c = threadIdx.x; c < nv; c += 256) {
-        const float4 v = load4(z + base + 4 * c);
-        float f[4] = {v.x, v.y, v.z, v.w};
+    auto emit = [&](int c, const float (&f)[8]) {
+        float r[8];
 #pragma unroll
-        for (int j = 0; j < 4; ++j) f[j] = 4 * c + j < n ? fmaf(f[j], fmaf(f[j], fmaf(f[j], c2, c1), c0), c3) : 0.f;
-        store4(out + base + 4 * c, make_float4(f[0], f[1], f[2], f[3]));
-    }
+        for (int j = 0; j < 8; ++j) r[j] = 8 * c + j < n ? fmaf(f[j], fmaf(f[j], fmaf(f[j], c2, c1), c0), c3) : 0.f;
+        store8(out + base + 8 * c, r);
+    };
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+        if ((int)threadIdx.x + 256 * i < nv) emit(threadIdx.x + 256 * i, keep[i]);
+    for (int c = threadIdx.x + 256 * KEEP; c < nv; c += 256) { float f[8]; load8(z + base + 8 * c, f); emit(c, f); }
 }
 
 // out[row][c] = gelu_tanh(s[row][c]) * table[id(row)][off + c] for c < n, zero in the pads.

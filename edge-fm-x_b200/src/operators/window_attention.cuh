@@ -37,33 +37,61 @@ template <> __device__ __forceinline__ float round_as<float>(float v) { return v
 template <> __device__ __forceinline__ float round_as<__nv_bfloat16>(float v) { return round_bf16(v); }
 
 // ---- many rows: norms and scatter --------------------------------------------------------------------------------
-// One block per row, one warp per head at a time.  TI: projections, TQ: q operand, TC: cache.
+template <typename T>
+__device__ __forceinline__ void load_head8(const T* x, int d, int D, bool vec, float (&f)[8]) {
+    if (vec && d + 8 <= D) {
+        if constexpr (sizeof(T) == 2) {
+            unpack8(ld_cached(x + d), f);
+        } else {
+            const float4 a = *reinterpret_cast<const float4*>(x + d), b = *reinterpret_cast<const float4*>(x + d + 4);
+            f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+        }
+    } else {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) f[j] = d + j < D ? to_f32(x[d + j]) : 0.f;
+    }
+}
+template <typename T>
+__device__ __forceinline__ void store_head8(T* p, const float (&f)[8]) {          // 16-byte aligned
+    if constexpr (sizeof(T) == 2) {
+        *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
+    } else {
+        *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+        *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
+    }
+}
+
+// One block per row; `lanes` (8, 16 or 32) threads share a head, 8 channels each.  TI: projections, TQ: q operand, TC: cache.
 template <typename TI, typename TQ, typename TC>
 __global__ void __launch_bounds__(256) qk_scatter_rows_kernel(const TI* __restrict__ qkv, int ld, TQ* __restrict__ q_out, TC* __restrict__ k_pool,
-                                                              TC* __restrict__ v_pool, const WindowAttnShape s, const RowPlan plan) {
-    const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+                                                              TC* __restrict__ v_pool, const WindowAttnShape s, const RowPlan plan, int lanes) {
+    const int row = blockIdx.x, l = threadIdx.x & (lanes - 1), per = 256 / lanes;
     const RowEntry e = plan.of_row(row);
     const size_t cr = plan.cache_row(e, e.pos0 + row - e.row0);
-    const TI* src = qkv + (size_t)row * ld;
-    for (int u = warp; u < s.H + 2 * s.G; u += 8) {
-        if (u < s.H + s.G) {
-            const bool is_q = u < s.H;
-            const TI* x = src + (size_t)u * s.D;                       // q heads, then k heads
-            const __nv_bfloat16* w = is_q ? s.q_norm : s.k_norm;
-            float ss = 0.f;
-            for (int d = lane; d < s.D; d += 32) { const float v = to_f32(x[d]); ss = fmaf(v, v, ss); }
-            const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)s.D + s.eps);
-            TQ* qd = q_out + ((size_t)row * s.H + u) * s.Dp;
-            TC* kd = k_pool + (cr * s.G + (u - s.H)) * s.Dp;
-            for (int d = lane; d < s.Dp; d += 32) {
-                const float v = d < s.D ? to_f32(x[d]) * inv * __bfloat162float(w[d]) : 0.f;
-                if (is_q) store_f32(qd + d, v); else store_f32(kd + d, v);
+    const TI* src = qkv + (size_t)row * ld;                            // ld % 8 == 0
+    const bool vec = (s.D & 7) == 0, vecv = vec && (s.Dv & 7) == 0;
+    const int units = s.H + 2 * s.G, d = 8 * l;
+    for (int u0 = 0; u0 < units; u0 += per) {                          // every thread takes part in the shuffles
+        const int u = u0 + threadIdx.x / lanes;
+        const bool qk = u < s.H + s.G;
+        float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+        if (qk) load_head8(src + (size_t)u * s.D, d, s.D, vec, f);     // q heads, then k heads
+        else if (u < units) load_head8(src + (size_t)(s.H + s.G) * s.D + (size_t)(u - s.H - s.G) * s.Dv, d, s.Dv, vecv, f);
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) ss = fmaf(f[j], f[j], ss);
+        for (int x = lanes / 2; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+        if (qk) {
+            const float inv = 1.0f / sqrtf(ss / (float)s.D + s.eps);
+            const __nv_bfloat16* w = u < s.H ? s.q_norm : s.k_norm;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) f[j] = d + j < s.D ? f[j] * inv * __bfloat162float(w[d + j]) : 0.f;
+            if (d < s.Dp) {
+                if (u < s.H) store_head8(q_out + ((size_t)row * s.H + u) * s.Dp + d, f);
+                else store_head8(k_pool + (cr * s.G + (u - s.H)) * s.Dp + d, f);
             }
-        } else {
-            const int g = u - s.H - s.G;
-            const TI* x = src + (size_t)(s.H + s.G) * s.D + (size_t)g * s.Dv;
-            TC* vd = v_pool + (cr * s.G + g) * s.Vp;
-            for (int d = lane; d < s.Vp; d += 32) store_f32(vd + d, d < s.Dv ? to_f32(x[d]) : 0.f);
+        } else if (u < units && d < s.Vp) {
+            store_head8(v_pool + (cr * s.G + (u - s.H - s.G)) * s.Vp + d, f);
         }
     }
 }

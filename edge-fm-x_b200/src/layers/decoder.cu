@@ -107,9 +107,9 @@ void launch_attn_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, con
     p.state = c.state;
     p.out = m.d_mix;
     p.early = early ? 1 : 0;
-    // one block per page of the visible range, up to the cluster width (a power of two)
+    // one block per 64 keys of the visible range, up to the cluster width (a power of two)
     int pages = slot.n_pages;
-    if (l.d.window > 0) pages = std::min(pages, (l.d.window + kPageTokens - 2) / kPageTokens + 1);
+    if (l.d.window > 0) pages = std::min(pages, (l.d.window + kPageTokens - 1) / kPageTokens);
     int cluster = 1;
     while (cluster < pages && cluster < m.attn_cluster) cluster *= 2;
     const int v = std::max(l.Dp, l.Vp);

@@ -7,6 +7,8 @@
 #pragma once
 #include <cooperative_groups.h>
 
+#include <utility>
+
 #include "gemv.cuh"
 
 namespace efm {
@@ -51,6 +53,7 @@ __global__ void __launch_bounds__(kGemvThreads, 1) token_side_kernel(const Token
     float* g = reinterpret_cast<float*>(ts_smem + l.off_g);
     float* red = reinterpret_cast<float*>(ts_smem + l.off_red);
     const int g0 = rank * l.gate_rows, ng = max(0, min(l.gate_rows, q.side_p - g0)), o0 = rank * l.proj_rows, no = max(0, min(l.proj_rows, q.n_out - o0));
+    auto started = cl.barrier_arrive();                              // waited for before the first store into another block
     pdl_launch_dependents();
     auto cp16 = [](void* dst, const void* src) {
         asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
@@ -66,6 +69,7 @@ __global__ void __launch_bounds__(kGemvThreads, 1) token_side_kernel(const Token
     gemv_stage_ext(p, p.K >> 3, ts_smem, gemv_xbytes(p.K));
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
+    cl.barrier_wait(std::move(started));
     const float* xs = reinterpret_cast<const float*>(ts_smem);
     // ---- gate rows: `parts` warps share a row ----------------------------------------------------------------------
     int parts = 1;

@@ -12,6 +12,8 @@
 #pragma once
 #include <cooperative_groups.h>
 
+#include <utility>
+
 #include "common.cuh"
 #include "row_plan.cuh"
 
@@ -216,7 +218,9 @@ struct Smem {
     float knew[MAXP], vnew[MAXP];
     float p[kHeads][kPageTokens];
     float alpha[kHeads], m[kHeads], l[kHeads];
-    float out[kHeads][MAXP];                   // this block's un-normalised output
+    // what the blocks of the cluster hand to this one: its share of their un-normalised outputs, and everybody's (m, l)
+    float rm[16][kHeads], rl[16][kHeads];
+    float rout[kHeads * MAXP + 16 * 16];       // [split][share of the outputs]
     float red[8192];                           // [key groups][kHeads][Vp]: at most 256 / (Vp / 4) * 8 * Vp = 8192
 };
 }  // namespace wd
@@ -258,8 +262,8 @@ template <> struct Row4<float> {
     __device__ __forceinline__ void get(float (&f)[4]) const { f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w; }
 };
 
-// grid (splits = cluster size, kv_heads * head blocks); block `split` walks every splits-th page of the visible range.
-// VM: upper bound of Dp and Vp.
+// grid (splits = cluster size, kv_heads * head blocks); the visible keys are dealt out evenly, block `split` walks its share in
+// tiles of 64.  VM: upper bound of Dp and Vp.
 template <typename TC, int VM>
 __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(const WindowDecodeParams<TC> p) {
     using namespace wd;
@@ -276,33 +280,37 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
     const int tpr = s.Vp / 4, kg = kThreads / tpr, dpart = tid % tpr, tg = tid / tpr;     // P.V phase: 4 channels per thread
     const bool pv = tg < kg;
 
+    namespace cg = cooperative_groups;
+    cg::cluster_group cl = cg::this_cluster();
+    auto started = cl.barrier_arrive();                                // waited for before the first store into another block
     if (!p.early) { pdl_wait(); pdl_launch_dependents(); }
     const int kv_len = (int)p.state->kv_len, pos = kv_len - 1;
     const bool ok = kv_len > 0 && kv_len <= p.max_pages * kPageTokens;
     const int lo = s.window > 0 ? max(0, kv_len - s.window) : 0;
-    const int pg0 = lo / kPageTokens, pg1 = ok ? pos / kPageTokens : pg0 - 1;
+    const int chunk = ok ? (kv_len - lo + n_splits - 1) / n_splits : 0;
+    const int begin = lo + split * chunk, end = ok ? min(kv_len, begin + chunk) : begin;
 
     Row8<TC> kr[KC];
     Row4<TC> vr[VK];
-    // rows of page `pg` except the one this launch appends
-    auto load_page = [&](int pg) {
-        const size_t base = (size_t)p.pages[pg] * kPageTokens;
-        const int j = pg * kPageTokens + key;
-        if (j >= lo && j < pos) {
+    auto pool_row = [&](int j) { return (size_t)p.pages[j / kPageTokens] * kPageTokens + j % kPageTokens; };
+    // 64 keys from j0, except the one this launch appends
+    auto load_tile = [&](int j0) {
+        const int j = j0 + key;
+        if (j < end && j != pos) {
+            const TC* src = p.k_pool + (pool_row(j) * s.G + g) * s.Dp;
 #pragma unroll
             for (int c = 0; c < KC; ++c)
-                if ((c * 4 + part) * 8 < s.Dp) kr[c].load(p.k_pool + ((base + key) * s.G + g) * s.Dp + (c * 4 + part) * 8);
+                if ((c * 4 + part) * 8 < s.Dp) kr[c].load(src + (c * 4 + part) * 8);
         }
         if (pv) {
 #pragma unroll
             for (int i = 0; i < VK; ++i) {
-                const int kk = tg + i * kg, jj = pg * kPageTokens + kk;
-                if (kk < kPageTokens && jj >= lo && jj < pos) vr[i].load(p.v_pool + ((base + kk) * s.G + g) * s.Vp + dpart * 4);
+                const int kk = tg + i * kg, jj = j0 + kk;
+                if (kk < kPageTokens && jj < end && jj != pos) vr[i].load(p.v_pool + (pool_row(jj) * s.G + g) * s.Vp + dpart * 4);
             }
         }
     };
-    int pg = pg0 + split;
-    if (pg <= pg1) load_page(pg);
+    if (begin < end) load_tile(begin);
     if (p.early) { pdl_wait(); pdl_launch_dependents(); }
 
     // ---- norms of this token's q heads and k, v ------------------------------------------------------------------
@@ -310,11 +318,20 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
         const bool is_q = u < nh;
         const float* x = is_q ? p.qkv + (size_t)(h0 + u) * s.D : p.qkv + (size_t)(s.H + g) * s.D;
         const __nv_bfloat16* w = is_q ? s.q_norm : s.k_norm;
-        float ss = 0.f;
-        for (int d = lane; d < s.D; d += 32) { const float v = __ldcg(x + d); ss = fmaf(v, v, ss); }
+        float f[VM / 32], ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < VM / 32; ++i) {
+            const int d = lane + 32 * i;
+            f[i] = d < s.D ? __ldcg(x + d) : 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < VM / 32; ++i) ss = fmaf(f[i], f[i], ss);
         const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)s.D + s.eps);
-        for (int d = lane; d < s.Dp; d += 32) {
-            const float v = d < s.D ? __ldcg(x + d) * inv * __bfloat162float(w[d]) : 0.f;
+#pragma unroll
+        for (int i = 0; i < VM / 32; ++i) {
+            const int d = lane + 32 * i;
+            if (d >= s.Dp) continue;
+            const float v = d < s.D ? f[i] * inv * __bfloat162float(w[d]) : 0.f;
             if (is_q) sm.q[u][d] = v; else sm.knew[d] = round_as<TC>(v);
         }
     }
@@ -322,8 +339,8 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
         sm.vnew[d] = d < s.Dv ? round_as<TC>(__ldcg(p.qkv + (size_t)(s.H + s.G) * s.D + (size_t)g * s.Dv + d)) : 0.f;
     if (tid < kHeads) { sm.m[tid] = -INFINITY; sm.l[tid] = 0.f; }
     __syncthreads();
-    if (ok && pg1 % n_splits == (split + pg0) % n_splits && pg1 >= pg0 + split && blockIdx.y % hb == 0) {     // the block that walks the last page appends
-        const size_t cr = (size_t)p.pages[pg1] * kPageTokens + pos % kPageTokens;
+    if (begin <= pos && pos < end && blockIdx.y % hb == 0) {           // the block that walks the newest key appends it
+        const size_t cr = pool_row(pos);
         for (int d = tid; d < s.Dp; d += kThreads) store_f32(p.k_pool + (cr * s.G + g) * s.Dp + d, sm.knew[d]);
         for (int d = tid; d < s.Vp; d += kThreads) store_f32(p.v_pool + (cr * s.G + g) * s.Vp + d, sm.vnew[d]);
     }
@@ -335,9 +352,9 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
 #pragma unroll
         for (int j = 0; j < 4; ++j) acc[h][j] = 0.f;
 
-    for (; pg <= pg1; pg += n_splits) {
-        const int j = pg * kPageTokens + key;
-        const bool vis = j >= lo && j <= pos;
+    for (int j0 = begin; j0 < end; j0 += kPageTokens) {
+        const int j = j0 + key;
+        const bool vis = j < end;
         // ---- scores: 4 threads per key ----------------------------------------------------------------------------
         float kf[KC][8];
 #pragma unroll
@@ -374,7 +391,7 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
         // ---- online softmax: one warp per head --------------------------------------------------------------------
         if (warp < nh) {
             const float s0 = sm.p[warp][lane], s1 = sm.p[warp][lane + 32];
-            const float m_old = sm.m[warp], mn = fmaxf(m_old, warp_max(fmaxf(s0, s1)));       // the page holds a visible key
+            const float m_old = sm.m[warp], mn = fmaxf(m_old, warp_max(fmaxf(s0, s1)));       // the tile holds a visible key
             const float p0 = expf(s0 - mn), p1 = expf(s1 - mn);
             sm.p[warp][lane] = p0;
             sm.p[warp][lane + 32] = p1;
@@ -397,8 +414,8 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
                 }
 #pragma unroll
             for (int i = 0; i < VK; ++i) {
-                const int kk = tg + i * kg, jj = pg * kPageTokens + kk;
-                if (kk < kPageTokens && jj >= lo && jj <= pos) {
+                const int kk = tg + i * kg, jj = j0 + kk;
+                if (kk < kPageTokens && jj < end) {
                     float v[4];
                     if (jj == pos) {
 #pragma unroll
@@ -416,7 +433,7 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
                 }
             }
         }
-        if (pg + n_splits <= pg1) load_page(pg + n_splits);
+        if (j0 + kPageTokens < end) load_tile(j0 + kPageTokens);
         __syncthreads();
     }
     // ---- sum over the key groups, then over the splits -------------------------------------------------------------
@@ -426,29 +443,34 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
             if (h < nh) *reinterpret_cast<float4*>(sm.red + ((size_t)tg * kHeads + h) * s.Vp + dpart * 4) = make_float4(acc[h][0], acc[h][1], acc[h][2], acc[h][3]);
     }
     __syncthreads();
-    for (int i = tid; i < nh * s.Vp; i += kThreads) {
-        const int h = i / s.Vp, d = i - h * s.Vp;
+    // every output belongs to one block of the cluster: hand it over, then merge the shares locally
+    cl.barrier_wait(std::move(started));
+    const int n_out = nh * s.Dv, share = (n_out + n_splits - 1) / n_splits;
+    for (int i = tid; i < n_out; i += kThreads) {
+        const int h = i / s.Dv, d = i - h * s.Dv;
         float v = 0.f;
         for (int t = 0; t < kg; ++t) v += sm.red[((size_t)t * kHeads + h) * s.Vp + d];
-        sm.out[h][d] = v;
+        const int owner = i / share;
+        *cl.map_shared_rank(&sm.rout[split * share + i - owner * share], owner) = v;
     }
-    namespace cg = cooperative_groups;
-    cg::cluster_group cl = cg::this_cluster();
+    for (int i = tid; i < n_splits * kHeads; i += kThreads) {
+        const int r = i / kHeads, h = i - r * kHeads;
+        *cl.map_shared_rank(&sm.rm[split][h], r) = sm.m[h];
+        *cl.map_shared_rank(&sm.rl[split][h], r) = sm.l[h];
+    }
     cl.sync();
-    for (int i = split * kThreads + tid; i < nh * s.Dv; i += n_splits * kThreads) {
-        const int h = i / s.Dv, d = i - h * s.Dv;
+    for (int i = tid; i < share && split * share + i < n_out; i += kThreads) {
+        const int o = split * share + i, h = o / s.Dv, d = o - h * s.Dv;
         float m = -INFINITY;
-        for (int r = 0; r < n_splits; ++r) m = fmaxf(m, *cl.map_shared_rank(&sm.m[h], r));
+        for (int r = 0; r < n_splits; ++r) m = fmaxf(m, sm.rm[r][h]);
         float num = 0.f, den = 0.f;
         for (int r = 0; r < n_splits; ++r) {
-            const float mr = *cl.map_shared_rank(&sm.m[h], r);
-            const float w = mr == -INFINITY ? 0.f : expf(mr - m);
-            num = fmaf(w, *cl.map_shared_rank(&sm.out[h][d], r), num);
-            den = fmaf(w, *cl.map_shared_rank(&sm.l[h], r), den);
+            const float mr = sm.rm[r][h], w = mr == -INFINITY ? 0.f : expf(mr - m);
+            num = fmaf(w, sm.rout[r * share + i], num);
+            den = fmaf(w, sm.rl[r][h], den);
         }
         p.out[(size_t)(h0 + h) * s.Dv + d] = den > 0.f ? num / den : 0.f;
     }
-    cl.sync();
 }
 
 }  // namespace efm

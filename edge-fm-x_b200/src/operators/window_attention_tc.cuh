@@ -3,7 +3,8 @@
 // two threads per query row) over a paged cache, with the per-head multiplier and the distance bias applied to the scores
 // in fp32.  A key tile is exactly one 64-token page: its TMA coordinate is the page number of the sequence's table.
 // Block = 128 rows of one entry x one head, 256 threads.  Rows of the tile that belong to the next entry are computed and
-// not stored.  Every mbarrier wait is bounded and raises *error.
+// not stored.  The weights enter P V as a bf16 pair high + low (16 bits of mantissa), written straight into tensor memory.
+// Every mbarrier wait is bounded and raises *error.
 #pragma once
 #include "attention_tc.cuh"
 #include "window_attention.cuh"
@@ -17,17 +18,33 @@ constexpr int BM = 128, BN = kPageTokens, kThreads = 256, kMaxTiles = 1024;
 template <int DP, int VP>
 struct Cfg {
     static constexpr int QB = DP / 64, VB = VP / 64;         // 64-channel boxes per row
-    static constexpr int Q_BYTES = BM * 128 * QB, K_BYTES = BN * 128 * QB, V_BYTES = BN * 128 * VB, P_BYTES = BM * 128;
-    static constexpr int O_COL = 64;
-    static constexpr int TMEM_COLS = VP == 64 ? 128 : 256;   // S (64 columns) + O tile, power of two
+    static constexpr int Q_BYTES = BM * 128 * QB, K_BYTES = BN * 128 * QB, V_BYTES = BN * 128 * VB;
+    static constexpr int P_COL = 64, O_COL = 128;
+    static constexpr int TMEM_COLS = 256;                    // S (64 columns) | P high, P low (32 each) | O tile, power of two
     static constexpr int HALF = VP / 2;
-    static constexpr size_t SMEM = (size_t)Q_BYTES + 2 * K_BYTES + V_BYTES + P_BYTES + 2 * BM * 4 + 128 + kMaxTiles * 4 + 1024;
+    static constexpr size_t SMEM = (size_t)Q_BYTES + 2 * K_BYTES + V_BYTES + 2 * BM * 4 + 128 + kMaxTiles * 4 + 1024;
 };
+
+__device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16]) {
+    asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};" ::"r"(taddr), "r"(r[0]), "r"(r[1]),
+                 "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]),
+                 "r"(r[14]), "r"(r[15]) : "memory");
+}
+// D = A . B with A in tensor memory (bf16 pairs along K in 32-bit columns) and B by shared-memory descriptor
+__device__ __forceinline__ void umma_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+    asm volatile(
+        "{\n"
+        ".reg .pred p;\n"
+        "setp.ne.b32 p, %4, 0;\n"
+        "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n"
+        "}\n"
+        ::"r"(tmem_d), "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate) : "memory");
+}
 
 }  // namespace wt
 
 template <int DP, int VP>
-__global__ void __launch_bounds__(wt::kThreads) window_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
+__global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                                                                            const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out,
                                                                            int ld_out, const WindowAttnShape s, const RowPlan plan,
                                                                            const RowTile* __restrict__ tiles, int* error) {
@@ -46,10 +63,10 @@ __global__ void __launch_bounds__(wt::kThreads) window_attention_tc_kernel(const
     const uint32_t raw = smem_u32(wt_smem);
     const uint32_t base = (raw + 1023u) & ~1023u;
     unsigned char* base_ptr = wt_smem + (base - raw);
-    const uint32_t sQ = base, sK = sQ + C::Q_BYTES, sV = sK + 2 * C::K_BYTES, sP = sV + C::V_BYTES;
-    constexpr int XCH = C::Q_BYTES + 2 * C::K_BYTES + C::V_BYTES + C::P_BYTES;
+    const uint32_t sQ = base, sK = sQ + C::Q_BYTES, sV = sK + 2 * C::K_BYTES;
+    constexpr int XCH = C::Q_BYTES + 2 * C::K_BYTES + C::V_BYTES;
     float* xch = reinterpret_cast<float*>(base_ptr + XCH);                       // [2][BM]
-    const uint32_t bars = sP + C::P_BYTES + 2 * BM * 4;
+    const uint32_t bars = sV + C::V_BYTES + 2 * BM * 4;
     const uint32_t qfull = bars, kfull0 = bars + 8, vfull = bars + 24, sbar = bars + 32, obar = bars + 40;
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(base_ptr + XCH + 2 * BM * 4 + 48);
     volatile int* abort_s = reinterpret_cast<volatile int*>(tmem_slot + 1);
@@ -151,24 +168,20 @@ __global__ void __launch_bounds__(wt::kThreads) window_attention_tc_kernel(const
         const float alpha = m == -INFINITY ? 0.f : at::ex2(m - mb);
         m = m_new;
         float rs = 0.f;
-        uint32_t pk[16];
+        uint32_t pk[16], pl[16];
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
             const float a = at::ex2(sc[i] - mb), b = at::ex2(sc[i + 1] - mb);      // exp2(-inf) = 0 for masked keys
             rs += a + b;
-            pk[i >> 1] = pack_bf16(a, b);
+            pk[i >> 1] = pack_bf16(a, b);                            // the weights as a bf16 pair high + low: 16 bits of mantissa
+            pl[i >> 1] = pack_bf16(a - bf16lo(pk[i >> 1]), b - bf16hi(pk[i >> 1]));
         }
         l = l * alpha + rs;
-        {   // P row into the K-major, 128-byte-swizzled operand layout: chunk c of row r lives at chunk c ^ (r % 8)
-            const uint32_t prow = sP + (uint32_t)(row >> 3) * 1024u + (uint32_t)(row & 7) * 128u;
-#pragma unroll
-            for (int c = 0; c < 4; ++c) {
-                const uint32_t addr = prow + (uint32_t)(((hf * 4 + c) ^ (row & 7)) << 4);
-                asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(addr), "r"(pk[4 * c]), "r"(pk[4 * c + 1]), "r"(pk[4 * c + 2]),
-                             "r"(pk[4 * c + 3]) : "memory");
-            }
-        }
-        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+        // P into tensor memory, where the MMA takes it as its A operand: lane = row, one column = two neighbouring keys
+        const uint32_t prow = tmem + ((uint32_t)((warp & 3) * 32) << 16) + (uint32_t)(C::P_COL + hf * 16);
+        wt::tmem_st16(prow, pk);
+        wt::tmem_st16(prow + 32u, pl);
+        asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
         asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
         __syncthreads();
         if (tid == 0) {
@@ -176,8 +189,8 @@ __global__ void __launch_bounds__(wt::kThreads) window_attention_tc_kernel(const
             bool ok = mbar_wait(vfull, (uint32_t)j & 1u, abort_s);
             if (ok) {
 #pragma unroll
-                for (int k = 0; k < BN / 16; ++k)
-                    umma_d(tmem + C::O_COL, umma_desc(sP) + (uint64_t)(k * 2), vdesc + (uint64_t)(k * (2048 >> 4)), kDescO, k != 0 ? 1u : 0u);
+                for (int k = 0; k < 2 * (BN / 16); ++k)              // high halves, then low halves
+                    wt::umma_ts(tmem + C::O_COL, tmem + (uint32_t)(C::P_COL + 8 * k), vdesc + (uint64_t)((k % (BN / 16)) * (2048 >> 4)), kDescO, k != 0 ? 1u : 0u);
                 umma_commit(obar);
                 if (j + 1 < ntiles) {
                     ok = mbar_wait(kfull0 + 8 * ((j + 1) & 1), (uint32_t)((j + 1) >> 1) & 1u, abort_s);

@@ -29,6 +29,10 @@ public:
     int32_t take_state();
     int32_t free_pages() const { return (int32_t)free_.size(); }
     int32_t free_states() const { return (int32_t)states_.size(); }
+    int32_t pages_held(int32_t slot) const {
+        auto it = seqs_.find(slot);
+        return it == seqs_.end() ? 0 : (int32_t)it->second.pages.size();
+    }
     bool holds(int32_t slot) const { return seqs_.count(slot) > 0; }
     static int32_t pages_for(int32_t tokens) { return (tokens + kCachePageTokens - 1) / kCachePageTokens; }
 

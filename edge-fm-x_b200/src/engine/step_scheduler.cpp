@@ -1,5 +1,6 @@
 #include "step_scheduler.h"
 
+#include <algorithm>
 #include <set>
 
 namespace edge_fm {
@@ -32,12 +33,20 @@ std::vector<PlannedEntry> StepScheduler::plan(const std::vector<StepEntry>& entr
         if (e.tokens.empty()) throw InvalidRequestError("step entry without tokens: " + e.id);
         if (!seen.insert(e.id).second) throw InvalidRequestError("request appears twice in one step: " + e.id);
     }
+    int32_t pages = 0, fresh = 0;
+    for (const StepEntry& e : entries) {
+        auto it = live_.find(e.id);
+        const int32_t have = it == live_.end() ? 0 : cache_->pages_held(it->second.slot);
+        pages += std::max(0, PagedCache::pages_for(length(e.id) + (int32_t)e.tokens.size()) - have);
+        fresh += it == live_.end() ? 1 : 0;
+    }
+    if (fresh > (int32_t)free_slots_.size()) throw InvalidRequestError("no free slot for the step's new requests");
+    if (pages > cache_->free_pages()) throw InvalidRequestError("the cache pool has no room for the step's tokens");
     std::vector<PlannedEntry> out;
     for (const StepEntry& e : entries) {
         const int32_t len = length(e.id);
         if (!try_admit(e.id, len + (int32_t)e.tokens.size()))
-            throw InvalidRequestError(is_live(e.id) || !free_slots_.empty() ? "the cache pool has no room for the tokens of request " + e.id
-                                                                            : "no free slot for request " + e.id);
+            throw InvalidRequestError("no cache pages or state slot for request " + e.id);
         PlannedEntry p;
         p.slot = live_.at(e.id).slot;
         p.kv_offset = len;

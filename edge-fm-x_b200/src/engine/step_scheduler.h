@@ -23,8 +23,7 @@ class StepScheduler {
 public:
     // Sequences get the slot numbers first_slot, first_slot + 1, ...; max_live of them at a time.
     StepScheduler(std::shared_ptr<PagedCache> cache, int32_t first_slot, int32_t max_live);
-    // Admits and places every entry of one step, or throws InvalidRequestError (nothing of the step has run then; requests
-    // that were admitted stay admitted with what they held).
+    // Admits and places every entry of one step, or throws InvalidRequestError and changes nothing.
     std::vector<PlannedEntry> plan(const std::vector<StepEntry>& entries);
     // The step has run: the entries' tokens are in the cache.
     void commit(const std::vector<StepEntry>& entries);

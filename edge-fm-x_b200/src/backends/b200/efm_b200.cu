@@ -189,6 +189,7 @@ efm_status efm_b200_prefill(efm_b200_ctx* c, int32_t slot, const int32_t* token_
     if (n_tokens <= 0 || kv_offset < 0) return fail(c, EFM_ERR_INVALID_ARGUMENT, "n_tokens must be > 0 and kv_offset >= 0");
     if ((int64_t)kv_offset + n_tokens > s.max_tokens)
         return fail(c, EFM_ERR_INVALID_ARGUMENT, "prefill exceeds the slot's max_tokens");
+    if (pos_ids3 != nullptr && c->pos3 == nullptr) return fail(c, EFM_ERR_UNSUPPORTED, "this model takes no position ids");
     if (c->d.use_mrope && pos_ids3 == nullptr) return fail(c, EFM_ERR_INVALID_ARGUMENT, "M-RoPE model needs position ids");
     EFM_CK(c, cudaSetDevice(c->device));
     if (c->ops->prefill_begin != nullptr) {
@@ -451,6 +452,7 @@ efm_status efm_b200_launch_count(efm_b200_ctx* c, int64_t* count) {
 
 efm_status efm_b200_decode_breakdown(efm_b200_ctx* c, int32_t n_steps, float* ms_out) {
     if (c == nullptr || ms_out == nullptr) return fail(c, EFM_ERR_INVALID_ARGUMENT, "null argument");
+    if (c->decoder != nullptr) return fail(c, EFM_ERR_UNSUPPORTED, "the breakdown is laid out for the text tower's five kernels per layer");
     if (c->bound_slot < 0) return fail(c, EFM_ERR_STATE, "decode_begin has not been called");
     KvSlot& s = c->slots[c->bound_slot];
     EFM_CK(c, cudaSetDevice(c->device));

@@ -112,12 +112,15 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     for (int i = 0; i < C::HALF; ++i) o[i] = 0.f;
     float m = -INFINITY, l = 0.f;
 
+    int last_k[2] = {-1, -1}, last_v = -1;                       // thread 0: tiles requested last
     auto load_k = [&](int tile, int buf) {
+        last_k[buf] = tile;
         mbar_expect_tx(kfull0 + 8 * buf, C::K_BYTES);
 #pragma unroll
         for (int b = 0; b < C::QB; ++b) tma_load_3d(sK + buf * C::K_BYTES + b * (BN * 128), &map_k, b * 64, g, pages[tile], kfull0 + 8 * buf);
     };
     auto load_v = [&](int tile) {
+        last_v = tile;
         mbar_expect_tx(vfull, C::V_BYTES);
 #pragma unroll
         for (int b = 0; b < C::VB; ++b) tma_load_3d(sV + b * (BN * 128), &map_v, b * 64, g, pages[tile], vfull);
@@ -212,6 +215,13 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
         }
     }
 
+    if (tid == 0 && *abort_s != 0) {                             // given up: let the copies in flight land (bounded) before leaving
+        volatile int go_on = 0;
+        (void)mbar_wait(qfull, 0, &go_on);
+        for (int b = 0; b < 2; ++b)
+            if (last_k[b] >= 0) (void)mbar_wait(kfull0 + 8 * b, (uint32_t)(last_k[b] >> 1) & 1u, &go_on);
+        if (last_v >= 0) (void)mbar_wait(vfull, (uint32_t)last_v & 1u, &go_on);
+    }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();
     xch[hf * BM + row] = l;

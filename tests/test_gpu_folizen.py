@@ -157,7 +157,7 @@ def spotlight(size, heads=4, kv_heads=2, dim=64, vdim=32, scale=0.75):
 
 
 @pytest.mark.parametrize("dtype", ["fp32", "bf16"])
-@pytest.mark.parametrize("size", [64, 65, 72, 128, 200])
+@pytest.mark.parametrize("size", [64, 65, 90, 128, 200])
 def test_window_edge(built, tmp_path, size, dtype):
     cfg, w = spotlight(size)
     wrong = {}

@@ -1,12 +1,14 @@
 // Layered decoders behind the C ABI: context creation, weight ingestion (fused projections, zero-padded rows), the
 // paged cache and the recurrent state slots, batched steps.
 #include <algorithm>
+#include <cmath>
 #include <cstdio>
 #include <cstring>
 
 #include "../../layers/decoder.h"
 #include "../../layers/shared_launch.h"
 #include "../../operators/gemv.cuh"
+#include "../../operators/rotary.cuh"
 #define EFM_DECLARATIONS_ONLY
 #include "../../operators/sample.cuh"
 #undef EFM_DECLARATIONS_ONLY
@@ -26,28 +28,65 @@ efm_status validate(const efm_decoder_desc& d, const efm_decoder_layer* layers) 
         d.max_slots <= 0 || d.cache_pages < 0 || d.state_slots < 0)
         return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, "non-positive decoder dimension");
     if (d.compute_dtype != EFM_BF16 && d.compute_dtype != EFM_F32) return fail(nullptr, EFM_ERR_UNSUPPORTED, "compute_dtype must be bf16 or fp32");
+    if (d.norm_layout != EFM_NORM_OUTPUT && d.norm_layout != EFM_NORM_SANDWICH) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, "unknown norm_layout");
+    if (d.norm_layout == EFM_NORM_SANDWICH && d.side_dim > 0) return fail(nullptr, EFM_ERR_UNSUPPORTED, "a token input behind normalised sublayer inputs");
+    if (d.loop_times < 0 || (d.loop_times > 1 && (d.loop_start < 0 || d.loop_stop <= d.loop_start || d.loop_stop > d.num_layers)))
+        return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, "the looped layers must be a span of the layers");
     for (int i = 0; i < d.num_layers; ++i) {
         const efm_decoder_layer& l = layers[i];
         const std::string at = "layer " + std::to_string(i) + ": ";
-        if (l.heads <= 0 || l.dim <= 0 || l.ff < 0) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "non-positive dimension");
+        if (l.heads <= 0 || l.dim <= 0 || l.ff < 0 || l.experts < 0) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "non-positive dimension");
         if (l.dim > 256) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "dim above 256");
         if (l.mixer == EFM_MIXER_ATTENTION) {
             if (l.kv_heads <= 0 || l.heads % l.kv_heads != 0 || l.vdim <= 0 || l.window < 0)
                 return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "heads must be a multiple of kv_heads, vdim positive, window >= 0");
             if (l.vdim > 256) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "vdim above 256");
+            if (l.keep_first < 0 || (l.qk_norm != EFM_QK_NORM_WEIGHTED && l.qk_norm != EFM_QK_NORM_PLAIN)) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "keep_first or qk_norm");
+            if (l.rot_kind != EFM_ROT_NONE && l.rot_dims > l.dim) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "more rotated channels than dim");
+            if (l.sink || l.out_gate) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "sink and out_gate belong to latent attention");
+        } else if (l.mixer == EFM_MIXER_LATENT_ATTENTION) {
+            if (l.vdim <= 0 || l.window < 0 || l.q_rank <= 0 || l.kv_rank <= 0) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "non-positive dimension");
+            if (l.vdim > 256 || l.kv_rank > 1024) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "vdim above 256 or kv_rank above 1024");
+            if (l.rot_kind == EFM_ROT_NONE) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "latent attention has a rotated part");
+            if (l.keep_first != 0) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "keep_first belongs to attention");
         } else if (l.mixer == EFM_MIXER_GENERAL_DELTA) {
             if (l.decay_rank <= 0) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "decay_rank must be positive");
             if (l.decay_rank > 512) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "decay_rank above 512");
         } else {
             return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "unknown mixer");
         }
+        if (l.rot_kind != EFM_ROT_NONE) {
+            if ((l.rot_kind != EFM_ROT_HALF && l.rot_kind != EFM_ROT_PAIRS) || l.rot_dims <= 0 || l.rot_dims % 2 != 0 || !(l.rot_base > 0.f))
+                return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "rotation needs a kind, an even number of channels and a base");
+            if (l.rot_dims > 2 * kRotMaxPairs) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "more than 256 rotated channels");
+        }
+        if (l.experts > 0) {
+            if (l.ff > 0 || l.expert_ff <= 0 || l.expert_top <= 0 || l.expert_groups <= 0 || l.expert_groups_kept <= 0 ||
+                l.expert_groups_kept > l.expert_groups || l.experts % l.expert_groups != 0 ||
+                l.expert_top > l.experts / l.expert_groups * l.expert_groups_kept)
+                return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "experts: equal groups, some of them kept, with at least expert_top experts");
+            if (l.experts > kMaxExperts || l.expert_top > kMaxExpertTop || l.expert_groups > kMaxExpertGroups)
+                return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "more experts, choices or groups than the router takes");
+        }
     }
     return EFM_OK;
 }
 
-cudaError_t alloc_linear(efm_b200_ctx* c, DecLinear& w, int N, int K) {
-    w.N = N; w.K = K; w.Np = round_up(N, 8); w.Kp = round_up(K, 8);
-    return dev_alloc(c, &w.w, (size_t)w.Np * w.Kp);
+cudaError_t alloc_linear(efm_b200_ctx* c, DecLinear& w, int N, int K, bool bias = false, int pad_k = 8) {
+    w.N = N; w.K = K; w.Np = round_up(N, 8); w.Kp = round_up(K, pad_k);
+    cudaError_t e = dev_alloc(c, &w.w, (size_t)w.Np * w.Kp);
+    if (e == cudaSuccess && bias) e = dev_alloc(c, &w.bias, w.Np);
+    return e;
+}
+
+// base^(-2 i / dims), rounded once
+cudaError_t alloc_inv_freq(efm_b200_ctx* c, DecoderLayer& l) {
+    if (l.d.rot_kind == EFM_ROT_NONE) return cudaSuccess;
+    std::vector<float> f((size_t)l.d.rot_dims / 2);
+    for (size_t i = 0; i < f.size(); ++i) f[i] = (float)std::pow((double)l.d.rot_base, -2.0 * (double)i / l.d.rot_dims);
+    cudaError_t e = dev_alloc(c, &l.inv_freq, f.size());
+    if (e == cudaSuccess) e = cudaStreamSynchronize(c->stream);
+    return e == cudaSuccess ? cudaMemcpy(l.inv_freq, f.data(), f.size() * sizeof(float), cudaMemcpyHostToDevice) : e;
 }
 
 }  // namespace
@@ -95,33 +134,67 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
     EFM_TRY(cudaDeviceGetAttribute(&c->num_sms, cudaDevAttrMultiProcessorCount, device_id));
     EFM_TRY(cudaStreamCreateWithFlags(&c->stream, cudaStreamNonBlocking));
     for (auto& ev : c->events) EFM_TRY(cudaEventCreate(&ev));
-    EFM_TRY(configure_decoder(*m));
     EFM_TRY(configure_sampler());
+    const bool sandwich = desc->norm_layout == EFM_NORM_SANDWICH;
+    for (int i = 0; i < desc->num_layers; ++i) {
+        const int times = desc->loop_times > 1 && i == desc->loop_start ? desc->loop_times : 1;
+        const int stop = times > 1 ? desc->loop_stop : i + 1;
+        for (int t = 0; t < times; ++t)
+            for (int k = i; k < stop; ++k) {
+                DecoderRun r;
+                r.layer = k;
+                m->runs.push_back(r);
+            }
+        i = stop - 1;
+    }
 
     const size_t rows = (size_t)std::max(desc->cache_pages, 1) * EFM_PAGE_TOKENS, es = act_bytes(*m);
-    size_t w_in = 8, w_mix = 8, w_ff = 8, w_q = 8, w_delta_in = 8, n_pack = 8, w_rank = 8, k_max = Wp;
-    bool any_delta = false;
+    size_t w_in = 8, w_mix = 8, w_ff = 8, w_q = 8, w_delta_in = 8, n_pack = 8, w_rank = 8, w_cq = 8, k_max = Wp;
+    size_t ws_c = 0, ws_kv = 0, n_experts = 0, w_route = 8, ex_ff = 0, top = 0, w_act = 8;
+    bool any_delta = false, any_dense = false, ws_full = false;
     m->layers.resize(desc->num_layers);
     for (int i = 0; i < desc->num_layers; ++i) {
         DecoderLayer& l = m->layers[i];
         l.d = layers[i];
         const efm_decoder_layer& d = l.d;
-        EFM_TRY(dev_alloc(c, &l.norm1, Wp));
+        EFM_TRY(dev_alloc(c, &l.post1, Wp));
+        if (sandwich) EFM_TRY(dev_alloc(c, &l.pre1, Wp));
+        EFM_TRY(alloc_inv_freq(c, l));
         if (d.mixer == EFM_MIXER_ATTENTION) {
             l.Dp = round_up(d.dim, 64);
             l.Vp = round_up(d.vdim, 64);
             l.mix_w = d.heads * d.vdim;
-            EFM_TRY(alloc_linear(c, l.in, (d.heads + d.kv_heads) * d.dim + d.kv_heads * d.vdim, m->W));
-            EFM_TRY(dev_alloc(c, &l.q_norm, d.dim));
-            EFM_TRY(dev_alloc(c, &l.k_norm, d.dim));
-            EFM_TRY(dev_alloc(c, &l.temp, d.heads));
-            char *k = nullptr, *v = nullptr;
-            EFM_TRY(dev_alloc(c, &k, rows * d.kv_heads * l.Dp * es));
-            EFM_TRY(dev_alloc(c, &v, rows * d.kv_heads * l.Vp * es));
-            l.k_pool = k;
-            l.v_pool = v;
+            EFM_TRY(alloc_linear(c, l.in, (d.heads + d.kv_heads) * d.dim + d.kv_heads * d.vdim, m->W, d.qkv_bias != 0));
+            if (d.qk_norm == EFM_QK_NORM_WEIGHTED) {
+                EFM_TRY(dev_alloc(c, &l.q_norm, d.dim));
+                EFM_TRY(dev_alloc(c, &l.k_norm, d.dim));
+            }
+            if (d.head_temp) EFM_TRY(dev_alloc(c, &l.temp, d.heads));
             w_q = std::max(w_q, (size_t)d.heads * l.Dp);
             w_in = std::max(w_in, (size_t)l.in.Np);
+        } else if (d.mixer == EFM_MIXER_LATENT_ATTENTION) {
+            l.Dp = round_up(d.dim, 8);
+            l.Vp = round_up(d.vdim, 8);
+            l.Qp = round_up(d.q_rank, 8);
+            l.Lc = round_up(d.kv_rank, 8);
+            l.Rc = round_up(d.rot_dims, 8);
+            l.mix_w = d.heads * d.vdim;
+            EFM_TRY(alloc_linear(c, l.in, l.Qp + l.Lc + l.Rc + (d.out_gate ? d.heads * d.vdim : 0), m->W));
+            EFM_TRY(alloc_linear(c, l.uq, d.heads * (l.Dp + l.Rc), d.q_rank));
+            EFM_TRY(alloc_linear(c, l.ukv, d.heads * (l.Dp + l.Vp), d.kv_rank));
+            EFM_TRY(dev_alloc(c, &l.q_norm, l.Qp));
+            EFM_TRY(dev_alloc(c, &l.k_norm, l.Lc));
+            if (d.sink) EFM_TRY(dev_alloc(c, &l.sink, d.heads));
+            w_q = std::max(w_q, (size_t)l.uq.Np);
+            w_cq = std::max(w_cq, (size_t)l.Qp);
+            w_in = std::max(w_in, (size_t)l.in.Np);
+            k_max = std::max(k_max, (size_t)l.uq.Kp);
+            if (decoder_layer_tc(*m, l)) {
+                ws_c = std::max(ws_c, (size_t)(l.Lc + l.Rc));
+                ws_kv = std::max(ws_kv, (size_t)l.ukv.Np);
+                ws_full = ws_full || d.window == 0;
+                m->ws_window = std::max(m->ws_window, d.window);
+            }
         } else {
             any_delta = true;
             const int HD = d.heads * d.dim;
@@ -131,8 +204,6 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
             EFM_TRY(dev_alloc(c, &l.w0, HD));
             EFM_TRY(dev_alloc(c, &l.a_bias, HD));
             EFM_TRY(dev_alloc(c, &l.mix_norm, HD));
-            l.state_off = m->state_stride;
-            m->state_stride += (size_t)HD * d.dim;
             w_delta_in = std::max(w_delta_in, (size_t)l.in.Np);
             n_pack = std::max(n_pack, decoder_delta_pack_floats(d.heads, d.dim, S, std::min(desc->max_slots, S)));
             w_rank = std::max(w_rank, (size_t)l.w2.Kp);
@@ -140,11 +211,26 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
         l.mix_wp = round_up(l.mix_w, 8);
         w_mix = std::max(w_mix, (size_t)l.mix_wp);
         EFM_TRY(alloc_linear(c, l.out, m->W, l.mix_w));
-        if (d.ff > 0) {
+        if (l.mlp()) {
+            EFM_TRY(dev_alloc(c, &l.post2, Wp));
+            if (sandwich) EFM_TRY(dev_alloc(c, &l.pre2, Wp));
+        }
+        if (l.moe()) {
+            l.ffp = round_up(d.expert_ff, 64);
+            EFM_TRY(alloc_linear(c, l.router, d.experts, m->W));
+            EFM_TRY(alloc_linear(c, l.expert_in, d.experts * 2 * l.ffp, m->W));
+            EFM_TRY(alloc_linear(c, l.expert_out, d.experts * Wp, d.expert_ff, false, 64));
+            n_experts = std::max(n_experts, (size_t)d.experts);
+            w_route = std::max(w_route, (size_t)l.router.Np);
+            ex_ff = std::max(ex_ff, (size_t)l.ffp);
+            top = std::max(top, (size_t)d.expert_top);
+            w_act = std::max(w_act, (size_t)d.expert_top * l.ffp);
+            k_max = std::max(k_max, (size_t)d.expert_top * l.ffp);
+        } else if (d.ff > 0) {
+            any_dense = true;
             EFM_TRY(alloc_linear(c, l.up, d.ff, m->W));
             EFM_TRY(alloc_linear(c, l.down, m->W, d.ff));
             EFM_TRY(dev_alloc(c, &l.act, 4));
-            EFM_TRY(dev_alloc(c, &l.norm2, Wp));
             w_ff = std::max(w_ff, (size_t)l.up.Np);
         }
         if (desc->side_dim > 0) {
@@ -154,10 +240,26 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
         }
         k_max = std::max(k_max, std::max((size_t)l.out.Kp, (size_t)(d.ff > 0 ? l.down.Kp : 0)));
     }
+    EFM_TRY(configure_decoder(*m));
+    for (DecoderRun& r : m->runs) {
+        const DecoderLayer& l = m->layers[r.layer];
+        char *k = nullptr, *v = nullptr;
+        if (l.d.mixer == EFM_MIXER_ATTENTION) {
+            EFM_TRY(dev_alloc(c, &k, rows * l.d.kv_heads * l.Dp * es));
+            EFM_TRY(dev_alloc(c, &v, rows * l.d.kv_heads * l.Vp * es));
+        } else if (l.d.mixer == EFM_MIXER_LATENT_ATTENTION) {
+            EFM_TRY(dev_alloc(c, &k, rows * (l.Lc + l.Rc) * es));
+        } else {
+            r.state_off = m->state_stride;
+            m->state_stride += (size_t)l.d.heads * l.d.dim * l.d.dim;
+        }
+        r.k_pool = k;
+        r.v_pool = v;
+    }
     {   // the longest GEMV input must fit the kernel's shared memory as fp32
         int optin = 0;
         EFM_TRY(cudaDeviceGetAttribute(&optin, cudaDevAttrMaxSharedMemoryPerBlockOptin, device_id));
-        if (std::max(gemv_smem_bytes((int)k_max), gemv_ext_smem_bytes(Wp)) + 2048 > (size_t)optin) {
+        if (std::max(std::max(gemv_smem_bytes((int)k_max), gemv_ext_smem_bytes(Wp)), gemv_ext_smem_bytes((int)w_cq)) + 2048 > (size_t)optin) {
             efm_status s = fail(nullptr, EFM_ERR_UNSUPPORTED, "width / feed-forward size exceeds what the decode GEMV stages in shared memory");
             efm_b200_destroy(c);
             return s;
@@ -182,12 +284,45 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
     };
     EFM_TRY(dev_alloc(c, &c->ids, S));
     EFM_TRY(dev_alloc(c, &c->resid, (size_t)S * Wp));
-    if (!m->f32) EFM_TRY(act(&m->xa, (size_t)S * Wp));
+    if (!m->f32 || sandwich) EFM_TRY(act(&m->xa, (size_t)S * Wp));
+    EFM_TRY(act(&m->cq, S * w_cq));
+    if (ws_c > 0) {
+        // the rows' own pages plus, for every entry long enough, those of a window
+        if (ws_full) m->ws_window = 0;
+        const size_t entries = std::min(desc->max_slots, std::max(1, S / kTcMinRows));
+        size_t pages = (size_t)std::max(desc->cache_pages, 1);
+        if (!ws_full) pages = std::min(pages, (size_t)S / EFM_PAGE_TOKENS + 1 + entries * ((size_t)m->ws_window / EFM_PAGE_TOKENS + 3));
+        m->ws_pages = (int)pages;
+        EFM_TRY(dev_alloc(c, &m->ws_c, pages * EFM_PAGE_TOKENS * ws_c));
+        EFM_TRY(dev_alloc(c, &m->ws_kv, pages * EFM_PAGE_TOKENS * ws_kv));
+    }
+    if (n_experts > 0) {
+        const size_t picks = (size_t)S * top;
+        m->ex_rows = (int)((picks / kExpertTile + std::min(picks, n_experts)) * kExpertTile);
+        EFM_TRY(act(&m->ex_in, (size_t)m->ex_rows * Wp));
+        EFM_TRY(act(&m->ex_act, (size_t)m->ex_rows * ex_ff));
+        if (m->f32) EFM_TRY(dev_alloc(c, &m->ex_gu, (size_t)m->ex_rows * 2 * ex_ff));
+        EFM_TRY(dev_alloc(c, &m->ex_y, (size_t)m->ex_rows * Wp));
+        EFM_TRY(dev_alloc(c, &m->route_logits, S * w_route));
+        EFM_TRY(dev_alloc(c, &m->ex.id, picks));
+        EFM_TRY(dev_alloc(c, &m->ex.weight, picks));
+        EFM_TRY(dev_alloc(c, &m->ex.place, picks));
+        EFM_TRY(dev_alloc(c, &m->ex.count, n_experts));
+        EFM_TRY(dev_alloc(c, &m->ex.tile_expert, (size_t)m->ex_rows / kExpertTile));
+        EFM_TRY(dev_alloc(c, &m->ex.n_tiles, 1));
+        EFM_TRY(dev_alloc(c, &m->d_h, Wp));
+        EFM_TRY(dev_alloc(c, &m->d_route, w_route));
+        EFM_TRY(dev_alloc(c, &m->d_act, w_act));
+        EFM_TRY(dev_alloc(c, &m->d_route_id, top));
+        EFM_TRY(dev_alloc(c, &m->d_route_w, top));
+    }
     EFM_TRY(act(&m->proj_a, S * w_in));
     EFM_TRY(act(&m->q, S * w_q));
     EFM_TRY(act(&m->mix, S * w_mix));
-    EFM_TRY(act(&m->ff, S * w_ff));
-    EFM_TRY(act(&m->ff2, S * w_ff));
+    if (any_dense) {
+        EFM_TRY(act(&m->ff, S * w_ff));
+        EFM_TRY(act(&m->ff2, S * w_ff));
+    }
     EFM_TRY(act(&m->side_a, (size_t)S * m->side_p));
     EFM_TRY(dev_alloc(c, &m->side_f, (size_t)S * m->side_p));
     EFM_TRY(dev_alloc(c, &m->y, (size_t)S * Wp));
@@ -201,13 +336,14 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
     m->max_want = std::min(S, 256);
     EFM_TRY(act(&m->head_a, (size_t)m->max_want * Wp));
     EFM_TRY(dev_alloc(c, &m->logits_rows, (size_t)m->max_want * m->head.Np));
-    // per pass: ids, row entries, wanted rows, two tile lists, entries
-    m->step_words = (size_t)S * 3 + 2 * (size_t)S * 2 + (size_t)S * (sizeof(RowEntry) / 4) + 64;
+    // per pass: ids, row entries, wanted rows, short rows, tile and page lists, entries
+    m->step_words = (size_t)S * 4 + 2 * (size_t)S * 2 + (size_t)m->ws_pages * 2 + (size_t)S * (sizeof(RowEntry) / 4) + 64;
     EFM_TRY(dev_alloc(c, &m->step_buf, m->step_words));
 
     EFM_TRY(dev_alloc(c, &c->resid_d, Wp));
     EFM_TRY(dev_alloc(c, &c->resid_d2, Wp));
     EFM_TRY(dev_alloc(c, &m->d_in, std::max(w_in, w_delta_in)));
+    EFM_TRY(dev_alloc(c, &m->d_q, w_q));
     EFM_TRY(dev_alloc(c, &m->d_mix, w_mix));
     EFM_TRY(dev_alloc(c, &m->d_y, Wp));
     EFM_TRY(dev_alloc(c, &m->d_y2, Wp));
@@ -380,7 +516,8 @@ efm_status efm_b200_decoder_step(efm_b200_ctx* c, const efm_step_entry* entries,
     while (first < n_entries) {
         std::vector<RowEntry> re;
         std::vector<int32_t> ids, row_entry;
-        std::vector<RowTile> tc, simt;
+        std::vector<RowTile> tc, simt, ws;
+        std::vector<int32_t> short_rows;
         struct Want { int32_t row; int64_t idx; uint32_t rng_step; };
         std::vector<Want> wants;
         int rows = 0;
@@ -388,9 +525,16 @@ efm_status efm_b200_decoder_step(efm_b200_ctx* c, const efm_step_entry* entries,
             const efm_step_entry& en = entries[e];
             const int n = std::min(en.n_tokens - done[e], c->max_s - rows);
             KvSlot& s = c->slots.at(en.slot);
-            RowEntry r{rows, n, en.kv_offset + done[e], s.table, s.state_slot};
+            RowEntry r{rows, n, en.kv_offset + done[e], s.table, s.state_slot, 0};
             const int idx = (int)re.size(), step = n >= kTcMinRows ? decoder_tc_tile_rows() : decoder_simt_tile_rows();
             for (int i = 0; i < n; i += step) (n >= kTcMinRows ? tc : simt).push_back(RowTile{idx, i});
+            if (n < kTcMinRows)
+                for (int i = 0; i < n; ++i) short_rows.push_back(rows + i);
+            else if (m.ws_pages > 0) {
+                const int p0 = decoder_ws_page0(m, r.pos0), p1 = (r.pos0 + n - 1) / EFM_PAGE_TOKENS;
+                r.ws0 = ((int)ws.size() - p0) * EFM_PAGE_TOKENS;
+                for (int p = p0; p <= p1; ++p) ws.push_back(RowTile{idx, p});
+            }
             for (int i = 0; i < n; ++i) { ids.push_back(en.tokens[done[e] + i]); row_entry.push_back(idx); }
             for (int i = 0; i < en.n_want; ++i)
                 if (en.want[i] >= done[e] && en.want[i] < done[e] + n) wants.push_back(Want{rows + en.want[i] - done[e], want0[e] + i, en.rng_step});
@@ -401,6 +545,7 @@ efm_status efm_b200_decoder_step(efm_b200_ctx* c, const efm_step_entry* entries,
             if (done[e] == en.n_tokens && e == first) ++first;
         }
         while (first < n_entries && done[first] == entries[first].n_tokens) ++first;
+        if ((int)ws.size() > m.ws_pages) return fail(c, EFM_ERR_STATE, "the entries see more cache pages than the pool has");
         // tiles of the tensor-core form go to the CUDA-core form in layers it does not take: list them in its units too
         std::vector<RowTile> all_simt;
         for (size_t i = 0; i < re.size(); ++i)
@@ -416,7 +561,8 @@ efm_status efm_b200_decoder_step(efm_b200_ctx* c, const efm_step_entry* entries,
         for (const Want& w : wants) want_rows.push_back(w.row);
         const size_t o_ids = put(ids.data(), ids.size()), o_re = put(re.data(), re.size() * sizeof(RowEntry) / 4),
                      o_row = put(row_entry.data(), row_entry.size()), o_tc = put(tc.data(), tc.size() * 2), o_simt = put(simt.data(), simt.size() * 2),
-                     o_all = put(all_simt.data(), all_simt.size() * 2), o_want = put(want_rows.data(), want_rows.size());
+                     o_all = put(all_simt.data(), all_simt.size() * 2), o_want = put(want_rows.data(), want_rows.size()),
+                     o_short = put(short_rows.data(), short_rows.size()), o_ws = put(ws.data(), ws.size() * 2);
         if (pk.size() > m.step_words) {
             EFM_CK(c, cudaStreamSynchronize(c->stream));
             EFM_CK(c, dev_alloc(c, &m.step_buf, pk.size() * 2, false));
@@ -438,6 +584,10 @@ efm_status efm_b200_decoder_step(efm_b200_ctx* c, const efm_step_entry* entries,
         tiles.n_simt = (int)simt.size();
         tiles.all = reinterpret_cast<const RowTile*>(m.step_buf + o_all);
         tiles.n_all = (int)all_simt.size();
+        tiles.short_rows = m.step_buf + o_short;
+        tiles.n_short = (int)short_rows.size();
+        tiles.ws_pages = reinterpret_cast<const RowTile*>(m.step_buf + o_ws);
+        tiles.n_ws = (int)ws.size();
         decoder_rows_pass(*c, plan, m.step_buf + o_ids, tiles, L);
         m.tap_row0 += rows;
         for (size_t w0 = 0; w0 < wants.size(); w0 += (size_t)m.max_want) {
@@ -473,14 +623,14 @@ efm_status efm_b200_decoder_set_taps(efm_b200_ctx* c, int32_t rows) {
     drop_prefill_graphs(c);
     m.tap = nullptr;
     m.tap_rows = rows;
-    if (rows > 0) EFM_CK(c, dev_alloc(c, &m.tap, (size_t)m.d.num_layers * rows * m.Wp));
+    if (rows > 0) EFM_CK(c, dev_alloc(c, &m.tap, m.runs.size() * rows * m.Wp));
     return EFM_OK;
 }
 
 efm_status efm_b200_decoder_read_taps(efm_b200_ctx* c, float* host_out) {
     if (c == nullptr || c->decoder == nullptr || host_out == nullptr || c->decoder->tap == nullptr) return fail(c, EFM_ERR_INVALID_ARGUMENT, "no taps are set");
     DecoderModel& m = *c->decoder;
-    EFM_CK(c, cudaMemcpy2DAsync(host_out, (size_t)m.W * 4, m.tap, (size_t)m.Wp * 4, (size_t)m.W * 4, (size_t)m.d.num_layers * m.tap_rows,
+    EFM_CK(c, cudaMemcpy2DAsync(host_out, (size_t)m.W * 4, m.tap, (size_t)m.Wp * 4, (size_t)m.W * 4, m.runs.size() * m.tap_rows,
                                 cudaMemcpyDeviceToHost, c->stream));
     return ctx_sync(c);
 }
@@ -490,11 +640,17 @@ efm_status efm_b200_decoder_read_taps(efm_b200_ctx* c, float* host_out) {
 namespace {
 
 // ---- weights -------------------------------------------------------------------------------------------------------
-efm_status put_rows(efm_b200_ctx* c, const DecLinear& w, int row0, int rows, const void* data, const std::string& name, const int64_t* shape, int ndim,
-                    int mem_kind) {
+// Rows [src, src + n) of a tensor become rows [dst, dst + n) of a (fused, padded) linear.
+struct Piece { int dst, src, n; };
+
+efm_status put_rows(efm_b200_ctx* c, const DecLinear& w, const std::vector<Piece>& pieces, const void* data, const std::string& name, const int64_t* shape,
+                    int ndim, int mem_kind) {
+    int rows = 0;
+    for (const Piece& p : pieces) rows += p.n;
     if (!shape_is(shape, ndim, rows, w.K)) return fail(c, EFM_ERR_INVALID_ARGUMENT, "unexpected shape for " + name);
-    EFM_CK(c, cudaMemcpy2DAsync(w.w + (size_t)row0 * w.Kp, (size_t)w.Kp * 2, data, (size_t)w.K * 2, (size_t)w.K * 2, (size_t)rows,
-                                mem_kind == EFM_MEM_DEVICE ? cudaMemcpyDeviceToDevice : cudaMemcpyHostToDevice, c->stream));
+    for (const Piece& p : pieces)
+        EFM_CK(c, cudaMemcpy2DAsync(w.w + (size_t)p.dst * w.Kp, (size_t)w.Kp * 2, static_cast<const char*>(data) + (size_t)p.src * w.K * 2, (size_t)w.K * 2,
+                                    (size_t)w.K * 2, (size_t)p.n, mem_kind == EFM_MEM_DEVICE ? cudaMemcpyDeviceToDevice : cudaMemcpyHostToDevice, c->stream));
     return EFM_OK;
 }
 efm_status put_vec(efm_b200_ctx* c, __nv_bfloat16* dst, int n, const void* data, const std::string& name, const int64_t* shape, int ndim, int mem_kind) {
@@ -503,14 +659,26 @@ efm_status put_vec(efm_b200_ctx* c, __nv_bfloat16* dst, int n, const void* data,
 }
 
 // Where a tensor goes: a row range of a (fused) linear or a vector.
-struct Target { DecLinear* lin = nullptr; int row0 = 0, rows = 0; __nv_bfloat16* vec = nullptr; int n = 0; };
+struct Target { DecLinear* lin = nullptr; std::vector<Piece> pieces; __nv_bfloat16* vec = nullptr; int n = 0; };
 
 bool layer_target(DecoderModel& m, DecoderLayer& l, const std::string& rest, Target* t) {
     const efm_decoder_layer& d = l.d;
-    auto lin = [&](DecLinear& w, int row0, int rows) { t->lin = &w; t->row0 = row0; t->rows = rows; return true; };
+    auto lin = [&](DecLinear& w, int row0, int rows) { t->lin = &w; t->pieces.push_back(Piece{row0, 0, rows}); return true; };
     auto vec = [&](__nv_bfloat16* v, int n) { t->vec = v; t->n = n; return v != nullptr; };
-    if (rest == "norm1") return vec(l.norm1, m.W);
-    if (rest == "norm2") return vec(l.norm2, m.W);
+    // heads of `n` rows, laid out from row0 on with `ld` rows each, `gap` more behind the first `cut` rows
+    auto heads = [&](DecLinear& w, int row0, int ld, int n, int cut, int gap) {
+        t->lin = &w;
+        for (int h = 0; h < d.heads; ++h) {
+            t->pieces.push_back(Piece{row0 + h * ld, h * n, cut});
+            if (n > cut) t->pieces.push_back(Piece{row0 + h * ld + cut + gap, h * n + cut, n - cut});
+        }
+        return true;
+    };
+    const bool sandwich = m.d.norm_layout == EFM_NORM_SANDWICH;
+    if (rest == "norm1") return vec(sandwich ? l.pre1 : l.post1, m.W);
+    if (rest == "norm2") return vec(sandwich ? l.pre2 : l.post2, m.W);
+    if (sandwich && rest == "norm1b") return vec(l.post1, m.W);
+    if (sandwich && rest == "norm2b") return vec(l.post2, m.W);
     if (rest == "mix.o") return lin(l.out, 0, m.W);
     if (d.mixer == EFM_MIXER_ATTENTION) {
         const int q = d.heads * d.dim, k = d.kv_heads * d.dim;
@@ -520,6 +688,25 @@ bool layer_target(DecoderModel& m, DecoderLayer& l, const std::string& rest, Tar
         if (rest == "mix.q.norm") return vec(l.q_norm, d.dim);
         if (rest == "mix.k.norm") return vec(l.k_norm, d.dim);
         if (rest == "mix.temp") return vec(l.temp, d.heads);
+        if (d.qkv_bias) {
+            if (rest == "mix.q.b") return vec(l.in.bias, q);
+            if (rest == "mix.k.b") return vec(l.in.bias + q, k);
+            if (rest == "mix.v.b") return vec(l.in.bias + q + k, d.kv_heads * d.vdim);
+        }
+    } else if (d.mixer == EFM_MIXER_LATENT_ATTENTION) {
+        if (rest == "mix.dq") return lin(l.in, 0, d.q_rank);
+        if (rest == "mix.dkv") {
+            lin(l.in, l.Qp, d.kv_rank);
+            t->pieces.push_back(Piece{l.Qp + l.Lc, d.kv_rank, d.rot_dims});
+            return true;
+        }
+        if (rest == "mix.g" && d.out_gate) return lin(l.in, l.Qp + l.Lc + l.Rc, d.heads * d.vdim);
+        if (rest == "mix.uq") return heads(l.uq, 0, l.Dp + l.Rc, d.dim + d.rot_dims, d.dim, l.Dp - d.dim);
+        if (rest == "mix.uk") return heads(l.ukv, 0, l.Dp, d.dim, d.dim, 0);
+        if (rest == "mix.uv") return heads(l.ukv, d.heads * l.Dp, l.Vp, d.vdim, d.vdim, 0);
+        if (rest == "mix.dq.norm") return vec(l.q_norm, d.q_rank);
+        if (rest == "mix.dkv.norm") return vec(l.k_norm, d.kv_rank);
+        if (rest == "mix.sink") return vec(l.sink, d.heads);
     } else {
         const int HD = d.heads * d.dim;
         static const char* seg[5] = {"mix.r", "mix.k", "mix.v", "mix.g", "mix.a"};
@@ -531,7 +718,21 @@ bool layer_target(DecoderModel& m, DecoderLayer& l, const std::string& rest, Tar
         if (rest == "mix.a.b") return vec(l.a_bias, HD);
         if (rest == "mix.norm") return vec(l.mix_norm, HD);
     }
-    if (d.ff > 0) {
+    if (l.moe()) {
+        if (rest == "mlp.router") return lin(l.router, 0, d.experts);
+        const size_t dot = rest.find('.', 5);
+        if (rest.compare(0, 5, "mlp.e") == 0 && dot != std::string::npos && dot > 5) {
+            const int e = std::atoi(rest.c_str() + 5);
+            const std::string what = rest.substr(dot + 1);
+            if (rest.substr(5, dot - 5) != std::to_string(e) || e >= d.experts) return false;
+            if (what == "down") return lin(l.expert_out, e * m.Wp, m.W);
+            if (what != "gate" && what != "up") return false;
+            t->lin = &l.expert_in;                     // 64 gate rows, the 64 matching up rows, ...
+            for (int r = 0; r < d.expert_ff; r += 64)
+                t->pieces.push_back(Piece{e * 2 * l.ffp + 2 * r + (what == "up" ? 64 : 0), r, std::min(64, d.expert_ff - r)});
+            return true;
+        }
+    } else if (d.ff > 0) {
         if (rest == "mlp.up") return lin(l.up, 0, d.ff);
         if (rest == "mlp.down") return lin(l.down, 0, m.W);
         if (rest == "mlp.act") return vec(l.act, 4);
@@ -549,12 +750,12 @@ efm_status decoder_set_weight(efm_b200_ctx* c, const char* raw, const void* data
     const std::string name(raw);
     Target t;
     DecLinear table;                       // plain row tables share the padded copy
-    if (name == "embed") { table.w = c->embed; table.K = m.W; table.Kp = m.Wp; t.lin = &table; t.rows = m.d.vocab; }
+    if (name == "embed") { table.w = c->embed; table.K = m.W; table.Kp = m.Wp; t.lin = &table; t.pieces.push_back(Piece{0, 0, m.d.vocab}); }
     else if (name == "side.embed" && m.side_embed != nullptr) {
         table.w = m.side_embed; table.K = table.Kp = m.d.side_dim * m.d.num_layers;
-        t.lin = &table; t.rows = m.d.vocab;
+        t.lin = &table; t.pieces.push_back(Piece{0, 0, m.d.vocab});
     }
-    else if (name == "head") { t.lin = &m.head; t.rows = m.d.vocab; }
+    else if (name == "head") { t.lin = &m.head; t.pieces.push_back(Piece{0, 0, m.d.vocab}); }
     else if (name == "final.norm") { t.vec = m.final_norm; t.n = m.W; }
     else if (name.size() > 1 && name[0] == 'l' && name[1] >= '0' && name[1] <= '9') {
         const size_t dot = name.find('.');
@@ -564,7 +765,7 @@ efm_status decoder_set_weight(efm_b200_ctx* c, const char* raw, const void* data
         return EFM_OK;                     // not part of this model
     }
     if (dtype != EFM_BF16) return fail(c, EFM_ERR_UNSUPPORTED, "weights must be bf16: " + name);
-    const efm_status st = t.lin != nullptr ? put_rows(c, *t.lin, t.row0, t.rows, data, name, shape, ndim, mem_kind)
+    const efm_status st = t.lin != nullptr ? put_rows(c, *t.lin, t.pieces, data, name, shape, ndim, mem_kind)
                                            : put_vec(c, t.vec, t.n, data, name, shape, ndim, mem_kind);
     if (st != EFM_OK) return st;
     EFM_CK(c, cudaStreamSynchronize(c->stream));          // the caller may release `data` on return
@@ -580,9 +781,28 @@ efm_status decoder_finalize(efm_b200_ctx* c) {
         const efm_decoder_layer& d = m.layers[i].d;
         auto add = [&](std::initializer_list<const char*> names) { for (const char* n : names) need.push_back("l" + std::to_string(i) + "." + n); };
         add({"norm1", "mix.o"});
-        if (d.mixer == EFM_MIXER_ATTENTION) add({"mix.q", "mix.k", "mix.v", "mix.q.norm", "mix.k.norm", "mix.temp"});
-        else add({"mix.r", "mix.k", "mix.v", "mix.g", "mix.a", "mix.a.b", "mix.w1", "mix.w2", "mix.w0", "mix.norm"});
-        if (d.ff > 0) add({"norm2", "mlp.up", "mlp.down", "mlp.act"});
+        if (m.d.norm_layout == EFM_NORM_SANDWICH) add({"norm1b"});
+        if (d.mixer == EFM_MIXER_ATTENTION) {
+            add({"mix.q", "mix.k", "mix.v"});
+            if (d.qk_norm == EFM_QK_NORM_WEIGHTED) add({"mix.q.norm", "mix.k.norm"});
+            if (d.head_temp) add({"mix.temp"});
+            if (d.qkv_bias) add({"mix.q.b", "mix.k.b", "mix.v.b"});
+        } else if (d.mixer == EFM_MIXER_LATENT_ATTENTION) {
+            add({"mix.dq", "mix.dq.norm", "mix.uq", "mix.dkv", "mix.dkv.norm", "mix.uk", "mix.uv"});
+            if (d.sink) add({"mix.sink"});
+            if (d.out_gate) add({"mix.g"});
+        } else add({"mix.r", "mix.k", "mix.v", "mix.g", "mix.a", "mix.a.b", "mix.w1", "mix.w2", "mix.w0", "mix.norm"});
+        if (d.experts > 0 || d.ff > 0) {
+            add({"norm2"});
+            if (m.d.norm_layout == EFM_NORM_SANDWICH) add({"norm2b"});
+        }
+        if (d.experts > 0) {
+            add({"mlp.router"});
+            for (int e = 0; e < d.experts; ++e)
+                for (const char* what : {".gate", ".up", ".down"}) add({("mlp.e" + std::to_string(e) + what).c_str()});
+        } else if (d.ff > 0) {
+            add({"mlp.up", "mlp.down", "mlp.act"});
+        }
         if (m.d.side_dim > 0) add({"side.gate", "side.proj", "side.norm"});
     }
     for (const std::string& n : need)
@@ -612,12 +832,18 @@ efm_status decoder_decode_begin(efm_b200_ctx* c, KvSlot& s, int kv_len) {
 void decoder_prefill_chunk(efm_b200_ctx& c, KvSlot& slot, int S, int kv_offset, int, int, bool sample_last, Launcher& L) {
     DecoderModel& m = *c.decoder;
     RowPlan plan{};
-    plan.one = RowEntry{0, S, kv_offset, slot.table, slot.state_slot};
+    plan.one = RowEntry{0, S, kv_offset, slot.table, slot.state_slot, 0};
+    RowTiles tiles;
+    if (m.ws_pages > 0) {
+        tiles.ws_page0 = decoder_ws_page0(m, kv_offset);
+        tiles.n_ws = (kv_offset + S - 1) / EFM_PAGE_TOKENS - tiles.ws_page0 + 1;
+        plan.one.ws0 = -tiles.ws_page0 * EFM_PAGE_TOKENS;
+    }
     plan.page_table = m.page_table;
     plan.max_pages = m.d.cache_pages;
     plan.n_entries = 1;
     plan.rows = S;
-    decoder_rows_pass(c, plan, c.ids, RowTiles{}, L);
+    decoder_rows_pass(c, plan, c.ids, tiles, L);
     if (sample_last && L.err == cudaSuccess) L.err = cudaErrorNotSupported;     // a sampled prefill ends with a decode step
 }
 void decoder_step_op(efm_b200_ctx& c, KvSlot& slot, Launcher& L) { decoder_decode_step(c, slot, L, true, true); }
@@ -626,14 +852,14 @@ int64_t decoder_step_bytes(const efm_b200_ctx& c, int32_t kv_len) {
     const DecoderModel& m = *c.decoder;
     auto lin = [](const DecLinear& w) { return (int64_t)w.N * w.K * 2; };
     int64_t b = lin(m.head) + (int64_t)m.W * 2 * 2;
-    for (const DecoderLayer& l : m.layers) {
-        b += lin(l.in) + lin(l.out) + lin(l.w2) + lin(l.up) + lin(l.down) + lin(l.gate) + lin(l.proj);
-        if (l.d.mixer == EFM_MIXER_ATTENTION) {
-            const int64_t n = l.d.window > 0 ? std::min(kv_len, l.d.window) : kv_len;
-            b += n * l.d.kv_heads * (l.d.dim + l.d.vdim) * (m.f32 ? 4 : 2);
-        } else {
-            b += 2 * (int64_t)l.d.heads * l.d.dim * l.d.dim * 4;
-        }
+    for (const DecoderRun& r : m.runs) {
+        const DecoderLayer& l = m.layers[r.layer];
+        b += lin(l.in) + lin(l.out) + lin(l.w2) + lin(l.up) + lin(l.down) + lin(l.gate) + lin(l.proj) + lin(l.uq) + lin(l.ukv) + lin(l.router);
+        if (l.moe()) b += (int64_t)l.d.expert_top * 3 * l.d.expert_ff * m.W * 2;
+        const int64_t n = l.d.window > 0 ? std::min(kv_len, l.d.window + l.d.keep_first) : kv_len;
+        if (l.d.mixer == EFM_MIXER_ATTENTION) b += n * l.d.kv_heads * (l.d.dim + l.d.vdim) * (m.f32 ? 4 : 2);
+        else if (l.d.mixer == EFM_MIXER_LATENT_ATTENTION) b += n * (l.d.kv_rank + l.d.rot_dims) * (m.f32 ? 4 : 2);
+        else b += 2 * (int64_t)l.d.heads * l.d.dim * l.d.dim * 4;
     }
     return b;
 }

@@ -4,6 +4,11 @@
 // Folizen: "layers" lists {type, mixer, mlp}; type "attention" {heads, kv_heads, dim, vdim, scale, mask.size} or
 // "general_delta" {heads, dim}; mlp null or {kind: "dense", ff}; "norm.eps", "token_side.dim", "vocab", "width".  Sizes
 // the JSON does not give (rank of the decay projection) are read from the tensors' shapes.
+//
+// Temuvik: "layers" lists {type, mixer, mlp}; type "attention" {heads, kv_heads, dim, vdim, scale, rot {base, dims},
+// mask {size, keep_first}} or "latent_attention" {heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, rot {base, dims},
+// mask {size}}; mlp null or {kind: "moe", expert.ff, router {experts, top, groups {count, keep}}}; "norm.eps",
+// "embedding.scale", "loop" {start, stop, times}, "vocab", "width".
 #include <efm_b200.h>
 
 #include <algorithm>
@@ -34,17 +39,39 @@ int32_t positive(const json::Value& v, const char* key, const std::string& where
     return (int32_t)(m.is_int ? m.inum : (int64_t)m.num);
 }
 
-DecoderConfig folizen_config(const json::Value& cfg, const Shapes& shapes) {
-    DecoderConfig out;
-    efm_decoder_desc& d = out.desc;
+float number(const json::Value& v, const char* key, const std::string& where) {
+    const json::Value& m = member(v, key, where);
+    if (!m.is_number()) throw ConfigurationError("config.json: " + where + "." + key + " must be a number");
+    return (float)m.num;
+}
+int32_t whole(const json::Value& v, const char* key, const std::string& where) {
+    const json::Value& m = member(v, key, where);
+    if (!m.is_number() || m.num < 0) throw ConfigurationError("config.json: " + where + "." + key + " must be a number, zero or more");
+    return (int32_t)(m.is_int ? m.inum : (int64_t)m.num);
+}
+bool given(const json::Value* v) { return v != nullptr && v->is_object(); }
+
+// What the layered decoders' configurations share.
+void read_model(const json::Value& cfg, efm_decoder_desc& d) {
     d.struct_size = (int32_t)sizeof(d);
     d.vocab = positive(cfg, "vocab", "model");
     d.width = positive(cfg, "width", "model");
     d.norm_eps = (float)member(member(cfg, "norm", "model"), "eps", "norm").num;
-    const json::Value* side = cfg.find("token_side");
-    if (side != nullptr && side->is_object()) d.side_dim = positive(*side, "dim", "token_side");
+    d.embed_scale = 1.0f;
+}
+const json::Value& layer_list(const json::Value& cfg) {
     const json::Value& layers = member(cfg, "layers", "model");
     if (!layers.is_array() || layers.arr.empty()) throw ConfigurationError("config.json: \"layers\" must be a non-empty list");
+    return layers;
+}
+
+DecoderConfig folizen_config(const json::Value& cfg, const Shapes& shapes) {
+    DecoderConfig out;
+    efm_decoder_desc& d = out.desc;
+    read_model(cfg, d);
+    const json::Value* side = cfg.find("token_side");
+    if (side != nullptr && side->is_object()) d.side_dim = positive(*side, "dim", "token_side");
+    const json::Value& layers = layer_list(cfg);
     for (size_t i = 0; i < layers.arr.size(); ++i) {
         const json::Value& l = layers.arr[i];
         const std::string where = "layers[" + std::to_string(i) + "]";
@@ -59,6 +86,7 @@ DecoderConfig folizen_config(const json::Value& cfg, const Shapes& shapes) {
             e.vdim = positive(mix, "vdim", where + ".mixer");
             e.scale = (float)member(mix, "scale", where + ".mixer").num;
             e.distance_bias = 1;
+            e.head_temp = 1;
             const json::Value* mask = mix.find("mask");
             if (mask != nullptr && mask->is_object()) e.window = positive(*mask, "size", where + ".mixer.mask");
         } else if (type == "general_delta") {
@@ -78,6 +106,80 @@ DecoderConfig folizen_config(const json::Value& cfg, const Shapes& shapes) {
         out.layers.push_back(e);
     }
     d.num_layers = (int32_t)out.layers.size();
+    return out;
+}
+
+void read_rotation(const json::Value& mix, int32_t kind, const std::string& where, efm_decoder_layer& e) {
+    const json::Value& rot = member(mix, "rot", where);
+    e.rot_kind = kind;
+    e.rot_dims = positive(rot, "dims", where + ".rot");
+    e.rot_base = number(rot, "base", where + ".rot");
+}
+
+void read_experts(const json::Value& mlp, const std::string& where, efm_decoder_layer& e) {
+    const std::string kind = mlp.get_string("kind", "");
+    if (kind != "moe") throw ConfigurationError("config.json: " + where + " has an unknown kind \"" + kind + "\"");
+    e.expert_ff = positive(member(mlp, "expert", where), "ff", where + ".expert");
+    const json::Value& router = member(mlp, "router", where);
+    e.experts = positive(router, "experts", where + ".router");
+    e.expert_top = positive(router, "top", where + ".router");
+    e.expert_groups = e.expert_groups_kept = 1;
+    const json::Value* groups = router.find("groups");
+    if (given(groups)) {
+        e.expert_groups = positive(*groups, "count", where + ".router.groups");
+        e.expert_groups_kept = positive(*groups, "keep", where + ".router.groups");
+    }
+}
+
+DecoderConfig temuvik_config(const json::Value& cfg, const Shapes&) {
+    DecoderConfig out;
+    efm_decoder_desc& d = out.desc;
+    read_model(cfg, d);
+    d.norm_layout = EFM_NORM_SANDWICH;
+    d.embed_scale = number(member(cfg, "embedding", "model"), "scale", "embedding");
+    const json::Value& layers = layer_list(cfg);
+    for (size_t i = 0; i < layers.arr.size(); ++i) {
+        const json::Value& l = layers.arr[i];
+        const std::string where = "layers[" + std::to_string(i) + "]", in = where + ".mixer";
+        const json::Value& mix = member(l, "mixer", where);
+        const std::string type = l.get_string("type", "");
+        efm_decoder_layer e{};
+        e.heads = positive(mix, "heads", in);
+        e.dim = positive(mix, "dim", in);
+        e.vdim = positive(mix, "vdim", in);
+        e.scale = number(mix, "scale", in);
+        const json::Value* mask = mix.find("mask");
+        if (given(mask)) e.window = positive(*mask, "size", in + ".mask");
+        if (type == "attention") {
+            e.mixer = EFM_MIXER_ATTENTION;
+            e.kv_heads = positive(mix, "kv_heads", in);
+            e.qk_norm = EFM_QK_NORM_PLAIN;
+            e.qkv_bias = 1;
+            if (given(mask) && mask->find("keep_first") != nullptr) e.keep_first = whole(*mask, "keep_first", in + ".mask");
+            read_rotation(mix, EFM_ROT_HALF, in, e);
+        } else if (type == "latent_attention") {
+            e.mixer = EFM_MIXER_LATENT_ATTENTION;
+            e.q_rank = positive(mix, "q_rank", in);
+            e.kv_rank = positive(mix, "kv_rank", in);
+            e.sink = 1;
+            e.out_gate = 1;
+            read_rotation(mix, EFM_ROT_PAIRS, in, e);
+            if (positive(mix, "rot_dim", in) != e.rot_dims) throw ConfigurationError("config.json: " + in + ".rot.dims must be rot_dim");
+        } else {
+            throw ConfigurationError("config.json: " + where + " has an unknown type \"" + type + "\"");
+        }
+        const json::Value* mlp = l.find("mlp");
+        if (given(mlp)) read_experts(*mlp, where + ".mlp", e);
+        out.layers.push_back(e);
+    }
+    d.num_layers = (int32_t)out.layers.size();
+    const json::Value* loop = cfg.find("loop");
+    if (given(loop)) {
+        d.loop_start = whole(*loop, "start", "loop");
+        d.loop_stop = whole(*loop, "stop", "loop");
+        d.loop_times = positive(*loop, "times", "loop");
+        if (d.loop_stop <= d.loop_start || d.loop_stop > d.num_layers) throw ConfigurationError("config.json: loop.start .. loop.stop must be a span of the layers");
+    }
     return out;
 }
 
@@ -151,7 +253,7 @@ ModelSetup build_decoder(const EngineConfig& config, DecoderConfig (*read)(const
         states += 1 + (r.prefix_token_ids.empty() ? 0 : 1);
     }
     if (pages <= 0) throw ConfigurationError("kvcache declares neither requests nor pool_tokens");
-    const bool recurrent = std::any_of(dc.layers.begin(), dc.layers.end(), [](const efm_decoder_layer& l) { return l.mixer != EFM_MIXER_ATTENTION; });
+    const bool recurrent = std::any_of(dc.layers.begin(), dc.layers.end(), [](const efm_decoder_layer& l) { return l.mixer == EFM_MIXER_GENERAL_DELTA; });
     d.cache_pages = (int32_t)pages;
     d.state_slots = recurrent ? states : 0;
     d.max_slots = (int32_t)reqs.size() + live;
@@ -185,8 +287,12 @@ ModelSetup build_decoder(const EngineConfig& config, DecoderConfig (*read)(const
         KVGeometry geo;
         geo.paged = true;
         geo.dtype = cache_dtype;
-        for (const efm_decoder_layer& l : dc.layers)
-            if (l.mixer == EFM_MIXER_ATTENTION) geo.token_bytes += (size_t)l.kv_heads * (l.dim + l.vdim) * get_dtype_size(cache_dtype);
+        for (int32_t i = 0; i < d.num_layers; ++i) {
+            const efm_decoder_layer& l = dc.layers[i];
+            const size_t times = d.loop_times > 1 && i >= d.loop_start && i < d.loop_stop ? d.loop_times : 1;
+            if (l.mixer == EFM_MIXER_ATTENTION) geo.token_bytes += times * l.kv_heads * (l.dim + l.vdim) * get_dtype_size(cache_dtype);
+            if (l.mixer == EFM_MIXER_LATENT_ATTENTION) geo.token_bytes += times * (l.kv_rank + l.rot_dims) * get_dtype_size(cache_dtype);
+        }
         setup.kv_manager = std::make_shared<KVManager>(reqs, geo, attention_type_from_string(config.kvcache_attention_type()), setup.device_id,
                                                        std::make_shared<PagedKVAllocator>(setup.paged_cache));
     } catch (...) {
@@ -198,7 +304,10 @@ ModelSetup build_decoder(const EngineConfig& config, DecoderConfig (*read)(const
 
 ModelSetup build_folizen(const EngineConfig& config) { return build_decoder(config, folizen_config); }
 
+ModelSetup build_temuvik(const EngineConfig& config) { return build_decoder(config, temuvik_config); }
+
 const ModelRegistrar kFolizen({"folizen", {"Folizen"}, build_folizen});
+const ModelRegistrar kTemuvik({"temuvik", {"Temuvik"}, build_temuvik});
 
 }  // namespace
 

@@ -1,9 +1,10 @@
 // Launch sequences of the layered decoders.
 //
-// Decode (one row), per layer:  [pending output norm + residual add] + input projections | mixer (norms, cache / state
-// update, attention or recurrence) | W_o | [norm1 + add] + W_up | [PolyNorm] + W_down | [norm2 + add] + token
-// input; what stands in brackets is the prologue of the kernel that follows it: four launches for a layer without a
-// feed-forward, six with one.
+// Decode (one row), per layer:  [pending output norm + residual add (+ input norm)] + input projections | mixer (norms,
+// cache / state update, attention or recurrence) | W_o | [norm + add] + W_up | [PolyNorm] + W_down | [norm + add] + token
+// input; what stands in brackets is the prologue of the kernel that follows it: three launches for a layer without a
+// feed-forward and token input, two more for a dense feed-forward, one more for the token input.  Latent attention adds
+// [query norm] + W_uq; routed experts are [norms + add] + router | [choice] + gate, up, silu | [weights] + down.
 // Many rows: tensor-core GEMMs (bf16 operands) or fp32 FMAs (32-bit mode) between row kernels.
 #include "decoder.h"
 
@@ -13,7 +14,9 @@
 #include "../operators/decoder_rows.cuh"
 #include "../operators/delta_chunk.cuh"
 #include "../operators/delta_rule.cuh"
+#include "../operators/experts.cuh"
 #include "../operators/gemm_tc.cuh"
+#include "../operators/latent_attention.cuh"
 #include "../operators/token_side.cuh"
 #include "../operators/window_attention.cuh"
 #include "../operators/window_attention_tc.cuh"
@@ -38,6 +41,16 @@ struct Pending {
 };
 
 template <Epi EPI>
+void launch_gemv_ext(efm_b200_ctx& c, Launcher& L, const GemvParams& p) {
+    const int ks = plan_gemv_ksplit(p.n_items, p.K, c.num_sms);
+    // Logits publishes one maximum per block of a full grid; the others launch no idle blocks
+    const int per = kGemvWarps / ks, need = (p.n_items + per - 1) / per;
+    const int grid = EPI == Epi::Logits ? c.num_sms : std::min(c.num_sms, need);
+    const size_t smem = p.prologue == kProAddNorm || p.prologue == kProNorm ? gemv_ext_smem_bytes(p.K) : gemv_smem_bytes(p.K);
+    L.launch(gemv_kernel<EPI, true>, dim3(grid), dim3(kGemvThreads), smem, p, ks);
+}
+
+template <Epi EPI>
 void gemv_ext(efm_b200_ctx& c, Launcher& L, const DecLinear& w, GemvParams& p) {
     p.W = w.w;
     p.N = w.N;
@@ -46,21 +59,20 @@ void gemv_ext(efm_b200_ctx& c, Launcher& L, const DecLinear& w, GemvParams& p) {
     p.eps = c.decoder->d.norm_eps;
     p.state = c.state;
     p.vocab = c.d.vocab;
-    const int ks = plan_gemv_ksplit(p.n_items, p.K, c.num_sms);
-    // Logits publishes one maximum per block of a full grid; the others launch no idle blocks
-    const int per = kGemvWarps / ks, need = (p.n_items + per - 1) / per;
-    const int grid = EPI == Epi::Logits ? c.num_sms : std::min(c.num_sms, need);
-    const size_t smem = p.prologue == kProAddNorm ? gemv_ext_smem_bytes(p.K) : gemv_smem_bytes(p.K);
-    L.launch(gemv_kernel<EPI, true>, dim3(grid), dim3(kGemvThreads), smem, p, ks);
+    p.bias = w.bias;
+    launch_gemv_ext<EPI>(c, L, p);
 }
 
-// Input of a product that reads the residual stream: embedding row (first layer) or stream + pending output.
-void stream_input(efm_b200_ctx& c, GemvParams& p, Pending& pend, bool first) {
+// Input of a product that reads the residual stream: embedding row (first layer) or stream + pending output; with `pre` the
+// product reads the norm of it.
+void stream_input(efm_b200_ctx& c, GemvParams& p, Pending& pend, bool first, const __nv_bfloat16* pre) {
     float* bufs[2] = {c.resid_d, c.resid_d2};
     p.k_true = c.decoder->W;
+    p.norm2_w = pre;
     if (first) {
         p.prologue = kProEmbed;
         p.embed_table = c.embed;
+        p.embed_scale = c.decoder->d.embed_scale;
         p.resid_out = bufs[pend.flip];
         return;
     }
@@ -74,13 +86,31 @@ void stream_input(efm_b200_ctx& c, GemvParams& p, Pending& pend, bool first) {
     pend.y = nullptr;
 }
 
+RotShape rot_shape(const DecoderLayer& l) {
+    const int kind = l.d.rot_kind == EFM_ROT_HALF ? kRotHalf : l.d.rot_kind == EFM_ROT_PAIRS ? kRotPairs : kRotNone;
+    return RotShape{kind, kind == kRotNone ? 0 : l.d.rot_dims, l.inv_freq};
+}
 WindowAttnShape attn_shape(const DecoderModel& m, const DecoderLayer& l) {
     WindowAttnShape s{};
     s.H = l.d.heads; s.G = l.d.kv_heads; s.D = l.d.dim; s.Dv = l.d.vdim; s.Dp = l.Dp; s.Vp = l.Vp;
-    s.window = l.d.window; s.bias = l.d.distance_bias; s.scale = l.d.scale; s.eps = m.d.norm_eps;
+    s.window = l.d.window; s.keep = l.d.window > 0 ? l.d.keep_first : 0;
+    s.bias = l.d.distance_bias; s.scale = l.d.scale; s.eps = m.d.norm_eps;
     s.q_norm = l.q_norm; s.k_norm = l.k_norm; s.temp = l.temp;
+    s.rot = rot_shape(l);
     return s;
 }
+LatentShape latent_shape(const DecoderModel& m, const DecoderLayer& l) {
+    LatentShape s{};
+    s.H = l.d.heads; s.D = l.d.dim; s.R = l.d.rot_dims; s.Dv = l.d.vdim; s.L = l.d.kv_rank;
+    s.Dp = l.Dp; s.Vp = l.Vp; s.Qp = l.Qp; s.Lc = l.Lc; s.Rc = l.Rc;
+    s.q_rank = l.d.q_rank; s.window = l.d.window; s.scale = l.d.scale; s.eps = m.d.norm_eps;
+    s.rot = rot_shape(l);
+    s.q_norm = l.q_norm; s.kv_norm = l.k_norm; s.sink = l.sink;
+    s.wk = l.ukv.w; s.wv = l.ukv.w + (size_t)l.d.heads * l.Dp * l.Lc;
+    s.gate = l.d.out_gate;
+    return s;
+}
+RouteShape route_shape(const DecoderLayer& l) { return RouteShape{l.d.experts, l.d.expert_top, l.d.expert_groups, l.d.expert_groups_kept}; }
 DeltaShape delta_shape(const DecoderModel& m, const DecoderLayer& l) {
     DeltaShape s{};
     s.heads = l.d.heads; s.D = l.d.dim; s.Dp = round_up(l.d.dim, 32); s.rank = l.d.decay_rank; s.ld = l.in.Np;
@@ -95,13 +125,13 @@ void launch_attn_decode_v(Launcher& L, const WindowDecodeParams<TC>& p, int clus
     L.launch(window_attention_decode_kernel<TC, VM>, dim3(cluster, p.s.G * hb), dim3(wd::kThreads), sizeof(wd::Smem<VM>), p);
 }
 template <typename TC>
-void launch_attn_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const KvSlot& slot, bool early) {
+void launch_attn_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const KvSlot& slot, bool early) {
     DecoderModel& m = *c.decoder;
     WindowDecodeParams<TC> p{};
     p.s = attn_shape(m, l);
     p.qkv = m.d_in;
-    p.k_pool = static_cast<TC*>(l.k_pool);
-    p.v_pool = static_cast<TC*>(l.v_pool);
+    p.k_pool = static_cast<TC*>(run.k_pool);
+    p.v_pool = static_cast<TC*>(run.v_pool);
     p.pages = m.page_table + (size_t)slot.table * m.d.cache_pages;
     p.max_pages = slot.n_pages;
     p.state = c.state;
@@ -109,7 +139,7 @@ void launch_attn_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, con
     p.early = early ? 1 : 0;
     // one block per 64 keys of the visible range, up to the cluster width (a power of two)
     int pages = slot.n_pages;
-    if (l.d.window > 0) pages = std::min(pages, (l.d.window + kPageTokens - 1) / kPageTokens);
+    if (l.d.window > 0) pages = std::min(pages, (l.d.window + p.s.keep + kPageTokens - 1) / kPageTokens);
     int cluster = 1;
     while (cluster < pages && cluster < m.attn_cluster) cluster *= 2;
     const int v = std::max(l.Dp, l.Vp);
@@ -118,14 +148,77 @@ void launch_attn_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, con
     else launch_attn_decode_v<TC, 256>(L, p, cluster);
 }
 
-void launch_delta_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const KvSlot& slot, bool early) {
+// ---- latent attention, absorbed form: a decode step, or rows of a pass ---------------------------------------------------
+// keys per tile that the block's shared memory takes next to everything else
+int latent_tile(const LatentShape& s, int nh, int splits, int es) {
+    int kt = 64;
+    while (kt > 8 && la::layout(s, nh, splits, es, kt).bytes > 200u * 1024u) kt /= 2;
+    return kt;
+}
+// blocks that share a row: one per 64 visible keys or 64 latent channels, a power of two
+int latent_splits(const DecoderLayer& l, int pages, int limit) {
+    if (l.d.window > 0) pages = std::min(pages, (l.d.window + kPageTokens - 1) / kPageTokens);
+    const int want = std::max(pages, l.Lc / 64);
+    int n = 1;
+    while (n < want && n < limit) n *= 2;
+    return std::min(n, limit);
+}
+template <typename TC, bool DECODE, typename P>
+void launch_latent_kernel(Launcher& L, const DecoderLayer& l, P& p, int splits, int rows) {
+    p.kt = latent_tile(p.s, l.la_heads, splits, sizeof(TC));
+    const size_t smem = la::layout(p.s, l.la_heads, splits, sizeof(TC), p.kt).bytes;
+    const dim3 grid(splits, (l.d.heads + l.la_heads - 1) / l.la_heads, rows), block(la::kThreads);
+    L.cluster_x = splits;
+    if (l.la_heads == 1) L.launch(latent_attention_kernel<TC, DECODE, 1>, grid, block, smem, p);
+    else if (l.la_heads == 2) L.launch(latent_attention_kernel<TC, DECODE, 2>, grid, block, smem, p);
+    else L.launch(latent_attention_kernel<TC, DECODE, 4>, grid, block, smem, p);
+}
+template <typename TC>
+void launch_latent_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const KvSlot& slot, bool early) {
+    DecoderModel& m = *c.decoder;
+    LatentParams<TC, float, float> p{};
+    p.s = latent_shape(m, l);
+    p.q = m.d_q;
+    p.proj = m.d_in;
+    p.ld = l.in.Np;
+    p.pool = static_cast<TC*>(run.k_pool);
+    p.out = m.d_mix;
+    p.ld_out = l.mix_wp;
+    p.pages = m.page_table + (size_t)slot.table * m.d.cache_pages;
+    p.max_pages = slot.n_pages;
+    p.early = early ? 1 : 0;
+    p.state = c.state;
+    launch_latent_kernel<TC, true>(L, l, p, latent_splits(l, slot.n_pages, l.la_cluster), 1);
+}
+template <typename TA>
+void launch_latent_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const RowPlan& plan, const int32_t* list, int n) {
+    DecoderModel& m = *c.decoder;
+    LatentParams<TA, TA, TA> p{};
+    p.s = latent_shape(m, l);
+    p.q = static_cast<const TA*>(m.q);
+    p.proj = static_cast<const TA*>(m.proj_a);
+    p.ld = l.in.Np;
+    p.pool = static_cast<TA*>(run.k_pool);
+    p.out = static_cast<TA*>(m.mix);
+    p.ld_out = l.mix_wp;
+    p.plan = plan;
+    const int groups = (l.d.heads + l.la_heads - 1) / l.la_heads;
+    int splits = latent_splits(l, m.d.cache_pages, l.la_cluster);
+    while (splits > 1 && (int64_t)splits * groups * n > 4 * c.num_sms) splits /= 2;       // many rows fill the GPU by themselves
+    for (int r0 = 0; r0 < n; r0 += 32768) {                          // grid.z
+        p.rows = list != nullptr ? list + r0 : nullptr;
+        launch_latent_kernel<TA, false>(L, l, p, splits, std::min(n - r0, 32768));
+    }
+}
+
+void launch_delta_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const KvSlot& slot, bool early) {
     DecoderModel& m = *c.decoder;
     DeltaDecodeParams p{};
     p.s = delta_shape(m, l);
     p.proj = m.d_in;
     p.w2 = l.w2.w;
     p.ld_w2 = l.w2.Kp;
-    p.pool = m.state_pool + (size_t)slot.state_slot * m.state_stride + l.state_off;
+    p.pool = m.state_pool + (size_t)slot.state_slot * m.state_stride + run.state_off;
     p.state = c.state;
     p.out = m.d_mix;
     p.early = early ? 1 : 0;
@@ -147,24 +240,35 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
         if (L.err == cudaSuccess)
             L.err = cudaMemcpyAsync(m.tap + ((size_t)layer * m.tap_rows + m.tap_row0) * m.Wp, src, (size_t)m.Wp * 4, cudaMemcpyDeviceToDevice, L.stream);
     };
-    for (size_t i = 0; i < m.layers.size(); ++i) {
-        const DecoderLayer& l = m.layers[i];
+    for (size_t i = 0; i < m.runs.size(); ++i) {
+        const DecoderRun& run = m.runs[i];
+        const DecoderLayer& l = m.layers[run.layer];
         // From the second layer on a mixer may read the device state and what earlier steps left in its cache before its
         // dependency wait: the mixer one layer up releases its dependents only after its own wait, so nothing of an
         // earlier step is still running.
         const bool early = i > 0;
         {
             GemvParams p{};
-            stream_input(c, p, pend, i == 0);
+            stream_input(c, p, pend, i == 0, l.pre1);
             p.out_f = m.d_in;
             gemv_ext<Epi::Store32>(c, L, l.in, p);
             if (i > 0) tap((int)i - 1);
         }
         if (l.d.mixer == EFM_MIXER_ATTENTION) {
-            if (m.f32) launch_attn_decode<float>(c, L, l, slot, early);
-            else launch_attn_decode<__nv_bfloat16>(c, L, l, slot, early);
+            if (m.f32) launch_attn_decode<float>(c, L, l, run, slot, early);
+            else launch_attn_decode<__nv_bfloat16>(c, L, l, run, slot, early);
+        } else if (l.d.mixer == EFM_MIXER_LATENT_ATTENTION) {
+            GemvParams p{};
+            p.prologue = kProNorm;
+            p.xf = m.d_in;
+            p.norm_w = l.q_norm;
+            p.k_true = l.d.q_rank;
+            p.out_f = m.d_q;
+            gemv_ext<Epi::Store32>(c, L, l.uq, p);
+            if (m.f32) launch_latent_decode<float>(c, L, l, run, slot, early);
+            else launch_latent_decode<__nv_bfloat16>(c, L, l, run, slot, early);
         } else {
-            launch_delta_decode(c, L, l, slot, early);
+            launch_delta_decode(c, L, l, run, slot, early);
         }
         {
             GemvParams p{};
@@ -173,11 +277,45 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
             p.out_f = m.d_y;
             gemv_ext<Epi::Store32>(c, L, l.out, p);
             pend.y = m.d_y;
-            pend.norm = l.norm1;
+            pend.norm = l.post1;
         }
-        if (l.d.ff > 0) {
+        if (l.moe()) {
+            GemvParams r{};
+            stream_input(c, r, pend, false, l.pre2);
+            r.x_out = m.d_h;
+            r.out_f = m.d_route;
+            gemv_ext<Epi::Store32>(c, L, l.router, r);
             GemvParams p{};
-            stream_input(c, p, pend, false);
+            p.prologue = kProPlain;
+            p.W = l.expert_in.w;
+            p.xf = m.d_h;
+            p.K = l.expert_in.Kp;
+            p.n_items = l.d.expert_top * l.d.expert_ff;
+            p.N = 2 * p.n_items;
+            p.state = c.state;
+            p.route = route_shape(l);
+            p.route_logits = m.d_route;
+            p.route_id = m.d_route_id;
+            p.route_w = m.d_route_w;
+            p.ff = l.d.expert_ff;
+            p.ffp = l.ffp;
+            p.expert_rows = 2 * l.ffp;
+            p.out_f = m.d_act;
+            launch_gemv_ext<Epi::ExpertUp>(c, L, p);
+            GemvParams q = p;
+            q.W = l.expert_out.w;
+            q.xf = m.d_act;
+            q.K = l.d.expert_top * l.ffp;
+            q.n_items = m.Wp / 2;
+            q.N = m.W;
+            q.expert_rows = m.Wp;
+            q.out_f = m.d_y;
+            launch_gemv_ext<Epi::ExpertDown>(c, L, q);
+            pend.y = m.d_y;
+            pend.norm = l.post2;
+        } else if (l.d.ff > 0) {
+            GemvParams p{};
+            stream_input(c, p, pend, false, l.pre2);
             p.out_f = m.d_ff;
             gemv_ext<Epi::Store32>(c, L, l.up, p);
             GemvParams q{};
@@ -188,15 +326,15 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
             q.out_f = m.d_y;
             gemv_ext<Epi::Store32>(c, L, l.down, q);
             pend.y = m.d_y;
-            pend.norm = l.norm2;
+            pend.norm = l.post2;
         }
         if (m.d.side_dim > 0) {
             GemvParams p{};
-            stream_input(c, p, pend, false);
+            stream_input(c, p, pend, false, nullptr);
             p.out_f = m.d_gate;
             p.gate_table = m.side_embed;
             p.gate_ld = m.d.side_dim * m.d.num_layers;
-            p.gate_off = (int)i * m.d.side_dim;
+            p.gate_off = run.layer * m.d.side_dim;
             if (m.side_cluster > 1 && p.prologue == kProAddNorm) {
                 TokenSideParams q{};
                 p.W = l.gate.w;
@@ -228,13 +366,12 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
     if (!want_logits && !sample && m.tap == nullptr) return;
     {
         GemvParams p{};
-        stream_input(c, p, pend, false);
-        p.norm2_w = m.final_norm;
+        stream_input(c, p, pend, false, m.final_norm);
         p.logits = c.logits;
         p.part_val = c.part_val;
         p.part_idx = c.part_idx;
         gemv_ext<Epi::Logits>(c, L, m.head, p);
-        tap((int)m.layers.size() - 1);
+        tap((int)m.runs.size() - 1);
     }
     if (!sample) return;
     SampleParams s{};
@@ -262,8 +399,8 @@ int decoder_simt_tile_rows() { return wa::QT; }
 bool decoder_layer_tc(const DecoderModel& m, const DecoderLayer& l) {
     static const bool off = [] { const char* e = std::getenv("EFM_B200_ATTN_TC"); return e != nullptr && e[0] == '0'; }();
     int pages = m.d.cache_pages;
-    if (l.d.window > 0) pages = std::min(pages, (l.d.window + wt::BM) / kPageTokens + 2);
-    return !off && !m.f32 && l.Dp <= 128 && l.Vp <= 128 && pages <= wt::kMaxTiles;
+    if (l.d.window > 0) pages = std::min(pages, (l.d.window + wt::BM) / kPageTokens + 2 + (l.d.keep_first + kPageTokens - 1) / kPageTokens);
+    return !off && !m.f32 && l.Dp <= 128 && l.Vp <= 128 && l.Rc <= 64 && pages <= wt::kMaxTiles;
 }
 
 namespace {
@@ -272,72 +409,112 @@ namespace {
 void linear_f32(efm_b200_ctx& c, Launcher& L, const DecLinear& w, const void* a, float* out, int rows) {
     if (c.decoder->f32) {
         L.launch(gemm_f32_kernel, dim3((w.Np + 63) / 64, (rows + 63) / 64), dim3(256), 0, static_cast<const float*>(a), w.Kp,
-                 (const __nv_bfloat16*)w.w, w.Kp, out, w.Np, rows, w.Np, w.Kp);
+                 (const __nv_bfloat16*)w.w, w.Kp, out, w.Np, rows, w.Np, w.Kp, (const __nv_bfloat16*)w.bias, RowGroups{});
         return;
     }
-    GemmParams g{static_cast<const __nv_bfloat16*>(a), w.w, nullptr, nullptr, out, rows, w.Np, w.Kp};
+    GemmParams g{static_cast<const __nv_bfloat16*>(a), w.w, w.bias, nullptr, out, rows, w.Np, w.Kp};
     launch_gemm_epi(L, GemmEpi::F32, g, &c.state->error);
 }
 // the same with the activation type of the pass as output
 void linear_act(efm_b200_ctx& c, Launcher& L, const DecLinear& w, const void* a, void* out, int rows) {
     if (c.decoder->f32) { linear_f32(c, L, w, a, static_cast<float*>(out), rows); return; }
-    GemmParams g{static_cast<const __nv_bfloat16*>(a), w.w, nullptr, static_cast<__nv_bfloat16*>(out), nullptr, rows, w.Np, w.Kp};
+    GemmParams g{static_cast<const __nv_bfloat16*>(a), w.w, w.bias, static_cast<__nv_bfloat16*>(out), nullptr, rows, w.Np, w.Kp};
     launch_gemm_epi(L, GemmEpi::Bf16Bias, g, &c.state->error);
 }
 
 template <int NC>
-void launch_delta_scan(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const RowPlan& plan) {
+void launch_delta_scan(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const RowPlan& plan) {
     DecoderModel& m = *c.decoder;
     const DeltaShape s = delta_shape(m, l);
     const int groups = (s.Dp + ds::kCols - 1) / ds::kCols;
     L.launch(delta_scan_kernel<NC>, dim3(l.d.heads * groups, plan.n_entries), dim3(ds::kThreads), ds::smem_bytes(s.Dp), (const float*)m.pack, m.o, l.mix_wp,
-             m.state_pool, m.state_stride, l.state_off, s, plan);
+             m.state_pool, m.state_stride, run.state_off, s, plan);
 }
 
-template <int DP, int VP>
-void launch_attention_tc_v(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const WindowAttnShape& s, const RowPlan& plan, const RowTile* list, int n) {
+// The maps of attention and latent attention differ; what is launched is the same.
+template <int DP, int VP, int RP>
+void launch_attention_tc_v(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const WindowAttnShape& s, const WindowTcMaps& maps, const RowPlan& plan,
+                           const RowTile* list, int n) {
+    L.launch(window_attention_tc_kernel<DP, VP, RP>, dim3(n, s.H), dim3(wt::kThreads), wt::Cfg<DP, VP, RP>::SMEM, maps, static_cast<__nv_bfloat16*>(c.decoder->mix),
+             l.mix_wp, s, plan, list, RP > 0 ? 1 : 0, &c.state->error);
+}
+template <int RP>
+void launch_attention_tc_r(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const WindowAttnShape& s, const WindowTcMaps& maps, const RowPlan& plan,
+                           const RowTile* list, int n) {
+    if (l.Dp <= 64 && l.Vp <= 64) launch_attention_tc_v<64, 64, RP>(c, L, l, s, maps, plan, list, n);
+    else if (l.Dp <= 64) launch_attention_tc_v<64, 128, RP>(c, L, l, s, maps, plan, list, n);
+    else if (l.Vp <= 64) launch_attention_tc_v<128, 64, RP>(c, L, l, s, maps, plan, list, n);
+    else launch_attention_tc_v<128, 128, RP>(c, L, l, s, maps, plan, list, n);
+}
+// [rows][heads][channels] with strides in elements
+bool head_map(CUtensorMap* map, const void* base, int channels, int heads, int rows, int head_stride, int row_stride, int box_rows) {
+    const uint64_t d[3] = {(uint64_t)channels, (uint64_t)heads, (uint64_t)rows}, st[2] = {(uint64_t)head_stride * 2, (uint64_t)row_stride * 2};
+    const uint32_t b[3] = {64, 1, (uint32_t)box_rows};
+    return make_map_nd(map, base, 3, d, st, b);
+}
+void launch_attention_tc(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const WindowAttnShape& s, const RowPlan& plan,
+                         const RowTile* list, int n) {
+    if (n <= 0) return;
     DecoderModel& m = *c.decoder;
-    CUtensorMap mq, mk, mv;
-    const uint64_t rows = (uint64_t)m.d.cache_pages * kPageTokens;
-    const uint64_t qd[3] = {(uint64_t)DP, (uint64_t)s.H, (uint64_t)plan.rows}, qs[2] = {(uint64_t)DP * 2, (uint64_t)s.H * DP * 2};
-    const uint64_t kd[3] = {(uint64_t)DP, (uint64_t)s.G, rows}, ks[2] = {(uint64_t)DP * 2, (uint64_t)s.G * DP * 2};
-    const uint64_t vd[3] = {(uint64_t)VP, (uint64_t)s.G, rows}, vs[2] = {(uint64_t)VP * 2, (uint64_t)s.G * VP * 2};
-    const uint32_t qb[3] = {64, 1, (uint32_t)wt::BM}, kb[3] = {64, 1, (uint32_t)wt::BN};
-    if (!make_map_nd(&mq, m.q, 3, qd, qs, qb) || !make_map_nd(&mk, l.k_pool, 3, kd, ks, kb) || !make_map_nd(&mv, l.v_pool, 3, vd, vs, kb)) {
+    WindowTcMaps maps;
+    const int rows = m.d.cache_pages * kPageTokens;
+    if (!head_map(&maps.q, m.q, s.Dp, s.H, plan.rows, s.Dp, s.H * s.Dp, wt::BM) || !head_map(&maps.k, run.k_pool, s.Dp, s.G, rows, s.Dp, s.G * s.Dp, wt::BN) ||
+        !head_map(&maps.v, run.v_pool, s.Vp, s.G, rows, s.Vp, s.G * s.Vp, wt::BN)) {
         if (L.err == cudaSuccess) L.err = cudaErrorInvalidValue;
         return;
     }
-    L.launch(window_attention_tc_kernel<DP, VP>, dim3(n, s.H), dim3(wt::kThreads), wt::Cfg<DP, VP>::SMEM, mq, mk, mv, static_cast<__nv_bfloat16*>(m.mix), l.mix_wp,
-             s, plan, list, &c.state->error);
+    maps.qr = maps.q;
+    maps.kr = maps.k;
+    launch_attention_tc_r<0>(c, L, l, s, maps, plan, list, n);
 }
-void launch_attention_tc(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const WindowAttnShape& s, const RowPlan& plan, const RowTile* list, int n) {
-    if (n <= 0) return;
-    if (l.Dp == 64 && l.Vp == 64) launch_attention_tc_v<64, 64>(c, L, l, s, plan, list, n);
-    else if (l.Dp == 64) launch_attention_tc_v<64, 128>(c, L, l, s, plan, list, n);
-    else if (l.Vp == 64) launch_attention_tc_v<128, 64>(c, L, l, s, plan, list, n);
-    else launch_attention_tc_v<128, 128>(c, L, l, s, plan, list, n);
+// Long entries of a latent layer: visible cache rows into the workspace, keys and values of all heads by one product,
+// attention over those.
+void launch_latent_tc(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const RowPlan& plan, const RowTiles& tiles,
+                      const RowTile* list, int n) {
+    DecoderModel& m = *c.decoder;
+    const LatentShape z = latent_shape(m, l);
+    const int LR = z.Lc + z.Rc, n_ws = tiles.n_ws * kPageTokens, ld = l.ukv.Np;
+    L.launch(latent_gather_rows_kernel<__nv_bfloat16>, dim3(tiles.n_ws), dim3(256), 0, static_cast<const __nv_bfloat16*>(run.k_pool), m.ws_c, LR, plan,
+             tiles.ws_pages, tiles.ws_page0);
+    GemmParams g{m.ws_c, l.ukv.w, nullptr, m.ws_kv, nullptr, n_ws, l.ukv.Np, l.ukv.Kp};
+    g.lda = LR;
+    launch_gemm_epi(L, GemmEpi::Bf16Bias, g, &c.state->error);
+    WindowAttnShape s{};
+    s.H = s.G = z.H; s.D = z.D; s.Dv = z.Dv; s.Dp = z.Dp; s.Vp = z.Vp;
+    s.window = z.window; s.scale = z.scale; s.eps = z.eps; s.sink = z.sink;
+    if (z.gate) { s.gate = static_cast<const __nv_bfloat16*>(m.proj_a) + z.off_gate(); s.gate_ld = l.in.Np; }
+    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(m.q);
+    WindowTcMaps maps;
+    const int qh = z.Dp + z.Rc;
+    if (!head_map(&maps.q, q, z.Dp, z.H, plan.rows, qh, z.q_ld(), wt::BM) || !head_map(&maps.qr, q + z.Dp, z.Rc, z.H, plan.rows, qh, z.q_ld(), wt::BM) ||
+        !head_map(&maps.k, m.ws_kv, z.Dp, z.H, n_ws, z.Dp, ld, wt::BN) || !head_map(&maps.v, m.ws_kv + (size_t)z.H * z.Dp, z.Vp, z.H, n_ws, z.Vp, ld, wt::BN) ||
+        !head_map(&maps.kr, m.ws_c + z.Lc, z.Rc, 1, n_ws, LR, LR, wt::BN)) {
+        if (L.err == cudaSuccess) L.err = cudaErrorInvalidValue;
+        return;
+    }
+    launch_attention_tc_r<64>(c, L, l, s, maps, plan, list, n);
 }
 
 // Chunked recurrence: every chunk's state-independent part at once, then the chunks in sequence.
 template <int DP>
-void launch_delta_chunks(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const RowPlan& plan) {
+void launch_delta_chunks(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const RowPlan& plan) {
     DecoderModel& m = *c.decoder;
     const DeltaShape s = delta_shape(m, l);
     const int chunks = plan.n_entries == 1 ? (plan.rows + dc::C - 1) / dc::C : plan.rows / dc::C + plan.n_entries;     // at most
     L.launch(delta_prepare_kernel<DP>, dim3(chunks, l.d.heads), dim3(dc::kThreads), sizeof(dc::PrepSmem<DP>), (const float*)m.proj_f, (const float*)m.decay,
              l.w2.Np, m.pack, s, plan);
     L.launch(delta_chunk_scan_kernel<DP>, dim3(l.d.heads * (DP / dc::kCols), plan.n_entries), dim3(dc::kScanThreads), sizeof(dc::ScanSmem<DP>), (const float*)m.pack,
-             m.o, l.mix_wp, m.state_pool, m.state_stride, l.state_off, s, plan);
+             m.o, l.mix_wp, m.state_pool, m.state_stride, run.state_off, s, plan);
 }
 
 // TA: activation and cache type of the pass
 template <typename TA>
-void attention_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const RowPlan& plan, const RowTiles& tiles) {
+void attention_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const void* x, const RowPlan& plan, const RowTiles& tiles) {
     DecoderModel& m = *c.decoder;
     const WindowAttnShape s = attn_shape(m, l);
-    linear_act(c, L, l.in, m.f32 ? (void*)c.resid : m.xa, m.proj_a, plan.rows);
-    TA* kp = static_cast<TA*>(l.k_pool);
-    TA* vp = static_cast<TA*>(l.v_pool);
+    linear_act(c, L, l.in, x, m.proj_a, plan.rows);
+    TA* kp = static_cast<TA*>(run.k_pool);
+    TA* vp = static_cast<TA*>(run.v_pool);
     int lanes = 8;                                                  // 8 channels each: at most 256 (padded) channels a head
     while (lanes * 8 < std::max(s.Dp, s.Vp)) lanes *= 2;
     L.launch(qk_scatter_rows_kernel<TA, TA, TA>, dim3(plan.rows), dim3(256), 0, static_cast<const TA*>(m.proj_a), l.in.Np, static_cast<TA*>(m.q), kp, vp, s, plan,
@@ -350,12 +527,12 @@ void attention_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const R
     if constexpr (std::is_same<TA, __nv_bfloat16>::value) {
         if (decoder_layer_tc(m, l)) {
             if (tiles.listed) {
-                launch_attention_tc(c, L, l, s, plan, tiles.tc, tiles.n_tc);
+                launch_attention_tc(c, L, l, run, s, plan, tiles.tc, tiles.n_tc);
                 cuda_cores(tiles.simt, tiles.n_simt);
                 return;
             }
             if (plan.rows >= kTcMinRows) {
-                launch_attention_tc(c, L, l, s, plan, nullptr, (plan.rows + wt::BM - 1) / wt::BM);
+                launch_attention_tc(c, L, l, run, s, plan, nullptr, (plan.rows + wt::BM - 1) / wt::BM);
                 return;
             }
         }
@@ -364,32 +541,93 @@ void attention_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const R
 }
 
 template <typename TA>
-void delta_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const RowPlan& plan) {
+void latent_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const void* x, const RowPlan& plan, const RowTiles& tiles) {
+    DecoderModel& m = *c.decoder;
+    const LatentShape s = latent_shape(m, l);
+    const int T = plan.rows;
+    linear_act(c, L, l.in, x, m.proj_a, T);
+    L.launch(latent_rows_kernel<TA>, dim3(T), dim3(256), 0, static_cast<const TA*>(m.proj_a), l.in.Np, static_cast<TA*>(m.cq), static_cast<TA*>(run.k_pool), s, plan);
+    linear_act(c, L, l.uq, m.cq, m.q, T);
+    L.launch(latent_rotate_rows_kernel<TA>, dim3(T), dim3(256), 0, static_cast<TA*>(m.q), s, plan);
+    if constexpr (std::is_same<TA, __nv_bfloat16>::value) {
+        if (decoder_layer_tc(m, l)) {
+            if (tiles.listed) {
+                if (tiles.n_tc > 0) launch_latent_tc(c, L, l, run, plan, tiles, tiles.tc, tiles.n_tc);
+                if (tiles.n_short > 0) launch_latent_rows<TA>(c, L, l, run, plan, tiles.short_rows, tiles.n_short);
+                return;
+            }
+            if (T >= kTcMinRows) {
+                launch_latent_tc(c, L, l, run, plan, tiles, nullptr, (T + wt::BM - 1) / wt::BM);
+                return;
+            }
+        }
+    }
+    launch_latent_rows<TA>(c, L, l, run, plan, nullptr, T);
+}
+
+// Routed experts of all rows: choice, rows sorted by expert, two grouped products.  The outputs stay sorted (m.ex_y); the norm
+// that follows sums them (SumOf).
+template <typename TA>
+SumOf expert_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const void* h, int T) {
+    DecoderModel& m = *c.decoder;
+    const RouteShape r = route_shape(l);
+    linear_f32(c, L, l.router, h, m.route_logits, T);
+    L.launch(expert_route_rows_kernel, dim3((T + 7) / 8), dim3(256), 0, (const float*)m.route_logits, l.router.Np, T, r, m.ex);
+    L.launch(expert_gather_rows_kernel<TA>, dim3(T), dim3(128), 0, static_cast<const TA*>(h), static_cast<TA*>(m.ex_in), m.Wp, r, m.ex);
+    // tiles in use at most: every row tile but the last of an expert is full
+    const int64_t picks = (int64_t)T * r.top;
+    const int max_rows = (int)std::min<int64_t>(m.ex_rows, (picks / kExpertTile + std::min<int64_t>(picks, r.experts)) * kExpertTile);
+    if constexpr (std::is_same<TA, float>::value) {
+        auto product = [&](const DecLinear& w, int n, const float* a, float* out) {
+            L.launch(gemm_f32_kernel, dim3((n + 63) / 64, (max_rows + 63) / 64), dim3(256), 0, a, w.Kp, (const __nv_bfloat16*)w.w, w.Kp, out, n, max_rows, n, w.Kp,
+                     (const __nv_bfloat16*)nullptr, RowGroups{m.ex.tile_expert, m.ex.n_tiles, n});
+        };
+        product(l.expert_in, 2 * l.ffp, static_cast<const float*>(m.ex_in), m.ex_gu);
+        L.launch(silu_mul_rows_kernel, dim3(max_rows / kExpertTile), dim3(256), 0, (const float*)m.ex_gu, static_cast<float*>(m.ex_act), l.ffp,
+                 (const int32_t*)m.ex.n_tiles);
+        product(l.expert_out, m.Wp, static_cast<const float*>(m.ex_act), m.ex_y);
+    } else {
+        auto product = [&](const DecLinear& w, int n, GemmEpi epi, const void* a, void* out, float* out_f) {
+            GemmParams g{static_cast<const __nv_bfloat16*>(a), w.w, nullptr, static_cast<__nv_bfloat16*>(out), out_f, max_rows, n, w.Kp};
+            g.group_tile = m.ex.tile_expert;
+            g.group_tiles = m.ex.n_tiles;
+            g.group_rows = n;
+            g.group_all = r.experts * n;
+            launch_gemm_epi(L, epi, g, &c.state->error);
+        };
+        product(l.expert_in, 2 * l.ffp, GemmEpi::SwiGlu, m.ex_in, m.ex_act, nullptr);
+        product(l.expert_out, m.Wp, GemmEpi::F32, m.ex_act, nullptr, m.ex_y);
+    }
+    return SumOf{m.ex.place, m.ex.weight, r.top, m.ex.count, r.experts};
+}
+
+template <typename TA>
+void delta_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const void* x, const RowPlan& plan) {
     DecoderModel& m = *c.decoder;
     const DeltaShape s = delta_shape(m, l);
-    linear_f32(c, L, l.in, m.f32 ? (void*)c.resid : m.xa, m.proj_f, plan.rows);
+    linear_f32(c, L, l.in, x, m.proj_f, plan.rows);
     L.launch(delta_tanh_rows_kernel, dim3(plan.rows), dim3(128), 0, (const float*)m.proj_f, m.tanh_w, l.w2.Kp, s);
     L.launch(gemm_f32_kernel, dim3((l.w2.Np + 63) / 64, (plan.rows + 63) / 64), dim3(256), 0, (const float*)m.tanh_w, l.w2.Kp, (const __nv_bfloat16*)l.w2.w,
-             l.w2.Kp, m.decay, l.w2.Np, plan.rows, l.w2.Np, l.w2.Kp);
+             l.w2.Kp, m.decay, l.w2.Np, plan.rows, l.w2.Np, l.w2.Kp, (const __nv_bfloat16*)nullptr, RowGroups{});
     const bool chunked = plan.rows >= dc::C && s.Dp <= 128;         // short passes and larger heads: token by token
     if (chunked) {
         switch (s.Dp / 32) {
-            case 1: launch_delta_chunks<32>(c, L, l, plan); break;
-            case 2: launch_delta_chunks<64>(c, L, l, plan); break;
-            case 3: launch_delta_chunks<96>(c, L, l, plan); break;
-            default: launch_delta_chunks<128>(c, L, l, plan); break;
+            case 1: launch_delta_chunks<32>(c, L, l, run, plan); break;
+            case 2: launch_delta_chunks<64>(c, L, l, run, plan); break;
+            case 3: launch_delta_chunks<96>(c, L, l, run, plan); break;
+            default: launch_delta_chunks<128>(c, L, l, run, plan); break;
         }
     } else {
         L.launch(delta_inputs_rows_kernel, dim3(plan.rows), dim3(256), 0, (const float*)m.proj_f, (const float*)m.decay, l.w2.Np, m.pack, s);
         switch (s.Dp / 32) {
-            case 1: launch_delta_scan<1>(c, L, l, plan); break;
-            case 2: launch_delta_scan<2>(c, L, l, plan); break;
-            case 3: launch_delta_scan<3>(c, L, l, plan); break;
-            case 4: launch_delta_scan<4>(c, L, l, plan); break;
-            case 5: launch_delta_scan<5>(c, L, l, plan); break;
-            case 6: launch_delta_scan<6>(c, L, l, plan); break;
-            case 7: launch_delta_scan<7>(c, L, l, plan); break;
-            default: launch_delta_scan<8>(c, L, l, plan); break;
+            case 1: launch_delta_scan<1>(c, L, l, run, plan); break;
+            case 2: launch_delta_scan<2>(c, L, l, run, plan); break;
+            case 3: launch_delta_scan<3>(c, L, l, run, plan); break;
+            case 4: launch_delta_scan<4>(c, L, l, run, plan); break;
+            case 5: launch_delta_scan<5>(c, L, l, run, plan); break;
+            case 6: launch_delta_scan<6>(c, L, l, run, plan); break;
+            case 7: launch_delta_scan<7>(c, L, l, run, plan); break;
+            default: launch_delta_scan<8>(c, L, l, run, plan); break;
         }
     }
     int lanes = 1;
@@ -402,32 +640,39 @@ template <typename TA>
 void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const RowTiles& tiles, Launcher& L) {
     DecoderModel& m = *c.decoder;
     const int T = plan.rows;
-    TA* xa = m.f32 ? nullptr : static_cast<TA*>(m.xa);          // 32-bit mode reads the stream itself
-    const void* xin = m.f32 ? (const void*)c.resid : m.xa;
-    auto add_norm = [&](const float* y, const __nv_bfloat16* w) {
-        L.launch(add_norm_rows_kernel<TA>, dim3(T), dim3(256), 0, c.resid, y, w, xa, m.W, m.Wp, m.d.norm_eps);
+    TA* xa = static_cast<TA*>(m.xa);                            // null: 32-bit mode without input norms reads the stream itself
+    const void* xin = xa != nullptr ? (const void*)xa : c.resid;
+    // the stream takes a sublayer's normed output; xa becomes the next sublayer's input
+    auto add_norm = [&](const float* y, const __nv_bfloat16* w, const __nv_bfloat16* pre, const SumOf& sum = SumOf{}) {
+        L.launch(add_norm_rows_kernel<TA>, dim3(T), dim3(256), 0, c.resid, y, w, xa, pre, m.W, m.Wp, m.d.norm_eps, sum);
     };
-    launch_embed_rows(L, ids, c.embed, nullptr, c.resid, T, c.d.vocab, m.Wp, -1, 0);
-    if (xa != nullptr) add_norm(nullptr, nullptr);
-    for (size_t i = 0; i < m.layers.size(); ++i) {
-        const DecoderLayer& l = m.layers[i];
-        if (l.d.mixer == EFM_MIXER_ATTENTION) attention_rows<TA>(c, L, l, plan, tiles);
-        else delta_rows<TA>(c, L, l, plan);
+    launch_embed_rows(L, ids, c.embed, nullptr, c.resid, T, c.d.vocab, m.Wp, -1, 0, m.d.embed_scale);
+    if (xa != nullptr) add_norm(nullptr, nullptr, m.layers[m.runs[0].layer].pre1);
+    for (size_t i = 0; i < m.runs.size(); ++i) {
+        const DecoderRun& run = m.runs[i];
+        const DecoderLayer& l = m.layers[run.layer];
+        const __nv_bfloat16* next = i + 1 < m.runs.size() ? m.layers[m.runs[i + 1].layer].pre1 : nullptr;
+        if (l.d.mixer == EFM_MIXER_ATTENTION) attention_rows<TA>(c, L, l, run, xin, plan, tiles);
+        else if (l.d.mixer == EFM_MIXER_LATENT_ATTENTION) latent_rows<TA>(c, L, l, run, xin, plan, tiles);
+        else delta_rows<TA>(c, L, l, run, xin, plan);
         linear_f32(c, L, l.out, m.mix, m.y, T);
-        add_norm(m.y, l.norm1);
-        if (l.d.ff > 0) {
+        add_norm(m.y, l.post1, l.mlp() ? l.pre2 : next);
+        if (l.moe()) {
+            const SumOf sum = expert_rows<TA>(c, L, l, xin, T);
+            add_norm(m.ex_y, l.post2, next, sum);
+        } else if (l.d.ff > 0) {
             linear_act(c, L, l.up, xin, m.ff, T);
             L.launch(poly_norm_rows_kernel<TA>, dim3(T), dim3(256), 0, static_cast<const TA*>(m.ff), static_cast<TA*>(m.ff2), (const __nv_bfloat16*)l.act, l.d.ff,
                      l.down.Kp, m.d.norm_eps);
             linear_f32(c, L, l.down, m.ff2, m.y, T);
-            add_norm(m.y, l.norm2);
+            add_norm(m.y, l.post2, next);
         }
         if (m.d.side_dim > 0) {
             linear_f32(c, L, l.gate, xin, m.side_f, T);
             L.launch(token_gate_rows_kernel<TA>, dim3(T), dim3(128), 0, (const float*)m.side_f, ids, (const __nv_bfloat16*)m.side_embed,
-                     m.d.side_dim * m.d.num_layers, (int)i * m.d.side_dim, c.d.vocab, static_cast<TA*>(m.side_a), m.d.side_dim, m.side_p);
+                     m.d.side_dim * m.d.num_layers, run.layer * m.d.side_dim, c.d.vocab, static_cast<TA*>(m.side_a), m.d.side_dim, m.side_p);
             linear_f32(c, L, l.proj, m.side_a, m.y, T);
-            add_norm(m.y, l.side_norm);
+            add_norm(m.y, l.side_norm, nullptr);
         }
         if (m.tap != nullptr && m.tap_row0 + T <= m.tap_rows && L.err == cudaSuccess)
             L.err = cudaMemcpyAsync(m.tap + ((size_t)i * m.tap_rows + m.tap_row0) * m.Wp, c.resid, (size_t)T * m.Wp * 4, cudaMemcpyDeviceToDevice, L.stream);
@@ -524,6 +769,51 @@ static cudaError_t fit_side_cluster(DecoderModel& m, int optin) {
     return m.side_cluster > 1 ? smem_attr(token_side_kernel, (size_t)optin - 2048) : cudaSuccess;
 }
 
+// Heads per block and cluster width of the absorbed form: the widest cluster that fits, and as few heads per block as keep
+// all clusters resident at once.
+template <typename TC, int NH>
+static cudaError_t fit_latent_heads(const DecoderModel& m, DecoderLayer& l, int optin, bool& done) {
+    cudaError_t e = smem_attr(latent_attention_kernel<TC, true, NH>, (size_t)optin - 4096);
+    if (e == cudaSuccess) e = smem_attr(latent_attention_kernel<TC, false, NH>, (size_t)optin - 4096);
+    if (e != cudaSuccess) return e;
+    const bool wide = cudaFuncSetAttribute(latent_attention_kernel<TC, true, NH>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess &&
+                      cudaFuncSetAttribute(latent_attention_kernel<TC, false, NH>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess;
+    if (done) return cudaSuccess;
+    const LatentShape s = latent_shape(m, l);
+    const int groups = (l.d.heads + NH - 1) / NH, most = latent_splits(l, m.d.cache_pages, wide ? 16 : 8);
+    for (int cs = most; cs >= 1; cs >>= 1) {
+        const size_t bytes = la::layout(s, NH, cs, sizeof(TC), latent_tile(s, NH, cs, sizeof(TC))).bytes;
+        if (bytes > (size_t)optin - 4096) continue;
+        cudaLaunchConfig_t cfg = {};
+        cfg.gridDim = dim3(cs, 1, 1);
+        cfg.blockDim = dim3(la::kThreads);
+        cfg.dynamicSmemBytes = bytes;
+        cudaLaunchAttribute at;
+        at.id = cudaLaunchAttributeClusterDimension;
+        at.val.clusterDim.x = (unsigned)cs;
+        at.val.clusterDim.y = at.val.clusterDim.z = 1;
+        cfg.attrs = &at;
+        cfg.numAttrs = 1;
+        int n = 0;
+        if (cudaOccupancyMaxActiveClusters(&n, latent_attention_kernel<TC, true, NH>, &cfg) == cudaSuccess && n >= 1) {
+            l.la_heads = NH;
+            l.la_cluster = cs;
+            done = n >= groups || NH == 4;
+            break;
+        }
+    }
+    (void)cudaGetLastError();
+    return cudaSuccess;
+}
+template <typename TC>
+static cudaError_t fit_latent(const DecoderModel& m, DecoderLayer& l, int optin) {
+    bool done = false;
+    cudaError_t e = fit_latent_heads<TC, 1>(m, l, optin, done);
+    if (e == cudaSuccess) e = fit_latent_heads<TC, 2>(m, l, optin, done);
+    if (e == cudaSuccess) e = fit_latent_heads<TC, 4>(m, l, optin, done);
+    return e;
+}
+
 cudaError_t configure_decoder(DecoderModel& m) {
     int dev = 0, optin = 0;
     cudaError_t e = cudaGetDevice(&dev);
@@ -532,6 +822,8 @@ cudaError_t configure_decoder(DecoderModel& m) {
     if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::Store32, true>, gv);
     if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::TokenGate, true>, gv);
     if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::Logits, true>, gv);
+    if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::ExpertUp, true>, gv);
+    if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::ExpertDown, true>, gv);
     const size_t rows = wa::rows_smem_bytes(256, 256);
     if (e == cudaSuccess) e = smem_attr(window_attention_rows_kernel<float, float, float>, rows);
     if (e == cudaSuccess) e = smem_attr(window_attention_rows_kernel<__nv_bfloat16, __nv_bfloat16, __nv_bfloat16>, rows);
@@ -539,16 +831,22 @@ cudaError_t configure_decoder(DecoderModel& m) {
     if (e == cudaSuccess) e = smem_attr(delta_scan_kernel<6>, ds::smem_bytes(192));
     if (e == cudaSuccess) e = smem_attr(delta_scan_kernel<7>, ds::smem_bytes(224));
     if (e == cudaSuccess) e = smem_attr(delta_scan_kernel<8>, ds::smem_bytes(256));
-    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<64, 64>, wt::Cfg<64, 64>::SMEM);
-    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<64, 128>, wt::Cfg<64, 128>::SMEM);
-    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<128, 64>, wt::Cfg<128, 64>::SMEM);
-    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<128, 128>, wt::Cfg<128, 128>::SMEM);
+    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<64, 64, 0>, wt::Cfg<64, 64, 0>::SMEM);
+    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<64, 64, 64>, wt::Cfg<64, 64, 64>::SMEM);
+    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<64, 128, 0>, wt::Cfg<64, 128, 0>::SMEM);
+    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<64, 128, 64>, wt::Cfg<64, 128, 64>::SMEM);
+    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<128, 64, 0>, wt::Cfg<128, 64, 0>::SMEM);
+    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<128, 64, 64>, wt::Cfg<128, 64, 64>::SMEM);
+    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<128, 128, 0>, wt::Cfg<128, 128, 0>::SMEM);
+    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<128, 128, 64>, wt::Cfg<128, 128, 64>::SMEM);
     if (e == cudaSuccess) e = smem_attr(delta_prepare_kernel<96>, sizeof(dc::PrepSmem<96>));
     if (e == cudaSuccess) e = smem_attr(delta_prepare_kernel<128>, sizeof(dc::PrepSmem<128>));
     if (e == cudaSuccess) e = smem_attr(delta_chunk_scan_kernel<64>, sizeof(dc::ScanSmem<64>));
     if (e == cudaSuccess) e = smem_attr(delta_chunk_scan_kernel<96>, sizeof(dc::ScanSmem<96>));
     if (e == cudaSuccess) e = smem_attr(delta_chunk_scan_kernel<128>, sizeof(dc::ScanSmem<128>));
     if (e == cudaSuccess) e = fit_side_cluster(m, optin);
+    for (DecoderLayer& l : m.layers)
+        if (l.d.mixer == EFM_MIXER_LATENT_ATTENTION && e == cudaSuccess) e = m.f32 ? fit_latent<float>(m, l, optin) : fit_latent<__nv_bfloat16>(m, l, optin);
     m.attn_cluster = 16;
     if (e == cudaSuccess) e = m.f32 ? fit_cluster<float, 64>(m.attn_cluster) : fit_cluster<__nv_bfloat16, 64>(m.attn_cluster);
     if (e == cudaSuccess) e = m.f32 ? fit_cluster<float, 128>(m.attn_cluster) : fit_cluster<__nv_bfloat16, 128>(m.attn_cluster);

@@ -1,12 +1,15 @@
-// Layered decoder: a list of layers, each with its own mixer (attention | generalised delta rule) and an optional dense
-// feed-forward, sublayer outputs normalised before the residual add, optional per-layer token input.  Weights, buffers
-// and launch sequences (definitions in decoder.cu); the C ABI side is backends/b200/decoder_b200.cu.
+// Layered decoder: a list of layers, each with its own mixer (attention | latent attention | generalised delta rule) and an
+// optional feed-forward (dense | routed experts), sublayer outputs (and, sandwich layout, inputs) normalised, optional
+// per-layer token input; a span of layers may run several times.  Weights, buffers and launch sequences (definitions in
+// decoder.cu); the C ABI side is backends/b200/decoder_b200.cu.
 #pragma once
+#include <algorithm>
 #include <set>
 #include <string>
 #include <vector>
 
 #include "../backends/b200/ctx.h"
+#include "../operators/expert_rows.h"
 #include "../operators/row_plan.cuh"
 
 namespace efm {
@@ -18,21 +21,38 @@ inline int round_up(int n, int m) { return (n + m - 1) / m * m; }
 struct DecLinear {
     __nv_bfloat16* w = nullptr;
     int N = 0, K = 0, Np = 0, Kp = 0;
+    __nv_bfloat16* bias = nullptr;        // [Np] or null
 };
 
 struct DecoderLayer {
     efm_decoder_layer d{};
-    int Dp = 0, Vp = 0;                   // attention: padded channels of a cache row
+    int Dp = 0, Vp = 0;                   // attention: padded channels of a cache row; latent: padded head channels
     int mix_w = 0, mix_wp = 0;            // mixer output width (heads * value channels), padded
-    DecLinear in;                         // attention: q | k | v; delta: r | k | v | g | a | w1
+    DecLinear in;                         // attention: q | k | v; latent: dq | c | r | g, each padded to 8; delta: r | k | v | g | a | w1
     DecLinear out;                        // W_o
     DecLinear w2;                         // delta: decay projection
-    DecLinear up, down, gate, proj;       // feed-forward; token side
-    __nv_bfloat16 *norm1 = nullptr, *norm2 = nullptr, *side_norm = nullptr, *act = nullptr;
+    DecLinear up, down, gate, proj;       // dense feed-forward; token side
+    __nv_bfloat16 *pre1 = nullptr, *pre2 = nullptr, *post1 = nullptr, *post2 = nullptr, *side_norm = nullptr, *act = nullptr;
     __nv_bfloat16 *q_norm = nullptr, *k_norm = nullptr, *temp = nullptr;
     __nv_bfloat16 *w0 = nullptr, *a_bias = nullptr, *mix_norm = nullptr;
-    void *k_pool = nullptr, *v_pool = nullptr;       // [pages * 64][kv_heads][Dp / Vp], bf16 or fp32
-    size_t state_off = 0;                 // delta: first float of this layer inside a state slot
+    float* inv_freq = nullptr;            // rotation: [rot_dims / 2]
+    // latent attention
+    int Qp = 0, Lc = 0, Rc = 0;           // query latent, cached latent, rotated part: padded to 8
+    DecLinear uq, ukv;                    // [heads][Dp + Rc] rows; [heads][Dp] key rows, then [heads][Vp] value rows
+    __nv_bfloat16* sink = nullptr;
+    int la_heads = 1, la_cluster = 1;     // heads per block and widest cluster of the absorbed form
+    // routed experts
+    DecLinear router, expert_in, expert_out;   // [experts]; [experts][2 * ffp]; [experts][width][ffp]
+    int ffp = 0;
+    bool moe() const { return d.experts > 0; }
+    bool mlp() const { return d.experts > 0 || d.ff > 0; }
+};
+
+// One run of a layer: a looped layer runs several times, every time with its own cache or state.
+struct DecoderRun {
+    int layer = 0;
+    void *k_pool = nullptr, *v_pool = nullptr;       // attention: [pages * 64][kv_heads][Dp / Vp]; latent: [pages * 64][Lc + Rc] (k_pool); bf16 or fp32
+    size_t state_off = 0;                 // delta: first float of this run inside a state slot
 };
 
 struct DecoderModel {
@@ -41,6 +61,7 @@ struct DecoderModel {
     int W = 0, Wp = 0;                    // width, padded to 8
     int side_p = 0;                       // token-side width padded to 8
     std::vector<DecoderLayer> layers;
+    std::vector<DecoderRun> runs;         // in order
     __nv_bfloat16 *side_embed = nullptr, *final_norm = nullptr;
     DecLinear head;
     std::set<std::string> seen;
@@ -50,16 +71,26 @@ struct DecoderModel {
     size_t state_stride = 0;
     std::vector<int> free_tables;
     // many-row buffers; "act" ones are bf16 or (32-bit mode) fp32
-    void *xa = nullptr, *proj_a = nullptr, *q = nullptr, *mix = nullptr, *ff = nullptr, *ff2 = nullptr, *side_a = nullptr, *head_a = nullptr;
+    void *xa = nullptr, *proj_a = nullptr, *q = nullptr, *mix = nullptr, *ff = nullptr, *ff2 = nullptr, *side_a = nullptr, *head_a = nullptr, *cq = nullptr;
     float *y = nullptr, *proj_f = nullptr, *pack = nullptr, *tanh_w = nullptr, *decay = nullptr, *o = nullptr, *side_f = nullptr, *logits_rows = nullptr;
     int tanh_ld = 0;
+    // latent attention, long entries: visible cache rows and what they expand to
+    __nv_bfloat16 *ws_c = nullptr, *ws_kv = nullptr;
+    int ws_pages = 0, ws_window = 0;      // capacity (0: no layer uses it); largest window of the layers that use it (0: no window)
+    // routed experts: rows sorted by expert
+    void *ex_in = nullptr, *ex_act = nullptr;
+    float *ex_gu = nullptr, *ex_y = nullptr, *route_logits = nullptr;
+    ExpertRows ex{};
+    int ex_rows = 0;
     int32_t* step_buf = nullptr;          // packed per-step indices
     size_t step_words = 0;
     int max_want = 0;
-    float* tap = nullptr;                 // debugging / tests: residual stream after every layer [layers][rows][Wp]
+    float* tap = nullptr;                 // debugging / tests: residual stream after every layer run [runs][rows][Wp]
     int tap_rows = 0, tap_row0 = 0;
     // one-row buffers
     float *d_in = nullptr, *d_mix = nullptr, *d_y = nullptr, *d_y2 = nullptr, *d_ff = nullptr, *d_gate = nullptr;
+    float *d_q = nullptr, *d_h = nullptr, *d_route = nullptr, *d_act = nullptr, *d_route_w = nullptr;
+    int32_t* d_route_id = nullptr;
     int attn_cluster = 8, side_cluster = 1;
 };
 
@@ -71,6 +102,10 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
 struct RowTiles {
     const RowTile *tc = nullptr, *simt = nullptr, *all = nullptr;
     int n_tc = 0, n_simt = 0, n_all = 0;
+    // latent attention: rows of the short entries (absorbed form) and the cache pages the long entries see
+    const int32_t* short_rows = nullptr;
+    const RowTile* ws_pages = nullptr;
+    int n_short = 0, n_ws = 0, ws_page0 = 0;
     bool listed = false;
 };
 void decoder_rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const RowTiles& tiles, Launcher& L);
@@ -83,6 +118,8 @@ int decoder_simt_tile_rows();
 bool decoder_layer_tc(const DecoderModel& m, const DecoderLayer& l);
 // scratch of one recurrent layer for `rows` rows of at most `entries` sequences
 size_t decoder_delta_pack_floats(int heads, int dim, int rows, int entries);
-cudaError_t configure_decoder(DecoderModel& m);
+// first cache page (of its sequence) that a long entry at position pos0 needs in the workspace
+inline int decoder_ws_page0(const DecoderModel& m, int pos0) { return m.ws_window > 0 ? std::max(0, pos0 - m.ws_window + 1) / kPageTokens : 0; }
+cudaError_t configure_decoder(DecoderModel& m);      // after the layers are set up
 
 }  // namespace efm

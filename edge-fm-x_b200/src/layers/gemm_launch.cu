@@ -69,7 +69,7 @@ static void launch_gemm(Launcher& L, const GemmParams& p, int* error_word = null
         attr_set = true;
     }
     CUtensorMap ma, mb;
-    if (!make_tile_map(&ma, p.A, p.M, p.K, p.lda > 0 ? p.lda : p.K, tc::BM) || !make_tile_map(&mb, p.B, p.N, p.K, p.K, tc::BN)) {
+    if (!make_tile_map(&ma, p.A, p.M, p.K, p.lda > 0 ? p.lda : p.K, tc::BM) || !make_tile_map(&mb, p.B, p.group_tile != nullptr ? p.group_all : p.N, p.K, p.K, tc::BN)) {
         if (L.err == cudaSuccess) L.err = cudaErrorInvalidValue;
         return;
     }
@@ -77,6 +77,11 @@ static void launch_gemm(Launcher& L, const GemmParams& p, int* error_word = null
     const dim3 block(tc::kThreads);
     const bool pdl = L.pdl;
     L.pdl = false;     // prefill kernels do not use the dependent-launch protocol
+    if (p.group_tile != nullptr) {
+        L.launch(gemm_tc_kernel<EPI>, dim3(std::min(L.num_sms, tiles)), block, tc::SMEM_BYTES, ma, mb, p, error_word);
+        L.pdl = pdl;
+        return;
+    }
     // Few output tiles and a long K: split K so that the whole GPU works, fp32 partials to the workspace, then
     // a fixed-order sum with the epilogue.
     if constexpr (EPI == GemmEpi::Bf16Bias || EPI == GemmEpi::Residual || EPI == GemmEpi::F32 || EPI == GemmEpi::SwiGlu) {
@@ -159,8 +164,8 @@ void launch_rmsnorm_rows(Launcher& L, const float* x, const __nv_bfloat16* w, __
 }
 
 void launch_embed_rows(Launcher& L, const int32_t* ids, const __nv_bfloat16* table, const __nv_bfloat16* custom, float* out, int rows,
-                       int vocab, int hidden, int embed_token_id, int n_custom) {
-    L.launch(embed_rows_kernel, dim3(rows), dim3(128), 0, ids, table, custom, out, vocab, hidden, embed_token_id, n_custom);
+                       int vocab, int hidden, int embed_token_id, int n_custom, float scale) {
+    L.launch(embed_rows_kernel, dim3(rows), dim3(128), 0, ids, table, custom, out, vocab, hidden, embed_token_id, n_custom, scale);
 }
 
 void launch_gemm_epi(Launcher& L, GemmEpi epi, const GemmParams& p, int* error_word) {

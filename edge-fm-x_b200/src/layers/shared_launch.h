@@ -22,9 +22,9 @@ void launch_seg_attention(Launcher& L, const SegAttnParams& p, int D);
 void launch_seg_attention_short(Launcher& L, const SegAttnParams& p, int D, int max_keys);
 void launch_sample(Launcher& L, const SampleParams& p);
 cudaError_t configure_sampler();      // once per device at set-up, never inside a stream capture
-// out[r,:] = table[ids[r],:] (fp32), injected rows for ids in [embed_token_id, embed_token_id + n_custom).
+// out[r,:] = table[ids[r],:] * scale (fp32), injected rows for ids in [embed_token_id, embed_token_id + n_custom).
 void launch_embed_rows(Launcher& L, const int32_t* ids, const __nv_bfloat16* table, const __nv_bfloat16* custom, float* out, int rows,
-                       int vocab, int hidden, int embed_token_id, int n_custom);
+                       int vocab, int hidden, int embed_token_id, int n_custom, float scale = 1.0f);
 // y[r,:] = bf16(rmsnorm(x[r,:]) * w) over `rows` fp32 rows.
 void launch_rmsnorm_rows(Launcher& L, const float* x, const __nv_bfloat16* w, __nv_bfloat16* y, int rows, int hidden, float eps);
 void launch_prefill_attention(Launcher& L, const __nv_bfloat16* q, const __nv_bfloat16* k, const __nv_bfloat16* v,

@@ -27,30 +27,79 @@ __device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
     return make_float4(bf16lo(v.x), bf16hi(v.x), bf16lo(v.y), bf16hi(v.y));
 }
 
-// x += y / sqrt(mean(y^2) + eps) * w (y null: x unchanged); copy of x as T (null: none).  One block per row.
+// Where a row's sublayer output comes from: row i of y, or (experts) the weighted sum of the rows place[i][..] of y.
+struct SumOf {
+    const int32_t* place;             // [rows][top], null: the row itself
+    const float* weight;              // [rows][top]
+    int top;
+    int32_t* count;                   // rows per expert, zeroed for the next pass by block 0
+    int experts;
+};
+
+// x += y / sqrt(mean(y^2) + eps) * w (y null: x unchanged); out (null: none) = x as T, or with `pre` x / sqrt(mean(x^2) + eps) * pre,
+// the next sublayer's input.  One block per row; the first 1024 * KEEP channels stay in registers.
 template <typename T>
 __global__ void __launch_bounds__(256) add_norm_rows_kernel(float* __restrict__ x, const float* __restrict__ y, const __nv_bfloat16* __restrict__ w,
-                                                            T* __restrict__ copy, int n, int ld, float eps) {
-    __shared__ float part[8];
+                                                            T* __restrict__ out, const __nv_bfloat16* __restrict__ pre, int n, int ld, float eps,
+                                                            const SumOf sum) {
+    constexpr int KEEP = 4;
+    __shared__ float part[2][8];
     const size_t base = (size_t)blockIdx.x * ld;
-    const int nv = ld / 4;
+    const int nv = ld / 4, tid = threadIdx.x;
+    if (sum.count != nullptr && blockIdx.x == 0)
+        for (int e = tid; e < sum.experts; e += 256) sum.count[e] = 0;
+    auto load_y = [&](int c) {
+        if (sum.place == nullptr) return load4(y + base + 4 * c);
+        float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int k = 0; k < sum.top; ++k) {
+            const size_t i = (size_t)blockIdx.x * sum.top + k;
+            const float g = sum.weight[i];
+            const float4 v = load4(y + (size_t)sum.place[i] * ld + 4 * c);
+            a.x = fmaf(g, v.x, a.x); a.y = fmaf(g, v.y, a.y); a.z = fmaf(g, v.z, a.z); a.w = fmaf(g, v.w, a.w);
+        }
+        return a;
+    };
+    auto square = [](float s, const float4& v) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s)))); };
+    float4 keep[KEEP];
+    float s2 = 0.f;
     if (y != nullptr) {
         float ss = 0.f;
-        for (int c = threadIdx.x; c < nv; c += 256) {
-            const float4 v = load4(y + base + 4 * c);
-            ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
-        }
-        const float inv = 1.0f / sqrtf(block_sum_256(ss, part) / (float)n + eps);
-        for (int c = threadIdx.x; c < nv; c += 256) {
-            const float4 v = load4(y + base + 4 * c), g = load4(w + 4 * c);
+#pragma unroll
+        for (int i = 0; i < KEEP; ++i)
+            if (tid + 256 * i < nv) { keep[i] = load_y(tid + 256 * i); ss = square(ss, keep[i]); }
+        for (int c = tid + 256 * KEEP; c < nv; c += 256) ss = square(ss, load_y(c));
+        const float inv = 1.0f / sqrtf(block_sum_256(ss, part[0]) / (float)n + eps);
+        auto add = [&](int c, const float4& v) {
+            const float4 g = load4(w + 4 * c);
             float4 r = load4(x + base + 4 * c);
             r.x += v.x * inv * g.x; r.y += v.y * inv * g.y; r.z += v.z * inv * g.z; r.w += v.w * inv * g.w;
             store4(x + base + 4 * c, r);
-            if (copy != nullptr) store4(copy + base + 4 * c, r);
-        }
+            s2 = square(s2, r);
+            if (out != nullptr && pre == nullptr) store4(out + base + 4 * c, r);
+            return r;
+        };
+#pragma unroll
+        for (int i = 0; i < KEEP; ++i)
+            if (tid + 256 * i < nv) keep[i] = add(tid + 256 * i, keep[i]);
+        for (int c = tid + 256 * KEEP; c < nv; c += 256) (void)add(c, load_y(c));
     } else {
-        for (int c = threadIdx.x; c < nv; c += 256) store4(copy + base + 4 * c, load4(x + base + 4 * c));
+#pragma unroll
+        for (int i = 0; i < KEEP; ++i)
+            if (tid + 256 * i < nv) { keep[i] = load4(x + base + 4 * (tid + 256 * i)); s2 = square(s2, keep[i]); }
+        for (int c = tid + 256 * KEEP; c < nv; c += 256) s2 = square(s2, load4(x + base + 4 * c));
+        if (out != nullptr && pre == nullptr)
+            for (int c = tid; c < nv; c += 256) store4(out + base + 4 * c, load4(x + base + 4 * c));
     }
+    if (out == nullptr || pre == nullptr) return;
+    const float inv = 1.0f / sqrtf(block_sum_256(s2, part[1]) / (float)n + eps);
+    auto emit = [&](int c, const float4& v) {
+        const float4 g = load4(pre + 4 * c);
+        store4(out + base + 4 * c, make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w));
+    };
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+        if (tid + 256 * i < nv) emit(tid + 256 * i, keep[i]);
+    for (int c = tid + 256 * KEEP; c < nv; c += 256) emit(c, load4(x + base + 4 * c));
 }
 
 __device__ __forceinline__ void load8(const float* p, float (&f)[8]) {
@@ -136,12 +185,20 @@ __global__ void __launch_bounds__(256) gather_norm_rows_kernel(const float* __re
 }
 
 // C[M, N] = A[M, K] . W[N, K]^T in fp32 FMAs (fp32 activations, bf16 weights): the products of the all-32-bit mode and
-// the small ones that feed a recurrence.  64 x 64 tiles, 256 threads, 4 x 4 outputs per thread.
+// the small ones that feed a recurrence.  64 x 64 tiles, 256 threads, 4 x 4 outputs per thread.  bias may be null.  Grouped
+// (group.tile not null): rows sorted by group as in gemm_tc.cuh, rows [group of the tile * group.rows, + N) of W.
+struct RowGroups { const int32_t *tile, *n_tiles; int rows; };
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ W, int ldw,
-                                                       float* __restrict__ C, int ldc, int M, int N, int K) {
+                                                       float* __restrict__ C, int ldc, int M, int N, int K, const __nv_bfloat16* __restrict__ bias,
+                                                       const RowGroups group) {
     __shared__ float as[16][64 + 4], ws[16][64 + 4];
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
     const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+    if (group.tile != nullptr) {
+        const int t = m0 / kExpertTile;
+        if (t >= *group.n_tiles) return;
+        W += (size_t)group.tile[t] * group.rows * ldw;
+    }
     float acc[4][4];
 #pragma unroll
     for (int i = 0; i < 4; ++i)
@@ -173,7 +230,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
-            if (n < N) C[(size_t)m * ldc + n] = acc[i][j];
+            if (n < N) C[(size_t)m * ldc + n] = acc[i][j] + (bias != nullptr ? __bfloat162float(bias[n]) : 0.f);
         }
     }
 }

@@ -1,0 +1,21 @@
+// Routed experts: limits, the router's shape and where a pass keeps the rows' choices.
+#pragma once
+#include <stdint.h>
+
+namespace efm {
+
+constexpr int kMaxExperts = 512, kMaxExpertTop = 32, kMaxExpertGroups = 64;
+constexpr int kExpertTile = 128;      // rows of an expert start at multiples of this
+
+struct RouteShape { int experts, top, groups, keep; };
+
+struct ExpertRows {
+    int32_t* id;                      // [rows][top]
+    float* weight;                    // [rows][top]
+    int32_t* place;                   // [rows][top]: place among the expert's rows, then row of the sorted order
+    int32_t* count;                   // [experts], zero between passes
+    int32_t* tile_expert;             // [tiles]
+    int32_t* n_tiles;                 // tiles in use
+};
+
+}  // namespace efm

@@ -27,17 +27,19 @@
 // do not depend on the previous phase.
 #pragma once
 #include "common.cuh"
+#include "expert_route.cuh"
 
 namespace efm {
 
-enum class Epi : int { Plain = 0, Residual = 1, QkvRope = 2, SwiGlu = 3, Logits = 4, Peers = 5, Store32 = 6, TokenGate = 7 };
+enum class Epi : int { Plain = 0, Residual = 1, QkvRope = 2, SwiGlu = 3, Logits = 4, Peers = 5, Store32 = 6, TokenGate = 7, ExpertUp = 8, ExpertDown = 9 };
 constexpr int kMaxPeers = 8;
-// The last three (and the epilogues Store32, TokenGate) exist in the EXT instantiations only (layered decoders):
-//   Embed    x = embed_table[token], no norm
+// The last four (and the epilogues from Store32 on) exist in the EXT instantiations only (layered decoders):
+//   Embed    x = embed_table[token] * embed_scale; with norm2_w the product reads rmsnorm(x) * norm2_w
+//   Norm     x = rmsnorm(xf) * norm_w
 //   AddNorm  x = xr + rmsnorm(addend) * norm_w: a sublayer whose OUTPUT is normalised, folded into the next product;
 //            with norm2_w the product reads rmsnorm(x) * norm2_w instead of x
 //   PolyNorm x = c0 rms(z) + c1 rms(z^2) + c2 rms(z^3) + c3 with z = xf and the four numbers of `poly`
-enum : int { kProPlain = 0, kProRmsNorm = 1, kProEmbedRmsNorm = 2, kProEmbed = 3, kProAddNorm = 4, kProPolyNorm = 5 };
+enum : int { kProPlain = 0, kProRmsNorm = 1, kProEmbedRmsNorm = 2, kProEmbed = 3, kProAddNorm = 4, kProPolyNorm = 5, kProNorm = 6 };
 
 struct GemvParams {
     const __nv_bfloat16* W;   // [N, K] row-major
@@ -93,6 +95,16 @@ struct GemvParams {
     // TokenGate: out[n] = gelu_tanh(W x)[n] * gate_table[token][gate_off + n] for n < N, 0 beyond
     const __nv_bfloat16* gate_table;
     int gate_ld, gate_off;
+    float embed_scale;
+    float* x_out;             // not null: block 0 stores the input of the product here (what the norms left)
+    // ExpertUp: the experts of this token are chosen from route_logits (block 0 publishes ids and weights); item = (choice,
+    // channel), out_f[choice * ffp + channel] = silu(gate) * up.  ExpertDown: x = the choices' activations times their
+    // weights, K = choices * ffp, the row of W jumps from expert to expert.
+    RouteShape route;
+    const float* route_logits;
+    int32_t* route_id;        // [top]
+    float* route_w;           // [top]
+    int ff, ffp, expert_rows; // channels, padded channels, rows of one expert's matrix
 };
 
 __device__ __forceinline__ float gelu_tanh(float z) {
@@ -117,7 +129,8 @@ __device__ __forceinline__ void group_barrier(int id, int nthreads) {
 }
 
 template <Epi EPI>
-__device__ __forceinline__ void item_rows(const GemvParams& p, int item, int& r0, int& r1) {
+__device__ __forceinline__ void item_rows(const GemvParams& p, int item, int& r0, int& r1, const int* chosen = nullptr) {
+    (void)chosen;
     if constexpr (EPI == Epi::QkvRope) {
         const int half = p.head_dim >> 1;
         const int head = item / half, d = item - head * half;
@@ -126,6 +139,10 @@ __device__ __forceinline__ void item_rows(const GemvParams& p, int item, int& r0
     } else if constexpr (EPI == Epi::SwiGlu) {
         // fused weight: blocks of 64 gate rows followed by the 64 matching up rows
         r0 = ((item >> 6) << 7) + (item & 63);
+        r1 = r0 + 64;
+    } else if constexpr (EPI == Epi::ExpertUp) {
+        const int k = item / p.ff, j = item - k * p.ff;
+        r0 = chosen[k] * p.expert_rows + ((j >> 6) << 7) + (j & 63);
         r1 = r0 + 64;
     } else {
         r0 = item * 2;
@@ -159,7 +176,16 @@ __device__ __forceinline__ void item_epilogue(const GemvParams& p, int item, flo
         if (item * 2 + 1 >= p.N) a1 = -INFINITY;
         if (a0 > best_v) { best_v = a0; best_i = item * 2; }          // ascending ids: strict > keeps
         if (a1 > best_v) { best_v = a1; best_i = item * 2 + 1; }      // the lowest id on ties
+    } else if constexpr (EPI == Epi::ExpertUp) {
+        const int k = item / p.ff;
+        p.out_f[k * p.ffp + item - k * p.ff] = a0 / (1.0f + expf(-a0)) * a1;
+    } else if constexpr (EPI == Epi::ExpertDown) {
+        *reinterpret_cast<float2*>(p.out_f + item * 2) = make_float2(a0, a1);
     } else if constexpr (EPI == Epi::Store32) {
+        if (p.bias != nullptr) {
+            a0 += __bfloat162float(p.bias[item * 2]);
+            a1 += __bfloat162float(p.bias[item * 2 + 1]);
+        }
         *reinterpret_cast<float2*>(p.out_f + item * 2) = make_float2(a0, a1);
     } else if constexpr (EPI == Epi::TokenGate) {
         const int n = item * 2, tok = p.state->token;
@@ -245,11 +271,25 @@ __device__ __forceinline__ GemvSched gemv_sched(const GemvParams& p, const int k
 }
 
 template <Epi EPI>
-__device__ __forceinline__ void gemv_load_unit(const GemvParams& p, const GemvSched& sc, const int u, uint4 (&buf)[kGemvU][2]) {
+__device__ __forceinline__ void gemv_load_unit(const GemvParams& p, const GemvSched& sc, const int u, uint4 (&buf)[kGemvU][2], const int* chosen = nullptr) {
     if (u >= sc.total) return;
     const int j = u / sc.upi, part = u - j * sc.upi;
     int r0, r1;
-    item_rows<EPI>(p, sc.ig0 + j * sc.ig_stride, r0, r1);
+    item_rows<EPI>(p, sc.ig0 + j * sc.ig_stride, r0, r1, chosen);
+    if constexpr (EPI == Epi::ExpertDown) {
+        const int per = p.ffp >> 3;                                   // chunks of one expert's row
+#pragma unroll
+        for (int uu = 0; uu < kGemvU; ++uu) {
+            const int c = (part * kGemvU + uu) * sc.stride + sc.gl;
+            if (c < sc.nch) {
+                const int k = c / per;
+                const __nv_bfloat16* w = p.W + ((size_t)chosen[k] * p.expert_rows + r0) * p.ffp + (size_t)(c - k * per) * 8;
+                buf[uu][0] = ld_stream(w);
+                buf[uu][1] = ld_stream(w + p.ffp);
+            }
+        }
+        return;
+    }
     const __nv_bfloat16* a = p.W + (size_t)r0 * p.K;
     const __nv_bfloat16* b = p.W + (size_t)r1 * p.K;
 #pragma unroll
@@ -270,8 +310,8 @@ __host__ __device__ inline unsigned int gemv_wbytes(int K) { return ((unsigned i
 template <Epi EPI, bool EXT>
 __device__ __forceinline__ void gemv_prefetch(const GemvParams& p, const GemvSched& sc, GemvRegs& r, unsigned char* smem,
                                               const unsigned int xbytes) {
-    gemv_load_unit<EPI>(p, sc, 0, r.a);
-    if (EXT ? p.prologue == kProAddNorm : p.prologue != kProPlain) {
+    if constexpr (EPI != Epi::ExpertUp && EPI != Epi::ExpertDown) gemv_load_unit<EPI>(p, sc, 0, r.a);
+    if (EXT ? (p.prologue == kProAddNorm || p.prologue == kProNorm) : p.prologue != kProPlain) {
         uint4* gs = reinterpret_cast<uint4*>(smem + xbytes);        // xbytes = gemv_xbytes(K)
         for (int c = threadIdx.x; c < sc.nch; c += kGemvThreads) gs[c] = ld_cached(p.norm_w + (size_t)c * 8);
     }
@@ -312,6 +352,20 @@ __device__ __forceinline__ bool gemv_stage_ext(const GemvParams& p, const int nc
     __shared__ float red3[3 * kGemvWarps];
     float* xs = reinterpret_cast<float*>(smem);
     const int tid = threadIdx.x;
+    float sq[1] = {0.f};
+    // the second norm: the product reads rmsnorm(x) * norm2_w
+    auto norm2 = [&](float (&s2)[1]) {
+        gemv_block_sums<1>(s2, red3 + kGemvWarps);
+        const float inv2 = 1.0f / sqrtf(s2[0] / (float)p.k_true + p.eps);
+        for (int c = tid; c < nch; c += kGemvThreads) {
+            float w[8], x[8];
+            unpack8(ld_cached(p.norm2_w + (size_t)c * 8), w);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) x[j] = xs[8 * c + j] * inv2 * w[j];
+            st8f(xs + 8 * c, x);
+            if (p.x_out != nullptr && blockIdx.x == 0) st8f(p.x_out + 8 * c, x);
+        }
+    };
     if (p.prologue == kProEmbed) {
         const int tok = p.state->token;
         const bool zero = tok < 0 || tok >= p.vocab;
@@ -319,8 +373,32 @@ __device__ __forceinline__ bool gemv_stage_ext(const GemvParams& p, const int nc
         for (int c = tid; c < nch; c += kGemvThreads) {
             float f[8];
             unpack8(zero ? make_uint4(0, 0, 0, 0) : ld_cached(row + (size_t)c * 8), f);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                f[j] *= p.embed_scale;
+                sq[0] = fmaf(f[j], f[j], sq[0]);
+            }
             st8f(xs + 8 * c, f);
             if (blockIdx.x == 0) st8f(p.resid_out + 8 * c, f);
+        }
+        if (p.norm2_w != nullptr) norm2(sq);
+    } else if (p.prologue == kProNorm) {
+        const uint4* gs = reinterpret_cast<const uint4*>(smem + xbytes);
+        for (int c = tid; c < nch; c += kGemvThreads) {
+            float f[8];
+            ld8f(p.xf + 8 * c, f);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) sq[0] = fmaf(f[j], f[j], sq[0]);
+            st8f(xs + 8 * c, f);
+        }
+        gemv_block_sums<1>(sq, red3);
+        const float inv = 1.0f / sqrtf(sq[0] / (float)p.k_true + p.eps);
+        for (int c = tid; c < nch; c += kGemvThreads) {
+            float w[8], x[8];
+            unpack8(gs[c], w);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) x[j] = xs[8 * c + j] * inv * w[j];
+            st8f(xs + 8 * c, x);
         }
     } else if (p.prologue == kProAddNorm) {
         const uint4* gs = reinterpret_cast<const uint4*>(smem + xbytes);
@@ -349,17 +427,7 @@ __device__ __forceinline__ bool gemv_stage_ext(const GemvParams& p, const int nc
             st8f(xs + 8 * c, x);
             if (blockIdx.x == 0) st8f(p.resid_out + 8 * c, x);
         }
-        if (p.norm2_w != nullptr) {
-            gemv_block_sums<1>(s2, red3 + kGemvWarps);
-            const float inv2 = 1.0f / sqrtf(s2[0] / (float)p.k_true + p.eps);
-            for (int c = tid; c < nch; c += kGemvThreads) {
-                float w[8], x[8];
-                unpack8(ld_cached(p.norm2_w + (size_t)c * 8), w);
-#pragma unroll
-                for (int j = 0; j < 8; ++j) x[j] = xs[8 * c + j] * inv2 * w[j];
-                st8f(xs + 8 * c, x);
-            }
-        }
+        if (p.norm2_w != nullptr) norm2(s2);
     } else if (p.prologue == kProPolyNorm) {
         float s[3] = {0.f, 0.f, 0.f};
         for (int c = tid; c < nch; c += kGemvThreads) {
@@ -510,7 +578,30 @@ __device__ __forceinline__ void gemv_run(const GemvParams& p, const GemvSched& s
         if (sc.wk == 0 && lane == 0 && sc.total > 0)
             old_first = __ldcg(reinterpret_cast<const float2*>(p.residual + sc.ig0 * 2));
     }
-    if constexpr (EXT) {
+    __shared__ int chosen_s[EPI == Epi::ExpertUp || EPI == Epi::ExpertDown ? kMaxExpertTop : 1];
+    const int* chosen = nullptr;
+    if constexpr (EPI == Epi::ExpertUp) {
+        if (warp == 0)
+            route_token(p.route_logits, p.route, [&](int k, int e, float w) {
+                chosen_s[k] = e;
+                if (blockIdx.x == 0) { p.route_id[k] = e; p.route_w[k] = w; }
+            });
+        chosen = chosen_s;
+        gemv_stage(p, nch, smem, xbytes);                              // ends with a block barrier
+        gemv_load_unit<EPI>(p, sc, 0, r.a, chosen);
+    } else if constexpr (EPI == Epi::ExpertDown) {
+        if (tid < p.route.top) chosen_s[tid] = __ldcg(p.route_id + tid);
+        chosen = chosen_s;
+        __syncthreads();
+        gemv_load_unit<EPI>(p, sc, 0, r.a, chosen);
+        float* xw = reinterpret_cast<float*>(smem);
+        for (int c = tid; c < 2 * nch; c += kGemvThreads) {            // padded channels are zero
+            const float w = __ldcg(p.route_w + 4 * c / p.ffp);
+            const float4 v = __ldcg(reinterpret_cast<const float4*>(p.xf) + c);
+            reinterpret_cast<float4*>(xw)[c] = make_float4(v.x * w, v.y * w, v.z * w, v.w * w);
+        }
+        __syncthreads();
+    } else if constexpr (EXT) {
         if (!gemv_stage_ext(p, nch, smem, xbytes)) gemv_stage(p, nch, smem, xbytes);
     } else {
         gemv_stage(p, nch, smem, xbytes);
@@ -559,7 +650,7 @@ __device__ __forceinline__ void gemv_run(const GemvParams& p, const GemvSched& s
         }
     };
     for (int u = 0; u < sc.total; ++u) {
-        if (u > 0) gemv_load_unit<EPI>(p, sc, u, r.a);       // unit 0 was fetched before the dependency wait
+        if (u > 0) gemv_load_unit<EPI>(p, sc, u, r.a, chosen);       // unit 0 was fetched before the dependency wait
         compute_unit(u, r.a);
     }
 }

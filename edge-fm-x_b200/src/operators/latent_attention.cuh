@@ -1,0 +1,447 @@
+// Latent attention over a paged cache: keys and values of all heads are linear in one cached latent c per token,
+//   k[h] = [Wk[h] c | r],  v[h] = Wv[h] c,  score = (q[h] . k[h]) * scale,
+// r a rotated key part shared by the heads; sliding window, an optional extra term exp(sink[h]) in the softmax denominator,
+// heads multiplied by sigmoid(gate).  A cache row is [c: Lc | r: Rc] (Lc, Rc: kv_rank, rot_dim padded to 8 with zeros), normed
+// and rotated.  The projections arrive as one row [query latent: Qp | c: Lc | r: Rc | gate: H * Dv].
+//
+//   latent_rows          many rows: norms of the two latents, rotation of r, cache append
+//   latent_rotate_rows   many rows: rotation of the queries' rotated part, in place
+//   latent_gather_rows   long entries: the visible cache rows of every entry into a contiguous workspace; one product expands
+//                        them to keys and values of all heads, and the tensor-core attention (window_attention_tc.cuh) reads those
+//   latent_attention     one row per cluster, absorbed form: the query is moved into the latent space (qa = Wk[h]^T q), scores and
+//                        sums run over the cached rows as they are, the result goes through Wv[h] and the gate: decode steps,
+//                        short portions and the 32-bit mode.  Nothing per-head is ever stored for a key.
+#pragma once
+#include <cooperative_groups.h>
+
+#include <utility>
+
+#include "common.cuh"
+#include "rotary.cuh"
+#include "row_plan.cuh"
+#include "window_attention.cuh"
+
+namespace efm {
+
+struct LatentShape {
+    int H, D, R, Dv, L;               // heads, unrotated and rotated query channels, value channels, latent width
+    int Dp, Vp, Qp, Lc, Rc;           // padded to 8; Qp: query latent
+    int q_rank, window;
+    float scale, eps;
+    RotShape rot;                     // of the R channels
+    const __nv_bfloat16* q_norm;      // [Qp]
+    const __nv_bfloat16* kv_norm;     // [Lc]
+    const __nv_bfloat16* sink;        // [H] or null
+    const __nv_bfloat16* wk;          // [H * Dp][Lc]
+    const __nv_bfloat16* wv;          // [H * Vp][Lc]
+    int gate;                         // 1: the projections end with the gate
+    __host__ __device__ int off_c() const { return Qp; }
+    __host__ __device__ int off_r() const { return Qp + Lc; }
+    __host__ __device__ int off_gate() const { return Qp + Lc + Rc; }
+    __host__ __device__ int q_ld() const { return H * (Dp + Rc); }
+};
+
+// ---- many rows -----------------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256) latent_rows_kernel(const T* __restrict__ proj, int ld, T* __restrict__ cq, T* __restrict__ pool, const LatentShape s,
+                                                          const RowPlan plan) {
+    __shared__ float part[2][8], cs[kRotMaxPairs], sn[kRotMaxPairs], rot[256];
+    const int row = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const RowEntry e = plan.of_row(row);
+    const int pos = e.pos0 + row - e.row0;
+    const T* src = proj + (size_t)row * ld;
+    T* dst = pool + plan.cache_row(e, pos) * (s.Lc + s.Rc);
+    rot_table(s.rot, pos, cs, sn);
+    float a = 0.f, b = 0.f;                                             // pads are zero
+    for (int c = tid; c < s.Qp; c += 256) { const float v = to_f32(src[c]); a = fmaf(v, v, a); }
+    for (int c = tid; c < s.Lc; c += 256) { const float v = to_f32(src[s.off_c() + c]); b = fmaf(v, v, b); }
+    for (int c = tid; c < s.Rc; c += 256) rot[c] = to_f32(src[s.off_r() + c]);
+    a = warp_sum(a);
+    b = warp_sum(b);
+    if (lane == 0) { part[0][warp] = a; part[1][warp] = b; }
+    __syncthreads();
+    a = b = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) { a += part[0][i]; b += part[1][i]; }
+    const float ia = 1.0f / sqrtf(a / (float)s.q_rank + s.eps), ib = 1.0f / sqrtf(b / (float)s.L + s.eps);
+    for (int c = tid; c < s.Qp; c += 256) store_f32(cq + (size_t)row * s.Qp + c, to_f32(src[c]) * ia * __bfloat162float(s.q_norm[c]));
+    for (int c = tid; c < s.Lc; c += 256) store_f32(dst + c, to_f32(src[s.off_c() + c]) * ib * __bfloat162float(s.kv_norm[c]));
+    for (int c = tid; c < s.Rc; c += 256) store_f32(dst + s.Lc + c, rot_channel(s.rot, rot, c, cs, sn));
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) latent_rotate_rows_kernel(T* __restrict__ q, const LatentShape s, const RowPlan plan) {
+    __shared__ float cs[kRotMaxPairs], sn[kRotMaxPairs];
+    const int row = blockIdx.x, pairs = s.rot.dims / 2;
+    const RowEntry e = plan.of_row(row);
+    rot_table(s.rot, e.pos0 + row - e.row0, cs, sn);
+    __syncthreads();
+    const int step = s.rot.kind == kRotHalf ? 1 : 2, apart = s.rot.kind == kRotHalf ? pairs : 1;
+    for (int n = threadIdx.x; n < s.H * pairs; n += 256) {
+        const int h = n / pairs, i = n - h * pairs;
+        T* x = q + (size_t)row * s.q_ld() + (size_t)h * (s.Dp + s.Rc) + s.Dp + i * step;
+        const float u = to_f32(x[0]), v = to_f32(x[apart]);
+        store_f32(x, u * cs[i] - v * sn[i]);
+        store_f32(x + apart, v * cs[i] + u * sn[i]);
+    }
+}
+
+// One block per page: pages[i] = (entry, page of its sequence); null: page0 + i of the single entry.
+template <typename T>
+__global__ void __launch_bounds__(256) latent_gather_rows_kernel(const T* __restrict__ pool, T* __restrict__ ws, int row_elems, const RowPlan plan,
+                                                                 const RowTile* __restrict__ pages, int page0) {
+    const RowTile t = pages != nullptr ? pages[blockIdx.x] : RowTile{0, page0 + (int)blockIdx.x};
+    const RowEntry e = plan.entry(t.entry);
+    const uint4* src = reinterpret_cast<const uint4*>(pool + plan.cache_row(e, t.row * kPageTokens) * row_elems);
+    uint4* dst = reinterpret_cast<uint4*>(ws + (size_t)(e.ws0 + t.row * kPageTokens) * row_elems);
+    // rows past the entry's last token hold what an earlier owner of the page left: any finite values, never visible
+    const int n = min(kPageTokens, e.pos0 + e.n - t.row * kPageTokens), per = row_elems * (int)sizeof(T) / 16;
+    for (int i = threadIdx.x; i < kPageTokens * per; i += 256) dst[i] = i < n * per ? src[i] : make_uint4(0, 0, 0, 0);
+}
+
+// ---- one row, absorbed -----------------------------------------------------------------------------------------------
+namespace la {
+constexpr int kThreads = 256;
+struct Layout {
+    int kt, ldk, slice;               // keys per tile, elements between key rows, latent channels per block of the cluster
+    unsigned int q, qin, cnew, keys, scr, rout, olat, bytes;
+};
+// Shared memory of one block: heads per block, cluster width, bytes per cache element.
+__host__ __device__ inline Layout layout(const LatentShape& s, int nh, int splits, int es, int kt) {
+    Layout l;
+    l.kt = kt;
+    l.ldk = s.Lc + s.Rc + 16 / es;
+    l.slice = (s.Lc / 8 + splits - 1) / splits * 8;
+    unsigned int at = 0;
+    auto take = [&](unsigned int bytes) { const unsigned int a = at; at = (at + bytes + 15u) & ~15u; return a; };
+    l.q = take((unsigned int)nh * (s.Lc + s.Rc) * 4u);
+    l.qin = take((unsigned int)nh * (s.Dp + s.Rc) * 4u);
+    l.cnew = take((unsigned int)(s.Lc + s.Rc) * 4u);
+    const unsigned int kb = 2u * kt * l.ldk * es, rb = (unsigned int)nh * 1024u * 4u;       // keys; afterwards sums of the key groups
+    l.keys = take(kb > rb ? kb : rb);
+    l.scr = take(kThreads * 8u * 4u);
+    l.rout = take((unsigned int)splits * nh * l.slice * 4u);
+    l.olat = take((unsigned int)nh * s.Lc * 4u);
+    l.bytes = at;
+    return l;
+}
+}  // namespace la
+
+template <typename TC, typename TI, typename TO>
+struct LatentParams {
+    LatentShape s;
+    const TI* q;                      // [rows][H][Dp + Rc]; decode: not rotated yet
+    const TI* proj;                   // [rows][ld]
+    int ld;
+    TC* pool;                         // [pages * 64][Lc + Rc]
+    TO* out;                          // [rows][ld_out]
+    int ld_out, kt;
+    // many rows: the plan and the rows to compute (null: all)
+    RowPlan plan;
+    const int32_t* rows;
+    // one row (decode)
+    const int32_t* pages;
+    int max_pages, early;
+    DecodeState* state;
+};
+
+// grid (cluster width, ceil(H / NH), rows).  The blocks of a cluster share the visible keys, the latent channels of the query
+// and of the result, and the value rows.
+template <typename TC, bool DECODE, int NH>
+__global__ void __launch_bounds__(la::kThreads) latent_attention_kernel(const LatentParams<TC, typename std::conditional<DECODE, float, TC>::type,
+                                                                                           typename std::conditional<DECODE, float, TC>::type> p) {
+    namespace cg = cooperative_groups;
+    using namespace la;
+    using TI = typename std::conditional<DECODE, float, TC>::type;
+    extern __shared__ __align__(16) unsigned char la_smem[];
+    __shared__ float cs[kRotMaxPairs], sn[kRotMaxPairs], part[8], sp[NH][64], sal[NH], sm_m[NH], sm_l[NH], rm[16][NH], rl[16][NH];
+    const LatentShape& s = p.s;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, split = blockIdx.x, n_splits = gridDim.x;
+    const int h0 = blockIdx.y * NH, nh = min(NH, s.H - h0), LR = s.Lc + s.Rc;
+    const Layout l = layout(s, NH, n_splits, sizeof(TC), p.kt);
+    float* q = reinterpret_cast<float*>(la_smem + l.q);
+    float* qin = reinterpret_cast<float*>(la_smem + l.qin);
+    float* cnew = reinterpret_cast<float*>(la_smem + l.cnew);
+    TC* keys = reinterpret_cast<TC*>(la_smem + l.keys);
+    float* red = reinterpret_cast<float*>(la_smem + l.keys);
+    float* scr = reinterpret_cast<float*>(la_smem + l.scr);
+    float* rout = reinterpret_cast<float*>(la_smem + l.rout);
+    float* olat = reinterpret_cast<float*>(la_smem + l.olat);
+    cg::cluster_group cl = cg::this_cluster();
+    auto started = cl.barrier_arrive();                                // waited for before the first store into another block
+
+    const int s0 = min(split * l.slice, s.Lc), s1 = min(s0 + l.slice, s.Lc), sl8 = (s1 - s0) / 8;
+    const int n_val = nh * s.Dv, vals = (n_val + n_splits - 1) / n_splits, v0 = split * vals, v1 = min(n_val, v0 + vals);
+    auto to_l2 = [](const void* a) { asm volatile("prefetch.global.L2 [%0];" ::"l"(a)); };
+    if constexpr (DECODE) {                                            // weights of this block on their way
+        const int lines = ((s1 - s0) * 2 + 127) / 128;
+        for (int i = tid; i < nh * s.Dp * lines; i += kThreads) to_l2(s.wk + ((size_t)h0 * s.Dp + i / lines) * s.Lc + s0 + (i % lines) * 64);
+        const int vl = (s.Lc * 2 + 127) / 128;
+        for (int i = tid; i < (v1 - v0) * vl; i += kThreads) {
+            const int v = v0 + i / vl;
+            to_l2(s.wv + ((size_t)(h0 + v / s.Dv) * s.Vp + v % s.Dv) * s.Lc + (i % vl) * 64);
+        }
+        if (!p.early) { pdl_wait(); pdl_launch_dependents(); }
+    }
+    const int row = DECODE ? 0 : (p.rows != nullptr ? p.rows[blockIdx.z] : (int)blockIdx.z);
+    RowEntry e{};
+    int pos;
+    bool ok = true;
+    const int32_t* pages;
+    if constexpr (DECODE) {
+        const int kv_len = (int)p.state->kv_len;
+        ok = kv_len > 0 && kv_len <= p.max_pages * kPageTokens;
+        pos = kv_len - 1;
+        pages = p.pages;
+    } else {
+        e = p.plan.of_row(row);
+        pos = e.pos0 + row - e.row0;
+        pages = p.plan.page_table + (size_t)e.table * p.plan.max_pages;
+    }
+    const int lo = s.window > 0 ? max(0, pos + 1 - s.window) : 0, n_vis = pos + 1 - lo;
+    const int chunk = ok ? (n_vis + n_splits - 1) / n_splits : 0;
+    const int begin = lo + split * chunk, end = ok ? min(pos + 1, begin + chunk) : begin;
+    const int n_tiles = end > begin ? (end - begin + l.kt - 1) / l.kt : 0;
+    const bool append = DECODE && n_tiles > 0 && end == pos + 1;       // this block walks the newest key
+    auto pool_row = [&](int j) { return (size_t)pages[j / kPageTokens] * kPageTokens + j % kPageTokens; };
+    const int per = LR * (int)sizeof(TC) / 16;                         // 16-byte pieces of a cache row
+    auto load_tile = [&](int t) {
+        if (t < n_tiles) {
+            const int j0 = begin + t * l.kt;
+            TC* dst = keys + (size_t)(t & 1) * l.kt * l.ldk;
+            for (int i = tid; i < l.kt * per; i += kThreads) {
+                const int r = i / per, c = i - r * per, j = j0 + r;
+                if (j < end && !(DECODE && j == pos))
+                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst + (size_t)r * l.ldk) + 16u * c),
+                                 "l"(reinterpret_cast<const char*>(p.pool + pool_row(j) * LR) + 16 * c) : "memory");
+            }
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    load_tile(0);
+    load_tile(1);
+    if (ok) rot_table(s.rot, pos, cs, sn);
+    if constexpr (DECODE) {
+        if (p.early) { pdl_wait(); pdl_launch_dependents(); }
+    }
+
+    // ---- this token's queries (and, decode, its cache row) -------------------------------------------------------------
+    const int qw = s.Dp + s.Rc;
+    for (int i = tid; i < nh * qw; i += kThreads) {
+        const TI* src = p.q + (size_t)row * s.q_ld() + (size_t)h0 * qw + i;
+        if constexpr (DECODE) qin[i] = __ldcg(src); else qin[i] = to_f32(*src);
+    }
+    float ss = 0.f;
+    if constexpr (DECODE) {
+        for (int c = tid; c < LR; c += kThreads) {
+            const float v = __ldcg(reinterpret_cast<const float*>(p.proj) + s.off_c() + c);
+            cnew[c] = v;
+            if (c < s.Lc) ss = fmaf(v, v, ss);
+        }
+        ss = warp_sum(ss);
+        if (lane == 0) part[warp] = ss;
+    }
+    if (tid < NH) { sm_m[tid] = -INFINITY; sm_l[tid] = 0.f; }
+    __syncthreads();
+    for (int i = tid; i < nh * s.Rc; i += kThreads) {
+        const int h = i / s.Rc, c = i - h * s.Rc;
+        q[h * LR + s.Lc + c] = (DECODE ? rot_channel(s.rot, qin + h * qw + s.Dp, c, cs, sn) : qin[h * qw + s.Dp + c]) * s.scale;
+    }
+    if constexpr (DECODE) {
+        if (append) {
+            ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < 8; ++i) ss += part[i];
+            const float inv = 1.0f / sqrtf(ss / (float)s.L + s.eps);
+            const int t = n_tiles - 1;
+            TC* mine = keys + (size_t)(t & 1) * l.kt * l.ldk + (size_t)(pos - begin - t * l.kt) * l.ldk;
+            // from the third tile on the row is written when the tile's turn comes: another tile still uses the buffer
+            TC* dst = p.pool + pool_row(pos) * LR;
+            for (int c = tid; c < LR; c += kThreads) {
+                const float v = c < s.Lc ? cnew[c] * inv * __bfloat162float(s.kv_norm[c]) : rot_channel(s.rot, cnew + s.Lc, c - s.Lc, cs, sn);
+                if (t < 2) store_f32(mine + c, v);
+                if (blockIdx.y == 0) store_f32(dst + c, v);
+                scr[c] = v;                                            // at most kThreads * 8 channels
+            }
+            __syncthreads();
+            for (int c = tid; c < LR; c += kThreads) cnew[c] = scr[c];
+            __syncthreads();
+        }
+    }
+
+    // ---- the queries in the latent space: this block's channels for all of its heads, sent to every block ------------------
+    {
+        const int cols = nh * sl8;                                     // 8-channel columns
+        int dl = 1;
+        while (dl * 2 * cols <= kThreads && dl < 32) dl *= 2;
+        const int wide = kThreads / dl;
+        cl.barrier_wait(std::move(started));
+        for (int c0 = 0; c0 < cols; c0 += wide) {
+            const int c = c0 + tid % wide, d0 = tid / wide;
+            float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+            if (c < cols) {
+                const int h = c / sl8;
+                const __nv_bfloat16* w = s.wk + (size_t)(h0 + h) * s.Dp * s.Lc + s0 + (c - h * sl8) * 8;
+#pragma unroll 4
+                for (int d = d0; d < s.Dp; d += dl) {
+                    float f[8];
+                    unpack8(ld_cached(w + (size_t)d * s.Lc), f);
+                    const float x = qin[h * qw + d];
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) acc[j] = fmaf(x, f[j], acc[j]);
+                }
+            }
+            __syncthreads();
+#pragma unroll
+            for (int j = 0; j < 8; ++j) scr[tid * 8 + j] = acc[j];
+            __syncthreads();
+            for (int i = tid; i < min(wide, cols - c0) * 8; i += kThreads) {
+                float v = 0.f;
+                for (int d = 0; d < dl; ++d) v += scr[(d * wide) * 8 + i];
+                const int cc = c0 + i / 8, h = cc / sl8, ch = s0 + (cc - h * sl8) * 8 + (i & 7);
+                v *= s.scale;
+                if (n_splits == 1) q[h * LR + ch] = v;
+                else
+                    for (int r = 0; r < n_splits; ++r) *cl.map_shared_rank(q + h * LR + ch, r) = v;
+            }
+        }
+    }
+    if (n_splits > 1) cl.sync(); else __syncthreads();
+
+    // ---- attention over this block's keys ----------------------------------------------------------------------------------
+    const int parts = kThreads / l.kt, key = tid / parts, pt = tid % parts;
+    const int tpr = s.Lc / 4, kg = kThreads / tpr, dpart = tid % tpr, tg = tid / tpr;
+    const bool pv = tg < kg;
+    float acc[NH][4];
+#pragma unroll
+    for (int h = 0; h < NH; ++h)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[h][j] = 0.f;
+    for (int t = 0; t < n_tiles; ++t) {
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        TC* kt = keys + (size_t)(t & 1) * l.kt * l.ldk;
+        const int j0 = begin + t * l.kt;
+        if (append && t >= 2 && t == n_tiles - 1)
+            for (int c = tid; c < LR; c += kThreads) store_f32(kt + (size_t)(pos - j0) * l.ldk + c, cnew[c]);
+        __syncthreads();
+        const bool vis = j0 + key < end;
+        float d[NH];
+#pragma unroll
+        for (int h = 0; h < NH; ++h) d[h] = 0.f;
+        if (vis) {
+            for (int c = pt; c < LR / 8; c += parts) {
+                float f[8];
+                load8_as_f32(kt + (size_t)key * l.ldk + c * 8, f);
+#pragma unroll
+                for (int h = 0; h < NH; ++h)
+                    if (h < nh) {
+                        const float4 a = *reinterpret_cast<const float4*>(q + h * LR + c * 8), b = *reinterpret_cast<const float4*>(q + h * LR + c * 8 + 4);
+                        d[h] = fmaf(a.x, f[0], d[h]); d[h] = fmaf(a.y, f[1], d[h]); d[h] = fmaf(a.z, f[2], d[h]); d[h] = fmaf(a.w, f[3], d[h]);
+                        d[h] = fmaf(b.x, f[4], d[h]); d[h] = fmaf(b.y, f[5], d[h]); d[h] = fmaf(b.z, f[6], d[h]); d[h] = fmaf(b.w, f[7], d[h]);
+                    }
+            }
+        }
+#pragma unroll
+        for (int h = 0; h < NH; ++h) {
+            for (int x = parts / 2; x > 0; x >>= 1) d[h] += __shfl_xor_sync(0xffffffffu, d[h], x);
+            if (pt == 0) sp[h][key] = vis && h < nh ? d[h] : -INFINITY;
+        }
+        __syncthreads();
+        if (warp < nh) {
+            const float x0 = lane < l.kt ? sp[warp][lane] : -INFINITY, x1 = lane + 32 < l.kt ? sp[warp][lane + 32] : -INFINITY;
+            const float mo = sm_m[warp], mn = fmaxf(mo, warp_max(fmaxf(x0, x1)));       // the tile holds a visible key
+            const float p0 = expf(x0 - mn), p1 = expf(x1 - mn);
+            sp[warp][lane] = p0;
+            sp[warp][lane + 32] = p1;
+            const float sum = warp_sum(p0 + p1);
+            if (lane == 0) {
+                const float al = expf(mo - mn);
+                sal[warp] = al;
+                sm_m[warp] = mn;
+                sm_l[warp] = sm_l[warp] * al + sum;
+            }
+        }
+        __syncthreads();
+        if (pv) {
+#pragma unroll
+            for (int h = 0; h < NH; ++h)
+                if (h < nh) {
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) acc[h][j] *= sal[h];
+                }
+            const int n = min(l.kt, end - j0);
+            for (int kk = tg; kk < n; kk += kg) {
+                const float4 v = load4_as_f32(kt + (size_t)kk * l.ldk + dpart * 4);
+#pragma unroll
+                for (int h = 0; h < NH; ++h)
+                    if (h < nh) {
+                        const float w = sp[h][kk];
+                        acc[h][0] = fmaf(w, v.x, acc[h][0]); acc[h][1] = fmaf(w, v.y, acc[h][1]);
+                        acc[h][2] = fmaf(w, v.z, acc[h][2]); acc[h][3] = fmaf(w, v.w, acc[h][3]);
+                    }
+            }
+        }
+        __syncthreads();
+        load_tile(t + 2);
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    // ---- sums over the key groups, then over the cluster: every latent channel belongs to one block ------------------------
+    if (pv) {
+#pragma unroll
+        for (int h = 0; h < NH; ++h)
+            *reinterpret_cast<float4*>(red + ((size_t)tg * NH + h) * s.Lc + dpart * 4) = make_float4(acc[h][0], acc[h][1], acc[h][2], acc[h][3]);
+    }
+    __syncthreads();
+    for (int i = tid; i < nh * s.Lc; i += kThreads) {
+        const int h = i / s.Lc, c = i - h * s.Lc, owner = c / l.slice;
+        float v = 0.f;
+        for (int g = 0; g < kg; ++g) v += red[((size_t)g * NH + h) * s.Lc + c];
+        *cl.map_shared_rank(rout + ((size_t)split * NH + h) * l.slice + c - owner * l.slice, owner) = v;
+    }
+    for (int i = tid; i < n_splits * nh; i += kThreads) {
+        const int r = i / nh, h = i - r * nh;
+        *cl.map_shared_rank(&rm[split][h], r) = sm_m[h];
+        *cl.map_shared_rank(&rl[split][h], r) = sm_l[h];
+    }
+    if (n_splits > 1) cl.sync(); else __syncthreads();
+    for (int i = tid; i < nh * (s1 - s0); i += kThreads) {
+        const int h = i / (s1 - s0), c = i - h * (s1 - s0);
+        float m = s.sink != nullptr ? __bfloat162float(s.sink[h0 + h]) : -INFINITY;
+        const float sk = m;
+        for (int r = 0; r < n_splits; ++r) m = fmaxf(m, rm[r][h]);
+        float num = 0.f, den = s.sink != nullptr ? expf(sk - m) : 0.f;
+        for (int r = 0; r < n_splits; ++r) {
+            const float w = rm[r][h] == -INFINITY ? 0.f : expf(rm[r][h] - m);
+            num = fmaf(w, rout[((size_t)r * NH + h) * l.slice + c], num);
+            den = fmaf(w, rl[r][h], den);
+        }
+        const float v = den > 0.f ? num / den : 0.f;
+        for (int r = 0; r < n_splits; ++r) *cl.map_shared_rank(olat + h * s.Lc + s0 + c, r) = v;
+    }
+    if (n_splits > 1) cl.sync(); else __syncthreads();
+    // ---- values and gate: one warp per value row -------------------------------------------------------------------------------
+    for (int v = v0 + warp; v < v1; v += kThreads / 32) {
+        const int h = v / s.Dv, c = v - h * s.Dv;
+        const __nv_bfloat16* w = s.wv + ((size_t)(h0 + h) * s.Vp + c) * s.Lc;
+        float a = 0.f;
+        for (int i = lane; i < s.Lc / 8; i += 32) {
+            const float4 x = *reinterpret_cast<const float4*>(olat + h * s.Lc + i * 8), y = *reinterpret_cast<const float4*>(olat + h * s.Lc + i * 8 + 4);
+            const float f[8] = {x.x, x.y, x.z, x.w, y.x, y.y, y.z, y.w};
+            a = dot8(ld_cached(w + i * 8), f, a);
+        }
+        a = warp_sum(a);
+        if (lane == 0) {
+            if (s.gate) {
+                const TI* gp = p.proj + (size_t)row * p.ld + s.off_gate() + (h0 + h) * s.Dv + c;
+                float g;
+                if constexpr (DECODE) g = __ldcg(gp); else g = to_f32(*gp);
+                a *= 1.0f / (1.0f + expf(-g));
+            }
+            store_f32(p.out + (size_t)row * p.ld_out + (h0 + h) * s.Dv + c, a);
+        }
+    }
+    if (DECODE && !ok && tid == 0) p.state->error = 2;
+}
+
+}  // namespace efm

@@ -12,6 +12,7 @@ struct RowEntry {
     int32_t row0, n, pos0;            // rows [row0, row0 + n) hold positions [pos0, pos0 + n) of the sequence
     int32_t table;                    // row of the page table
     int32_t state;                    // recurrent-state slot
+    int32_t ws0;                      // workspace row of position 0 (may be negative: only the positions a pass needs have one)
 };
 
 // One block's share of attention rows: rows [row, row + tile) of an entry.

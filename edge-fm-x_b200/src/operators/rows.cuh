@@ -13,7 +13,7 @@ __global__ void __launch_bounds__(128) embed_rows_kernel(const int32_t* __restri
                                                          const __nv_bfloat16* __restrict__ table,
                                                          const __nv_bfloat16* __restrict__ custom,
                                                          float* __restrict__ out, int vocab, int hidden,
-                                                         int embed_token_id, int n_custom) {
+                                                         int embed_token_id, int n_custom, float scale) {
     const int t = blockIdx.x;
     const int id = ids[t];
     const __nv_bfloat16* src = nullptr;
@@ -25,8 +25,8 @@ __global__ void __launch_bounds__(128) embed_rows_kernel(const int32_t* __restri
     for (int c = threadIdx.x; c < hidden / 8; c += blockDim.x) {
         float f[8];
         unpack8(src != nullptr ? ld_cached(src + (size_t)c * 8) : make_uint4(0, 0, 0, 0), f);
-        dst[2 * c] = make_float4(f[0], f[1], f[2], f[3]);
-        dst[2 * c + 1] = make_float4(f[4], f[5], f[6], f[7]);
+        dst[2 * c] = make_float4(f[0] * scale, f[1] * scale, f[2] * scale, f[3] * scale);
+        dst[2 * c + 1] = make_float4(f[4] * scale, f[5] * scale, f[6] * scale, f[7] * scale);
     }
 }
 

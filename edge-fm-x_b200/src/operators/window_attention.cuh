@@ -1,10 +1,11 @@
-// Causal softmax attention over a paged cache with a sliding window and per-head score modification:
-//   score(i, j) = (q_i . k_j) * scale * temp[h] - slope_h * (i - j),   0 <= i - j < window   (window 0: no lower bound)
-// with slope_h = 2^(-8 (h + 1) / H), q and k RMS-normalised per head before they are used / cached, value width free.
+// Causal softmax attention over a paged cache with a sliding window, kept first tokens and per-head score modification:
+//   score(i, j) = (q_i . k_j) * scale * temp[h] - slope_h * (i - j),   0 <= i - j < window (window 0: no lower bound) or j < keep
+// with slope_h = 2^(-8 (h + 1) / H), q and k RMS-normalised per head (with or without a weight) and then rotated before they
+// are used / cached, value width free.  A weightless norm commutes with the rotation, which keeps a head's length.
 // Cache: per layer a K pool [pages * 64][kv_heads][Dp] and a V pool [pages * 64][kv_heads][Vp], channels zero-padded to
 // Dp / Vp (multiples of 64); a sequence's pages are listed in a page table.  TC = bf16 or fp32 (the all-32-bit mode).
 //
-//   qk_scatter_rows      many rows: per-head norms, q -> [T][H][Dp], k and v -> cache rows
+//   qk_scatter_rows      many rows: per-head norms and rotation, q -> [T][H][Dp], k and v -> cache rows
 //   window_attention_rows many rows on the CUDA cores, fp32 throughout (32-bit mode, short portions, head sizes the
 //                        tensor-core form does not take)
 //   window_attention_decode one row: norms of q and k, cache append and split-key attention in one launch; the splits of
@@ -15,6 +16,7 @@
 #include <utility>
 
 #include "common.cuh"
+#include "rotary.cuh"
 #include "row_plan.cuh"
 
 namespace efm {
@@ -22,12 +24,22 @@ namespace efm {
 struct WindowAttnShape {
     int H, G, D, Dv, Dp, Vp;          // query heads, kv heads, channels and padded channels
     int window;                       // 0: full causal
+    int keep;                         // first tokens that stay visible (with a window)
     int bias;                         // 1: distance bias
     float scale, eps;
-    const __nv_bfloat16* q_norm;      // [D]
+    const __nv_bfloat16* q_norm;      // [D], null: norm without a weight
     const __nv_bfloat16* k_norm;      // [D]
-    const __nv_bfloat16* temp;        // [H]
+    const __nv_bfloat16* temp;        // [H], null: 1
+    RotShape rot;
+    // tensor-core form only: extra term exp(sink[h]) of the softmax denominator, and heads multiplied by sigmoid(gate)
+    const __nv_bfloat16* sink;        // [H], null: none
+    const __nv_bfloat16* gate;        // [T][H * Dv] with row stride gate_ld, null: none
+    int gate_ld;
 };
+
+__device__ __forceinline__ float head_multiplier(const WindowAttnShape& s, int h) {
+    return s.temp != nullptr ? s.scale * __bfloat162float(s.temp[h]) : s.scale;
+}
 
 __device__ __forceinline__ float to_f32(float v) { return v; }
 __device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
@@ -37,6 +49,17 @@ __device__ __forceinline__ float distance_slope(int h, int H) { return exp2f(-8.
 template <typename T> __device__ __forceinline__ float round_as(float v);
 template <> __device__ __forceinline__ float round_as<float>(float v) { return v; }
 template <> __device__ __forceinline__ float round_as<__nv_bfloat16>(float v) { return round_bf16(v); }
+
+__device__ __forceinline__ void load8_as_f32(const float* p, float (&f)[8]) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+__device__ __forceinline__ void load8_as_f32(const __nv_bfloat16* p, float (&f)[8]) { unpack8(ld_cached(p), f); }
+__device__ __forceinline__ float4 load4_as_f32(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4_as_f32(const __nv_bfloat16* p) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    return make_float4(bf16lo(v.x), bf16hi(v.x), bf16lo(v.y), bf16hi(v.y));
+}
 
 // ---- many rows: norms and scatter --------------------------------------------------------------------------------
 template <typename T>
@@ -67,8 +90,14 @@ __device__ __forceinline__ void store_head8(T* p, const float (&f)[8]) {        
 template <typename TI, typename TQ, typename TC>
 __global__ void __launch_bounds__(256) qk_scatter_rows_kernel(const TI* __restrict__ qkv, int ld, TQ* __restrict__ q_out, TC* __restrict__ k_pool,
                                                               TC* __restrict__ v_pool, const WindowAttnShape s, const RowPlan plan, int lanes) {
+    __shared__ float cs[kRotMaxPairs], sn[kRotMaxPairs], stage[256 * 8];
     const int row = blockIdx.x, l = threadIdx.x & (lanes - 1), per = 256 / lanes;
     const RowEntry e = plan.of_row(row);
+    float* st = stage + (threadIdx.x & ~(lanes - 1)) * 8;              // this head's channels
+    if (s.rot.kind != kRotNone) {
+        rot_table(s.rot, e.pos0 + row - e.row0, cs, sn);
+        __syncthreads();
+    }
     const size_t cr = plan.cache_row(e, e.pos0 + row - e.row0);
     const TI* src = qkv + (size_t)row * ld;                            // ld % 8 == 0
     const bool vec = (s.D & 7) == 0, vecv = vec && (s.Dv & 7) == 0;
@@ -87,7 +116,19 @@ __global__ void __launch_bounds__(256) qk_scatter_rows_kernel(const TI* __restri
             const float inv = 1.0f / sqrtf(ss / (float)s.D + s.eps);
             const __nv_bfloat16* w = u < s.H ? s.q_norm : s.k_norm;
 #pragma unroll
-            for (int j = 0; j < 8; ++j) f[j] = d + j < s.D ? f[j] * inv * __bfloat162float(w[d + j]) : 0.f;
+            for (int j = 0; j < 8; ++j) f[j] = d + j < s.D ? f[j] * inv * (w != nullptr ? __bfloat162float(w[d + j]) : 1.f) : 0.f;
+        }
+        if (s.rot.kind != kRotNone) {                                  // the lanes of a head exchange channels
+#pragma unroll
+            for (int j = 0; j < 8; ++j) st[d + j] = f[j];
+            __syncwarp();
+            if (qk && d < s.rot.dims) {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) f[j] = rot_channel(s.rot, st, d + j, cs, sn);
+            }
+            __syncwarp();
+        }
+        if (qk) {
             if (d < s.Dp) {
                 if (u < s.H) store_head8(q_out + ((size_t)row * s.H + u) * s.Dp + d, f);
                 else store_head8(k_pool + (cr * s.G + (u - s.H)) * s.Dp + d, f);
@@ -132,7 +173,8 @@ __global__ void __launch_bounds__(256) window_attention_rows_kernel(const TQ* __
     const int lo = s.window > 0 ? max(0, i_pos - s.window + 1) : 0;
     const int first = s.window > 0 ? max(0, e.pos0 + r0 - s.window + 1) : 0;
     const int end = e.pos0 + r0 + nq;                                  // one past the last visible key of the block
-    const float mul = s.scale * __bfloat162float(s.temp[h]);
+    const int first_tile = first & ~(KT - 1), kept = s.window > 0 ? min(s.keep, first) : 0;    // kept keys ahead of the window
+    const float mul = head_multiplier(s, h);
     const float slope = s.bias ? distance_slope(h, s.H) : 0.f;
     float acc[4][4];
 #pragma unroll
@@ -140,7 +182,7 @@ __global__ void __launch_bounds__(256) window_attention_rows_kernel(const TQ* __
 #pragma unroll
         for (int j = 0; j < 4; ++j) acc[n][j] = 0.f;
     float m = -INFINITY, l = 0.f;
-    for (int k0 = first & ~(KT - 1); k0 < end; k0 += KT) {
+    for (int k0 = kept > 0 ? 0 : first_tile; k0 < end; k0 = k0 + KT >= kept ? max(k0 + KT, first_tile) : k0 + KT) {
         __syncthreads();
         for (int i = tid; i < KT * s.Dp; i += 256) {
             const int kr = i / s.Dp, d = i - kr * s.Dp;
@@ -162,7 +204,7 @@ __global__ void __launch_bounds__(256) window_attention_rows_kernel(const TQ* __
                 const float4 x = a[t], y = b[t];
                 d0 = fmaf(x.x, y.x, d0); d1 = fmaf(x.y, y.y, d1); d0 = fmaf(x.z, y.z, d0); d1 = fmaf(x.w, y.w, d1);
             }
-            sc[u] = (j >= lo && j <= i_pos) ? (d0 + d1) * mul - slope * (float)(i_pos - j) : -INFINITY;
+            sc[u] = ((j >= lo || j < s.keep) && j <= i_pos) ? (d0 + d1) * mul - slope * (float)(i_pos - j) : -INFINITY;
         }
         float mx = fmaxf(sc[0], sc[1]);
 #pragma unroll
@@ -218,6 +260,7 @@ struct Smem {
     float knew[MAXP], vnew[MAXP];
     float p[kHeads][kPageTokens];
     float alpha[kHeads], m[kHeads], l[kHeads];
+    float cs[kRotMaxPairs], sn[kRotMaxPairs];
     // what the blocks of the cluster hand to this one: its share of their un-normalised outputs, and everybody's (m, l)
     float rm[16][kHeads], rl[16][kHeads];
     float rout[kHeads * MAXP + 16 * 16];       // [split][share of the outputs]
@@ -262,8 +305,8 @@ template <> struct Row4<float> {
     __device__ __forceinline__ void get(float (&f)[4]) const { f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w; }
 };
 
-// grid (splits = cluster size, kv_heads * head blocks); the visible keys are dealt out evenly, block `split` walks its share in
-// tiles of 64.  VM: upper bound of Dp and Vp.
+// grid (splits = cluster size, kv_heads * head blocks); the visible keys (kept first tokens, then the window) are numbered in
+// order and dealt out evenly, block `split` walks its share in tiles of 64.  VM: upper bound of Dp and Vp.
 template <typename TC, int VM>
 __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(const WindowDecodeParams<TC> p) {
     using namespace wd;
@@ -287,17 +330,20 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
     const int kv_len = (int)p.state->kv_len, pos = kv_len - 1;
     const bool ok = kv_len > 0 && kv_len <= p.max_pages * kPageTokens;
     const int lo = s.window > 0 ? max(0, kv_len - s.window) : 0;
-    const int chunk = ok ? (kv_len - lo + n_splits - 1) / n_splits : 0;
-    const int begin = lo + split * chunk, end = ok ? min(kv_len, begin + chunk) : begin;
+    const int kept = s.window > 0 ? min(s.keep, lo) : 0;               // visible key n stands at position n or, behind the kept ones, n + skip
+    const int skip = lo - kept, n_vis = kv_len - skip, newest = n_vis - 1;
+    const int chunk = ok ? (n_vis + n_splits - 1) / n_splits : 0;
+    const int begin = split * chunk, end = ok ? min(n_vis, begin + chunk) : begin;
 
     Row8<TC> kr[KC];
     Row4<TC> vr[VK];
+    auto position = [&](int n) { return n < kept ? n : n + skip; };
     auto pool_row = [&](int j) { return (size_t)p.pages[j / kPageTokens] * kPageTokens + j % kPageTokens; };
-    // 64 keys from j0, except the one this launch appends
+    // 64 keys from number j0, except the one this launch appends
     auto load_tile = [&](int j0) {
         const int j = j0 + key;
-        if (j < end && j != pos) {
-            const TC* src = p.k_pool + (pool_row(j) * s.G + g) * s.Dp;
+        if (j < end && j != newest) {
+            const TC* src = p.k_pool + (pool_row(position(j)) * s.G + g) * s.Dp;
 #pragma unroll
             for (int c = 0; c < KC; ++c)
                 if ((c * 4 + part) * 8 < s.Dp) kr[c].load(src + (c * 4 + part) * 8);
@@ -306,14 +352,16 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
 #pragma unroll
             for (int i = 0; i < VK; ++i) {
                 const int kk = tg + i * kg, jj = j0 + kk;
-                if (kk < kPageTokens && jj < end && jj != pos) vr[i].load(p.v_pool + (pool_row(jj) * s.G + g) * s.Vp + dpart * 4);
+                if (kk < kPageTokens && jj < end && jj != newest) vr[i].load(p.v_pool + (pool_row(position(jj)) * s.G + g) * s.Vp + dpart * 4);
             }
         }
     };
     if (begin < end) load_tile(begin);
+    if (ok) rot_table(s.rot, pos, sm.cs, sm.sn);
     if (p.early) { pdl_wait(); pdl_launch_dependents(); }
+    if (s.rot.kind != kRotNone) __syncthreads();
 
-    // ---- norms of this token's q heads and k, v ------------------------------------------------------------------
+    // ---- norms and rotation of this token's q heads and k, v ------------------------------------------------------------------
     for (int u = warp; u < nh + 1; u += 8) {
         const bool is_q = u < nh;
         const float* x = is_q ? p.qkv + (size_t)(h0 + u) * s.D : p.qkv + (size_t)(s.H + g) * s.D;
@@ -331,15 +379,29 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
         for (int i = 0; i < VM / 32; ++i) {
             const int d = lane + 32 * i;
             if (d >= s.Dp) continue;
-            const float v = d < s.D ? f[i] * inv * __bfloat162float(w[d]) : 0.f;
-            if (is_q) sm.q[u][d] = v; else sm.knew[d] = round_as<TC>(v);
+            const float v = d < s.D ? f[i] * inv * (w != nullptr ? __bfloat162float(w[d]) : 1.f) : 0.f;
+            if (is_q) sm.q[u][d] = v; else sm.knew[d] = v;
         }
+        float* y = is_q ? sm.q[u] : sm.knew;
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < VM / 32; ++i) {
+            const int d = lane + 32 * i;
+            if (d < s.Dp) {
+                f[i] = s.rot.kind != kRotNone ? rot_channel(s.rot, y, d, sm.cs, sm.sn) : y[d];
+                if (!is_q) f[i] = round_as<TC>(f[i]);
+            }
+        }
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < VM / 32; ++i)
+            if (lane + 32 * i < s.Dp) y[lane + 32 * i] = f[i];
     }
     for (int d = tid; d < s.Vp; d += kThreads)
         sm.vnew[d] = d < s.Dv ? round_as<TC>(__ldcg(p.qkv + (size_t)(s.H + s.G) * s.D + (size_t)g * s.Dv + d)) : 0.f;
     if (tid < kHeads) { sm.m[tid] = -INFINITY; sm.l[tid] = 0.f; }
     __syncthreads();
-    if (begin <= pos && pos < end && blockIdx.y % hb == 0) {           // the block that walks the newest key appends it
+    if (begin <= newest && newest < end && blockIdx.y % hb == 0) {     // the block that walks the newest key appends it
         const size_t cr = pool_row(pos);
         for (int d = tid; d < s.Dp; d += kThreads) store_f32(p.k_pool + (cr * s.G + g) * s.Dp + d, sm.knew[d]);
         for (int d = tid; d < s.Vp; d += kThreads) store_f32(p.v_pool + (cr * s.G + g) * s.Vp + d, sm.vnew[d]);
@@ -360,7 +422,7 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
 #pragma unroll
         for (int c = 0; c < KC; ++c) {
             const int d0 = (c * 4 + part) * 8;
-            if (d0 < s.Dp && j == pos) {
+            if (d0 < s.Dp && j == newest) {
 #pragma unroll
                 for (int i = 0; i < 8; ++i) kf[c][i] = sm.knew[d0 + i];
             } else {
@@ -384,7 +446,7 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
             d += __shfl_xor_sync(0xffffffffu, d, 2);
             if (part == 0) {
                 const float slope = s.bias ? distance_slope(h0 + h, s.H) : 0.f;
-                sm.p[h][key] = vis ? d * (s.scale * __bfloat162float(s.temp[h0 + h])) - slope * (float)(pos - j) : -INFINITY;
+                sm.p[h][key] = vis ? d * head_multiplier(s, h0 + h) - slope * (float)(pos - position(j)) : -INFINITY;
             }
         }
         __syncthreads();
@@ -417,7 +479,7 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
                 const int kk = tg + i * kg, jj = j0 + kk;
                 if (kk < kPageTokens && jj < end) {
                     float v[4];
-                    if (jj == pos) {
+                    if (jj == newest) {
 #pragma unroll
                         for (int c = 0; c < 4; ++c) v[c] = sm.vnew[dpart * 4 + c];
                     } else {

@@ -1,7 +1,10 @@
 // Many-row form of the windowed attention (window_attention.cuh) on the 5th-generation tensor cores: the structure of
 // attention_tc.cuh (S = Q K^T and O_tile = P V as tcgen05.mma with TMEM accumulators, operands by TMA, online softmax with
 // two threads per query row) over a paged cache, with the per-head multiplier and the distance bias applied to the scores
-// in fp32.  A key tile is exactly one 64-token page: its TMA coordinate is the page number of the sequence's table.
+// in fp32.  A key tile is exactly one 64-token page: its TMA coordinate is the page number of the sequence's table, or the
+// place of the page in a workspace of keys and values expanded for this pass (latent attention).
+// Keys may come from two tensors: DP channels per kv head, and RP more that all heads share (a rotated part); the query rows
+// are split the same way.  Channels that a tensor does not have are filled with zeros by TMA.
 // Block = 128 rows of one entry x one head, 256 threads.  Rows of the tile that belong to the next entry are computed and
 // not stored.  The weights enter P V as a bf16 pair high + low (16 bits of mantissa), written straight into tensor memory.
 // Every mbarrier wait is bounded and raises *error.
@@ -15,9 +18,9 @@ namespace wt {
 
 constexpr int BM = 128, BN = kPageTokens, kThreads = 256, kMaxTiles = 1024;
 
-template <int DP, int VP>
+template <int DP, int VP, int RP = 0>
 struct Cfg {
-    static constexpr int QB = DP / 64, VB = VP / 64;         // 64-channel boxes per row
+    static constexpr int QB = (DP + RP) / 64, VB = VP / 64;  // 64-channel boxes per row
     static constexpr int Q_BYTES = BM * 128 * QB, K_BYTES = BN * 128 * QB, V_BYTES = BN * 128 * VB;
     static constexpr int P_COL = 64, O_COL = 128;
     static constexpr int TMEM_COLS = 256;                    // S (64 columns) | P high, P low (32 each) | O tile, power of two
@@ -43,11 +46,15 @@ __device__ __forceinline__ void umma_ts(uint32_t tmem_d, uint32_t tmem_a, uint64
 
 }  // namespace wt
 
-template <int DP, int VP>
-__global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
-                                                                           const __grid_constant__ CUtensorMap map_v, __nv_bfloat16* __restrict__ out,
+struct WindowTcMaps {
+    CUtensorMap q, k, v;              // [rows][heads][channels]
+    CUtensorMap qr, kr;               // RP > 0: rotated parts, [rows][heads][channels] and [rows][1][channels]
+};
+
+template <int DP, int VP, int RP>
+__global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(const __grid_constant__ WindowTcMaps maps, __nv_bfloat16* __restrict__ out,
                                                                            int ld_out, const WindowAttnShape s, const RowPlan plan,
-                                                                           const RowTile* __restrict__ tiles, int* error) {
+                                                                           const RowTile* __restrict__ tiles, int workspace, int* error) {
     using namespace wt;
     using at::instr_desc;
     using at::tma_load_3d;
@@ -58,7 +65,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     using tc::smem_u32;
     using tc::umma_commit;
     using tc::umma_desc;
-    using C = Cfg<DP, VP>;
+    using C = Cfg<DP, VP, RP>;
     extern __shared__ unsigned char wt_smem[];
     const uint32_t raw = smem_u32(wt_smem);
     const uint32_t base = (raw + 1023u) & ~1023u;
@@ -84,7 +91,10 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     const bool valid = row < nq;
     const int lo = s.window > 0 ? max(0, i_pos - s.window + 1) : 0, hi = i_pos + 1;
     const int first = s.window > 0 ? max(0, p0 - s.window + 1) : 0, lo_max = s.window > 0 ? max(0, p0 + nq - s.window) : 0, hi_min = p0 + 1;
-    const int pg0 = first / BN, ntiles = min((p0 + nq - 1) / BN - pg0 + 1, kMaxTiles), kb0 = pg0 * BN;
+    // tiles: the pages with kept first tokens ahead of the window's first page, then the pages of the window
+    const int pg0 = first / BN, nk = s.window > 0 ? min((min(s.keep, first) + BN - 1) / BN, pg0) : 0;
+    const int ntiles = min(nk + (p0 + nq - 1) / BN - pg0 + 1, kMaxTiles);
+    auto tile_page = [&](int i) { return i < nk ? i : pg0 + i - nk; };
 
     if (tid == 0) {
         mbar_init(qfull, 1); mbar_init(kfull0, 1); mbar_init(kfull0 + 8, 1); mbar_init(vfull, 1); mbar_init(sbar, 1); mbar_init(obar, 1);
@@ -95,7 +105,8 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_slot)), "r"(C::TMEM_COLS) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
-    for (int i = tid; i < ntiles; i += kThreads) pages[i] = plan.page_table[(size_t)e.table * plan.max_pages + pg0 + i] * BN;
+    for (int i = tid; i < ntiles; i += kThreads) 
+        pages[i] = workspace ? e.ws0 + tile_page(i) * BN : plan.page_table[(size_t)e.table * plan.max_pages + tile_page(i)] * BN;
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -105,7 +116,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     constexpr uint32_t kDescO = instr_desc(BM, VP) | (1u << 16);
     const uint64_t vdesc = at::umma_desc_mn(sV, (uint32_t)(BN * 128), 1024u);
     constexpr float kLog2e = 1.4426950408889634f;
-    const float f2 = s.scale * __bfloat162float(s.temp[h]) * kLog2e;
+    const float f2 = head_multiplier(s, h) * kLog2e;
     const float b2 = (s.bias ? distance_slope(h, s.H) : 0.f) * kLog2e;
     float o[C::HALF];
 #pragma unroll
@@ -117,17 +128,19 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
         last_k[buf] = tile;
         mbar_expect_tx(kfull0 + 8 * buf, C::K_BYTES);
 #pragma unroll
-        for (int b = 0; b < C::QB; ++b) tma_load_3d(sK + buf * C::K_BYTES + b * (BN * 128), &map_k, b * 64, g, pages[tile], kfull0 + 8 * buf);
+        for (int b = 0; b < C::QB; ++b)
+            if (b < DP / 64) tma_load_3d(sK + buf * C::K_BYTES + b * (BN * 128), &maps.k, b * 64, g, pages[tile], kfull0 + 8 * buf);
+            else tma_load_3d(sK + buf * C::K_BYTES + b * (BN * 128), &maps.kr, b * 64 - DP, 0, pages[tile], kfull0 + 8 * buf);
     };
     auto load_v = [&](int tile) {
         last_v = tile;
         mbar_expect_tx(vfull, C::V_BYTES);
 #pragma unroll
-        for (int b = 0; b < C::VB; ++b) tma_load_3d(sV + b * (BN * 128), &map_v, b * 64, g, pages[tile], vfull);
+        for (int b = 0; b < C::VB; ++b) tma_load_3d(sV + b * (BN * 128), &maps.v, b * 64, g, pages[tile], vfull);
     };
     auto issue_s = [&](int buf) {
 #pragma unroll
-        for (int k = 0; k < DP / 16; ++k) {
+        for (int k = 0; k < (DP + RP) / 16; ++k) {
             const uint64_t da = umma_desc(sQ + (k >> 2) * (BM * 128)) + (uint64_t)((k & 3) * 2);
             const uint64_t db = umma_desc(sK + buf * C::K_BYTES + (k >> 2) * (BN * 128)) + (uint64_t)((k & 3) * 2);
             umma_d(tmem, da, db, kDescS, k != 0 ? 1u : 0u);
@@ -137,7 +150,9 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     if (tid == 0) {
         mbar_expect_tx(qfull, C::Q_BYTES);
 #pragma unroll
-        for (int b = 0; b < C::QB; ++b) tma_load_3d(sQ + b * (BM * 128), &map_q, b * 64, h, e.row0 + r0, qfull);
+        for (int b = 0; b < C::QB; ++b)
+            if (b < DP / 64) tma_load_3d(sQ + b * (BM * 128), &maps.q, b * 64, h, e.row0 + r0, qfull);
+            else tma_load_3d(sQ + b * (BM * 128), &maps.qr, b * 64 - DP, h, e.row0 + r0, qfull);
         load_k(0, 0);
         if (ntiles > 1) load_k(1, 1);
         load_v(0);
@@ -153,15 +168,15 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
         if (tid == 0 && j + 2 < ntiles && *abort_s == 0) load_k(j + 2, j & 1);      // S_j has read K buffer j % 2
         uint32_t sr[32];
         tc::tmem_ld32(tmem + ((uint32_t)((warp & 3) * 32) << 16) + (uint32_t)(hf * 32), sr);
-        const int key0 = kb0 + j * BN + hf * 32;
+        const int kb = tile_page(j) * BN, key0 = kb + hf * 32;
         float sc[32];                                            // scores in units of log2
         float mx = -INFINITY;
         const float bias0 = b2 * (float)(key0 - i_pos);
-        const bool interior = kb0 + j * BN >= lo_max && kb0 + (j + 1) * BN <= hi_min;
+        const bool interior = (kb >= lo_max || kb + BN <= s.keep) && kb + BN <= hi_min;
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
             const float v = fmaf(__uint_as_float(sr[i]), f2, fmaf(b2, (float)i, bias0));
-            sc[i] = interior || (key0 + i >= lo && key0 + i < hi) ? v : -INFINITY;
+            sc[i] = interior || ((key0 + i >= lo || key0 + i < s.keep) && key0 + i < hi) ? v : -INFINITY;
             mx = fmaxf(mx, sc[i]);
         }
         xch[hf * BM + row] = mx;
@@ -226,11 +241,30 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     __syncthreads();
     xch[hf * BM + row] = l;
     __syncthreads();
-    const float L = xch[row] + xch[BM + row];
-    const float inv = L > 0.f ? 1.0f / L : 0.f;
+    float L = xch[row] + xch[BM + row], up = 1.0f;
+    if (s.sink != nullptr) {                                     // one more term of the denominator
+        const float sk = __bfloat162float(s.sink[h]) * kLog2e, mx = fmaxf(m, sk);
+        up = at::ex2(m - mx);
+        L = fmaf(L, up, at::ex2(sk - mx));
+    }
+    const float inv = L > 0.f ? up / L : 0.f;
     if (valid && *abort_s == 0) {
         __nv_bfloat16* dst = out + (size_t)(e.row0 + r0 + row) * ld_out + (size_t)h * s.Dv;
         const bool vec = (s.Dv & 7) == 0;                        // ld_out is a multiple of 8
+        if (s.gate != nullptr) {
+            const __nv_bfloat16* gt = s.gate + (size_t)(e.row0 + r0 + row) * s.gate_ld + (size_t)h * s.Dv;
+#pragma unroll
+            for (int i = 0; i < C::HALF; i += 8) {
+                const int d = hf * C::HALF + i;
+                float f[8];
+                if (vec && d + 8 <= s.Dv) unpack8(ld_cached(gt + d), f);
+                else
+#pragma unroll
+                    for (int c = 0; c < 8; ++c) f[c] = d + c < s.Dv ? __bfloat162float(gt[d + c]) : 0.f;
+#pragma unroll
+                for (int c = 0; c < 8; ++c) o[i + c] *= 1.0f / (1.0f + expf(-f[c]));
+            }
+        }
 #pragma unroll
         for (int i = 0; i < C::HALF; i += 8) {
             const int d = hf * C::HALF + i;

@@ -360,30 +360,52 @@ EFM_API efm_status efm_b200_vit_encode(efm_b200_vit* vit, const void* pixels, in
                                        int32_t out_mem);
 
 /* ---- layered decoders ---------------------------------------------------------------------
- * A decoder described layer by layer: every layer names its mixer (softmax attention or the generalised delta rule), the
- * mixer's sizes and an optional dense feed-forward; sublayer outputs are RMS-normalised before the residual add; an
- * optional per-layer token input follows.  (No counterpart in the reference.)  Such a context serves the same calls as
- * the text tower (set_weight, finalize_weights, prefill, decode_begin, decode_steps, read_tokens, read_logits, ...) and,
- * in addition, batched steps over a paged cache: one pool of 64-token pages per attention layer and one pool of recurrent
- * state slots, handed out by the caller (who maps page numbers to sequences).
+ * A decoder described layer by layer: every layer names its mixer (softmax attention, latent attention or the generalised
+ * delta rule), the mixer's sizes and an optional feed-forward (dense or routed experts); sublayer outputs are
+ * RMS-normalised before the residual add, and with EFM_NORM_SANDWICH sublayer inputs are normalised too; an optional
+ * per-layer token input follows.  A span of layers may run several times in a row with the same weights, every pass with
+ * its own cache and state.  (No counterpart in the reference.)  Such a context serves the same calls as the text tower
+ * (set_weight, finalize_weights, prefill, decode_begin, decode_steps, read_tokens, read_logits, ...) and, in addition,
+ * batched steps over a paged cache: one pool of 64-token pages per attention layer run and one pool of recurrent state
+ * slots, handed out by the caller (who maps page numbers to sequences).
  *
- * Tensor names: embed, side.embed, final.norm, head and, for layer i, l<i>.norm1 / norm2, l<i>.mix.{q,k,v,o,q.norm,k.norm,
- * temp} (attention) or l<i>.mix.{r,k,v,g,a,a.b,w1,w2,w0,norm,o} (delta rule), l<i>.mlp.{up,down,act},
- * l<i>.side.{gate,proj,norm}; bf16. */
-enum { EFM_MIXER_ATTENTION = 0, EFM_MIXER_GENERAL_DELTA = 1 };
+ * Tensor names: embed, side.embed, final.norm, head and, for layer i, l<i>.norm1 / norm2 (sandwich: before the sublayers,
+ * l<i>.norm1b / norm2b behind them), l<i>.mix.{q,k,v,o} with, as the layer asks, {q.b,k.b,v.b}, {q.norm,k.norm}, temp
+ * (attention), l<i>.mix.{dq,dq.norm,uq,dkv,dkv.norm,uk,uv,o} with sink, g (latent attention) or
+ * l<i>.mix.{r,k,v,g,a,a.b,w1,w2,w0,norm,o} (delta rule), l<i>.mlp.{up,down,act} (dense) or l<i>.mlp.router and
+ * l<i>.mlp.e<j>.{gate,up,down} (experts), l<i>.side.{gate,proj,norm}; bf16. */
+enum { EFM_MIXER_ATTENTION = 0, EFM_MIXER_GENERAL_DELTA = 1, EFM_MIXER_LATENT_ATTENTION = 2 };
 enum { EFM_PAGE_TOKENS = 64 };
+enum { EFM_QK_NORM_WEIGHTED = 0, EFM_QK_NORM_PLAIN = 1 };            /* RMS norm of q and k per head, with / without a weight */
+enum { EFM_ROT_NONE = 0, EFM_ROT_HALF = 1, EFM_ROT_PAIRS = 2 };      /* channel i turns with i + dims / 2; 2 i with 2 i + 1 */
+enum { EFM_NORM_OUTPUT = 0, EFM_NORM_SANDWICH = 1 };
 
 typedef struct efm_decoder_layer {
     int32_t mixer;                /* EFM_MIXER_* */
     int32_t heads;
     int32_t kv_heads;             /* attention only */
-    int32_t dim;                  /* per-head key channels (delta rule: value channels too), <= 256 */
-    int32_t vdim;                 /* attention: per-head value channels, <= 256 */
-    int32_t window;               /* attention: position i sees j with 0 <= i - j < window; 0: all j <= i */
+    int32_t dim;                  /* per-head key channels (delta rule: value channels too; latent: the unrotated ones), <= 256 */
+    int32_t vdim;                 /* attention, latent attention: per-head value channels, <= 256 */
+    int32_t window;               /* both attentions: position i sees j with 0 <= i - j < window; 0: all j <= i */
     int32_t distance_bias;        /* attention: 1 = subtract 2^(-8 (h+1) / heads) * (i - j) from the score of head h */
-    float scale;                  /* attention: score multiplier */
+    float scale;                  /* both attentions: score multiplier */
     int32_t decay_rank;           /* delta rule: rows of w1, <= 512 */
-    int32_t ff;                   /* feed-forward width, 0: none */
+    int32_t ff;                   /* dense feed-forward (PolyNorm) width, 0: none */
+    int32_t keep_first;           /* attention with a window: the first keep_first tokens stay visible */
+    int32_t qk_norm;              /* attention: EFM_QK_NORM_* */
+    int32_t head_temp;            /* attention: 1 = a learned score multiplier per head */
+    int32_t qkv_bias;             /* attention: 1 = q, k and v have biases */
+    int32_t rot_kind;             /* EFM_ROT_*; latent: of the rotated part */
+    int32_t rot_dims;             /* rotated channels of a head (the first ones), even; latent: the rotated key part, <= 256 */
+    float rot_base;               /* pair i of position p turns by p * rot_base^(-2 i / rot_dims) */
+    int32_t q_rank, kv_rank;      /* latent: widths of the query latent and of the cached key / value latent (<= 1024) */
+    int32_t sink;                 /* latent: 1 = a learned extra term exp(sink[h]) in the softmax denominator */
+    int32_t out_gate;             /* latent: 1 = heads multiplied by sigmoid(W_g h) */
+    int32_t experts;              /* routed feed-forward: number of experts (<= 512), 0: none */
+    int32_t expert_ff;            /* width of an expert */
+    int32_t expert_top;           /* experts a token uses (<= 32) */
+    int32_t expert_groups;        /* equal groups of neighbouring experts (<= 64) ... */
+    int32_t expert_groups_kept;   /* ... of which those with the best single scores stay open */
 } efm_decoder_layer;
 
 typedef struct efm_decoder_desc {
@@ -397,6 +419,9 @@ typedef struct efm_decoder_desc {
     int32_t cache_pages;          /* pages of each attention layer's pool */
     int32_t state_slots;          /* recurrent state slots */
     int32_t max_slots;            /* sequences mapped at a time */
+    int32_t norm_layout;          /* EFM_NORM_* */
+    float embed_scale;            /* embedding rows are multiplied by this */
+    int32_t loop_start, loop_stop, loop_times;   /* layers [start, stop) run `times` times in a row; times <= 1: once */
 } efm_decoder_desc;
 
 EFM_API efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decoder_layer* layers, int32_t device_id,
@@ -429,8 +454,8 @@ typedef struct efm_step_entry {
  * and the entry's random counter.  Synchronises when something is returned. */
 EFM_API efm_status efm_b200_decoder_step(efm_b200_ctx* ctx, const efm_step_entry* entries, int32_t n_entries,
                                          float* logits, int32_t* sampled);
-/* Residual stream after every layer of the steps that follow: copied to host_out [num_layers, rows, width] by
- * efm_b200_decoder_read_taps.  rows = 0 switches it off. */
+/* Residual stream after every layer run (a looped layer counts each time) of the steps that follow: copied to host_out
+ * [layer runs, rows, width] by efm_b200_decoder_read_taps.  rows = 0 switches it off. */
 EFM_API efm_status efm_b200_decoder_set_taps(efm_b200_ctx* ctx, int32_t rows);
 EFM_API efm_status efm_b200_decoder_read_taps(efm_b200_ctx* ctx, float* host_out);
 

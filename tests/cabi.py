@@ -44,13 +44,16 @@ class VlaDesc(C.Structure):
 
 class DecoderLayer(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "kv_heads", "dim", "vdim", "window", "distance_bias")] + \
-        [("scale", C.c_float), ("decay_rank", C.c_int32), ("ff", C.c_int32)]
+        [("scale", C.c_float)] + [(n, C.c_int32) for n in ("decay_rank", "ff", "keep_first", "qk_norm", "head_temp", "qkv_bias", "rot_kind", "rot_dims")] + \
+        [("rot_base", C.c_float)] + [(n, C.c_int32) for n in (
+            "q_rank", "kv_rank", "sink", "out_gate", "experts", "expert_ff", "expert_top", "expert_groups", "expert_groups_kept")]
 
 
 class DecoderDesc(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("struct_size", "num_layers", "vocab", "width", "side_dim")] + \
         [("norm_eps", C.c_float)] + [(n, C.c_int32) for n in (
-            "compute_dtype", "max_step_tokens", "max_response_tokens", "cache_pages", "state_slots", "max_slots")]
+            "compute_dtype", "max_step_tokens", "max_response_tokens", "cache_pages", "state_slots", "max_slots",
+            "norm_layout")] + [("embed_scale", C.c_float)] + [(n, C.c_int32) for n in ("loop_start", "loop_stop", "loop_times")]
 
 
 class StepEntry(C.Structure):
@@ -469,23 +472,38 @@ class VlaPolicy:
 
 
 class Decoder(Backend):
-    """A layered-decoder context described by a Folizen configuration dict; one mapped slot per call of map_slot."""
+    """A layered-decoder context described by a Folizen or Temuvik configuration dict; one mapped slot per call of map_slot."""
 
     def __init__(self, config, *, decay_rank=64, cache_pages=64, state_slots=4, max_slots=4, max_step_tokens=2048,
                  max_response_tokens=512, dtype=EFM_BF16, device_id=0):
         self.L = lib()
         layers = (DecoderLayer * len(config["layers"]))()
+        temuvik = config["architecture"] == "Temuvik"
         for e, l in zip(layers, config["layers"]):
-            m = l["mixer"]
-            e.heads, e.dim, e.ff = m["heads"], m["dim"], l["mlp"]["ff"] if l["mlp"] else 0
+            m, mask = l["mixer"], l["mixer"].get("mask") or {}
+            e.heads, e.dim, e.window = m["heads"], m["dim"], mask.get("size", 0)
+            if temuvik:
+                e.vdim, e.scale, e.rot_dims, e.rot_base = m["vdim"], m["scale"], m["rot"]["dims"], m["rot"]["base"]
+                if l["type"] == "attention":
+                    e.mixer, e.kv_heads, e.keep_first, e.qk_norm, e.qkv_bias, e.rot_kind = 0, m["kv_heads"], mask.get("keep_first", 0), 1, 1, 1
+                else:
+                    e.mixer, e.q_rank, e.kv_rank, e.sink, e.out_gate, e.rot_kind = 2, m["q_rank"], m["kv_rank"], 1, 1, 2
+                if l["mlp"]:
+                    r = l["mlp"]["router"]
+                    g = r.get("groups") or {"count": 1, "keep": 1}
+                    e.experts, e.expert_ff, e.expert_top = r["experts"], l["mlp"]["expert"]["ff"], r["top"]
+                    e.expert_groups, e.expert_groups_kept = g["count"], g["keep"]
+                continue
+            e.ff = l["mlp"]["ff"] if l["mlp"] else 0
             if l["type"] == "attention":
-                e.mixer, e.kv_heads, e.vdim, e.scale, e.distance_bias = 0, m["kv_heads"], m["vdim"], m["scale"], 1
-                e.window = m["mask"]["size"] if m.get("mask") else 0
+                e.mixer, e.kv_heads, e.vdim, e.scale, e.distance_bias, e.head_temp = 0, m["kv_heads"], m["vdim"], m["scale"], 1, 1
             else:
                 e.mixer, e.decay_rank = 1, decay_rank
+        loop = config.get("loop") or {"start": 0, "stop": 0, "times": 0}
         d = DecoderDesc(C.sizeof(DecoderDesc), len(layers), config["vocab"], config["width"],
                         (config.get("token_side") or {}).get("dim", 0), config["norm"]["eps"], dtype, max_step_tokens,
-                        max_response_tokens, cache_pages, state_slots, max_slots)
+                        max_response_tokens, cache_pages, state_slots, max_slots, int(temuvik),
+                        config["embedding"]["scale"] if temuvik else 1.0, loop["start"], loop["stop"], loop["times"])
         self.cfg = type("Cfg", (), {"vocab": config["vocab"], "mrope_section": None})()
         self.ctx = P()
         st = self.L.efm_b200_decoder_create(C.byref(d), layers, device_id, C.byref(self.ctx))

@@ -919,7 +919,7 @@ def summarise(line):
     return out
 
 
-# ---- layered decoder (Folizen) beside the text tower at equal size -----------------------------------------------------
+# ---- layered decoders beside the text tower at equal size -----------------------------------------------------------------
 DESIGN_SIZES = {        # width, heads, kv heads (head dim 128), attention feed-forward, vocabulary
     "1024": (1024, 8, 2, 4096, 32768),
     "2048": (2048, 16, 4, 8192, 32768),
@@ -928,7 +928,40 @@ DESIGN_SIZES = {        # width, heads, kv heads (head dim 128), attention feed-
 DESIGN_LAYERS, DESIGN_WINDOW, DESIGN_PROMPT, DESIGN_DECODE, DESIGN_RANK = 8, 1024, 2048, 64, 64
 
 
-def design_config(size):
+DESIGN_EXPERTS = {"count": 32, "top": 4, "groups": 4, "keep": 2}
+
+
+def temuvik_config(size):
+    """Latent attention and attention with kept first tokens in turn, routed experts everywhere; active feed-forward = `ff`."""
+    W, H, G, ff, V = DESIGN_SIZES[size]
+    e = DESIGN_EXPERTS
+    mlp = {"kind": "moe", "expert": {"ff": ff // e["top"]}, "router": {"experts": e["count"], "top": e["top"], "groups": {"count": e["groups"], "keep": e["keep"]}}}
+    att = {"type": "attention", "mlp": mlp, "mixer": {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                                      "mask": {"size": DESIGN_WINDOW, "keep_first": 16}, "rot": {"base": 1e5, "dims": 128}}}
+    lat = {"type": "latent_attention", "mlp": mlp, "mixer": {"heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": 3 * W // 8, "kv_rank": 512,
+                                                             "scale": 192 ** -0.5, "mask": {"size": DESIGN_WINDOW}, "rot": {"base": 1e5, "dims": 64}}}
+    return {"architecture": "Temuvik", "width": W, "vocab": V, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "layers": [lat if i % 2 == 0 else att for i in range(DESIGN_LAYERS)]}
+
+
+def temuvik_flops(cfg, n):
+    """Matrix products of the experts a token uses and everything else, plus visible attention pairs, 2 per multiply-add."""
+    W, out = cfg["width"], 0
+    for l in cfg["layers"]:
+        m = l["mixer"]
+        H, D, Dv = m["heads"], m["dim"], m["vdim"]
+        seen = sum(min(i + 1, m["mask"]["size"]) for i in range(n)) + sum(min(m["mask"].get("keep_first", 0), max(0, i + 1 - m["mask"]["size"])) for i in range(n))
+        if l["type"] == "attention":
+            out += 2 * n * W * (H * D + m["kv_heads"] * (D + Dv) + H * Dv) + 2 * H * (D + Dv) * seen
+        else:
+            R, q, L = m["rot_dim"], m["q_rank"], m["kv_rank"]
+            out += 2 * n * (W * (q + L + R + 2 * H * Dv) + q * H * (D + R) + L * H * (D + Dv)) + 2 * H * (D + R + Dv) * seen
+        r = l["mlp"]["router"]
+        out += 2 * n * W * (r["experts"] + 3 * r["top"] * l["mlp"]["expert"]["ff"])
+    return out
+
+
+def folizen_config(size):
     W, H, G, ff, V = DESIGN_SIZES[size]
     att = {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": DESIGN_WINDOW}},
            "mlp": {"kind": "dense", "ff": ff}}
@@ -937,7 +970,7 @@ def design_config(size):
             "layers": [att if i % 2 == 0 else delta for i in range(DESIGN_LAYERS)]}
 
 
-def design_flops(cfg, n):
+def folizen_flops(cfg, n):
     """Matrix products plus visible attention pairs plus the recurrence (7 D^2 multiply-adds per token and head), 2 per multiply-add."""
     W, side, out = cfg["width"], cfg["token_side"]["dim"], 0
     for l in cfg["layers"]:
@@ -981,16 +1014,19 @@ def time_model(be, slot, prompt, steps, warmup):
 
 
 def run_design(args):
-    """Prefill and decode throughput of the Folizen design at sizes that resemble real layers (random weights), and of the
-    text tower with the same width, heads, depth and number of weights."""
+    """Prefill and decode throughput of a layered design at sizes that resemble real layers (random weights), and of the text
+    tower with the same width, heads, depth and number of weights (experts: the weights one token uses)."""
     import torch
     import cabi
     import folizen_util as fu
+    import temuvik_util as tu
     from oracle import qwen_text, synth
     hbm, _ = peaks()
     tf, _ = tensor_peak()
     clocks = ClockSampler(0)
-    out = {"metric": "Folizen prefill / decode throughput beside the text tower at equal size", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic",
+    name_ = args.design.capitalize()
+    design_config, design_flops = (folizen_config, folizen_flops) if args.design == "folizen" else (temuvik_config, temuvik_flops)
+    out = {"metric": name_ + " prefill / decode throughput beside the text tower at equal size", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic",
            "config": {"layers": DESIGN_LAYERS, "prompt": DESIGN_PROMPT, "decode_steps": DESIGN_DECODE, "window": DESIGN_WINDOW}, "sizes": {}}
     clocks.start()
     for size in args.design_sizes.split(","):
@@ -999,11 +1035,12 @@ def run_design(args):
         g = torch.Generator(device="cuda").manual_seed(0)
         be = cabi.Decoder(cfg, decay_rank=DESIGN_RANK, cache_pages=pages, state_slots=1, max_slots=1)
         n_weights = 0
-        for name, shape in fu.shapes(cfg, DESIGN_RANK).items():
+        for name, shape in (fu.shapes(cfg, DESIGN_RANK) if args.design == "folizen" else tu.shapes(cfg)).items():
             t = torch.randn(shape, generator=g, device="cuda") * (shape[-1] ** -0.5 if len(shape) == 2 else 0.1)
             if "norm" in name or name.endswith("temp"):
                 t += 1.0
-            n_weights += t.numel() if len(shape) == 2 and "embed" not in name else 0
+            used = DESIGN_EXPERTS["top"] / DESIGN_EXPERTS["count"] if ".mlp.e" in name else 1
+            n_weights += int(t.numel() * used) if len(shape) == 2 and "embed" not in name else 0
             be.load_weights_partial({name: t.to(torch.bfloat16)})
         be.finalize()
         be.map_slot(0, list(range(pages)), 0)
@@ -1027,9 +1064,9 @@ def run_design(args):
         def report(p, d, f, b):
             return {"prefill_ms": p, "prefill_tokens_per_s": DESIGN_PROMPT / p * 1e3, "prefill_frac_of_bf16_peak": f / p / 1e9 / tf,
                     "decode_ms": d, "decode_tokens_per_s": 1e3 / d, "bytes_per_step": b, "decode_frac_of_hbm": b / d / 1e6 / hbm}
-        out["sizes"][size] = {"folizen": report(pre, dec, fl, nbytes), "text_tower": dict(report(qpre, qdec, qfl, qbytes), intermediate=q.intermediate)}
+        out["sizes"][size] = {args.design: report(pre, dec, fl, nbytes), "text_tower": dict(report(qpre, qdec, qfl, qbytes), intermediate=q.intermediate)}
     out["clocks"] = clocks.stop()
-    out["value"] = out["sizes"][args.design_sizes.split(",")[-1]]["folizen"]["decode_tokens_per_s"]
+    out["value"] = out["sizes"][args.design_sizes.split(",")[-1]][args.design]["decode_tokens_per_s"]
     print(json.dumps(out), flush=True)
 
 
@@ -1042,7 +1079,7 @@ def main():
     ap.add_argument("--config", type=int, default=None, choices=[0, 1, 2, 3, 4],
                     help="run one configuration alone; default: configuration 3 (tensor parallel over the ranks) plus, on one GPU, "
                          "a short pass over the other four")
-    ap.add_argument("--design", choices=["folizen"], default=None, help="layered decoder beside the text tower at equal size (one GPU)")
+    ap.add_argument("--design", choices=["folizen", "temuvik"], default=None, help="layered decoder beside the text tower at equal size (one GPU)")
     ap.add_argument("--design-sizes", default="1024,2048,4096", help="comma-separated widths for --design")
     ap.add_argument("--tokens", type=int, default=0, help="override the number of generated tokens")
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")

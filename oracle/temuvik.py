@@ -6,7 +6,6 @@ Notation: x [T, width] is the residual stream of one sequence, t / i / j are pos
 """
 from __future__ import annotations
 
-import math
 from dataclasses import dataclass, field
 from typing import Callable, Dict, List, Optional
 
@@ -21,27 +20,25 @@ def rms(v: torch.Tensor, eps: float) -> torch.Tensor:
     return v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps)
 
 
-def rotate_half(x: torch.Tensor, base: float, dims: int, first: int = 0) -> torch.Tensor:
-    """x [T, heads, D]: channels i and i + dims / 2 turn by (first + t) * base^(-2 i / dims); channels >= dims pass."""
+def turn(u: torch.Tensor, v: torch.Tensor, base: float, dims: int, i: int):
+    """Pair i of a head at every position t: turned by t * base^(-2 i / dims).  u, v [T, heads]."""
+    a = torch.arange(u.shape[0], dtype=u.dtype)[:, None] * base ** (-2.0 * i / dims)
+    return u * torch.cos(a) - v * torch.sin(a), v * torch.cos(a) + u * torch.sin(a)
+
+
+def rotate_half(x: torch.Tensor, base: float, dims: int) -> torch.Tensor:
+    """x [T, heads, D]: channels i and i + dims / 2 are pair i; channels >= dims pass."""
     out = x.clone()
-    for t in range(x.shape[0]):
-        for i in range(dims // 2):
-            a = (first + t) * base ** (-2.0 * i / dims)
-            u, v = x[t, :, i], x[t, :, i + dims // 2]
-            out[t, :, i] = u * math.cos(a) - v * math.sin(a)
-            out[t, :, i + dims // 2] = v * math.cos(a) + u * math.sin(a)
+    for i in range(dims // 2):
+        out[:, :, i], out[:, :, i + dims // 2] = turn(x[:, :, i], x[:, :, i + dims // 2], base, dims, i)
     return out
 
 
-def rotate_pairs(x: torch.Tensor, base: float, dims: int, first: int = 0) -> torch.Tensor:
-    """The same with neighbouring channels 2 i and 2 i + 1 as the pair."""
+def rotate_pairs(x: torch.Tensor, base: float, dims: int) -> torch.Tensor:
+    """The same with the neighbours 2 i and 2 i + 1 as pair i."""
     out = x.clone()
-    for t in range(x.shape[0]):
-        for i in range(dims // 2):
-            a = (first + t) * base ** (-2.0 * i / dims)
-            u, v = x[t, :, 2 * i], x[t, :, 2 * i + 1]
-            out[t, :, 2 * i] = u * math.cos(a) - v * math.sin(a)
-            out[t, :, 2 * i + 1] = v * math.cos(a) + u * math.sin(a)
+    for i in range(dims // 2):
+        out[:, :, 2 * i], out[:, :, 2 * i + 1] = turn(x[:, :, 2 * i], x[:, :, 2 * i + 1], base, dims, i)
     return out
 
 

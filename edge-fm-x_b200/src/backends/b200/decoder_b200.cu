@@ -302,7 +302,7 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
         EFM_TRY(act(&m->ex_in, (size_t)m->ex_rows * Wp));
         EFM_TRY(act(&m->ex_act, (size_t)m->ex_rows * ex_ff));
         if (m->f32) EFM_TRY(dev_alloc(c, &m->ex_gu, (size_t)m->ex_rows * 2 * ex_ff));
-        EFM_TRY(dev_alloc(c, &m->ex_y, (size_t)m->ex_rows * Wp));
+        EFM_TRY(act(&m->ex_y, (size_t)m->ex_rows * Wp));
         EFM_TRY(dev_alloc(c, &m->route_logits, S * w_route));
         EFM_TRY(dev_alloc(c, &m->ex.id, picks));
         EFM_TRY(dev_alloc(c, &m->ex.weight, picks));
@@ -315,6 +315,7 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
         EFM_TRY(dev_alloc(c, &m->d_act, w_act));
         EFM_TRY(dev_alloc(c, &m->d_route_id, top));
         EFM_TRY(dev_alloc(c, &m->d_route_w, top));
+        EFM_TRY(dev_alloc(c, &m->d_route_ticket, 1));
     }
     EFM_TRY(act(&m->proj_a, S * w_in));
     EFM_TRY(act(&m->q, S * w_q));

@@ -42,7 +42,9 @@ struct Pending {
 
 template <Epi EPI>
 void launch_gemv_ext(efm_b200_ctx& c, Launcher& L, const GemvParams& p) {
-    const int ks = plan_gemv_ksplit(p.n_items, p.K, c.num_sms);
+    int ks = plan_gemv_ksplit(p.n_items, p.K, c.num_sms);
+    if (EPI == Epi::Router)                                            // few rows: one chunk per lane, over as many blocks as that takes
+        while (ks * 2 <= kGemvWarps && ks * 32 < p.K / 8 && p.n_items * ks * 2 <= c.num_sms * kGemvWarps) ks *= 2;
     // Logits publishes one maximum per block of a full grid; the others launch no idle blocks
     const int per = kGemvWarps / ks, need = (p.n_items + per - 1) / per;
     const int grid = EPI == Epi::Logits ? c.num_sms : std::min(c.num_sms, need);
@@ -118,11 +120,11 @@ DeltaShape delta_shape(const DecoderModel& m, const DecoderLayer& l) {
     return s;
 }
 
-template <typename TC, int VM>
+template <typename TC, int VM, bool ROT>
 void launch_attn_decode_v(Launcher& L, const WindowDecodeParams<TC>& p, int cluster) {
     const int hb = (p.s.H / p.s.G + wd::kHeads - 1) / wd::kHeads;
     L.cluster_x = cluster;
-    L.launch(window_attention_decode_kernel<TC, VM>, dim3(cluster, p.s.G * hb), dim3(wd::kThreads), sizeof(wd::Smem<VM>), p);
+    L.launch(window_attention_decode_kernel<TC, VM, ROT>, dim3(cluster, p.s.G * hb), dim3(wd::kThreads), sizeof(wd::Smem<VM>), p);
 }
 template <typename TC>
 void launch_attn_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const KvSlot& slot, bool early) {
@@ -143,9 +145,10 @@ void launch_attn_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, con
     int cluster = 1;
     while (cluster < pages && cluster < m.attn_cluster) cluster *= 2;
     const int v = std::max(l.Dp, l.Vp);
-    if (v <= 64) launch_attn_decode_v<TC, 64>(L, p, cluster);
-    else if (v <= 128) launch_attn_decode_v<TC, 128>(L, p, cluster);
-    else launch_attn_decode_v<TC, 256>(L, p, cluster);
+    const bool rot = p.s.rot.kind != kRotNone;
+    if (v <= 64) rot ? launch_attn_decode_v<TC, 64, true>(L, p, cluster) : launch_attn_decode_v<TC, 64, false>(L, p, cluster);
+    else if (v <= 128) rot ? launch_attn_decode_v<TC, 128, true>(L, p, cluster) : launch_attn_decode_v<TC, 128, false>(L, p, cluster);
+    else rot ? launch_attn_decode_v<TC, 256, true>(L, p, cluster) : launch_attn_decode_v<TC, 256, false>(L, p, cluster);
 }
 
 // ---- latent attention, absorbed form: a decode step, or rows of a pass ---------------------------------------------------
@@ -284,7 +287,11 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
             stream_input(c, r, pend, false, l.pre2);
             r.x_out = m.d_h;
             r.out_f = m.d_route;
-            gemv_ext<Epi::Store32>(c, L, l.router, r);
+            r.route = route_shape(l);
+            r.route_id = m.d_route_id;
+            r.route_w = m.d_route_w;
+            r.route_ticket = m.d_route_ticket;
+            gemv_ext<Epi::Router>(c, L, l.router, r);
             GemvParams p{};
             p.prologue = kProPlain;
             p.W = l.expert_in.w;
@@ -294,7 +301,6 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
             p.N = 2 * p.n_items;
             p.state = c.state;
             p.route = route_shape(l);
-            p.route_logits = m.d_route;
             p.route_id = m.d_route_id;
             p.route_w = m.d_route_w;
             p.ff = l.d.expert_ff;
@@ -474,7 +480,7 @@ void launch_latent_tc(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const
     DecoderModel& m = *c.decoder;
     const LatentShape z = latent_shape(m, l);
     const int LR = z.Lc + z.Rc, n_ws = tiles.n_ws * kPageTokens, ld = l.ukv.Np;
-    L.launch(latent_gather_rows_kernel<__nv_bfloat16>, dim3(tiles.n_ws), dim3(256), 0, static_cast<const __nv_bfloat16*>(run.k_pool), m.ws_c, LR, plan,
+    L.launch(latent_gather_rows_kernel<__nv_bfloat16>, dim3(tiles.n_ws, 4), dim3(256), 0, static_cast<const __nv_bfloat16*>(run.k_pool), m.ws_c, LR, plan,
              tiles.ws_pages, tiles.ws_page0);
     GemmParams g{m.ws_c, l.ukv.w, nullptr, m.ws_kv, nullptr, n_ws, l.ukv.Np, l.ukv.Kp};
     g.lda = LR;
@@ -517,8 +523,8 @@ void attention_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const D
     TA* vp = static_cast<TA*>(run.v_pool);
     int lanes = 8;                                                  // 8 channels each: at most 256 (padded) channels a head
     while (lanes * 8 < std::max(s.Dp, s.Vp)) lanes *= 2;
-    L.launch(qk_scatter_rows_kernel<TA, TA, TA>, dim3(plan.rows), dim3(256), 0, static_cast<const TA*>(m.proj_a), l.in.Np, static_cast<TA*>(m.q), kp, vp, s, plan,
-             lanes);
+    L.launch(s.rot.kind != kRotNone ? qk_scatter_rows_kernel<TA, TA, TA, true> : qk_scatter_rows_kernel<TA, TA, TA, false>, dim3(plan.rows), dim3(256), 0,
+             static_cast<const TA*>(m.proj_a), l.in.Np, static_cast<TA*>(m.q), kp, vp, s, plan, lanes);
     auto cuda_cores = [&](const RowTile* list, int n) {
         if (n > 0)
             L.launch(window_attention_rows_kernel<TA, TA, TA>, dim3(n, s.H), dim3(256), wa::rows_smem_bytes(s.Dp, s.Vp), static_cast<const TA*>(m.q),
@@ -568,7 +574,7 @@ void latent_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const Deco
 // Routed experts of all rows: choice, rows sorted by expert, two grouped products.  The outputs stay sorted (m.ex_y); the norm
 // that follows sums them (SumOf).
 template <typename TA>
-SumOf expert_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const void* h, int T) {
+SumOf<TA> expert_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const void* h, int T) {
     DecoderModel& m = *c.decoder;
     const RouteShape r = route_shape(l);
     linear_f32(c, L, l.router, h, m.route_logits, T);
@@ -585,20 +591,20 @@ SumOf expert_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const voi
         product(l.expert_in, 2 * l.ffp, static_cast<const float*>(m.ex_in), m.ex_gu);
         L.launch(silu_mul_rows_kernel, dim3(max_rows / kExpertTile), dim3(256), 0, (const float*)m.ex_gu, static_cast<float*>(m.ex_act), l.ffp,
                  (const int32_t*)m.ex.n_tiles);
-        product(l.expert_out, m.Wp, static_cast<const float*>(m.ex_act), m.ex_y);
+        product(l.expert_out, m.Wp, static_cast<const float*>(m.ex_act), static_cast<float*>(m.ex_y));
     } else {
-        auto product = [&](const DecLinear& w, int n, GemmEpi epi, const void* a, void* out, float* out_f) {
-            GemmParams g{static_cast<const __nv_bfloat16*>(a), w.w, nullptr, static_cast<__nv_bfloat16*>(out), out_f, max_rows, n, w.Kp};
+        auto product = [&](const DecLinear& w, int n, GemmEpi epi, const void* a, void* out) {
+            GemmParams g{static_cast<const __nv_bfloat16*>(a), w.w, nullptr, static_cast<__nv_bfloat16*>(out), nullptr, max_rows, n, w.Kp};
             g.group_tile = m.ex.tile_expert;
             g.group_tiles = m.ex.n_tiles;
             g.group_rows = n;
             g.group_all = r.experts * n;
             launch_gemm_epi(L, epi, g, &c.state->error);
         };
-        product(l.expert_in, 2 * l.ffp, GemmEpi::SwiGlu, m.ex_in, m.ex_act, nullptr);
-        product(l.expert_out, m.Wp, GemmEpi::F32, m.ex_act, nullptr, m.ex_y);
+        product(l.expert_in, 2 * l.ffp, GemmEpi::SwiGlu, m.ex_in, m.ex_act);
+        product(l.expert_out, m.Wp, GemmEpi::Bf16Bias, m.ex_act, m.ex_y);
     }
-    return SumOf{m.ex.place, m.ex.weight, r.top, m.ex.count, r.experts};
+    return SumOf<TA>{static_cast<const TA*>(m.ex_y), m.ex.place, m.ex.weight, r.top, m.ex.count, r.experts};
 }
 
 template <typename TA>
@@ -643,7 +649,7 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
     TA* xa = static_cast<TA*>(m.xa);                            // null: 32-bit mode without input norms reads the stream itself
     const void* xin = xa != nullptr ? (const void*)xa : c.resid;
     // the stream takes a sublayer's normed output; xa becomes the next sublayer's input
-    auto add_norm = [&](const float* y, const __nv_bfloat16* w, const __nv_bfloat16* pre, const SumOf& sum = SumOf{}) {
+    auto add_norm = [&](const float* y, const __nv_bfloat16* w, const __nv_bfloat16* pre, const SumOf<TA>& sum = SumOf<TA>{}) {
         L.launch(add_norm_rows_kernel<TA>, dim3(T), dim3(256), 0, c.resid, y, w, xa, pre, m.W, m.Wp, m.d.norm_eps, sum);
     };
     launch_embed_rows(L, ids, c.embed, nullptr, c.resid, T, c.d.vocab, m.Wp, -1, 0, m.d.embed_scale);
@@ -658,8 +664,7 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
         linear_f32(c, L, l.out, m.mix, m.y, T);
         add_norm(m.y, l.post1, l.mlp() ? l.pre2 : next);
         if (l.moe()) {
-            const SumOf sum = expert_rows<TA>(c, L, l, xin, T);
-            add_norm(m.ex_y, l.post2, next, sum);
+            add_norm(nullptr, l.post2, next, expert_rows<TA>(c, L, l, xin, T));
         } else if (l.d.ff > 0) {
             linear_act(c, L, l.up, xin, m.ff, T);
             L.launch(poly_norm_rows_kernel<TA>, dim3(T), dim3(256), 0, static_cast<const TA*>(m.ff), static_cast<TA*>(m.ff2), (const __nv_bfloat16*)l.act, l.d.ff,
@@ -709,11 +714,11 @@ template <typename K>
 cudaError_t smem_attr(K kernel, size_t bytes) { return cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes); }
 
 // widest cluster the decode attention kernel can be placed with
-template <typename TC, int VM>
+template <typename TC, int VM, bool ROT>
 cudaError_t fit_cluster(int& width) {
-    cudaError_t e = smem_attr(window_attention_decode_kernel<TC, VM>, sizeof(wd::Smem<VM>));
+    cudaError_t e = smem_attr(window_attention_decode_kernel<TC, VM, ROT>, sizeof(wd::Smem<VM>));
     if (e != cudaSuccess) return e;
-    const bool wide = cudaFuncSetAttribute(window_attention_decode_kernel<TC, VM>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess;
+    const bool wide = cudaFuncSetAttribute(window_attention_decode_kernel<TC, VM, ROT>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess;
     int cs = wide ? 16 : 8;
     for (; cs > 1; cs >>= 1) {
         cudaLaunchConfig_t cfg = {};
@@ -727,7 +732,7 @@ cudaError_t fit_cluster(int& width) {
         cfg.attrs = &at;
         cfg.numAttrs = 1;
         int n = 0;
-        if (cudaOccupancyMaxActiveClusters(&n, window_attention_decode_kernel<TC, VM>, &cfg) == cudaSuccess && n >= 1) break;
+        if (cudaOccupancyMaxActiveClusters(&n, window_attention_decode_kernel<TC, VM, ROT>, &cfg) == cudaSuccess && n >= 1) break;
     }
     (void)cudaGetLastError();
     width = std::min(width, cs);
@@ -769,18 +774,18 @@ static cudaError_t fit_side_cluster(DecoderModel& m, int optin) {
     return m.side_cluster > 1 ? smem_attr(token_side_kernel, (size_t)optin - 2048) : cudaSuccess;
 }
 
-// Heads per block and cluster width of the absorbed form: the widest cluster that fits, and as few heads per block as keep
-// all clusters resident at once.
+// Heads per block and cluster width of the absorbed form.  A block reads its keys from shared memory once and the queries of
+// its heads along with them; every further block of a cluster costs exchange; clusters that are not resident wait.
 template <typename TC, int NH>
-static cudaError_t fit_latent_heads(const DecoderModel& m, DecoderLayer& l, int optin, bool& done) {
+static cudaError_t fit_latent_heads(const DecoderModel& m, DecoderLayer& l, int optin, double& best) {
     cudaError_t e = smem_attr(latent_attention_kernel<TC, true, NH>, (size_t)optin - 4096);
     if (e == cudaSuccess) e = smem_attr(latent_attention_kernel<TC, false, NH>, (size_t)optin - 4096);
     if (e != cudaSuccess) return e;
     const bool wide = cudaFuncSetAttribute(latent_attention_kernel<TC, true, NH>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess &&
                       cudaFuncSetAttribute(latent_attention_kernel<TC, false, NH>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess;
-    if (done) return cudaSuccess;
     const LatentShape s = latent_shape(m, l);
     const int groups = (l.d.heads + NH - 1) / NH, most = latent_splits(l, m.d.cache_pages, wide ? 16 : 8);
+    const int keys = std::min(m.d.cache_pages * kPageTokens, l.d.window > 0 ? l.d.window : 1 << 30);
     for (int cs = most; cs >= 1; cs >>= 1) {
         const size_t bytes = la::layout(s, NH, cs, sizeof(TC), latent_tile(s, NH, cs, sizeof(TC))).bytes;
         if (bytes > (size_t)optin - 4096) continue;
@@ -795,22 +800,23 @@ static cudaError_t fit_latent_heads(const DecoderModel& m, DecoderLayer& l, int 
         cfg.attrs = &at;
         cfg.numAttrs = 1;
         int n = 0;
-        if (cudaOccupancyMaxActiveClusters(&n, latent_attention_kernel<TC, true, NH>, &cfg) == cudaSuccess && n >= 1) {
+        if (cudaOccupancyMaxActiveClusters(&n, latent_attention_kernel<TC, true, NH>, &cfg) != cudaSuccess || n < 1) continue;
+        const double cost = ((double)keys / cs * (4 + 2 * NH) + 40.0 * cs + 400.0) * ((groups + n - 1) / n);
+        if (best < 0.0 || cost < best) {
+            best = cost;
             l.la_heads = NH;
             l.la_cluster = cs;
-            done = n >= groups || NH == 4;
-            break;
         }
     }
     (void)cudaGetLastError();
-    return cudaSuccess;
+    return best < 0.0 && NH == 4 ? cudaErrorInvalidConfiguration : cudaSuccess;
 }
 template <typename TC>
 static cudaError_t fit_latent(const DecoderModel& m, DecoderLayer& l, int optin) {
-    bool done = false;
-    cudaError_t e = fit_latent_heads<TC, 1>(m, l, optin, done);
-    if (e == cudaSuccess) e = fit_latent_heads<TC, 2>(m, l, optin, done);
-    if (e == cudaSuccess) e = fit_latent_heads<TC, 4>(m, l, optin, done);
+    double best = -1.0;
+    cudaError_t e = fit_latent_heads<TC, 1>(m, l, optin, best);
+    if (e == cudaSuccess) e = fit_latent_heads<TC, 2>(m, l, optin, best);
+    if (e == cudaSuccess) e = fit_latent_heads<TC, 4>(m, l, optin, best);
     return e;
 }
 
@@ -824,6 +830,7 @@ cudaError_t configure_decoder(DecoderModel& m) {
     if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::Logits, true>, gv);
     if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::ExpertUp, true>, gv);
     if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::ExpertDown, true>, gv);
+    if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::Router, true>, gv);
     const size_t rows = wa::rows_smem_bytes(256, 256);
     if (e == cudaSuccess) e = smem_attr(window_attention_rows_kernel<float, float, float>, rows);
     if (e == cudaSuccess) e = smem_attr(window_attention_rows_kernel<__nv_bfloat16, __nv_bfloat16, __nv_bfloat16>, rows);
@@ -848,9 +855,17 @@ cudaError_t configure_decoder(DecoderModel& m) {
     for (DecoderLayer& l : m.layers)
         if (l.d.mixer == EFM_MIXER_LATENT_ATTENTION && e == cudaSuccess) e = m.f32 ? fit_latent<float>(m, l, optin) : fit_latent<__nv_bfloat16>(m, l, optin);
     m.attn_cluster = 16;
-    if (e == cudaSuccess) e = m.f32 ? fit_cluster<float, 64>(m.attn_cluster) : fit_cluster<__nv_bfloat16, 64>(m.attn_cluster);
-    if (e == cudaSuccess) e = m.f32 ? fit_cluster<float, 128>(m.attn_cluster) : fit_cluster<__nv_bfloat16, 128>(m.attn_cluster);
-    if (e == cudaSuccess) e = m.f32 ? fit_cluster<float, 256>(m.attn_cluster) : fit_cluster<__nv_bfloat16, 256>(m.attn_cluster);
+    auto fit = [&](auto type) {
+        using TC = decltype(type);
+        if (e == cudaSuccess) e = fit_cluster<TC, 64, false>(m.attn_cluster);
+        if (e == cudaSuccess) e = fit_cluster<TC, 128, false>(m.attn_cluster);
+        if (e == cudaSuccess) e = fit_cluster<TC, 256, false>(m.attn_cluster);
+        if (e == cudaSuccess) e = fit_cluster<TC, 64, true>(m.attn_cluster);
+        if (e == cudaSuccess) e = fit_cluster<TC, 128, true>(m.attn_cluster);
+        if (e == cudaSuccess) e = fit_cluster<TC, 256, true>(m.attn_cluster);
+    };
+    if (m.f32) fit(float());
+    else fit(__nv_bfloat16());
     return e;
 }
 

@@ -78,8 +78,8 @@ struct DecoderModel {
     __nv_bfloat16 *ws_c = nullptr, *ws_kv = nullptr;
     int ws_pages = 0, ws_window = 0;      // capacity (0: no layer uses it); largest window of the layers that use it (0: no window)
     // routed experts: rows sorted by expert
-    void *ex_in = nullptr, *ex_act = nullptr;
-    float *ex_gu = nullptr, *ex_y = nullptr, *route_logits = nullptr;
+    void *ex_in = nullptr, *ex_act = nullptr, *ex_y = nullptr;
+    float *ex_gu = nullptr, *route_logits = nullptr;
     ExpertRows ex{};
     int ex_rows = 0;
     int32_t* step_buf = nullptr;          // packed per-step indices
@@ -91,6 +91,7 @@ struct DecoderModel {
     float *d_in = nullptr, *d_mix = nullptr, *d_y = nullptr, *d_y2 = nullptr, *d_ff = nullptr, *d_gate = nullptr;
     float *d_q = nullptr, *d_h = nullptr, *d_route = nullptr, *d_act = nullptr, *d_route_w = nullptr;
     int32_t* d_route_id = nullptr;
+    unsigned int* d_route_ticket = nullptr;
     int attn_cluster = 8, side_cluster = 1;
 };
 

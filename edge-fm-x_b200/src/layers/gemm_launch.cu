@@ -77,10 +77,17 @@ static void launch_gemm(Launcher& L, const GemmParams& p, int* error_word = null
     const dim3 block(tc::kThreads);
     const bool pdl = L.pdl;
     L.pdl = false;     // prefill kernels do not use the dependent-launch protocol
-    if (p.group_tile != nullptr) {
-        L.launch(gemm_tc_kernel<EPI>, dim3(std::min(L.num_sms, tiles)), block, tc::SMEM_BYTES, ma, mb, p, error_word);
-        L.pdl = pdl;
-        return;
+    if constexpr (EPI == GemmEpi::Bf16Bias || EPI == GemmEpi::SwiGlu) {
+        if (p.group_tile != nullptr) {
+            static bool attr_group = false;
+            if (!attr_group) {
+                cudaFuncSetAttribute(gemm_tc_kernel<EPI, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)tc::SMEM_BYTES);
+                attr_group = true;
+            }
+            L.launch(gemm_tc_kernel<EPI, true>, dim3(std::min(L.num_sms, tiles)), block, tc::SMEM_BYTES, ma, mb, p, error_word);
+            L.pdl = pdl;
+            return;
+        }
     }
     // Few output tiles and a long K: split K so that the whole GPU works, fp32 partials to the workspace, then
     // a fixed-order sum with the epilogue.

@@ -27,8 +27,10 @@ __device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
     return make_float4(bf16lo(v.x), bf16hi(v.x), bf16lo(v.y), bf16hi(v.y));
 }
 
-// Where a row's sublayer output comes from: row i of y, or (experts) the weighted sum of the rows place[i][..] of y.
+// Where a row's sublayer output comes from: row i of y, or (experts) the weighted sum of the rows place[i][..] of ye.
+template <typename T>
 struct SumOf {
+    const T* ye;
     const int32_t* place;             // [rows][top], null: the row itself
     const float* weight;              // [rows][top]
     int top;
@@ -36,12 +38,12 @@ struct SumOf {
     int experts;
 };
 
-// x += y / sqrt(mean(y^2) + eps) * w (y null: x unchanged); out (null: none) = x as T, or with `pre` x / sqrt(mean(x^2) + eps) * pre,
+// x += y / sqrt(mean(y^2) + eps) * w (w null: x unchanged); out (null: none) = x as T, or with `pre` x / sqrt(mean(x^2) + eps) * pre,
 // the next sublayer's input.  One block per row; the first 1024 * KEEP channels stay in registers.
 template <typename T>
 __global__ void __launch_bounds__(256) add_norm_rows_kernel(float* __restrict__ x, const float* __restrict__ y, const __nv_bfloat16* __restrict__ w,
                                                             T* __restrict__ out, const __nv_bfloat16* __restrict__ pre, int n, int ld, float eps,
-                                                            const SumOf sum) {
+                                                            const SumOf<T> sum) {
     constexpr int KEEP = 4;
     __shared__ float part[2][8];
     const size_t base = (size_t)blockIdx.x * ld;
@@ -54,24 +56,26 @@ __global__ void __launch_bounds__(256) add_norm_rows_kernel(float* __restrict__ 
         for (int k = 0; k < sum.top; ++k) {
             const size_t i = (size_t)blockIdx.x * sum.top + k;
             const float g = sum.weight[i];
-            const float4 v = load4(y + (size_t)sum.place[i] * ld + 4 * c);
+            const float4 v = load4(sum.ye + (size_t)sum.place[i] * ld + 4 * c);
             a.x = fmaf(g, v.x, a.x); a.y = fmaf(g, v.y, a.y); a.z = fmaf(g, v.z, a.z); a.w = fmaf(g, v.w, a.w);
         }
         return a;
     };
     auto square = [](float s, const float4& v) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s)))); };
-    float4 keep[KEEP];
+    float4 keep[KEEP], old[KEEP];
     float s2 = 0.f;
-    if (y != nullptr) {
+    if (w != nullptr) {
         float ss = 0.f;
 #pragma unroll
         for (int i = 0; i < KEEP; ++i)
-            if (tid + 256 * i < nv) { keep[i] = load_y(tid + 256 * i); ss = square(ss, keep[i]); }
+            if (tid + 256 * i < nv) { old[i] = load4(x + base + 4 * (tid + 256 * i)); keep[i] = load_y(tid + 256 * i); }
+#pragma unroll
+        for (int i = 0; i < KEEP; ++i)
+            if (tid + 256 * i < nv) ss = square(ss, keep[i]);
         for (int c = tid + 256 * KEEP; c < nv; c += 256) ss = square(ss, load_y(c));
         const float inv = 1.0f / sqrtf(block_sum_256(ss, part[0]) / (float)n + eps);
-        auto add = [&](int c, const float4& v) {
+        auto add = [&](int c, const float4& v, float4 r) {
             const float4 g = load4(w + 4 * c);
-            float4 r = load4(x + base + 4 * c);
             r.x += v.x * inv * g.x; r.y += v.y * inv * g.y; r.z += v.z * inv * g.z; r.w += v.w * inv * g.w;
             store4(x + base + 4 * c, r);
             s2 = square(s2, r);
@@ -80,8 +84,8 @@ __global__ void __launch_bounds__(256) add_norm_rows_kernel(float* __restrict__ 
         };
 #pragma unroll
         for (int i = 0; i < KEEP; ++i)
-            if (tid + 256 * i < nv) keep[i] = add(tid + 256 * i, keep[i]);
-        for (int c = tid + 256 * KEEP; c < nv; c += 256) (void)add(c, load_y(c));
+            if (tid + 256 * i < nv) keep[i] = add(tid + 256 * i, keep[i], old[i]);
+        for (int c = tid + 256 * KEEP; c < nv; c += 256) (void)add(c, load_y(c), load4(x + base + 4 * c));
     } else {
 #pragma unroll
         for (int i = 0; i < KEEP; ++i)

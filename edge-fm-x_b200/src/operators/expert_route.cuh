@@ -7,9 +7,8 @@ namespace efm {
 
 // z: router logits of all experts.  Scores softmax(z); the groups whose best scores are the largest stay open; the best `top`
 // experts of those are handed to store(k, expert, score) in lane 0.  Ties go to the lower number.
-template <typename Store>
-__device__ __forceinline__ void route_token(const float* z, const RouteShape& r, Store store) {
-    constexpr int N = kMaxExperts / 32;
+template <int N, typename Store>
+__device__ __forceinline__ void route_token_n(const float* z, const RouteShape& r, Store store) {      // at most 32 N experts
     const int lane = threadIdx.x & 31, per = r.experts / r.groups;
     float v[N], mx = -INFINITY, sum = 0.f;
 #pragma unroll
@@ -68,6 +67,14 @@ __device__ __forceinline__ void route_token(const float* z, const RouteShape& r,
         for (int i = 0; i < N; ++i)
             if (e == lane + 32 * i) v[i] = -2.f;
     }
+}
+template <typename Store>
+__device__ __forceinline__ void route_token(const float* z, const RouteShape& r, Store store) {
+    static_assert(kMaxExperts == 32 * 16, "widest instantiation");
+    if (r.experts <= 32) route_token_n<1>(z, r, store);
+    else if (r.experts <= 64) route_token_n<2>(z, r, store);
+    else if (r.experts <= 128) route_token_n<4>(z, r, store);
+    else route_token_n<16>(z, r, store);
 }
 
 }  // namespace efm

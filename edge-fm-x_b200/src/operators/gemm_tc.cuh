@@ -41,7 +41,7 @@ struct GemmParams {
     int tile_count = 0;       // m-fastest tile order (0: all of them).  With kb_per_split > 0 and tile_count > 0 the
                               // partial of (split z, tile t) goes to the compact slot Cf + (z * tile_count + t -
                               // tile_begin) * 128 * 256, row-major inside the tile ("tail split", see the launcher)
-    // grouped product (routed experts): rows arrive sorted by group, every group from a multiple of 128 rows on; row tile t
+    // GROUPED instantiations (routed experts): rows arrive sorted by group, every group from a multiple of 128 rows on; row tile t
     // is multiplied with rows [group_tile[t] * group_rows, + N) of B; *group_tiles row tiles are in use
     const int32_t* group_tile = nullptr;
     const int32_t* group_tiles = nullptr;
@@ -128,7 +128,7 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&r)[32]) {
 
 }  // namespace tc
 
-template <GemmEpi EPI>
+template <GemmEpi EPI, bool GROUPED = false>
 __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a,
                                                                const __grid_constant__ CUtensorMap map_b,
                                                                const GemmParams p, int* error) {
@@ -147,7 +147,7 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
     volatile int* abort_s = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int tiles_m = p.group_tiles != nullptr ? max(1, *p.group_tiles) : (p.M + BM - 1) / BM, tiles_n = (p.N + BN - 1) / BN;
+    const int tiles_m = GROUPED ? *p.group_tiles : (p.M + BM - 1) / BM, tiles_n = (p.N + BN - 1) / BN;
     const int KB_all = (p.K + BK - 1) / BK;
     const int splits = p.kb_per_split > 0 ? (KB_all + p.kb_per_split - 1) / p.kb_per_split : 1;
     const int n_tiles = p.tile_count > 0 ? p.tile_count : tiles_m * tiles_n;
@@ -185,7 +185,8 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
             for (int item = blockIdx.x; item < n_items && *abort_s == 0; item += gridDim.x) {
                 int m0, n0, kb0, kb1, z;
                 item_coords(item, m0, n0, kb0, kb1, z);
-                const int b_row = n0 + (p.group_tile != nullptr ? p.group_tile[m0 / BM] * p.group_rows : 0);
+                int b_row = n0;
+                if constexpr (GROUPED) b_row += p.group_tile[m0 / BM] * p.group_rows;
                 for (int kb = kb0; kb < kb1; ++kb, ++it) {
                     const int s = it % STAGES;
                     const uint32_t ph = (it / STAGES) & 1u;

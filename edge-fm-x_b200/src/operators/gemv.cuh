@@ -31,7 +31,7 @@
 
 namespace efm {
 
-enum class Epi : int { Plain = 0, Residual = 1, QkvRope = 2, SwiGlu = 3, Logits = 4, Peers = 5, Store32 = 6, TokenGate = 7, ExpertUp = 8, ExpertDown = 9 };
+enum class Epi : int { Plain = 0, Residual = 1, QkvRope = 2, SwiGlu = 3, Logits = 4, Peers = 5, Store32 = 6, TokenGate = 7, ExpertUp = 8, ExpertDown = 9, Router = 10 };
 constexpr int kMaxPeers = 8;
 // The last four (and the epilogues from Store32 on) exist in the EXT instantiations only (layered decoders):
 //   Embed    x = embed_table[token] * embed_scale; with norm2_w the product reads rmsnorm(x) * norm2_w
@@ -97,11 +97,11 @@ struct GemvParams {
     int gate_ld, gate_off;
     float embed_scale;
     float* x_out;             // not null: block 0 stores the input of the product here (what the norms left)
-    // ExpertUp: the experts of this token are chosen from route_logits (block 0 publishes ids and weights); item = (choice,
-    // channel), out_f[choice * ffp + channel] = silu(gate) * up.  ExpertDown: x = the choices' activations times their
-    // weights, K = choices * ffp, the row of W jumps from expert to expert.
+    // Router: out_f = logits; the block that finishes last chooses this token's experts and publishes ids and weights.
+    // ExpertUp: item = (choice, channel), out_f[choice * ffp + channel] = silu(gate) * up.  ExpertDown: x = the choices'
+    // activations times their weights, K = choices * ffp, the row of W jumps from expert to expert.
     RouteShape route;
-    const float* route_logits;
+    unsigned int* route_ticket;           // zero between launches
     int32_t* route_id;        // [top]
     float* route_w;           // [top]
     int ff, ffp, expert_rows; // channels, padded channels, rows of one expert's matrix
@@ -181,6 +181,8 @@ __device__ __forceinline__ void item_epilogue(const GemvParams& p, int item, flo
         p.out_f[k * p.ffp + item - k * p.ff] = a0 / (1.0f + expf(-a0)) * a1;
     } else if constexpr (EPI == Epi::ExpertDown) {
         *reinterpret_cast<float2*>(p.out_f + item * 2) = make_float2(a0, a1);
+    } else if constexpr (EPI == Epi::Router) {
+        __stcg(reinterpret_cast<float2*>(p.out_f + item * 2), make_float2(a0, a1));
     } else if constexpr (EPI == Epi::Store32) {
         if (p.bias != nullptr) {
             a0 += __bfloat162float(p.bias[item * 2]);
@@ -566,7 +568,7 @@ __device__ __forceinline__ void gemv_stage(const GemvParams& p, const int nch, u
 // Stage activations (with the fused norm), stream the rows, reduce, epilogue.
 template <Epi EPI, bool EXT>
 __device__ __forceinline__ void gemv_run(const GemvParams& p, const GemvSched& sc, GemvRegs& r, unsigned char* smem,
-                                         const unsigned int xbytes, float& best_v, int& best_i) {
+                                         const unsigned int xbytes, float& best_v, int& best_i, const int* early_chosen = nullptr) {
     const float* xs = reinterpret_cast<const float*>(smem);
     float* red = reinterpret_cast<float*>(smem + xbytes + gemv_wbytes(p.K));
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -578,22 +580,16 @@ __device__ __forceinline__ void gemv_run(const GemvParams& p, const GemvSched& s
         if (sc.wk == 0 && lane == 0 && sc.total > 0)
             old_first = __ldcg(reinterpret_cast<const float2*>(p.residual + sc.ig0 * 2));
     }
-    __shared__ int chosen_s[EPI == Epi::ExpertUp || EPI == Epi::ExpertDown ? kMaxExpertTop : 1];
+    __shared__ int chosen_s[EPI == Epi::ExpertUp ? kMaxExpertTop : 1];
     const int* chosen = nullptr;
     if constexpr (EPI == Epi::ExpertUp) {
-        if (warp == 0)
-            route_token(p.route_logits, p.route, [&](int k, int e, float w) {
-                chosen_s[k] = e;
-                if (blockIdx.x == 0) { p.route_id[k] = e; p.route_w[k] = w; }
-            });
-        chosen = chosen_s;
-        gemv_stage(p, nch, smem, xbytes);                              // ends with a block barrier
-        gemv_load_unit<EPI>(p, sc, 0, r.a, chosen);
-    } else if constexpr (EPI == Epi::ExpertDown) {
         if (tid < p.route.top) chosen_s[tid] = __ldcg(p.route_id + tid);
         chosen = chosen_s;
         __syncthreads();
         gemv_load_unit<EPI>(p, sc, 0, r.a, chosen);
+        gemv_stage(p, nch, smem, xbytes);
+    } else if constexpr (EPI == Epi::ExpertDown) {
+        chosen = early_chosen;
         float* xw = reinterpret_cast<float*>(smem);
         for (int c = tid; c < 2 * nch; c += kGemvThreads) {            // padded channels are zero
             const float w = __ldcg(p.route_w + 4 * c / p.ffp);
@@ -607,6 +603,7 @@ __device__ __forceinline__ void gemv_run(const GemvParams& p, const GemvSched& s
         gemv_stage(p, nch, smem, xbytes);
     }
     (void)tid;
+    (void)early_chosen;
 
     // ---- rows ------------------------------------------------------------------------------------
     float acc0 = 0.f, acc1 = 0.f;
@@ -688,12 +685,35 @@ __global__ void __launch_bounds__(kGemvThreads, 1) gemv_kernel(const GemvParams 
     int best_i = 0x7fffffff;
     // Let the next kernel of the step start its own weight prefetch as soon as every block of this
     // one is resident, then prefetch (independent of every earlier kernel), then wait.
-    pdl_launch_dependents();
+    // ExpertUp holds its dependents back until its own wait is over: the choice it waits for is then there for ExpertDown,
+    // which fetches its first weights before its wait.
+    if constexpr (EPI != Epi::ExpertUp) pdl_launch_dependents();
     const GemvSched sc = gemv_sched(p, ks, blockIdx.x, gridDim.x);
+    __shared__ int early_s[EPI == Epi::ExpertDown ? kMaxExpertTop : 1];
+    if constexpr (EPI == Epi::ExpertDown) {
+        if ((int)threadIdx.x < p.route.top) early_s[threadIdx.x] = __ldcg(p.route_id + threadIdx.x);
+        __syncthreads();
+        gemv_load_unit<EPI>(p, sc, 0, regs.a, early_s);
+    }
     gemv_prefetch<EPI, EXT>(p, sc, regs, gemv_smem, xbytes);
     pdl_wait();
+    if constexpr (EPI == Epi::ExpertUp) pdl_launch_dependents();
     if constexpr (EPI == Epi::Peers) best_i = (int)(__ldcg(p.epoch) + 1u);      // this launch's exchange count rides in best_i
-    gemv_run<EPI, EXT>(p, sc, regs, gemv_smem, xbytes, best_v, best_i);
+    gemv_run<EPI, EXT>(p, sc, regs, gemv_smem, xbytes, best_v, best_i, EPI == Epi::ExpertDown ? early_s : nullptr);
+    if constexpr (EPI == Epi::Router) {
+        __shared__ unsigned int last;
+        __syncthreads();
+        if (threadIdx.x == 0) {
+            __threadfence();
+            last = atomicAdd(p.route_ticket, 1u) == gridDim.x - 1 ? 1u : 0u;
+            __threadfence();
+        }
+        __syncthreads();
+        if (last != 0u && threadIdx.x < 32) {
+            route_token(p.out_f, p.route, [&](int k, int e, float w) { p.route_id[k] = e; p.route_w[k] = w; });
+            if (threadIdx.x == 0) *p.route_ticket = 0u;
+        }
+    }
     if constexpr (EPI == Epi::Logits) gemv_publish_best(p, best_v, best_i, bv, bi);
     if constexpr (EPI == Epi::Peers) {
         // every block has read the count by now; the one that draws the last ticket advances it for the consumer

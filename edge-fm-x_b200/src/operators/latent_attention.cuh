@@ -42,20 +42,33 @@ struct LatentShape {
 };
 
 // ---- many rows -----------------------------------------------------------------------------------------------------
+// One block per row, 8 channels per thread and turn (every part is a multiple of 8); the first 8 * 256 channels stay in registers.
 template <typename T>
 __global__ void __launch_bounds__(256) latent_rows_kernel(const T* __restrict__ proj, int ld, T* __restrict__ cq, T* __restrict__ pool, const LatentShape s,
                                                           const RowPlan plan) {
-    __shared__ float part[2][8], cs[kRotMaxPairs], sn[kRotMaxPairs], rot[256];
+    __shared__ float part[2][8], cs[kRotMaxPairs], sn[kRotMaxPairs];
+    __shared__ __align__(16) float rot[256];
     const int row = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const RowEntry e = plan.of_row(row);
-    const int pos = e.pos0 + row - e.row0;
+    const int pos = e.pos0 + row - e.row0, nq = s.Qp / 8, nc = s.Lc / 8, n = nq + nc + s.Rc / 8;
     const T* src = proj + (size_t)row * ld;
-    T* dst = pool + plan.cache_row(e, pos) * (s.Lc + s.Rc);
+    float keep[8], a = 0.f, b = 0.f;                                    // pads are zero
+    for (int c = tid; c < n; c += 256) {
+        float f[8];
+        load8_as_f32(src + 8 * c, f);
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            ss = fmaf(f[j], f[j], ss);
+            if (c == tid) keep[j] = f[j];
+        }
+        if (c < nq) a += ss;
+        else if (c < nq + nc) b += ss;
+        else
+#pragma unroll
+            for (int j = 0; j < 8; ++j) rot[8 * (c - nq - nc) + j] = f[j];
+    }
     rot_table(s.rot, pos, cs, sn);
-    float a = 0.f, b = 0.f;                                             // pads are zero
-    for (int c = tid; c < s.Qp; c += 256) { const float v = to_f32(src[c]); a = fmaf(v, v, a); }
-    for (int c = tid; c < s.Lc; c += 256) { const float v = to_f32(src[s.off_c() + c]); b = fmaf(v, v, b); }
-    for (int c = tid; c < s.Rc; c += 256) rot[c] = to_f32(src[s.off_r() + c]);
     a = warp_sum(a);
     b = warp_sum(b);
     if (lane == 0) { part[0][warp] = a; part[1][warp] = b; }
@@ -64,9 +77,24 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const T* __restrict__ 
 #pragma unroll
     for (int i = 0; i < 8; ++i) { a += part[0][i]; b += part[1][i]; }
     const float ia = 1.0f / sqrtf(a / (float)s.q_rank + s.eps), ib = 1.0f / sqrtf(b / (float)s.L + s.eps);
-    for (int c = tid; c < s.Qp; c += 256) store_f32(cq + (size_t)row * s.Qp + c, to_f32(src[c]) * ia * __bfloat162float(s.q_norm[c]));
-    for (int c = tid; c < s.Lc; c += 256) store_f32(dst + c, to_f32(src[s.off_c() + c]) * ib * __bfloat162float(s.kv_norm[c]));
-    for (int c = tid; c < s.Rc; c += 256) store_f32(dst + s.Lc + c, rot_channel(s.rot, rot, c, cs, sn));
+    T* dst = pool + plan.cache_row(e, pos) * (s.Lc + s.Rc);
+    for (int c = tid; c < n; c += 256) {
+        float f[8], w[8];
+        if (c == tid)
+#pragma unroll
+            for (int j = 0; j < 8; ++j) f[j] = keep[j];
+        else load8_as_f32(src + 8 * c, f);
+        if (c < nq + nc) {
+            unpack8(ld_cached(c < nq ? s.q_norm + 8 * c : s.kv_norm + 8 * (c - nq)), w);
+            const float inv = c < nq ? ia : ib;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) f[j] *= inv * w[j];
+        } else {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) f[j] = rot_channel(s.rot, rot, 8 * (c - nq - nc) + j, cs, sn);
+        }
+        store_head8(c < nq ? cq + (size_t)row * s.Qp + 8 * c : dst + 8 * (c - nq), f);
+    }
 }
 
 template <typename T>
@@ -76,17 +104,37 @@ __global__ void __launch_bounds__(256) latent_rotate_rows_kernel(T* __restrict__
     const RowEntry e = plan.of_row(row);
     rot_table(s.rot, e.pos0 + row - e.row0, cs, sn);
     __syncthreads();
-    const int step = s.rot.kind == kRotHalf ? 1 : 2, apart = s.rot.kind == kRotHalf ? pairs : 1;
+    T* base = q + (size_t)row * s.q_ld() + s.Dp;
+    const int ld = s.Dp + s.Rc;
+    if (s.rot.kind == kRotPairs) {                                      // pairs are neighbours: 8 channels per thread
+        const int per = s.Rc / 8;
+        for (int n = threadIdx.x; n < s.H * per; n += 256) {
+            const int h = n / per, c = (n - h * per) * 8;
+            T* x = base + (size_t)h * ld + c;
+            float f[8];
+            load8_as_f32(x, f);
+#pragma unroll
+            for (int j = 0; j < 8; j += 2) {
+                const int i = (c + j) >> 1;
+                if (i >= pairs) continue;
+                const float u = f[j], v = f[j + 1];
+                f[j] = u * cs[i] - v * sn[i];
+                f[j + 1] = v * cs[i] + u * sn[i];
+            }
+            store_head8(x, f);
+        }
+        return;
+    }
     for (int n = threadIdx.x; n < s.H * pairs; n += 256) {
         const int h = n / pairs, i = n - h * pairs;
-        T* x = q + (size_t)row * s.q_ld() + (size_t)h * (s.Dp + s.Rc) + s.Dp + i * step;
-        const float u = to_f32(x[0]), v = to_f32(x[apart]);
+        T* x = base + (size_t)h * ld + i;
+        const float u = to_f32(x[0]), v = to_f32(x[pairs]);
         store_f32(x, u * cs[i] - v * sn[i]);
-        store_f32(x + apart, v * cs[i] + u * sn[i]);
+        store_f32(x + pairs, v * cs[i] + u * sn[i]);
     }
 }
 
-// One block per page: pages[i] = (entry, page of its sequence); null: page0 + i of the single entry.
+// Grid (pages, parts of a page): pages[i] = (entry, page of its sequence); null: page0 + i of the single entry.
 template <typename T>
 __global__ void __launch_bounds__(256) latent_gather_rows_kernel(const T* __restrict__ pool, T* __restrict__ ws, int row_elems, const RowPlan plan,
                                                                  const RowTile* __restrict__ pages, int page0) {
@@ -94,9 +142,9 @@ __global__ void __launch_bounds__(256) latent_gather_rows_kernel(const T* __rest
     const RowEntry e = plan.entry(t.entry);
     const uint4* src = reinterpret_cast<const uint4*>(pool + plan.cache_row(e, t.row * kPageTokens) * row_elems);
     uint4* dst = reinterpret_cast<uint4*>(ws + (size_t)(e.ws0 + t.row * kPageTokens) * row_elems);
-    // rows past the entry's last token hold what an earlier owner of the page left: any finite values, never visible
+    // rows past the entry's last token hold what an earlier owner of the page left: zeros instead, never visible
     const int n = min(kPageTokens, e.pos0 + e.n - t.row * kPageTokens), per = row_elems * (int)sizeof(T) / 16;
-    for (int i = threadIdx.x; i < kPageTokens * per; i += 256) dst[i] = i < n * per ? src[i] : make_uint4(0, 0, 0, 0);
+    for (int i = blockIdx.y * 256 + threadIdx.x; i < kPageTokens * per; i += 256 * gridDim.y) dst[i] = i < n * per ? src[i] : make_uint4(0, 0, 0, 0);
 }
 
 // ---- one row, absorbed -----------------------------------------------------------------------------------------------
@@ -420,18 +468,23 @@ __global__ void __launch_bounds__(la::kThreads) latent_attention_kernel(const La
         for (int r = 0; r < n_splits; ++r) *cl.map_shared_rank(olat + h * s.Lc + s0 + c, r) = v;
     }
     if (n_splits > 1) cl.sync(); else __syncthreads();
-    // ---- values and gate: one warp per value row -------------------------------------------------------------------------------
-    for (int v = v0 + warp; v < v1; v += kThreads / 32) {
-        const int h = v / s.Dv, c = v - h * s.Dv;
-        const __nv_bfloat16* w = s.wv + ((size_t)(h0 + h) * s.Vp + c) * s.Lc;
+    // ---- values and gate: as many lanes per value row as keep every warp's rows in flight together --------------------------
+    int lanes = 32;
+    while (lanes > 4 && (kThreads / lanes) < v1 - v0) lanes /= 2;
+    for (int vb = v0; vb < v1; vb += kThreads / lanes) {
+        const int v = vb + tid / lanes, li = tid % lanes, h = v < v1 ? v / s.Dv : 0, c = v - h * s.Dv;
         float a = 0.f;
-        for (int i = lane; i < s.Lc / 8; i += 32) {
-            const float4 x = *reinterpret_cast<const float4*>(olat + h * s.Lc + i * 8), y = *reinterpret_cast<const float4*>(olat + h * s.Lc + i * 8 + 4);
-            const float f[8] = {x.x, x.y, x.z, x.w, y.x, y.y, y.z, y.w};
-            a = dot8(ld_cached(w + i * 8), f, a);
+        if (v < v1) {
+            const __nv_bfloat16* w = s.wv + ((size_t)(h0 + h) * s.Vp + c) * s.Lc;
+#pragma unroll 4
+            for (int i = li; i < s.Lc / 8; i += lanes) {
+                const float4 x = *reinterpret_cast<const float4*>(olat + h * s.Lc + i * 8), y = *reinterpret_cast<const float4*>(olat + h * s.Lc + i * 8 + 4);
+                const float f[8] = {x.x, x.y, x.z, x.w, y.x, y.y, y.z, y.w};
+                a = dot8(ld_cached(w + i * 8), f, a);
+            }
         }
-        a = warp_sum(a);
-        if (lane == 0) {
+        for (int o = lanes / 2; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
+        if (li == 0 && v < v1) {
             if (s.gate) {
                 const TI* gp = p.proj + (size_t)row * p.ld + s.off_gate() + (h0 + h) * s.Dv + c;
                 float g;

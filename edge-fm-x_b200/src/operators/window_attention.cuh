@@ -87,14 +87,15 @@ __device__ __forceinline__ void store_head8(T* p, const float (&f)[8]) {        
 }
 
 // One block per row; `lanes` (8, 16 or 32) threads share a head, 8 channels each.  TI: projections, TQ: q operand, TC: cache.
-template <typename TI, typename TQ, typename TC>
+template <typename TI, typename TQ, typename TC, bool ROT>
 __global__ void __launch_bounds__(256) qk_scatter_rows_kernel(const TI* __restrict__ qkv, int ld, TQ* __restrict__ q_out, TC* __restrict__ k_pool,
                                                               TC* __restrict__ v_pool, const WindowAttnShape s, const RowPlan plan, int lanes) {
-    __shared__ float cs[kRotMaxPairs], sn[kRotMaxPairs], stage[256 * 8];
+    __shared__ __align__(16) float cs[kRotMaxPairs], sn[kRotMaxPairs], stage[ROT ? 256 * 8 : 1];
     const int row = blockIdx.x, l = threadIdx.x & (lanes - 1), per = 256 / lanes;
     const RowEntry e = plan.of_row(row);
-    float* st = stage + (threadIdx.x & ~(lanes - 1)) * 8;              // this head's channels
-    if (s.rot.kind != kRotNone) {
+    const int half = s.rot.dims / 2;
+    const bool by_lanes = s.rot.kind == kRotHalf && (half & 7) == 0;   // a channel's partner sits in the same place of another lane
+    if constexpr (ROT) {
         rot_table(s.rot, e.pos0 + row - e.row0, cs, sn);
         __syncthreads();
     }
@@ -118,15 +119,26 @@ __global__ void __launch_bounds__(256) qk_scatter_rows_kernel(const TI* __restri
 #pragma unroll
             for (int j = 0; j < 8; ++j) f[j] = d + j < s.D ? f[j] * inv * (w != nullptr ? __bfloat162float(w[d + j]) : 1.f) : 0.f;
         }
-        if (s.rot.kind != kRotNone) {                                  // the lanes of a head exchange channels
+        if constexpr (ROT) {
+            if (by_lanes) {
+                const bool low = d < half, in = d < s.rot.dims;
+                const int src = in ? (low ? l + half / 8 : l - half / 8) : l, i0 = in ? (low ? d : d - half) : 0;
 #pragma unroll
-            for (int j = 0; j < 8; ++j) st[d + j] = f[j];
-            __syncwarp();
-            if (qk && d < s.rot.dims) {
+                for (int j = 0; j < 8; ++j) {
+                    const float o = __shfl_sync(0xffffffffu, f[j], src, lanes);
+                    if (qk && in) f[j] = low ? f[j] * cs[i0 + j] - o * sn[i0 + j] : f[j] * cs[i0 + j] + o * sn[i0 + j];
+                }
+            } else {
+                float* st = stage + (threadIdx.x & ~(lanes - 1)) * 8;  // this head's channels
 #pragma unroll
-                for (int j = 0; j < 8; ++j) f[j] = rot_channel(s.rot, st, d + j, cs, sn);
+                for (int j = 0; j < 8; ++j) st[d + j] = f[j];
+                __syncwarp();
+                if (qk && d < s.rot.dims) {
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) f[j] = rot_channel(s.rot, st, d + j, cs, sn);
+                }
+                __syncwarp();
             }
-            __syncwarp();
         }
         if (qk) {
             if (d < s.Dp) {
@@ -307,7 +319,7 @@ template <> struct Row4<float> {
 
 // grid (splits = cluster size, kv_heads * head blocks); the visible keys (kept first tokens, then the window) are numbered in
 // order and dealt out evenly, block `split` walks its share in tiles of 64.  VM: upper bound of Dp and Vp.
-template <typename TC, int VM>
+template <typename TC, int VM, bool ROT>
 __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(const WindowDecodeParams<TC> p) {
     using namespace wd;
     constexpr int KC = VM / 32;                                        // 8-channel chunks per thread and key (4 threads per key)
@@ -357,9 +369,11 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
         }
     };
     if (begin < end) load_tile(begin);
-    if (ok) rot_table(s.rot, pos, sm.cs, sm.sn);
+    if constexpr (ROT) {
+        if (ok) rot_table(s.rot, pos, sm.cs, sm.sn);
+        __syncthreads();
+    }
     if (p.early) { pdl_wait(); pdl_launch_dependents(); }
-    if (s.rot.kind != kRotNone) __syncthreads();
 
     // ---- norms and rotation of this token's q heads and k, v ------------------------------------------------------------------
     for (int u = warp; u < nh + 1; u += 8) {
@@ -380,22 +394,24 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
             const int d = lane + 32 * i;
             if (d >= s.Dp) continue;
             const float v = d < s.D ? f[i] * inv * (w != nullptr ? __bfloat162float(w[d]) : 1.f) : 0.f;
-            if (is_q) sm.q[u][d] = v; else sm.knew[d] = v;
+            if (is_q) sm.q[u][d] = v; else sm.knew[d] = ROT ? v : round_as<TC>(v);
         }
-        float* y = is_q ? sm.q[u] : sm.knew;
-        __syncwarp();
+        if constexpr (ROT) {
+            float* y = is_q ? sm.q[u] : sm.knew;
+            __syncwarp();
 #pragma unroll
-        for (int i = 0; i < VM / 32; ++i) {
-            const int d = lane + 32 * i;
-            if (d < s.Dp) {
-                f[i] = s.rot.kind != kRotNone ? rot_channel(s.rot, y, d, sm.cs, sm.sn) : y[d];
-                if (!is_q) f[i] = round_as<TC>(f[i]);
+            for (int i = 0; i < VM / 32; ++i) {
+                const int d = lane + 32 * i;
+                if (d < s.Dp) {
+                    f[i] = rot_channel(s.rot, y, d, sm.cs, sm.sn);
+                    if (!is_q) f[i] = round_as<TC>(f[i]);
+                }
             }
-        }
-        __syncwarp();
+            __syncwarp();
 #pragma unroll
-        for (int i = 0; i < VM / 32; ++i)
-            if (lane + 32 * i < s.Dp) y[lane + 32 * i] = f[i];
+            for (int i = 0; i < VM / 32; ++i)
+                if (lane + 32 * i < s.Dp) y[lane + 32 * i] = f[i];
+        }
     }
     for (int d = tid; d < s.Vp; d += kThreads)
         sm.vnew[d] = d < s.Dv ? round_as<TC>(__ldcg(p.qkv + (size_t)(s.H + s.G) * s.D + (size_t)g * s.Dv + d)) : 0.f;

@@ -21,11 +21,14 @@ constexpr int BM = 128, BN = kPageTokens, kThreads = 256, kMaxTiles = 1024;
 template <int DP, int VP, int RP = 0>
 struct Cfg {
     static constexpr int QB = (DP + RP) / 64, VB = VP / 64;  // 64-channel boxes per row
+    // Wide keys have one buffer: the next tile is requested when S of this one is done and has the softmax's time to arrive,
+    // and two blocks fit on an SM.
+    static constexpr int KBUF = DP + RP > 128 ? 1 : 2;
     static constexpr int Q_BYTES = BM * 128 * QB, K_BYTES = BN * 128 * QB, V_BYTES = BN * 128 * VB;
     static constexpr int P_COL = 64, O_COL = 128;
     static constexpr int TMEM_COLS = 256;                    // S (64 columns) | P high, P low (32 each) | O tile, power of two
     static constexpr int HALF = VP / 2;
-    static constexpr size_t SMEM = (size_t)Q_BYTES + 2 * K_BYTES + V_BYTES + 2 * BM * 4 + 128 + kMaxTiles * 4 + 1024;
+    static constexpr size_t SMEM = (size_t)Q_BYTES + KBUF * K_BYTES + V_BYTES + 2 * BM * 4 + 128 + kMaxTiles * 4 + 1024;
 };
 
 __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16]) {
@@ -70,8 +73,8 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     const uint32_t raw = smem_u32(wt_smem);
     const uint32_t base = (raw + 1023u) & ~1023u;
     unsigned char* base_ptr = wt_smem + (base - raw);
-    const uint32_t sQ = base, sK = sQ + C::Q_BYTES, sV = sK + 2 * C::K_BYTES;
-    constexpr int XCH = C::Q_BYTES + 2 * C::K_BYTES + C::V_BYTES;
+    const uint32_t sQ = base, sK = sQ + C::Q_BYTES, sV = sK + C::KBUF * C::K_BYTES;
+    constexpr int XCH = C::Q_BYTES + C::KBUF * C::K_BYTES + C::V_BYTES;
     float* xch = reinterpret_cast<float*>(base_ptr + XCH);                       // [2][BM]
     const uint32_t bars = sV + C::V_BYTES + 2 * BM * 4;
     const uint32_t qfull = bars, kfull0 = bars + 8, vfull = bars + 24, sbar = bars + 32, obar = bars + 40;
@@ -154,7 +157,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
             if (b < DP / 64) tma_load_3d(sQ + b * (BM * 128), &maps.q, b * 64, h, e.row0 + r0, qfull);
             else tma_load_3d(sQ + b * (BM * 128), &maps.qr, b * 64 - DP, h, e.row0 + r0, qfull);
         load_k(0, 0);
-        if (ntiles > 1) load_k(1, 1);
+        if (C::KBUF > 1 && ntiles > 1) load_k(1, 1);
         load_v(0);
         const bool ok = mbar_wait(qfull, 0, abort_s) && mbar_wait(kfull0, 0, abort_s);
         if (!ok) *abort_s = 1;
@@ -165,7 +168,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     for (int j = 0; j < ntiles; ++j) {
         if (!mbar_wait(sbar, (uint32_t)j & 1u, abort_s)) *abort_s = 1;
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        if (tid == 0 && j + 2 < ntiles && *abort_s == 0) load_k(j + 2, j & 1);      // S_j has read K buffer j % 2
+        if (tid == 0 && j + C::KBUF < ntiles && *abort_s == 0) load_k(j + C::KBUF, j % C::KBUF);      // S_j has read its K buffer
         uint32_t sr[32];
         tc::tmem_ld32(tmem + ((uint32_t)((warp & 3) * 32) << 16) + (uint32_t)(hf * 32), sr);
         const int kb = tile_page(j) * BN, key0 = kb + hf * 32;
@@ -211,8 +214,8 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
                     wt::umma_ts(tmem + C::O_COL, tmem + (uint32_t)(C::P_COL + 8 * k), vdesc + (uint64_t)((k % (BN / 16)) * (2048 >> 4)), kDescO, k != 0 ? 1u : 0u);
                 umma_commit(obar);
                 if (j + 1 < ntiles) {
-                    ok = mbar_wait(kfull0 + 8 * ((j + 1) & 1), (uint32_t)((j + 1) >> 1) & 1u, abort_s);
-                    if (ok) issue_s((j + 1) & 1);
+                    ok = mbar_wait(kfull0 + 8 * ((j + 1) % C::KBUF), (uint32_t)((j + 1) / C::KBUF) & 1u, abort_s);
+                    if (ok) issue_s((j + 1) % C::KBUF);
                 }
             }
             if (!ok) *abort_s = 1;
@@ -234,7 +237,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
         volatile int go_on = 0;
         (void)mbar_wait(qfull, 0, &go_on);
         for (int b = 0; b < 2; ++b)
-            if (last_k[b] >= 0) (void)mbar_wait(kfull0 + 8 * b, (uint32_t)(last_k[b] >> 1) & 1u, &go_on);
+            if (last_k[b] >= 0) (void)mbar_wait(kfull0 + 8 * b, (uint32_t)(last_k[b] / C::KBUF) & 1u, &go_on);
         if (last_v >= 0) (void)mbar_wait(vfull, (uint32_t)last_v & 1u, &go_on);
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");

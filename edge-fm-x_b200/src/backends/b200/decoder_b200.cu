@@ -308,7 +308,7 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
         EFM_TRY(dev_alloc(c, &m->ex.weight, picks));
         EFM_TRY(dev_alloc(c, &m->ex.place, picks));
         EFM_TRY(dev_alloc(c, &m->ex.count, n_experts));
-        EFM_TRY(dev_alloc(c, &m->ex.tile_expert, (size_t)m->ex_rows / kExpertTile));
+        EFM_TRY(dev_alloc(c, &m->ex.tile, (size_t)m->ex_rows / kExpertTile));
         EFM_TRY(dev_alloc(c, &m->ex.n_tiles, 1));
         EFM_TRY(dev_alloc(c, &m->d_h, Wp));
         EFM_TRY(dev_alloc(c, &m->d_route, w_route));

@@ -49,7 +49,10 @@ void launch_gemv_ext(efm_b200_ctx& c, Launcher& L, const GemvParams& p) {
     const int per = kGemvWarps / ks, need = (p.n_items + per - 1) / per;
     const int grid = EPI == Epi::Logits ? c.num_sms : std::min(c.num_sms, need);
     const size_t smem = p.prologue == kProAddNorm || p.prologue == kProNorm ? gemv_ext_smem_bytes(p.K) : gemv_smem_bytes(p.K);
-    L.launch(gemv_kernel<EPI, true>, dim3(grid), dim3(kGemvThreads), smem, p, ks);
+    constexpr bool kExperts = EPI == Epi::Router || EPI == Epi::ExpertUp || EPI == Epi::ExpertDown || EPI == Epi::Store32Bias;
+    if constexpr (kExperts) L.launch(gemv_kernel<EPI, 2>, dim3(grid), dim3(kGemvThreads), smem, p, ks);
+    else if constexpr (EPI == Epi::TokenGate) L.launch(gemv_kernel<EPI, 1>, dim3(grid), dim3(kGemvThreads), smem, p, ks);
+    else L.launch(c.decoder->input_norms() ? gemv_kernel<EPI, 2> : gemv_kernel<EPI, 1>, dim3(grid), dim3(kGemvThreads), smem, p, ks);
 }
 
 template <Epi EPI>
@@ -152,10 +155,10 @@ void launch_attn_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, con
 }
 
 // ---- latent attention, absorbed form: a decode step, or rows of a pass ---------------------------------------------------
-// keys per tile that the block's shared memory takes next to everything else
-int latent_tile(const LatentShape& s, int nh, int splits, int es) {
-    int kt = 64;
-    while (kt > 8 && la::layout(s, nh, splits, es, kt).bytes > 200u * 1024u) kt /= 2;
+// keys per tile, at most `most`, that the block's shared memory takes next to everything else
+int latent_tile(const LatentShape& s, int nh, int splits, int es, int most) {
+    int kt = most;
+    while (kt > 16 && la::layout(s, nh, splits, es, kt).bytes > 200u * 1024u) kt /= 2;
     return kt;
 }
 // blocks that share a row: one per 64 visible keys or 64 latent channels, a power of two
@@ -168,7 +171,7 @@ int latent_splits(const DecoderLayer& l, int pages, int limit) {
 }
 template <typename TC, bool DECODE, typename P>
 void launch_latent_kernel(Launcher& L, const DecoderLayer& l, P& p, int splits, int rows) {
-    p.kt = latent_tile(p.s, l.la_heads, splits, sizeof(TC));
+    p.kt = latent_tile(p.s, l.la_heads, splits, sizeof(TC), l.la_tile);
     const size_t smem = la::layout(p.s, l.la_heads, splits, sizeof(TC), p.kt).bytes;
     const dim3 grid(splits, (l.d.heads + l.la_heads - 1) / l.la_heads, rows), block(la::kThreads);
     L.cluster_x = splits;
@@ -254,7 +257,8 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
             GemvParams p{};
             stream_input(c, p, pend, i == 0, l.pre1);
             p.out_f = m.d_in;
-            gemv_ext<Epi::Store32>(c, L, l.in, p);
+            if (l.in.bias != nullptr) gemv_ext<Epi::Store32Bias>(c, L, l.in, p);
+            else gemv_ext<Epi::Store32>(c, L, l.in, p);
             if (i > 0) tap((int)i - 1);
         }
         if (l.d.mixer == EFM_MIXER_ATTENTION) {
@@ -438,19 +442,19 @@ void launch_delta_scan(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, cons
 }
 
 // The maps of attention and latent attention differ; what is launched is the same.
-template <int DP, int VP, int RP>
+template <int DP, int VP, int RP, bool KEEP>
 void launch_attention_tc_v(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const WindowAttnShape& s, const WindowTcMaps& maps, const RowPlan& plan,
                            const RowTile* list, int n) {
-    L.launch(window_attention_tc_kernel<DP, VP, RP>, dim3(n, s.H), dim3(wt::kThreads), wt::Cfg<DP, VP, RP>::SMEM, maps, static_cast<__nv_bfloat16*>(c.decoder->mix),
+    L.launch(window_attention_tc_kernel<DP, VP, RP, KEEP>, dim3(n, s.H), dim3(wt::kThreads), wt::Cfg<DP, VP, RP>::SMEM, maps, static_cast<__nv_bfloat16*>(c.decoder->mix),
              l.mix_wp, s, plan, list, RP > 0 ? 1 : 0, &c.state->error);
 }
-template <int RP>
+template <int RP, bool KEEP = false>
 void launch_attention_tc_r(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const WindowAttnShape& s, const WindowTcMaps& maps, const RowPlan& plan,
                            const RowTile* list, int n) {
-    if (l.Dp <= 64 && l.Vp <= 64) launch_attention_tc_v<64, 64, RP>(c, L, l, s, maps, plan, list, n);
-    else if (l.Dp <= 64) launch_attention_tc_v<64, 128, RP>(c, L, l, s, maps, plan, list, n);
-    else if (l.Vp <= 64) launch_attention_tc_v<128, 64, RP>(c, L, l, s, maps, plan, list, n);
-    else launch_attention_tc_v<128, 128, RP>(c, L, l, s, maps, plan, list, n);
+    if (l.Dp <= 64 && l.Vp <= 64) launch_attention_tc_v<64, 64, RP, KEEP>(c, L, l, s, maps, plan, list, n);
+    else if (l.Dp <= 64) launch_attention_tc_v<64, 128, RP, KEEP>(c, L, l, s, maps, plan, list, n);
+    else if (l.Vp <= 64) launch_attention_tc_v<128, 64, RP, KEEP>(c, L, l, s, maps, plan, list, n);
+    else launch_attention_tc_v<128, 128, RP, KEEP>(c, L, l, s, maps, plan, list, n);
 }
 // [rows][heads][channels] with strides in elements
 bool head_map(CUtensorMap* map, const void* base, int channels, int heads, int rows, int head_stride, int row_stride, int box_rows) {
@@ -471,7 +475,8 @@ void launch_attention_tc(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, co
     }
     maps.qr = maps.q;
     maps.kr = maps.k;
-    launch_attention_tc_r<0>(c, L, l, s, maps, plan, list, n);
+    if (s.keep > 0) launch_attention_tc_r<0, true>(c, L, l, s, maps, plan, list, n);
+    else launch_attention_tc_r<0>(c, L, l, s, maps, plan, list, n);
 }
 // Long entries of a latent layer: visible cache rows into the workspace, keys and values of all heads by one product,
 // attention over those.
@@ -586,7 +591,7 @@ SumOf<TA> expert_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const
     if constexpr (std::is_same<TA, float>::value) {
         auto product = [&](const DecLinear& w, int n, const float* a, float* out) {
             L.launch(gemm_f32_kernel, dim3((n + 63) / 64, (max_rows + 63) / 64), dim3(256), 0, a, w.Kp, (const __nv_bfloat16*)w.w, w.Kp, out, n, max_rows, n, w.Kp,
-                     (const __nv_bfloat16*)nullptr, RowGroups{m.ex.tile_expert, m.ex.n_tiles, n});
+                     (const __nv_bfloat16*)nullptr, RowGroups{m.ex.tile, m.ex.n_tiles, n});
         };
         product(l.expert_in, 2 * l.ffp, static_cast<const float*>(m.ex_in), m.ex_gu);
         L.launch(silu_mul_rows_kernel, dim3(max_rows / kExpertTile), dim3(256), 0, (const float*)m.ex_gu, static_cast<float*>(m.ex_act), l.ffp,
@@ -595,7 +600,7 @@ SumOf<TA> expert_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const
     } else {
         auto product = [&](const DecLinear& w, int n, GemmEpi epi, const void* a, void* out) {
             GemmParams g{static_cast<const __nv_bfloat16*>(a), w.w, nullptr, static_cast<__nv_bfloat16*>(out), nullptr, max_rows, n, w.Kp};
-            g.group_tile = m.ex.tile_expert;
+            g.group_tile = reinterpret_cast<const GroupTile*>(m.ex.tile);
             g.group_tiles = m.ex.n_tiles;
             g.group_rows = n;
             g.group_all = r.experts * n;
@@ -650,7 +655,10 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
     const void* xin = xa != nullptr ? (const void*)xa : c.resid;
     // the stream takes a sublayer's normed output; xa becomes the next sublayer's input
     auto add_norm = [&](const float* y, const __nv_bfloat16* w, const __nv_bfloat16* pre, const SumOf<TA>& sum = SumOf<TA>{}) {
-        L.launch(add_norm_rows_kernel<TA>, dim3(T), dim3(256), 0, c.resid, y, w, xa, pre, m.W, m.Wp, m.d.norm_eps, sum);
+        const bool experts = sum.place != nullptr;
+        L.launch(pre != nullptr ? (experts ? add_norm_rows_kernel<TA, true, true> : add_norm_rows_kernel<TA, true, false>)
+                                : (experts ? add_norm_rows_kernel<TA, false, true> : add_norm_rows_kernel<TA, false, false>),
+                 dim3(T), dim3(256), 0, c.resid, y, w, xa, pre, m.W, m.Wp, m.d.norm_eps, sum);
     };
     launch_embed_rows(L, ids, c.embed, nullptr, c.resid, T, c.d.vocab, m.Wp, -1, 0, m.d.embed_scale);
     if (xa != nullptr) add_norm(nullptr, nullptr, m.layers[m.runs[0].layer].pre1);
@@ -778,36 +786,38 @@ static cudaError_t fit_side_cluster(DecoderModel& m, int optin) {
 // its heads along with them; every further block of a cluster costs exchange; clusters that are not resident wait.
 template <typename TC, int NH>
 static cudaError_t fit_latent_heads(const DecoderModel& m, DecoderLayer& l, int optin, double& best) {
-    cudaError_t e = smem_attr(latent_attention_kernel<TC, true, NH>, (size_t)optin - 4096);
-    if (e == cudaSuccess) e = smem_attr(latent_attention_kernel<TC, false, NH>, (size_t)optin - 4096);
+    cudaError_t e = smem_attr(latent_attention_kernel<TC, true, NH>, (size_t)optin - 8192);
+    if (e == cudaSuccess) e = smem_attr(latent_attention_kernel<TC, false, NH>, (size_t)optin - 8192);
     if (e != cudaSuccess) return e;
     const bool wide = cudaFuncSetAttribute(latent_attention_kernel<TC, true, NH>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess &&
                       cudaFuncSetAttribute(latent_attention_kernel<TC, false, NH>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess;
     const LatentShape s = latent_shape(m, l);
     const int groups = (l.d.heads + NH - 1) / NH, most = latent_splits(l, m.d.cache_pages, wide ? 16 : 8);
     const int keys = std::min(m.d.cache_pages * kPageTokens, l.d.window > 0 ? l.d.window : 1 << 30);
-    for (int cs = most; cs >= 1; cs >>= 1) {
-        const size_t bytes = la::layout(s, NH, cs, sizeof(TC), latent_tile(s, NH, cs, sizeof(TC))).bytes;
-        if (bytes > (size_t)optin - 4096) continue;
-        cudaLaunchConfig_t cfg = {};
-        cfg.gridDim = dim3(cs, 1, 1);
-        cfg.blockDim = dim3(la::kThreads);
-        cfg.dynamicSmemBytes = bytes;
-        cudaLaunchAttribute at;
-        at.id = cudaLaunchAttributeClusterDimension;
-        at.val.clusterDim.x = (unsigned)cs;
-        at.val.clusterDim.y = at.val.clusterDim.z = 1;
-        cfg.attrs = &at;
-        cfg.numAttrs = 1;
-        int n = 0;
-        if (cudaOccupancyMaxActiveClusters(&n, latent_attention_kernel<TC, true, NH>, &cfg) != cudaSuccess || n < 1) continue;
-        const double cost = ((double)keys / cs * (4 + 2 * NH) + 40.0 * cs + 400.0) * ((groups + n - 1) / n);
-        if (best < 0.0 || cost < best) {
-            best = cost;
-            l.la_heads = NH;
-            l.la_cluster = cs;
+    for (int tile = 64; tile >= 32; tile /= 2)                       // shorter tiles: two blocks may share an SM
+        for (int cs = most; cs >= 1; cs >>= 1) {
+            const size_t bytes = la::layout(s, NH, cs, sizeof(TC), latent_tile(s, NH, cs, sizeof(TC), tile)).bytes;
+            if (bytes > (size_t)optin - 8192) continue;
+            cudaLaunchConfig_t cfg = {};
+            cfg.gridDim = dim3(cs, 1, 1);
+            cfg.blockDim = dim3(la::kThreads);
+            cfg.dynamicSmemBytes = bytes;
+            cudaLaunchAttribute at;
+            at.id = cudaLaunchAttributeClusterDimension;
+            at.val.clusterDim.x = (unsigned)cs;
+            at.val.clusterDim.y = at.val.clusterDim.z = 1;
+            cfg.attrs = &at;
+            cfg.numAttrs = 1;
+            int n = 0;
+            if (cudaOccupancyMaxActiveClusters(&n, latent_attention_kernel<TC, true, NH>, &cfg) != cudaSuccess || n < 1) continue;
+            const double cost = ((double)keys / cs * (4 + 2 * NH) + 40.0 * cs + 400.0 + (tile < 64 ? 20.0 : 0.0)) * ((groups + n - 1) / n);
+            if (best < 0.0 || cost < best) {
+                best = cost;
+                l.la_heads = NH;
+                l.la_cluster = cs;
+                l.la_tile = tile;
+            }
         }
-    }
     (void)cudaGetLastError();
     return best < 0.0 && NH == 4 ? cudaErrorInvalidConfiguration : cudaSuccess;
 }
@@ -825,12 +835,9 @@ cudaError_t configure_decoder(DecoderModel& m) {
     cudaError_t e = cudaGetDevice(&dev);
     if (e == cudaSuccess) e = cudaDeviceGetAttribute(&optin, cudaDevAttrMaxSharedMemoryPerBlockOptin, dev);
     const size_t gv = (size_t)optin - 2048;
-    if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::Store32, true>, gv);
-    if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::TokenGate, true>, gv);
-    if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::Logits, true>, gv);
-    if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::ExpertUp, true>, gv);
-    if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::ExpertDown, true>, gv);
-    if (e == cudaSuccess) e = smem_attr(gemv_kernel<Epi::Router, true>, gv);
+    auto gemv_attr = [&](auto... kernels) { ((e = e == cudaSuccess ? smem_attr(kernels, gv) : e), ...); };
+    gemv_attr(gemv_kernel<Epi::Store32, 1>, gemv_kernel<Epi::TokenGate, 1>, gemv_kernel<Epi::Logits, 1>, gemv_kernel<Epi::Store32, 2>, gemv_kernel<Epi::Logits, 2>,
+              gemv_kernel<Epi::Store32Bias, 2>, gemv_kernel<Epi::Router, 2>, gemv_kernel<Epi::ExpertUp, 2>, gemv_kernel<Epi::ExpertDown, 2>);
     const size_t rows = wa::rows_smem_bytes(256, 256);
     if (e == cudaSuccess) e = smem_attr(window_attention_rows_kernel<float, float, float>, rows);
     if (e == cudaSuccess) e = smem_attr(window_attention_rows_kernel<__nv_bfloat16, __nv_bfloat16, __nv_bfloat16>, rows);
@@ -838,14 +845,15 @@ cudaError_t configure_decoder(DecoderModel& m) {
     if (e == cudaSuccess) e = smem_attr(delta_scan_kernel<6>, ds::smem_bytes(192));
     if (e == cudaSuccess) e = smem_attr(delta_scan_kernel<7>, ds::smem_bytes(224));
     if (e == cudaSuccess) e = smem_attr(delta_scan_kernel<8>, ds::smem_bytes(256));
-    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<64, 64, 0>, wt::Cfg<64, 64, 0>::SMEM);
-    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<64, 64, 64>, wt::Cfg<64, 64, 64>::SMEM);
-    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<64, 128, 0>, wt::Cfg<64, 128, 0>::SMEM);
-    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<64, 128, 64>, wt::Cfg<64, 128, 64>::SMEM);
-    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<128, 64, 0>, wt::Cfg<128, 64, 0>::SMEM);
-    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<128, 64, 64>, wt::Cfg<128, 64, 64>::SMEM);
-    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<128, 128, 0>, wt::Cfg<128, 128, 0>::SMEM);
-    if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<128, 128, 64>, wt::Cfg<128, 128, 64>::SMEM);
+    auto tc_attr = [&](auto dp, auto vp) {
+        constexpr int DP = decltype(dp)::value, VP = decltype(vp)::value;
+        if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<DP, VP, 0, false>, wt::Cfg<DP, VP, 0>::SMEM);
+        if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<DP, VP, 0, true>, wt::Cfg<DP, VP, 0>::SMEM);
+        if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<DP, VP, 64, false>, wt::Cfg<DP, VP, 64>::SMEM);
+    };
+    const std::integral_constant<int, 64> k64{};
+    const std::integral_constant<int, 128> k128{};
+    tc_attr(k64, k64); tc_attr(k64, k128); tc_attr(k128, k64); tc_attr(k128, k128);
     if (e == cudaSuccess) e = smem_attr(delta_prepare_kernel<96>, sizeof(dc::PrepSmem<96>));
     if (e == cudaSuccess) e = smem_attr(delta_prepare_kernel<128>, sizeof(dc::PrepSmem<128>));
     if (e == cudaSuccess) e = smem_attr(delta_chunk_scan_kernel<64>, sizeof(dc::ScanSmem<64>));

@@ -40,7 +40,7 @@ struct DecoderLayer {
     int Qp = 0, Lc = 0, Rc = 0;           // query latent, cached latent, rotated part: padded to 8
     DecLinear uq, ukv;                    // [heads][Dp + Rc] rows; [heads][Dp] key rows, then [heads][Vp] value rows
     __nv_bfloat16* sink = nullptr;
-    int la_heads = 1, la_cluster = 1;     // heads per block and widest cluster of the absorbed form
+    int la_heads = 1, la_cluster = 1, la_tile = 64;       // absorbed form: heads per block, widest cluster, keys per tile
     // routed experts
     DecLinear router, expert_in, expert_out;   // [experts]; [experts][2 * ffp]; [experts][width][ffp]
     int ffp = 0;
@@ -60,6 +60,8 @@ struct DecoderModel {
     bool f32 = false;
     int W = 0, Wp = 0;                    // width, padded to 8
     int side_p = 0;                       // token-side width padded to 8
+    // decode GEMV level 2 (gemv.cuh): input norms, embedding scale
+    bool input_norms() const { return d.norm_layout == EFM_NORM_SANDWICH || d.embed_scale != 1.0f; }
     std::vector<DecoderLayer> layers;
     std::vector<DecoderRun> runs;         // in order
     __nv_bfloat16 *side_embed = nullptr, *final_norm = nullptr;

@@ -27,7 +27,7 @@ __device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
     return make_float4(bf16lo(v.x), bf16hi(v.x), bf16lo(v.y), bf16hi(v.y));
 }
 
-// Where a row's sublayer output comes from: row i of y, or (experts) the weighted sum of the rows place[i][..] of ye.
+// Where a row's sublayer output comes from: row i of y, or (SUM) the weighted sum of the rows place[i][..] of ye.
 template <typename T>
 struct SumOf {
     const T* ye;
@@ -38,9 +38,9 @@ struct SumOf {
     int experts;
 };
 
-// x += y / sqrt(mean(y^2) + eps) * w (w null: x unchanged); out (null: none) = x as T, or with `pre` x / sqrt(mean(x^2) + eps) * pre,
+// x += y / sqrt(mean(y^2) + eps) * w (w null: x unchanged); out (null: none) = x as T, or (PRE) x / sqrt(mean(x^2) + eps) * pre,
 // the next sublayer's input.  One block per row; the first 1024 * KEEP channels stay in registers.
-template <typename T>
+template <typename T, bool PRE, bool SUM>
 __global__ void __launch_bounds__(256) add_norm_rows_kernel(float* __restrict__ x, const float* __restrict__ y, const __nv_bfloat16* __restrict__ w,
                                                             T* __restrict__ out, const __nv_bfloat16* __restrict__ pre, int n, int ld, float eps,
                                                             const SumOf<T> sum) {
@@ -48,10 +48,10 @@ __global__ void __launch_bounds__(256) add_norm_rows_kernel(float* __restrict__ 
     __shared__ float part[2][8];
     const size_t base = (size_t)blockIdx.x * ld;
     const int nv = ld / 4, tid = threadIdx.x;
-    if (sum.count != nullptr && blockIdx.x == 0)
+    if (SUM && blockIdx.x == 0)
         for (int e = tid; e < sum.experts; e += 256) sum.count[e] = 0;
     auto load_y = [&](int c) {
-        if (sum.place == nullptr) return load4(y + base + 4 * c);
+        if constexpr (!SUM) return load4(y + base + 4 * c);
         float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
         for (int k = 0; k < sum.top; ++k) {
             const size_t i = (size_t)blockIdx.x * sum.top + k;
@@ -78,8 +78,8 @@ __global__ void __launch_bounds__(256) add_norm_rows_kernel(float* __restrict__ 
             const float4 g = load4(w + 4 * c);
             r.x += v.x * inv * g.x; r.y += v.y * inv * g.y; r.z += v.z * inv * g.z; r.w += v.w * inv * g.w;
             store4(x + base + 4 * c, r);
-            s2 = square(s2, r);
-            if (out != nullptr && pre == nullptr) store4(out + base + 4 * c, r);
+            if constexpr (PRE) s2 = square(s2, r);
+            if (!PRE && out != nullptr) store4(out + base + 4 * c, r);
             return r;
         };
 #pragma unroll
@@ -91,10 +91,10 @@ __global__ void __launch_bounds__(256) add_norm_rows_kernel(float* __restrict__ 
         for (int i = 0; i < KEEP; ++i)
             if (tid + 256 * i < nv) { keep[i] = load4(x + base + 4 * (tid + 256 * i)); s2 = square(s2, keep[i]); }
         for (int c = tid + 256 * KEEP; c < nv; c += 256) s2 = square(s2, load4(x + base + 4 * c));
-        if (out != nullptr && pre == nullptr)
+        if (!PRE && out != nullptr)
             for (int c = tid; c < nv; c += 256) store4(out + base + 4 * c, load4(x + base + 4 * c));
     }
-    if (out == nullptr || pre == nullptr) return;
+    if constexpr (!PRE) return;
     const float inv = 1.0f / sqrtf(block_sum_256(s2, part[1]) / (float)n + eps);
     auto emit = [&](int c, const float4& v) {
         const float4 g = load4(pre + 4 * c);
@@ -191,7 +191,7 @@ __global__ void __launch_bounds__(256) gather_norm_rows_kernel(const float* __re
 // C[M, N] = A[M, K] . W[N, K]^T in fp32 FMAs (fp32 activations, bf16 weights): the products of the all-32-bit mode and
 // the small ones that feed a recurrence.  64 x 64 tiles, 256 threads, 4 x 4 outputs per thread.  bias may be null.  Grouped
 // (group.tile not null): rows sorted by group as in gemm_tc.cuh, rows [group of the tile * group.rows, + N) of W.
-struct RowGroups { const int32_t *tile, *n_tiles; int rows; };
+struct RowGroups { const int4* tile; const int32_t* n_tiles; int rows; };
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ W, int ldw,
                                                        float* __restrict__ C, int ldc, int M, int N, int K, const __nv_bfloat16* __restrict__ bias,
                                                        const RowGroups group) {
@@ -201,7 +201,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
     if (group.tile != nullptr) {
         const int t = m0 / kExpertTile;
         if (t >= *group.n_tiles) return;
-        W += (size_t)group.tile[t] * group.rows * ldw;
+        W += (size_t)group.tile[t].x * group.rows * ldw;
     }
     float acc[4][4];
 #pragma unroll

@@ -1,5 +1,6 @@
 // Routed experts: limits, the router's shape and where a pass keeps the rows' choices.
 #pragma once
+#include <cuda_runtime.h>
 #include <stdint.h>
 
 namespace efm {
@@ -14,7 +15,7 @@ struct ExpertRows {
     float* weight;                    // [rows][top]
     int32_t* place;                   // [rows][top]: place among the expert's rows, then row of the sorted order
     int32_t* count;                   // [experts], zero between passes
-    int32_t* tile_expert;             // [tiles]
+    int4* tile;                       // [tiles]: expert, its first tile, its number of tiles
     int32_t* n_tiles;                 // tiles in use
 };
 

@@ -27,7 +27,7 @@ __global__ void __launch_bounds__(256) expert_route_rows_kernel(const float* __r
     });
 }
 
-// First row of every expert in the sorted order, by the first warp; block 0 writes the tiles' experts.
+// First row of every expert in the sorted order, by the first warp; block 0 describes the tiles.
 __device__ __forceinline__ void expert_offsets(const int32_t* count, int experts, int32_t* off, const ExpertRows* publish) {
     const int lane = threadIdx.x & 31;
     int base = 0;
@@ -42,7 +42,7 @@ __device__ __forceinline__ void expert_offsets(const int32_t* count, int experts
         const int first = base + x - n;
         if (e < experts) off[e] = first * kExpertTile;
         if (publish != nullptr)
-            for (int t = 0; t < n; ++t) publish->tile_expert[first + t] = e;
+            for (int t = 0; t < n; ++t) publish->tile[first + t] = make_int4(e, first, n, 0);
         base += __shfl_sync(0xffffffffu, x, 31);
     }
     if (publish != nullptr && lane == 0) *publish->n_tiles = base;

@@ -27,6 +27,8 @@ namespace efm {
 
 enum class GemmEpi : int { Bf16Bias = 0, Residual = 1, F32 = 2, Bf16Gelu = 3, SwiGlu = 4, Bf16GeluTanh = 5 };
 
+struct GroupTile { int32_t group, first, count, pad; };      // row tile: its group, the group's first row tile and number of them
+
 struct GemmParams {
     const __nv_bfloat16* A;   // [M, K] (row stride lda)
     const __nv_bfloat16* B;   // [N, K]
@@ -42,8 +44,9 @@ struct GemmParams {
                               // partial of (split z, tile t) goes to the compact slot Cf + (z * tile_count + t -
                               // tile_begin) * 128 * 256, row-major inside the tile ("tail split", see the launcher)
     // GROUPED instantiations (routed experts): rows arrive sorted by group, every group from a multiple of 128 rows on; row tile t
-    // is multiplied with rows [group_tile[t] * group_rows, + N) of B; *group_tiles row tiles are in use
-    const int32_t* group_tile = nullptr;
+    // is multiplied with rows [group_tile[t].group * group_rows, + N) of B; *group_tiles row tiles are in use.  The tiles of a group
+    // are walked together (its row tiles fastest), so that its rows and its part of B are fetched from memory once
+    const GroupTile* group_tile = nullptr;
     const int32_t* group_tiles = nullptr;
     int group_rows = 0, group_all = 0;      // rows of B per group and altogether
 };
@@ -170,6 +173,16 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
     const uint32_t tmem = *tmem_slot;
 
     auto item_coords = [&](int item, int& m0, int& n0, int& kb0, int& kb1, int& z) {
+        if constexpr (GROUPED) {
+            const int4 g = *reinterpret_cast<const int4*>(p.group_tile + item / tiles_n);
+            const int i = item - g.y * tiles_n;
+            m0 = (g.y + i % g.z) * BM;
+            n0 = i / g.z * BN;
+            kb0 = 0;
+            kb1 = KB_all;
+            z = g.x;                                                  // the group, where nothing is split
+            return;
+        }
         z = item / n_tiles;
         const int tile = p.tile_begin + (item - z * n_tiles);
         const int mt = tile % tiles_m, nt = tile / tiles_m;
@@ -186,7 +199,7 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
                 int m0, n0, kb0, kb1, z;
                 item_coords(item, m0, n0, kb0, kb1, z);
                 int b_row = n0;
-                if constexpr (GROUPED) b_row += p.group_tile[m0 / BM] * p.group_rows;
+                if constexpr (GROUPED) b_row += z * p.group_rows;
                 for (int kb = kb0; kb < kb1; ++kb, ++it) {
                     const int s = it % STAGES;
                     const uint32_t ph = (it / STAGES) & 1u;
@@ -247,7 +260,7 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
             const int nc0 = EPI == GemmEpi::SwiGlu ? (n0 >> 1) : n0;           // first output column of the tile
             const bool vec = (ldc & 3) == 0;
             const size_t split_off = compact ? (size_t)item * (size_t)(BM * BN)
-                                             : (p.kb_per_split > 0 ? (size_t)z * (size_t)p.M * (size_t)p.N : 0);
+                                             : (!GROUPED && p.kb_per_split > 0 ? (size_t)z * (size_t)p.M * (size_t)p.N : 0);
 #pragma unroll 1
             for (int c0 = ch * (OUT_COLS / 2); c0 < (ch + 1) * (OUT_COLS / 2); c0 += 32) {
                 if (nc0 + c0 >= ldc) break;                                    // whole chunk outside the matrix

@@ -31,9 +31,10 @@
 
 namespace efm {
 
-enum class Epi : int { Plain = 0, Residual = 1, QkvRope = 2, SwiGlu = 3, Logits = 4, Peers = 5, Store32 = 6, TokenGate = 7, ExpertUp = 8, ExpertDown = 9, Router = 10 };
+enum class Epi : int { Plain = 0, Residual = 1, QkvRope = 2, SwiGlu = 3, Logits = 4, Peers = 5, Store32 = 6, TokenGate = 7, ExpertUp = 8, ExpertDown = 9, Router = 10, Store32Bias = 11 };
 constexpr int kMaxPeers = 8;
-// The last four (and the epilogues from Store32 on) exist in the EXT instantiations only (layered decoders):
+// The last four (and the epilogues from Store32 on) exist in the EXT instantiations only (layered decoders; level 2 adds input
+// norms: Norm, and the second norm and the scale of Embed):
 //   Embed    x = embed_table[token] * embed_scale; with norm2_w the product reads rmsnorm(x) * norm2_w
 //   Norm     x = rmsnorm(xf) * norm_w
 //   AddNorm  x = xr + rmsnorm(addend) * norm_w: a sublayer whose OUTPUT is normalised, folded into the next product;
@@ -183,11 +184,9 @@ __device__ __forceinline__ void item_epilogue(const GemvParams& p, int item, flo
         *reinterpret_cast<float2*>(p.out_f + item * 2) = make_float2(a0, a1);
     } else if constexpr (EPI == Epi::Router) {
         __stcg(reinterpret_cast<float2*>(p.out_f + item * 2), make_float2(a0, a1));
+    } else if constexpr (EPI == Epi::Store32Bias) {
+        *reinterpret_cast<float2*>(p.out_f + item * 2) = make_float2(a0 + __bfloat162float(p.bias[item * 2]), a1 + __bfloat162float(p.bias[item * 2 + 1]));
     } else if constexpr (EPI == Epi::Store32) {
-        if (p.bias != nullptr) {
-            a0 += __bfloat162float(p.bias[item * 2]);
-            a1 += __bfloat162float(p.bias[item * 2 + 1]);
-        }
         *reinterpret_cast<float2*>(p.out_f + item * 2) = make_float2(a0, a1);
     } else if constexpr (EPI == Epi::TokenGate) {
         const int n = item * 2, tok = p.state->token;
@@ -280,11 +279,12 @@ __device__ __forceinline__ void gemv_load_unit(const GemvParams& p, const GemvSc
     item_rows<EPI>(p, sc.ig0 + j * sc.ig_stride, r0, r1, chosen);
     if constexpr (EPI == Epi::ExpertDown) {
         const int per = p.ffp >> 3;                                   // chunks of one expert's row
+        const float inv = 1.0f / (float)per;                           // c / per exactly: half a chunk is far above the rounding
 #pragma unroll
         for (int uu = 0; uu < kGemvU; ++uu) {
             const int c = (part * kGemvU + uu) * sc.stride + sc.gl;
             if (c < sc.nch) {
-                const int k = c / per;
+                const int k = (int)(((float)c + 0.5f) * inv);
                 const __nv_bfloat16* w = p.W + ((size_t)chosen[k] * p.expert_rows + r0) * p.ffp + (size_t)(c - k * per) * 8;
                 buf[uu][0] = ld_stream(w);
                 buf[uu][1] = ld_stream(w + p.ffp);
@@ -309,11 +309,11 @@ __host__ __device__ inline unsigned int gemv_xbytes(int K) { return ((unsigned i
 __host__ __device__ inline unsigned int gemv_wbytes(int K) { return ((unsigned int)K * 2u + 15u) & ~15u; }
 
 // Weights only: the first two units into registers, the norm weight into shared memory.
-template <Epi EPI, bool EXT>
+template <Epi EPI, int EXT>
 __device__ __forceinline__ void gemv_prefetch(const GemvParams& p, const GemvSched& sc, GemvRegs& r, unsigned char* smem,
                                               const unsigned int xbytes) {
     if constexpr (EPI != Epi::ExpertUp && EPI != Epi::ExpertDown) gemv_load_unit<EPI>(p, sc, 0, r.a);
-    if (EXT ? (p.prologue == kProAddNorm || p.prologue == kProNorm) : p.prologue != kProPlain) {
+    if (EXT ? (p.prologue == kProAddNorm || (EXT > 1 && p.prologue == kProNorm)) : p.prologue != kProPlain) {
         uint4* gs = reinterpret_cast<uint4*>(smem + xbytes);        // xbytes = gemv_xbytes(K)
         for (int c = threadIdx.x; c < sc.nch; c += kGemvThreads) gs[c] = ld_cached(p.norm_w + (size_t)c * 8);
     }
@@ -350,6 +350,7 @@ __device__ __forceinline__ void st8f(float* p, const float (&f)[8]) {
 __host__ __device__ inline unsigned int gemv_ext_off(int K) { return gemv_xbytes(K) + gemv_wbytes(K) + (2 * 16 * 2 + 16) * 4u; }
 
 // EXT prologues; false: not one of them.  Ends with a block barrier.
+template <int EXT>
 __device__ __forceinline__ bool gemv_stage_ext(const GemvParams& p, const int nch, unsigned char* smem, const unsigned int xbytes) {
     __shared__ float red3[3 * kGemvWarps];
     float* xs = reinterpret_cast<float*>(smem);
@@ -365,7 +366,7 @@ __device__ __forceinline__ bool gemv_stage_ext(const GemvParams& p, const int nc
 #pragma unroll
             for (int j = 0; j < 8; ++j) x[j] = xs[8 * c + j] * inv2 * w[j];
             st8f(xs + 8 * c, x);
-            if (p.x_out != nullptr && blockIdx.x == 0) st8f(p.x_out + 8 * c, x);
+            if (EXT > 1 && p.x_out != nullptr && blockIdx.x == 0) st8f(p.x_out + 8 * c, x);
         }
     };
     if (p.prologue == kProEmbed) {
@@ -375,16 +376,20 @@ __device__ __forceinline__ bool gemv_stage_ext(const GemvParams& p, const int nc
         for (int c = tid; c < nch; c += kGemvThreads) {
             float f[8];
             unpack8(zero ? make_uint4(0, 0, 0, 0) : ld_cached(row + (size_t)c * 8), f);
+            if constexpr (EXT > 1) {
 #pragma unroll
-            for (int j = 0; j < 8; ++j) {
-                f[j] *= p.embed_scale;
-                sq[0] = fmaf(f[j], f[j], sq[0]);
+                for (int j = 0; j < 8; ++j) {
+                    f[j] *= p.embed_scale;
+                    sq[0] = fmaf(f[j], f[j], sq[0]);
+                }
             }
             st8f(xs + 8 * c, f);
             if (blockIdx.x == 0) st8f(p.resid_out + 8 * c, f);
         }
-        if (p.norm2_w != nullptr) norm2(sq);
-    } else if (p.prologue == kProNorm) {
+        if constexpr (EXT > 1) {
+            if (p.norm2_w != nullptr) norm2(sq);
+        }
+    } else if (EXT > 1 && p.prologue == kProNorm) {
         const uint4* gs = reinterpret_cast<const uint4*>(smem + xbytes);
         for (int c = tid; c < nch; c += kGemvThreads) {
             float f[8];
@@ -566,7 +571,7 @@ __device__ __forceinline__ void gemv_stage(const GemvParams& p, const int nch, u
 }
 
 // Stage activations (with the fused norm), stream the rows, reduce, epilogue.
-template <Epi EPI, bool EXT>
+template <Epi EPI, int EXT>
 __device__ __forceinline__ void gemv_run(const GemvParams& p, const GemvSched& sc, GemvRegs& r, unsigned char* smem,
                                          const unsigned int xbytes, float& best_v, int& best_i, const int* early_chosen = nullptr) {
     const float* xs = reinterpret_cast<const float*>(smem);
@@ -591,14 +596,16 @@ __device__ __forceinline__ void gemv_run(const GemvParams& p, const GemvSched& s
     } else if constexpr (EPI == Epi::ExpertDown) {
         chosen = early_chosen;
         float* xw = reinterpret_cast<float*>(smem);
+        const float* weight = reinterpret_cast<const float*>(early_chosen + kMaxExpertTop);
+        const float inv = 4.0f / (float)p.ffp;
         for (int c = tid; c < 2 * nch; c += kGemvThreads) {            // padded channels are zero
-            const float w = __ldcg(p.route_w + 4 * c / p.ffp);
+            const float w = weight[(int)(((float)c + 0.5f) * inv)];
             const float4 v = __ldcg(reinterpret_cast<const float4*>(p.xf) + c);
             reinterpret_cast<float4*>(xw)[c] = make_float4(v.x * w, v.y * w, v.z * w, v.w * w);
         }
         __syncthreads();
     } else if constexpr (EXT) {
-        if (!gemv_stage_ext(p, nch, smem, xbytes)) gemv_stage(p, nch, smem, xbytes);
+        if (!gemv_stage_ext<EXT>(p, nch, smem, xbytes)) gemv_stage(p, nch, smem, xbytes);
     } else {
         gemv_stage(p, nch, smem, xbytes);
     }
@@ -674,7 +681,7 @@ __device__ __forceinline__ void gemv_publish_best(const GemvParams& p, float bes
 }
 
 // One GEMV phase as its own launch (phase-per-launch decode form, prefill lm_head, operator API).
-template <Epi EPI, bool EXT = false>
+template <Epi EPI, int EXT = 0>
 __global__ void __launch_bounds__(kGemvThreads, 1) gemv_kernel(const GemvParams p, const int ks) {
     extern __shared__ __align__(16) unsigned char gemv_smem[];
     __shared__ float bv[kGemvWarps];
@@ -689,9 +696,12 @@ __global__ void __launch_bounds__(kGemvThreads, 1) gemv_kernel(const GemvParams 
     // which fetches its first weights before its wait.
     if constexpr (EPI != Epi::ExpertUp) pdl_launch_dependents();
     const GemvSched sc = gemv_sched(p, ks, blockIdx.x, gridDim.x);
-    __shared__ int early_s[EPI == Epi::ExpertDown ? kMaxExpertTop : 1];
+    __shared__ int early_s[EPI == Epi::ExpertDown ? 2 * kMaxExpertTop : 1];      // ids | weights
     if constexpr (EPI == Epi::ExpertDown) {
-        if ((int)threadIdx.x < p.route.top) early_s[threadIdx.x] = __ldcg(p.route_id + threadIdx.x);
+        if ((int)threadIdx.x < p.route.top) {
+            early_s[threadIdx.x] = __ldcg(p.route_id + threadIdx.x);
+            early_s[kMaxExpertTop + threadIdx.x] = __float_as_int(__ldcg(p.route_w + threadIdx.x));
+        }
         __syncthreads();
         gemv_load_unit<EPI>(p, sc, 0, regs.a, early_s);
     }

@@ -149,7 +149,7 @@ __global__ void __launch_bounds__(256) latent_gather_rows_kernel(const T* __rest
 
 // ---- one row, absorbed -----------------------------------------------------------------------------------------------
 namespace la {
-constexpr int kThreads = 256;
+constexpr int kThreads = 512, kWarps = kThreads / 32;
 struct Layout {
     int kt, ldk, slice;               // keys per tile, elements between key rows, latent channels per block of the cluster
     unsigned int q, qin, cnew, keys, scr, rout, olat, bytes;
@@ -165,7 +165,7 @@ __host__ __device__ inline Layout layout(const LatentShape& s, int nh, int split
     l.q = take((unsigned int)nh * (s.Lc + s.Rc) * 4u);
     l.qin = take((unsigned int)nh * (s.Dp + s.Rc) * 4u);
     l.cnew = take((unsigned int)(s.Lc + s.Rc) * 4u);
-    const unsigned int kb = 2u * kt * l.ldk * es, rb = (unsigned int)nh * 1024u * 4u;       // keys; afterwards sums of the key groups
+    const unsigned int kb = 2u * kt * l.ldk * es, rb = (unsigned int)nh * 4u * kThreads * 4u;       // keys; afterwards sums of the key groups
     l.keys = take(kb > rb ? kb : rb);
     l.scr = take(kThreads * 8u * 4u);
     l.rout = take((unsigned int)splits * nh * l.slice * 4u);
@@ -202,7 +202,7 @@ __global__ void __launch_bounds__(la::kThreads) latent_attention_kernel(const La
     using namespace la;
     using TI = typename std::conditional<DECODE, float, TC>::type;
     extern __shared__ __align__(16) unsigned char la_smem[];
-    __shared__ float cs[kRotMaxPairs], sn[kRotMaxPairs], part[8], sp[NH][64], sal[NH], sm_m[NH], sm_l[NH], rm[16][NH], rl[16][NH];
+    __shared__ float cs[kRotMaxPairs], sn[kRotMaxPairs], part[kWarps], sp[NH][64], sal[NH], sm_m[NH], sm_l[NH], rm[16][NH], rl[16][NH];
     const LatentShape& s = p.s;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, split = blockIdx.x, n_splits = gridDim.x;
     const int h0 = blockIdx.y * NH, nh = min(NH, s.H - h0), LR = s.Lc + s.Rc;
@@ -257,11 +257,13 @@ __global__ void __launch_bounds__(la::kThreads) latent_attention_kernel(const La
         if (t < n_tiles) {
             const int j0 = begin + t * l.kt;
             TC* dst = keys + (size_t)(t & 1) * l.kt * l.ldk;
-            for (int i = tid; i < l.kt * per; i += kThreads) {
-                const int r = i / per, c = i - r * per, j = j0 + r;
-                if (j < end && !(DECODE && j == pos))
-                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst + (size_t)r * l.ldk) + 16u * c),
-                                 "l"(reinterpret_cast<const char*>(p.pool + pool_row(j) * LR) + 16 * c) : "memory");
+            for (int r = warp; r < l.kt; r += kWarps) {                // a warp per cache row
+                const int j = j0 + r;
+                if (j >= end || (DECODE && j == pos)) continue;
+                const char* src = reinterpret_cast<const char*>(p.pool + pool_row(j) * LR);
+                const uint32_t to = (uint32_t)__cvta_generic_to_shared(dst + (size_t)r * l.ldk);
+                for (int c = lane; c < per; c += 32)
+                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(to + 16u * c), "l"(src + 16 * c) : "memory");
             }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -299,7 +301,7 @@ __global__ void __launch_bounds__(la::kThreads) latent_attention_kernel(const La
         if (append) {
             ss = 0.f;
 #pragma unroll
-            for (int i = 0; i < 8; ++i) ss += part[i];
+            for (int i = 0; i < kWarps; ++i) ss += part[i];
             const float inv = 1.0f / sqrtf(ss / (float)s.L + s.eps);
             const int t = n_tiles - 1;
             TC* mine = keys + (size_t)(t & 1) * l.kt * l.ldk + (size_t)(pos - begin - t * l.kt) * l.ldk;
@@ -441,11 +443,16 @@ __global__ void __launch_bounds__(la::kThreads) latent_attention_kernel(const La
             *reinterpret_cast<float4*>(red + ((size_t)tg * NH + h) * s.Lc + dpart * 4) = make_float4(acc[h][0], acc[h][1], acc[h][2], acc[h][3]);
     }
     __syncthreads();
-    for (int i = tid; i < nh * s.Lc; i += kThreads) {
-        const int h = i / s.Lc, c = i - h * s.Lc, owner = c / l.slice;
-        float v = 0.f;
-        for (int g = 0; g < kg; ++g) v += red[((size_t)g * NH + h) * s.Lc + c];
-        *cl.map_shared_rank(rout + ((size_t)split * NH + h) * l.slice + c - owner * l.slice, owner) = v;
+    for (int c = tid; c < s.Lc; c += kThreads) {
+        const int owner = c / l.slice;
+        float* to = cl.map_shared_rank(rout + (size_t)split * NH * l.slice + c - owner * l.slice, owner);
+#pragma unroll
+        for (int h = 0; h < NH; ++h)
+            if (h < nh) {
+                float v = 0.f;
+                for (int g = 0; g < kg; ++g) v += red[((size_t)g * NH + h) * s.Lc + c];
+                to[h * l.slice] = v;
+            }
     }
     for (int i = tid; i < n_splits * nh; i += kThreads) {
         const int r = i / nh, h = i - r * nh;

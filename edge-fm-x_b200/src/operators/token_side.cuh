@@ -66,7 +66,7 @@ __global__ void __launch_bounds__(kGemvThreads, 1) token_side_kernel(const Token
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
     pdl_wait();
-    gemv_stage_ext(p, p.K >> 3, ts_smem, gemv_xbytes(p.K));
+    gemv_stage_ext<1>(p, p.K >> 3, ts_smem, gemv_xbytes(p.K));
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
     cl.barrier_wait(std::move(started));

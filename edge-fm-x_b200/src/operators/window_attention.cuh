@@ -88,9 +88,11 @@ __device__ __forceinline__ void store_head8(T* p, const float (&f)[8]) {        
 
 // One block per row; `lanes` (8, 16 or 32) threads share a head, 8 channels each.  TI: projections, TQ: q operand, TC: cache.
 template <typename TI, typename TQ, typename TC, bool ROT>
-__global__ void __launch_bounds__(256) qk_scatter_rows_kernel(const TI* __restrict__ qkv, int ld, TQ* __restrict__ q_out, TC* __restrict__ k_pool,
+__global__ void __launch_bounds__(256, 4) qk_scatter_rows_kernel(const TI* __restrict__ qkv, int ld, TQ* __restrict__ q_out, TC* __restrict__ k_pool,
                                                               TC* __restrict__ v_pool, const WindowAttnShape s, const RowPlan plan, int lanes) {
-    __shared__ __align__(16) float cs[kRotMaxPairs], sn[kRotMaxPairs], stage[ROT ? 256 * 8 : 1];
+    __shared__ __align__(16) float cs[kRotMaxPairs];
+    __shared__ __align__(16) float sn[kRotMaxPairs];
+    __shared__ float stage[ROT ? 256 * 8 : 1];
     const int row = blockIdx.x, l = threadIdx.x & (lanes - 1), per = 256 / lanes;
     const RowEntry e = plan.of_row(row);
     const int half = s.rot.dims / 2;
@@ -117,16 +119,26 @@ __global__ void __launch_bounds__(256) qk_scatter_rows_kernel(const TI* __restri
             const float inv = 1.0f / sqrtf(ss / (float)s.D + s.eps);
             const __nv_bfloat16* w = u < s.H ? s.q_norm : s.k_norm;
 #pragma unroll
-            for (int j = 0; j < 8; ++j) f[j] = d + j < s.D ? f[j] * inv * (w != nullptr ? __bfloat162float(w[d + j]) : 1.f) : 0.f;
+            for (int j = 0; j < 8; ++j) f[j] *= inv;                   // channels past D are zero
+            if (w != nullptr) {
+                float g[8];
+                load_head8(w, d, s.D, vec, g);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) f[j] *= g[j];
+            }
         }
         if constexpr (ROT) {
             if (by_lanes) {
-                const bool low = d < half, in = d < s.rot.dims;
+                const bool low = d < half, in = qk && d < s.rot.dims;
                 const int src = in ? (low ? l + half / 8 : l - half / 8) : l, i0 = in ? (low ? d : d - half) : 0;
+                float c[8], n[8];
+                load8_as_f32(cs + i0, c);
+                load8_as_f32(sn + i0, n);
+                const float sign = low ? -1.f : 1.f;
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
                     const float o = __shfl_sync(0xffffffffu, f[j], src, lanes);
-                    if (qk && in) f[j] = low ? f[j] * cs[i0 + j] - o * sn[i0 + j] : f[j] * cs[i0 + j] + o * sn[i0 + j];
+                    if (in) f[j] = fmaf(f[j], c[j], sign * o * n[j]);
                 }
             } else {
                 float* st = stage + (threadIdx.x & ~(lanes - 1)) * 8;  // this head's channels

@@ -54,7 +54,7 @@ struct WindowTcMaps {
     CUtensorMap qr, kr;               // RP > 0: rotated parts, [rows][heads][channels] and [rows][1][channels]
 };
 
-template <int DP, int VP, int RP>
+template <int DP, int VP, int RP, bool KEEP>
 __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(const __grid_constant__ WindowTcMaps maps, __nv_bfloat16* __restrict__ out,
                                                                            int ld_out, const WindowAttnShape s, const RowPlan plan,
                                                                            const RowTile* __restrict__ tiles, int workspace, int* error) {
@@ -95,9 +95,9 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     const int lo = s.window > 0 ? max(0, i_pos - s.window + 1) : 0, hi = i_pos + 1;
     const int first = s.window > 0 ? max(0, p0 - s.window + 1) : 0, lo_max = s.window > 0 ? max(0, p0 + nq - s.window) : 0, hi_min = p0 + 1;
     // tiles: the pages with kept first tokens ahead of the window's first page, then the pages of the window
-    const int pg0 = first / BN, nk = s.window > 0 ? min((min(s.keep, first) + BN - 1) / BN, pg0) : 0;
+    const int pg0 = first / BN, nk = KEEP && s.window > 0 ? min((min(s.keep, first) + BN - 1) / BN, pg0) : 0, keep = KEEP ? s.keep : 0;
     const int ntiles = min(nk + (p0 + nq - 1) / BN - pg0 + 1, kMaxTiles);
-    auto tile_page = [&](int i) { return i < nk ? i : pg0 + i - nk; };
+    auto tile_page = [&](int i) { return KEEP && i < nk ? i : pg0 + i - nk; };
 
     if (tid == 0) {
         mbar_init(qfull, 1); mbar_init(kfull0, 1); mbar_init(kfull0 + 8, 1); mbar_init(vfull, 1); mbar_init(sbar, 1); mbar_init(obar, 1);
@@ -175,11 +175,11 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
         float sc[32];                                            // scores in units of log2
         float mx = -INFINITY;
         const float bias0 = b2 * (float)(key0 - i_pos);
-        const bool interior = (kb >= lo_max || kb + BN <= s.keep) && kb + BN <= hi_min;
+        const bool interior = (kb >= lo_max || (KEEP && kb + BN <= keep)) && kb + BN <= hi_min;
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
             const float v = fmaf(__uint_as_float(sr[i]), f2, fmaf(b2, (float)i, bias0));
-            sc[i] = interior || ((key0 + i >= lo || key0 + i < s.keep) && key0 + i < hi) ? v : -INFINITY;
+            sc[i] = interior || ((key0 + i >= lo || (KEEP && key0 + i < keep)) && key0 + i < hi) ? v : -INFINITY;
             mx = fmaxf(mx, sc[i]);
         }
         xch[hf * BM + row] = mx;

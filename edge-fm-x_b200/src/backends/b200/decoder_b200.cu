@@ -519,6 +519,7 @@ efm_status efm_b200_decoder_step(efm_b200_ctx* c, const efm_step_entry* entries,
         std::vector<int32_t> ids, row_entry;
         std::vector<RowTile> tc, simt, ws;
         std::vector<int32_t> short_rows;
+        int n_ws = 0;
         struct Want { int32_t row; int64_t idx; uint32_t rng_step; };
         std::vector<Want> wants;
         int rows = 0;
@@ -533,8 +534,9 @@ efm_status efm_b200_decoder_step(efm_b200_ctx* c, const efm_step_entry* entries,
                 for (int i = 0; i < n; ++i) short_rows.push_back(rows + i);
             else if (m.ws_pages > 0) {
                 const int p0 = decoder_ws_page0(m, r.pos0), p1 = (r.pos0 + n - 1) / EFM_PAGE_TOKENS;
-                r.ws0 = ((int)ws.size() - p0) * EFM_PAGE_TOKENS;
-                for (int p = p0; p <= p1; ++p) ws.push_back(RowTile{idx, p});
+                r.ws0 = (n_ws - p0) * EFM_PAGE_TOKENS;
+                n_ws += p1 - p0 + 1;
+                for (int p = p0; p * EFM_PAGE_TOKENS < r.pos0; ++p) ws.push_back(RowTile{idx, p});
             }
             for (int i = 0; i < n; ++i) { ids.push_back(en.tokens[done[e] + i]); row_entry.push_back(idx); }
             for (int i = 0; i < en.n_want; ++i)
@@ -546,7 +548,7 @@ efm_status efm_b200_decoder_step(efm_b200_ctx* c, const efm_step_entry* entries,
             if (done[e] == en.n_tokens && e == first) ++first;
         }
         while (first < n_entries && done[first] == entries[first].n_tokens) ++first;
-        if ((int)ws.size() > m.ws_pages) return fail(c, EFM_ERR_STATE, "the entries see more cache pages than the pool has");
+        if (n_ws > m.ws_pages) return fail(c, EFM_ERR_STATE, "the entries see more cache pages than the pool has");
         // tiles of the tensor-core form go to the CUDA-core form in layers it does not take: list them in its units too
         std::vector<RowTile> all_simt;
         for (size_t i = 0; i < re.size(); ++i)
@@ -588,7 +590,8 @@ efm_status efm_b200_decoder_step(efm_b200_ctx* c, const efm_step_entry* entries,
         tiles.short_rows = m.step_buf + o_short;
         tiles.n_short = (int)short_rows.size();
         tiles.ws_pages = reinterpret_cast<const RowTile*>(m.step_buf + o_ws);
-        tiles.n_ws = (int)ws.size();
+        tiles.n_ws = n_ws;
+        tiles.n_gather = (int)ws.size();
         decoder_rows_pass(*c, plan, m.step_buf + o_ids, tiles, L);
         m.tap_row0 += rows;
         for (size_t w0 = 0; w0 < wants.size(); w0 += (size_t)m.max_want) {
@@ -838,6 +841,7 @@ void decoder_prefill_chunk(efm_b200_ctx& c, KvSlot& slot, int S, int kv_offset, 
     if (m.ws_pages > 0) {
         tiles.ws_page0 = decoder_ws_page0(m, kv_offset);
         tiles.n_ws = (kv_offset + S - 1) / EFM_PAGE_TOKENS - tiles.ws_page0 + 1;
+        tiles.n_gather = std::max(0, (kv_offset + EFM_PAGE_TOKENS - 1) / EFM_PAGE_TOKENS - tiles.ws_page0);
         plan.one.ws0 = -tiles.ws_page0 * EFM_PAGE_TOKENS;
     }
     plan.page_table = m.page_table;

@@ -485,8 +485,9 @@ void launch_latent_tc(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const
     DecoderModel& m = *c.decoder;
     const LatentShape z = latent_shape(m, l);
     const int LR = z.Lc + z.Rc, n_ws = tiles.n_ws * kPageTokens, ld = l.ukv.Np;
-    L.launch(latent_gather_rows_kernel<__nv_bfloat16>, dim3(tiles.n_ws, 4), dim3(256), 0, static_cast<const __nv_bfloat16*>(run.k_pool), m.ws_c, LR, plan,
-             tiles.ws_pages, tiles.ws_page0);
+    if (tiles.n_gather > 0)
+        L.launch(latent_gather_rows_kernel<__nv_bfloat16>, dim3(tiles.n_gather, 4), dim3(256), 0, static_cast<const __nv_bfloat16*>(run.k_pool), m.ws_c, LR, plan,
+                 tiles.ws_pages, tiles.ws_page0);
     GemmParams g{m.ws_c, l.ukv.w, nullptr, m.ws_kv, nullptr, n_ws, l.ukv.Np, l.ukv.Kp};
     g.lda = LR;
     launch_gemm_epi(L, GemmEpi::Bf16Bias, g, &c.state->error);
@@ -557,7 +558,12 @@ void latent_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const Deco
     const LatentShape s = latent_shape(m, l);
     const int T = plan.rows;
     linear_act(c, L, l.in, x, m.proj_a, T);
-    L.launch(latent_rows_kernel<TA>, dim3(T), dim3(256), 0, static_cast<const TA*>(m.proj_a), l.in.Np, static_cast<TA*>(m.cq), static_cast<TA*>(run.k_pool), s, plan);
+    TA* ws = nullptr;
+    if constexpr (std::is_same<TA, __nv_bfloat16>::value) {
+        if (decoder_layer_tc(m, l)) ws = m.ws_c;
+    }
+    L.launch(latent_rows_kernel<TA>, dim3((T + kLatentRowsPerBlock - 1) / kLatentRowsPerBlock), dim3(32 * kLatentRowsPerBlock), 0, static_cast<const TA*>(m.proj_a),
+             l.in.Np, static_cast<TA*>(m.cq), static_cast<TA*>(run.k_pool), ws, kTcMinRows, s, plan);
     linear_act(c, L, l.uq, m.cq, m.q, T);
     L.launch(latent_rotate_rows_kernel<TA>, dim3(T), dim3(256), 0, static_cast<TA*>(m.q), s, plan);
     if constexpr (std::is_same<TA, __nv_bfloat16>::value) {
@@ -794,7 +800,7 @@ static cudaError_t fit_latent_heads(const DecoderModel& m, DecoderLayer& l, int 
     const LatentShape s = latent_shape(m, l);
     const int groups = (l.d.heads + NH - 1) / NH, most = latent_splits(l, m.d.cache_pages, wide ? 16 : 8);
     const int keys = std::min(m.d.cache_pages * kPageTokens, l.d.window > 0 ? l.d.window : 1 << 30);
-    for (int tile = 64; tile >= 32; tile /= 2)                       // shorter tiles: two blocks may share an SM
+    for (int tile = la::kMaxTile; tile >= 32; tile /= 2)             // shorter tiles: two blocks may share an SM
         for (int cs = most; cs >= 1; cs >>= 1) {
             const size_t bytes = la::layout(s, NH, cs, sizeof(TC), latent_tile(s, NH, cs, sizeof(TC), tile)).bytes;
             if (bytes > (size_t)optin - 8192) continue;
@@ -810,7 +816,7 @@ static cudaError_t fit_latent_heads(const DecoderModel& m, DecoderLayer& l, int 
             cfg.numAttrs = 1;
             int n = 0;
             if (cudaOccupancyMaxActiveClusters(&n, latent_attention_kernel<TC, true, NH>, &cfg) != cudaSuccess || n < 1) continue;
-            const double cost = ((double)keys / cs * (4 + 2 * NH) + 40.0 * cs + 400.0 + (tile < 64 ? 20.0 : 0.0)) * ((groups + n - 1) / n);
+            const double cost = ((double)keys / cs * (4 + 2 * NH) + 40.0 * cs + 400.0 + 100.0 * ((keys + cs * tile - 1) / (cs * tile))) * ((groups + n - 1) / n);
             if (best < 0.0 || cost < best) {
                 best = cost;
                 l.la_heads = NH;

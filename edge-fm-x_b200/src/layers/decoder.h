@@ -105,10 +105,11 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
 struct RowTiles {
     const RowTile *tc = nullptr, *simt = nullptr, *all = nullptr;
     int n_tc = 0, n_simt = 0, n_all = 0;
-    // latent attention: rows of the short entries (absorbed form) and the cache pages the long entries see
+    // latent attention: rows of the short entries (absorbed form); workspace pages of the long entries and those of them that
+    // hold earlier tokens (listed, or from ws_page0 on)
     const int32_t* short_rows = nullptr;
     const RowTile* ws_pages = nullptr;
-    int n_short = 0, n_ws = 0, ws_page0 = 0;
+    int n_short = 0, n_ws = 0, n_gather = 0, ws_page0 = 0;
     bool listed = false;
 };
 void decoder_rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const RowTiles& tiles, Launcher& L);

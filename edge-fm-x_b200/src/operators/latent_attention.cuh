@@ -6,8 +6,9 @@
 //
 //   latent_rows          many rows: norms of the two latents, rotation of r, cache append
 //   latent_rotate_rows   many rows: rotation of the queries' rotated part, in place
-//   latent_gather_rows   long entries: the visible cache rows of every entry into a contiguous workspace; one product expands
-//                        them to keys and values of all heads, and the tensor-core attention (window_attention_tc.cuh) reads those
+//   latent_gather_rows   long entries: the earlier cache rows an entry sees into a contiguous workspace, where latent_rows has put
+//                        its new ones; one product expands all of them to keys and values of all heads, and the tensor-core
+//                        attention (window_attention_tc.cuh) reads those
 //   latent_attention     one row per cluster, absorbed form: the query is moved into the latent space (qa = Wk[h]^T q), scores and
 //                        sums run over the cached rows as they are, the result goes through Wv[h] and the gate: decode steps,
 //                        short portions and the 32-bit mode.  Nothing per-head is ever stored for a key.
@@ -42,49 +43,50 @@ struct LatentShape {
 };
 
 // ---- many rows -----------------------------------------------------------------------------------------------------
-// One block per row, 8 channels per thread and turn (every part is a multiple of 8); the first 8 * 256 channels stay in registers.
+// One warp per row, 8 channels per lane and turn (every part is a multiple of 8); the first 32 * 8 * KEEP channels stay in
+// registers.  ws (may be null): rows of the long entries go to the workspace too.
+constexpr int kLatentRowsPerBlock = 4;
 template <typename T>
-__global__ void __launch_bounds__(256) latent_rows_kernel(const T* __restrict__ proj, int ld, T* __restrict__ cq, T* __restrict__ pool, const LatentShape s,
-                                                          const RowPlan plan) {
-    __shared__ float part[2][8], cs[kRotMaxPairs], sn[kRotMaxPairs];
-    __shared__ __align__(16) float rot[256];
-    const int row = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const RowEntry e = plan.of_row(row);
-    const int pos = e.pos0 + row - e.row0, nq = s.Qp / 8, nc = s.Lc / 8, n = nq + nc + s.Rc / 8;
+__global__ void __launch_bounds__(32 * kLatentRowsPerBlock) latent_rows_kernel(const T* __restrict__ proj, int ld, T* __restrict__ cq, T* __restrict__ pool,
+                                                                                T* __restrict__ ws, int ws_min_rows, const LatentShape s, const RowPlan plan) {
+    constexpr int KEEP = 6;
+    __shared__ float cs_s[kLatentRowsPerBlock][kRotMaxPairs], sn_s[kLatentRowsPerBlock][kRotMaxPairs], rot_s[kLatentRowsPerBlock][2 * kRotMaxPairs];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, row = blockIdx.x * kLatentRowsPerBlock + warp;
+    if (row >= plan.rows) return;                                       // no block barriers below
+    float *cs = cs_s[warp], *sn = sn_s[warp], *rot = rot_s[warp];
+    const int nq = s.Qp / 8, nc = s.Lc / 8, n = nq + nc + s.Rc / 8;
     const T* src = proj + (size_t)row * ld;
-    float keep[8], a = 0.f, b = 0.f;                                    // pads are zero
-    for (int c = tid; c < n; c += 256) {
-        float f[8];
-        load8_as_f32(src + 8 * c, f);
+    float keep[KEEP][8];
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+        if (lane + 32 * i < n) load8_as_f32(src + 8 * (lane + 32 * i), keep[i]);
+    const RowEntry e = plan.of_row(row);
+    const int pos = e.pos0 + row - e.row0;
+    for (int i = lane; i < s.rot.dims / 2; i += 32) sincosf((float)pos * s.rot.inv_freq[i], sn + i, cs + i);
+    float a = 0.f, b = 0.f;                                             // pads are zero
+    auto take = [&](int c, const float (&f)[8]) {
         float ss = 0.f;
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            ss = fmaf(f[j], f[j], ss);
-            if (c == tid) keep[j] = f[j];
-        }
+        for (int j = 0; j < 8; ++j) ss = fmaf(f[j], f[j], ss);
         if (c < nq) a += ss;
         else if (c < nq + nc) b += ss;
         else
 #pragma unroll
             for (int j = 0; j < 8; ++j) rot[8 * (c - nq - nc) + j] = f[j];
-    }
-    rot_table(s.rot, pos, cs, sn);
+    };
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+        if (lane + 32 * i < n) take(lane + 32 * i, keep[i]);
+    for (int c = lane + 32 * KEEP; c < n; c += 32) { float f[8]; load8_as_f32(src + 8 * c, f); take(c, f); }
     a = warp_sum(a);
     b = warp_sum(b);
-    if (lane == 0) { part[0][warp] = a; part[1][warp] = b; }
-    __syncthreads();
-    a = b = 0.f;
-#pragma unroll
-    for (int i = 0; i < 8; ++i) { a += part[0][i]; b += part[1][i]; }
+    __syncwarp();
     const float ia = 1.0f / sqrtf(a / (float)s.q_rank + s.eps), ib = 1.0f / sqrtf(b / (float)s.L + s.eps);
     T* dst = pool + plan.cache_row(e, pos) * (s.Lc + s.Rc);
-    for (int c = tid; c < n; c += 256) {
-        float f[8], w[8];
-        if (c == tid)
-#pragma unroll
-            for (int j = 0; j < 8; ++j) f[j] = keep[j];
-        else load8_as_f32(src + 8 * c, f);
+    T* dst2 = ws != nullptr && e.n >= ws_min_rows ? ws + (size_t)(e.ws0 + pos) * (s.Lc + s.Rc) : nullptr;
+    auto emit = [&](int c, float (&f)[8]) {
         if (c < nq + nc) {
+            float w[8];
             unpack8(ld_cached(c < nq ? s.q_norm + 8 * c : s.kv_norm + 8 * (c - nq)), w);
             const float inv = c < nq ? ia : ib;
 #pragma unroll
@@ -94,7 +96,12 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const T* __restrict__ 
             for (int j = 0; j < 8; ++j) f[j] = rot_channel(s.rot, rot, 8 * (c - nq - nc) + j, cs, sn);
         }
         store_head8(c < nq ? cq + (size_t)row * s.Qp + 8 * c : dst + 8 * (c - nq), f);
-    }
+        if (c >= nq && dst2 != nullptr) store_head8(dst2 + 8 * (c - nq), f);
+    };
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+        if (lane + 32 * i < n) emit(lane + 32 * i, keep[i]);
+    for (int c = lane + 32 * KEEP; c < n; c += 32) { float f[8]; load8_as_f32(src + 8 * c, f); emit(c, f); }
 }
 
 template <typename T>
@@ -142,16 +149,15 @@ __global__ void __launch_bounds__(256) latent_gather_rows_kernel(const T* __rest
     const RowEntry e = plan.entry(t.entry);
     const uint4* src = reinterpret_cast<const uint4*>(pool + plan.cache_row(e, t.row * kPageTokens) * row_elems);
     uint4* dst = reinterpret_cast<uint4*>(ws + (size_t)(e.ws0 + t.row * kPageTokens) * row_elems);
-    // rows past the entry's last token hold what an earlier owner of the page left: zeros instead, never visible
-    const int n = min(kPageTokens, e.pos0 + e.n - t.row * kPageTokens), per = row_elems * (int)sizeof(T) / 16;
-    for (int i = blockIdx.y * 256 + threadIdx.x; i < kPageTokens * per; i += 256 * gridDim.y) dst[i] = i < n * per ? src[i] : make_uint4(0, 0, 0, 0);
+    const int n = min(kPageTokens, e.pos0 - t.row * kPageTokens) * (row_elems * (int)sizeof(T) / 16);      // rows from pos0 on are new
+    for (int i = blockIdx.y * 256 + threadIdx.x; i < n; i += 256 * gridDim.y) dst[i] = src[i];
 }
 
 // ---- one row, absorbed -----------------------------------------------------------------------------------------------
 namespace la {
-constexpr int kThreads = 512, kWarps = kThreads / 32;
+constexpr int kThreads = 512, kWarps = kThreads / 32, kMaxTile = 128;
 struct Layout {
-    int kt, ldk, slice;               // keys per tile, elements between key rows, latent channels per block of the cluster
+    int kt, ldk, slice;               // keys per tile (at most kMaxTile), elements between key rows, latent channels per block of the cluster
     unsigned int q, qin, cnew, keys, scr, rout, olat, bytes;
 };
 // Shared memory of one block: heads per block, cluster width, bytes per cache element.
@@ -165,7 +171,7 @@ __host__ __device__ inline Layout layout(const LatentShape& s, int nh, int split
     l.q = take((unsigned int)nh * (s.Lc + s.Rc) * 4u);
     l.qin = take((unsigned int)nh * (s.Dp + s.Rc) * 4u);
     l.cnew = take((unsigned int)(s.Lc + s.Rc) * 4u);
-    const unsigned int kb = 2u * kt * l.ldk * es, rb = (unsigned int)nh * 4u * kThreads * 4u;       // keys; afterwards sums of the key groups
+    const unsigned int kb = (unsigned int)kt * l.ldk * es, rb = (unsigned int)nh * 4u * kThreads * 4u;       // keys; afterwards sums of the key groups
     l.keys = take(kb > rb ? kb : rb);
     l.scr = take(kThreads * 8u * 4u);
     l.rout = take((unsigned int)splits * nh * l.slice * 4u);
@@ -202,7 +208,7 @@ __global__ void __launch_bounds__(la::kThreads) latent_attention_kernel(const La
     using namespace la;
     using TI = typename std::conditional<DECODE, float, TC>::type;
     extern __shared__ __align__(16) unsigned char la_smem[];
-    __shared__ float cs[kRotMaxPairs], sn[kRotMaxPairs], part[kWarps], sp[NH][64], sal[NH], sm_m[NH], sm_l[NH], rm[16][NH], rl[16][NH];
+    __shared__ float cs[kRotMaxPairs], sn[kRotMaxPairs], part[kWarps], sp[NH][kMaxTile], sal[NH], sm_m[NH], sm_l[NH], rm[16][NH], rl[16][NH];
     const LatentShape& s = p.s;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, split = blockIdx.x, n_splits = gridDim.x;
     const int h0 = blockIdx.y * NH, nh = min(NH, s.H - h0), LR = s.Lc + s.Rc;
@@ -256,7 +262,7 @@ __global__ void __launch_bounds__(la::kThreads) latent_attention_kernel(const La
     auto load_tile = [&](int t) {
         if (t < n_tiles) {
             const int j0 = begin + t * l.kt;
-            TC* dst = keys + (size_t)(t & 1) * l.kt * l.ldk;
+            TC* dst = keys;
             for (int r = warp; r < l.kt; r += kWarps) {                // a warp per cache row
                 const int j = j0 + r;
                 if (j >= end || (DECODE && j == pos)) continue;
@@ -268,8 +274,7 @@ __global__ void __launch_bounds__(la::kThreads) latent_attention_kernel(const La
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    load_tile(0);
-    load_tile(1);
+    load_tile(0);                                                      // a window's share is one tile as a rule
     if (ok) rot_table(s.rot, pos, cs, sn);
     if constexpr (DECODE) {
         if (p.early) { pdl_wait(); pdl_launch_dependents(); }
@@ -303,13 +308,9 @@ __global__ void __launch_bounds__(la::kThreads) latent_attention_kernel(const La
 #pragma unroll
             for (int i = 0; i < kWarps; ++i) ss += part[i];
             const float inv = 1.0f / sqrtf(ss / (float)s.L + s.eps);
-            const int t = n_tiles - 1;
-            TC* mine = keys + (size_t)(t & 1) * l.kt * l.ldk + (size_t)(pos - begin - t * l.kt) * l.ldk;
-            // from the third tile on the row is written when the tile's turn comes: another tile still uses the buffer
             TC* dst = p.pool + pool_row(pos) * LR;
             for (int c = tid; c < LR; c += kThreads) {
                 const float v = c < s.Lc ? cnew[c] * inv * __bfloat162float(s.kv_norm[c]) : rot_channel(s.rot, cnew + s.Lc, c - s.Lc, cs, sn);
-                if (t < 2) store_f32(mine + c, v);
                 if (blockIdx.y == 0) store_f32(dst + c, v);
                 scr[c] = v;                                            // at most kThreads * 8 channels
             }
@@ -345,14 +346,19 @@ __global__ void __launch_bounds__(la::kThreads) latent_attention_kernel(const La
 #pragma unroll
             for (int j = 0; j < 8; ++j) scr[tid * 8 + j] = acc[j];
             __syncthreads();
-            for (int i = tid; i < min(wide, cols - c0) * 8; i += kThreads) {
+            const int n = min(wide, cols - c0) * 8;                    // sums over d0: eight lanes each
+            for (int i0 = 0; i0 < n; i0 += kThreads / 8) {
+                const int i = i0 + tid / 8, x = tid & 7;
                 float v = 0.f;
-                for (int d = 0; d < dl; ++d) v += scr[(d * wide) * 8 + i];
-                const int cc = c0 + i / 8, h = cc / sl8, ch = s0 + (cc - h * sl8) * 8 + (i & 7);
-                v *= s.scale;
-                if (n_splits == 1) q[h * LR + ch] = v;
-                else
-                    for (int r = 0; r < n_splits; ++r) *cl.map_shared_rank(q + h * LR + ch, r) = v;
+                if (i < n)
+                    for (int d = x; d < dl; d += 8) v += scr[d * wide * 8 + i];
+#pragma unroll
+                for (int o = 4; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+                if (i < n) {
+                    const int cc = c0 + i / 8, h = cc / sl8, ch = s0 + (cc - h * sl8) * 8 + (i & 7);
+                    v *= s.scale;
+                    for (int r = x; r < n_splits; r += 8) *cl.map_shared_rank(q + h * LR + ch, r) = v;
+                }
             }
         }
     }
@@ -368,10 +374,10 @@ __global__ void __launch_bounds__(la::kThreads) latent_attention_kernel(const La
 #pragma unroll
         for (int j = 0; j < 4; ++j) acc[h][j] = 0.f;
     for (int t = 0; t < n_tiles; ++t) {
-        asm volatile("cp.async.wait_group 1;" ::: "memory");
-        TC* kt = keys + (size_t)(t & 1) * l.kt * l.ldk;
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        TC* kt = keys;
         const int j0 = begin + t * l.kt;
-        if (append && t >= 2 && t == n_tiles - 1)
+        if (append && t == n_tiles - 1)
             for (int c = tid; c < LR; c += kThreads) store_f32(kt + (size_t)(pos - j0) * l.ldk + c, cnew[c]);
         __syncthreads();
         const bool vis = j0 + key < end;
@@ -398,12 +404,20 @@ __global__ void __launch_bounds__(la::kThreads) latent_attention_kernel(const La
         }
         __syncthreads();
         if (warp < nh) {
-            const float x0 = lane < l.kt ? sp[warp][lane] : -INFINITY, x1 = lane + 32 < l.kt ? sp[warp][lane + 32] : -INFINITY;
-            const float mo = sm_m[warp], mn = fmaxf(mo, warp_max(fmaxf(x0, x1)));       // the tile holds a visible key
-            const float p0 = expf(x0 - mn), p1 = expf(x1 - mn);
-            sp[warp][lane] = p0;
-            sp[warp][lane + 32] = p1;
-            const float sum = warp_sum(p0 + p1);
+            float x[kMaxTile / 32], mx = -INFINITY, sum = 0.f;
+#pragma unroll
+            for (int i = 0; i < kMaxTile / 32; ++i) {
+                x[i] = lane + 32 * i < l.kt ? sp[warp][lane + 32 * i] : -INFINITY;
+                mx = fmaxf(mx, x[i]);
+            }
+            const float mo = sm_m[warp], mn = fmaxf(mo, warp_max(mx));          // the tile holds a visible key
+#pragma unroll
+            for (int i = 0; i < kMaxTile / 32; ++i) {
+                x[i] = expf(x[i] - mn);
+                if (lane + 32 * i < l.kt) sp[warp][lane + 32 * i] = x[i];
+                sum += x[i];
+            }
+            sum = warp_sum(sum);
             if (lane == 0) {
                 const float al = expf(mo - mn);
                 sal[warp] = al;
@@ -432,10 +446,8 @@ __global__ void __launch_bounds__(la::kThreads) latent_attention_kernel(const La
             }
         }
         __syncthreads();
-        load_tile(t + 2);
+        if (t + 1 < n_tiles) load_tile(t + 1);
     }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();
     // ---- sums over the key groups, then over the cluster: every latent channel belongs to one block ------------------------
     if (pv) {
 #pragma unroll

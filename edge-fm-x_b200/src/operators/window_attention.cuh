@@ -31,7 +31,7 @@ struct WindowAttnShape {
     const __nv_bfloat16* k_norm;      // [D]
     const __nv_bfloat16* temp;        // [H], null: 1
     RotShape rot;
-    // tensor-core form only: extra term exp(sink[h]) of the softmax denominator, and heads multiplied by sigmoid(gate)
+    // tensor-core form with a shared key part only: extra term exp(sink[h]) of the softmax denominator, and heads multiplied by sigmoid(gate)
     const __nv_bfloat16* sink;        // [H], null: none
     const __nv_bfloat16* gate;        // [T][H * Dv] with row stride gate_ld, null: none
     int gate_ld;
@@ -111,18 +111,17 @@ __global__ void __launch_bounds__(256, 4) qk_scatter_rows_kernel(const TI* __res
         float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
         if (qk) load_head8(src + (size_t)u * s.D, d, s.D, vec, f);     // q heads, then k heads
         else if (u < units) load_head8(src + (size_t)(s.H + s.G) * s.D + (size_t)(u - s.H - s.G) * s.Dv, d, s.Dv, vecv, f);
-        float ss = 0.f;
+        const __nv_bfloat16* w = u < s.H ? s.q_norm : s.k_norm;
+        float ss = 0.f, g[8];
+        if (qk && w != nullptr) load_head8(w, d, s.D, vec, g);
 #pragma unroll
         for (int j = 0; j < 8; ++j) ss = fmaf(f[j], f[j], ss);
         for (int x = lanes / 2; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
         if (qk) {
             const float inv = 1.0f / sqrtf(ss / (float)s.D + s.eps);
-            const __nv_bfloat16* w = u < s.H ? s.q_norm : s.k_norm;
 #pragma unroll
             for (int j = 0; j < 8; ++j) f[j] *= inv;                   // channels past D are zero
             if (w != nullptr) {
-                float g[8];
-                load_head8(w, d, s.D, vec, g);
 #pragma unroll
                 for (int j = 0; j < 8; ++j) f[j] *= g[j];
             }

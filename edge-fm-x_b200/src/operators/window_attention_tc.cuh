@@ -245,7 +245,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     xch[hf * BM + row] = l;
     __syncthreads();
     float L = xch[row] + xch[BM + row], up = 1.0f;
-    if (s.sink != nullptr) {                                     // one more term of the denominator
+    if (RP > 0 && s.sink != nullptr) {                           // one more term of the denominator
         const float sk = __bfloat162float(s.sink[h]) * kLog2e, mx = fmaxf(m, sk);
         up = at::ex2(m - mx);
         L = fmaf(L, up, at::ex2(sk - mx));
@@ -254,7 +254,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     if (valid && *abort_s == 0) {
         __nv_bfloat16* dst = out + (size_t)(e.row0 + r0 + row) * ld_out + (size_t)h * s.Dv;
         const bool vec = (s.Dv & 7) == 0;                        // ld_out is a multiple of 8
-        if (s.gate != nullptr) {
+        if (RP > 0 && s.gate != nullptr) {
             const __nv_bfloat16* gt = s.gate + (size_t)(e.row0 + r0 + row) * s.gate_ld + (size_t)h * s.Dv;
 #pragma unroll
             for (int i = 0; i < C::HALF; i += 8) {

@@ -280,16 +280,18 @@ __device__ __forceinline__ void gemv_load_unit(const GemvParams& p, const GemvSc
     if constexpr (EPI == Epi::ExpertDown) {
         const int per = p.ffp >> 3;                                   // chunks of one expert's row
         const float inv = 1.0f / (float)per;                           // c / per exactly: half a chunk is far above the rounding
+        const __nv_bfloat16* w[kGemvU];                                // all addresses first: the loads then leave back to back
 #pragma unroll
         for (int uu = 0; uu < kGemvU; ++uu) {
-            const int c = (part * kGemvU + uu) * sc.stride + sc.gl;
-            if (c < sc.nch) {
-                const int k = (int)(((float)c + 0.5f) * inv);
-                const __nv_bfloat16* w = p.W + ((size_t)chosen[k] * p.expert_rows + r0) * p.ffp + (size_t)(c - k * per) * 8;
-                buf[uu][0] = ld_stream(w);
-                buf[uu][1] = ld_stream(w + p.ffp);
-            }
+            const int c = min((part * kGemvU + uu) * sc.stride + sc.gl, sc.nch - 1), k = (int)(((float)c + 0.5f) * inv);
+            w[uu] = p.W + ((size_t)chosen[k] * p.expert_rows + r0) * p.ffp + (size_t)(c - k * per) * 8;
         }
+#pragma unroll
+        for (int uu = 0; uu < kGemvU; ++uu)
+            if ((part * kGemvU + uu) * sc.stride + sc.gl < sc.nch) {
+                buf[uu][0] = ld_stream(w[uu]);
+                buf[uu][1] = ld_stream(w[uu] + p.ffp);
+            }
         return;
     }
     const __nv_bfloat16* a = p.W + (size_t)r0 * p.K;

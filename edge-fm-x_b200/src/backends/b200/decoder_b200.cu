@@ -28,8 +28,11 @@ efm_status validate(const efm_decoder_desc& d, const efm_decoder_layer* layers) 
         d.max_slots <= 0 || d.cache_pages < 0 || d.state_slots < 0)
         return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, "non-positive decoder dimension");
     if (d.compute_dtype != EFM_BF16 && d.compute_dtype != EFM_F32) return fail(nullptr, EFM_ERR_UNSUPPORTED, "compute_dtype must be bf16 or fp32");
-    if (d.norm_layout != EFM_NORM_OUTPUT && d.norm_layout != EFM_NORM_SANDWICH) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, "unknown norm_layout");
-    if (d.norm_layout == EFM_NORM_SANDWICH && d.side_dim > 0) return fail(nullptr, EFM_ERR_UNSUPPORTED, "a token input behind normalised sublayer inputs");
+    if (d.norm_layout < EFM_NORM_OUTPUT || d.norm_layout > EFM_NORM_INPUT) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, "unknown norm_layout");
+    if (d.logit_softcap < 0.f) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, "logit_softcap must not be negative");
+    if (d.norm_layout != EFM_NORM_INPUT && (d.logit_scale != 1.0f || d.logit_softcap > 0.f))
+        return fail(nullptr, EFM_ERR_UNSUPPORTED, "scaled or capped logits behind output norms");
+    if (d.norm_layout != EFM_NORM_OUTPUT && d.side_dim > 0) return fail(nullptr, EFM_ERR_UNSUPPORTED, "a token input behind normalised sublayer inputs");
     if (d.loop_times < 0 || (d.loop_times > 1 && (d.loop_start < 0 || d.loop_stop <= d.loop_start || d.loop_stop > d.num_layers)))
         return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, "the looped layers must be a span of the layers");
     for (int i = 0; i < d.num_layers; ++i) {
@@ -37,18 +40,29 @@ efm_status validate(const efm_decoder_desc& d, const efm_decoder_layer* layers) 
         const std::string at = "layer " + std::to_string(i) + ": ";
         if (l.heads <= 0 || l.dim <= 0 || l.ff < 0 || l.experts < 0) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "non-positive dimension");
         if (l.dim > 256) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "dim above 256");
-        if (l.mixer == EFM_MIXER_ATTENTION) {
+        const bool input = d.norm_layout == EFM_NORM_INPUT;
+        if (l.mixer == EFM_MIXER_ATTENTION || l.mixer == EFM_MIXER_PARALLEL) {
             if (l.kv_heads <= 0 || l.heads % l.kv_heads != 0 || l.vdim <= 0 || l.window < 0)
                 return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "heads must be a multiple of kv_heads, vdim positive, window >= 0");
             if (l.vdim > 256) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "vdim above 256");
-            if (l.keep_first < 0 || (l.qk_norm != EFM_QK_NORM_WEIGHTED && l.qk_norm != EFM_QK_NORM_PLAIN)) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "keep_first or qk_norm");
+            if (l.keep_first < 0 || l.qk_norm < EFM_QK_NORM_WEIGHTED || l.qk_norm > EFM_QK_NORM_NONE) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "keep_first or qk_norm");
             if (l.rot_kind != EFM_ROT_NONE && l.rot_dims > l.dim) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "more rotated channels than dim");
             if (l.sink || l.out_gate) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "sink and out_gate belong to latent attention");
+            if (input && l.qkv_bias) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "biases behind elementwise input norms");
+            if (l.mixer == EFM_MIXER_PARALLEL) {
+                if (!input) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "parallel mixers need input norms");
+                if (l.linear_heads <= 0 || l.linear_dim <= 0 || l.linear_vdim <= 0 || l.linear_decay == nullptr)
+                    return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "linear attention needs positive sizes and a decay per head");
+                if (l.linear_dim > 256 || l.linear_vdim > 256) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "linear attention heads above 256 channels");
+                for (int h = 0; h < l.linear_heads; ++h)
+                    if (!(l.linear_decay[h] >= 0.0 && l.linear_decay[h] <= 1.0)) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "decays must lie between 0 and 1");
+            }
         } else if (l.mixer == EFM_MIXER_LATENT_ATTENTION) {
             if (l.vdim <= 0 || l.window < 0 || l.q_rank <= 0 || l.kv_rank <= 0) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "non-positive dimension");
             if (l.vdim > 256 || l.kv_rank > 1024) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "vdim above 256 or kv_rank above 1024");
             if (l.rot_kind == EFM_ROT_NONE) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "latent attention has a rotated part");
             if (l.keep_first != 0) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "keep_first belongs to attention");
+            if (l.out_gate < EFM_GATE_NONE || l.out_gate > EFM_GATE_HEADS) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "unknown out_gate");
         } else if (l.mixer == EFM_MIXER_GENERAL_DELTA) {
             if (l.decay_rank <= 0) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "decay_rank must be positive");
             if (l.decay_rank > 512) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "decay_rank above 512");
@@ -59,8 +73,16 @@ efm_status validate(const efm_decoder_desc& d, const efm_decoder_layer* layers) 
             if ((l.rot_kind != EFM_ROT_HALF && l.rot_kind != EFM_ROT_PAIRS) || l.rot_dims <= 0 || l.rot_dims % 2 != 0 || !(l.rot_base > 0.f))
                 return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "rotation needs a kind, an even number of channels and a base");
             if (l.rot_dims > 2 * kRotMaxPairs) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "more than 256 rotated channels");
+            if (l.rot_factor < 0.f || (l.rot_factor > 0.f && !(l.rot_original > 0.f && l.rot_fast > 0.f && l.rot_slow > 0.f && l.rot_base != 1.0f)))
+                return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "a scaled rotation needs a positive factor, context and limits");
         }
+        if (l.ff > 0 && l.ff_act != EFM_ACT_POLYNORM && l.ff_act != EFM_ACT_RELU2) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "unknown ff_act");
+        if (l.ff > 0 && l.ff_act == EFM_ACT_RELU2 && !input) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "a squared ReLU behind output norms");
         if (l.experts > 0) {
+            if (!input && (l.expert_glu != EFM_GLU_SILU || l.expert_weight_input || l.shared_ff > 0))
+                return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "clamped, input-weighted or shared experts behind output norms");
+            if (l.shared_ff < 0 || l.expert_glu < EFM_GLU_SILU || l.expert_glu > EFM_GLU_CLAMPED || l.expert_score < EFM_SCORE_SOFTMAX || l.expert_score > EFM_SCORE_SIGMOID)
+                return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "unknown form of the experts");
             if (l.ff > 0 || l.expert_ff <= 0 || l.expert_top <= 0 || l.expert_groups <= 0 || l.expert_groups_kept <= 0 ||
                 l.expert_groups_kept > l.expert_groups || l.experts % l.expert_groups != 0 ||
                 l.expert_top > l.experts / l.expert_groups * l.expert_groups_kept)
@@ -79,14 +101,46 @@ cudaError_t alloc_linear(efm_b200_ctx* c, DecLinear& w, int N, int K, bool bias 
     return e;
 }
 
-// base^(-2 i / dims), rounded once
+// base^(-2 i / dims), rounded once.  Scaled: the pairs that turn rot_fast and rot_slow times within the original context bound a
+// ramp from the frequency itself to a rot_factor-th of it.
 cudaError_t alloc_inv_freq(efm_b200_ctx* c, DecoderLayer& l) {
     if (l.d.rot_kind == EFM_ROT_NONE) return cudaSuccess;
     std::vector<float> f((size_t)l.d.rot_dims / 2);
-    for (size_t i = 0; i < f.size(); ++i) f[i] = (float)std::pow((double)l.d.rot_base, -2.0 * (double)i / l.d.rot_dims);
+    const double dims = l.d.rot_dims, base = l.d.rot_base, factor = l.d.rot_factor;
+    double lo = 0.0, hi = 0.0;
+    if (factor > 0.0) {
+        auto pair = [&](double turns) { return dims * std::log(l.d.rot_original / (2.0 * M_PI * turns)) / (2.0 * std::log(base)); };
+        lo = std::max(std::floor(pair(l.d.rot_fast)), 0.0);
+        hi = std::min(std::ceil(pair(l.d.rot_slow)), dims - 1.0);
+    }
+    for (size_t i = 0; i < f.size(); ++i) {
+        double w = std::pow(base, -2.0 * (double)i / dims);
+        if (factor > 0.0) {
+            const double ramp = std::min(std::max(((double)i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+            w = w / factor * ramp + w * (1.0 - ramp);
+        }
+        f[i] = (float)w;
+    }
     cudaError_t e = dev_alloc(c, &l.inv_freq, f.size());
     if (e == cudaSuccess) e = cudaStreamSynchronize(c->stream);
     return e == cudaSuccess ? cudaMemcpy(l.inv_freq, f.data(), f.size() * sizeof(float), cudaMemcpyHostToDevice) : e;
+}
+
+// decay^i of every head, rounded once
+cudaError_t alloc_powers(efm_b200_ctx* c, DecoderLayer& l) {
+    std::vector<float> f;
+    for (int h = 0; h < l.d.linear_heads; ++h)
+        for (int i = 0; i <= kLinearChunk; ++i) f.push_back((float)std::pow(l.d.linear_decay[h], (double)i));
+    cudaError_t e = dev_alloc(c, &l.lin_powers, f.size());
+    if (e == cudaSuccess) e = cudaStreamSynchronize(c->stream);
+    return e == cudaSuccess ? cudaMemcpy(l.lin_powers, f.data(), f.size() * sizeof(float), cudaMemcpyHostToDevice) : e;
+}
+
+cudaError_t alloc_norm(efm_b200_ctx* c, DecNorm& n, int width, bool tanh) {
+    cudaError_t e = dev_alloc(c, &n.w, width);
+    if (e == cudaSuccess && tanh) e = dev_alloc(c, &n.b, width);
+    if (e == cudaSuccess && tanh) e = dev_alloc(c, &n.alpha, 1);
+    return e;
 }
 
 }  // namespace
@@ -135,7 +189,7 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
     EFM_TRY(cudaStreamCreateWithFlags(&c->stream, cudaStreamNonBlocking));
     for (auto& ev : c->events) EFM_TRY(cudaEventCreate(&ev));
     EFM_TRY(configure_sampler());
-    const bool sandwich = desc->norm_layout == EFM_NORM_SANDWICH;
+    const bool outputs = desc->norm_layout != EFM_NORM_INPUT, inputs = desc->norm_layout != EFM_NORM_OUTPUT, tanh = !outputs;
     for (int i = 0; i < desc->num_layers; ++i) {
         const int times = desc->loop_times > 1 && i == desc->loop_start ? desc->loop_times : 1;
         const int stop = times > 1 ? desc->loop_stop : i + 1;
@@ -150,21 +204,35 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
 
     const size_t rows = (size_t)std::max(desc->cache_pages, 1) * EFM_PAGE_TOKENS, es = act_bytes(*m);
     size_t w_in = 8, w_mix = 8, w_ff = 8, w_q = 8, w_delta_in = 8, n_pack = 8, w_rank = 8, w_cq = 8, k_max = Wp;
-    size_t ws_c = 0, ws_kv = 0, n_experts = 0, w_route = 8, ex_ff = 0, top = 0, w_act = 8;
+    size_t ws_c = 0, ws_kv = 0, n_experts = 0, w_route = 8, ex_ff = 0, top = 0, w_act = 8, n_lin = 0, w_lin = 0, sh_ff = 0;
     bool any_delta = false, any_dense = false, ws_full = false;
     m->layers.resize(desc->num_layers);
     for (int i = 0; i < desc->num_layers; ++i) {
         DecoderLayer& l = m->layers[i];
         l.d = layers[i];
         const efm_decoder_layer& d = l.d;
-        EFM_TRY(dev_alloc(c, &l.post1, Wp));
-        if (sandwich) EFM_TRY(dev_alloc(c, &l.pre1, Wp));
+        if (outputs) EFM_TRY(dev_alloc(c, &l.post1, Wp));
+        if (inputs) EFM_TRY(alloc_norm(c, l.pre1, Wp, tanh));
         EFM_TRY(alloc_inv_freq(c, l));
-        if (d.mixer == EFM_MIXER_ATTENTION) {
+        if (l.attention()) {
             l.Dp = round_up(d.dim, 64);
             l.Vp = round_up(d.vdim, 64);
             l.mix_w = d.heads * d.vdim;
-            EFM_TRY(alloc_linear(c, l.in, (d.heads + d.kv_heads) * d.dim + d.kv_heads * d.vdim, m->W, d.qkv_bias != 0));
+            int n_in = (d.heads + d.kv_heads) * d.dim + d.kv_heads * d.vdim;
+            if (l.linear()) {
+                const int qk = d.linear_heads * d.linear_dim, v = d.linear_heads * d.linear_vdim;
+                l.lin_vp = round_up(d.linear_vdim, 4);
+                l.lin_in = round_up(n_in, 8);
+                n_in = l.lin_in + 2 * round_up(qk, 8) + 2 * round_up(v, 8);
+                l.lin_mix = round_up(l.mix_w, 8);
+                l.mix_w = l.lin_mix + v;
+                EFM_TRY(dev_alloc(c, &l.mix_norm, round_up(v, 8)));
+                EFM_TRY(alloc_powers(c, l));
+                n_lin = std::max(n_lin, decoder_linear_ws_floats(l, S, std::min(desc->max_slots, S)));
+                w_lin = std::max(w_lin, (size_t)round_up(v, 8));
+            }
+            l.d.linear_decay = nullptr;
+            EFM_TRY(alloc_linear(c, l.in, n_in, m->W, d.qkv_bias != 0));
             if (d.qk_norm == EFM_QK_NORM_WEIGHTED) {
                 EFM_TRY(dev_alloc(c, &l.q_norm, d.dim));
                 EFM_TRY(dev_alloc(c, &l.k_norm, d.dim));
@@ -179,7 +247,7 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
             l.Lc = round_up(d.kv_rank, 8);
             l.Rc = round_up(d.rot_dims, 8);
             l.mix_w = d.heads * d.vdim;
-            EFM_TRY(alloc_linear(c, l.in, l.Qp + l.Lc + l.Rc + (d.out_gate ? d.heads * d.vdim : 0), m->W));
+            EFM_TRY(alloc_linear(c, l.in, l.Qp + l.Lc + l.Rc + (d.out_gate == EFM_GATE_HEADS ? d.heads : d.out_gate ? d.heads * d.vdim : 0), m->W));
             EFM_TRY(alloc_linear(c, l.uq, d.heads * (l.Dp + l.Rc), d.q_rank));
             EFM_TRY(alloc_linear(c, l.ukv, d.heads * (l.Dp + l.Vp), d.kv_rank));
             EFM_TRY(dev_alloc(c, &l.q_norm, l.Qp));
@@ -212,25 +280,31 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
         w_mix = std::max(w_mix, (size_t)l.mix_wp);
         EFM_TRY(alloc_linear(c, l.out, m->W, l.mix_w));
         if (l.mlp()) {
-            EFM_TRY(dev_alloc(c, &l.post2, Wp));
-            if (sandwich) EFM_TRY(dev_alloc(c, &l.pre2, Wp));
+            if (outputs) EFM_TRY(dev_alloc(c, &l.post2, Wp));
+            if (inputs) EFM_TRY(alloc_norm(c, l.pre2, Wp, tanh));
         }
         if (l.moe()) {
             l.ffp = round_up(d.expert_ff, 64);
-            EFM_TRY(alloc_linear(c, l.router, d.experts, m->W));
+            EFM_TRY(alloc_linear(c, l.router, d.experts + (d.shared_ff > 0 ? 1 : 0), m->W));
             EFM_TRY(alloc_linear(c, l.expert_in, d.experts * 2 * l.ffp, m->W));
             EFM_TRY(alloc_linear(c, l.expert_out, d.experts * Wp, d.expert_ff, false, 64));
             n_experts = std::max(n_experts, (size_t)d.experts);
             w_route = std::max(w_route, (size_t)l.router.Np);
             ex_ff = std::max(ex_ff, (size_t)l.ffp);
             top = std::max(top, (size_t)d.expert_top);
-            w_act = std::max(w_act, (size_t)d.expert_top * l.ffp);
-            k_max = std::max(k_max, (size_t)d.expert_top * l.ffp);
+            if (d.shared_ff > 0) {
+                l.sfp = round_up(d.shared_ff, 64);
+                EFM_TRY(alloc_linear(c, l.shared_in, 2 * l.sfp, m->W));
+                EFM_TRY(alloc_linear(c, l.shared_out, m->W, d.shared_ff, false, 64));
+                sh_ff = std::max(sh_ff, (size_t)l.sfp);
+            }
+            w_act = std::max(w_act, (size_t)d.expert_top * l.ffp + l.sfp);
+            k_max = std::max(k_max, (size_t)d.expert_top * l.ffp + l.sfp);
         } else if (d.ff > 0) {
             any_dense = true;
             EFM_TRY(alloc_linear(c, l.up, d.ff, m->W));
             EFM_TRY(alloc_linear(c, l.down, m->W, d.ff));
-            EFM_TRY(dev_alloc(c, &l.act, 4));
+            if (d.ff_act == EFM_ACT_POLYNORM) EFM_TRY(dev_alloc(c, &l.act, 4));
             w_ff = std::max(w_ff, (size_t)l.up.Np);
         }
         if (desc->side_dim > 0) {
@@ -244,14 +318,18 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
     for (DecoderRun& r : m->runs) {
         const DecoderLayer& l = m->layers[r.layer];
         char *k = nullptr, *v = nullptr;
-        if (l.d.mixer == EFM_MIXER_ATTENTION) {
+        if (l.linear()) {
+            r.state_off = m->state_stride;
+            m->state_stride += (size_t)l.d.linear_heads * l.d.linear_dim * l.lin_vp;
+        }
+        if (l.attention()) {
             EFM_TRY(dev_alloc(c, &k, rows * l.d.kv_heads * l.Dp * es));
             EFM_TRY(dev_alloc(c, &v, rows * l.d.kv_heads * l.Vp * es));
         } else if (l.d.mixer == EFM_MIXER_LATENT_ATTENTION) {
             EFM_TRY(dev_alloc(c, &k, rows * (l.Lc + l.Rc) * es));
         } else {
             r.state_off = m->state_stride;
-            m->state_stride += (size_t)l.d.heads * l.d.dim * l.d.dim;
+            m->state_stride += ((size_t)l.d.heads * l.d.dim * l.d.dim + 3) / 4 * 4;
         }
         r.k_pool = k;
         r.v_pool = v;
@@ -259,18 +337,22 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
     {   // the longest GEMV input must fit the kernel's shared memory as fp32
         int optin = 0;
         EFM_TRY(cudaDeviceGetAttribute(&optin, cudaDevAttrMaxSharedMemoryPerBlockOptin, device_id));
-        if (std::max(std::max(gemv_smem_bytes((int)k_max), gemv_ext_smem_bytes(Wp)), gemv_ext_smem_bytes((int)w_cq)) + 2048 > (size_t)optin) {
+        size_t need = std::max(std::max(gemv_smem_bytes((int)k_max), gemv_ext_smem_bytes(Wp)), gemv_ext_smem_bytes((int)w_cq));
+        for (const DecoderLayer& l : m->layers)
+            if (l.linear()) need = std::max(need, gemv_ext_smem_bytes(l.out.Kp));
+        if (need + 2048 > (size_t)optin) {
             efm_status s = fail(nullptr, EFM_ERR_UNSUPPORTED, "width / feed-forward size exceeds what the decode GEMV stages in shared memory");
             efm_b200_destroy(c);
             return s;
         }
     }
-    EFM_TRY(dev_alloc(c, &c->embed, (size_t)desc->vocab * Wp));
-    if (desc->side_dim > 0) EFM_TRY(dev_alloc(c, &m->side_embed, (size_t)desc->vocab * desc->side_dim * desc->num_layers));
-    EFM_TRY(dev_alloc(c, &m->final_norm, Wp));
     EFM_TRY(alloc_linear(c, m->head, desc->vocab, m->W));
+    if (desc->tied_head) c->embed = m->head.w;
+    else EFM_TRY(dev_alloc(c, &c->embed, (size_t)desc->vocab * Wp));
+    if (desc->side_dim > 0) EFM_TRY(dev_alloc(c, &m->side_embed, (size_t)desc->vocab * desc->side_dim * desc->num_layers));
+    EFM_TRY(alloc_norm(c, m->final_norm, Wp, tanh));
     c->lm_head = m->head.w;
-    c->final_norm = m->final_norm;
+    c->final_norm = m->final_norm.w;
 
     EFM_TRY(dev_alloc(c, &m->page_table, (size_t)desc->max_slots * std::max(desc->cache_pages, 1)));
     if (m->state_stride > 0) EFM_TRY(dev_alloc(c, &m->state_pool, m->state_stride * std::max(desc->state_slots, 1)));
@@ -284,7 +366,7 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
     };
     EFM_TRY(dev_alloc(c, &c->ids, S));
     EFM_TRY(dev_alloc(c, &c->resid, (size_t)S * Wp));
-    if (!m->f32 || sandwich) EFM_TRY(act(&m->xa, (size_t)S * Wp));
+    if (!m->f32 || inputs) EFM_TRY(act(&m->xa, (size_t)S * Wp));
     EFM_TRY(act(&m->cq, S * w_cq));
     if (ws_c > 0) {
         // the rows' own pages plus, for every entry long enough, those of a window
@@ -310,13 +392,21 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
         EFM_TRY(dev_alloc(c, &m->ex.count, n_experts));
         EFM_TRY(dev_alloc(c, &m->ex.tile, (size_t)m->ex_rows / kExpertTile));
         EFM_TRY(dev_alloc(c, &m->ex.n_tiles, 1));
+        EFM_TRY(dev_alloc(c, &m->ex.shared, S));
+        if (sh_ff > 0) {
+            EFM_TRY(act(&m->sh_act, S * sh_ff));
+            EFM_TRY(act(&m->sh_y, (size_t)S * Wp));
+            if (m->f32) EFM_TRY(dev_alloc(c, &m->sh_gu, S * 2 * sh_ff));
+        }
         EFM_TRY(dev_alloc(c, &m->d_h, Wp));
         EFM_TRY(dev_alloc(c, &m->d_route, w_route));
         EFM_TRY(dev_alloc(c, &m->d_act, w_act));
         EFM_TRY(dev_alloc(c, &m->d_route_id, top));
-        EFM_TRY(dev_alloc(c, &m->d_route_w, top));
+        EFM_TRY(dev_alloc(c, &m->d_route_w, top + 1));
         EFM_TRY(dev_alloc(c, &m->d_route_ticket, 1));
     }
+    if (n_lin > 0) EFM_TRY(dev_alloc(c, &m->lin_ws, n_lin));
+    if (n_lin > 0 || any_delta) EFM_TRY(dev_alloc(c, &m->o, S * std::max(w_lin, any_delta ? w_mix : 0)));
     EFM_TRY(act(&m->proj_a, S * w_in));
     EFM_TRY(act(&m->q, S * w_q));
     EFM_TRY(act(&m->mix, S * w_mix));
@@ -332,7 +422,6 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
         EFM_TRY(dev_alloc(c, &m->pack, n_pack));
         EFM_TRY(dev_alloc(c, &m->tanh_w, S * w_rank));
         EFM_TRY(dev_alloc(c, &m->decay, S * w_mix));
-        EFM_TRY(dev_alloc(c, &m->o, S * w_mix));
     }
     m->max_want = std::min(S, 256);
     EFM_TRY(act(&m->head_a, (size_t)m->max_want * Wp));
@@ -644,26 +733,36 @@ efm_status efm_b200_decoder_read_taps(efm_b200_ctx* c, float* host_out) {
 namespace {
 
 // ---- weights -------------------------------------------------------------------------------------------------------
-// Rows [src, src + n) of a tensor become rows [dst, dst + n) of a (fused, padded) linear.
-struct Piece { int dst, src, n; };
+// Rows [src, src + n) of a tensor become rows [dst, dst + n) of a (fused, padded) linear, from column `col` on.
+struct Piece { int dst, src, n, col = 0; };
 
 efm_status put_rows(efm_b200_ctx* c, const DecLinear& w, const std::vector<Piece>& pieces, const void* data, const std::string& name, const int64_t* shape,
-                    int ndim, int mem_kind) {
+                    int ndim, int mem_kind, int cols) {
+    const int K = cols > 0 ? cols : w.K;             // a part of the linear's columns, or all
     int rows = 0;
     for (const Piece& p : pieces) rows += p.n;
-    if (!shape_is(shape, ndim, rows, w.K)) return fail(c, EFM_ERR_INVALID_ARGUMENT, "unexpected shape for " + name);
+    if (!shape_is(shape, ndim, rows, K)) return fail(c, EFM_ERR_INVALID_ARGUMENT, "unexpected shape for " + name);
     for (const Piece& p : pieces)
-        EFM_CK(c, cudaMemcpy2DAsync(w.w + (size_t)p.dst * w.Kp, (size_t)w.Kp * 2, static_cast<const char*>(data) + (size_t)p.src * w.K * 2, (size_t)w.K * 2,
-                                    (size_t)w.K * 2, (size_t)p.n, mem_kind == EFM_MEM_DEVICE ? cudaMemcpyDeviceToDevice : cudaMemcpyHostToDevice, c->stream));
+        EFM_CK(c, cudaMemcpy2DAsync(w.w + (size_t)p.dst * w.Kp + p.col, (size_t)w.Kp * 2, static_cast<const char*>(data) + (size_t)p.src * K * 2, (size_t)K * 2,
+                                    (size_t)K * 2, (size_t)p.n, mem_kind == EFM_MEM_DEVICE ? cudaMemcpyDeviceToDevice : cudaMemcpyHostToDevice, c->stream));
     return EFM_OK;
 }
 efm_status put_vec(efm_b200_ctx* c, __nv_bfloat16* dst, int n, const void* data, const std::string& name, const int64_t* shape, int ndim, int mem_kind) {
-    if (!shape_is(shape, ndim, n)) return fail(c, EFM_ERR_INVALID_ARGUMENT, "unexpected shape for " + name);
+    if (!(n == 1 && ndim == 0) && !shape_is(shape, ndim, n)) return fail(c, EFM_ERR_INVALID_ARGUMENT, "unexpected shape for " + name);
     return copy_rows(c, dst, data, (size_t)n * 2, mem_kind);
 }
 
 // Where a tensor goes: a row range of a (fused) linear or a vector.
-struct Target { DecLinear* lin = nullptr; std::vector<Piece> pieces; __nv_bfloat16* vec = nullptr; int n = 0; };
+struct Target { DecLinear* lin = nullptr; std::vector<Piece> pieces; int cols = 0; __nv_bfloat16* vec = nullptr; int n = 0; };
+
+// `name`, `name`.b or `name`.alpha of an input norm
+bool norm_target(const DecoderModel& m, const DecNorm& n, const std::string& what, const char* name, Target* t) {
+    const std::string base(name);
+    if (what == base) { t->vec = n.w; t->n = m.W; }
+    else if (what == base + ".b") { t->vec = n.b; t->n = m.W; }
+    else if (what == base + ".alpha") { t->vec = n.alpha; t->n = 1; }
+    return t->vec != nullptr;
+}
 
 bool layer_target(DecoderModel& m, DecoderLayer& l, const std::string& rest, Target* t) {
     const efm_decoder_layer& d = l.d;
@@ -679,12 +778,30 @@ bool layer_target(DecoderModel& m, DecoderLayer& l, const std::string& rest, Tar
         return true;
     };
     const bool sandwich = m.d.norm_layout == EFM_NORM_SANDWICH;
-    if (rest == "norm1") return vec(sandwich ? l.pre1 : l.post1, m.W);
-    if (rest == "norm2") return vec(sandwich ? l.pre2 : l.post2, m.W);
+    if (m.d.norm_layout == EFM_NORM_OUTPUT) {
+        if (rest == "norm1") return vec(l.post1, m.W);
+        if (rest == "norm2") return vec(l.post2, m.W);
+    } else if (norm_target(m, l.pre1, rest, "norm1", t) || norm_target(m, l.pre2, rest, "norm2", t)) {
+        return true;
+    }
     if (sandwich && rest == "norm1b") return vec(l.post1, m.W);
     if (sandwich && rest == "norm2b") return vec(l.post2, m.W);
-    if (rest == "mix.o") return lin(l.out, 0, m.W);
-    if (d.mixer == EFM_MIXER_ATTENTION) {
+    if (rest == "mix.o" && !l.linear()) return lin(l.out, 0, m.W);
+    if (l.linear()) {                                  // the two halves share one projection and one output product
+        const int q = d.heads * d.dim, k = d.kv_heads * d.dim, lv = d.linear_heads * d.linear_vdim, lq = d.linear_heads * d.linear_dim;
+        auto out = [&](int col, int cols) { t->lin = &l.out; t->cols = cols; t->pieces.push_back(Piece{0, 0, m.W, col}); return true; };
+        if (rest == "mix.left.q") return lin(l.in, 0, q);
+        if (rest == "mix.left.k") return lin(l.in, q, k);
+        if (rest == "mix.left.v") return lin(l.in, q + k, d.kv_heads * d.vdim);
+        if (rest == "mix.left.o") return out(0, d.heads * d.vdim);
+        const int qp = round_up(lq, 8), vp = round_up(lv, 8);
+        if (rest == "mix.right.q") return lin(l.in, l.lin_in, lq);
+        if (rest == "mix.right.k") return lin(l.in, l.lin_in + qp, lq);
+        if (rest == "mix.right.v") return lin(l.in, l.lin_in + 2 * qp, lv);
+        if (rest == "mix.right.g") return lin(l.in, l.lin_in + 2 * qp + vp, lv);
+        if (rest == "mix.right.o") return out(l.lin_mix, lv);
+        if (rest == "mix.right.norm") return vec(l.mix_norm, lv);
+    } else if (d.mixer == EFM_MIXER_ATTENTION) {
         const int q = d.heads * d.dim, k = d.kv_heads * d.dim;
         if (rest == "mix.q") return lin(l.in, 0, q);
         if (rest == "mix.k") return lin(l.in, q, k);
@@ -704,7 +821,7 @@ bool layer_target(DecoderModel& m, DecoderLayer& l, const std::string& rest, Tar
             t->pieces.push_back(Piece{l.Qp + l.Lc, d.kv_rank, d.rot_dims});
             return true;
         }
-        if (rest == "mix.g" && d.out_gate) return lin(l.in, l.Qp + l.Lc + l.Rc, d.heads * d.vdim);
+        if (rest == "mix.g" && d.out_gate) return lin(l.in, l.Qp + l.Lc + l.Rc, d.out_gate == EFM_GATE_HEADS ? d.heads : d.heads * d.vdim);
         if (rest == "mix.uq") return heads(l.uq, 0, l.Dp + l.Rc, d.dim + d.rot_dims, d.dim, l.Dp - d.dim);
         if (rest == "mix.uk") return heads(l.ukv, 0, l.Dp, d.dim, d.dim, 0);
         if (rest == "mix.uv") return heads(l.ukv, d.heads * l.Dp, l.Vp, d.vdim, d.vdim, 0);
@@ -724,6 +841,16 @@ bool layer_target(DecoderModel& m, DecoderLayer& l, const std::string& rest, Tar
     }
     if (l.moe()) {
         if (rest == "mlp.router") return lin(l.router, 0, d.experts);
+        auto gate_up = [&](DecLinear& w, int row0, int n, bool up) {     // 64 gate rows, the 64 matching up rows, ...
+            t->lin = &w;
+            for (int r = 0; r < n; r += 64) t->pieces.push_back(Piece{row0 + 2 * r + (up ? 64 : 0), r, std::min(64, n - r)});
+            return true;
+        };
+        if (d.shared_ff > 0) {
+            if (rest == "mlp.shared.gate" || rest == "mlp.shared.up") return gate_up(l.shared_in, 0, d.shared_ff, rest == "mlp.shared.up");
+            if (rest == "mlp.shared.down") return lin(l.shared_out, 0, m.W);
+            if (rest == "mlp.shared.sg") return lin(l.router, d.experts, 1);
+        }
         const size_t dot = rest.find('.', 5);
         if (rest.compare(0, 5, "mlp.e") == 0 && dot != std::string::npos && dot > 5) {
             const int e = std::atoi(rest.c_str() + 5);
@@ -731,15 +858,12 @@ bool layer_target(DecoderModel& m, DecoderLayer& l, const std::string& rest, Tar
             if (rest.substr(5, dot - 5) != std::to_string(e) || e >= d.experts) return false;
             if (what == "down") return lin(l.expert_out, e * m.Wp, m.W);
             if (what != "gate" && what != "up") return false;
-            t->lin = &l.expert_in;                     // 64 gate rows, the 64 matching up rows, ...
-            for (int r = 0; r < d.expert_ff; r += 64)
-                t->pieces.push_back(Piece{e * 2 * l.ffp + 2 * r + (what == "up" ? 64 : 0), r, std::min(64, d.expert_ff - r)});
-            return true;
+            return gate_up(l.expert_in, e * 2 * l.ffp, d.expert_ff, what == "up");
         }
     } else if (d.ff > 0) {
         if (rest == "mlp.up") return lin(l.up, 0, d.ff);
         if (rest == "mlp.down") return lin(l.down, 0, m.W);
-        if (rest == "mlp.act") return vec(l.act, 4);
+        if (rest == "mlp.act" && l.act != nullptr) return vec(l.act, 4);
     }
     if (m.d.side_dim > 0) {
         if (rest == "side.gate") return lin(l.gate, 0, m.d.side_dim);
@@ -759,8 +883,8 @@ efm_status decoder_set_weight(efm_b200_ctx* c, const char* raw, const void* data
         table.w = m.side_embed; table.K = table.Kp = m.d.side_dim * m.d.num_layers;
         t.lin = &table; t.pieces.push_back(Piece{0, 0, m.d.vocab});
     }
-    else if (name == "head") { t.lin = &m.head; t.pieces.push_back(Piece{0, 0, m.d.vocab}); }
-    else if (name == "final.norm") { t.vec = m.final_norm; t.n = m.W; }
+    else if (name == "head" && !m.d.tied_head) { t.lin = &m.head; t.pieces.push_back(Piece{0, 0, m.d.vocab}); }
+    else if (norm_target(m, m.final_norm, name, "final.norm", &t)) {}
     else if (name.size() > 1 && name[0] == 'l' && name[1] >= '0' && name[1] <= '9') {
         const size_t dot = name.find('.');
         const int i = std::atoi(name.c_str() + 1);
@@ -769,7 +893,7 @@ efm_status decoder_set_weight(efm_b200_ctx* c, const char* raw, const void* data
         return EFM_OK;                     // not part of this model
     }
     if (dtype != EFM_BF16) return fail(c, EFM_ERR_UNSUPPORTED, "weights must be bf16: " + name);
-    const efm_status st = t.lin != nullptr ? put_rows(c, *t.lin, t.pieces, data, name, shape, ndim, mem_kind)
+    const efm_status st = t.lin != nullptr ? put_rows(c, *t.lin, t.pieces, data, name, shape, ndim, mem_kind, t.cols)
                                            : put_vec(c, t.vec, t.n, data, name, shape, ndim, mem_kind);
     if (st != EFM_OK) return st;
     EFM_CK(c, cudaStreamSynchronize(c->stream));          // the caller may release `data` on return
@@ -779,18 +903,25 @@ efm_status decoder_set_weight(efm_b200_ctx* c, const char* raw, const void* data
 
 efm_status decoder_finalize(efm_b200_ctx* c) {
     DecoderModel& m = *c->decoder;
-    std::vector<std::string> need = {"embed", "head", "final.norm"};
+    const bool tanh = m.tanh_norms();
+    std::vector<std::string> need = {"embed", "final.norm"};
+    if (!m.d.tied_head) need.push_back("head");
+    if (tanh) for (const char* n : {"final.norm.b", "final.norm.alpha"}) need.push_back(n);
     if (m.d.side_dim > 0) need.push_back("side.embed");
     for (int i = 0; i < m.d.num_layers; ++i) {
         const efm_decoder_layer& d = m.layers[i].d;
         auto add = [&](std::initializer_list<const char*> names) { for (const char* n : names) need.push_back("l" + std::to_string(i) + "." + n); };
-        add({"norm1", "mix.o"});
+        add({"norm1"});
+        if (tanh) add({"norm1.b", "norm1.alpha"});
+        if (d.mixer != EFM_MIXER_PARALLEL) add({"mix.o"});
         if (m.d.norm_layout == EFM_NORM_SANDWICH) add({"norm1b"});
         if (d.mixer == EFM_MIXER_ATTENTION) {
             add({"mix.q", "mix.k", "mix.v"});
             if (d.qk_norm == EFM_QK_NORM_WEIGHTED) add({"mix.q.norm", "mix.k.norm"});
             if (d.head_temp) add({"mix.temp"});
             if (d.qkv_bias) add({"mix.q.b", "mix.k.b", "mix.v.b"});
+        } else if (d.mixer == EFM_MIXER_PARALLEL) {
+            add({"mix.left.q", "mix.left.k", "mix.left.v", "mix.left.o", "mix.right.q", "mix.right.k", "mix.right.v", "mix.right.g", "mix.right.o", "mix.right.norm"});
         } else if (d.mixer == EFM_MIXER_LATENT_ATTENTION) {
             add({"mix.dq", "mix.dq.norm", "mix.uq", "mix.dkv", "mix.dkv.norm", "mix.uk", "mix.uv"});
             if (d.sink) add({"mix.sink"});
@@ -798,14 +929,17 @@ efm_status decoder_finalize(efm_b200_ctx* c) {
         } else add({"mix.r", "mix.k", "mix.v", "mix.g", "mix.a", "mix.a.b", "mix.w1", "mix.w2", "mix.w0", "mix.norm"});
         if (d.experts > 0 || d.ff > 0) {
             add({"norm2"});
+            if (tanh) add({"norm2.b", "norm2.alpha"});
             if (m.d.norm_layout == EFM_NORM_SANDWICH) add({"norm2b"});
         }
         if (d.experts > 0) {
             add({"mlp.router"});
+            if (d.shared_ff > 0) add({"mlp.shared.gate", "mlp.shared.up", "mlp.shared.down", "mlp.shared.sg"});
             for (int e = 0; e < d.experts; ++e)
                 for (const char* what : {".gate", ".up", ".down"}) add({("mlp.e" + std::to_string(e) + what).c_str()});
         } else if (d.ff > 0) {
-            add({"mlp.up", "mlp.down", "mlp.act"});
+            add({"mlp.up", "mlp.down"});
+            if (d.ff_act == EFM_ACT_POLYNORM) add({"mlp.act"});
         }
         if (m.d.side_dim > 0) add({"side.gate", "side.proj", "side.norm"});
     }
@@ -859,10 +993,11 @@ int64_t decoder_step_bytes(const efm_b200_ctx& c, int32_t kv_len) {
     int64_t b = lin(m.head) + (int64_t)m.W * 2 * 2;
     for (const DecoderRun& r : m.runs) {
         const DecoderLayer& l = m.layers[r.layer];
-        b += lin(l.in) + lin(l.out) + lin(l.w2) + lin(l.up) + lin(l.down) + lin(l.gate) + lin(l.proj) + lin(l.uq) + lin(l.ukv) + lin(l.router);
+        b += lin(l.in) + lin(l.out) + lin(l.w2) + lin(l.up) + lin(l.down) + lin(l.gate) + lin(l.proj) + lin(l.uq) + lin(l.ukv) + lin(l.router) + lin(l.shared_in) + lin(l.shared_out);
         if (l.moe()) b += (int64_t)l.d.expert_top * 3 * l.d.expert_ff * m.W * 2;
         const int64_t n = l.d.window > 0 ? std::min(kv_len, l.d.window + l.d.keep_first) : kv_len;
-        if (l.d.mixer == EFM_MIXER_ATTENTION) b += n * l.d.kv_heads * (l.d.dim + l.d.vdim) * (m.f32 ? 4 : 2);
+        if (l.linear()) b += 2 * (int64_t)l.d.linear_heads * l.d.linear_dim * l.lin_vp * 4;
+        if (l.attention()) b += n * l.d.kv_heads * (l.d.dim + l.d.vdim) * (m.f32 ? 4 : 2);
         else if (l.d.mixer == EFM_MIXER_LATENT_ATTENTION) b += n * (l.d.kv_rank + l.d.rot_dims) * (m.f32 ? 4 : 2);
         else b += 2 * (int64_t)l.d.heads * l.d.dim * l.d.dim * 4;
     }

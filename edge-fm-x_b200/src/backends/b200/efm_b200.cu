@@ -110,7 +110,7 @@ efm_status efm_b200_destroy(efm_b200_ctx* c) {
 
 efm_status efm_b200_set_weight(efm_b200_ctx* c, const char* hf_name, const void* data, const int64_t* shape,
                                int32_t ndim, int32_t dtype, int32_t mem_kind) {
-    if (c == nullptr || hf_name == nullptr || data == nullptr || shape == nullptr)
+    if (c == nullptr || hf_name == nullptr || data == nullptr || (shape == nullptr && ndim != 0))
         return fail(c, EFM_ERR_INVALID_ARGUMENT, "null argument");
     if (c->finalized) return fail(c, EFM_ERR_STATE, "weights are already finalized");
     EFM_CK(c, cudaSetDevice(c->device));

@@ -9,6 +9,11 @@
 // mask {size, keep_first}} or "latent_attention" {heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, rot {base, dims},
 // mask {size}}; mlp null or {kind: "moe", expert.ff, router {experts, top, groups {count, keep}}}; "norm.eps",
 // "embedding.scale", "loop" {start, stop, times}, "vocab", "width".
+//
+// Vekolix: "layers" lists {type, mixer, mlp}; type "latent_attention" {heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, rot} or
+// "parallel" {left {heads, kv_heads, dim, vdim, scale, rot}, right {heads, dim, vdim, decay}, left_scale, right_scale}; rot {base,
+// dims, scaling {factor, original, fast, slow}}; mlp null, {kind: "dense", ff} or {kind: "moe", expert {ff, limit}, router
+// {experts, top}, shared {ff, limit}}; "norm.eps", "residual_mult", "logit_scale", "logit_softcap", "vocab", "width".
 #include <efm_b200.h>
 
 #include <algorithm>
@@ -25,6 +30,7 @@ namespace {
 struct DecoderConfig {
     efm_decoder_desc desc{};
     std::vector<efm_decoder_layer> layers;
+    std::vector<std::vector<double>> decays;             // by layer; efm_decoder_layer::linear_decay points here once all are read
 };
 using Shapes = std::map<std::string, std::vector<int64_t>>;
 
@@ -58,6 +64,7 @@ void read_model(const json::Value& cfg, efm_decoder_desc& d) {
     d.width = positive(cfg, "width", "model");
     d.norm_eps = (float)member(member(cfg, "norm", "model"), "eps", "norm").num;
     d.embed_scale = 1.0f;
+    d.logit_scale = 1.0f;
 }
 const json::Value& layer_list(const json::Value& cfg) {
     const json::Value& layers = member(cfg, "layers", "model");
@@ -114,6 +121,15 @@ void read_rotation(const json::Value& mix, int32_t kind, const std::string& wher
     e.rot_kind = kind;
     e.rot_dims = positive(rot, "dims", where + ".rot");
     e.rot_base = number(rot, "base", where + ".rot");
+    const json::Value* scaling = rot.find("scaling");
+    if (!given(scaling)) return;
+    const std::string in = where + ".rot.scaling";
+    for (const char* key : {"factor", "original", "fast", "slow"})
+        if (number(*scaling, key, in) <= 0.f) throw ConfigurationError("config.json: " + in + "." + key + " must be positive");
+    e.rot_factor = number(*scaling, "factor", in);
+    e.rot_original = number(*scaling, "original", in);
+    e.rot_fast = number(*scaling, "fast", in);
+    e.rot_slow = number(*scaling, "slow", in);
 }
 
 void read_experts(const json::Value& mlp, const std::string& where, efm_decoder_layer& e) {
@@ -131,6 +147,18 @@ void read_experts(const json::Value& mlp, const std::string& where, efm_decoder_
     }
 }
 
+void read_latent(const json::Value& mix, const std::string& in, efm_decoder_layer& e) {
+    e.mixer = EFM_MIXER_LATENT_ATTENTION;
+    e.heads = positive(mix, "heads", in);
+    e.dim = positive(mix, "dim", in);
+    e.vdim = positive(mix, "vdim", in);
+    e.scale = number(mix, "scale", in);
+    e.q_rank = positive(mix, "q_rank", in);
+    e.kv_rank = positive(mix, "kv_rank", in);
+    read_rotation(mix, EFM_ROT_PAIRS, in, e);
+    if (positive(mix, "rot_dim", in) != e.rot_dims) throw ConfigurationError("config.json: " + in + ".rot.dims must be rot_dim");
+}
+
 DecoderConfig temuvik_config(const json::Value& cfg, const Shapes&) {
     DecoderConfig out;
     efm_decoder_desc& d = out.desc;
@@ -144,27 +172,23 @@ DecoderConfig temuvik_config(const json::Value& cfg, const Shapes&) {
         const json::Value& mix = member(l, "mixer", where);
         const std::string type = l.get_string("type", "");
         efm_decoder_layer e{};
-        e.heads = positive(mix, "heads", in);
-        e.dim = positive(mix, "dim", in);
-        e.vdim = positive(mix, "vdim", in);
-        e.scale = number(mix, "scale", in);
         const json::Value* mask = mix.find("mask");
         if (given(mask)) e.window = positive(*mask, "size", in + ".mask");
         if (type == "attention") {
             e.mixer = EFM_MIXER_ATTENTION;
+            e.heads = positive(mix, "heads", in);
+            e.dim = positive(mix, "dim", in);
+            e.vdim = positive(mix, "vdim", in);
+            e.scale = number(mix, "scale", in);
             e.kv_heads = positive(mix, "kv_heads", in);
             e.qk_norm = EFM_QK_NORM_PLAIN;
             e.qkv_bias = 1;
             if (given(mask) && mask->find("keep_first") != nullptr) e.keep_first = whole(*mask, "keep_first", in + ".mask");
             read_rotation(mix, EFM_ROT_HALF, in, e);
         } else if (type == "latent_attention") {
-            e.mixer = EFM_MIXER_LATENT_ATTENTION;
-            e.q_rank = positive(mix, "q_rank", in);
-            e.kv_rank = positive(mix, "kv_rank", in);
+            read_latent(mix, in, e);
             e.sink = 1;
-            e.out_gate = 1;
-            read_rotation(mix, EFM_ROT_PAIRS, in, e);
-            if (positive(mix, "rot_dim", in) != e.rot_dims) throw ConfigurationError("config.json: " + in + ".rot.dims must be rot_dim");
+            e.out_gate = EFM_GATE_CHANNELS;
         } else {
             throw ConfigurationError("config.json: " + where + " has an unknown type \"" + type + "\"");
         }
@@ -180,6 +204,77 @@ DecoderConfig temuvik_config(const json::Value& cfg, const Shapes&) {
         d.loop_times = positive(*loop, "times", "loop");
         if (d.loop_stop <= d.loop_start || d.loop_stop > d.num_layers) throw ConfigurationError("config.json: loop.start .. loop.stop must be a span of the layers");
     }
+    return out;
+}
+
+void read_parallel(const json::Value& mix, const std::string& in, efm_decoder_layer& e, std::vector<double>& decay) {
+    e.mixer = EFM_MIXER_PARALLEL;
+    const json::Value &left = member(mix, "left", in), &right = member(mix, "right", in);
+    const std::string l = in + ".left", r = in + ".right";
+    e.heads = positive(left, "heads", l);
+    e.kv_heads = positive(left, "kv_heads", l);
+    e.dim = positive(left, "dim", l);
+    e.vdim = positive(left, "vdim", l);
+    e.scale = number(left, "scale", l);
+    e.qk_norm = EFM_QK_NORM_NONE;
+    read_rotation(left, EFM_ROT_HALF, l, e);
+    e.linear_heads = positive(right, "heads", r);
+    e.linear_dim = positive(right, "dim", r);
+    e.linear_vdim = positive(right, "vdim", r);
+    e.mix_scale = number(mix, "left_scale", in);
+    e.linear_scale = number(mix, "right_scale", in);
+    const json::Value& d = member(right, "decay", r);
+    if (!d.is_array() || (int32_t)d.arr.size() != e.linear_heads) throw ConfigurationError("config.json: " + r + ".decay must list one number per head");
+    for (const json::Value& v : d.arr) {
+        if (!v.is_number()) throw ConfigurationError("config.json: " + r + ".decay must list one number per head");
+        decay.push_back(v.num);
+    }
+}
+
+DecoderConfig vekolix_config(const json::Value& cfg, const Shapes&) {
+    DecoderConfig out;
+    efm_decoder_desc& d = out.desc;
+    read_model(cfg, d);
+    d.norm_layout = EFM_NORM_INPUT;
+    d.tied_head = 1;
+    d.residual_mult = number(cfg, "residual_mult", "model");
+    d.logit_scale = number(cfg, "logit_scale", "model");
+    d.logit_softcap = number(cfg, "logit_softcap", "model");
+    const json::Value& layers = layer_list(cfg);
+    out.decays.resize(layers.arr.size());
+    for (size_t i = 0; i < layers.arr.size(); ++i) {
+        const json::Value& l = layers.arr[i];
+        const std::string where = "layers[" + std::to_string(i) + "]", in = where + ".mixer", ff = where + ".mlp";
+        const json::Value& mix = member(l, "mixer", where);
+        const std::string type = l.get_string("type", "");
+        efm_decoder_layer e{};
+        if (type == "latent_attention") {
+            read_latent(mix, in, e);
+            e.out_gate = EFM_GATE_HEADS;
+        } else if (type == "parallel") {
+            read_parallel(mix, in, e, out.decays[i]);
+        } else {
+            throw ConfigurationError("config.json: " + where + " has an unknown type \"" + type + "\"");
+        }
+        const json::Value* mlp = l.find("mlp");
+        if (given(mlp) && mlp->get_string("kind", "") == "dense") {
+            e.ff = positive(*mlp, "ff", ff);
+            e.ff_act = EFM_ACT_RELU2;
+        } else if (given(mlp)) {
+            read_experts(*mlp, ff, e);
+            e.expert_glu = EFM_GLU_CLAMPED;
+            e.expert_score = EFM_SCORE_SIGMOID;
+            e.expert_weight_input = 1;
+            e.expert_limit = number(member(*mlp, "expert", ff), "limit", ff + ".expert");
+            const json::Value* shared = mlp->find("shared");
+            if (given(shared)) {
+                e.shared_ff = positive(*shared, "ff", ff + ".shared");
+                e.shared_limit = number(*shared, "limit", ff + ".shared");
+            }
+        }
+        out.layers.push_back(e);
+    }
+    d.num_layers = (int32_t)out.layers.size();
     return out;
 }
 
@@ -231,6 +326,8 @@ ModelSetup build_decoder(const EngineConfig& config, DecoderConfig (*read)(const
     }
     DecoderConfig dc = read(config.prefill_model_config(), shapes);
     efm_decoder_desc& d = dc.desc;
+    for (size_t i = 0; i < dc.decays.size(); ++i)
+        if (!dc.decays[i].empty()) dc.layers[i].linear_decay = dc.decays[i].data();
 
     const std::string compute = config.compute_dtype();
     if (compute != "bf16" && compute != "fp32") throw ConfigurationError("runtime.compute_dtype must be \"bf16\" or \"fp32\", got " + compute);
@@ -253,7 +350,7 @@ ModelSetup build_decoder(const EngineConfig& config, DecoderConfig (*read)(const
         states += 1 + (r.prefix_token_ids.empty() ? 0 : 1);
     }
     if (pages <= 0) throw ConfigurationError("kvcache declares neither requests nor pool_tokens");
-    const bool recurrent = std::any_of(dc.layers.begin(), dc.layers.end(), [](const efm_decoder_layer& l) { return l.mixer == EFM_MIXER_GENERAL_DELTA; });
+    const bool recurrent = std::any_of(dc.layers.begin(), dc.layers.end(), [](const efm_decoder_layer& l) { return l.mixer == EFM_MIXER_GENERAL_DELTA || l.mixer == EFM_MIXER_PARALLEL; });
     d.cache_pages = (int32_t)pages;
     d.state_slots = recurrent ? states : 0;
     d.max_slots = (int32_t)reqs.size() + live;
@@ -290,7 +387,7 @@ ModelSetup build_decoder(const EngineConfig& config, DecoderConfig (*read)(const
         for (int32_t i = 0; i < d.num_layers; ++i) {
             const efm_decoder_layer& l = dc.layers[i];
             const size_t times = d.loop_times > 1 && i >= d.loop_start && i < d.loop_stop ? d.loop_times : 1;
-            if (l.mixer == EFM_MIXER_ATTENTION) geo.token_bytes += times * l.kv_heads * (l.dim + l.vdim) * get_dtype_size(cache_dtype);
+            if (l.mixer == EFM_MIXER_ATTENTION || l.mixer == EFM_MIXER_PARALLEL) geo.token_bytes += times * l.kv_heads * (l.dim + l.vdim) * get_dtype_size(cache_dtype);
             if (l.mixer == EFM_MIXER_LATENT_ATTENTION) geo.token_bytes += times * (l.kv_rank + l.rot_dims) * get_dtype_size(cache_dtype);
         }
         setup.kv_manager = std::make_shared<KVManager>(reqs, geo, attention_type_from_string(config.kvcache_attention_type()), setup.device_id,
@@ -306,8 +403,11 @@ ModelSetup build_folizen(const EngineConfig& config) { return build_decoder(conf
 
 ModelSetup build_temuvik(const EngineConfig& config) { return build_decoder(config, temuvik_config); }
 
+ModelSetup build_vekolix(const EngineConfig& config) { return build_decoder(config, vekolix_config); }
+
 const ModelRegistrar kFolizen({"folizen", {"Folizen"}, build_folizen});
 const ModelRegistrar kTemuvik({"temuvik", {"Temuvik"}, build_temuvik});
+const ModelRegistrar kVekolix({"vekolix", {"Vekolix"}, build_vekolix});
 
 }  // namespace
 

@@ -4,10 +4,12 @@
 // cache / state update, attention or recurrence) | W_o | [norm + add] + W_up | [PolyNorm] + W_down | [norm + add] + token
 // input; what stands in brackets is the prologue of the kernel that follows it: three launches for a layer without a
 // feed-forward and token input, two more for a dense feed-forward, one more for the token input.  Latent attention adds
-// [query norm] + W_uq; routed experts are [norms + add] + router | [choice] + gate, up, silu | [weights] + down.
+// [query norm] + W_uq; routed experts are [norms + add] + router | [choice] + gate, up, gated unit | [weights] + down, a shared expert
+// among them.  Linear attention runs in the launch of the attention beside it, its norm and gate are a prologue of W_o.
 // Many rows: tensor-core GEMMs (bf16 operands) or fp32 FMAs (32-bit mode) between row kernels.
 #include "decoder.h"
 
+#include <cmath>
 #include <cstdlib>
 #include <type_traits>
 
@@ -17,6 +19,7 @@
 #include "../operators/experts.cuh"
 #include "../operators/gemm_tc.cuh"
 #include "../operators/latent_attention.cuh"
+#include "../operators/linear_attention.cuh"
 #include "../operators/token_side.cuh"
 #include "../operators/window_attention.cuh"
 #include "../operators/window_attention_tc.cuh"
@@ -58,14 +61,19 @@ void launch_gemv_ext(efm_b200_ctx& c, Launcher& L, const GemvParams& p) {
     // Logits publishes one maximum per block of a full grid; the others launch no idle blocks
     const int per = kGemvWarps / ks, need = (p.n_items + per - 1) / per;
     const int grid = EPI == Epi::Logits ? c.num_sms : std::min(c.num_sms, need);
-    const size_t smem = p.prologue == kProAddNorm || p.prologue == kProNorm ? gemv_ext_smem_bytes(p.K) : gemv_smem_bytes(p.K);
-    constexpr bool kExperts = EPI == Epi::Router || EPI == Epi::ExpertUp || EPI == Epi::ExpertDown || EPI == Epi::Store32Bias;
+    const bool two = p.prologue == kProAddNorm || p.prologue == kProNorm || p.prologue == kProAddTanh || p.prologue == kProMerge;
+    const size_t smem = two ? gemv_ext_smem_bytes(p.K) : gemv_smem_bytes(p.K);
+    constexpr bool kExperts = EPI == Epi::Router || EPI == Epi::ExpertUp || EPI == Epi::ExpertDown;
+    const int level = c.decoder->gemv_level();
+    auto run = [&](auto kernel) { L.launch(kernel, dim3(grid), dim3(kGemvThreads), smem, p, ks); };
     if constexpr (EPI == Epi::Router) {
         InOrder serial(L);
-        L.launch(gemv_kernel<EPI, 2>, dim3(grid), dim3(kGemvThreads), smem, p, ks);
-    } else if constexpr (kExperts) L.launch(gemv_kernel<EPI, 2>, dim3(grid), dim3(kGemvThreads), smem, p, ks);
-    else if constexpr (EPI == Epi::TokenGate) L.launch(gemv_kernel<EPI, 1>, dim3(grid), dim3(kGemvThreads), smem, p, ks);
-    else L.launch(c.decoder->input_norms() ? gemv_kernel<EPI, 2> : gemv_kernel<EPI, 1>, dim3(grid), dim3(kGemvThreads), smem, p, ks);
+        run(level == 3 ? gemv_kernel<EPI, 3> : gemv_kernel<EPI, 2>);
+    } else if constexpr (kExperts) run(level == 3 ? gemv_kernel<EPI, 3> : gemv_kernel<EPI, 2>);
+    else if constexpr (EPI == Epi::Store32Bias) run(gemv_kernel<EPI, 2>);
+    else if constexpr (EPI == Epi::TokenGate) run(gemv_kernel<EPI, 1>);
+    else if constexpr (EPI == Epi::Relu2) run(gemv_kernel<EPI, 3>);
+    else run(level == 3 ? gemv_kernel<EPI, 3> : level == 2 ? gemv_kernel<EPI, 2> : gemv_kernel<EPI, 1>);
 }
 
 template <Epi EPI>
@@ -83,10 +91,18 @@ void gemv_ext(efm_b200_ctx& c, Launcher& L, const DecLinear& w, GemvParams& p) {
 
 // Input of a product that reads the residual stream: embedding row (first layer) or stream + pending output; with `pre` the
 // product reads the norm of it.
-void stream_input(efm_b200_ctx& c, GemvParams& p, Pending& pend, bool first, const __nv_bfloat16* pre) {
+void stream_input(efm_b200_ctx& c, GemvParams& p, Pending& pend, bool first, const DecNorm& pre) {
     float* bufs[2] = {c.resid_d, c.resid_d2};
+    const bool tanh = c.decoder->tanh_norms();
     p.k_true = c.decoder->W;
-    p.norm2_w = pre;
+    if (tanh) {
+        p.norm_w = pre.w;
+        p.norm_b = pre.b;
+        p.norm_alpha = pre.alpha;
+        p.add_mult = c.decoder->d.residual_mult;
+    } else {
+        p.norm2_w = pre.w;
+    }
     if (first) {
         p.prologue = kProEmbed;
         p.embed_table = c.embed;
@@ -95,10 +111,10 @@ void stream_input(efm_b200_ctx& c, GemvParams& p, Pending& pend, bool first, con
         return;
     }
     if (pend.y == nullptr) { p.prologue = kProPlain; p.xf = bufs[pend.flip]; return; }
-    p.prologue = kProAddNorm;
+    p.prologue = tanh ? kProAddTanh : kProAddNorm;
     p.xr = bufs[pend.flip];
     p.addend = pend.y;
-    p.norm_w = pend.norm;
+    if (!tanh) p.norm_w = pend.norm;
     pend.flip ^= 1;                      // other blocks still read the old row: the new one goes to the other buffer
     p.resid_out = bufs[pend.flip];
     pend.y = nullptr;
@@ -106,13 +122,14 @@ void stream_input(efm_b200_ctx& c, GemvParams& p, Pending& pend, bool first, con
 
 RotShape rot_shape(const DecoderLayer& l) {
     const int kind = l.d.rot_kind == EFM_ROT_HALF ? kRotHalf : l.d.rot_kind == EFM_ROT_PAIRS ? kRotPairs : kRotNone;
-    return RotShape{kind, kind == kRotNone ? 0 : l.d.rot_dims, l.inv_freq};
+    return RotShape{kind, kind == kRotNone ? 0 : l.d.rot_dims, l.inv_freq, l.d.rot_factor > 0.f ? 0.1f * std::log(l.d.rot_factor) + 1.0f : 1.0f};
 }
 WindowAttnShape attn_shape(const DecoderModel& m, const DecoderLayer& l) {
     WindowAttnShape s{};
     s.H = l.d.heads; s.G = l.d.kv_heads; s.D = l.d.dim; s.Dv = l.d.vdim; s.Dp = l.Dp; s.Vp = l.Vp;
     s.window = l.d.window; s.keep = l.d.window > 0 ? l.d.keep_first : 0;
     s.bias = l.d.distance_bias; s.scale = l.d.scale; s.eps = m.d.norm_eps;
+    s.qk_norm = l.d.qk_norm != EFM_QK_NORM_NONE; s.out_scale = l.linear() ? l.d.mix_scale : 1.0f;
     s.q_norm = l.q_norm; s.k_norm = l.k_norm; s.temp = l.temp;
     s.rot = rot_shape(l);
     return s;
@@ -128,7 +145,17 @@ LatentShape latent_shape(const DecoderModel& m, const DecoderLayer& l) {
     s.gate = l.d.out_gate;
     return s;
 }
-RouteShape route_shape(const DecoderLayer& l) { return RouteShape{l.d.experts, l.d.expert_top, l.d.expert_groups, l.d.expert_groups_kept}; }
+LinearShape linear_shape(const DecoderModel& m, const DecoderLayer& l) {
+    LinearShape s{};
+    s.heads = l.d.linear_heads; s.D = l.d.linear_dim; s.Dv = l.d.linear_vdim; s.Vp = l.lin_vp;
+    const int qk = round_up(s.heads * s.D, 8), v = round_up(s.heads * s.Dv, 8);
+    s.off_q = l.lin_in; s.off_k = l.lin_in + qk; s.off_v = l.lin_in + 2 * qk; s.off_g = l.lin_in + 2 * qk + v;
+    s.ld = l.in.Np; s.powers = l.lin_powers; s.norm = l.mix_norm; s.eps = m.d.norm_eps; s.scale = l.d.linear_scale;
+    return s;
+}
+RouteShape route_shape(const DecoderLayer& l) {
+    return RouteShape{l.d.experts, l.d.expert_top, l.d.expert_groups, l.d.expert_groups_kept, l.d.expert_score == EFM_SCORE_SIGMOID, l.d.shared_ff > 0};
+}
 DeltaShape delta_shape(const DecoderModel& m, const DecoderLayer& l) {
     DeltaShape s{};
     s.heads = l.d.heads; s.D = l.d.dim; s.Dp = round_up(l.d.dim, 32); s.rank = l.d.decay_rank; s.ld = l.in.Np;
@@ -138,11 +165,12 @@ DeltaShape delta_shape(const DecoderModel& m, const DecoderLayer& l) {
 
 template <typename TC, int VM, bool ROT>
 void launch_attn_decode_v(Launcher& L, const WindowDecodeParams<TC>& p, int cluster) {
-    const int hb = (p.s.H / p.s.G + wd::kHeads - 1) / wd::kHeads;
+    const int hb = (p.s.H / p.s.G + wd::kHeads - 1) / wd::kHeads, lin = (p.lin.units + cluster - 1) / cluster;
     L.cluster_x = cluster;
     const bool pdl = L.pdl;
     L.pdl = pdl && !ROT;                                               // see InOrder
-    L.launch(window_attention_decode_kernel<TC, VM, ROT>, dim3(cluster, p.s.G * hb), dim3(wd::kThreads), sizeof(wd::Smem<VM>), p);
+    L.launch(lin > 0 ? window_attention_decode_kernel<TC, VM, ROT, true> : window_attention_decode_kernel<TC, VM, ROT, false>, dim3(cluster, p.s.G * hb + lin),
+             dim3(wd::kThreads), sizeof(wd::Smem<VM>), p);
     L.pdl = pdl;
 }
 template <typename TC>
@@ -158,6 +186,12 @@ void launch_attn_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, con
     p.state = c.state;
     p.out = m.d_mix;
     p.early = early ? 1 : 0;
+    if (l.linear()) {
+        p.lin.s = linear_shape(m, l);
+        p.lin.pool = m.state_pool + (size_t)slot.state_slot * m.state_stride + run.state_off;
+        p.lin.out = m.d_mix + l.lin_mix;
+        p.lin.units = ln::decode_units(p.lin.s);
+    }
     // one block per 64 keys of the visible range, up to the cluster width (a power of two)
     int pages = slot.n_pages;
     if (l.d.window > 0) pages = std::min(pages, (l.d.window + p.s.keep + kPageTokens - 1) / kPageTokens);
@@ -278,7 +312,7 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
             else gemv_ext<Epi::Store32>(c, L, l.in, p);
             if (i > 0) tap((int)i - 1);
         }
-        if (l.d.mixer == EFM_MIXER_ATTENTION) {
+        if (l.attention()) {
             if (m.f32) launch_attn_decode<float>(c, L, l, run, slot, early);
             else launch_attn_decode<__nv_bfloat16>(c, L, l, run, slot, early);
         } else if (l.d.mixer == EFM_MIXER_LATENT_ATTENTION) {
@@ -298,6 +332,14 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
             GemvParams p{};
             p.prologue = kProPlain;
             p.xf = m.d_mix;
+            if (l.linear()) {
+                p.prologue = kProMerge;
+                p.merge0 = l.lin_mix;
+                p.merge_gate = m.d_in + linear_shape(m, l).off_g;
+                p.merge_scale = l.d.linear_scale;
+                p.norm_w = l.mix_norm;
+                p.k_true = l.d.linear_heads * l.d.linear_vdim;
+            }
             p.out_f = m.d_y;
             gemv_ext<Epi::Store32>(c, L, l.out, p);
             pend.y = m.d_y;
@@ -318,7 +360,14 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
             p.W = l.expert_in.w;
             p.xf = m.d_h;
             p.K = l.expert_in.Kp;
-            p.n_items = l.d.expert_top * l.d.expert_ff;
+            p.n_items = l.d.expert_top * l.d.expert_ff + l.d.shared_ff;
+            p.glu = l.d.expert_glu == EFM_GLU_CLAMPED ? kGluClamped : kGluSilu;
+            p.weight_input = l.d.expert_weight_input;
+            p.limit = l.d.expert_limit;
+            p.shared_limit = l.d.shared_limit;
+            p.shared_ff = l.d.shared_ff;
+            p.shared_ffp = l.sfp;
+            p.W2 = l.shared_in.w;
             p.N = 2 * p.n_items;
             p.state = c.state;
             p.route = route_shape(l);
@@ -331,8 +380,9 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
             launch_gemv_ext<Epi::ExpertUp>(c, L, p);
             GemvParams q = p;
             q.W = l.expert_out.w;
+            q.W2 = l.shared_out.w;
             q.xf = m.d_act;
-            q.K = l.d.expert_top * l.ffp;
+            q.K = l.d.expert_top * l.ffp + l.sfp;
             q.n_items = m.Wp / 2;
             q.N = m.W;
             q.expert_rows = m.Wp;
@@ -344,9 +394,11 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
             GemvParams p{};
             stream_input(c, p, pend, false, l.pre2);
             p.out_f = m.d_ff;
-            gemv_ext<Epi::Store32>(c, L, l.up, p);
+            const bool poly = l.d.ff_act == EFM_ACT_POLYNORM;
+            if (poly) gemv_ext<Epi::Store32>(c, L, l.up, p);
+            else gemv_ext<Epi::Relu2>(c, L, l.up, p);
             GemvParams q{};
-            q.prologue = kProPolyNorm;
+            q.prologue = poly ? kProPolyNorm : kProPlain;
             q.xf = m.d_ff;
             q.k_true = l.d.ff;
             q.poly = l.act;
@@ -357,7 +409,7 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
         }
         if (m.d.side_dim > 0) {
             GemvParams p{};
-            stream_input(c, p, pend, false, nullptr);
+            stream_input(c, p, pend, false, DecNorm{});
             p.out_f = m.d_gate;
             p.gate_table = m.side_embed;
             p.gate_ld = m.d.side_dim * m.d.num_layers;
@@ -395,6 +447,8 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
         GemvParams p{};
         stream_input(c, p, pend, false, m.final_norm);
         p.logits = c.logits;
+        p.logit_scale = m.d.logit_scale;
+        p.logit_softcap = m.d.logit_softcap;
         p.part_val = c.part_val;
         p.part_idx = c.part_idx;
         gemv_ext<Epi::Logits>(c, L, m.head, p);
@@ -422,12 +476,12 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
 // ---- many rows ---------------------------------------------------------------------------------------------------
 int decoder_tc_tile_rows() { return wt::BM; }
 int decoder_simt_tile_rows() { return wa::QT; }
-// bf16 heads of at most 128 channels whose visible pages fit the kernel's page list
+// bf16 heads of at most 128 key channels whose visible pages fit the kernel's page list
 bool decoder_layer_tc(const DecoderModel& m, const DecoderLayer& l) {
     static const bool off = [] { const char* e = std::getenv("EFM_B200_ATTN_TC"); return e != nullptr && e[0] == '0'; }();
     int pages = m.d.cache_pages;
     if (l.d.window > 0) pages = std::min(pages, (l.d.window + wt::BM) / kPageTokens + 2 + (l.d.keep_first + kPageTokens - 1) / kPageTokens);
-    return !off && !m.f32 && l.Dp <= 128 && l.Vp <= 128 && l.Rc <= 64 && pages <= wt::kMaxTiles;
+    return !off && !m.f32 && l.Dp <= 128 && l.Vp <= 256 && l.Rc <= 64 && pages <= wt::kMaxTiles;
 }
 
 namespace {
@@ -462,7 +516,7 @@ void launch_delta_scan(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, cons
 template <int DP, int VP, int RP, bool KEEP>
 void launch_attention_tc_v(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const WindowAttnShape& s, const WindowTcMaps& maps, const RowPlan& plan,
                            const RowTile* list, int n) {
-    L.launch(window_attention_tc_kernel<DP, VP, RP, KEEP>, dim3(n, s.H), dim3(wt::kThreads), wt::Cfg<DP, VP, RP>::SMEM, maps, static_cast<__nv_bfloat16*>(c.decoder->mix),
+    L.launch(window_attention_tc_kernel<DP, VP, RP, KEEP>, dim3(n, s.H, (s.Vp + VP - 1) / VP), dim3(wt::kThreads), wt::Cfg<DP, VP, RP>::SMEM, maps, static_cast<__nv_bfloat16*>(c.decoder->mix),
              l.mix_wp, s, plan, list, RP > 0 ? 1 : 0, &c.state->error);
 }
 template <int RP, bool KEEP = false>
@@ -510,8 +564,8 @@ void launch_latent_tc(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const
     launch_gemm_epi(L, GemmEpi::Bf16Bias, g, &c.state->error);
     WindowAttnShape s{};
     s.H = s.G = z.H; s.D = z.D; s.Dv = z.Dv; s.Dp = z.Dp; s.Vp = z.Vp;
-    s.window = z.window; s.scale = z.scale; s.eps = z.eps; s.sink = z.sink;
-    if (z.gate) { s.gate = static_cast<const __nv_bfloat16*>(m.proj_a) + z.off_gate(); s.gate_ld = l.in.Np; }
+    s.window = z.window; s.scale = z.scale; s.eps = z.eps; s.sink = z.sink; s.out_scale = 1.0f;
+    if (z.gate) { s.gate = static_cast<const __nv_bfloat16*>(m.proj_a) + z.off_gate(); s.gate_ld = l.in.Np; s.gate_heads = z.gate == EFM_GATE_HEADS; }
     const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(m.q);
     WindowTcMaps maps;
     const int qh = z.Dp + z.Rc;
@@ -536,12 +590,42 @@ void launch_delta_chunks(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, co
              m.o, l.mix_wp, m.state_pool, m.state_stride, run.state_off, s, plan);
 }
 
+// Linear attention of rows whose projections are in proj_a, into its columns of the mixer output.
+template <typename TA>
+void linear_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const RowPlan& plan) {
+    DecoderModel& m = *c.decoder;
+    const LinearShape s = linear_shape(m, l);
+    const TA* proj = static_cast<const TA*>(m.proj_a);
+    const int chunks = max_chunks(plan, kLinearChunk), ld_o = round_up(s.width(), 8);
+    auto chunk = [&](auto rm, auto rn) {
+        constexpr int RM = decltype(rm)::value, RN = decltype(rn)::value;
+        L.launch(linear_chunk_rows_kernel<TA, RM, RN>, dim3(chunks, s.heads, ((s.D + 16 * RM - 1) / (16 * RM)) * ((s.Vp + 16 * RN - 1) / (16 * RN))), dim3(ln::kThreads),
+                 ln::chunk_smem_bytes(RM, RN), proj, m.lin_ws, s, plan);
+    };
+    auto attend = [&](auto rn) {
+        constexpr int RN = decltype(rn)::value;
+        L.launch(linear_attend_rows_kernel<TA, RN>, dim3(chunks, s.heads, (s.Dv + 16 * RN - 1) / (16 * RN)), dim3(ln::kThreads), ln::attend_smem_bytes(s.D, RN), proj,
+                 (const float*)m.lin_ws, m.o, ld_o, s, plan);
+    };
+    const std::integral_constant<int, 4> k4{};
+    const std::integral_constant<int, 8> k8{};
+    if (s.D <= 64) { if (s.Dv <= 64) chunk(k4, k4); else chunk(k4, k8); }
+    else if (s.Dv <= 64) chunk(k8, k4);
+    else chunk(k8, k8);
+    L.launch(linear_chain_rows_kernel, dim3((unsigned)((s.heads * s.head_floats() + 1023) / 1024), plan.n_entries), dim3(256), 0, m.lin_ws, m.state_pool, m.state_stride,
+             run.state_off, s, plan);
+    if (s.Dv <= 64) attend(k4); else attend(k8);
+    L.launch(linear_output_rows_kernel<TA>, dim3(plan.rows), dim3(256), 0, (const float*)m.o, ld_o, proj, static_cast<TA*>(m.mix) + l.lin_mix, l.mix_wp,
+             l.mix_wp - l.lin_mix, s);
+}
+
 // TA: activation and cache type of the pass
 template <typename TA>
 void attention_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const void* x, const RowPlan& plan, const RowTiles& tiles) {
     DecoderModel& m = *c.decoder;
     const WindowAttnShape s = attn_shape(m, l);
     linear_act(c, L, l.in, x, m.proj_a, plan.rows);
+    if (l.linear()) linear_rows<TA>(c, L, l, run, plan);
     TA* kp = static_cast<TA*>(run.k_pool);
     TA* vp = static_cast<TA*>(run.v_pool);
     int lanes = 8;                                                  // 8 channels each: at most 256 (padded) channels a head
@@ -607,7 +691,7 @@ SumOf<TA> expert_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const
     const RouteShape r = route_shape(l);
     linear_f32(c, L, l.router, h, m.route_logits, T);
     L.launch(expert_route_rows_kernel, dim3((T + 7) / 8), dim3(256), 0, (const float*)m.route_logits, l.router.Np, T, r, m.ex);
-    L.launch(expert_gather_rows_kernel<TA>, dim3(T), dim3(128), 0, static_cast<const TA*>(h), static_cast<TA*>(m.ex_in), m.Wp, r, m.ex);
+    L.launch(l.d.expert_weight_input ? expert_gather_rows_kernel<TA, true> : expert_gather_rows_kernel<TA, false>, dim3(T), dim3(128), 0, static_cast<const TA*>(h), static_cast<TA*>(m.ex_in), m.Wp, r, m.ex);
     // tiles in use at most: every row tile but the last of an expert is full
     const int64_t picks = (int64_t)T * r.top;
     const int max_rows = (int)std::min<int64_t>(m.ex_rows, (picks / kExpertTile + std::min<int64_t>(picks, r.experts)) * kExpertTile);
@@ -617,9 +701,16 @@ SumOf<TA> expert_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const
                      (const __nv_bfloat16*)nullptr, RowGroups{m.ex.tile, m.ex.n_tiles, n});
         };
         product(l.expert_in, 2 * l.ffp, static_cast<const float*>(m.ex_in), m.ex_gu);
-        L.launch(silu_mul_rows_kernel, dim3(max_rows / kExpertTile), dim3(256), 0, (const float*)m.ex_gu, static_cast<float*>(m.ex_act), l.ffp,
-                 (const int32_t*)m.ex.n_tiles);
+        const int glu = l.d.expert_glu == EFM_GLU_CLAMPED ? kGluClamped : kGluSilu;
+        L.launch(glu_rows_kernel, dim3(max_rows / kExpertTile), dim3(256), 0, (const float*)m.ex_gu, static_cast<float*>(m.ex_act), max_rows, l.ffp,
+                 (const int32_t*)m.ex.n_tiles, glu, l.d.expert_limit);
         product(l.expert_out, m.Wp, static_cast<const float*>(m.ex_act), static_cast<float*>(m.ex_y));
+        if (l.d.shared_ff > 0) {
+            linear_f32(c, L, l.shared_in, h, m.sh_gu, T);
+            L.launch(glu_rows_kernel, dim3((T + kExpertTile - 1) / kExpertTile), dim3(256), 0, (const float*)m.sh_gu, static_cast<float*>(m.sh_act), T, l.sfp,
+                     (const int32_t*)nullptr, glu, l.d.shared_limit);
+            linear_f32(c, L, l.shared_out, m.sh_act, static_cast<float*>(m.sh_y), T);
+        }
     } else {
         auto product = [&](const DecLinear& w, int n, GemmEpi epi, const void* a, void* out) {
             GemmParams g{static_cast<const __nv_bfloat16*>(a), w.w, nullptr, static_cast<__nv_bfloat16*>(out), nullptr, max_rows, n, w.Kp};
@@ -627,12 +718,21 @@ SumOf<TA> expert_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const
             g.group_tiles = m.ex.n_tiles;
             g.group_rows = n;
             g.group_all = r.experts * n;
+            g.limit = l.d.expert_limit;
             launch_gemm_epi(L, epi, g, &c.state->error);
         };
-        product(l.expert_in, 2 * l.ffp, GemmEpi::SwiGlu, m.ex_in, m.ex_act);
+        const GemmEpi glu = l.d.expert_glu == EFM_GLU_CLAMPED ? GemmEpi::ClampGlu : GemmEpi::SwiGlu;
+        product(l.expert_in, 2 * l.ffp, glu, m.ex_in, m.ex_act);
         product(l.expert_out, m.Wp, GemmEpi::Bf16Bias, m.ex_act, m.ex_y);
+        if (l.d.shared_ff > 0) {
+            GemmParams g{static_cast<const __nv_bfloat16*>(h), l.shared_in.w, nullptr, static_cast<__nv_bfloat16*>(m.sh_act), nullptr, T, l.shared_in.Np, l.shared_in.Kp};
+            g.limit = l.d.shared_limit;
+            launch_gemm_epi(L, glu, g, &c.state->error);
+            linear_act(c, L, l.shared_out, m.sh_act, m.sh_y, T);
+        }
     }
-    return SumOf<TA>{static_cast<const TA*>(m.ex_y), m.ex.place, m.ex.weight, r.top, m.ex.count, r.experts};
+    return SumOf<TA>{static_cast<const TA*>(m.ex_y), m.ex.place, m.ex.weight, r.top, m.ex.count, r.experts, l.d.expert_weight_input,
+                     l.d.shared_ff > 0 ? static_cast<const TA*>(m.sh_y) : nullptr, m.ex.shared};
 }
 
 template <typename TA>
@@ -677,8 +777,14 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
     TA* xa = static_cast<TA*>(m.xa);                            // null: 32-bit mode without input norms reads the stream itself
     const void* xin = xa != nullptr ? (const void*)xa : c.resid;
     // the stream takes a sublayer's normed output; xa becomes the next sublayer's input
-    auto add_norm = [&](const float* y, const __nv_bfloat16* w, const __nv_bfloat16* pre, const SumOf<TA>& sum = SumOf<TA>{}) {
+    auto add_norm = [&](const float* y, const __nv_bfloat16* w, const DecNorm& norm, const SumOf<TA>& sum = SumOf<TA>{}) {
         const bool experts = sum.place != nullptr;
+        const __nv_bfloat16* pre = norm.w;
+        if (m.tanh_norms()) {
+            L.launch(experts ? add_tanh_rows_kernel<TA, true> : add_tanh_rows_kernel<TA, false>, dim3((m.Wp + 1023) / 1024, T), dim3(256), 0, c.resid, y,
+                     m.d.residual_mult, xa, norm.w, norm.b, norm.alpha, m.Wp, sum);
+            return;
+        }
         L.launch(pre != nullptr ? (experts ? add_norm_rows_kernel<TA, true, true> : add_norm_rows_kernel<TA, true, false>)
                                 : (experts ? add_norm_rows_kernel<TA, false, true> : add_norm_rows_kernel<TA, false, false>),
                  dim3(T), dim3(256), 0, c.resid, y, w, xa, pre, m.W, m.Wp, m.d.norm_eps, sum);
@@ -688,8 +794,8 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
     for (size_t i = 0; i < m.runs.size(); ++i) {
         const DecoderRun& run = m.runs[i];
         const DecoderLayer& l = m.layers[run.layer];
-        const __nv_bfloat16* next = i + 1 < m.runs.size() ? m.layers[m.runs[i + 1].layer].pre1 : nullptr;
-        if (l.d.mixer == EFM_MIXER_ATTENTION) attention_rows<TA>(c, L, l, run, xin, plan, tiles);
+        const DecNorm next = i + 1 < m.runs.size() ? m.layers[m.runs[i + 1].layer].pre1 : DecNorm{};
+        if (l.attention()) attention_rows<TA>(c, L, l, run, xin, plan, tiles);
         else if (l.d.mixer == EFM_MIXER_LATENT_ATTENTION) latent_rows<TA>(c, L, l, run, xin, plan, tiles);
         else delta_rows<TA>(c, L, l, run, xin, plan);
         linear_f32(c, L, l.out, m.mix, m.y, T);
@@ -697,10 +803,20 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
         if (l.moe()) {
             add_norm(nullptr, l.post2, next, expert_rows<TA>(c, L, l, xin, T));
         } else if (l.d.ff > 0) {
-            linear_act(c, L, l.up, xin, m.ff, T);
-            L.launch(poly_norm_rows_kernel<TA>, dim3(T), dim3(256), 0, static_cast<const TA*>(m.ff), static_cast<TA*>(m.ff2), (const __nv_bfloat16*)l.act, l.d.ff,
-                     l.down.Kp, m.d.norm_eps);
-            linear_f32(c, L, l.down, m.ff2, m.y, T);
+            const bool poly = l.d.ff_act == EFM_ACT_POLYNORM;
+            if (poly) {
+                linear_act(c, L, l.up, xin, m.ff, T);
+                L.launch(poly_norm_rows_kernel<TA>, dim3(T), dim3(256), 0, static_cast<const TA*>(m.ff), static_cast<TA*>(m.ff2), (const __nv_bfloat16*)l.act, l.d.ff,
+                         l.down.Kp, m.d.norm_eps);
+            } else if (m.f32) {
+                linear_f32(c, L, l.up, xin, static_cast<float*>(m.ff), T);
+                const size_t n = (size_t)T * l.up.Np;
+                L.launch(relu2_kernel, dim3((unsigned)((n + 1023) / 1024)), dim3(256), 0, static_cast<float*>(m.ff), n);
+            } else {
+                GemmParams g{static_cast<const __nv_bfloat16*>(xin), l.up.w, nullptr, static_cast<__nv_bfloat16*>(m.ff), nullptr, T, l.up.Np, l.up.Kp};
+                launch_gemm_epi(L, GemmEpi::Bf16Relu2, g, &c.state->error);
+            }
+            linear_f32(c, L, l.down, poly ? m.ff2 : m.ff, m.y, T);
             add_norm(m.y, l.post2, next);
         }
         if (m.d.side_dim > 0) {
@@ -708,7 +824,7 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
             L.launch(token_gate_rows_kernel<TA>, dim3(T), dim3(128), 0, (const float*)m.side_f, ids, (const __nv_bfloat16*)m.side_embed,
                      m.d.side_dim * m.d.num_layers, run.layer * m.d.side_dim, c.d.vocab, static_cast<TA*>(m.side_a), m.d.side_dim, m.side_p);
             linear_f32(c, L, l.proj, m.side_a, m.y, T);
-            add_norm(m.y, l.side_norm, nullptr);
+            add_norm(m.y, l.side_norm, DecNorm{});
         }
         if (m.tap != nullptr && m.tap_row0 + T <= m.tap_rows && L.err == cudaSuccess)
             L.err = cudaMemcpyAsync(m.tap + ((size_t)i * m.tap_rows + m.tap_row0) * m.Wp, c.resid, (size_t)T * m.Wp * 4, cudaMemcpyDeviceToDevice, L.stream);
@@ -729,13 +845,20 @@ void decoder_rows_logits(efm_b200_ctx& c, const int32_t* rows, int n, Launcher& 
     DecoderModel& m = *c.decoder;
     const bool pdl = L.pdl;
     L.pdl = false;
-    if (m.f32)
-        L.launch(gather_norm_rows_kernel<float>, dim3(n), dim3(256), 0, (const float*)c.resid, rows, (const __nv_bfloat16*)m.final_norm,
-                 static_cast<float*>(m.head_a), m.W, m.Wp, m.d.norm_eps);
-    else
-        L.launch(gather_norm_rows_kernel<__nv_bfloat16>, dim3(n), dim3(256), 0, (const float*)c.resid, rows, (const __nv_bfloat16*)m.final_norm,
-                 static_cast<__nv_bfloat16*>(m.head_a), m.W, m.Wp, m.d.norm_eps);
+    auto gather = [&](auto* out) {
+        using TA = std::remove_pointer_t<decltype(out)>;
+        const DecNorm& f = m.final_norm;
+        if (m.tanh_norms())
+            L.launch(gather_tanh_rows_kernel<TA>, dim3(n), dim3(256), 0, (const float*)c.resid, rows, (const __nv_bfloat16*)f.w, (const __nv_bfloat16*)f.b,
+                     (const __nv_bfloat16*)f.alpha, out, m.Wp);
+        else
+            L.launch(gather_norm_rows_kernel<TA>, dim3(n), dim3(256), 0, (const float*)c.resid, rows, (const __nv_bfloat16*)f.w, out, m.W, m.Wp, m.d.norm_eps);
+    };
+    if (m.f32) gather(static_cast<float*>(m.head_a));
+    else gather(static_cast<__nv_bfloat16*>(m.head_a));
     linear_f32(c, L, m.head, m.head_a, m.logits_rows, n);
+    if (m.d.logit_softcap > 0.f || m.d.logit_scale != 1.0f)
+        L.launch(cap_logits_rows_kernel, dim3((m.d.vocab + 255) / 256, n), dim3(256), 0, m.logits_rows, m.d.vocab, m.head.Np, m.d.logit_scale, m.d.logit_softcap);
     L.pdl = pdl;
 }
 
@@ -745,11 +868,12 @@ template <typename K>
 cudaError_t smem_attr(K kernel, size_t bytes) { return cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes); }
 
 // widest cluster the decode attention kernel can be placed with
-template <typename TC, int VM, bool ROT>
-cudaError_t fit_cluster(int& width) {
-    cudaError_t e = smem_attr(window_attention_decode_kernel<TC, VM, ROT>, sizeof(wd::Smem<VM>));
+template <typename TC, int VM, bool ROT, bool LIN>
+cudaError_t fit_cluster_v(int& width) {
+    const auto kernel = window_attention_decode_kernel<TC, VM, ROT, LIN>;
+    cudaError_t e = smem_attr(kernel, sizeof(wd::Smem<VM>));
     if (e != cudaSuccess) return e;
-    const bool wide = cudaFuncSetAttribute(window_attention_decode_kernel<TC, VM, ROT>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess;
+    const bool wide = cudaFuncSetAttribute(kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) == cudaSuccess;
     int cs = wide ? 16 : 8;
     for (; cs > 1; cs >>= 1) {
         cudaLaunchConfig_t cfg = {};
@@ -763,11 +887,16 @@ cudaError_t fit_cluster(int& width) {
         cfg.attrs = &at;
         cfg.numAttrs = 1;
         int n = 0;
-        if (cudaOccupancyMaxActiveClusters(&n, window_attention_decode_kernel<TC, VM, ROT>, &cfg) == cudaSuccess && n >= 1) break;
+        if (cudaOccupancyMaxActiveClusters(&n, kernel, &cfg) == cudaSuccess && n >= 1) break;
     }
     (void)cudaGetLastError();
     width = std::min(width, cs);
     return cudaSuccess;
+}
+template <typename TC, int VM, bool ROT>
+cudaError_t fit_cluster(int& width) {
+    const cudaError_t e = fit_cluster_v<TC, VM, ROT, false>(width);
+    return e == cudaSuccess ? fit_cluster_v<TC, VM, ROT, true>(width) : e;
 }
 }  // namespace
 
@@ -777,6 +906,10 @@ size_t decoder_delta_pack_floats(int heads, int dim, int rows, int entries) {
     size_t n = (size_t)rows * heads * kDeltaParts * Dp;
     if (Dp <= 128) n = std::max(n, (size_t)(rows / dc::C + 1 + entries) * heads * dc::pack_floats(Dp));
     return n;
+}
+
+size_t decoder_linear_ws_floats(const DecoderLayer& l, int rows, int entries) {
+    return (size_t)(rows / kLinearChunk + 1 + entries) * l.d.linear_heads * l.d.linear_dim * l.lin_vp;
 }
 
 // Widest cluster the one-launch token input fits; 1: two products instead.
@@ -861,6 +994,18 @@ cudaError_t configure_decoder(DecoderModel& m) {
     auto gemv_attr = [&](auto... kernels) { ((e = e == cudaSuccess ? smem_attr(kernels, gv) : e), ...); };
     gemv_attr(gemv_kernel<Epi::Store32, 1>, gemv_kernel<Epi::TokenGate, 1>, gemv_kernel<Epi::Logits, 1>, gemv_kernel<Epi::Store32, 2>, gemv_kernel<Epi::Logits, 2>,
               gemv_kernel<Epi::Store32Bias, 2>, gemv_kernel<Epi::Router, 2>, gemv_kernel<Epi::ExpertUp, 2>, gemv_kernel<Epi::ExpertDown, 2>);
+    gemv_attr(gemv_kernel<Epi::Store32, 3>, gemv_kernel<Epi::Logits, 3>, gemv_kernel<Epi::Relu2, 3>, gemv_kernel<Epi::Router, 3>, gemv_kernel<Epi::ExpertUp, 3>,
+              gemv_kernel<Epi::ExpertDown, 3>);
+    auto linear_attr = [&](auto type) {
+        using T = decltype(type);
+        auto chunk = [&](auto kernel, int rm, int rn) { if (e == cudaSuccess) e = smem_attr(kernel, ln::chunk_smem_bytes(rm, rn)); };
+        chunk(linear_chunk_rows_kernel<T, 4, 4>, 4, 4); chunk(linear_chunk_rows_kernel<T, 4, 8>, 4, 8);
+        chunk(linear_chunk_rows_kernel<T, 8, 4>, 8, 4); chunk(linear_chunk_rows_kernel<T, 8, 8>, 8, 8);
+        if (e == cudaSuccess) e = smem_attr(linear_attend_rows_kernel<T, 4>, ln::attend_smem_bytes(256, 4));
+        if (e == cudaSuccess) e = smem_attr(linear_attend_rows_kernel<T, 8>, ln::attend_smem_bytes(256, 8));
+    };
+    linear_attr(float());
+    linear_attr(__nv_bfloat16());
     const size_t rows = wa::rows_smem_bytes(256, 256);
     if (e == cudaSuccess) e = smem_attr(window_attention_rows_kernel<float, float, float>, rows);
     if (e == cudaSuccess) e = smem_attr(window_attention_rows_kernel<__nv_bfloat16, __nv_bfloat16, __nv_bfloat16>, rows);

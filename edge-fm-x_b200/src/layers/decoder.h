@@ -1,6 +1,6 @@
-// Layered decoder: a list of layers, each with its own mixer (attention | latent attention | generalised delta rule) and an
-// optional feed-forward (dense | routed experts), sublayer outputs (and, sandwich layout, inputs) normalised, optional
-// per-layer token input; a span of layers may run several times.  Weights, buffers and launch sequences (definitions in
+// Layered decoder: a list of layers, each with its own mixer (attention | latent attention | generalised delta rule | attention and
+// linear attention side by side) and an optional feed-forward (dense | routed experts), sublayer outputs (and, sandwich layout,
+// inputs; or the inputs alone, elementwise) normalised, optional per-layer token input; a span of layers may run several times.  Weights, buffers and launch sequences (definitions in
 // decoder.cu); the C ABI side is backends/b200/decoder_b200.cu.
 #pragma once
 #include <algorithm>
@@ -24,15 +24,20 @@ struct DecLinear {
     __nv_bfloat16* bias = nullptr;        // [Np] or null
 };
 
+// Weight of an RMS norm; with b and alpha tanh(alpha x) w + b.
+struct DecNorm { __nv_bfloat16 *w = nullptr, *b = nullptr, *alpha = nullptr; };
+
 struct DecoderLayer {
     efm_decoder_layer d{};
     int Dp = 0, Vp = 0;                   // attention: padded channels of a cache row; latent: padded head channels
-    int mix_w = 0, mix_wp = 0;            // mixer output width (heads * value channels), padded
-    DecLinear in;                         // attention: q | k | v; latent: dq | c | r | g, each padded to 8; delta: r | k | v | g | a | w1
-    DecLinear out;                        // W_o
+    int mix_w = 0, mix_wp = 0;            // mixer output width (heads * value channels; parallel: both halves), padded
+    DecLinear in;                         // attention: q | k | v; latent: dq | c | r | g, each padded to 8; delta: r | k | v | g | a | w1;
+                                          // parallel: attention's, then q | k | v | g of linear attention, each padded to 8
+    DecLinear out;                        // W_o (parallel: the two side by side)
     DecLinear w2;                         // delta: decay projection
     DecLinear up, down, gate, proj;       // dense feed-forward; token side
-    __nv_bfloat16 *pre1 = nullptr, *pre2 = nullptr, *post1 = nullptr, *post2 = nullptr, *side_norm = nullptr, *act = nullptr;
+    DecNorm pre1, pre2;
+    __nv_bfloat16 *post1 = nullptr, *post2 = nullptr, *side_norm = nullptr, *act = nullptr;
     __nv_bfloat16 *q_norm = nullptr, *k_norm = nullptr, *temp = nullptr;
     __nv_bfloat16 *w0 = nullptr, *a_bias = nullptr, *mix_norm = nullptr;
     float* inv_freq = nullptr;            // rotation: [rot_dims / 2]
@@ -41,9 +46,16 @@ struct DecoderLayer {
     DecLinear uq, ukv;                    // [heads][Dp + Rc] rows; [heads][Dp] key rows, then [heads][Vp] value rows
     __nv_bfloat16* sink = nullptr;
     int la_heads = 1, la_cluster = 1, la_tile = 64;       // absorbed form: heads per block, widest cluster, keys per tile
+    // linear attention beside attention
+    int lin_in = 0, lin_mix = 0;          // its first column in the projections and in the mixer output
+    int lin_vp = 0;                       // value channels padded to 4 (state rows)
+    float* lin_powers = nullptr;          // [linear_heads][kLinearChunk + 1]
+    bool linear() const { return d.mixer == EFM_MIXER_PARALLEL; }
+    bool attention() const { return d.mixer == EFM_MIXER_ATTENTION || d.mixer == EFM_MIXER_PARALLEL; }
     // routed experts
-    DecLinear router, expert_in, expert_out;   // [experts]; [experts][2 * ffp]; [experts][width][ffp]
-    int ffp = 0;
+    DecLinear router, expert_in, expert_out;   // [experts], a shared expert's gate behind; [experts][2 * ffp]; [experts][width][ffp]
+    DecLinear shared_in, shared_out;      // [2 * sfp]; [width][sfp]
+    int ffp = 0, sfp = 0;
     bool moe() const { return d.experts > 0; }
     bool mlp() const { return d.experts > 0 || d.ff > 0; }
 };
@@ -52,7 +64,7 @@ struct DecoderLayer {
 struct DecoderRun {
     int layer = 0;
     void *k_pool = nullptr, *v_pool = nullptr;       // attention: [pages * 64][kv_heads][Dp / Vp]; latent: [pages * 64][Lc + Rc] (k_pool); bf16 or fp32
-    size_t state_off = 0;                 // delta: first float of this run inside a state slot
+    size_t state_off = 0;                 // recurrent mixers: first float of this run inside a state slot
 };
 
 struct DecoderModel {
@@ -60,11 +72,13 @@ struct DecoderModel {
     bool f32 = false;
     int W = 0, Wp = 0;                    // width, padded to 8
     int side_p = 0;                       // token-side width padded to 8
-    // decode GEMV level 2 (gemv.cuh): input norms, embedding scale
-    bool input_norms() const { return d.norm_layout == EFM_NORM_SANDWICH || d.embed_scale != 1.0f; }
+    bool tanh_norms() const { return d.norm_layout == EFM_NORM_INPUT; }
+    // level of the decode GEMV (gemv.cuh)
+    int gemv_level() const { return tanh_norms() ? 3 : d.norm_layout == EFM_NORM_SANDWICH || d.embed_scale != 1.0f ? 2 : 1; }
     std::vector<DecoderLayer> layers;
     std::vector<DecoderRun> runs;         // in order
-    __nv_bfloat16 *side_embed = nullptr, *final_norm = nullptr;
+    __nv_bfloat16* side_embed = nullptr;
+    DecNorm final_norm;
     DecLinear head;
     std::set<std::string> seen;
     // caches
@@ -79,9 +93,11 @@ struct DecoderModel {
     // latent attention, long entries: visible cache rows and what they expand to
     __nv_bfloat16 *ws_c = nullptr, *ws_kv = nullptr;
     int ws_pages = 0, ws_window = 0;      // capacity (0: no layer uses it); largest window of the layers that use it (0: no window)
+    float* lin_ws = nullptr;              // linear attention: states of a pass's chunks
     // routed experts: rows sorted by expert
     void *ex_in = nullptr, *ex_act = nullptr, *ex_y = nullptr;
-    float *ex_gu = nullptr, *route_logits = nullptr;
+    void *sh_act = nullptr, *sh_y = nullptr;              // shared expert
+    float *ex_gu = nullptr, *sh_gu = nullptr, *route_logits = nullptr;
     ExpertRows ex{};
     int ex_rows = 0;
     int32_t* step_buf = nullptr;          // packed per-step indices
@@ -122,6 +138,8 @@ int decoder_simt_tile_rows();
 bool decoder_layer_tc(const DecoderModel& m, const DecoderLayer& l);
 // scratch of one recurrent layer for `rows` rows of at most `entries` sequences
 size_t decoder_delta_pack_floats(int heads, int dim, int rows, int entries);
+// the same of a layer with linear attention: chunk states
+size_t decoder_linear_ws_floats(const DecoderLayer& l, int rows, int entries);
 // first cache page (of its sequence) that a long entry at position pos0 needs in the workspace
 inline int decoder_ws_page0(const DecoderModel& m, int pos0) { return m.ws_window > 0 ? std::max(0, pos0 - m.ws_window + 1) / kPageTokens : 0; }
 cudaError_t configure_decoder(DecoderModel& m);      // after the layers are set up

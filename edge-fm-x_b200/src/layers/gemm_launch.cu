@@ -77,7 +77,7 @@ static void launch_gemm(Launcher& L, const GemmParams& p, int* error_word = null
     const dim3 block(tc::kThreads);
     const bool pdl = L.pdl;
     L.pdl = false;     // prefill kernels do not use the dependent-launch protocol
-    if constexpr (EPI == GemmEpi::Bf16Bias || EPI == GemmEpi::SwiGlu) {
+    if constexpr (EPI == GemmEpi::Bf16Bias || gemm_is_glu(EPI)) {
         if (p.group_tile != nullptr) {
             static bool attr_group = false;
             if (!attr_group) {
@@ -91,10 +91,10 @@ static void launch_gemm(Launcher& L, const GemmParams& p, int* error_word = null
     }
     // Few output tiles and a long K: split K so that the whole GPU works, fp32 partials to the workspace, then
     // a fixed-order sum with the epilogue.
-    if constexpr (EPI == GemmEpi::Bf16Bias || EPI == GemmEpi::Residual || EPI == GemmEpi::F32 || EPI == GemmEpi::SwiGlu) {
+    if constexpr (EPI == GemmEpi::Bf16Bias || EPI == GemmEpi::Residual || EPI == GemmEpi::F32 || EPI == GemmEpi::Bf16Relu2 || gemm_is_glu(EPI)) {
         const int KB = (p.K + tc::BK - 1) / tc::BK;
         int splits = std::min(L.num_sms / std::max(1, tiles), KB / min_kb_per_split());
-        if (L.gemm_ws != nullptr && splits >= 2 && (p.N & 3) == 0 && (EPI != GemmEpi::SwiGlu || (p.N & 127) == 0) &&
+        if (L.gemm_ws != nullptr && splits >= 2 && (p.N & 3) == 0 && (!gemm_is_glu(EPI) || (p.N & 127) == 0) &&
             (size_t)splits * p.M * p.N <= L.gemm_ws_floats) {
             const int per = (KB + splits - 1) / splits;
             splits = (KB + per - 1) / per;                 // no empty split
@@ -108,7 +108,7 @@ static void launch_gemm(Launcher& L, const GemmParams& p, int* error_word = null
                 attr_f32 = true;
             }
             L.launch(gemm_tc_kernel<GemmEpi::F32>, dim3(std::min(L.num_sms, tiles * splits)), block, tc::SMEM_BYTES, ma, mb, q, error_word);
-            const size_t total4 = (size_t)p.M * p.N / (EPI == GemmEpi::SwiGlu ? 8 : 4);
+            const size_t total4 = (size_t)p.M * p.N / (gemm_is_glu(EPI) ? 8 : 4);
             const int fin = (int)std::min<size_t>((total4 + 255) / 256, (size_t)L.num_sms * 4);
             L.launch(gemm_splitk_finish_kernel<EPI>, dim3(fin), dim3(256), 0, (const float*)L.gemm_ws, splits, p);
             L.pdl = pdl;
@@ -183,6 +183,8 @@ void launch_gemm_epi(Launcher& L, GemmEpi epi, const GemmParams& p, int* error_w
         case GemmEpi::Bf16Gelu: launch_gemm<GemmEpi::Bf16Gelu>(L, p, error_word); break;
         case GemmEpi::Bf16GeluTanh: launch_gemm<GemmEpi::Bf16GeluTanh>(L, p, error_word); break;
         case GemmEpi::SwiGlu: launch_gemm<GemmEpi::SwiGlu>(L, p, error_word); break;
+        case GemmEpi::Bf16Relu2: launch_gemm<GemmEpi::Bf16Relu2>(L, p, error_word); break;
+        case GemmEpi::ClampGlu: launch_gemm<GemmEpi::ClampGlu>(L, p, error_word); break;
     }
 }
 

@@ -1,5 +1,5 @@
-// Row kernels of the layered decoders' many-row pass: output norms with the residual add, PolyNorm, the per-layer token
-// input, gathered final norms, and the all-32-bit matrix product.  T = bf16 (tensor-core operands) or fp32.
+// Row kernels of the layered decoders' many-row pass: norms with the residual add, PolyNorm, the per-layer token input,
+// gathered final norms, the cap of the logits, and the all-32-bit matrix product.  T = bf16 (tensor-core operands) or fp32.
 #pragma once
 #include "common.cuh"
 #include "gemv.cuh"
@@ -36,6 +36,9 @@ struct SumOf {
     int top;
     int32_t* count;                   // rows per expert, zeroed for the next pass by block 0
     int experts;
+    int plain;                        // 1: the weights are in the experts' inputs already
+    const T* shared;                  // output of a shared expert (null: none) ...
+    const float* shared_weight;       // ... and its weight, [rows]
 };
 
 // x += y / sqrt(mean(y^2) + eps) * w (w null: x unchanged); out (null: none) = x as T, or (PRE) x / sqrt(mean(x^2) + eps) * pre,
@@ -168,6 +171,68 @@ __global__ void __launch_bounds__(128) token_gate_rows_kernel(const float* __res
     const __nv_bfloat16* e = table + (size_t)(ok ? id : 0) * table_ld + off;
     for (int c = threadIdx.x; c < ld; c += 128)
         store_f32(out + (size_t)row * ld + c, ok && c < n ? gelu_tanh(s[(size_t)row * ld + c]) * __bfloat162float(e[c]) : 0.f);
+}
+
+// Elementwise input norm: x += mult * y, out = tanh(alpha x) w + b.  y: null (SUM: the experts' outputs of the row instead); w null: no
+// output.  Grid (parts of a row, rows): a thread has four channels.
+template <typename T, bool SUM>
+__global__ void __launch_bounds__(256) add_tanh_rows_kernel(float* __restrict__ x, const float* __restrict__ y, float mult, T* __restrict__ out,
+                                                            const __nv_bfloat16* __restrict__ w, const __nv_bfloat16* __restrict__ b,
+                                                            const __nv_bfloat16* __restrict__ alpha, int ld, const SumOf<T> sum) {
+    const int c = 4 * (blockIdx.x * 256 + threadIdx.x);
+    const size_t row = blockIdx.y, base = row * ld;
+    if (SUM && row == 0)
+        for (int e = blockIdx.x * 256 + threadIdx.x; e < sum.experts; e += 256 * gridDim.x) sum.count[e] = 0;
+    if (c >= ld) return;
+    float4 r = load4(x + base + c);
+    if (SUM || y != nullptr) {
+        float4 a;
+        if constexpr (SUM) {
+            a = make_float4(0.f, 0.f, 0.f, 0.f);
+            auto add = [&](float g, const float4& v) { a.x = fmaf(g, v.x, a.x); a.y = fmaf(g, v.y, a.y); a.z = fmaf(g, v.z, a.z); a.w = fmaf(g, v.w, a.w); };
+            for (int k = 0; k < sum.top; ++k) {
+                const size_t i = row * sum.top + k;
+                add(sum.plain ? 1.0f : sum.weight[i], load4(sum.ye + (size_t)sum.place[i] * ld + c));
+            }
+            if (sum.shared != nullptr) add(sum.shared_weight[row], load4(sum.shared + base + c));
+        } else {
+            a = load4(y + base + c);
+        }
+        r.x = fmaf(mult, a.x, r.x); r.y = fmaf(mult, a.y, r.y); r.z = fmaf(mult, a.z, r.z); r.w = fmaf(mult, a.w, r.w);
+        store4(x + base + c, r);
+    }
+    if (w == nullptr) return;
+    const float al = __bfloat162float(*alpha);
+    const float4 g = load4(w + c), h = load4(b + c);
+    store4(out + base + c, make_float4(tanh_norm(r.x, al, g.x, h.x), tanh_norm(r.y, al, g.y, h.y), tanh_norm(r.z, al, g.z, h.z), tanh_norm(r.w, al, g.w, h.w)));
+}
+
+// out[i] = tanh(alpha x[rows[i]]) w + b
+template <typename T>
+__global__ void __launch_bounds__(256) gather_tanh_rows_kernel(const float* __restrict__ x, const int32_t* __restrict__ rows, const __nv_bfloat16* __restrict__ w,
+                                                               const __nv_bfloat16* __restrict__ b, const __nv_bfloat16* __restrict__ alpha, T* __restrict__ out, int ld) {
+    const float al = __bfloat162float(*alpha);
+    const float* src = x + (size_t)rows[blockIdx.x] * ld;
+    for (int c = threadIdx.x; c < ld / 4; c += 256) {
+        const float4 v = load4(src + 4 * c), g = load4(w + 4 * c), h = load4(b + 4 * c);
+        store4(out + (size_t)blockIdx.x * ld + 4 * c,
+               make_float4(tanh_norm(v.x, al, g.x, h.x), tanh_norm(v.y, al, g.y, h.y), tanh_norm(v.z, al, g.z, h.z), tanh_norm(v.w, al, g.w, h.w)));
+    }
+}
+
+// logits in place; grid (parts of a row, rows)
+__global__ void __launch_bounds__(256) cap_logits_rows_kernel(float* __restrict__ z, int n, int ld, float scale, float softcap) {
+    const int c = blockIdx.x * 256 + threadIdx.x;
+    if (c < n) z[(size_t)blockIdx.y * ld + c] = cap_logit(z[(size_t)blockIdx.y * ld + c], scale, softcap);
+}
+
+// z = relu(z)^2, n numbers, a multiple of 4
+__global__ void __launch_bounds__(256) relu2_kernel(float* __restrict__ z, size_t n) {
+    const size_t i = ((size_t)blockIdx.x * 256 + threadIdx.x) * 4;
+    if (i >= n) return;
+    float4 v = load4(z + i);
+    v.x = fmaxf(v.x, 0.f); v.y = fmaxf(v.y, 0.f); v.z = fmaxf(v.z, 0.f); v.w = fmaxf(v.w, 0.f);
+    store4(z + i, make_float4(v.x * v.x, v.y * v.y, v.z * v.z, v.w * v.w));
 }
 
 // out[i] = rms(x[rows[i]]) * w

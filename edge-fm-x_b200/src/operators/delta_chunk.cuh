@@ -19,18 +19,6 @@ namespace dc {
 constexpr int C = 16, kThreads = 128, kScanThreads = 256, kCols = 16;
 __host__ __device__ constexpr int pack_floats(int DP) { return 113 * DP; }
 
-// Chunk `idx` of the pass -> entry, first token; false past the last chunk.  first: index of the entry's first chunk.
-__device__ __forceinline__ bool locate(const RowPlan& plan, int idx, RowEntry& e, int& t0) {
-    int at = 0;
-    for (int i = 0; i < plan.n_entries; ++i) {
-        e = plan.entry(i);
-        const int n = (e.n + C - 1) / C;
-        if (idx < at + n) { t0 = (idx - at) * C; return true; }
-        at += n;
-    }
-    return false;
-}
-
 template <int DP>
 struct PrepSmem {
     float xq[32][DP + 4];             // X rows, then Q rows
@@ -60,7 +48,7 @@ __global__ void __launch_bounds__(dc::kThreads) delta_prepare_kernel(const float
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y, HD = s.heads * s.D, c0 = h * s.D;
     RowEntry e;
     int t0;
-    if (!locate(plan, blockIdx.x, e, t0)) return;
+    if (!locate_chunk<C>(plan, blockIdx.x, e, t0)) return;
     const int nv = min(C, e.n - t0);
     // ---- step inputs: a warp per token ----------------------------------------------------------------------------
     constexpr int NT = C / 4, NI = DP / 32;

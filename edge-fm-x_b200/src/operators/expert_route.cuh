@@ -5,7 +5,7 @@
 
 namespace efm {
 
-// z: router logits of all experts.  Scores softmax(z); the groups whose best scores are the largest stay open; the best `top`
+// z: router logits of all experts.  Scores softmax(z) or sigmoid(z); the groups whose best scores are the largest stay open; the best `top`
 // experts of those are handed to store(k, expert, score) in lane 0.  Ties go to the lower number.
 template <int N, typename Store>
 __device__ __forceinline__ void route_token_n(const float* z, const RouteShape& r, Store store) {      // at most 32 N experts
@@ -17,15 +17,20 @@ __device__ __forceinline__ void route_token_n(const float* z, const RouteShape& 
         v[i] = e < r.experts ? __ldcg(z + e) : -INFINITY;
         mx = fmaxf(mx, v[i]);
     }
-    mx = warp_max(mx);
+    if (r.sigmoid) {
 #pragma unroll
-    for (int i = 0; i < N; ++i) {
-        v[i] = lane + 32 * i < r.experts ? expf(v[i] - mx) : 0.f;
-        sum += v[i];
+        for (int i = 0; i < N; ++i) v[i] = lane + 32 * i < r.experts ? 1.0f / (1.0f + expf(-v[i])) : -1.f;
+    } else {
+        mx = warp_max(mx);
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            v[i] = lane + 32 * i < r.experts ? expf(v[i] - mx) : 0.f;
+            sum += v[i];
+        }
+        const float inv = 1.0f / warp_sum(sum);
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = lane + 32 * i < r.experts ? v[i] * inv : -1.f;
     }
-    const float inv = 1.0f / warp_sum(sum);
-#pragma unroll
-    for (int i = 0; i < N; ++i) v[i] = lane + 32 * i < r.experts ? v[i] * inv : -1.f;
     if (r.keep < r.groups) {                                            // close all but the best groups
         float best[2] = {-1.f, -1.f};                                   // lane l: groups l and l + 32
         for (int g = 0; g < r.groups; ++g) {

@@ -8,7 +8,11 @@ namespace efm {
 constexpr int kMaxExperts = 512, kMaxExpertTop = 32, kMaxExpertGroups = 64;
 constexpr int kExpertTile = 128;      // rows of an expert start at multiples of this
 
-struct RouteShape { int experts, top, groups, keep; };
+struct RouteShape {
+    int experts, top, groups, keep;
+    int sigmoid;                      // scores: 0 softmax of the logits, 1 sigmoid of each
+    int shared;                       // 1: logit `experts` gates a shared expert
+};
 
 struct ExpertRows {
     int32_t* id;                      // [rows][top]
@@ -17,6 +21,7 @@ struct ExpertRows {
     int32_t* count;                   // [experts], zero between passes
     int4* tile;                       // [tiles]: expert, its first tile, its number of tiles
     int32_t* n_tiles;                 // tiles in use
+    float* shared;                    // [rows]: gate of the shared expert
 };
 
 }  // namespace efm

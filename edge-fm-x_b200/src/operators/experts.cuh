@@ -1,18 +1,20 @@
 // Routed feed-forward: every token uses `top` of `experts` small gated feed-forwards,
-//   y = sum_k s_k W_down[e_k] (silu(W_gate[e_k] h) * W_up[e_k] h),   s = softmax(W_router h),
+//   y = sum_k s_k W_down[e_k] (silu(W_gate[e_k] h) * W_up[e_k] h),   s = softmax(W_router h) or sigmoid(W_router h),
 // where e_k are the best experts of the best groups (a group's score is its largest expert score) and s_k their scores as they
-// are.  Weights: [experts][2 * ffp rows][K] with blocks of 64 gate rows followed by the 64 matching up rows, and
+// are; they may scale the experts' inputs instead of their outputs.  A shared expert runs for every token beside them.
+// Weights: [experts][2 * ffp rows][K] with blocks of 64 gate rows followed by the 64 matching up rows, and
 // [experts][n_out][ffp]; ffp is the expert width padded to 64 with zero rows / columns.
 //
 //   route_token          one token's choice, by one warp (expert_route.cuh; the decode GEMV of gemv.cuh chooses the same way)
 //   expert_route_rows    many rows: choices, weights, and each choice's place among its expert's rows
 //   expert_gather_rows   the rows sorted by expert, every expert's share starting at a multiple of kExpertTile rows, and the
 //                        expert of each such tile: the A operand of the grouped products (gemm_tc.cuh, gemm_f32)
-//   silu_mul_rows        32-bit mode: silu(gate) * up
+//   glu_rows             32-bit mode: the gated unit (gemv.cuh)
 // The weighted sum of the expert outputs is part of the output norm (add_norm_rows, decoder_rows.cuh).
 #pragma once
 #include "common.cuh"
 #include "expert_route.cuh"
+#include "gemv.cuh"
 
 namespace efm {
 
@@ -25,6 +27,7 @@ __global__ void __launch_bounds__(256) expert_route_rows_kernel(const float* __r
         o.weight[(size_t)row * r.top + k] = w;
         o.place[(size_t)row * r.top + k] = atomicAdd(o.count + e, 1);
     });
+    if (r.shared && (threadIdx.x & 31) == 0) o.shared[row] = 1.0f / (1.0f + expf(-logits[(size_t)row * ld + r.experts]));
 }
 
 // First row of every expert in the sorted order, by the first warp; block 0 describes the tiles.
@@ -48,11 +51,12 @@ __device__ __forceinline__ void expert_offsets(const int32_t* count, int experts
     if (publish != nullptr && lane == 0) *publish->n_tiles = base;
 }
 
-// Row `row` of h to its places in the sorted order.  One block per row; ld % 8 == 0.
-template <typename T>
+// Row `row` of h, or (SCALE) each choice's weight times it, to its places in the sorted order.  One block per row; ld % 8 == 0.
+template <typename T, bool SCALE>
 __global__ void __launch_bounds__(128) expert_gather_rows_kernel(const T* __restrict__ h, T* __restrict__ out, int ld, const RouteShape r, const ExpertRows o) {
     __shared__ int32_t off[kMaxExperts];
     __shared__ int32_t dst[kMaxExpertTop];
+    __shared__ float weight[SCALE ? kMaxExpertTop : 1];
     const int row = blockIdx.x;
     if (threadIdx.x < 32) {
         expert_offsets(o.count, r.experts, off, row == 0 ? &o : nullptr);
@@ -62,25 +66,40 @@ __global__ void __launch_bounds__(128) expert_gather_rows_kernel(const T* __rest
             const int d = off[o.id[i]] + o.place[i];
             dst[threadIdx.x] = d;
             o.place[i] = d;
+            if constexpr (SCALE) weight[threadIdx.x] = o.weight[i];
         }
     }
     __syncthreads();
     constexpr int V = 16 / sizeof(T);
     for (int c = threadIdx.x; c < ld / V; c += 128) {
         const uint4 v = ld_cached(h + (size_t)row * ld + c * V);
-        for (int k = 0; k < r.top; ++k) *reinterpret_cast<uint4*>(out + (size_t)dst[k] * ld + c * V) = v;
+        for (int k = 0; k < r.top; ++k) {
+            uint4 x = v;
+            if constexpr (SCALE) {
+                const float w = weight[k];
+                if constexpr (sizeof(T) == 2)
+                    x = make_uint4(pack_bf16(w * bf16lo(v.x), w * bf16hi(v.x)), pack_bf16(w * bf16lo(v.y), w * bf16hi(v.y)),
+                                   pack_bf16(w * bf16lo(v.z), w * bf16hi(v.z)), pack_bf16(w * bf16lo(v.w), w * bf16hi(v.w)));
+                else
+                    x = make_uint4(__float_as_uint(w * __uint_as_float(v.x)), __float_as_uint(w * __uint_as_float(v.y)),
+                                   __float_as_uint(w * __uint_as_float(v.z)), __float_as_uint(w * __uint_as_float(v.w)));
+            }
+            *reinterpret_cast<uint4*>(out + (size_t)dst[k] * ld + c * V) = x;
+        }
     }
 }
 
-// gu: rows of 64 gate values followed by the 64 matching up values -> silu(gate) * up, ffp columns.  Grid: tiles of kExpertTile rows.
-__global__ void __launch_bounds__(256) silu_mul_rows_kernel(const float* __restrict__ gu, float* __restrict__ out, int ffp, const int32_t* __restrict__ n_tiles) {
+// gu: rows of 64 gate values followed by the 64 matching up values -> gated unit, ffp columns.  Grid: tiles of kExpertTile rows, of
+// which *n_tiles (null: all) are in use.
+__global__ void __launch_bounds__(256) glu_rows_kernel(const float* __restrict__ gu, float* __restrict__ out, int rows, int ffp, const int32_t* __restrict__ n_tiles,
+                                                       int kind, float limit) {
     const int tile = blockIdx.x;
-    if (tile >= *n_tiles) return;
+    if (n_tiles != nullptr && tile >= *n_tiles) return;
     for (int i = threadIdx.x; i < kExpertTile * ffp; i += 256) {
         const int r = i / ffp, c = i - r * ffp;
+        if (tile * kExpertTile + r >= rows) return;
         const float* src = gu + (size_t)(tile * kExpertTile + r) * 2 * ffp + (c >> 6) * 128 + (c & 63);
-        const float g = src[0], u = src[64];
-        out[(size_t)(tile * kExpertTile + r) * ffp + c] = g / (1.0f + expf(-g)) * u;
+        out[(size_t)(tile * kExpertTile + r) * ffp + c] = glu(kind, src[0], src[64], limit);
     }
 }
 

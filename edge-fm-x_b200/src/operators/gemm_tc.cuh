@@ -14,7 +14,7 @@
 //               longer than its MMAs whenever K was short):
 //               tcgen05.ld (row = TMEM lane, 32 columns at a time), bias / activation, staging through
 //               shared memory (XOR-swizzled 16-byte columns) so that global rows are written as contiguous segments:
-//               bf16 (+bias, optionally erf-GELU) | fp32 residual add | fp32 | silu(gate)*up in bf16.
+//               bf16 (+bias, optionally erf-GELU, tanh-GELU or squared ReLU) | fp32 residual add | fp32 | a gated unit in bf16.
 // Rows past M and columns past N are zero-filled by TMA on load and masked on store.
 // Every mbarrier wait is bounded; a wait that gives up raises *error, all roles leave their loops, the
 // block frees its TMEM and returns.  Bound: tensor pipe (2 M N K flops).
@@ -25,7 +25,7 @@
 
 namespace efm {
 
-enum class GemmEpi : int { Bf16Bias = 0, Residual = 1, F32 = 2, Bf16Gelu = 3, SwiGlu = 4, Bf16GeluTanh = 5 };
+enum class GemmEpi : int { Bf16Bias = 0, Residual = 1, F32 = 2, Bf16Gelu = 3, SwiGlu = 4, Bf16GeluTanh = 5, Bf16Relu2 = 6, ClampGlu = 7 };
 
 struct GroupTile { int32_t group, first, count, pad; };      // row tile: its group, the group's first row tile and number of them
 
@@ -49,7 +49,21 @@ struct GemmParams {
     const GroupTile* group_tile = nullptr;
     const int32_t* group_tiles = nullptr;
     int group_rows = 0, group_all = 0;      // rows of B per group and altogether
+    float limit = 0.f;        // ClampGlu
 };
+
+// Gated units over a fused gate|up weight: half as many output columns.
+constexpr bool gemm_is_glu(GemmEpi e) { return e == GemmEpi::SwiGlu || e == GemmEpi::ClampGlu; }
+template <GemmEpi EPI>
+__device__ __forceinline__ float gemm_glu(float g, float u, float limit) {
+    if constexpr (EPI == GemmEpi::ClampGlu) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit) + 1.0f;
+        return __fdividef(g, 1.0f + __expf(-1.702f * g)) * u;
+    }
+    // the approximate reciprocal instead of an IEEE division: the epilogue warps' issue slots are the limit when K is short
+    return __fdividef(g, 1.0f + __expf(-g)) * u;
+}
 
 namespace tc {
 
@@ -255,9 +269,9 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
             if (!mbar_wait(accf0 + 8 * a, use, abort_s)) { *abort_s = 1; break; }
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const uint32_t acc = tmem + ((uint32_t)(q * 32) << 16) + (uint32_t)(a * BN);
-            constexpr int OUT_COLS = EPI == GemmEpi::SwiGlu ? BN / 2 : BN;
-            const int ldc = EPI == GemmEpi::SwiGlu ? (p.N >> 1) : p.N;         // output row length
-            const int nc0 = EPI == GemmEpi::SwiGlu ? (n0 >> 1) : n0;           // first output column of the tile
+            constexpr int OUT_COLS = gemm_is_glu(EPI) ? BN / 2 : BN;
+            const int ldc = gemm_is_glu(EPI) ? (p.N >> 1) : p.N;               // output row length
+            const int nc0 = gemm_is_glu(EPI) ? (n0 >> 1) : n0;           // first output column of the tile
             const bool vec = (ldc & 3) == 0;
             const size_t split_off = compact ? (size_t)item * (size_t)(BM * BN)
                                              : (!GROUPED && p.kb_per_split > 0 ? (size_t)z * (size_t)p.M * (size_t)p.N : 0);
@@ -278,9 +292,9 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
                     }
                 }
                 float o[32];
-                if constexpr (EPI == GemmEpi::SwiGlu) {
+                if constexpr (gemm_is_glu(EPI)) {
                     // fused gate|up weight: in every 128 columns the first 64 are gate rows and the last 64 the up
-                    // rows of the same channels; out[m, n/2 + j] = silu(gate_j) * up_j
+                    // rows of the same channels; out[m, n/2 + j] = unit(gate_j, up_j)
                     const int blk = c0 >> 6, cc = c0 & 63;
                     uint32_t rg[32], ru[32];
                     tmem_ld32(acc + (uint32_t)(blk * 128 + cc), rg);
@@ -298,9 +312,7 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
                             g += __shfl_sync(0xffffffffu, bias_g, e);
                             u += __shfl_sync(0xffffffffu, bias_u, e);
                         }
-                        // four epilogue warps drain a tile while one warp feeds the tensor cores: their issue slots are
-                        // the limit when K is short, hence the approximate reciprocal instead of an IEEE division
-                        o[e] = __fdividef(g, 1.0f + __expf(-g)) * u;
+                        o[e] = gemm_glu<EPI>(g, u, p.limit);
                     }
                 } else {
                     uint32_t r[32];
@@ -312,6 +324,7 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
                     for (int e = 0; e < 32; ++e) {
                         o[e] = __uint_as_float(r[e]) + __shfl_sync(0xffffffffu, bias_l, e);
                         if constexpr (EPI == GemmEpi::Bf16Gelu) o[e] = 0.5f * o[e] * (1.0f + erff(o[e] * 0.70710678118654752f));
+                        if constexpr (EPI == GemmEpi::Bf16Relu2) { o[e] = fmaxf(o[e], 0.f); o[e] *= o[e]; }
                         if constexpr (EPI == GemmEpi::Bf16GeluTanh)
                         {
                             float th;           // hardware tanh (relative error ~2^-11, below the bf16 rounding of the result)
@@ -377,8 +390,8 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
 template <GemmEpi EPI>
 __global__ void __launch_bounds__(256) gemm_splitk_finish_kernel(const float* __restrict__ ws, int splits, const GemmParams p) {
     const size_t plane = (size_t)p.M * p.N;
-    if constexpr (EPI == GemmEpi::SwiGlu) {
-        // fused gate|up partials [M, N] (64 gate columns, 64 up columns, ...) -> out [M, N / 2] = silu(gate) * up
+    if constexpr (gemm_is_glu(EPI)) {
+        // fused gate|up partials [M, N] (64 gate columns, 64 up columns, ...) -> out [M, N / 2] = unit(gate, up)
         const int half = p.N >> 1;
         const size_t out4 = (size_t)p.M * half / 4;        // N % 128 == 0 (checked by the launcher)
         for (size_t i = (size_t)blockIdx.x * 256 + threadIdx.x; i < out4; i += (size_t)gridDim.x * 256) {
@@ -397,8 +410,8 @@ __global__ void __launch_bounds__(256) gemm_splitk_finish_kernel(const float* __
                 g.x += __bfloat162float(bg[0]); g.y += __bfloat162float(bg[1]); g.z += __bfloat162float(bg[2]); g.w += __bfloat162float(bg[3]);
                 u.x += __bfloat162float(bg[64]); u.y += __bfloat162float(bg[65]); u.z += __bfloat162float(bg[66]); u.w += __bfloat162float(bg[67]);
             }
-            const float o0 = g.x / (1.0f + __expf(-g.x)) * u.x, o1 = g.y / (1.0f + __expf(-g.y)) * u.y;
-            const float o2 = g.z / (1.0f + __expf(-g.z)) * u.z, o3 = g.w / (1.0f + __expf(-g.w)) * u.w;
+            const float o0 = gemm_glu<EPI>(g.x, u.x, p.limit), o1 = gemm_glu<EPI>(g.y, u.y, p.limit);
+            const float o2 = gemm_glu<EPI>(g.z, u.z, p.limit), o3 = gemm_glu<EPI>(g.w, u.w, p.limit);
             *reinterpret_cast<uint2*>(p.C + m * half + j) = make_uint2(pack_bf16(o0, o1), pack_bf16(o2, o3));
         }
         return;
@@ -421,6 +434,10 @@ __global__ void __launch_bounds__(256) gemm_splitk_finish_kernel(const float* __
             const float4 o = *reinterpret_cast<const float4*>(p.Cf + i * 4);
             *reinterpret_cast<float4*>(p.Cf + i * 4) = make_float4(o.x + a.x, o.y + a.y, o.z + a.z, o.w + a.w);
         } else {
+            if constexpr (EPI == GemmEpi::Bf16Relu2) {
+                a.x = fmaxf(a.x, 0.f); a.y = fmaxf(a.y, 0.f); a.z = fmaxf(a.z, 0.f); a.w = fmaxf(a.w, 0.f);
+                a.x *= a.x; a.y *= a.y; a.z *= a.z; a.w *= a.w;
+            }
             *reinterpret_cast<uint2*>(p.C + i * 4) = make_uint2(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w));
         }
     }

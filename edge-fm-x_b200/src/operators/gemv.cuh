@@ -31,16 +31,19 @@
 
 namespace efm {
 
-enum class Epi : int { Plain = 0, Residual = 1, QkvRope = 2, SwiGlu = 3, Logits = 4, Peers = 5, Store32 = 6, TokenGate = 7, ExpertUp = 8, ExpertDown = 9, Router = 10, Store32Bias = 11 };
+enum class Epi : int { Plain = 0, Residual = 1, QkvRope = 2, SwiGlu = 3, Logits = 4, Peers = 5, Store32 = 6, TokenGate = 7, ExpertUp = 8, ExpertDown = 9, Router = 10, Store32Bias = 11, Relu2 = 12 };
 constexpr int kMaxPeers = 8;
-// The last four (and the epilogues from Store32 on) exist in the EXT instantiations only (layered decoders; level 2 adds input
-// norms: Norm, and the second norm and the scale of Embed):
+// Embed and what follows it (and the epilogues from Store32 on) exist in the EXT instantiations only (layered decoders; level 2 adds
+// input norms: Norm, and the second norm and the scale of Embed; level 3 elementwise input norms, AddTanh and Merge, the clamped
+// and the shared expert and the cap of the logits):
 //   Embed    x = embed_table[token] * embed_scale; with norm2_w the product reads rmsnorm(x) * norm2_w
 //   Norm     x = rmsnorm(xf) * norm_w
 //   AddNorm  x = xr + rmsnorm(addend) * norm_w: a sublayer whose OUTPUT is normalised, folded into the next product;
 //            with norm2_w the product reads rmsnorm(x) * norm2_w instead of x
 //   PolyNorm x = c0 rms(z) + c1 rms(z^2) + c2 rms(z^3) + c3 with z = xf and the four numbers of `poly`
-enum : int { kProPlain = 0, kProRmsNorm = 1, kProEmbedRmsNorm = 2, kProEmbed = 3, kProAddNorm = 4, kProPolyNorm = 5, kProNorm = 6 };
+//   AddTanh  x = xr + add_mult * addend; the product reads tanh(alpha x) * norm_w + norm_b (Embed does the same when norm_b is given)
+//   Merge    channels [0, merge0) of xf as they are, the others rmsnorm(xf) * norm_w * sigmoid(merge_gate) * merge_scale
+enum : int { kProPlain = 0, kProRmsNorm = 1, kProEmbedRmsNorm = 2, kProEmbed = 3, kProAddNorm = 4, kProPolyNorm = 5, kProNorm = 6, kProAddTanh = 7, kProMerge = 8 };
 
 struct GemvParams {
     const __nv_bfloat16* W;   // [N, K] row-major
@@ -106,7 +109,35 @@ struct GemvParams {
     int32_t* route_id;        // [top]
     float* route_w;           // [top]
     int ff, ffp, expert_rows; // channels, padded channels, rows of one expert's matrix
+    // level 3
+    const __nv_bfloat16* norm_b;
+    const __nv_bfloat16* norm_alpha;      // one number
+    float add_mult;
+    int merge0;
+    const float* merge_gate;
+    float merge_scale;
+    float logit_scale, logit_softcap;     // Logits: softcap * tanh(logit_scale * z / softcap); softcap 0: logit_scale * z
+    // ExpertUp / ExpertDown: the gated unit's form; a shared expert behind the chosen ones (rows of W2, activations behind theirs,
+    // weight at route_w[top])
+    int glu, weight_input;
+    float limit, shared_limit;
+    const __nv_bfloat16* W2;
+    int shared_ff, shared_ffp;
 };
+
+// gated units: silu(g) u, or (clamped) g sigmoid(1.702 g) (u + 1) with g at most and u within +- limit
+enum : int { kGluSilu = 0, kGluClamped = 1 };
+__device__ __forceinline__ float glu(int kind, float g, float u, float limit) {
+    if (kind == kGluSilu) return g / (1.0f + expf(-g)) * u;
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
+__device__ __forceinline__ float tanh_norm(float x, float alpha, float w, float b) { return fmaf(tanhf(alpha * x), w, b); }
+__device__ __forceinline__ float cap_logit(float z, float scale, float softcap) {
+    z *= scale;
+    return softcap > 0.f ? softcap * tanhf(z / softcap) : z;
+}
 
 __device__ __forceinline__ float gelu_tanh(float z) {
     return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
@@ -129,7 +160,7 @@ __device__ __forceinline__ void group_barrier(int id, int nthreads) {
     asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(nthreads) : "memory");
 }
 
-template <Epi EPI>
+template <Epi EPI, int EXT = 0>
 __device__ __forceinline__ void item_rows(const GemvParams& p, int item, int& r0, int& r1, const int* chosen = nullptr) {
     (void)chosen;
     if constexpr (EPI == Epi::QkvRope) {
@@ -142,8 +173,8 @@ __device__ __forceinline__ void item_rows(const GemvParams& p, int item, int& r0
         r0 = ((item >> 6) << 7) + (item & 63);
         r1 = r0 + 64;
     } else if constexpr (EPI == Epi::ExpertUp) {
-        const int k = item / p.ff, j = item - k * p.ff;
-        r0 = chosen[k] * p.expert_rows + ((j >> 6) << 7) + (j & 63);
+        const int k = item / p.ff, j = item - (EXT > 2 && k >= p.route.top ? p.route.top : k) * p.ff;
+        r0 = (EXT > 2 && k >= p.route.top ? 0 : chosen[k] * p.expert_rows) + ((j >> 6) << 7) + (j & 63);
         r1 = r0 + 64;
     } else {
         r0 = item * 2;
@@ -151,9 +182,10 @@ __device__ __forceinline__ void item_rows(const GemvParams& p, int item, int& r0
     }
 }
 
-template <Epi EPI>
+template <Epi EPI, int EXT = 0>
 __device__ __forceinline__ void item_epilogue(const GemvParams& p, int item, float a0, float a1,
-                                              float& best_v, int& best_i) {
+                                              float& best_v, int& best_i, const int* chosen = nullptr) {
+    (void)chosen;
     if constexpr (EPI == Epi::Plain) {
         p.y[item * 2] = __float2bfloat16_rn(a0);
         p.y[item * 2 + 1] = __float2bfloat16_rn(a1);
@@ -172,6 +204,10 @@ __device__ __forceinline__ void item_epilogue(const GemvParams& p, int item, flo
         for (int r = 0; r < kMaxPeers; ++r)
             if (r < p.n_peers) st_peer_words(p.peer_out[r] + item * 2, w0, w1);
     } else if constexpr (EPI == Epi::Logits) {
+        if constexpr (EXT > 2) {
+            a0 = cap_logit(a0, p.logit_scale, p.logit_softcap);
+            a1 = cap_logit(a1, p.logit_scale, p.logit_softcap);
+        }
         *reinterpret_cast<float2*>(p.logits + item * 2) = make_float2(a0, a1);
         if (item * 2 >= p.N) a0 = -INFINITY;                          // padding rows
         if (item * 2 + 1 >= p.N) a1 = -INFINITY;
@@ -179,13 +215,24 @@ __device__ __forceinline__ void item_epilogue(const GemvParams& p, int item, flo
         if (a1 > best_v) { best_v = a1; best_i = item * 2 + 1; }      // the lowest id on ties
     } else if constexpr (EPI == Epi::ExpertUp) {
         const int k = item / p.ff;
-        p.out_f[k * p.ffp + item - k * p.ff] = a0 / (1.0f + expf(-a0)) * a1;
+        if constexpr (EXT > 2) {
+            const bool shared = k >= p.route.top;
+            const float w = !shared && p.weight_input ? __int_as_float(chosen[kMaxExpertTop + k]) : 1.0f;      // a product is linear in its input
+            p.out_f[shared ? p.route.top * p.ffp + item - p.route.top * p.ff : k * p.ffp + item - k * p.ff] =
+                glu(p.glu, a0 * w, a1 * w, shared ? p.shared_limit : p.limit);
+        } else {
+            p.out_f[k * p.ffp + item - k * p.ff] = a0 / (1.0f + expf(-a0)) * a1;
+        }
     } else if constexpr (EPI == Epi::ExpertDown) {
         *reinterpret_cast<float2*>(p.out_f + item * 2) = make_float2(a0, a1);
     } else if constexpr (EPI == Epi::Router) {
         __stcg(reinterpret_cast<float2*>(p.out_f + item * 2), make_float2(a0, a1));
     } else if constexpr (EPI == Epi::Store32Bias) {
         *reinterpret_cast<float2*>(p.out_f + item * 2) = make_float2(a0 + __bfloat162float(p.bias[item * 2]), a1 + __bfloat162float(p.bias[item * 2 + 1]));
+    } else if constexpr (EPI == Epi::Relu2) {
+        a0 = fmaxf(a0, 0.f);
+        a1 = fmaxf(a1, 0.f);
+        *reinterpret_cast<float2*>(p.out_f + item * 2) = make_float2(a0 * a0, a1 * a1);
     } else if constexpr (EPI == Epi::Store32) {
         *reinterpret_cast<float2*>(p.out_f + item * 2) = make_float2(a0, a1);
     } else if constexpr (EPI == Epi::TokenGate) {
@@ -271,31 +318,42 @@ __device__ __forceinline__ GemvSched gemv_sched(const GemvParams& p, const int k
     return sc;
 }
 
-template <Epi EPI>
+template <Epi EPI, int EXT = 0>
 __device__ __forceinline__ void gemv_load_unit(const GemvParams& p, const GemvSched& sc, const int u, uint4 (&buf)[kGemvU][2], const int* chosen = nullptr) {
     if (u >= sc.total) return;
     const int j = u / sc.upi, part = u - j * sc.upi;
     int r0, r1;
-    item_rows<EPI>(p, sc.ig0 + j * sc.ig_stride, r0, r1, chosen);
+    item_rows<EPI, EXT>(p, sc.ig0 + j * sc.ig_stride, r0, r1, chosen);
     if constexpr (EPI == Epi::ExpertDown) {
         const int per = p.ffp >> 3;                                   // chunks of one expert's row
         const float inv = 1.0f / (float)per;                           // c / per exactly: half a chunk is far above the rounding
         const __nv_bfloat16* w[kGemvU];                                // all addresses first: the loads then leave back to back
+        int ld[kGemvU];
 #pragma unroll
         for (int uu = 0; uu < kGemvU; ++uu) {
             const int c = min((part * kGemvU + uu) * sc.stride + sc.gl, sc.nch - 1), k = (int)(((float)c + 0.5f) * inv);
-            w[uu] = p.W + ((size_t)chosen[k] * p.expert_rows + r0) * p.ffp + (size_t)(c - k * per) * 8;
+            ld[uu] = p.ffp;
+            if (EXT > 2 && c >= p.route.top * per) {
+                ld[uu] = p.shared_ffp;
+                w[uu] = p.W2 + (size_t)r0 * p.shared_ffp + (size_t)(c - p.route.top * per) * 8;
+            } else {
+                w[uu] = p.W + ((size_t)chosen[k] * p.expert_rows + r0) * p.ffp + (size_t)(c - k * per) * 8;
+            }
         }
 #pragma unroll
         for (int uu = 0; uu < kGemvU; ++uu)
             if ((part * kGemvU + uu) * sc.stride + sc.gl < sc.nch) {
                 buf[uu][0] = ld_stream(w[uu]);
-                buf[uu][1] = ld_stream(w[uu] + p.ffp);
+                buf[uu][1] = ld_stream(w[uu] + ld[uu]);
             }
         return;
     }
-    const __nv_bfloat16* a = p.W + (size_t)r0 * p.K;
-    const __nv_bfloat16* b = p.W + (size_t)r1 * p.K;
+    const __nv_bfloat16* W = p.W;
+    if constexpr (EPI == Epi::ExpertUp && EXT > 2) {
+        if (sc.ig0 + j * sc.ig_stride >= p.route.top * p.ff) W = p.W2;
+    }
+    const __nv_bfloat16* a = W + (size_t)r0 * p.K;
+    const __nv_bfloat16* b = W + (size_t)r1 * p.K;
 #pragma unroll
     for (int uu = 0; uu < kGemvU; ++uu) {
         const int c = (part * kGemvU + uu) * sc.stride + sc.gl;
@@ -310,14 +368,28 @@ __device__ __forceinline__ void gemv_load_unit(const GemvParams& p, const GemvSc
 __host__ __device__ inline unsigned int gemv_xbytes(int K) { return ((unsigned int)K * 4u + 15u) & ~15u; }
 __host__ __device__ inline unsigned int gemv_wbytes(int K) { return ((unsigned int)K * 2u + 15u) & ~15u; }
 
+// Offset of the second staged vector of the EXT prologues (behind red + misc).
+__host__ __device__ inline unsigned int gemv_ext_off(int K) { return gemv_xbytes(K) + gemv_wbytes(K) + (2 * 16 * 2 + 16) * 4u; }
+
 // Weights only: the first two units into registers, the norm weight into shared memory.
 template <Epi EPI, int EXT>
 __device__ __forceinline__ void gemv_prefetch(const GemvParams& p, const GemvSched& sc, GemvRegs& r, unsigned char* smem,
                                               const unsigned int xbytes) {
-    if constexpr (EPI != Epi::ExpertUp && EPI != Epi::ExpertDown) gemv_load_unit<EPI>(p, sc, 0, r.a);
-    if (EXT ? (p.prologue == kProAddNorm || (EXT > 1 && p.prologue == kProNorm)) : p.prologue != kProPlain) {
+    if constexpr (EPI != Epi::ExpertUp && EPI != Epi::ExpertDown) gemv_load_unit<EPI, EXT>(p, sc, 0, r.a);
+    if (EXT ? (p.prologue == kProAddNorm || (EXT > 1 && p.prologue == kProNorm) || (EXT > 2 && p.prologue == kProAddTanh)) : p.prologue != kProPlain) {
         uint4* gs = reinterpret_cast<uint4*>(smem + xbytes);        // xbytes = gemv_xbytes(K)
         for (int c = threadIdx.x; c < sc.nch; c += kGemvThreads) gs[c] = ld_cached(p.norm_w + (size_t)c * 8);
+        if constexpr (EXT > 2) {
+            uint4* bs = reinterpret_cast<uint4*>(smem + gemv_ext_off(p.K));
+            if (p.prologue == kProAddTanh)
+                for (int c = threadIdx.x; c < sc.nch; c += kGemvThreads) bs[c] = ld_cached(p.norm_b + (size_t)c * 8);
+        }
+    }
+    if constexpr (EXT > 2) {
+        if (p.prologue == kProMerge) {
+            uint4* gs = reinterpret_cast<uint4*>(smem + xbytes);
+            for (int c = threadIdx.x; c < sc.nch - p.merge0 / 8; c += kGemvThreads) gs[c] = ld_cached(p.norm_w + (size_t)c * 8);
+        }
     }
 }
 
@@ -348,9 +420,6 @@ __device__ __forceinline__ void st8f(float* p, const float (&f)[8]) {
     reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
 }
 
-// Offset of the second staged vector of the AddNorm prologue (behind red + misc).
-__host__ __device__ inline unsigned int gemv_ext_off(int K) { return gemv_xbytes(K) + gemv_wbytes(K) + (2 * 16 * 2 + 16) * 4u; }
-
 // EXT prologues; false: not one of them.  Ends with a block barrier.
 template <int EXT>
 __device__ __forceinline__ bool gemv_stage_ext(const GemvParams& p, const int nch, unsigned char* smem, const unsigned int xbytes) {
@@ -371,6 +440,16 @@ __device__ __forceinline__ bool gemv_stage_ext(const GemvParams& p, const int nc
             if (EXT > 1 && p.x_out != nullptr && blockIdx.x == 0) st8f(p.x_out + 8 * c, x);
         }
     };
+    const float alpha = EXT > 2 && p.norm_alpha != nullptr ? __bfloat162float(*p.norm_alpha) : 0.f;
+    auto tanh8 = [&](int c, float (&f)[8], const uint4& wv, const uint4& bv) {
+        float w[8], b[8];
+        unpack8(wv, w);
+        unpack8(bv, b);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) f[j] = tanh_norm(f[j], alpha, w[j], b[j]);
+        if (p.x_out != nullptr && blockIdx.x == 0) st8f(p.x_out + 8 * c, f);
+    };
+    (void)tanh8;
     if (p.prologue == kProEmbed) {
         const int tok = p.state->token;
         const bool zero = tok < 0 || tok >= p.vocab;
@@ -385,8 +464,11 @@ __device__ __forceinline__ bool gemv_stage_ext(const GemvParams& p, const int nc
                     sq[0] = fmaf(f[j], f[j], sq[0]);
                 }
             }
-            st8f(xs + 8 * c, f);
             if (blockIdx.x == 0) st8f(p.resid_out + 8 * c, f);
+            if constexpr (EXT > 2) {
+                if (p.norm_b != nullptr) tanh8(c, f, ld_cached(p.norm_w + (size_t)c * 8), ld_cached(p.norm_b + (size_t)c * 8));
+            }
+            st8f(xs + 8 * c, f);
         }
         if constexpr (EXT > 1) {
             if (p.norm2_w != nullptr) norm2(sq);
@@ -408,6 +490,48 @@ __device__ __forceinline__ bool gemv_stage_ext(const GemvParams& p, const int nc
 #pragma unroll
             for (int j = 0; j < 8; ++j) x[j] = xs[8 * c + j] * inv * w[j];
             st8f(xs + 8 * c, x);
+        }
+    } else if (EXT > 2 && p.prologue == kProAddTanh) {
+        const uint4 *gs = reinterpret_cast<const uint4*>(smem + xbytes), *bs = reinterpret_cast<const uint4*>(smem + gemv_ext_off(p.K));
+        for (int c = tid; c < nch; c += kGemvThreads) {       // same thread, same chunks as in the prefetch
+            float y[8], x[8];
+            ld8f(p.addend + 8 * c, y);
+            ld8f(p.xr + 8 * c, x);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) x[j] = fmaf(p.add_mult, y[j], x[j]);
+            if (blockIdx.x == 0) st8f(p.resid_out + 8 * c, x);
+            tanh8(c, x, gs[c], bs[c]);
+            st8f(xs + 8 * c, x);
+        }
+    } else if (EXT > 2 && p.prologue == kProMerge) {
+        const uint4* gs = reinterpret_cast<const uint4*>(smem + xbytes);
+        float* xs2 = reinterpret_cast<float*>(smem + gemv_ext_off(p.K));
+        const int c0 = p.merge0 / 8;
+        for (int c = tid; c < c0; c += kGemvThreads) {
+            float x[8];
+            ld8f(p.xf + 8 * c, x);
+            st8f(xs + 8 * c, x);
+        }
+        for (int c = tid; c < nch - c0; c += kGemvThreads) {
+            float x[8], g[8], w[8];
+            ld8f(p.xf + 8 * (c0 + c), x);
+            ld8f(p.merge_gate + 8 * c, g);
+            unpack8(gs[c], w);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                if (8 * c + j >= p.k_true) x[j] = 0.f;                // pads
+                sq[0] = fmaf(x[j], x[j], sq[0]);
+                g[j] = w[j] / (1.0f + expf(-g[j]));
+            }
+            st8f(xs + 8 * (c0 + c), x);
+            st8f(xs2 + 8 * c, g);
+        }
+        gemv_block_sums<1>(sq, red3);
+        const float inv = p.merge_scale / sqrtf(sq[0] / (float)p.k_true + p.eps);
+        for (int c = tid; c < nch - c0; c += kGemvThreads) {
+            float* x = xs + 8 * (c0 + c);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) x[j] *= inv * xs2[8 * c + j];
         }
     } else if (p.prologue == kProAddNorm) {
         const uint4* gs = reinterpret_cast<const uint4*>(smem + xbytes);
@@ -587,13 +711,16 @@ __device__ __forceinline__ void gemv_run(const GemvParams& p, const GemvSched& s
         if (sc.wk == 0 && lane == 0 && sc.total > 0)
             old_first = __ldcg(reinterpret_cast<const float2*>(p.residual + sc.ig0 * 2));
     }
-    __shared__ int chosen_s[EPI == Epi::ExpertUp ? kMaxExpertTop : 1];
+    __shared__ int chosen_s[EPI == Epi::ExpertUp ? 2 * kMaxExpertTop : 1];
     const int* chosen = nullptr;
     if constexpr (EPI == Epi::ExpertUp) {
-        if (tid < p.route.top) chosen_s[tid] = __ldcg(p.route_id + tid);
+        if (tid < p.route.top) {
+            chosen_s[tid] = __ldcg(p.route_id + tid);
+            if constexpr (EXT > 2) chosen_s[kMaxExpertTop + tid] = __float_as_int(__ldcg(p.route_w + tid));
+        }
         chosen = chosen_s;
         __syncthreads();
-        gemv_load_unit<EPI>(p, sc, 0, r.a, chosen);
+        gemv_load_unit<EPI, EXT>(p, sc, 0, r.a, chosen);
         gemv_stage(p, nch, smem, xbytes);
     } else if constexpr (EPI == Epi::ExpertDown) {
         chosen = early_chosen;
@@ -601,7 +728,7 @@ __device__ __forceinline__ void gemv_run(const GemvParams& p, const GemvSched& s
         const float* weight = reinterpret_cast<const float*>(early_chosen + kMaxExpertTop);
         const float inv = 4.0f / (float)p.ffp;
         for (int c = tid; c < 2 * nch; c += kGemvThreads) {            // padded channels are zero
-            const float w = weight[(int)(((float)c + 0.5f) * inv)];
+            const float w = weight[EXT > 2 ? min((int)(((float)c + 0.5f) * inv), p.route.top) : (int)(((float)c + 0.5f) * inv)];
             const float4 v = __ldcg(reinterpret_cast<const float4*>(p.xf) + c);
             reinterpret_cast<float4*>(xw)[c] = make_float4(v.x * w, v.y * w, v.z * w, v.w * w);
         }
@@ -651,12 +778,12 @@ __device__ __forceinline__ void gemv_run(const GemvParams& p, const GemvSched& s
                 const float2 old = j == 0 ? old_first : __ldcg(reinterpret_cast<const float2*>(p.residual + ig * 2));
                 *reinterpret_cast<float2*>(p.residual + ig * 2) = make_float2(old.x + t0, old.y + t1);
             } else {
-                item_epilogue<EPI>(p, ig, t0, t1, best_v, best_i);
+                item_epilogue<EPI, EXT>(p, ig, t0, t1, best_v, best_i, chosen);
             }
         }
     };
     for (int u = 0; u < sc.total; ++u) {
-        if (u > 0) gemv_load_unit<EPI>(p, sc, u, r.a, chosen);       // unit 0 was fetched before the dependency wait
+        if (u > 0) gemv_load_unit<EPI, EXT>(p, sc, u, r.a, chosen);       // unit 0 was fetched before the dependency wait
         compute_unit(u, r.a);
     }
 }
@@ -698,14 +825,15 @@ __global__ void __launch_bounds__(kGemvThreads, 1) gemv_kernel(const GemvParams 
     // which fetches its first weights before its wait.
     if constexpr (EPI != Epi::ExpertUp) pdl_launch_dependents();
     const GemvSched sc = gemv_sched(p, ks, blockIdx.x, gridDim.x);
-    __shared__ int early_s[EPI == Epi::ExpertDown ? 2 * kMaxExpertTop : 1];      // ids | weights
+    __shared__ int early_s[EPI == Epi::ExpertDown ? 2 * kMaxExpertTop + 1 : 1];  // ids | weights (and that of the shared expert)
     if constexpr (EPI == Epi::ExpertDown) {
         if ((int)threadIdx.x < p.route.top) {
             early_s[threadIdx.x] = __ldcg(p.route_id + threadIdx.x);
-            early_s[kMaxExpertTop + threadIdx.x] = __float_as_int(__ldcg(p.route_w + threadIdx.x));
+            early_s[kMaxExpertTop + threadIdx.x] = EXT > 2 && p.weight_input ? __float_as_int(1.0f) : __float_as_int(__ldcg(p.route_w + threadIdx.x));
         }
+        if (EXT > 2 && threadIdx.x == 0 && p.shared_ff > 0) early_s[kMaxExpertTop + p.route.top] = __float_as_int(__ldcg(p.route_w + p.route.top));
         __syncthreads();
-        gemv_load_unit<EPI>(p, sc, 0, regs.a, early_s);
+        gemv_load_unit<EPI, EXT>(p, sc, 0, regs.a, early_s);
     }
     gemv_prefetch<EPI, EXT>(p, sc, regs, gemv_smem, xbytes);
     pdl_wait();
@@ -723,7 +851,10 @@ __global__ void __launch_bounds__(kGemvThreads, 1) gemv_kernel(const GemvParams 
         __syncthreads();
         if (last != 0u && threadIdx.x < 32) {
             route_token(p.out_f, p.route, [&](int k, int e, float w) { p.route_id[k] = e; p.route_w[k] = w; });
-            if (threadIdx.x == 0) *p.route_ticket = 0u;
+            if (threadIdx.x == 0) {
+                if (p.route.shared) p.route_w[p.route.top] = 1.0f / (1.0f + expf(-__ldcg(p.out_f + p.route.experts)));
+                *p.route_ticket = 0u;
+            }
         }
     }
     if constexpr (EPI == Epi::Logits) gemv_publish_best(p, best_v, best_i, bv, bi);
@@ -744,7 +875,7 @@ __host__ __device__ inline size_t gemv_smem_bytes(int K) {      // xs (fp32) | n
     return (size_t)gemv_xbytes(K) + gemv_wbytes(K) + (size_t)(2 * kGemvWarps * 2 + 16) * sizeof(float);
 }
 
-// EXT instantiations: room for the second vector of the AddNorm prologue.
+// EXT instantiations: room for the second vector of a prologue.
 __host__ __device__ inline size_t gemv_ext_smem_bytes(int K) { return (size_t)gemv_ext_off(K) + (size_t)K * 4; }
 
 }  // namespace efm

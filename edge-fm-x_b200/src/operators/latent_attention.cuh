@@ -1,8 +1,8 @@
 // Latent attention over a paged cache: keys and values of all heads are linear in one cached latent c per token,
 //   k[h] = [Wk[h] c | r],  v[h] = Wv[h] c,  score = (q[h] . k[h]) * scale,
 // r a rotated key part shared by the heads; sliding window, an optional extra term exp(sink[h]) in the softmax denominator,
-// heads multiplied by sigmoid(gate).  A cache row is [c: Lc | r: Rc] (Lc, Rc: kv_rank, rot_dim padded to 8 with zeros), normed
-// and rotated.  The projections arrive as one row [query latent: Qp | c: Lc | r: Rc | gate: H * Dv].
+// heads multiplied by sigmoid(gate), one gate per channel or per head.  A cache row is [c: Lc | r: Rc] (Lc, Rc: kv_rank, rot_dim padded to 8 with zeros), normed
+// and rotated.  The projections arrive as one row [query latent: Qp | c: Lc | r: Rc | gate: H * Dv or H].
 //
 //   latent_rows          many rows: norms of the two latents, rotation of r, cache append
 //   latent_rotate_rows   many rows: rotation of the queries' rotated part, in place
@@ -35,7 +35,7 @@ struct LatentShape {
     const __nv_bfloat16* sink;        // [H] or null
     const __nv_bfloat16* wk;          // [H * Dp][Lc]
     const __nv_bfloat16* wv;          // [H * Vp][Lc]
-    int gate;                         // 1: the projections end with the gate
+    int gate;                         // the projections end with a gate per 1: channel, 2: head; 0: no gate
     __host__ __device__ int off_c() const { return Qp; }
     __host__ __device__ int off_r() const { return Qp + Lc; }
     __host__ __device__ int off_gate() const { return Qp + Lc + Rc; }
@@ -62,7 +62,7 @@ __global__ void __launch_bounds__(32 * kLatentRowsPerBlock) latent_rows_kernel(c
         if (lane + 32 * i < n) load8_as_f32(src + 8 * (lane + 32 * i), keep[i]);
     const RowEntry e = plan.of_row(row);
     const int pos = e.pos0 + row - e.row0;
-    for (int i = lane; i < s.rot.dims / 2; i += 32) sincosf((float)pos * s.rot.inv_freq[i], sn + i, cs + i);
+    for (int i = lane; i < s.rot.dims / 2; i += 32) rot_sincos(s.rot, pos, i, sn + i, cs + i);
     float a = 0.f, b = 0.f;                                             // pads are zero
     auto take = [&](int c, const float (&f)[8]) {
         float ss = 0.f;
@@ -505,7 +505,7 @@ __global__ void __launch_bounds__(la::kThreads) latent_attention_kernel(const La
         for (int o = lanes / 2; o > 0; o >>= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
         if (li == 0 && v < v1) {
             if (s.gate) {
-                const TI* gp = p.proj + (size_t)row * p.ld + s.off_gate() + (h0 + h) * s.Dv + c;
+                const TI* gp = p.proj + (size_t)row * p.ld + s.off_gate() + (s.gate == 2 ? h0 + h : (h0 + h) * s.Dv + c);
                 float g;
                 if constexpr (DECODE) g = __ldcg(gp); else g = to_f32(*gp);
                 a *= 1.0f / (1.0f + expf(-g));

@@ -1,0 +1,386 @@
+// Linear attention with a constant decay per head: a state S [D key channels x Dv value channels], fp32,
+//   S_t = a S_{t-1} + k_t v_t^T,   o_t = S_t^T q_t,   q, k, v = silu(projections),
+// then one RMS norm over the channels of all heads, a plain weight, a sigmoid gate and a multiplier.  The projections are four
+// column ranges of a row, each starting at a multiple of 8.
+//
+// Many rows, in chunks of up to 64 tokens of one entry.  A chunk's own contribution does not depend on the state it starts from, so
+// all chunks run at once and only their sums are chained:
+//   linear_chunk_rows    U_c = sum_t a^(n-1-t) k_t v_t^T of every chunk (n tokens)
+//   linear_chain_rows    the states the chunks start from, S_{c+1} = a^n S_c + U_c, in place of the U_c; the last one to the pool
+//   linear_attend_rows   o_t = a^(t+1) S_c^T q_t + sum_{s<=t} a^(t-s) (q_t . k_s) v_s
+//   linear_output_rows   norm, weight, gate, multiplier
+// One row: linear_decode_block, part of the launch of the attention beside it (window_attention.cuh).
+// State pool: [slots][slot_stride] floats, this layer at `offset`, head h at + h * D * Vp, row = key channel (Vp: Dv padded to 4,
+// pads zero).  The powers of the decays come from the host, rounded once.
+#pragma once
+#include "common.cuh"
+#include "row_plan.cuh"
+
+namespace efm {
+
+struct LinearShape {
+    int heads, D, Dv, Vp;
+    int off_q, off_k, off_v, off_g;   // columns of the projections
+    int ld;                           // row length of the projections
+    const float* powers;              // [heads][kLinearChunk + 1]: decay^i
+    const __nv_bfloat16* norm;        // [heads * Dv]
+    float eps, scale;
+    __host__ __device__ int width() const { return heads * Dv; }
+    __host__ __device__ size_t head_floats() const { return (size_t)D * Vp; }
+};
+
+__device__ __forceinline__ float silu_f(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float lin_f32(float v) { return v; }
+__device__ __forceinline__ float lin_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+
+namespace ln {
+constexpr int C = kLinearChunk, kThreads = 256;
+
+// dst[r][0 .. cols) (row stride ld_dst, cols % 4 == 0) = silu of channels [c0, c0 + cols) of a head, zero past `width` and past row n
+template <typename T, typename F>
+__device__ __forceinline__ void stage_rows(float* dst, int ld_dst, const T* src, int ld_src, int c0, int cols, int width, int n, F mul) {
+    const int per = cols / 4;
+    const bool vec = ((reinterpret_cast<uintptr_t>(src) | (uintptr_t)(ld_src * sizeof(T))) & (4 * sizeof(T) - 1)) == 0;
+    for (int i = threadIdx.x; i < C * per; i += kThreads) {
+        const int r = i / per, c = (i - r * per) * 4;
+        float f[4] = {0.f, 0.f, 0.f, 0.f};
+        if (r < n) {
+            const T* p = src + (size_t)r * ld_src + c0 + c;
+            if (vec && c0 + c + 4 <= width) {
+                if constexpr (sizeof(T) == 2) {
+                    const uint2 v = *reinterpret_cast<const uint2*>(p);
+                    f[0] = bf16lo(v.x); f[1] = bf16hi(v.x); f[2] = bf16lo(v.y); f[3] = bf16hi(v.y);
+                } else {
+                    const float4 v = *reinterpret_cast<const float4*>(p);
+                    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+                }
+            } else {
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+                    if (c0 + c + j < width) f[j] = lin_f32(p[j]);
+            }
+            const float m = mul(r);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) f[j] = silu_f(f[j]) * m;
+        }
+        *reinterpret_cast<float4*>(dst + (size_t)r * ld_dst + c) = make_float4(f[0], f[1], f[2], f[3]);
+    }
+}
+__host__ __device__ constexpr size_t chunk_smem_bytes(int RM, int RN) { return (size_t)C * (16 * RM + 16 * RN) * sizeof(float); }
+// queries | keys, afterwards values | products | a slice of the state
+__host__ __device__ inline int attend_key_floats(int D4, int RN) { const int k = C * (D4 + 4), v = C * 16 * RN; return k > v ? k : v; }
+__host__ __device__ inline size_t attend_smem_bytes(int D, int RN) {
+    const int D4 = (D + 3) / 4 * 4;
+    return (size_t)(C * (D4 + 4) + attend_key_floats(D4, RN) + C * (C + 4) + 32 * 16 * RN) * sizeof(float);
+}
+}  // namespace ln
+
+// grid (chunks, heads, tiles of the state); a tile is 16 RM key channels x 16 RN value channels.  ws: [chunks][heads][D][Vp]
+template <typename T, int RM, int RN>
+__global__ void __launch_bounds__(ln::kThreads) linear_chunk_rows_kernel(const T* __restrict__ proj, float* __restrict__ ws, const LinearShape s, const RowPlan plan) {
+    using namespace ln;
+    constexpr int TM = 16 * RM, TN = 16 * RN;
+    extern __shared__ __align__(16) float ln_smem[];
+    float *ks = ln_smem, *vs = ln_smem + C * TM;
+    RowEntry e;
+    int t0;
+    if (!locate_chunk<C>(plan, blockIdx.x, e, t0)) return;
+    const int h = blockIdx.y, n = min(C, e.n - t0), tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+    const int tiles_n = (s.Vp + TN - 1) / TN, d0 = blockIdx.z / tiles_n * TM, v0 = blockIdx.z % tiles_n * TN;
+    const float* pw = s.powers + (size_t)h * (C + 1);
+    const T* row = proj + (size_t)(e.row0 + t0) * s.ld;
+    stage_rows(ks, TM, row + s.off_k + h * s.D, s.ld, d0, TM, s.D, n, [&](int r) { return pw[n - 1 - r]; });
+    stage_rows(vs, TN, row + s.off_v + h * s.Dv, s.ld, v0, TN, s.Dv, n, [](int) { return 1.0f; });
+    __syncthreads();
+    float acc[RM][RN];
+#pragma unroll
+    for (int i = 0; i < RM; ++i)
+#pragma unroll
+        for (int j = 0; j < RN; ++j) acc[i][j] = 0.f;
+#pragma unroll 2
+    for (int t = 0; t < n; ++t) {
+        float a[RM], b[RN];
+#pragma unroll
+        for (int i = 0; i < RM; i += 4) *reinterpret_cast<float4*>(a + i) = *reinterpret_cast<const float4*>(ks + t * TM + i * 16 + ty * 4);
+#pragma unroll
+        for (int j = 0; j < RN; j += 4) *reinterpret_cast<float4*>(b + j) = *reinterpret_cast<const float4*>(vs + t * TN + j * 16 + tx * 4);
+#pragma unroll
+        for (int i = 0; i < RM; ++i)
+#pragma unroll
+            for (int j = 0; j < RN; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+    }
+    float* out = ws + ((size_t)blockIdx.x * s.heads + h) * s.head_floats();
+#pragma unroll
+    for (int i = 0; i < RM; ++i) {
+        const int d = d0 + (i & ~3) * 16 + ty * 4 + (i & 3);
+        if (d >= s.D) continue;
+#pragma unroll
+        for (int j = 0; j < RN; j += 4) {
+            const int v = v0 + j * 16 + tx * 4;
+            if (v < s.Vp) *reinterpret_cast<float4*>(out + (size_t)d * s.Vp + v) = make_float4(acc[i][j], acc[i][j + 1], acc[i][j + 2], acc[i][j + 3]);
+        }
+    }
+}
+
+// grid (groups of 256 x 4 state numbers, entries)
+__global__ void __launch_bounds__(256) linear_chain_rows_kernel(float* __restrict__ ws, float* __restrict__ pool, size_t slot_stride, size_t offset,
+                                                                const LinearShape s, const RowPlan plan) {
+    constexpr int C = kLinearChunk, U = 8;
+    const size_t all = s.heads * s.head_floats(), i = ((size_t)blockIdx.x * 256 + threadIdx.x) * 4;
+    if (i >= all) return;
+    const RowEntry e = plan.entry(blockIdx.y);
+    const float* pw = s.powers + i / s.head_floats() * (C + 1);
+    int chunk0 = 0;
+    for (int k = 0; k < (int)blockIdx.y; ++k) chunk0 += (plan.entry(k).n + C - 1) / C;
+    const int n_chunks = (e.n + C - 1) / C;
+    float* st = pool + (size_t)e.state * slot_stride + offset + i;
+    float* w = ws + (size_t)chunk0 * all + i;
+    float4 S = e.pos0 > 0 ? *reinterpret_cast<const float4*>(st) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float full = pw[C], last = pw[e.n - (n_chunks - 1) * C];
+    for (int c0 = 0; c0 < n_chunks; c0 += U) {
+        float4 u[U];
+#pragma unroll
+        for (int k = 0; k < U; ++k)
+            if (c0 + k < n_chunks) u[k] = *reinterpret_cast<const float4*>(w + (size_t)(c0 + k) * all);
+#pragma unroll
+        for (int k = 0; k < U; ++k)
+            if (c0 + k < n_chunks) {
+                *reinterpret_cast<float4*>(w + (size_t)(c0 + k) * all) = S;
+                const float a = c0 + k == n_chunks - 1 ? last : full;
+                S.x = fmaf(a, S.x, u[k].x); S.y = fmaf(a, S.y, u[k].y); S.z = fmaf(a, S.z, u[k].z); S.w = fmaf(a, S.w, u[k].w);
+            }
+    }
+    *reinterpret_cast<float4*>(st) = S;
+}
+
+// grid (chunks, heads, tiles of 16 RN value channels)
+template <typename T, int RN>
+__global__ void __launch_bounds__(ln::kThreads) linear_attend_rows_kernel(const T* __restrict__ proj, const float* __restrict__ ws, float* __restrict__ o, int ld_o,
+                                                                          const LinearShape s, const RowPlan plan) {
+    using namespace ln;
+    constexpr int TN = 16 * RN, LP = C + 4;
+    extern __shared__ __align__(16) float ln_smem[];
+    RowEntry e;
+    int t0;
+    if (!locate_chunk<C>(plan, blockIdx.x, e, t0)) return;
+    const int h = blockIdx.y, v0 = blockIdx.z * TN, n = min(C, e.n - t0), tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+    const int D4 = (s.D + 3) / 4 * 4, LD = D4 + 4;
+    float *qs = ln_smem, *ks = qs + C * LD, *vs = ks, *ps = ks + attend_key_floats(D4, RN), *ss = ps + C * LP;
+    __shared__ float pw[C + 1];
+    if (tid <= C) pw[tid] = s.powers[(size_t)h * (C + 1) + tid];
+    const T* row = proj + (size_t)(e.row0 + t0) * s.ld;
+    auto one = [](int) { return 1.0f; };
+    stage_rows(qs, LD, row + s.off_q + h * s.D, s.ld, 0, D4, s.D, n, one);
+    stage_rows(ks, LD, row + s.off_k + h * s.D, s.ld, 0, D4, s.D, n, one);
+    __syncthreads();
+    {   // products of queries and keys, decayed; row ty + 16 i, column tx + 16 j
+        float p[4][4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) p[i][j] = 0.f;
+        for (int d = 0; d < D4; d += 4) {
+            float4 a[4], b[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) a[i] = *reinterpret_cast<const float4*>(qs + (ty + 16 * i) * LD + d);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) b[j] = *reinterpret_cast<const float4*>(ks + (tx + 16 * j) * LD + d);
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    p[i][j] = fmaf(a[i].x, b[j].x, p[i][j]); p[i][j] = fmaf(a[i].y, b[j].y, p[i][j]);
+                    p[i][j] = fmaf(a[i].z, b[j].z, p[i][j]); p[i][j] = fmaf(a[i].w, b[j].w, p[i][j]);
+                }
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const int t = ty + 16 * i, u = tx + 16 * j;
+                ps[t * LP + u] = u <= t ? p[i][j] * pw[t - u] : 0.f;
+            }
+    }
+    __syncthreads();
+    stage_rows(vs, TN, row + s.off_v + h * s.Dv, s.ld, v0, TN, s.Dv, n, one);      // in place of the keys
+    float acc[4][RN];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < RN; ++j) acc[i][j] = 0.f;
+    // four rows of b (row stride TN) times four columns of a (row stride lda)
+    auto step = [&](const float* a, int lda, const float* b) {
+        float x[4][4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(x[i]) = *reinterpret_cast<const float4*>(a + (ty + 16 * i) * lda);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            float y[RN];
+#pragma unroll
+            for (int j = 0; j < RN; j += 4) *reinterpret_cast<float4*>(y + j) = *reinterpret_cast<const float4*>(b + k * TN + j * 16 + tx * 4);
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < RN; ++j) acc[i][j] = fmaf(x[i][k], y[j], acc[i][j]);
+        }
+    };
+    const float* S = ws + ((size_t)blockIdx.x * s.heads + h) * s.head_floats();
+    if (e.pos0 + t0 > 0)                                               // the first chunk of a sequence starts from zero
+        for (int d0 = 0; d0 < D4; d0 += 32) {
+            for (int i = tid; i < 32 * TN / 4; i += kThreads) {
+                const int r = i / (TN / 4), c = (i - r * (TN / 4)) * 4;
+                *reinterpret_cast<float4*>(ss + r * TN + c) = d0 + r < s.D && v0 + c < s.Vp ? *reinterpret_cast<const float4*>(S + (size_t)(d0 + r) * s.Vp + v0 + c)
+                                                                                            : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+            __syncthreads();
+            for (int d = 0; d < min(32, D4 - d0); d += 4) step(qs + d0 + d, LD, ss + d * TN);
+            __syncthreads();
+        }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < RN; ++j) acc[i][j] *= pw[ty + 16 * i + 1];
+    __syncthreads();
+    for (int u = 0; u < n; u += 4) step(ps + u, LP, vs + u * TN);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int t = ty + 16 * i;
+        if (t >= n) continue;
+        float* dst = o + (size_t)(e.row0 + t0 + t) * ld_o + h * s.Dv;
+#pragma unroll
+        for (int j = 0; j < RN; j += 4) {
+            const int v = v0 + j * 16 + tx * 4;
+            if ((s.Dv & 3) == 0) {
+                if (v < s.Dv) *reinterpret_cast<float4*>(dst + v) = make_float4(acc[i][j], acc[i][j + 1], acc[i][j + 2], acc[i][j + 3]);
+            } else {
+#pragma unroll
+                for (int k = 0; k < 4; ++k)
+                    if (v + k < s.Dv) dst[v + k] = acc[i][j + k];
+            }
+        }
+    }
+}
+
+// out[row][0 .. width) = rms(o) * norm * sigmoid(gate) * scale, columns up to `cols` zero.  One block per row; ld_o, cols multiples
+// of 4.  The first 1024 * KEEP channels stay in registers.
+template <typename T>
+__global__ void __launch_bounds__(256) linear_output_rows_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ proj, T* __restrict__ out, int ld_out,
+                                                                 int cols, const LinearShape s) {
+    constexpr int KEEP = 4;
+    __shared__ float part[8];
+    const int row = blockIdx.x, tid = threadIdx.x, n = s.width();
+    const float* src = o + (size_t)row * ld_o;
+    const T* gate = proj + (size_t)row * s.ld + s.off_g;
+    T* dst = out + (size_t)row * ld_out;
+    auto load = [&](int c) {
+        float4 v = *reinterpret_cast<const float4*>(src + c);           // ld_o covers the pads
+        if (c + 4 > n) { if (c >= n) v.x = 0.f; if (c + 1 >= n) v.y = 0.f; if (c + 2 >= n) v.z = 0.f; v.w = 0.f; }
+        return v;
+    };
+    float4 keep[KEEP];
+    float ss = 0.f;
+    auto square = [&](const float4& v) { ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss)))); };
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+        if (4 * (tid + 256 * i) < cols) keep[i] = load(4 * (tid + 256 * i));
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+        if (4 * (tid + 256 * i) < cols) square(keep[i]);
+    for (int c = 4 * (tid + 256 * KEEP); c < cols; c += 1024) square(load(c));
+    ss = warp_sum(ss);
+    if ((tid & 31) == 0) part[tid >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ss += part[i];
+    const float inv = s.scale / sqrtf(ss / (float)n + s.eps);
+    auto emit = [&](int c, const float4& v) {
+        const float f[4] = {v.x, v.y, v.z, v.w};
+        float g[4], w[4], r[4];
+        const uint2 wv = *reinterpret_cast<const uint2*>(s.norm + c);     // padded with zeros
+        w[0] = bf16lo(wv.x); w[1] = bf16hi(wv.x); w[2] = bf16lo(wv.y); w[3] = bf16hi(wv.y);
+        if constexpr (sizeof(T) == 2) {
+            const uint2 x = *reinterpret_cast<const uint2*>(gate + c);
+            g[0] = bf16lo(x.x); g[1] = bf16hi(x.x); g[2] = bf16lo(x.y); g[3] = bf16hi(x.y);
+        } else {
+            const float4 x = *reinterpret_cast<const float4*>(gate + c);
+            g[0] = x.x; g[1] = x.y; g[2] = x.z; g[3] = x.w;
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) r[j] = f[j] * inv * w[j] / (1.0f + expf(-g[j]));
+        if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2*>(dst + c) = make_uint2(pack_bf16(r[0], r[1]), pack_bf16(r[2], r[3]));
+        else *reinterpret_cast<float4*>(dst + c) = make_float4(r[0], r[1], r[2], r[3]);
+    };
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i)
+        if (4 * (tid + 256 * i) < cols) emit(4 * (tid + 256 * i), keep[i]);
+    for (int c = 4 * (tid + 256 * KEEP); c < cols; c += 1024) emit(c, load(c));
+}
+
+// ---- one row -----------------------------------------------------------------------------------------------------------
+namespace ln {
+constexpr int kCols = 64;             // value channels per decode block
+struct DecodeSmem { float q[256], k[256], red[16][kCols]; };
+inline int decode_units(const LinearShape& s) { return s.heads * ((s.Dv + kCols - 1) / kCols); }
+}  // namespace ln
+
+struct LinearDecodeParams {
+    LinearShape s;
+    float* pool;                      // this layer's state of the sequence
+    float* out;                       // [heads * Dv], before the norm
+    int units;                        // blocks: (head, 64 value channels); 0: no linear attention in this launch
+};
+
+// One block of 256 threads: 16 threads per state row (4 channels each), 16 rows at a time.  The state is read before the
+// dependency wait when `early`.
+__device__ __forceinline__ void linear_decode_block(const LinearDecodeParams& p, int unit, const float* proj, const DecodeState* state, int max_tokens, int early,
+                                                    ln::DecodeSmem& sm) {
+    using namespace ln;
+    constexpr int NR = 16;
+    const LinearShape& s = p.s;
+    const int slices = (s.Dv + kCols - 1) / kCols, h = unit / slices, tid = threadIdx.x, rg = tid >> 4, c = unit % slices * kCols + (tid & 15) * 4;
+    const bool act = c < s.Vp;
+    float* S = p.pool + h * s.head_floats() + c;
+    if (!early) { pdl_wait(); pdl_launch_dependents(); }
+    const int kv_len = (int)state->kv_len;
+    const bool ok = kv_len > 0 && kv_len <= max_tokens, fresh = kv_len <= 1;
+    float4 r[NR];
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+        const int d = rg + 16 * i;
+        r[i] = act && d < s.D && !fresh ? __ldcg(reinterpret_cast<const float4*>(S + (size_t)d * s.Vp)) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    const float a = s.powers[(size_t)h * (kLinearChunk + 1) + 1];
+    if (early) { pdl_wait(); pdl_launch_dependents(); }
+    float v[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) v[j] = c + j < s.Dv ? silu_f(__ldcg(proj + s.off_v + h * s.Dv + c + j)) : 0.f;
+    for (int d = tid; d < s.D; d += 256) {
+        sm.q[d] = silu_f(__ldcg(proj + s.off_q + h * s.D + d));
+        sm.k[d] = silu_f(__ldcg(proj + s.off_k + h * s.D + d));
+    }
+    __syncthreads();
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+        const int d = rg + 16 * i;
+        if (d < s.D) {
+            const float k = sm.k[d], q = sm.q[d];
+            r[i].x = fmaf(a, r[i].x, k * v[0]); r[i].y = fmaf(a, r[i].y, k * v[1]);
+            r[i].z = fmaf(a, r[i].z, k * v[2]); r[i].w = fmaf(a, r[i].w, k * v[3]);
+            if (act && ok) *reinterpret_cast<float4*>(S + (size_t)d * s.Vp) = r[i];
+            o.x = fmaf(q, r[i].x, o.x); o.y = fmaf(q, r[i].y, o.y); o.z = fmaf(q, r[i].z, o.z); o.w = fmaf(q, r[i].w, o.w);
+        }
+    }
+    *reinterpret_cast<float4*>(&sm.red[rg][(tid & 15) * 4]) = o;
+    __syncthreads();
+    if (tid < kCols) {
+        float t = 0.f;
+#pragma unroll
+        for (int g = 0; g < 16; ++g) t += sm.red[g][tid];
+        const int ch = unit % slices * kCols + tid;
+        if (ch < s.Dv) p.out[h * s.Dv + ch] = t;
+    }
+}
+
+}  // namespace efm

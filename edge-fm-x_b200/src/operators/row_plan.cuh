@@ -7,6 +7,7 @@
 namespace efm {
 
 constexpr int kPageTokens = 64;       // cache rows per page
+constexpr int kLinearChunk = 64;      // tokens per chunk of linear attention
 
 struct RowEntry {
     int32_t row0, n, pos0;            // rows [row0, row0 + n) hold positions [pos0, pos0 + n) of the sequence
@@ -33,5 +34,22 @@ struct RowPlan {
     }
 #endif
 };
+
+#ifdef __CUDACC__
+// Chunk `idx` of the pass, entries cut into chunks of C tokens each -> entry, first token; false past the last chunk.
+template <int C>
+__device__ __forceinline__ bool locate_chunk(const RowPlan& plan, int idx, RowEntry& e, int& t0) {
+    int at = 0;
+    for (int i = 0; i < plan.n_entries; ++i) {
+        e = plan.entry(i);
+        const int n = (e.n + C - 1) / C;
+        if (idx < at + n) { t0 = (idx - at) * C; return true; }
+        at += n;
+    }
+    return false;
+}
+#endif
+// chunks of a pass, at most
+inline int max_chunks(const RowPlan& plan, int C) { return plan.n_entries == 1 ? (plan.rows + C - 1) / C : plan.rows / C + plan.n_entries; }
 
 }  // namespace efm

@@ -1,7 +1,7 @@
 // Causal softmax attention over a paged cache with a sliding window, kept first tokens and per-head score modification:
 //   score(i, j) = (q_i . k_j) * scale * temp[h] - slope_h * (i - j),   0 <= i - j < window (window 0: no lower bound) or j < keep
-// with slope_h = 2^(-8 (h + 1) / H), q and k RMS-normalised per head (with or without a weight) and then rotated before they
-// are used / cached, value width free.  A weightless norm commutes with the rotation, which keeps a head's length.
+// with slope_h = 2^(-8 (h + 1) / H), q and k RMS-normalised per head (with or without a weight, or not at all) and then rotated
+// before they are used / cached, value width free.  A weightless norm commutes with the rotation, which keeps a head's length.
 // Cache: per layer a K pool [pages * 64][kv_heads][Dp] and a V pool [pages * 64][kv_heads][Vp], channels zero-padded to
 // Dp / Vp (multiples of 64); a sequence's pages are listed in a page table.  TC = bf16 or fp32 (the all-32-bit mode).
 //
@@ -16,6 +16,7 @@
 #include <utility>
 
 #include "common.cuh"
+#include "linear_attention.cuh"
 #include "rotary.cuh"
 #include "row_plan.cuh"
 
@@ -26,15 +27,17 @@ struct WindowAttnShape {
     int window;                       // 0: full causal
     int keep;                         // first tokens that stay visible (with a window)
     int bias;                         // 1: distance bias
+    int qk_norm;                      // 0: q and k as they are
     float scale, eps;
+    float out_scale;                  // of the result
     const __nv_bfloat16* q_norm;      // [D], null: norm without a weight
     const __nv_bfloat16* k_norm;      // [D]
     const __nv_bfloat16* temp;        // [H], null: 1
     RotShape rot;
     // tensor-core form with a shared key part only: extra term exp(sink[h]) of the softmax denominator, and heads multiplied by sigmoid(gate)
     const __nv_bfloat16* sink;        // [H], null: none
-    const __nv_bfloat16* gate;        // [T][H * Dv] with row stride gate_ld, null: none
-    int gate_ld;
+    const __nv_bfloat16* gate;        // [T][H * Dv], or (gate_heads) [T][H], with row stride gate_ld, null: none
+    int gate_ld, gate_heads;
 };
 
 __device__ __forceinline__ float head_multiplier(const WindowAttnShape& s, int h) {
@@ -118,7 +121,7 @@ __global__ void __launch_bounds__(256, 4) qk_scatter_rows_kernel(const TI* __res
         for (int j = 0; j < 8; ++j) ss = fmaf(f[j], f[j], ss);
         for (int x = lanes / 2; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
         if (qk) {
-            const float inv = 1.0f / sqrtf(ss / (float)s.D + s.eps);
+            const float inv = s.qk_norm ? 1.0f / sqrtf(ss / (float)s.D + s.eps) : 1.0f;
 #pragma unroll
             for (int j = 0; j < 8; ++j) f[j] *= inv;                   // channels past D are zero
             if (w != nullptr) {
@@ -262,7 +265,7 @@ __global__ void __launch_bounds__(256) window_attention_rows_kernel(const TQ* __
         }
     }
     if (r >= nq) return;
-    const float inv = l > 0.f ? 1.0f / l : 0.f;
+    const float inv = l > 0.f ? s.out_scale / l : 0.f;
     TO* dst = out + (size_t)(e.row0 + r0 + r) * ld_out + (size_t)h * s.Dv;
 #pragma unroll
     for (int n = 0; n < 4; ++n)
@@ -302,6 +305,7 @@ struct WindowDecodeParams {
     DecodeState* state;
     float* out;                       // [H * Dv]
     int early;                        // 1: state and the older cache rows may be read before the dependency wait
+    LinearDecodeParams lin;           // linear attention beside this one: its blocks follow in grid.y
 };
 
 // 8 channels of a cache row as fp32
@@ -329,8 +333,9 @@ template <> struct Row4<float> {
 };
 
 // grid (splits = cluster size, kv_heads * head blocks); the visible keys (kept first tokens, then the window) are numbered in
-// order and dealt out evenly, block `split` walks its share in tiles of 64.  VM: upper bound of Dp and Vp.
-template <typename TC, int VM, bool ROT>
+// order and dealt out evenly, block `split` walks its share in tiles of 64.  VM: upper bound of Dp and Vp.  Further rows of
+// clusters (LIN) compute the linear attention that reads the same projections.
+template <typename TC, int VM, bool ROT, bool LIN>
 __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(const WindowDecodeParams<TC> p) {
     using namespace wd;
     constexpr int KC = VM / 32;                                        // 8-channel chunks per thread and key (4 threads per key)
@@ -341,6 +346,15 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int split = blockIdx.x, n_splits = gridDim.x;
     const int group = s.H / s.G, hb = (group + kHeads - 1) / kHeads;
+    if constexpr (LIN) {
+        if ((int)blockIdx.y >= s.G * hb) {                             // a whole cluster
+            const int unit = ((int)blockIdx.y - s.G * hb) * n_splits + split;
+            if (unit < p.lin.units)
+                linear_decode_block(p.lin, unit, p.qkv, p.state, p.max_pages * kPageTokens, p.early, *reinterpret_cast<ln::DecodeSmem*>(wd_smem));
+            else { pdl_wait(); pdl_launch_dependents(); }
+            return;
+        }
+    }
     const int g = blockIdx.y / hb, h0 = g * group + (blockIdx.y % hb) * kHeads, nh = min(kHeads, (g + 1) * group - h0);
     const int key = tid >> 2, part = tid & 3;                          // score phase
     const int tpr = s.Vp / 4, kg = kThreads / tpr, dpart = tid % tpr, tg = tid / tpr;     // P.V phase: 4 channels per thread
@@ -399,7 +413,7 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
         }
 #pragma unroll
         for (int i = 0; i < VM / 32; ++i) ss = fmaf(f[i], f[i], ss);
-        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)s.D + s.eps);
+        const float inv = s.qk_norm ? 1.0f / sqrtf(warp_sum(ss) / (float)s.D + s.eps) : 1.0f;
 #pragma unroll
         for (int i = 0; i < VM / 32; ++i) {
             const int d = lane + 32 * i;
@@ -558,7 +572,7 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
             num = fmaf(w, sm.rout[r * share + i], num);
             den = fmaf(w, sm.rl[r][h], den);
         }
-        p.out[(size_t)(h0 + h) * s.Dv + d] = den > 0.f ? num / den : 0.f;
+        p.out[(size_t)(h0 + h) * s.Dv + d] = den > 0.f ? s.out_scale * (num / den) : 0.f;
     }
 }
 

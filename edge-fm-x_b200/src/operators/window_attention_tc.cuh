@@ -5,7 +5,8 @@
 // place of the page in a workspace of keys and values expanded for this pass (latent attention).
 // Keys may come from two tensors: DP channels per kv head, and RP more that all heads share (a rotated part); the query rows
 // are split the same way.  Channels that a tensor does not have are filled with zeros by TMA.
-// Block = 128 rows of one entry x one head, 256 threads.  Rows of the tile that belong to the next entry are computed and
+// Block = 128 rows of one entry x one head x (grid.z) VP value channels, 256 threads.  Wider values take several blocks, each of
+// which computes the scores for itself.  Rows of the tile that belong to the next entry are computed and
 // not stored.  The weights enter P V as a bf16 pair high + low (16 bits of mantissa), written straight into tensor memory.
 // Every mbarrier wait is bounded and raises *error.
 #pragma once
@@ -84,6 +85,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int row = (warp & 3) * 32 + lane, hf = warp >> 2;       // TMEM lane = query row; which half of the columns
+    const int v0 = blockIdx.z * VP;                               // first value channel
     const int bx = (int)gridDim.x - 1 - (int)blockIdx.x, h = blockIdx.y, g = h / (s.H / s.G);     // late rows first: they see most keys
     RowEntry e;
     int r0;
@@ -139,7 +141,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
         last_v = tile;
         mbar_expect_tx(vfull, C::V_BYTES);
 #pragma unroll
-        for (int b = 0; b < C::VB; ++b) tma_load_3d(sV + b * (BN * 128), &maps.v, b * 64, g, pages[tile], vfull);
+        for (int b = 0; b < C::VB; ++b) tma_load_3d(sV + b * (BN * 128), &maps.v, v0 + b * 64, g, pages[tile], vfull);
     };
     auto issue_s = [&](int buf) {
 #pragma unroll
@@ -250,15 +252,17 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
         up = at::ex2(m - mx);
         L = fmaf(L, up, at::ex2(sk - mx));
     }
-    const float inv = L > 0.f ? up / L : 0.f;
+    float inv = L > 0.f ? s.out_scale * up / L : 0.f;
     if (valid && *abort_s == 0) {
         __nv_bfloat16* dst = out + (size_t)(e.row0 + r0 + row) * ld_out + (size_t)h * s.Dv;
         const bool vec = (s.Dv & 7) == 0;                        // ld_out is a multiple of 8
-        if (RP > 0 && s.gate != nullptr) {
+        if (RP > 0 && s.gate != nullptr && s.gate_heads) {
+            inv *= 1.0f / (1.0f + expf(-__bfloat162float(s.gate[(size_t)(e.row0 + r0 + row) * s.gate_ld + h])));
+        } else if (RP > 0 && s.gate != nullptr) {
             const __nv_bfloat16* gt = s.gate + (size_t)(e.row0 + r0 + row) * s.gate_ld + (size_t)h * s.Dv;
 #pragma unroll
             for (int i = 0; i < C::HALF; i += 8) {
-                const int d = hf * C::HALF + i;
+                const int d = v0 + hf * C::HALF + i;
                 float f[8];
                 if (vec && d + 8 <= s.Dv) unpack8(ld_cached(gt + d), f);
                 else
@@ -270,7 +274,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
         }
 #pragma unroll
         for (int i = 0; i < C::HALF; i += 8) {
-            const int d = hf * C::HALF + i;
+            const int d = v0 + hf * C::HALF + i;
             if (vec && d + 8 <= s.Dv)
                 *reinterpret_cast<uint4*>(dst + d) = make_uint4(pack_bf16(o[i] * inv, o[i + 1] * inv), pack_bf16(o[i + 2] * inv, o[i + 3] * inv),
                                                                 pack_bf16(o[i + 4] * inv, o[i + 5] * inv), pack_bf16(o[i + 6] * inv, o[i + 7] * inv));

@@ -360,28 +360,35 @@ EFM_API efm_status efm_b200_vit_encode(efm_b200_vit* vit, const void* pixels, in
                                        int32_t out_mem);
 
 /* ---- layered decoders ---------------------------------------------------------------------
- * A decoder described layer by layer: every layer names its mixer (softmax attention, latent attention or the generalised
- * delta rule), the mixer's sizes and an optional feed-forward (dense or routed experts); sublayer outputs are
- * RMS-normalised before the residual add, and with EFM_NORM_SANDWICH sublayer inputs are normalised too; an optional
- * per-layer token input follows.  A span of layers may run several times in a row with the same weights, every pass with
+ * A decoder described layer by layer: every layer names its mixer (softmax attention, latent attention, the generalised
+ * delta rule, or softmax attention and decayed linear attention side by side), the mixer's sizes and an optional
+ * feed-forward (dense or routed experts).  Sublayer outputs are RMS-normalised before the residual add, with
+ * EFM_NORM_SANDWICH sublayer inputs too; with EFM_NORM_INPUT only the inputs are normalised, by tanh(alpha x) w + b.  An
+ * optional per-layer token input follows.  A span of layers may run several times in a row with the same weights, every pass with
  * its own cache and state.  (No counterpart in the reference.)  Such a context serves the same calls as the text tower
  * (set_weight, finalize_weights, prefill, decode_begin, decode_steps, read_tokens, read_logits, ...) and, in addition,
  * batched steps over a paged cache: one pool of 64-token pages per attention layer run and one pool of recurrent state
  * slots, handed out by the caller (who maps page numbers to sequences).
  *
- * Tensor names: embed, side.embed, final.norm, head and, for layer i, l<i>.norm1 / norm2 (sandwich: before the sublayers,
- * l<i>.norm1b / norm2b behind them), l<i>.mix.{q,k,v,o} with, as the layer asks, {q.b,k.b,v.b}, {q.norm,k.norm}, temp
+ * Tensor names: embed, side.embed, final.norm, head (untied) and, for layer i, l<i>.norm1 / norm2 (sandwich: before the
+ * sublayers, l<i>.norm1b / norm2b behind them; input norms: each with .alpha and .b, final.norm too), l<i>.mix.{q,k,v,o} with, as the layer asks, {q.b,k.b,v.b}, {q.norm,k.norm}, temp
  * (attention), l<i>.mix.{dq,dq.norm,uq,dkv,dkv.norm,uk,uv,o} with sink, g (latent attention) or
- * l<i>.mix.{r,k,v,g,a,a.b,w1,w2,w0,norm,o} (delta rule), l<i>.mlp.{up,down,act} (dense) or l<i>.mlp.router and
- * l<i>.mlp.e<j>.{gate,up,down} (experts), l<i>.side.{gate,proj,norm}; bf16. */
-enum { EFM_MIXER_ATTENTION = 0, EFM_MIXER_GENERAL_DELTA = 1, EFM_MIXER_LATENT_ATTENTION = 2 };
+ * l<i>.mix.{r,k,v,g,a,a.b,w1,w2,w0,norm,o} (delta rule) or l<i>.mix.left.* (as attention) and
+ * l<i>.mix.right.{q,k,v,g,norm,o} (parallel), l<i>.mlp.{up,down} with act (dense) or l<i>.mlp.router,
+ * l<i>.mlp.e<j>.{gate,up,down} and, with a shared expert, l<i>.mlp.shared.{gate,up,down,sg} (experts),
+ * l<i>.side.{gate,proj,norm}; bf16. */
+enum { EFM_MIXER_ATTENTION = 0, EFM_MIXER_GENERAL_DELTA = 1, EFM_MIXER_LATENT_ATTENTION = 2, EFM_MIXER_PARALLEL = 3 };
 enum { EFM_PAGE_TOKENS = 64 };
-enum { EFM_QK_NORM_WEIGHTED = 0, EFM_QK_NORM_PLAIN = 1 };            /* RMS norm of q and k per head, with / without a weight */
+enum { EFM_QK_NORM_WEIGHTED = 0, EFM_QK_NORM_PLAIN = 1, EFM_QK_NORM_NONE = 2 };   /* RMS norm of q and k per head, with / without a weight */
 enum { EFM_ROT_NONE = 0, EFM_ROT_HALF = 1, EFM_ROT_PAIRS = 2 };      /* channel i turns with i + dims / 2; 2 i with 2 i + 1 */
-enum { EFM_NORM_OUTPUT = 0, EFM_NORM_SANDWICH = 1 };
+enum { EFM_NORM_OUTPUT = 0, EFM_NORM_SANDWICH = 1, EFM_NORM_INPUT = 2 };
+enum { EFM_GATE_NONE = 0, EFM_GATE_CHANNELS = 1, EFM_GATE_HEADS = 2 };   /* sigmoid gate per output channel / per head */
+enum { EFM_ACT_POLYNORM = 0, EFM_ACT_RELU2 = 1 };                    /* dense feed-forward */
+enum { EFM_GLU_SILU = 0, EFM_GLU_CLAMPED = 1 };   /* experts: silu(g) u; g' sigmoid(1.702 g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit) */
+enum { EFM_SCORE_SOFTMAX = 0, EFM_SCORE_SIGMOID = 1 };               /* router scores */
 
 typedef struct efm_decoder_layer {
-    int32_t mixer;                /* EFM_MIXER_* */
+    int32_t mixer;                /* EFM_MIXER_*; parallel: the attention fields describe its left half */
     int32_t heads;
     int32_t kv_heads;             /* attention only */
     int32_t dim;                  /* per-head key channels (delta rule: value channels too; latent: the unrotated ones), <= 256 */
@@ -390,7 +397,7 @@ typedef struct efm_decoder_layer {
     int32_t distance_bias;        /* attention: 1 = subtract 2^(-8 (h+1) / heads) * (i - j) from the score of head h */
     float scale;                  /* both attentions: score multiplier */
     int32_t decay_rank;           /* delta rule: rows of w1, <= 512 */
-    int32_t ff;                   /* dense feed-forward (PolyNorm) width, 0: none */
+    int32_t ff;                   /* dense feed-forward width, 0: none */
     int32_t keep_first;           /* attention with a window: the first keep_first tokens stay visible */
     int32_t qk_norm;              /* attention: EFM_QK_NORM_* */
     int32_t head_temp;            /* attention: 1 = a learned score multiplier per head */
@@ -400,12 +407,27 @@ typedef struct efm_decoder_layer {
     float rot_base;               /* pair i of position p turns by p * rot_base^(-2 i / rot_dims) */
     int32_t q_rank, kv_rank;      /* latent: widths of the query latent and of the cached key / value latent (<= 1024) */
     int32_t sink;                 /* latent: 1 = a learned extra term exp(sink[h]) in the softmax denominator */
-    int32_t out_gate;             /* latent: 1 = heads multiplied by sigmoid(W_g h) */
+    int32_t out_gate;             /* latent: EFM_GATE_* */
     int32_t experts;              /* routed feed-forward: number of experts (<= 512), 0: none */
     int32_t expert_ff;            /* width of an expert */
     int32_t expert_top;           /* experts a token uses (<= 32) */
     int32_t expert_groups;        /* equal groups of neighbouring experts (<= 64) ... */
     int32_t expert_groups_kept;   /* ... of which those with the best single scores stay open */
+    /* rotation scaled to a longer context (YaRN): pairs that turn at most rot_slow times within rot_original positions are
+     * slowed down by rot_factor, those that turn more than rot_fast times keep their frequency, a ramp lies between, and
+     * cos and sin are multiplied by 0.1 ln(rot_factor) + 1.  rot_factor 0: off */
+    float rot_factor, rot_original, rot_fast, rot_slow;
+    int32_t ff_act;               /* EFM_ACT_* */
+    int32_t expert_glu;           /* EFM_GLU_* */
+    float expert_limit;
+    int32_t expert_score;         /* EFM_SCORE_* */
+    int32_t expert_weight_input;  /* 1: a choice's weight multiplies the expert's input, 0: its output */
+    int32_t shared_ff;            /* expert every token uses, output multiplied by sigmoid(W_sg h): width, 0: none */
+    float shared_limit;
+    /* parallel: S_t = decay_h S_{t-1} + silu(k_t) silu(v_t)^T, o_t = S_t^T silu(q_t), RMS norm over all heads, weight, gate */
+    int32_t linear_heads, linear_dim, linear_vdim;    /* dims <= 256 */
+    float mix_scale, linear_scale;                    /* multipliers of the two halves */
+    const double* linear_decay;                       /* [linear_heads], read by efm_b200_decoder_create */
 } efm_decoder_layer;
 
 typedef struct efm_decoder_desc {
@@ -422,6 +444,10 @@ typedef struct efm_decoder_desc {
     int32_t norm_layout;          /* EFM_NORM_* */
     float embed_scale;            /* embedding rows are multiplied by this */
     int32_t loop_start, loop_stop, loop_times;   /* layers [start, stop) run `times` times in a row; times <= 1: once */
+    float residual_mult;          /* EFM_NORM_INPUT: sublayer outputs are multiplied by this */
+    int32_t tied_head;            /* 1: the head is the embedding table */
+    float logit_scale;            /* logits = logit_scale * head . x ... */
+    float logit_softcap;          /* ... then softcap * tanh(logits / softcap); 0: off */
 } efm_decoder_desc;
 
 EFM_API efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decoder_layer* layers, int32_t device_id,

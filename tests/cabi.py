@@ -46,14 +46,19 @@ class DecoderLayer(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "kv_heads", "dim", "vdim", "window", "distance_bias")] + \
         [("scale", C.c_float)] + [(n, C.c_int32) for n in ("decay_rank", "ff", "keep_first", "qk_norm", "head_temp", "qkv_bias", "rot_kind", "rot_dims")] + \
         [("rot_base", C.c_float)] + [(n, C.c_int32) for n in (
-            "q_rank", "kv_rank", "sink", "out_gate", "experts", "expert_ff", "expert_top", "expert_groups", "expert_groups_kept")]
+            "q_rank", "kv_rank", "sink", "out_gate", "experts", "expert_ff", "expert_top", "expert_groups", "expert_groups_kept")] + \
+        [(n, C.c_float) for n in ("rot_factor", "rot_original", "rot_fast", "rot_slow")] + [("ff_act", C.c_int32), ("expert_glu", C.c_int32),
+         ("expert_limit", C.c_float), ("expert_score", C.c_int32), ("expert_weight_input", C.c_int32), ("shared_ff", C.c_int32), ("shared_limit", C.c_float)] + \
+        [(n, C.c_int32) for n in ("linear_heads", "linear_dim", "linear_vdim")] + [("mix_scale", C.c_float), ("linear_scale", C.c_float),
+         ("linear_decay", C.POINTER(C.c_double))]
 
 
 class DecoderDesc(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("struct_size", "num_layers", "vocab", "width", "side_dim")] + \
         [("norm_eps", C.c_float)] + [(n, C.c_int32) for n in (
             "compute_dtype", "max_step_tokens", "max_response_tokens", "cache_pages", "state_slots", "max_slots",
-            "norm_layout")] + [("embed_scale", C.c_float)] + [(n, C.c_int32) for n in ("loop_start", "loop_stop", "loop_times")]
+            "norm_layout")] + [("embed_scale", C.c_float)] + [(n, C.c_int32) for n in ("loop_start", "loop_stop", "loop_times")] + \
+        [("residual_mult", C.c_float), ("tied_head", C.c_int32), ("logit_scale", C.c_float), ("logit_softcap", C.c_float)]
 
 
 class StepEntry(C.Structure):
@@ -472,14 +477,18 @@ class VlaPolicy:
 
 
 class Decoder(Backend):
-    """A layered-decoder context described by a Folizen or Temuvik configuration dict; one mapped slot per call of map_slot."""
+    """A layered-decoder context described by a Folizen, Temuvik or Vekolix configuration dict; one mapped slot per call of map_slot."""
 
     def __init__(self, config, *, decay_rank=64, cache_pages=64, state_slots=4, max_slots=4, max_step_tokens=2048,
                  max_response_tokens=512, dtype=EFM_BF16, device_id=0):
         self.L = lib()
         layers = (DecoderLayer * len(config["layers"]))()
-        temuvik = config["architecture"] == "Temuvik"
+        temuvik, vekolix = (config["architecture"] == n for n in ("Temuvik", "Vekolix"))
+        decays = []                                                   # read by decoder_create
         for e, l in zip(layers, config["layers"]):
+            if vekolix:
+                self._vekolix_layer(e, l, decays)
+                continue
             m, mask = l["mixer"], l["mixer"].get("mask") or {}
             e.heads, e.dim, e.window = m["heads"], m["dim"], mask.get("size", 0)
             if temuvik:
@@ -502,13 +511,39 @@ class Decoder(Backend):
         loop = config.get("loop") or {"start": 0, "stop": 0, "times": 0}
         d = DecoderDesc(C.sizeof(DecoderDesc), len(layers), config["vocab"], config["width"],
                         (config.get("token_side") or {}).get("dim", 0), config["norm"]["eps"], dtype, max_step_tokens,
-                        max_response_tokens, cache_pages, state_slots, max_slots, int(temuvik),
-                        config["embedding"]["scale"] if temuvik else 1.0, loop["start"], loop["stop"], loop["times"])
+                        max_response_tokens, cache_pages, state_slots, max_slots, 2 if vekolix else int(temuvik),
+                        config["embedding"]["scale"] if temuvik else 1.0, loop["start"], loop["stop"], loop["times"], config.get("residual_mult", 0.0),
+                        int(vekolix), config.get("logit_scale", 1.0), config.get("logit_softcap", 0.0))
         self.cfg = type("Cfg", (), {"vocab": config["vocab"], "mrope_section": None})()
         self.ctx = P()
         st = self.L.efm_b200_decoder_create(C.byref(d), layers, device_id, C.byref(self.ctx))
         if st != EFM_OK:
             raise BackendError(f"decoder_create failed ({st}): {self.L.efm_b200_last_error(None).decode()}")
+
+    @staticmethod
+    def _vekolix_layer(e, l, decays):
+        m, mlp = l["mixer"], l["mlp"]
+        a = m["left"] if l["type"] == "parallel" else m
+        e.heads, e.dim, e.vdim, e.scale = a["heads"], a["dim"], a["vdim"], a["scale"]
+        e.rot_dims, e.rot_base = a["rot"]["dims"], a["rot"]["base"]
+        s = a["rot"].get("scaling")
+        if s:
+            e.rot_factor, e.rot_original, e.rot_fast, e.rot_slow = s["factor"], s["original"], s["fast"], s["slow"]
+        if l["type"] == "parallel":
+            r = m["right"]
+            decays.append((C.c_double * r["heads"])(*r["decay"]))
+            e.mixer, e.kv_heads, e.qk_norm, e.rot_kind = 3, a["kv_heads"], 2, 1
+            e.linear_heads, e.linear_dim, e.linear_vdim, e.linear_decay = r["heads"], r["dim"], r["vdim"], decays[-1]
+            e.mix_scale, e.linear_scale = m["left_scale"], m["right_scale"]
+        else:
+            e.mixer, e.q_rank, e.kv_rank, e.out_gate, e.rot_kind = 2, m["q_rank"], m["kv_rank"], 2, 2
+        if mlp and mlp["kind"] == "dense":
+            e.ff, e.ff_act = mlp["ff"], 1
+        elif mlp:
+            e.experts, e.expert_ff, e.expert_limit, e.expert_top = mlp["router"]["experts"], mlp["expert"]["ff"], mlp["expert"]["limit"], mlp["router"]["top"]
+            e.expert_groups = e.expert_groups_kept = e.expert_glu = e.expert_score = e.expert_weight_input = 1
+            if mlp.get("shared"):
+                e.shared_ff, e.shared_limit = mlp["shared"]["ff"], mlp["shared"]["limit"]
 
     def map_slot(self, slot, pages, state_slot):
         self.check(self.L.efm_b200_decoder_map_slot(self.ctx, slot, _i32_array(pages), len(pages), state_slot), "decoder_map_slot")

@@ -989,6 +989,42 @@ def folizen_flops(cfg, n):
     return out
 
 
+def vekolix_config(size):
+    """Attention beside linear attention (dense feed-forward) and latent attention (routed experts and a shared one) in turn."""
+    W, H, G, ff, V = DESIGN_SIZES[size]
+    e = DESIGN_EXPERTS
+    moe = {"kind": "moe", "expert": {"ff": ff // 8, "limit": 7.0}, "router": {"experts": e["count"], "top": e["top"]}, "shared": {"ff": ff // 8, "limit": 7.0}}
+    par = {"type": "parallel", "mlp": {"kind": "dense", "ff": ff}, "mixer": {
+        "left": {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                 "rot": {"base": 1e5, "dims": 64, "scaling": {"factor": 8.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}, "left_scale": 1.0,
+        "right": {"heads": W // 128, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-3.0 - 8.0 * h / (W // 128)) for h in range(W // 128)]}, "right_scale": 1.0}}
+    lat = {"type": "latent_attention", "mlp": moe, "mixer": {"heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": 3 * W // 8, "kv_rank": 512,
+                                                             "scale": 192 ** -0.5, "rot": {"base": 1e5, "dims": 64}}}
+    return {"architecture": "Vekolix", "width": W, "vocab": V, "norm": {"eps": 1e-5}, "residual_mult": 0.3, "logit_scale": 0.5, "logit_softcap": 30.0,
+            "layers": [lat if i % 2 == 0 else par for i in range(DESIGN_LAYERS)]}
+
+
+def vekolix_flops(cfg, n):
+    """Matrix products (of the experts a token uses) plus visible attention pairs plus the recurrence (2 D Dv multiply-adds per token
+    and head), 2 per multiply-add."""
+    W, out, seen = cfg["width"], 0, n * (n + 1) // 2
+    for l in cfg["layers"]:
+        m, mlp = l["mixer"], l["mlp"]
+        if l["type"] == "parallel":
+            a, b = m["left"], m["right"]
+            out += 2 * n * W * (a["heads"] * (a["dim"] + a["vdim"]) + a["kv_heads"] * (a["dim"] + a["vdim"])) + 2 * a["heads"] * (a["dim"] + a["vdim"]) * seen
+            out += 2 * n * W * b["heads"] * (2 * b["dim"] + 3 * b["vdim"]) + 4 * n * b["heads"] * b["dim"] * b["vdim"]
+        else:
+            H, D, Dv, R, q, L = m["heads"], m["dim"], m["vdim"], m["rot_dim"], m["q_rank"], m["kv_rank"]
+            out += 2 * n * (W * (q + L + R + H + H * Dv) + q * H * (D + R) + L * H * (D + Dv)) + 2 * H * (D + R + Dv) * seen
+        if mlp["kind"] == "dense":
+            out += 4 * n * W * mlp["ff"]
+        else:
+            r = mlp["router"]
+            out += 2 * n * W * (r["experts"] + 3 * r["top"] * mlp["expert"]["ff"] + 3 * mlp["shared"]["ff"])
+    return out
+
+
 def time_model(be, slot, prompt, steps, warmup):
     """Median device times: prefill of the whole prompt (no sample), decode per token at that context (captured graph)."""
     pre, dec = [], []
@@ -1020,24 +1056,28 @@ def run_design(args):
     import cabi
     import folizen_util as fu
     import temuvik_util as tu
+    import vekolix_util as vu
     from oracle import qwen_text, synth
     hbm, _ = peaks()
     tf, _ = tensor_peak()
     clocks = ClockSampler(0)
     name_ = args.design.capitalize()
-    design_config, design_flops = (folizen_config, folizen_flops) if args.design == "folizen" else (temuvik_config, temuvik_flops)
+    design_config, design_flops, design_shapes = {"folizen": (folizen_config, folizen_flops, lambda cfg: fu.shapes(cfg, DESIGN_RANK)),
+                                                  "temuvik": (temuvik_config, temuvik_flops, tu.shapes),
+                                                  "vekolix": (vekolix_config, vekolix_flops, vu.shapes)}[args.design]
     out = {"metric": name_ + " prefill / decode throughput beside the text tower at equal size", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic",
-           "config": {"layers": DESIGN_LAYERS, "prompt": DESIGN_PROMPT, "decode_steps": DESIGN_DECODE, "window": DESIGN_WINDOW}, "sizes": {}}
+           "config": {"layers": DESIGN_LAYERS, "prompt": DESIGN_PROMPT, "decode_steps": DESIGN_DECODE, "window": 0 if args.design == "vekolix" else DESIGN_WINDOW}, "sizes": {}}
     clocks.start()
     for size in args.design_sizes.split(","):
         cfg = design_config(size)
         pages = (DESIGN_PROMPT + DESIGN_DECODE + 64) // 64
         g = torch.Generator(device="cuda").manual_seed(0)
         be = cabi.Decoder(cfg, decay_rank=DESIGN_RANK, cache_pages=pages, state_slots=1, max_slots=1)
-        n_weights = 0
-        for name, shape in (fu.shapes(cfg, DESIGN_RANK) if args.design == "folizen" else tu.shapes(cfg)).items():
+        shapes = design_shapes(cfg)
+        n_weights = 0 if "head" in shapes else cfg["vocab"] * cfg["width"]        # a tied head counts like any other
+        for name, shape in shapes.items():
             t = torch.randn(shape, generator=g, device="cuda") * (shape[-1] ** -0.5 if len(shape) == 2 else 0.1)
-            if "norm" in name or name.endswith("temp"):
+            if ("norm" in name and not name.endswith(".b")) or name.endswith("temp"):
                 t += 1.0
             used = DESIGN_EXPERTS["top"] / DESIGN_EXPERTS["count"] if ".mlp.e" in name else 1
             n_weights += int(t.numel() * used) if len(shape) == 2 and "embed" not in name else 0
@@ -1079,7 +1119,7 @@ def main():
     ap.add_argument("--config", type=int, default=None, choices=[0, 1, 2, 3, 4],
                     help="run one configuration alone; default: configuration 3 (tensor parallel over the ranks) plus, on one GPU, "
                          "a short pass over the other four")
-    ap.add_argument("--design", choices=["folizen", "temuvik"], default=None, help="layered decoder beside the text tower at equal size (one GPU)")
+    ap.add_argument("--design", choices=["folizen", "temuvik", "vekolix"], default=None, help="layered decoder beside the text tower at equal size (one GPU)")
     ap.add_argument("--design-sizes", default="1024,2048,4096", help="comma-separated widths for --design")
     ap.add_argument("--tokens", type=int, default=0, help="override the number of generated tokens")
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")

@@ -92,7 +92,7 @@ SIZES = {
     "tiny": config([parallel(heads=1, kv_heads=1, dim=8, vdim=8, rot=2, lin_heads=1, lin_dim=4, lin_vdim=4, mlp=experts(n=2, top=1, ff=8, shared=(8, 0.3))),
                     latent(heads=1, dim=8, rot=2, vdim=8, q_rank=8, kv_rank=8, mlp=dense(8))], width=16, vocab=32),
     "odd": config([latent(heads=3, dim=20, rot=6, vdim=12, q_rank=30, kv_rank=36, mlp=experts(n=9, top=3, ff=50, shared=(70, 1.0))),
-                   parallel(heads=5, kv_heads=1, dim=20, vdim=12, rot=6, lin_heads=3, lin_dim=7, lin_vdim=9, mlp=dense(90))], width=76, vocab=131, eps=1e-3, mult=1.0),
+                   parallel(heads=5, kv_heads=1, dim=20, vdim=12, rot=6, lin_heads=3, lin_dim=7, lin_vdim=9, mlp=dense(90))], width=76, vocab=131, eps=1e-1, mult=0.4),
     "unaligned_rows": config([parallel(heads=3, kv_heads=3, dim=9, vdim=5, rot=4, lin_heads=5, lin_dim=13, lin_vdim=3, mlp=dense(33))], width=50, vocab=77),
     "wide_group": config([parallel(heads=12, kv_heads=1, dim=64, vdim=96, rot=32, lin_heads=2, lin_dim=64, lin_vdim=128), latent(heads=12, dim=64, rot=32, vdim=96)],
                          width=192, vocab=301),
@@ -227,14 +227,14 @@ def test_long_decoding(built, tmp_path, dtype):
 def test_state_over_chunk_edges(built, tmp_path, decay, dtype):
     """The recurrence alone, cut at and beside the edges of its chunks; with decays near one a state that is lost, kept from
     another request or decayed once too often shows hundreds of tokens later."""
-    cfg = config([parallel(lin_heads=2, lin_dim=24, lin_vdim=20, decay=decay)])
+    cfg = config([parallel(lin_heads=2, lin_dim=24, lin_vdim=20, decay=decay, scales=(1.0, 2.0))])
     w = isolate(vu.weights(cfg, seed=4), "right")
     eng = vu.engine(tmp_path, cfg, w, dtype)
     for seed, cuts in enumerate(([300], [64, 64, 64, 108], [63, 2, 64, 1, 65, 105], [1, 2], [129, 1, 1, 62, 107], [192, 1])):
         toks = vu.tokens(cfg, 300, seed=50 + seed)
         ref = reference(cfg, w, toks).logits.numpy()
-        forgot = reference(cfg, w, toks[64:]).logits.numpy()
-        assert decay[-1] < 0.99 or vu.error(forgot[-20:], ref[-20:]) > 0.1
+        forgot = reference(cfg, w, toks[192:]).logits.numpy()
+        assert decay[-1] < 0.99 or vu.error(forgot[-20:], ref[-20:]) > 0.15
         assert vu.error(vu.run_portions(eng, "r", toks, cuts), ref) < vu.LIMIT[dtype], cuts
 
 

@@ -130,7 +130,7 @@ cudaError_t alloc_inv_freq(efm_b200_ctx* c, DecoderLayer& l) {
 cudaError_t alloc_powers(efm_b200_ctx* c, DecoderLayer& l) {
     std::vector<float> f;
     for (int h = 0; h < l.d.linear_heads; ++h)
-        for (int i = 0; i <= kLinearChunk; ++i) f.push_back((float)std::pow(l.d.linear_decay[h], (double)i));
+        for (int i = 0; i <= kLinearPowers; ++i) f.push_back((float)std::pow(l.d.linear_decay[h], (double)i));
     cudaError_t e = dev_alloc(c, &l.lin_powers, f.size());
     if (e == cudaSuccess) e = cudaStreamSynchronize(c->stream);
     return e == cudaSuccess ? cudaMemcpy(l.lin_powers, f.data(), f.size() * sizeof(float), cudaMemcpyHostToDevice) : e;

@@ -20,6 +20,7 @@
 #include "../operators/gemm_tc.cuh"
 #include "../operators/latent_attention.cuh"
 #include "../operators/linear_attention.cuh"
+#include "../operators/linear_attention_tc.cuh"
 #include "../operators/token_side.cuh"
 #include "../operators/window_attention.cuh"
 #include "../operators/window_attention_tc.cuh"
@@ -596,7 +597,34 @@ void linear_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const Deco
     DecoderModel& m = *c.decoder;
     const LinearShape s = linear_shape(m, l);
     const TA* proj = static_cast<const TA*>(m.proj_a);
-    const int chunks = max_chunks(plan, kLinearChunk), ld_o = round_up(s.width(), 8);
+    const int ld_o = round_up(s.width(), 8);
+    bool tensor_cores = false;
+    if constexpr (std::is_same<TA, __nv_bfloat16>::value) tensor_cores = s.D <= 128 && plan.rows >= kLinearChunk;      // short passes: CUDA cores
+    const int chunks = max_chunks(plan, tensor_cores ? kLinearChunkTc : kLinearChunk);
+    auto chain = [&](auto kernel) {
+        L.launch(kernel, dim3((unsigned)((s.heads * s.head_floats() + 1023) / 1024), plan.n_entries), dim3(256), 0, m.lin_ws, m.state_pool, m.state_stride, run.state_off,
+                 s, plan);
+    };
+    auto output = [&] {
+        L.launch(linear_output_rows_kernel<TA>, dim3(plan.rows), dim3(256), 0, (const float*)m.o, ld_o, proj, static_cast<TA*>(m.mix) + l.lin_mix, l.mix_wp,
+                 l.mix_wp - l.lin_mix, s);
+    };
+    if constexpr (std::is_same<TA, __nv_bfloat16>::value) {
+        if (tensor_cores) {
+            auto products = [&](auto vp) {
+                constexpr int VP = decltype(vp)::value;
+                const dim3 grid(chunks, s.heads, (s.Dv + VP - 1) / VP);
+                L.launch(linear_chunk_tc_kernel<VP>, grid, dim3(lt::kThreads), lt::Cfg<VP>::CHUNK_SMEM, proj, m.lin_ws, s, plan, &c.state->error);
+                chain(linear_chain_rows_kernel<kLinearChunkTc>);
+                L.launch(linear_attend_tc_kernel<VP>, grid, dim3(lt::kThreads), lt::Cfg<VP>::ATTEND_SMEM, proj, (const float*)m.lin_ws, m.o, ld_o, s, plan,
+                         &c.state->error);
+            };
+            if (s.Dv <= 64) products(std::integral_constant<int, 64>{});
+            else products(std::integral_constant<int, 128>{});
+            output();
+            return;
+        }
+    }
     auto chunk = [&](auto rm, auto rn) {
         constexpr int RM = decltype(rm)::value, RN = decltype(rn)::value;
         L.launch(linear_chunk_rows_kernel<TA, RM, RN>, dim3(chunks, s.heads, ((s.D + 16 * RM - 1) / (16 * RM)) * ((s.Vp + 16 * RN - 1) / (16 * RN))), dim3(ln::kThreads),
@@ -612,11 +640,9 @@ void linear_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const Deco
     if (s.D <= 64) { if (s.Dv <= 64) chunk(k4, k4); else chunk(k4, k8); }
     else if (s.Dv <= 64) chunk(k8, k4);
     else chunk(k8, k8);
-    L.launch(linear_chain_rows_kernel, dim3((unsigned)((s.heads * s.head_floats() + 1023) / 1024), plan.n_entries), dim3(256), 0, m.lin_ws, m.state_pool, m.state_stride,
-             run.state_off, s, plan);
+    chain(linear_chain_rows_kernel<kLinearChunk>);
     if (s.Dv <= 64) attend(k4); else attend(k8);
-    L.launch(linear_output_rows_kernel<TA>, dim3(plan.rows), dim3(256), 0, (const float*)m.o, ld_o, proj, static_cast<TA*>(m.mix) + l.lin_mix, l.mix_wp,
-             l.mix_wp - l.lin_mix, s);
+    output();
 }
 
 // TA: activation and cache type of the pass
@@ -624,8 +650,21 @@ template <typename TA>
 void attention_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const void* x, const RowPlan& plan, const RowTiles& tiles) {
     DecoderModel& m = *c.decoder;
     const WindowAttnShape s = attn_shape(m, l);
-    linear_act(c, L, l.in, x, m.proj_a, plan.rows);
-    if (l.linear()) linear_rows<TA>(c, L, l, run, plan);
+    if (l.linear()) {
+        const LinearShape z = linear_shape(m, l);
+        if constexpr (std::is_same<TA, float>::value) {
+            linear_f32(c, L, l.in, x, static_cast<float*>(m.proj_a), plan.rows);
+            L.launch(silu_columns_kernel, dim3((z.off_g - z.off_q + 1023) / 1024, plan.rows), dim3(256), 0, static_cast<float*>(m.proj_a), l.in.Np, z.off_q, z.off_g);
+        } else {
+            GemmParams g{static_cast<const __nv_bfloat16*>(x), l.in.w, l.in.bias, static_cast<__nv_bfloat16*>(m.proj_a), nullptr, plan.rows, l.in.Np, l.in.Kp};
+            g.silu0 = z.off_q;
+            g.silu1 = z.off_g;
+            launch_gemm_epi(L, GemmEpi::Bf16Silu, g, &c.state->error);
+        }
+        linear_rows<TA>(c, L, l, run, plan);
+    } else {
+        linear_act(c, L, l.in, x, m.proj_a, plan.rows);
+    }
     TA* kp = static_cast<TA*>(run.k_pool);
     TA* vp = static_cast<TA*>(run.v_pool);
     int lanes = 8;                                                  // 8 channels each: at most 256 (padded) channels a head
@@ -1006,6 +1045,10 @@ cudaError_t configure_decoder(DecoderModel& m) {
     };
     linear_attr(float());
     linear_attr(__nv_bfloat16());
+    if (e == cudaSuccess) e = smem_attr(linear_chunk_tc_kernel<64>, lt::Cfg<64>::CHUNK_SMEM);
+    if (e == cudaSuccess) e = smem_attr(linear_chunk_tc_kernel<128>, lt::Cfg<128>::CHUNK_SMEM);
+    if (e == cudaSuccess) e = smem_attr(linear_attend_tc_kernel<64>, lt::Cfg<64>::ATTEND_SMEM);
+    if (e == cudaSuccess) e = smem_attr(linear_attend_tc_kernel<128>, lt::Cfg<128>::ATTEND_SMEM);
     const size_t rows = wa::rows_smem_bytes(256, 256);
     if (e == cudaSuccess) e = smem_attr(window_attention_rows_kernel<float, float, float>, rows);
     if (e == cudaSuccess) e = smem_attr(window_attention_rows_kernel<__nv_bfloat16, __nv_bfloat16, __nv_bfloat16>, rows);

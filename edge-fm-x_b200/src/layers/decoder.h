@@ -49,7 +49,7 @@ struct DecoderLayer {
     // linear attention beside attention
     int lin_in = 0, lin_mix = 0;          // its first column in the projections and in the mixer output
     int lin_vp = 0;                       // value channels padded to 4 (state rows)
-    float* lin_powers = nullptr;          // [linear_heads][kLinearChunk + 1]
+    float* lin_powers = nullptr;          // [linear_heads][kLinearPowers + 1]
     bool linear() const { return d.mixer == EFM_MIXER_PARALLEL; }
     bool attention() const { return d.mixer == EFM_MIXER_ATTENTION || d.mixer == EFM_MIXER_PARALLEL; }
     // routed experts

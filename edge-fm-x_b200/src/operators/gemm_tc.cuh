@@ -14,7 +14,7 @@
 //               longer than its MMAs whenever K was short):
 //               tcgen05.ld (row = TMEM lane, 32 columns at a time), bias / activation, staging through
 //               shared memory (XOR-swizzled 16-byte columns) so that global rows are written as contiguous segments:
-//               bf16 (+bias, optionally erf-GELU, tanh-GELU or squared ReLU) | fp32 residual add | fp32 | a gated unit in bf16.
+//               bf16 (+bias, optionally erf-GELU, tanh-GELU, squared ReLU or silu of a column range) | fp32 residual add | fp32 | a gated unit in bf16.
 // Rows past M and columns past N are zero-filled by TMA on load and masked on store.
 // Every mbarrier wait is bounded; a wait that gives up raises *error, all roles leave their loops, the
 // block frees its TMEM and returns.  Bound: tensor pipe (2 M N K flops).
@@ -25,7 +25,7 @@
 
 namespace efm {
 
-enum class GemmEpi : int { Bf16Bias = 0, Residual = 1, F32 = 2, Bf16Gelu = 3, SwiGlu = 4, Bf16GeluTanh = 5, Bf16Relu2 = 6, ClampGlu = 7 };
+enum class GemmEpi : int { Bf16Bias = 0, Residual = 1, F32 = 2, Bf16Gelu = 3, SwiGlu = 4, Bf16GeluTanh = 5, Bf16Relu2 = 6, ClampGlu = 7, Bf16Silu = 8 };
 
 struct GroupTile { int32_t group, first, count, pad; };      // row tile: its group, the group's first row tile and number of them
 
@@ -50,6 +50,7 @@ struct GemmParams {
     const int32_t* group_tiles = nullptr;
     int group_rows = 0, group_all = 0;      // rows of B per group and altogether
     float limit = 0.f;        // ClampGlu
+    int silu0 = 0, silu1 = 0; // Bf16Silu: columns [silu0, silu1) become silu of themselves
 };
 
 // Gated units over a fused gate|up weight: half as many output columns.
@@ -63,6 +64,14 @@ __device__ __forceinline__ float gemm_glu(float g, float u, float limit) {
     }
     // the approximate reciprocal instead of an IEEE division: the epilogue warps' issue slots are the limit when K is short
     return __fdividef(g, 1.0f + __expf(-g)) * u;
+}
+
+__device__ __forceinline__ float4 gemm_silu_range(float4 a, int n, const GemmParams& p) {
+    float f[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+        if (n + j >= p.silu0 && n + j < p.silu1) f[j] = __fdividef(f[j], 1.0f + __expf(-f[j]));
+    return make_float4(f[0], f[1], f[2], f[3]);
 }
 
 namespace tc {
@@ -324,6 +333,7 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
                     for (int e = 0; e < 32; ++e) {
                         o[e] = __uint_as_float(r[e]) + __shfl_sync(0xffffffffu, bias_l, e);
                         if constexpr (EPI == GemmEpi::Bf16Gelu) o[e] = 0.5f * o[e] * (1.0f + erff(o[e] * 0.70710678118654752f));
+                        if constexpr (EPI == GemmEpi::Bf16Silu) { if (n + e >= p.silu0 && n + e < p.silu1) o[e] = __fdividef(o[e], 1.0f + __expf(-o[e])); }
                         if constexpr (EPI == GemmEpi::Bf16Relu2) { o[e] = fmaxf(o[e], 0.f); o[e] *= o[e]; }
                         if constexpr (EPI == GemmEpi::Bf16GeluTanh)
                         {
@@ -434,6 +444,7 @@ __global__ void __launch_bounds__(256) gemm_splitk_finish_kernel(const float* __
             const float4 o = *reinterpret_cast<const float4*>(p.Cf + i * 4);
             *reinterpret_cast<float4*>(p.Cf + i * 4) = make_float4(o.x + a.x, o.y + a.y, o.z + a.z, o.w + a.w);
         } else {
+            if constexpr (EPI == GemmEpi::Bf16Silu) a = gemm_silu_range(a, n, p);
             if constexpr (EPI == GemmEpi::Bf16Relu2) {
                 a.x = fmaxf(a.x, 0.f); a.y = fmaxf(a.y, 0.f); a.z = fmaxf(a.z, 0.f); a.w = fmaxf(a.w, 0.f);
                 a.x *= a.x; a.y *= a.y; a.z *= a.z; a.w *= a.w;
@@ -474,6 +485,7 @@ __global__ void __launch_bounds__(256) gemm_tail_finish_kernel(const float* __re
             const float4 o = *reinterpret_cast<const float4*>(p.Cf + off);
             *reinterpret_cast<float4*>(p.Cf + off) = make_float4(o.x + a.x, o.y + a.y, o.z + a.z, o.w + a.w);
         } else {
+            if constexpr (EPI == GemmEpi::Bf16Silu) a = gemm_silu_range(a, n, p);
             *reinterpret_cast<uint2*>(p.C + off) = make_uint2(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w));
         }
     }

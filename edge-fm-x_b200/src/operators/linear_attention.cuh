@@ -1,9 +1,10 @@
 // Linear attention with a constant decay per head: a state S [D key channels x Dv value channels], fp32,
 //   S_t = a S_{t-1} + k_t v_t^T,   o_t = S_t^T q_t,   q, k, v = silu(projections),
 // then one RMS norm over the channels of all heads, a plain weight, a sigmoid gate and a multiplier.  The projections are four
-// column ranges of a row, each starting at a multiple of 8.
+// column ranges of a row, each starting at a multiple of 8; in the many-row forms the product that makes them has applied silu (the
+// 32-bit mode: silu_columns), so that q, k and v are rounded once.
 //
-// Many rows, in chunks of up to 64 tokens of one entry.  A chunk's own contribution does not depend on the state it starts from, so
+// Many rows, in chunks of up to 64 tokens of one entry (128 on the tensor cores, linear_attention_tc.cuh).  A chunk's own contribution does not depend on the state it starts from, so
 // all chunks run at once and only their sums are chained:
 //   linear_chunk_rows    U_c = sum_t a^(n-1-t) k_t v_t^T of every chunk (n tokens)
 //   linear_chain_rows    the states the chunks start from, S_{c+1} = a^n S_c + U_c, in place of the U_c; the last one to the pool
@@ -22,7 +23,7 @@ struct LinearShape {
     int heads, D, Dv, Vp;
     int off_q, off_k, off_v, off_g;   // columns of the projections
     int ld;                           // row length of the projections
-    const float* powers;              // [heads][kLinearChunk + 1]: decay^i
+    const float* powers;              // [heads][kLinearPowers + 1]: decay^i
     const __nv_bfloat16* norm;        // [heads * Dv]
     float eps, scale;
     __host__ __device__ int width() const { return heads * Dv; }
@@ -36,7 +37,7 @@ __device__ __forceinline__ float lin_f32(__nv_bfloat16 v) { return __bfloat162fl
 namespace ln {
 constexpr int C = kLinearChunk, kThreads = 256;
 
-// dst[r][0 .. cols) (row stride ld_dst, cols % 4 == 0) = silu of channels [c0, c0 + cols) of a head, zero past `width` and past row n
+// dst[r][0 .. cols) (row stride ld_dst, cols % 4 == 0) = mul(r) times channels [c0, c0 + cols) of a head, zero past `width` and past row n
 template <typename T, typename F>
 __device__ __forceinline__ void stage_rows(float* dst, int ld_dst, const T* src, int ld_src, int c0, int cols, int width, int n, F mul) {
     const int per = cols / 4;
@@ -61,7 +62,7 @@ __device__ __forceinline__ void stage_rows(float* dst, int ld_dst, const T* src,
             }
             const float m = mul(r);
 #pragma unroll
-            for (int j = 0; j < 4; ++j) f[j] = silu_f(f[j]) * m;
+            for (int j = 0; j < 4; ++j) f[j] *= m;
         }
         *reinterpret_cast<float4*>(dst + (size_t)r * ld_dst + c) = make_float4(f[0], f[1], f[2], f[3]);
     }
@@ -75,6 +76,15 @@ __host__ __device__ inline size_t attend_smem_bytes(int D, int RN) {
 }
 }  // namespace ln
 
+// columns [c0, c1) of every row (multiples of 4).  Grid (parts of a row, rows)
+__global__ void __launch_bounds__(256) silu_columns_kernel(float* __restrict__ x, int ld, int c0, int c1) {
+    const int c = c0 + 4 * (blockIdx.x * 256 + threadIdx.x);
+    if (c >= c1) return;
+    float4* p = reinterpret_cast<float4*>(x + (size_t)blockIdx.y * ld + c);
+    const float4 v = *p;
+    *p = make_float4(silu_f(v.x), silu_f(v.y), silu_f(v.z), silu_f(v.w));
+}
+
 // grid (chunks, heads, tiles of the state); a tile is 16 RM key channels x 16 RN value channels.  ws: [chunks][heads][D][Vp]
 template <typename T, int RM, int RN>
 __global__ void __launch_bounds__(ln::kThreads) linear_chunk_rows_kernel(const T* __restrict__ proj, float* __restrict__ ws, const LinearShape s, const RowPlan plan) {
@@ -87,7 +97,7 @@ __global__ void __launch_bounds__(ln::kThreads) linear_chunk_rows_kernel(const T
     if (!locate_chunk<C>(plan, blockIdx.x, e, t0)) return;
     const int h = blockIdx.y, n = min(C, e.n - t0), tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
     const int tiles_n = (s.Vp + TN - 1) / TN, d0 = blockIdx.z / tiles_n * TM, v0 = blockIdx.z % tiles_n * TN;
-    const float* pw = s.powers + (size_t)h * (C + 1);
+    const float* pw = s.powers + (size_t)h * (kLinearPowers + 1);
     const T* row = proj + (size_t)(e.row0 + t0) * s.ld;
     stage_rows(ks, TM, row + s.off_k + h * s.D, s.ld, d0, TM, s.D, n, [&](int r) { return pw[n - 1 - r]; });
     stage_rows(vs, TN, row + s.off_v + h * s.Dv, s.ld, v0, TN, s.Dv, n, [](int) { return 1.0f; });
@@ -122,14 +132,15 @@ __global__ void __launch_bounds__(ln::kThreads) linear_chunk_rows_kernel(const T
     }
 }
 
-// grid (groups of 256 x 4 state numbers, entries)
+// grid (groups of 256 x 4 state numbers, entries); chunks of C tokens
+template <int C>
 __global__ void __launch_bounds__(256) linear_chain_rows_kernel(float* __restrict__ ws, float* __restrict__ pool, size_t slot_stride, size_t offset,
                                                                 const LinearShape s, const RowPlan plan) {
-    constexpr int C = kLinearChunk, U = 8;
+    constexpr int U = 8;
     const size_t all = s.heads * s.head_floats(), i = ((size_t)blockIdx.x * 256 + threadIdx.x) * 4;
     if (i >= all) return;
     const RowEntry e = plan.entry(blockIdx.y);
-    const float* pw = s.powers + i / s.head_floats() * (C + 1);
+    const float* pw = s.powers + i / s.head_floats() * (kLinearPowers + 1);
     int chunk0 = 0;
     for (int k = 0; k < (int)blockIdx.y; ++k) chunk0 += (plan.entry(k).n + C - 1) / C;
     const int n_chunks = (e.n + C - 1) / C;
@@ -167,7 +178,7 @@ __global__ void __launch_bounds__(ln::kThreads) linear_attend_rows_kernel(const 
     const int D4 = (s.D + 3) / 4 * 4, LD = D4 + 4;
     float *qs = ln_smem, *ks = qs + C * LD, *vs = ks, *ps = ks + attend_key_floats(D4, RN), *ss = ps + C * LP;
     __shared__ float pw[C + 1];
-    if (tid <= C) pw[tid] = s.powers[(size_t)h * (C + 1) + tid];
+    if (tid <= C) pw[tid] = s.powers[(size_t)h * (kLinearPowers + 1) + tid];
     const T* row = proj + (size_t)(e.row0 + t0) * s.ld;
     auto one = [](int) { return 1.0f; };
     stage_rows(qs, LD, row + s.off_q + h * s.D, s.ld, 0, D4, s.D, n, one);
@@ -277,12 +288,27 @@ __global__ void __launch_bounds__(256) linear_output_rows_kernel(const float* __
         if (c + 4 > n) { if (c >= n) v.x = 0.f; if (c + 1 >= n) v.y = 0.f; if (c + 2 >= n) v.z = 0.f; v.w = 0.f; }
         return v;
     };
+    struct Factors { float g[4], w[4]; };
+    auto factors = [&](int c) {
+        Factors f;
+        const uint2 w = *reinterpret_cast<const uint2*>(s.norm + c);       // padded with zeros
+        f.w[0] = bf16lo(w.x); f.w[1] = bf16hi(w.x); f.w[2] = bf16lo(w.y); f.w[3] = bf16hi(w.y);
+        if constexpr (sizeof(T) == 2) {
+            const uint2 x = *reinterpret_cast<const uint2*>(gate + c);
+            f.g[0] = bf16lo(x.x); f.g[1] = bf16hi(x.x); f.g[2] = bf16lo(x.y); f.g[3] = bf16hi(x.y);
+        } else {
+            const float4 x = *reinterpret_cast<const float4*>(gate + c);
+            f.g[0] = x.x; f.g[1] = x.y; f.g[2] = x.z; f.g[3] = x.w;
+        }
+        return f;
+    };
     float4 keep[KEEP];
+    Factors fac[KEEP];                                                  // requested ahead of the sum
     float ss = 0.f;
     auto square = [&](const float4& v) { ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss)))); };
 #pragma unroll
     for (int i = 0; i < KEEP; ++i)
-        if (4 * (tid + 256 * i) < cols) keep[i] = load(4 * (tid + 256 * i));
+        if (4 * (tid + 256 * i) < cols) { keep[i] = load(4 * (tid + 256 * i)); fac[i] = factors(4 * (tid + 256 * i)); }
 #pragma unroll
     for (int i = 0; i < KEEP; ++i)
         if (4 * (tid + 256 * i) < cols) square(keep[i]);
@@ -294,27 +320,18 @@ __global__ void __launch_bounds__(256) linear_output_rows_kernel(const float* __
 #pragma unroll
     for (int i = 0; i < 8; ++i) ss += part[i];
     const float inv = s.scale / sqrtf(ss / (float)n + s.eps);
-    auto emit = [&](int c, const float4& v) {
+    auto emit = [&](int c, const float4& v, const Factors& k) {
         const float f[4] = {v.x, v.y, v.z, v.w};
-        float g[4], w[4], r[4];
-        const uint2 wv = *reinterpret_cast<const uint2*>(s.norm + c);     // padded with zeros
-        w[0] = bf16lo(wv.x); w[1] = bf16hi(wv.x); w[2] = bf16lo(wv.y); w[3] = bf16hi(wv.y);
-        if constexpr (sizeof(T) == 2) {
-            const uint2 x = *reinterpret_cast<const uint2*>(gate + c);
-            g[0] = bf16lo(x.x); g[1] = bf16hi(x.x); g[2] = bf16lo(x.y); g[3] = bf16hi(x.y);
-        } else {
-            const float4 x = *reinterpret_cast<const float4*>(gate + c);
-            g[0] = x.x; g[1] = x.y; g[2] = x.z; g[3] = x.w;
-        }
+        float r[4];
 #pragma unroll
-        for (int j = 0; j < 4; ++j) r[j] = f[j] * inv * w[j] / (1.0f + expf(-g[j]));
+        for (int j = 0; j < 4; ++j) r[j] = f[j] * inv * k.w[j] / (1.0f + expf(-k.g[j]));
         if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2*>(dst + c) = make_uint2(pack_bf16(r[0], r[1]), pack_bf16(r[2], r[3]));
         else *reinterpret_cast<float4*>(dst + c) = make_float4(r[0], r[1], r[2], r[3]);
     };
 #pragma unroll
     for (int i = 0; i < KEEP; ++i)
-        if (4 * (tid + 256 * i) < cols) emit(4 * (tid + 256 * i), keep[i]);
-    for (int c = 4 * (tid + 256 * KEEP); c < cols; c += 1024) emit(c, load(c));
+        if (4 * (tid + 256 * i) < cols) emit(4 * (tid + 256 * i), keep[i], fac[i]);
+    for (int c = 4 * (tid + 256 * KEEP); c < cols; c += 1024) emit(c, load(c), factors(c));
 }
 
 // ---- one row -----------------------------------------------------------------------------------------------------------
@@ -350,7 +367,7 @@ __device__ __forceinline__ void linear_decode_block(const LinearDecodeParams& p,
         const int d = rg + 16 * i;
         r[i] = act && d < s.D && !fresh ? __ldcg(reinterpret_cast<const float4*>(S + (size_t)d * s.Vp)) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    const float a = s.powers[(size_t)h * (kLinearChunk + 1) + 1];
+    const float a = s.powers[(size_t)h * (kLinearPowers + 1) + 1];
     if (early) { pdl_wait(); pdl_launch_dependents(); }
     float v[4];
 #pragma unroll

@@ -7,7 +7,8 @@
 namespace efm {
 
 constexpr int kPageTokens = 64;       // cache rows per page
-constexpr int kLinearChunk = 64;      // tokens per chunk of linear attention
+constexpr int kLinearChunk = 64, kLinearChunkTc = 128;      // tokens per chunk of linear attention: CUDA cores, tensor cores
+constexpr int kLinearPowers = kLinearChunkTc;               // powers of a decay at hand
 
 struct RowEntry {
     int32_t row0, n, pos0;            // rows [row0, row0 + n) hold positions [pos0, pos0 + n) of the sequence

@@ -828,6 +828,18 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
                                 : (experts ? add_norm_rows_kernel<TA, false, true> : add_norm_rows_kernel<TA, false, false>),
                  dim3(T), dim3(256), 0, c.resid, y, w, xa, pre, m.W, m.Wp, m.d.norm_eps, sum);
     };
+    // a sublayer's last product and what follows it; elementwise norms are part of the product
+    auto sublayer_out = [&](const DecLinear& w, const void* a, const __nv_bfloat16* post, const DecNorm& norm) {
+        if (m.tanh_norms() && !m.f32) {
+            GemmParams g{static_cast<const __nv_bfloat16*>(a), w.w, nullptr, norm.w != nullptr ? static_cast<__nv_bfloat16*>(m.xa) : nullptr, c.resid, T, w.Np, w.Kp};
+            g.mult = m.d.residual_mult;
+            g.norm_w = norm.w; g.norm_b = norm.b; g.norm_alpha = norm.alpha;
+            launch_gemm_epi(L, GemmEpi::ResidualTanh, g, &c.state->error);
+            return;
+        }
+        linear_f32(c, L, w, a, m.y, T);
+        add_norm(m.y, post, norm);
+    };
     launch_embed_rows(L, ids, c.embed, nullptr, c.resid, T, c.d.vocab, m.Wp, -1, 0, m.d.embed_scale);
     if (xa != nullptr) add_norm(nullptr, nullptr, m.layers[m.runs[0].layer].pre1);
     for (size_t i = 0; i < m.runs.size(); ++i) {
@@ -837,8 +849,7 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
         if (l.attention()) attention_rows<TA>(c, L, l, run, xin, plan, tiles);
         else if (l.d.mixer == EFM_MIXER_LATENT_ATTENTION) latent_rows<TA>(c, L, l, run, xin, plan, tiles);
         else delta_rows<TA>(c, L, l, run, xin, plan);
-        linear_f32(c, L, l.out, m.mix, m.y, T);
-        add_norm(m.y, l.post1, l.mlp() ? l.pre2 : next);
+        sublayer_out(l.out, m.mix, l.post1, l.mlp() ? l.pre2 : next);
         if (l.moe()) {
             add_norm(nullptr, l.post2, next, expert_rows<TA>(c, L, l, xin, T));
         } else if (l.d.ff > 0) {
@@ -855,8 +866,7 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
                 GemmParams g{static_cast<const __nv_bfloat16*>(xin), l.up.w, nullptr, static_cast<__nv_bfloat16*>(m.ff), nullptr, T, l.up.Np, l.up.Kp};
                 launch_gemm_epi(L, GemmEpi::Bf16Relu2, g, &c.state->error);
             }
-            linear_f32(c, L, l.down, poly ? m.ff2 : m.ff, m.y, T);
-            add_norm(m.y, l.post2, next);
+            sublayer_out(l.down, poly ? m.ff2 : m.ff, l.post2, next);
         }
         if (m.d.side_dim > 0) {
             linear_f32(c, L, l.gate, xin, m.side_f, T);

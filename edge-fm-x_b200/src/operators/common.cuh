@@ -73,6 +73,9 @@ __device__ __forceinline__ float warp_max(float v) {
     return v;
 }
 
+// elementwise input norm
+__device__ __forceinline__ float tanh_norm(float x, float alpha, float w, float b) { return fmaf(tanhf(alpha * x), w, b); }
+
 // ---- programmatic dependent launch -----------------------------------------------------
 // Every kernel of the decode step calls pdl_wait() before it touches memory another kernel
 // writes, and calls it on every path (a grid that exits without waiting would let ITS

@@ -14,7 +14,8 @@
 //               longer than its MMAs whenever K was short):
 //               tcgen05.ld (row = TMEM lane, 32 columns at a time), bias / activation, staging through
 //               shared memory (XOR-swizzled 16-byte columns) so that global rows are written as contiguous segments:
-//               bf16 (+bias, optionally erf-GELU, tanh-GELU, squared ReLU or silu of a column range) | fp32 residual add | fp32 | a gated unit in bf16.
+//               bf16 (+bias, optionally erf-GELU, tanh-GELU, squared ReLU or silu of a column range) | fp32 residual add | fp32 | a gated unit in bf16 |
+//               fp32 residual add of a multiple and, in bf16, the elementwise norm tanh(alpha x) w + b of the new residual.
 // Rows past M and columns past N are zero-filled by TMA on load and masked on store.
 // Every mbarrier wait is bounded; a wait that gives up raises *error, all roles leave their loops, the
 // block frees its TMEM and returns.  Bound: tensor pipe (2 M N K flops).
@@ -25,7 +26,7 @@
 
 namespace efm {
 
-enum class GemmEpi : int { Bf16Bias = 0, Residual = 1, F32 = 2, Bf16Gelu = 3, SwiGlu = 4, Bf16GeluTanh = 5, Bf16Relu2 = 6, ClampGlu = 7, Bf16Silu = 8 };
+enum class GemmEpi : int { Bf16Bias = 0, Residual = 1, F32 = 2, Bf16Gelu = 3, SwiGlu = 4, Bf16GeluTanh = 5, Bf16Relu2 = 6, ClampGlu = 7, Bf16Silu = 8, ResidualTanh = 9 };
 
 struct GroupTile { int32_t group, first, count, pad; };      // row tile: its group, the group's first row tile and number of them
 
@@ -50,6 +51,9 @@ struct GemmParams {
     const int32_t* group_tiles = nullptr;
     int group_rows = 0, group_all = 0;      // rows of B per group and altogether
     float limit = 0.f;        // ClampGlu
+    // ResidualTanh: Cf += mult * product, C = tanh(alpha Cf) norm_w + norm_b (C null: none)
+    float mult = 1.f;
+    const __nv_bfloat16 *norm_w = nullptr, *norm_b = nullptr, *norm_alpha = nullptr;
     int silu0 = 0, silu1 = 0; // Bf16Silu: columns [silu0, silu1) become silu of themselves
 };
 
@@ -72,6 +76,17 @@ __device__ __forceinline__ float4 gemm_silu_range(float4 a, int n, const GemmPar
     for (int j = 0; j < 4; ++j)
         if (n + j >= p.silu0 && n + j < p.silu1) f[j] = __fdividef(f[j], 1.0f + __expf(-f[j]));
     return make_float4(f[0], f[1], f[2], f[3]);
+}
+
+// four columns from n on: the new residual and its norm
+__device__ __forceinline__ void gemm_residual_tanh(const GemmParams& p, const float4& old, const float4& v, size_t off, int n) {
+    const float4 x = make_float4(fmaf(p.mult, v.x, old.x), fmaf(p.mult, v.y, old.y), fmaf(p.mult, v.z, old.z), fmaf(p.mult, v.w, old.w));
+    *reinterpret_cast<float4*>(p.Cf + off) = x;
+    if (p.C == nullptr) return;
+    const float al = __bfloat162float(*p.norm_alpha);
+    const uint2 w = *reinterpret_cast<const uint2*>(p.norm_w + n), b = *reinterpret_cast<const uint2*>(p.norm_b + n);
+    *reinterpret_cast<uint2*>(p.C + off) = make_uint2(pack_bf16(tanh_norm(x.x, al, bf16lo(w.x), bf16lo(b.x)), tanh_norm(x.y, al, bf16hi(w.x), bf16hi(b.x))),
+                                                      pack_bf16(tanh_norm(x.z, al, bf16lo(w.y), bf16lo(b.y)), tanh_norm(x.w, al, bf16hi(w.y), bf16hi(b.y))));
 }
 
 namespace tc {
@@ -292,7 +307,7 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
                 // read and long before the first store (the
                 // compiler may not move a load of Cf above a store to Cf by itself), one round trip per chunk
                 float4 prev[8];
-                if constexpr (EPI == GemmEpi::Residual) {
+                if constexpr (EPI == GemmEpi::Residual || EPI == GemmEpi::ResidualTanh) {
 #pragma unroll
                     for (int r0 = 0; r0 < 32; r0 += 4) {
                         const int m = m0 + q * 32 + r0 + (lane >> 3), n = nc0 + c0 + cl;
@@ -365,6 +380,8 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
                         } else if constexpr (EPI == GemmEpi::Residual) {
                             const float4 old = prev[r0 >> 2];
                             *reinterpret_cast<float4*>(p.Cf + off) = make_float4(old.x + v.x, old.y + v.y, old.z + v.z, old.w + v.w);
+                        } else if constexpr (EPI == GemmEpi::ResidualTanh) {
+                            gemm_residual_tanh(p, prev[r0 >> 2], v, off, n);
                         } else {
                             *reinterpret_cast<uint2*>(p.C + off) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
                         }
@@ -375,6 +392,12 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
                             if (n + i >= ldc) break;
                             if constexpr (EPI == GemmEpi::F32) p.Cf[split_off + off + i] = e4[i];
                             else if constexpr (EPI == GemmEpi::Residual) p.Cf[off + i] += e4[i];
+                            else if constexpr (EPI == GemmEpi::ResidualTanh) {
+                                const float x = fmaf(p.mult, e4[i], p.Cf[off + i]);
+                                p.Cf[off + i] = x;
+                                if (p.C != nullptr)
+                                    p.C[off + i] = __float2bfloat16_rn(tanh_norm(x, __bfloat162float(*p.norm_alpha), __bfloat162float(p.norm_w[n + i]), __bfloat162float(p.norm_b[n + i])));
+                            }
                             else p.C[off + i] = __float2bfloat16_rn(e4[i]);
                         }
                     }
@@ -443,6 +466,8 @@ __global__ void __launch_bounds__(256) gemm_splitk_finish_kernel(const float* __
         } else if constexpr (EPI == GemmEpi::Residual) {
             const float4 o = *reinterpret_cast<const float4*>(p.Cf + i * 4);
             *reinterpret_cast<float4*>(p.Cf + i * 4) = make_float4(o.x + a.x, o.y + a.y, o.z + a.z, o.w + a.w);
+        } else if constexpr (EPI == GemmEpi::ResidualTanh) {
+            gemm_residual_tanh(p, *reinterpret_cast<const float4*>(p.Cf + i * 4), a, i * 4, n);
         } else {
             if constexpr (EPI == GemmEpi::Bf16Silu) a = gemm_silu_range(a, n, p);
             if constexpr (EPI == GemmEpi::Bf16Relu2) {
@@ -484,6 +509,8 @@ __global__ void __launch_bounds__(256) gemm_tail_finish_kernel(const float* __re
         } else if constexpr (EPI == GemmEpi::Residual) {
             const float4 o = *reinterpret_cast<const float4*>(p.Cf + off);
             *reinterpret_cast<float4*>(p.Cf + off) = make_float4(o.x + a.x, o.y + a.y, o.z + a.z, o.w + a.w);
+        } else if constexpr (EPI == GemmEpi::ResidualTanh) {
+            gemm_residual_tanh(p, *reinterpret_cast<const float4*>(p.Cf + off), a, off, n);
         } else {
             if constexpr (EPI == GemmEpi::Bf16Silu) a = gemm_silu_range(a, n, p);
             *reinterpret_cast<uint2*>(p.C + off) = make_uint2(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w));

@@ -133,7 +133,6 @@ __device__ __forceinline__ float glu(int kind, float g, float u, float limit) {
     u = fminf(fmaxf(u, -limit), limit);
     return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
 }
-__device__ __forceinline__ float tanh_norm(float x, float alpha, float w, float b) { return fmaf(tanhf(alpha * x), w, b); }
 __device__ __forceinline__ float cap_logit(float z, float scale, float softcap) {
     z *= scale;
     return softcap > 0.f ? softcap * tanhf(z / softcap) : z;

@@ -275,9 +275,9 @@ __global__ void __launch_bounds__(ln::kThreads) linear_attend_rows_kernel(const 
 // out[row][0 .. width) = rms(o) * norm * sigmoid(gate) * scale, columns up to `cols` zero.  One block per row; ld_o, cols multiples
 // of 4.  The first 1024 * KEEP channels stay in registers.
 template <typename T>
-__global__ void __launch_bounds__(256) linear_output_rows_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ proj, T* __restrict__ out, int ld_out,
+__global__ void __launch_bounds__(256, 5) linear_output_rows_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ proj, T* __restrict__ out, int ld_out,
                                                                  int cols, const LinearShape s) {
-    constexpr int KEEP = 4;
+    constexpr int KEEP = 2;
     __shared__ float part[8];
     const int row = blockIdx.x, tid = threadIdx.x, n = s.width();
     const float* src = o + (size_t)row * ld_o;

@@ -51,25 +51,23 @@ __device__ __forceinline__ uint4 load_head(const __nv_bfloat16* head, int c, int
         f[j] = (c + 2 * j < width ? (uint32_t)p[c + 2 * j] : 0u) | (c + 2 * j + 1 < width ? (uint32_t)p[c + 2 * j + 1] << 16 : 0u);
     return make_uint4(f[0], f[1], f[2], f[3]);
 }
-// rows [0, n) of a head into an image of `rows` rows and 8 cols8 channels, the rest zero; several loads of a thread in flight
+// rows [0, n) of a head into an image of `rows` rows and 8 cols8 channels, the rest zero: asynchronous copies where the head's
+// channels come in whole 16-byte pieces
 __device__ __forceinline__ void stage_head(unsigned char* dst, const __nv_bfloat16* head, int ld, int c0, int width, int n, int rows, int cols8) {
-    const bool vec = (reinterpret_cast<uintptr_t>(head) & 15) == 0;
-    constexpr int U = 4;
-    const int all = rows * cols8;
-    for (int i0 = threadIdx.x; i0 < all; i0 += U * kThreads) {
-        uint4 v[U];
-#pragma unroll
-        for (int u = 0; u < U; ++u) {
-            const int i = i0 + u * kThreads, r = i / cols8, c8 = i - r * cols8;
-            v[u] = i < all && r < n && c0 + 8 * c8 < width ? load_head(head + (size_t)r * ld, c0 + 8 * c8, width, vec) : make_uint4(0u, 0u, 0u, 0u);
-        }
-#pragma unroll
-        for (int u = 0; u < U; ++u) {
-            const int i = i0 + u * kThreads, r = i / cols8, c8 = i - r * cols8;
-            if (i < all) *reinterpret_cast<uint4*>(dst + image(r, c8)) = v[u];
-        }
+    const bool vec = ((reinterpret_cast<uintptr_t>(head) & 15) | (uintptr_t)(width & 7)) == 0;
+    const uint32_t to = tc::smem_u32(dst);
+    for (int i = threadIdx.x; i < rows * cols8; i += kThreads) {
+        const int r = i / cols8, c8 = i - r * cols8, c = c0 + 8 * c8;
+        const bool in = r < n && c < width;
+        if (vec)
+            asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(to + image(r, c8)), "l"(in ? head + (size_t)r * ld + c : head), "r"(in ? 16 : 0) : "memory");
+        else
+            *reinterpret_cast<uint4*>(dst + image(r, c8)) = in ? load_head(head + (size_t)r * ld, c, width, false) : make_uint4(0u, 0u, 0u, 0u);
     }
+    asm volatile("cp.async.commit_group;" ::: "memory");
 }
+template <int N>
+__device__ __forceinline__ void staged() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 __device__ __forceinline__ void fence_async_smem() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
 }  // namespace lt
 
@@ -101,8 +99,9 @@ __global__ void __launch_bounds__(lt::kThreads, 2) linear_chunk_tc_kernel(const 
     }
     const float* pw = s.powers + (size_t)h * (kLinearPowers + 1);
     const __nv_bfloat16 *k0 = proj + (size_t)(e.row0 + t0) * s.ld + s.off_k + h * s.D, *w0 = proj + (size_t)(e.row0 + t0) * s.ld + s.off_v + h * s.Dv;
+    stage_head(vs, w0, s.ld, v0, s.Dv, n, steps * 16, VP / 8);
     const bool vk = (reinterpret_cast<uintptr_t>(k0) & 15) == 0;
-    constexpr int U = 4;
+    constexpr int U = 8;
     for (int i0 = tid; i0 < steps * 16 * 16; i0 += U * kThreads) {   // all 128 key channels: the product has 128 rows
         uint4 x[U];
         float a[U];
@@ -123,7 +122,7 @@ __global__ void __launch_bounds__(lt::kThreads, 2) linear_chunk_tc_kernel(const 
             if (i < steps * 16 * 16) put_pair(khi, klo, i >> 4, i & 15, f);
         }
     }
-    stage_head(vs, w0, s.ld, v0, s.Dv, n, steps * 16, VP / 8);
+    staged<0>();
     fence_async_smem();
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();
@@ -201,22 +200,10 @@ __global__ void __launch_bounds__(lt::kThreads, 1) linear_attend_tc_kernel(const
     const __nv_bfloat16 *q0 = row + s.off_q + h * s.D, *k0 = row + s.off_k + h * s.D, *w0 = row + s.off_v + h * s.Dv;
     stage_head(p0, q0, s.ld, 0, s.D, n, C, 2 * dsteps);               // rows past n: zero, every row of the product is computed
     stage_head(p0 + K_OFF, k0, s.ld, 0, s.D, n, C, 2 * dsteps);
-    fence_async_smem();
-    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
-    __syncthreads();
-    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-    const uint32_t tmem = *tmem_slot;
-    if (tid == 0) {
-        constexpr uint32_t kDesc = at::instr_desc(128, 128);
-        for (int k = 0; k < dsteps; ++k)
-            at::umma_d(tmem, tc::umma_desc(base + (k >> 2) * BOX) + (uint64_t)((k & 3) * 2), tc::umma_desc(base + K_OFF + (k >> 2) * BOX) + (uint64_t)((k & 3) * 2), kDesc,
-                       k != 0 ? 1u : 0u);
-        tc::umma_commit(pbar);
-    }
-    // values and state while the products of queries and keys are under way
+    stage_head(p0 + V_OFF, w0, s.ld, v0, s.Dv, n, steps * 16, VP / 8);
     if (state) {
         const float* S = ws + ((size_t)blockIdx.x * s.heads + h) * s.head_floats();
-        constexpr int U = 2;
+        constexpr int U = 4;
         const int all = dsteps * 16 * (VP / 8);
         for (int i0 = tid; i0 < all; i0 += U * kThreads) {
             float4 a[U], b[U];
@@ -235,7 +222,20 @@ __global__ void __launch_bounds__(lt::kThreads, 1) linear_attend_tc_kernel(const
             }
         }
     }
-    stage_head(p0 + V_OFF, w0, s.ld, v0, s.Dv, n, steps * 16, VP / 8);
+    staged<1>();
+    fence_async_smem();
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    const uint32_t tmem = *tmem_slot;
+    if (tid == 0) {
+        constexpr uint32_t kDesc = at::instr_desc(128, 128);
+        for (int k = 0; k < dsteps; ++k)
+            at::umma_d(tmem, tc::umma_desc(base + (k >> 2) * BOX) + (uint64_t)((k & 3) * 2), tc::umma_desc(base + K_OFF + (k >> 2) * BOX) + (uint64_t)((k & 3) * 2), kDesc,
+                       k != 0 ? 1u : 0u);
+        tc::umma_commit(pbar);
+    }
+    staged<0>();
     fence_async_smem();
     bool ok = __all_sync(0xffffffffu, tc::mbar_wait(pbar, 0, abort_s));     // a warp accesses tensor memory as one
     if (!ok) *abort_s = 1;

@@ -169,7 +169,7 @@ void launch_attn_decode_v(Launcher& L, const WindowDecodeParams<TC>& p, int clus
     const int hb = (p.s.H / p.s.G + wd::kHeads - 1) / wd::kHeads, lin = (p.lin.units + cluster - 1) / cluster;
     L.cluster_x = cluster;
     const bool pdl = L.pdl;
-    L.pdl = pdl && !ROT;                                               // see InOrder
+    L.pdl = pdl && (!ROT || lin > 0);                                  // see InOrder; with linear attention the grid is larger
     L.launch(lin > 0 ? window_attention_decode_kernel<TC, VM, ROT, true> : window_attention_decode_kernel<TC, VM, ROT, false>, dim3(cluster, p.s.G * hb + lin),
              dim3(wd::kThreads), sizeof(wd::Smem<VM>), p);
     L.pdl = pdl;

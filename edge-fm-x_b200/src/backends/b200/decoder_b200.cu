@@ -638,6 +638,8 @@ efm_status efm_b200_decoder_step(efm_b200_ctx* c, const efm_step_entry* entries,
         }
         while (first < n_entries && done[first] == entries[first].n_tokens) ++first;
         if (n_ws > m.ws_pages) return fail(c, EFM_ERR_STATE, "the entries see more cache pages than the pool has");
+        // late rows see the most keys; the kernel takes the last tiles first
+        std::stable_sort(tc.begin(), tc.end(), [&](const RowTile& a, const RowTile& b) { return re[a.entry].pos0 + a.row < re[b.entry].pos0 + b.row; });
         // tiles of the tensor-core form go to the CUDA-core form in layers it does not take: list them in its units too
         std::vector<RowTile> all_simt;
         for (size_t i = 0; i < re.size(); ++i)

@@ -517,8 +517,9 @@ void launch_delta_scan(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, cons
 template <int DP, int VP, int RP, bool KEEP>
 void launch_attention_tc_v(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const WindowAttnShape& s, const WindowTcMaps& maps, const RowPlan& plan,
                            const RowTile* list, int n) {
-    L.launch(window_attention_tc_kernel<DP, VP, RP, KEEP>, dim3(n, s.H, (s.Vp + VP - 1) / VP), dim3(wt::kThreads), wt::Cfg<DP, VP, RP>::SMEM, maps, static_cast<__nv_bfloat16*>(c.decoder->mix),
-             l.mix_wp, s, plan, list, RP > 0 ? 1 : 0, &c.state->error);
+    const int blocks = n * s.H * ((s.Vp + VP - 1) / VP), first_wave = blocks <= 2 * c.num_sms ? std::min(blocks, c.num_sms) : blocks;
+    L.launch(window_attention_tc_kernel<DP, VP, RP, KEEP>, dim3(blocks), dim3(wt::kThreads), wt::Cfg<DP, VP, RP>::SMEM, maps, static_cast<__nv_bfloat16*>(c.decoder->mix),
+             l.mix_wp, s, plan, list, n, first_wave, RP > 0 ? 1 : 0, &c.state->error);
 }
 template <int RP, bool KEEP = false>
 void launch_attention_tc_r(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const WindowAttnShape& s, const WindowTcMaps& maps, const RowPlan& plan,

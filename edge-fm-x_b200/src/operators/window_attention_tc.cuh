@@ -5,9 +5,12 @@
 // place of the page in a workspace of keys and values expanded for this pass (latent attention).
 // Keys may come from two tensors: DP channels per kv head, and RP more that all heads share (a rotated part); the query rows
 // are split the same way.  Channels that a tensor does not have are filled with zeros by TMA.
-// Block = 128 rows of one entry x one head x (grid.z) VP value channels, 256 threads.  Wider values take several blocks, each of
-// which computes the scores for itself.  Rows of the tile that belong to the next entry are computed and
+// Block = 128 rows of one entry x one head x VP value channels, 256 threads.  Wider values take several blocks, each of which
+// computes the scores for itself.  Late rows see the most keys: blocks take them first, and the second half of what is resident at a
+// time from the other end, so that an SM's two blocks are a long and a short one.  Rows of the tile that belong to the next entry are computed and
 // not stored.  The weights enter P V as a bf16 pair high + low (16 bits of mantissa), written straight into tensor memory.
+// The products run behind the softmax: S of the next tile is issued as soon as every thread holds its scores, and P V of a tile is
+// folded into the registers one tile later, while the next weights are already on their way.
 // Every mbarrier wait is bounded and raises *error.
 #pragma once
 #include "attention_tc.cuh"
@@ -29,7 +32,7 @@ struct Cfg {
     static constexpr int P_COL = 64, O_COL = 128;
     static constexpr int TMEM_COLS = 256;                    // S (64 columns) | P high, P low (32 each) | O tile, power of two
     static constexpr int HALF = VP / 2;
-    static constexpr size_t SMEM = (size_t)Q_BYTES + KBUF * K_BYTES + V_BYTES + 2 * BM * 4 + 128 + kMaxTiles * 4 + 1024;
+    static constexpr size_t SMEM = (size_t)Q_BYTES + KBUF * K_BYTES + 2 * V_BYTES + 2 * BM * 4 + 128 + kMaxTiles * 4 + 1024;
 };
 
 __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16]) {
@@ -58,7 +61,8 @@ struct WindowTcMaps {
 template <int DP, int VP, int RP, bool KEEP>
 __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(const __grid_constant__ WindowTcMaps maps, __nv_bfloat16* __restrict__ out,
                                                                            int ld_out, const WindowAttnShape s, const RowPlan plan,
-                                                                           const RowTile* __restrict__ tiles, int workspace, int* error) {
+                                                                           const RowTile* __restrict__ tiles, int n_tiles_all, int first_wave, int workspace,
+                                                                           int* error) {
     using namespace wt;
     using at::instr_desc;
     using at::tma_load_3d;
@@ -75,18 +79,21 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     const uint32_t base = (raw + 1023u) & ~1023u;
     unsigned char* base_ptr = wt_smem + (base - raw);
     const uint32_t sQ = base, sK = sQ + C::Q_BYTES, sV = sK + C::KBUF * C::K_BYTES;
-    constexpr int XCH = C::Q_BYTES + C::KBUF * C::K_BYTES + C::V_BYTES;
+    constexpr int XCH = C::Q_BYTES + C::KBUF * C::K_BYTES + 2 * C::V_BYTES;
     float* xch = reinterpret_cast<float*>(base_ptr + XCH);                       // [2][BM]
-    const uint32_t bars = sV + C::V_BYTES + 2 * BM * 4;
-    const uint32_t qfull = bars, kfull0 = bars + 8, vfull = bars + 24, sbar = bars + 32, obar = bars + 40;
-    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(base_ptr + XCH + 2 * BM * 4 + 48);
+    const uint32_t bars = sV + 2 * C::V_BYTES + 2 * BM * 4;
+    const uint32_t qfull = bars, kfull0 = bars + 8, vfull0 = bars + 24, sbar = bars + 40, obar = bars + 48;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(base_ptr + XCH + 2 * BM * 4 + 56);
     volatile int* abort_s = reinterpret_cast<volatile int*>(tmem_slot + 1);
     int* pages = reinterpret_cast<int*>(base_ptr + XCH + 2 * BM * 4 + 128);
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int row = (warp & 3) * 32 + lane, hf = warp >> 2;       // TMEM lane = query row; which half of the columns
-    const int v0 = blockIdx.z * VP;                               // first value channel
-    const int bx = (int)gridDim.x - 1 - (int)blockIdx.x, h = blockIdx.y, g = h / (s.H / s.G);     // late rows first: they see most keys
+    // grid.x = tiles x (heads x slices); see the top
+    const int slices = (s.Vp + VP - 1) / VP, per_tile = s.H * slices;
+    const int rank = (int)blockIdx.x < first_wave ? (int)blockIdx.x : (int)gridDim.x - 1 - ((int)blockIdx.x - first_wave);
+    const int bx = n_tiles_all - 1 - rank / per_tile, h = rank % per_tile / slices, g = h / (s.H / s.G);
+    const int v0 = rank % slices * VP;                            // first value channel
     RowEntry e;
     int r0;
     if (tiles != nullptr) { const RowTile t = tiles[bx]; e = plan.entry(t.entry); r0 = t.row; }
@@ -102,7 +109,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     auto tile_page = [&](int i) { return KEEP && i < nk ? i : pg0 + i - nk; };
 
     if (tid == 0) {
-        mbar_init(qfull, 1); mbar_init(kfull0, 1); mbar_init(kfull0 + 8, 1); mbar_init(vfull, 1); mbar_init(sbar, 1); mbar_init(obar, 1);
+        mbar_init(qfull, 1); mbar_init(kfull0, 1); mbar_init(kfull0 + 8, 1); mbar_init(vfull0, 1); mbar_init(vfull0 + 8, 1); mbar_init(sbar, 1); mbar_init(obar, 1);
         *abort_s = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
@@ -119,7 +126,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
 
     constexpr uint32_t kDescS = instr_desc(BM, BN);
     constexpr uint32_t kDescO = instr_desc(BM, VP) | (1u << 16);
-    const uint64_t vdesc = at::umma_desc_mn(sV, (uint32_t)(BN * 128), 1024u);
+    const uint64_t vdesc[2] = {at::umma_desc_mn(sV, (uint32_t)(BN * 128), 1024u), at::umma_desc_mn(sV + C::V_BYTES, (uint32_t)(BN * 128), 1024u)};
     constexpr float kLog2e = 1.4426950408889634f;
     const float f2 = head_multiplier(s, h) * kLog2e;
     const float b2 = (s.bias ? distance_slope(h, s.H) : 0.f) * kLog2e;
@@ -128,7 +135,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     for (int i = 0; i < C::HALF; ++i) o[i] = 0.f;
     float m = -INFINITY, l = 0.f;
 
-    int last_k[2] = {-1, -1}, last_v = -1;                       // thread 0: tiles requested last
+    int last_k[2] = {-1, -1}, last_v[2] = {-1, -1};                       // thread 0: tiles requested last
     auto load_k = [&](int tile, int buf) {
         last_k[buf] = tile;
         mbar_expect_tx(kfull0 + 8 * buf, C::K_BYTES);
@@ -138,10 +145,11 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
             else tma_load_3d(sK + buf * C::K_BYTES + b * (BN * 128), &maps.kr, b * 64 - DP, 0, pages[tile], kfull0 + 8 * buf);
     };
     auto load_v = [&](int tile) {
-        last_v = tile;
+        const uint32_t b0 = (uint32_t)(tile & 1), vfull = vfull0 + 8 * b0;
+        last_v[tile & 1] = tile;
         mbar_expect_tx(vfull, C::V_BYTES);
 #pragma unroll
-        for (int b = 0; b < C::VB; ++b) tma_load_3d(sV + b * (BN * 128), &maps.v, v0 + b * 64, g, pages[tile], vfull);
+        for (int b = 0; b < C::VB; ++b) tma_load_3d(sV + b0 * C::V_BYTES + b * (BN * 128), &maps.v, v0 + b * 64, g, pages[tile], vfull);
     };
     auto issue_s = [&](int buf) {
 #pragma unroll
@@ -161,12 +169,25 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
         load_k(0, 0);
         if (C::KBUF > 1 && ntiles > 1) load_k(1, 1);
         load_v(0);
+        if (ntiles > 1) load_v(1);
         const bool ok = mbar_wait(qfull, 0, abort_s) && mbar_wait(kfull0, 0, abort_s);
         if (!ok) *abort_s = 1;
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         if (ok) issue_s(0);
     }
 
+    // O += P V of tile j, whose weights are relative to the maximum after that tile
+    float alpha_prev = 0.f;
+    auto fold = [&]() {
+        const uint32_t orow = tmem + ((uint32_t)((warp & 3) * 32) << 16) + (uint32_t)(C::O_COL + hf * C::HALF);
+#pragma unroll
+        for (int c0 = 0; c0 < C::HALF; c0 += 32) {
+            uint32_t r[32];
+            tc::tmem_ld32(orow + (uint32_t)c0, r);
+#pragma unroll
+            for (int i = 0; i < 32; ++i) o[c0 + i] = fmaf(o[c0 + i], alpha_prev, __uint_as_float(r[i]));
+        }
+    };
     for (int j = 0; j < ntiles; ++j) {
         if (!mbar_wait(sbar, (uint32_t)j & 1u, abort_s)) *abort_s = 1;
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -178,14 +199,29 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
         float mx = -INFINITY;
         const float bias0 = b2 * (float)(key0 - i_pos);
         const bool interior = (kb >= lo_max || (KEEP && kb + BN <= keep)) && kb + BN <= hi_min;
+        if (interior && b2 == 0.f) {                             // most tiles: every key visible
 #pragma unroll
-        for (int i = 0; i < 32; ++i) {
-            const float v = fmaf(__uint_as_float(sr[i]), f2, fmaf(b2, (float)i, bias0));
-            sc[i] = interior || ((key0 + i >= lo || (KEEP && key0 + i < keep)) && key0 + i < hi) ? v : -INFINITY;
-            mx = fmaxf(mx, sc[i]);
+            for (int i = 0; i < 32; ++i) {
+                sc[i] = __uint_as_float(sr[i]) * f2;
+                mx = fmaxf(mx, sc[i]);
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+                const float v = fmaf(__uint_as_float(sr[i]), f2, fmaf(b2, (float)i, bias0));
+                sc[i] = interior || ((key0 + i >= lo || (KEEP && key0 + i < keep)) && key0 + i < hi) ? v : -INFINITY;
+                mx = fmaxf(mx, sc[i]);
+            }
         }
         xch[hf * BM + row] = mx;
+        asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
         if (__syncthreads_or(*abort_s != 0)) break;             // every thread takes the same decision
+        if (C::KBUF > 1 && tid == 0 && j + 1 < ntiles) {         // every thread holds its scores: S of the next tile
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            if (mbar_wait(kfull0 + 8 * ((j + 1) % C::KBUF), (uint32_t)((j + 1) / C::KBUF) & 1u, abort_s)) issue_s((j + 1) % C::KBUF);
+            else *abort_s = 1;
+        }
+        __syncwarp();
         const float m_new = fmaxf(m, fmaxf(xch[row], xch[BM + row]));
         const float mb = m_new == -INFINITY ? 0.f : m_new;
         const float alpha = m == -INFINITY ? 0.f : at::ex2(m - mb);
@@ -200,39 +236,44 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
             pl[i >> 1] = pack_bf16(a - bf16lo(pk[i >> 1]), b - bf16hi(pk[i >> 1]));
         }
         l = l * alpha + rs;
+        if (j > 0) {                                             // P V of the previous tile has read its weights and values
+            if (!mbar_wait(obar, (uint32_t)(j - 1) & 1u, abort_s)) *abort_s = 1;
+            __syncwarp();
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            if (tid == 0 && j + 1 < ntiles && *abort_s == 0) load_v(j + 1);
+            __syncwarp();
+        }
         // P into tensor memory, where the MMA takes it as its A operand: lane = row, one column = two neighbouring keys
         const uint32_t prow = tmem + ((uint32_t)((warp & 3) * 32) << 16) + (uint32_t)(C::P_COL + hf * 16);
         wt::tmem_st16(prow, pk);
         wt::tmem_st16(prow + 32u, pl);
+        if (j > 0) fold();
+        alpha_prev = alpha;
         asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
         asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
         __syncthreads();
         if (tid == 0) {
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            bool ok = mbar_wait(vfull, (uint32_t)j & 1u, abort_s);
+            bool ok = mbar_wait(vfull0 + 8 * (j & 1), (uint32_t)(j >> 1) & 1u, abort_s);
             if (ok) {
 #pragma unroll
                 for (int k = 0; k < 2 * (BN / 16); ++k)              // high halves, then low halves
-                    wt::umma_ts(tmem + C::O_COL, tmem + (uint32_t)(C::P_COL + 8 * k), vdesc + (uint64_t)((k % (BN / 16)) * (2048 >> 4)), kDescO, k != 0 ? 1u : 0u);
+                    wt::umma_ts(tmem + C::O_COL, tmem + (uint32_t)(C::P_COL + 8 * k), vdesc[j & 1] + (uint64_t)((k % (BN / 16)) * (2048 >> 4)), kDescO, k != 0 ? 1u : 0u);
                 umma_commit(obar);
-                if (j + 1 < ntiles) {
+                if (C::KBUF == 1 && j + 1 < ntiles) {
                     ok = mbar_wait(kfull0 + 8 * ((j + 1) % C::KBUF), (uint32_t)((j + 1) / C::KBUF) & 1u, abort_s);
                     if (ok) issue_s((j + 1) % C::KBUF);
                 }
             }
             if (!ok) *abort_s = 1;
         }
-        if (!mbar_wait(obar, (uint32_t)j & 1u, abort_s)) *abort_s = 1;
+        __syncwarp();
+    }
+    if (!__syncthreads_or(*abort_s != 0)) {
+        if (!mbar_wait(obar, (uint32_t)(ntiles - 1) & 1u, abort_s)) *abort_s = 1;
+        __syncwarp();
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        if (tid == 0 && j + 1 < ntiles && *abort_s == 0) load_v(j + 1);             // P V of tile j has read the V buffer
-        const uint32_t orow = tmem + ((uint32_t)((warp & 3) * 32) << 16) + (uint32_t)(C::O_COL + hf * C::HALF);
-#pragma unroll
-        for (int c0 = 0; c0 < C::HALF; c0 += 32) {
-            uint32_t r[32];
-            tc::tmem_ld32(orow + (uint32_t)c0, r);
-#pragma unroll
-            for (int i = 0; i < 32; ++i) o[c0 + i] = fmaf(o[c0 + i], alpha, __uint_as_float(r[i]));
-        }
+        fold();
     }
 
     if (tid == 0 && *abort_s != 0) {                             // given up: let the copies in flight land (bounded) before leaving
@@ -240,7 +281,8 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
         (void)mbar_wait(qfull, 0, &go_on);
         for (int b = 0; b < 2; ++b)
             if (last_k[b] >= 0) (void)mbar_wait(kfull0 + 8 * b, (uint32_t)(last_k[b] / C::KBUF) & 1u, &go_on);
-        if (last_v >= 0) (void)mbar_wait(vfull, (uint32_t)last_v & 1u, &go_on);
+        for (int b = 0; b < 2; ++b)
+            if (last_v[b] >= 0) (void)mbar_wait(vfull0 + 8 * b, (uint32_t)(last_v[b] >> 1) & 1u, &go_on);
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();

@@ -86,12 +86,17 @@ __device__ __forceinline__ float gemm_tanh(float y) {
     return q < 0.02f ? p : t;
 }
 // four columns from n on: the new residual and its norm
-__device__ __forceinline__ void gemm_residual_tanh(const GemmParams& p, const float4& old, const float4& v, size_t off, int n) {
+struct GemmNorm { float alpha; uint2 w, b; };
+__device__ __forceinline__ GemmNorm gemm_norm(const GemmParams& p, int n) {
+    if (p.C == nullptr) return GemmNorm{0.f, make_uint2(0u, 0u), make_uint2(0u, 0u)};
+    return GemmNorm{__bfloat162float(*p.norm_alpha), *reinterpret_cast<const uint2*>(p.norm_w + n), *reinterpret_cast<const uint2*>(p.norm_b + n)};
+}
+__device__ __forceinline__ void gemm_residual_tanh(const GemmParams& p, const GemmNorm& k, const float4& old, const float4& v, size_t off) {
     const float4 x = make_float4(fmaf(p.mult, v.x, old.x), fmaf(p.mult, v.y, old.y), fmaf(p.mult, v.z, old.z), fmaf(p.mult, v.w, old.w));
     *reinterpret_cast<float4*>(p.Cf + off) = x;
     if (p.C == nullptr) return;
-    const float al = __bfloat162float(*p.norm_alpha);
-    const uint2 w = *reinterpret_cast<const uint2*>(p.norm_w + n), b = *reinterpret_cast<const uint2*>(p.norm_b + n);
+    const float al = k.alpha;
+    const uint2 w = k.w, b = k.b;
     *reinterpret_cast<uint2*>(p.C + off) = make_uint2(pack_bf16(fmaf(gemm_tanh(al * x.x), bf16lo(w.x), bf16lo(b.x)), fmaf(gemm_tanh(al * x.y), bf16hi(w.x), bf16hi(b.x))),
                                                       pack_bf16(fmaf(gemm_tanh(al * x.z), bf16lo(w.y), bf16lo(b.y)), fmaf(gemm_tanh(al * x.w), bf16hi(w.y), bf16hi(b.y))));
 }
@@ -297,30 +302,41 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
             item_coords(item, m0, n0, kb0, kb1, z);
             const int a = j & 1;
             const uint32_t use = (uint32_t)(j >> 1) & 1u;
-            if (!mbar_wait(accf0 + 8 * a, use, abort_s)) { *abort_s = 1; break; }
-            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            const uint32_t acc = tmem + ((uint32_t)(q * 32) << 16) + (uint32_t)(a * BN);
             constexpr int OUT_COLS = gemm_is_glu(EPI) ? BN / 2 : BN;
             const int ldc = gemm_is_glu(EPI) ? (p.N >> 1) : p.N;               // output row length
             const int nc0 = gemm_is_glu(EPI) ? (n0 >> 1) : n0;           // first output column of the tile
             const bool vec = (ldc & 3) == 0;
+            constexpr bool kPrev = EPI == GemmEpi::Residual || EPI == GemmEpi::ResidualTanh;
+            const int cl = (lane & 7) * 4;
+            // residual epilogues: the old values of a chunk are requested one chunk ahead, the first ones while the accumulator is
+            // still being computed
+            auto load_prev = [&](int c0, float4 (&pv)[8]) {
+#pragma unroll
+                for (int r0 = 0; r0 < 32; r0 += 4) {
+                    const int m = m0 + q * 32 + r0 + (lane >> 3), n = nc0 + c0 + cl;
+                    pv[r0 >> 2] = (vec && m < p.M && n + 3 < ldc) ? __ldcg(reinterpret_cast<const float4*>(p.Cf + (size_t)m * ldc + n))
+                                                                  : make_float4(0.f, 0.f, 0.f, 0.f);
+                }
+            };
+            float4 prev[8], next[8];
+            if constexpr (kPrev) load_prev(ch * (OUT_COLS / 2), next);
+            if (!mbar_wait(accf0 + 8 * a, use, abort_s)) { *abort_s = 1; break; }
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            const uint32_t acc = tmem + ((uint32_t)(q * 32) << 16) + (uint32_t)(a * BN);
             const size_t split_off = compact ? (size_t)item * (size_t)(BM * BN)
                                              : (!GROUPED && p.kb_per_split > 0 ? (size_t)z * (size_t)p.M * (size_t)p.N : 0);
 #pragma unroll 1
             for (int c0 = ch * (OUT_COLS / 2); c0 < (ch + 1) * (OUT_COLS / 2); c0 += 32) {
                 if (nc0 + c0 >= ldc) break;                                    // whole chunk outside the matrix
-                const int cl = (lane & 7) * 4;
-                // residual epilogue: all eight old values of the chunk are requested up front, before the accumulator is
-                // read and long before the first store (the
-                // compiler may not move a load of Cf above a store to Cf by itself), one round trip per chunk
-                float4 prev[8];
-                if constexpr (EPI == GemmEpi::Residual || EPI == GemmEpi::ResidualTanh) {
+                GemmNorm nk{};                                                 // of this lane's four columns
+                if constexpr (EPI == GemmEpi::ResidualTanh) {
+                    if (vec && nc0 + c0 + cl + 3 < ldc) nk = gemm_norm(p, nc0 + c0 + cl);
+                }
+                (void)nk;
+                if constexpr (kPrev) {
 #pragma unroll
-                    for (int r0 = 0; r0 < 32; r0 += 4) {
-                        const int m = m0 + q * 32 + r0 + (lane >> 3), n = nc0 + c0 + cl;
-                        prev[r0 >> 2] = (vec && m < p.M && n + 3 < ldc) ? __ldcg(reinterpret_cast<const float4*>(p.Cf + (size_t)m * ldc + n))
-                                                                     : make_float4(0.f, 0.f, 0.f, 0.f);
-                    }
+                    for (int i = 0; i < 8; ++i) prev[i] = next[i];
+                    if (c0 + 32 < (ch + 1) * (OUT_COLS / 2)) load_prev(c0 + 32, next);
                 }
                 float o[32];
                 if constexpr (gemm_is_glu(EPI)) {
@@ -388,7 +404,7 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
                             const float4 old = prev[r0 >> 2];
                             *reinterpret_cast<float4*>(p.Cf + off) = make_float4(old.x + v.x, old.y + v.y, old.z + v.z, old.w + v.w);
                         } else if constexpr (EPI == GemmEpi::ResidualTanh) {
-                            gemm_residual_tanh(p, prev[r0 >> 2], v, off, n);
+                            gemm_residual_tanh(p, nk, prev[r0 >> 2], v, off);
                         } else {
                             *reinterpret_cast<uint2*>(p.C + off) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
                         }
@@ -474,7 +490,7 @@ __global__ void __launch_bounds__(256) gemm_splitk_finish_kernel(const float* __
             const float4 o = *reinterpret_cast<const float4*>(p.Cf + i * 4);
             *reinterpret_cast<float4*>(p.Cf + i * 4) = make_float4(o.x + a.x, o.y + a.y, o.z + a.z, o.w + a.w);
         } else if constexpr (EPI == GemmEpi::ResidualTanh) {
-            gemm_residual_tanh(p, *reinterpret_cast<const float4*>(p.Cf + i * 4), a, i * 4, n);
+            gemm_residual_tanh(p, gemm_norm(p, n), *reinterpret_cast<const float4*>(p.Cf + i * 4), a, i * 4);
         } else {
             if constexpr (EPI == GemmEpi::Bf16Silu) a = gemm_silu_range(a, n, p);
             if constexpr (EPI == GemmEpi::Bf16Relu2) {
@@ -517,7 +533,7 @@ __global__ void __launch_bounds__(256) gemm_tail_finish_kernel(const float* __re
             const float4 o = *reinterpret_cast<const float4*>(p.Cf + off);
             *reinterpret_cast<float4*>(p.Cf + off) = make_float4(o.x + a.x, o.y + a.y, o.z + a.z, o.w + a.w);
         } else if constexpr (EPI == GemmEpi::ResidualTanh) {
-            gemm_residual_tanh(p, *reinterpret_cast<const float4*>(p.Cf + off), a, off, n);
+            gemm_residual_tanh(p, gemm_norm(p, n), *reinterpret_cast<const float4*>(p.Cf + off), a, off);
         } else {
             if constexpr (EPI == GemmEpi::Bf16Silu) a = gemm_silu_range(a, n, p);
             *reinterpret_cast<uint2*>(p.C + off) = make_uint2(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w));

@@ -7,6 +7,7 @@
 
 #include "../../layers/decoder.h"
 #include "../../layers/shared_launch.h"
+#include "../../operators/conv_limits.h"
 #include "../../operators/gemv.cuh"
 #include "../../operators/rotary.cuh"
 #define EFM_DECLARATIONS_ONLY
@@ -30,8 +31,11 @@ efm_status validate(const efm_decoder_desc& d, const efm_decoder_layer* layers) 
     if (d.compute_dtype != EFM_BF16 && d.compute_dtype != EFM_F32) return fail(nullptr, EFM_ERR_UNSUPPORTED, "compute_dtype must be bf16 or fp32");
     if (d.norm_layout < EFM_NORM_OUTPUT || d.norm_layout > EFM_NORM_INPUT) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, "unknown norm_layout");
     if (d.logit_softcap < 0.f) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, "logit_softcap must not be negative");
-    if (d.norm_layout != EFM_NORM_INPUT && (d.logit_scale != 1.0f || d.logit_softcap > 0.f))
-        return fail(nullptr, EFM_ERR_UNSUPPORTED, "scaled or capped logits behind output norms");
+    if (d.norm_layout != EFM_NORM_INPUT && (d.logit_scale != 1.0f || (d.logit_softcap > 0.f && d.norm_layout != EFM_NORM_OUTPUT)))
+        return fail(nullptr, EFM_ERR_UNSUPPORTED, "scaled logits, or capped ones behind a sandwich of norms");
+    if (d.conv_taps < 0 || d.conv_taps > kMaxConvTaps) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, "conv_taps must lie between 0 and 16");
+    if ((d.conv_taps > 0 || d.depth_average) && (d.norm_layout != EFM_NORM_OUTPUT || d.side_dim > 0 || d.loop_times > 1))
+        return fail(nullptr, EFM_ERR_UNSUPPORTED, "input convolutions and depth averages need output norms, no token input and no loop");
     if (d.norm_layout != EFM_NORM_OUTPUT && d.side_dim > 0) return fail(nullptr, EFM_ERR_UNSUPPORTED, "a token input behind normalised sublayer inputs");
     if (d.loop_times < 0 || (d.loop_times > 1 && (d.loop_start < 0 || d.loop_stop <= d.loop_start || d.loop_stop > d.num_layers)))
         return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, "the looped layers must be a span of the layers");
@@ -45,9 +49,14 @@ efm_status validate(const efm_decoder_desc& d, const efm_decoder_layer* layers) 
             if (l.kv_heads <= 0 || l.heads % l.kv_heads != 0 || l.vdim <= 0 || l.window < 0)
                 return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "heads must be a multiple of kv_heads, vdim positive, window >= 0");
             if (l.vdim > 256) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "vdim above 256");
-            if (l.keep_first < 0 || l.qk_norm < EFM_QK_NORM_WEIGHTED || l.qk_norm > EFM_QK_NORM_NONE) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "keep_first or qk_norm");
+            if (l.keep_first < 0 || l.qk_norm < EFM_QK_NORM_WEIGHTED || l.qk_norm > EFM_QK_NORM_ROW) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "keep_first or qk_norm");
             if (l.rot_kind != EFM_ROT_NONE && l.rot_dims > l.dim) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "more rotated channels than dim");
-            if (l.sink || l.out_gate) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "sink and out_gate belong to latent attention");
+            if (l.sink || (l.out_gate != EFM_GATE_NONE && l.out_gate != EFM_GATE_HEADS)) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "sinks and gates per channel belong to latent attention");
+            if (l.score_weights < EFM_WEIGHTS_SOFTMAX || l.score_weights > EFM_WEIGHTS_SIGMOID) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "unknown score_weights");
+            if (l.score_weights == EFM_WEIGHTS_SIGMOID && l.keep_first > 0) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "kept first tokens with sigmoid weights");
+            if ((l.score_weights != EFM_WEIGHTS_SOFTMAX || l.out_gate || l.out_bias || l.qk_norm == EFM_QK_NORM_ROW) && (l.mixer != EFM_MIXER_ATTENTION || d.norm_layout != EFM_NORM_OUTPUT))
+                return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "sigmoid weights, gates, output biases and norms over all heads belong to attention behind output norms");
+            if (l.score_weights != EFM_WEIGHTS_SOFTMAX && l.rot_kind != EFM_ROT_NONE) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "rotation with sigmoid weights");
             if (input && l.qkv_bias) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "biases behind elementwise input norms");
             if (l.mixer == EFM_MIXER_PARALLEL) {
                 if (!input) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "parallel mixers need input norms");
@@ -63,6 +72,17 @@ efm_status validate(const efm_decoder_desc& d, const efm_decoder_layer* layers) 
             if (l.rot_kind == EFM_ROT_NONE) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "latent attention has a rotated part");
             if (l.keep_first != 0) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "keep_first belongs to attention");
             if (l.out_gate < EFM_GATE_NONE || l.out_gate > EFM_GATE_HEADS) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "unknown out_gate");
+        } else if (l.mixer == EFM_MIXER_LINEAR) {
+            if (d.norm_layout != EFM_NORM_OUTPUT) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "linear attention alone needs output norms");
+            if (l.linear_heads <= 0 || l.linear_dim <= 0 || l.linear_vdim <= 0) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "linear attention needs positive sizes");
+            if (l.linear_dim > 256 || l.linear_vdim > 256) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "linear attention heads above 256 channels");
+            if (l.rot_kind != EFM_ROT_NONE && l.rot_dims > l.linear_dim) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "more rotated channels than dim");
+            if (!(l.linear_tau >= 0.f)) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "linear_tau must not be negative");
+            if (l.linear_tau > 0.f ? l.decay_rank <= 0 : l.linear_decay == nullptr) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "linear attention needs a decay per head, or decay_rank and linear_tau");
+            if (l.decay_rank > 512) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "decay_rank above 512");
+            if (l.linear_tau == 0.f)
+                for (int h = 0; h < l.linear_heads; ++h)
+                    if (!(l.linear_decay[h] >= 0.0 && l.linear_decay[h] <= 1.0)) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "decays must lie between 0 and 1");
         } else if (l.mixer == EFM_MIXER_GENERAL_DELTA) {
             if (l.decay_rank <= 0) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "decay_rank must be positive");
             if (l.decay_rank > 512) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "decay_rank above 512");
@@ -77,11 +97,15 @@ efm_status validate(const efm_decoder_desc& d, const efm_decoder_layer* layers) 
                 return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "a scaled rotation needs a positive factor, context and limits");
         }
         if (l.ff > 0 && l.ff_act != EFM_ACT_POLYNORM && l.ff_act != EFM_ACT_RELU2) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "unknown ff_act");
+        if (l.ff > 0 && (d.conv_taps > 0 || d.depth_average)) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "a dense feed-forward behind an input convolution");
         if (l.ff > 0 && l.ff_act == EFM_ACT_RELU2 && !input) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "a squared ReLU behind output norms");
         if (l.experts > 0) {
-            if (!input && (l.expert_glu != EFM_GLU_SILU || l.expert_weight_input || l.shared_ff > 0))
-                return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "clamped, input-weighted or shared experts behind output norms");
-            if (l.shared_ff < 0 || l.expert_glu < EFM_GLU_SILU || l.expert_glu > EFM_GLU_CLAMPED || l.expert_score < EFM_SCORE_SOFTMAX || l.expert_score > EFM_SCORE_SIGMOID)
+            const bool plain = l.expert_glu == EFM_GLU_NONE_RELU2;
+            if (!input && (l.expert_glu == EFM_GLU_CLAMPED || l.expert_weight_input || (l.shared_ff > 0 && !plain)))
+                return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "clamped, input-weighted or (with a gated unit) shared experts behind output norms");
+            if (plain && d.norm_layout != EFM_NORM_OUTPUT) return fail(nullptr, EFM_ERR_UNSUPPORTED, at + "experts without a gate need output norms");
+            if (l.expert_scale < 0.f || l.shared_gate < EFM_SHARED_GATED || l.shared_gate > EFM_SHARED_PLAIN) return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "expert_scale or shared_gate");
+            if (l.shared_ff < 0 || l.expert_glu < EFM_GLU_SILU || l.expert_glu > EFM_GLU_NONE_RELU2 || l.expert_score < EFM_SCORE_SOFTMAX || l.expert_score > EFM_SCORE_SIGMOID)
                 return fail(nullptr, EFM_ERR_INVALID_ARGUMENT, at + "unknown form of the experts");
             if (l.ff > 0 || l.expert_ff <= 0 || l.expert_top <= 0 || l.expert_groups <= 0 || l.expert_groups_kept <= 0 ||
                 l.expert_groups_kept > l.expert_groups || l.experts % l.expert_groups != 0 ||
@@ -189,6 +213,12 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
     EFM_TRY(cudaStreamCreateWithFlags(&c->stream, cudaStreamNonBlocking));
     for (auto& ev : c->events) EFM_TRY(cudaEventCreate(&ev));
     EFM_TRY(configure_sampler());
+    m->extended = desc->norm_layout == EFM_NORM_OUTPUT && (desc->conv_taps > 0 || desc->depth_average || desc->logit_softcap > 0.f);
+    for (int i = 0; i < desc->num_layers; ++i) {
+        const efm_decoder_layer& l = layers[i];
+        m->extended = m->extended || l.mixer == EFM_MIXER_LINEAR || l.out_bias || (l.experts > 0 && l.expert_glu == EFM_GLU_NONE_RELU2) ||
+                      (desc->norm_layout == EFM_NORM_OUTPUT && (l.experts > 0 || l.qkv_bias));
+    }
     const bool outputs = desc->norm_layout != EFM_NORM_INPUT, inputs = desc->norm_layout != EFM_NORM_OUTPUT, tanh = !outputs;
     for (int i = 0; i < desc->num_layers; ++i) {
         const int times = desc->loop_times > 1 && i == desc->loop_start ? desc->loop_times : 1;
@@ -205,6 +235,7 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
     const size_t rows = (size_t)std::max(desc->cache_pages, 1) * EFM_PAGE_TOKENS, es = act_bytes(*m);
     size_t w_in = 8, w_mix = 8, w_ff = 8, w_q = 8, w_delta_in = 8, n_pack = 8, w_rank = 8, w_cq = 8, k_max = Wp;
     size_t ws_c = 0, ws_kv = 0, n_experts = 0, w_route = 8, ex_ff = 0, top = 0, w_act = 8, n_lin = 0, w_lin = 0, sh_ff = 0;
+    size_t w_proj_f = 0, w_decay = 0;
     bool any_delta = false, any_dense = false, ws_full = false;
     m->layers.resize(desc->num_layers);
     for (int i = 0; i < desc->num_layers; ++i) {
@@ -213,17 +244,23 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
         const efm_decoder_layer& d = l.d;
         if (outputs) EFM_TRY(dev_alloc(c, &l.post1, Wp));
         if (inputs) EFM_TRY(alloc_norm(c, l.pre1, Wp, tanh));
+        if (desc->conv_taps > 0) {
+            EFM_TRY(dev_alloc(c, &l.canon1, (size_t)desc->conv_taps * Wp));
+            if (l.mlp()) EFM_TRY(dev_alloc(c, &l.canon2, (size_t)desc->conv_taps * Wp));
+        }
+        if (desc->depth_average) EFM_TRY(dev_alloc(c, &l.dwa, (size_t)i + 2));
         EFM_TRY(alloc_inv_freq(c, l));
         if (l.attention()) {
             l.Dp = round_up(d.dim, 64);
             l.Vp = round_up(d.vdim, 64);
             l.mix_w = d.heads * d.vdim;
             int n_in = (d.heads + d.kv_heads) * d.dim + d.kv_heads * d.vdim;
-            if (l.linear()) {
-                const int qk = d.linear_heads * d.linear_dim, v = d.linear_heads * d.linear_vdim;
+            if (d.out_gate) n_in += d.heads;
+            if (l.parallel()) {
+                const int v = d.linear_heads * d.linear_vdim;
                 l.lin_vp = round_up(d.linear_vdim, 4);
                 l.lin_in = round_up(n_in, 8);
-                n_in = l.lin_in + 2 * round_up(qk, 8) + 2 * round_up(v, 8);
+                n_in = l.lin_in + 2 * l.linear_qk() + 2 * l.linear_v();
                 l.lin_mix = round_up(l.mix_w, 8);
                 l.mix_w = l.lin_mix + v;
                 EFM_TRY(dev_alloc(c, &l.mix_norm, round_up(v, 8)));
@@ -233,10 +270,12 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
             }
             l.d.linear_decay = nullptr;
             EFM_TRY(alloc_linear(c, l.in, n_in, m->W, d.qkv_bias != 0));
-            if (d.qk_norm == EFM_QK_NORM_WEIGHTED) {
-                EFM_TRY(dev_alloc(c, &l.q_norm, d.dim));
-                EFM_TRY(dev_alloc(c, &l.k_norm, d.dim));
+            if (d.qk_norm == EFM_QK_NORM_WEIGHTED || d.qk_norm == EFM_QK_NORM_ROW) {
+                const bool row = d.qk_norm == EFM_QK_NORM_ROW;
+                EFM_TRY(dev_alloc(c, &l.q_norm, row ? d.heads * d.dim : d.dim));
+                EFM_TRY(dev_alloc(c, &l.k_norm, row ? d.kv_heads * d.dim : d.dim));
             }
+            if (d.score_weights == EFM_WEIGHTS_SIGMOID) EFM_TRY(dev_alloc(c, &l.shift, d.heads));
             if (d.head_temp) EFM_TRY(dev_alloc(c, &l.temp, d.heads));
             w_q = std::max(w_q, (size_t)d.heads * l.Dp);
             w_in = std::max(w_in, (size_t)l.in.Np);
@@ -263,6 +302,23 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
                 ws_full = ws_full || d.window == 0;
                 m->ws_window = std::max(m->ws_window, d.window);
             }
+        } else if (l.alone()) {
+            const int v = d.linear_heads * d.linear_vdim, rank = l.channel_decay() ? d.decay_rank : 0;
+            l.lin_vp = round_up(d.linear_vdim, 4);
+            l.mix_w = v;
+            EFM_TRY(alloc_linear(c, l.in, 2 * l.linear_qk() + 2 * l.linear_v() + rank, m->W));
+            if (d.linear_norm) EFM_TRY(dev_alloc(c, &l.mix_norm, d.linear_vdim));
+            if (rank > 0) {
+                EFM_TRY(alloc_linear(c, l.w2, d.linear_heads * d.linear_dim, rank, true));
+                w_decay = std::max(w_decay, (size_t)l.w2.Np);
+            } else {
+                EFM_TRY(alloc_powers(c, l));
+            }
+            l.d.linear_decay = nullptr;
+            n_lin = std::max(n_lin, decoder_linear_ws_floats(l, S, std::min(desc->max_slots, S)));
+            w_lin = std::max(w_lin, (size_t)l.linear_v());
+            w_in = std::max(w_in, (size_t)l.in.Np);
+            if (d.rot_kind != EFM_ROT_NONE && !m->f32) w_proj_f = std::max(w_proj_f, (size_t)l.in.Np);
         } else {
             any_delta = true;
             const int HD = d.heads * d.dim;
@@ -278,15 +334,15 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
         }
         l.mix_wp = round_up(l.mix_w, 8);
         w_mix = std::max(w_mix, (size_t)l.mix_wp);
-        EFM_TRY(alloc_linear(c, l.out, m->W, l.mix_w));
+        EFM_TRY(alloc_linear(c, l.out, m->W, l.mix_w, d.out_bias != 0));
         if (l.mlp()) {
             if (outputs) EFM_TRY(dev_alloc(c, &l.post2, Wp));
             if (inputs) EFM_TRY(alloc_norm(c, l.pre2, Wp, tanh));
         }
         if (l.moe()) {
             l.ffp = round_up(d.expert_ff, 64);
-            EFM_TRY(alloc_linear(c, l.router, d.experts + (d.shared_ff > 0 ? 1 : 0), m->W));
-            EFM_TRY(alloc_linear(c, l.expert_in, d.experts * 2 * l.ffp, m->W));
+            EFM_TRY(alloc_linear(c, l.router, d.experts + (d.shared_ff > 0 && d.shared_gate == EFM_SHARED_GATED ? 1 : 0), m->W));
+            EFM_TRY(alloc_linear(c, l.expert_in, d.experts * l.up_rows(l.ffp), m->W));
             EFM_TRY(alloc_linear(c, l.expert_out, d.experts * Wp, d.expert_ff, false, 64));
             n_experts = std::max(n_experts, (size_t)d.experts);
             w_route = std::max(w_route, (size_t)l.router.Np);
@@ -294,7 +350,7 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
             top = std::max(top, (size_t)d.expert_top);
             if (d.shared_ff > 0) {
                 l.sfp = round_up(d.shared_ff, 64);
-                EFM_TRY(alloc_linear(c, l.shared_in, 2 * l.sfp, m->W));
+                EFM_TRY(alloc_linear(c, l.shared_in, l.up_rows(l.sfp), m->W));
                 EFM_TRY(alloc_linear(c, l.shared_out, m->W, d.shared_ff, false, 64));
                 sh_ff = std::max(sh_ff, (size_t)l.sfp);
             }
@@ -322,12 +378,17 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
             r.state_off = m->state_stride;
             m->state_stride += (size_t)l.d.linear_heads * l.d.linear_dim * l.lin_vp;
         }
+        if (desc->conv_taps > 0) {
+            r.conv1_off = m->state_stride;
+            r.conv2_off = r.conv1_off + (size_t)desc->conv_taps * Wp;
+            m->state_stride = r.conv2_off + (l.mlp() ? (size_t)desc->conv_taps * Wp : 0);
+        }
         if (l.attention()) {
             EFM_TRY(dev_alloc(c, &k, rows * l.d.kv_heads * l.Dp * es));
             EFM_TRY(dev_alloc(c, &v, rows * l.d.kv_heads * l.Vp * es));
         } else if (l.d.mixer == EFM_MIXER_LATENT_ATTENTION) {
             EFM_TRY(dev_alloc(c, &k, rows * (l.Lc + l.Rc) * es));
-        } else {
+        } else if (!l.alone()) {
             r.state_off = m->state_stride;
             m->state_stride += ((size_t)l.d.heads * l.d.dim * l.d.dim + 3) / 4 * 4;
         }
@@ -338,8 +399,9 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
         int optin = 0;
         EFM_TRY(cudaDeviceGetAttribute(&optin, cudaDevAttrMaxSharedMemoryPerBlockOptin, device_id));
         size_t need = std::max(std::max(gemv_smem_bytes((int)k_max), gemv_ext_smem_bytes(Wp)), gemv_ext_smem_bytes((int)w_cq));
+        if (desc->conv_taps > 0) need = std::max(need, gemv_conv_smem_bytes(Wp));
         for (const DecoderLayer& l : m->layers)
-            if (l.linear()) need = std::max(need, gemv_ext_smem_bytes(l.out.Kp));
+            if (l.parallel()) need = std::max(need, gemv_ext_smem_bytes(l.out.Kp));
         if (need + 2048 > (size_t)optin) {
             efm_status s = fail(nullptr, EFM_ERR_UNSUPPORTED, "width / feed-forward size exceeds what the decode GEMV stages in shared memory");
             efm_b200_destroy(c);
@@ -366,7 +428,12 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
     };
     EFM_TRY(dev_alloc(c, &c->ids, S));
     EFM_TRY(dev_alloc(c, &c->resid, (size_t)S * Wp));
-    if (!m->f32 || inputs) EFM_TRY(act(&m->xa, (size_t)S * Wp));
+    if (!m->f32 || inputs || desc->conv_taps > 0) EFM_TRY(act(&m->xa, (size_t)S * Wp));
+    if (desc->depth_average) {
+        EFM_TRY(dev_alloc(c, &m->hist, ((size_t)desc->num_layers + 1) * S * Wp));
+        EFM_TRY(dev_alloc(c, &m->d_hist, ((size_t)desc->num_layers + 1) * Wp));
+        EFM_TRY(dev_alloc(c, &m->d_avg, Wp));
+    }
     EFM_TRY(act(&m->cq, S * w_cq));
     if (ws_c > 0) {
         // the rows' own pages plus, for every entry long enough, those of a window
@@ -418,11 +485,13 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
     EFM_TRY(dev_alloc(c, &m->side_f, (size_t)S * m->side_p));
     EFM_TRY(dev_alloc(c, &m->y, (size_t)S * Wp));
     if (any_delta) {
-        EFM_TRY(dev_alloc(c, &m->proj_f, S * w_delta_in));
         EFM_TRY(dev_alloc(c, &m->pack, n_pack));
         EFM_TRY(dev_alloc(c, &m->tanh_w, S * w_rank));
-        EFM_TRY(dev_alloc(c, &m->decay, S * w_mix));
+        w_proj_f = std::max(w_proj_f, w_delta_in);
+        w_decay = std::max(w_decay, w_mix);
     }
+    if (w_proj_f > 0) EFM_TRY(dev_alloc(c, &m->proj_f, S * w_proj_f));
+    if (w_decay > 0) EFM_TRY(dev_alloc(c, &m->decay, S * w_decay));
     m->max_want = std::min(S, 256);
     EFM_TRY(act(&m->head_a, (size_t)m->max_want * Wp));
     EFM_TRY(dev_alloc(c, &m->logits_rows, (size_t)m->max_want * m->head.Np));
@@ -735,7 +804,8 @@ efm_status efm_b200_decoder_read_taps(efm_b200_ctx* c, float* host_out) {
 namespace {
 
 // ---- weights -------------------------------------------------------------------------------------------------------
-// Rows [src, src + n) of a tensor become rows [dst, dst + n) of a (fused, padded) linear, from column `col` on.
+// Rows [src, src + n) of a tensor become rows [dst, dst + n) of a (fused, padded) linear, from column `col` on.  Several tensors may
+// be parts of one linear.
 struct Piece { int dst, src, n, col = 0; };
 
 efm_status put_rows(efm_b200_ctx* c, const DecLinear& w, const std::vector<Piece>& pieces, const void* data, const std::string& name, const int64_t* shape,
@@ -755,7 +825,15 @@ efm_status put_vec(efm_b200_ctx* c, __nv_bfloat16* dst, int n, const void* data,
 }
 
 // Where a tensor goes: a row range of a (fused) linear or a vector.
-struct Target { DecLinear* lin = nullptr; std::vector<Piece> pieces; int cols = 0; __nv_bfloat16* vec = nullptr; int n = 0; };
+// taps > 0: [n, taps] into the vector, tap by tap (row stride ld).
+struct Target { DecLinear* lin = nullptr; std::vector<Piece> pieces; int cols = 0; __nv_bfloat16* vec = nullptr; int n = 0, taps = 0, ld = 0; };
+efm_status put_taps(efm_b200_ctx* c, const Target& t, const void* data, const std::string& name, const int64_t* shape, int ndim, int mem_kind) {
+    if (!shape_is(shape, ndim, t.n, t.taps)) return fail(c, EFM_ERR_INVALID_ARGUMENT, "unexpected shape for " + name);
+    for (int j = 0; j < t.taps; ++j)
+        EFM_CK(c, cudaMemcpy2DAsync(t.vec + (size_t)j * t.ld, 2, static_cast<const char*>(data) + (size_t)j * 2, (size_t)t.taps * 2, 2, (size_t)t.n,
+                                    mem_kind == EFM_MEM_DEVICE ? cudaMemcpyDeviceToDevice : cudaMemcpyHostToDevice, c->stream));
+    return EFM_OK;
+}
 
 // `name`, `name`.b or `name`.alpha of an input norm
 bool norm_target(const DecoderModel& m, const DecNorm& n, const std::string& what, const char* name, Target* t) {
@@ -766,7 +844,7 @@ bool norm_target(const DecoderModel& m, const DecNorm& n, const std::string& wha
     return t->vec != nullptr;
 }
 
-bool layer_target(DecoderModel& m, DecoderLayer& l, const std::string& rest, Target* t) {
+bool layer_target(DecoderModel& m, DecoderLayer& l, int index, const std::string& rest, Target* t) {
     const efm_decoder_layer& d = l.d;
     auto lin = [&](DecLinear& w, int row0, int rows) { t->lin = &w; t->pieces.push_back(Piece{row0, 0, rows}); return true; };
     auto vec = [&](__nv_bfloat16* v, int n) { t->vec = v; t->n = n; return v != nullptr; };
@@ -788,8 +866,29 @@ bool layer_target(DecoderModel& m, DecoderLayer& l, const std::string& rest, Tar
     }
     if (sandwich && rest == "norm1b") return vec(l.post1, m.W);
     if (sandwich && rest == "norm2b") return vec(l.post2, m.W);
-    if (rest == "mix.o" && !l.linear()) return lin(l.out, 0, m.W);
-    if (l.linear()) {                                  // the two halves share one projection and one output product
+    if (rest == "canon1" || rest == "canon2") {
+        t->vec = rest == "canon1" ? l.canon1 : l.canon2;
+        t->n = m.W;
+        t->taps = m.d.conv_taps;
+        t->ld = m.Wp;
+        return t->vec != nullptr;
+    }
+    if (rest == "dwa") return vec(l.dwa, index + 2);
+    if (rest == "mix.o" && !l.parallel()) return lin(l.out, 0, m.W);
+    if (rest == "mix.o.b") return vec(l.out.bias, m.W);
+    if (l.alone()) {
+        const int qk = d.linear_heads * d.linear_dim, v = d.linear_heads * d.linear_vdim, g = 2 * l.linear_qk() + l.linear_v();
+        if (rest == "mix.q") return lin(l.in, 0, qk);
+        if (rest == "mix.k") return lin(l.in, l.linear_qk(), qk);
+        if (rest == "mix.v") return lin(l.in, 2 * l.linear_qk(), v);
+        if (rest == "mix.g") return lin(l.in, g, v);
+        if (rest == "mix.norm") return vec(l.mix_norm, d.linear_vdim);
+        if (l.channel_decay()) {
+            if (rest == "mix.a1") return lin(l.in, g + l.linear_v(), d.decay_rank);
+            if (rest == "mix.a2") return lin(l.w2, 0, qk);
+            if (rest == "mix.a2.b") return vec(l.w2.bias, qk);
+        }
+    } else if (l.parallel()) {                                  // the two halves share one projection and one output product
         const int q = d.heads * d.dim, k = d.kv_heads * d.dim, lv = d.linear_heads * d.linear_vdim, lq = d.linear_heads * d.linear_dim;
         auto out = [&](int col, int cols) { t->lin = &l.out; t->cols = cols; t->pieces.push_back(Piece{0, 0, m.W, col}); return true; };
         if (rest == "mix.left.q") return lin(l.in, 0, q);
@@ -808,8 +907,11 @@ bool layer_target(DecoderModel& m, DecoderLayer& l, const std::string& rest, Tar
         if (rest == "mix.q") return lin(l.in, 0, q);
         if (rest == "mix.k") return lin(l.in, q, k);
         if (rest == "mix.v") return lin(l.in, q + k, d.kv_heads * d.vdim);
-        if (rest == "mix.q.norm") return vec(l.q_norm, d.dim);
-        if (rest == "mix.k.norm") return vec(l.k_norm, d.dim);
+        const bool row = d.qk_norm == EFM_QK_NORM_ROW;
+        if (rest == "mix.q.norm") return vec(l.q_norm, row ? q : d.dim);
+        if (rest == "mix.k.norm") return vec(l.k_norm, row ? k : d.dim);
+        if (rest == "mix.pb") return vec(l.shift, d.heads);
+        if (rest == "mix.g" && d.out_gate) return lin(l.in, q + k + d.kv_heads * d.vdim, d.heads);
         if (rest == "mix.temp") return vec(l.temp, d.heads);
         if (d.qkv_bias) {
             if (rest == "mix.q.b") return vec(l.in.bias, q);
@@ -844,6 +946,7 @@ bool layer_target(DecoderModel& m, DecoderLayer& l, const std::string& rest, Tar
     if (l.moe()) {
         if (rest == "mlp.router") return lin(l.router, 0, d.experts);
         auto gate_up = [&](DecLinear& w, int row0, int n, bool up) {     // 64 gate rows, the 64 matching up rows, ...
+            if (!l.gated_experts()) return up && lin(w, row0, n);
             t->lin = &w;
             for (int r = 0; r < n; r += 64) t->pieces.push_back(Piece{row0 + 2 * r + (up ? 64 : 0), r, std::min(64, n - r)});
             return true;
@@ -851,7 +954,7 @@ bool layer_target(DecoderModel& m, DecoderLayer& l, const std::string& rest, Tar
         if (d.shared_ff > 0) {
             if (rest == "mlp.shared.gate" || rest == "mlp.shared.up") return gate_up(l.shared_in, 0, d.shared_ff, rest == "mlp.shared.up");
             if (rest == "mlp.shared.down") return lin(l.shared_out, 0, m.W);
-            if (rest == "mlp.shared.sg") return lin(l.router, d.experts, 1);
+            if (rest == "mlp.shared.sg" && d.shared_gate == EFM_SHARED_GATED) return lin(l.router, d.experts, 1);
         }
         const size_t dot = rest.find('.', 5);
         if (rest.compare(0, 5, "mlp.e") == 0 && dot != std::string::npos && dot > 5) {
@@ -860,7 +963,7 @@ bool layer_target(DecoderModel& m, DecoderLayer& l, const std::string& rest, Tar
             if (rest.substr(5, dot - 5) != std::to_string(e) || e >= d.experts) return false;
             if (what == "down") return lin(l.expert_out, e * m.Wp, m.W);
             if (what != "gate" && what != "up") return false;
-            return gate_up(l.expert_in, e * 2 * l.ffp, d.expert_ff, what == "up");
+            return gate_up(l.expert_in, e * l.up_rows(l.ffp), d.expert_ff, what == "up");
         }
     } else if (d.ff > 0) {
         if (rest == "mlp.up") return lin(l.up, 0, d.ff);
@@ -890,12 +993,12 @@ efm_status decoder_set_weight(efm_b200_ctx* c, const char* raw, const void* data
     else if (name.size() > 1 && name[0] == 'l' && name[1] >= '0' && name[1] <= '9') {
         const size_t dot = name.find('.');
         const int i = std::atoi(name.c_str() + 1);
-        if (dot == std::string::npos || i < 0 || i >= m.d.num_layers || !layer_target(m, m.layers[i], name.substr(dot + 1), &t)) return EFM_OK;
+        if (dot == std::string::npos || i < 0 || i >= m.d.num_layers || !layer_target(m, m.layers[i], i, name.substr(dot + 1), &t)) return EFM_OK;
     } else {
         return EFM_OK;                     // not part of this model
     }
     if (dtype != EFM_BF16) return fail(c, EFM_ERR_UNSUPPORTED, "weights must be bf16: " + name);
-    const efm_status st = t.lin != nullptr ? put_rows(c, *t.lin, t.pieces, data, name, shape, ndim, mem_kind, t.cols)
+    const efm_status st = t.taps > 0 ? put_taps(c, t, data, name, shape, ndim, mem_kind) : t.lin != nullptr ? put_rows(c, *t.lin, t.pieces, data, name, shape, ndim, mem_kind, t.cols)
                                            : put_vec(c, t.vec, t.n, data, name, shape, ndim, mem_kind);
     if (st != EFM_OK) return st;
     EFM_CK(c, cudaStreamSynchronize(c->stream));          // the caller may release `data` on return
@@ -914,12 +1017,18 @@ efm_status decoder_finalize(efm_b200_ctx* c) {
         const efm_decoder_layer& d = m.layers[i].d;
         auto add = [&](std::initializer_list<const char*> names) { for (const char* n : names) need.push_back("l" + std::to_string(i) + "." + n); };
         add({"norm1"});
+        if (m.d.conv_taps > 0) add({"canon1"});
+        if (m.layers[i].canon2 != nullptr) add({"canon2"});
+        if (m.d.depth_average) add({"dwa"});
+        if (d.out_bias) add({"mix.o.b"});
         if (tanh) add({"norm1.b", "norm1.alpha"});
         if (d.mixer != EFM_MIXER_PARALLEL) add({"mix.o"});
         if (m.d.norm_layout == EFM_NORM_SANDWICH) add({"norm1b"});
         if (d.mixer == EFM_MIXER_ATTENTION) {
             add({"mix.q", "mix.k", "mix.v"});
-            if (d.qk_norm == EFM_QK_NORM_WEIGHTED) add({"mix.q.norm", "mix.k.norm"});
+            if (d.qk_norm == EFM_QK_NORM_WEIGHTED || d.qk_norm == EFM_QK_NORM_ROW) add({"mix.q.norm", "mix.k.norm"});
+            if (d.score_weights == EFM_WEIGHTS_SIGMOID) add({"mix.pb"});
+            if (d.out_gate) add({"mix.g"});
             if (d.head_temp) add({"mix.temp"});
             if (d.qkv_bias) add({"mix.q.b", "mix.k.b", "mix.v.b"});
         } else if (d.mixer == EFM_MIXER_PARALLEL) {
@@ -928,6 +1037,10 @@ efm_status decoder_finalize(efm_b200_ctx* c) {
             add({"mix.dq", "mix.dq.norm", "mix.uq", "mix.dkv", "mix.dkv.norm", "mix.uk", "mix.uv"});
             if (d.sink) add({"mix.sink"});
             if (d.out_gate) add({"mix.g"});
+        } else if (d.mixer == EFM_MIXER_LINEAR) {
+            add({"mix.q", "mix.k", "mix.v", "mix.g"});
+            if (d.linear_norm) add({"mix.norm"});
+            if (d.linear_tau > 0.f) add({"mix.a1", "mix.a2", "mix.a2.b"});
         } else add({"mix.r", "mix.k", "mix.v", "mix.g", "mix.a", "mix.a.b", "mix.w1", "mix.w2", "mix.w0", "mix.norm"});
         if (d.experts > 0 || d.ff > 0) {
             add({"norm2"});
@@ -936,9 +1049,15 @@ efm_status decoder_finalize(efm_b200_ctx* c) {
         }
         if (d.experts > 0) {
             add({"mlp.router"});
-            if (d.shared_ff > 0) add({"mlp.shared.gate", "mlp.shared.up", "mlp.shared.down", "mlp.shared.sg"});
+            const bool gated = d.expert_glu != EFM_GLU_NONE_RELU2;
+            if (d.shared_ff > 0) {
+                add({"mlp.shared.up", "mlp.shared.down"});
+                if (gated) add({"mlp.shared.gate"});
+                if (d.shared_gate == EFM_SHARED_GATED) add({"mlp.shared.sg"});
+            }
             for (int e = 0; e < d.experts; ++e)
-                for (const char* what : {".gate", ".up", ".down"}) add({("mlp.e" + std::to_string(e) + what).c_str()});
+                for (const char* what : {".gate", ".up", ".down"})
+                    if (gated || what[1] != 'g') add({("mlp.e" + std::to_string(e) + what).c_str()});
         } else if (d.ff > 0) {
             add({"mlp.up", "mlp.down"});
             if (d.ff_act == EFM_ACT_POLYNORM) add({"mlp.act"});
@@ -996,12 +1115,13 @@ int64_t decoder_step_bytes(const efm_b200_ctx& c, int32_t kv_len) {
     for (const DecoderRun& r : m.runs) {
         const DecoderLayer& l = m.layers[r.layer];
         b += lin(l.in) + lin(l.out) + lin(l.w2) + lin(l.up) + lin(l.down) + lin(l.gate) + lin(l.proj) + lin(l.uq) + lin(l.ukv) + lin(l.router) + lin(l.shared_in) + lin(l.shared_out);
-        if (l.moe()) b += (int64_t)l.d.expert_top * 3 * l.d.expert_ff * m.W * 2;
+        if (l.moe()) b += (int64_t)l.d.expert_top * (l.gated_experts() ? 3 : 2) * l.d.expert_ff * m.W * 2;
+        if (m.d.conv_taps > 0) b += (int64_t)(l.mlp() ? 2 : 1) * m.d.conv_taps * m.W * 6;
         const int64_t n = l.d.window > 0 ? std::min(kv_len, l.d.window + l.d.keep_first) : kv_len;
         if (l.linear()) b += 2 * (int64_t)l.d.linear_heads * l.d.linear_dim * l.lin_vp * 4;
         if (l.attention()) b += n * l.d.kv_heads * (l.d.dim + l.d.vdim) * (m.f32 ? 4 : 2);
         else if (l.d.mixer == EFM_MIXER_LATENT_ATTENTION) b += n * (l.d.kv_rank + l.d.rot_dims) * (m.f32 ? 4 : 2);
-        else b += 2 * (int64_t)l.d.heads * l.d.dim * l.d.dim * 4;
+        else if (!l.alone()) b += 2 * (int64_t)l.d.heads * l.d.dim * l.d.dim * 4;
     }
     return b;
 }

@@ -14,6 +14,10 @@
 // "parallel" {left {heads, kv_heads, dim, vdim, scale, rot}, right {heads, dim, vdim, decay}, left_scale, right_scale}; rot {base,
 // dims, scaling {factor, original, fast, slow}}; mlp null, {kind: "dense", ff} or {kind: "moe", expert {ff, limit}, router
 // {experts, top}, shared {ff, limit}}; "norm.eps", "residual_mult", "logit_scale", "logit_softcap", "vocab", "width".
+//
+// Viladra: "layers" lists {type, mixer, mlp}; type "retention" {heads, dim, vdim, decay, rot {base, dims}}, "gla" {heads, dim, vdim, tau}
+// or "attention" {heads, kv_heads, dim, vdim, scale, mask.size}; mlp null or {kind: "moe", expert.ff, router {experts, top, scale},
+// shared.ff}; "canon.taps", "embedding.scale", "norm.eps", "logit_softcap", "vocab", "width".
 #include <efm_b200.h>
 
 #include <algorithm>
@@ -207,6 +211,15 @@ DecoderConfig temuvik_config(const json::Value& cfg, const Shapes&) {
     return out;
 }
 
+void read_decay(const json::Value& mix, int32_t heads, const std::string& in, std::vector<double>& decay) {
+    const json::Value& d = member(mix, "decay", in);
+    if (!d.is_array() || (int32_t)d.arr.size() != heads) throw ConfigurationError("config.json: " + in + ".decay must list one number per head");
+    for (const json::Value& v : d.arr) {
+        if (!v.is_number()) throw ConfigurationError("config.json: " + in + ".decay must list one number per head");
+        decay.push_back(v.num);
+    }
+}
+
 void read_parallel(const json::Value& mix, const std::string& in, efm_decoder_layer& e, std::vector<double>& decay) {
     e.mixer = EFM_MIXER_PARALLEL;
     const json::Value &left = member(mix, "left", in), &right = member(mix, "right", in);
@@ -223,12 +236,7 @@ void read_parallel(const json::Value& mix, const std::string& in, efm_decoder_la
     e.linear_vdim = positive(right, "vdim", r);
     e.mix_scale = number(mix, "left_scale", in);
     e.linear_scale = number(mix, "right_scale", in);
-    const json::Value& d = member(right, "decay", r);
-    if (!d.is_array() || (int32_t)d.arr.size() != e.linear_heads) throw ConfigurationError("config.json: " + r + ".decay must list one number per head");
-    for (const json::Value& v : d.arr) {
-        if (!v.is_number()) throw ConfigurationError("config.json: " + r + ".decay must list one number per head");
-        decay.push_back(v.num);
-    }
+    read_decay(right, e.linear_heads, r, decay);
 }
 
 DecoderConfig vekolix_config(const json::Value& cfg, const Shapes&) {
@@ -271,6 +279,74 @@ DecoderConfig vekolix_config(const json::Value& cfg, const Shapes&) {
                 e.shared_ff = positive(*shared, "ff", ff + ".shared");
                 e.shared_limit = number(*shared, "limit", ff + ".shared");
             }
+        }
+        out.layers.push_back(e);
+    }
+    d.num_layers = (int32_t)out.layers.size();
+    return out;
+}
+
+DecoderConfig viladra_config(const json::Value& cfg, const Shapes& shapes) {
+    DecoderConfig out;
+    efm_decoder_desc& d = out.desc;
+    read_model(cfg, d);
+    d.norm_layout = EFM_NORM_OUTPUT;
+    d.tied_head = 1;
+    d.depth_average = 1;
+    d.conv_taps = positive(member(cfg, "canon", "model"), "taps", "canon");
+    d.embed_scale = number(member(cfg, "embedding", "model"), "scale", "embedding");
+    d.logit_softcap = number(cfg, "logit_softcap", "model");
+    if (!(d.logit_softcap > 0.f)) throw ConfigurationError("config.json: logit_softcap must be positive");
+    const json::Value& layers = layer_list(cfg);
+    out.decays.resize(layers.arr.size());
+    for (size_t i = 0; i < layers.arr.size(); ++i) {
+        const json::Value& l = layers.arr[i];
+        const std::string where = "layers[" + std::to_string(i) + "]", in = where + ".mixer", ff = where + ".mlp";
+        const json::Value& mix = member(l, "mixer", where);
+        const std::string type = l.get_string("type", "");
+        efm_decoder_layer e{};
+        e.heads = positive(mix, "heads", in);
+        e.dim = positive(mix, "dim", in);
+        e.vdim = positive(mix, "vdim", in);
+        if (type == "attention") {
+            e.mixer = EFM_MIXER_ATTENTION;
+            e.kv_heads = positive(mix, "kv_heads", in);
+            e.scale = number(mix, "scale", in);
+            e.qk_norm = EFM_QK_NORM_ROW;
+            e.qkv_bias = e.out_bias = 1;
+            e.score_weights = EFM_WEIGHTS_SIGMOID;
+            e.out_gate = EFM_GATE_HEADS;
+            const json::Value* mask = mix.find("mask");
+            if (given(mask)) e.window = positive(*mask, "size", in + ".mask");
+        } else if (type == "retention" || type == "gla") {
+            e.mixer = EFM_MIXER_LINEAR;
+            e.linear_heads = e.heads;
+            e.linear_dim = e.dim;
+            e.linear_vdim = e.vdim;
+            if (type == "retention") {
+                read_rotation(mix, EFM_ROT_HALF, in, e);
+                read_decay(mix, e.heads, in, out.decays[i]);
+            } else {
+                e.linear_norm = 1;
+                e.linear_tau = number(mix, "tau", in);
+                if (!(e.linear_tau > 0.f)) throw ConfigurationError("config.json: " + in + ".tau must be positive");
+                const std::string a1 = "l" + std::to_string(i) + ".mix.a1";
+                const auto it = shapes.find(a1);
+                if (it == shapes.end() || it->second.size() != 2) throw ModelNotLoadedError("checkpoint lacks " + a1);
+                e.decay_rank = (int32_t)it->second[0];
+            }
+        } else {
+            throw ConfigurationError("config.json: " + where + " has an unknown type \"" + type + "\"");
+        }
+        const json::Value* mlp = l.find("mlp");
+        if (given(mlp)) {
+            read_experts(*mlp, ff, e);
+            e.expert_glu = EFM_GLU_NONE_RELU2;
+            e.expert_scale = number(member(*mlp, "router", ff), "scale", ff + ".router");
+            if (!(e.expert_scale > 0.f)) throw ConfigurationError("config.json: " + ff + ".router.scale must be positive");
+            e.shared_gate = EFM_SHARED_PLAIN;
+            const json::Value* shared = mlp->find("shared");
+            if (given(shared)) e.shared_ff = positive(*shared, "ff", ff + ".shared");
         }
         out.layers.push_back(e);
     }
@@ -350,7 +426,9 @@ ModelSetup build_decoder(const EngineConfig& config, DecoderConfig (*read)(const
         states += 1 + (r.prefix_token_ids.empty() ? 0 : 1);
     }
     if (pages <= 0) throw ConfigurationError("kvcache declares neither requests nor pool_tokens");
-    const bool recurrent = std::any_of(dc.layers.begin(), dc.layers.end(), [](const efm_decoder_layer& l) { return l.mixer == EFM_MIXER_GENERAL_DELTA || l.mixer == EFM_MIXER_PARALLEL; });
+    const bool recurrent = d.conv_taps > 0 || std::any_of(dc.layers.begin(), dc.layers.end(), [](const efm_decoder_layer& l) {
+        return l.mixer == EFM_MIXER_GENERAL_DELTA || l.mixer == EFM_MIXER_PARALLEL || l.mixer == EFM_MIXER_LINEAR;
+    });
     d.cache_pages = (int32_t)pages;
     d.state_slots = recurrent ? states : 0;
     d.max_slots = (int32_t)reqs.size() + live;
@@ -405,9 +483,12 @@ ModelSetup build_temuvik(const EngineConfig& config) { return build_decoder(conf
 
 ModelSetup build_vekolix(const EngineConfig& config) { return build_decoder(config, vekolix_config); }
 
+ModelSetup build_viladra(const EngineConfig& config) { return build_decoder(config, viladra_config); }
+
 const ModelRegistrar kFolizen({"folizen", {"Folizen"}, build_folizen});
 const ModelRegistrar kTemuvik({"temuvik", {"Temuvik"}, build_temuvik});
 const ModelRegistrar kVekolix({"vekolix", {"Vekolix"}, build_vekolix});
+const ModelRegistrar kViladra({"viladra", {"Viladra"}, build_viladra});
 
 }  // namespace
 

@@ -33,7 +33,7 @@ const ModelFamily& ModelRegistry::resolve(const EngineConfig& config) {
         if (f.name == name) return f;
     std::string known;
     for (const std::string& n : names()) known += (known.empty() ? "" : ", ") + n;
-    throw ConfigurationError("Unsupported or missing model_name in engine config. Supported values include: Qwen2.5, Qwen2.5-VL, Folizen, Temuvik, Vekolix (" + known + ")");
+    throw ConfigurationError("Unsupported or missing model_name in engine config. Supported values include: Qwen2.5, Qwen2.5-VL, Folizen, Temuvik, Vekolix, Viladra (" + known + ")");
 }
 
 void check_backend(int32_t st, const efm_b200_ctx* ctx, const char* what) {

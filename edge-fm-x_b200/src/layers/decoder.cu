@@ -5,7 +5,8 @@
 // input; what stands in brackets is the prologue of the kernel that follows it: three launches for a layer without a
 // feed-forward and token input, two more for a dense feed-forward, one more for the token input.  Latent attention adds
 // [query norm] + W_uq; routed experts are [norms + add] + router | [choice] + gate, up, gated unit | [weights] + down, a shared expert
-// among them.  Linear attention runs in the launch of the attention beside it, its norm and gate are a prologue of W_o.
+// among them.  Linear attention runs in the launch of the attention beside it, its norm and gate are a prologue of W_o; alone it is one
+// launch, norm and gate included.  Input convolutions and the average over depth are part of the prologues, too.
 // Many rows: tensor-core GEMMs (bf16 operands) or fp32 FMAs (32-bit mode) between row kernels.
 #include "decoder.h"
 
@@ -63,18 +64,18 @@ void launch_gemv_ext(efm_b200_ctx& c, Launcher& L, const GemvParams& p) {
     const int per = kGemvWarps / ks, need = (p.n_items + per - 1) / per;
     const int grid = EPI == Epi::Logits ? c.num_sms : std::min(c.num_sms, need);
     const bool two = p.prologue == kProAddNorm || p.prologue == kProNorm || p.prologue == kProAddTanh || p.prologue == kProMerge;
-    const size_t smem = two ? gemv_ext_smem_bytes(p.K) : gemv_smem_bytes(p.K);
+    const size_t smem = p.conv_w != nullptr ? gemv_conv_smem_bytes(p.K) : two ? gemv_ext_smem_bytes(p.K) : gemv_smem_bytes(p.K);
     constexpr bool kExperts = EPI == Epi::Router || EPI == Epi::ExpertUp || EPI == Epi::ExpertDown;
     const int level = c.decoder->gemv_level();
     auto run = [&](auto kernel) { L.launch(kernel, dim3(grid), dim3(kGemvThreads), smem, p, ks); };
     if constexpr (EPI == Epi::Router) {
         InOrder serial(L);
-        run(level == 3 ? gemv_kernel<EPI, 3> : gemv_kernel<EPI, 2>);
-    } else if constexpr (kExperts) run(level == 3 ? gemv_kernel<EPI, 3> : gemv_kernel<EPI, 2>);
-    else if constexpr (EPI == Epi::Store32Bias) run(gemv_kernel<EPI, 2>);
+        run(level == 4 ? gemv_kernel<EPI, 4> : level == 3 ? gemv_kernel<EPI, 3> : gemv_kernel<EPI, 2>);
+    } else if constexpr (kExperts) run(level == 4 ? gemv_kernel<EPI, 4> : level == 3 ? gemv_kernel<EPI, 3> : gemv_kernel<EPI, 2>);
+    else if constexpr (EPI == Epi::Store32Bias) run(level == 4 ? gemv_kernel<EPI, 4> : gemv_kernel<EPI, 2>);
     else if constexpr (EPI == Epi::TokenGate) run(gemv_kernel<EPI, 1>);
     else if constexpr (EPI == Epi::Relu2) run(gemv_kernel<EPI, 3>);
-    else run(level == 3 ? gemv_kernel<EPI, 3> : level == 2 ? gemv_kernel<EPI, 2> : gemv_kernel<EPI, 1>);
+    else run(level == 4 ? gemv_kernel<EPI, 4> : level == 3 ? gemv_kernel<EPI, 3> : level == 2 ? gemv_kernel<EPI, 2> : gemv_kernel<EPI, 1>);
 }
 
 template <Epi EPI>
@@ -130,7 +131,8 @@ WindowAttnShape attn_shape(const DecoderModel& m, const DecoderLayer& l) {
     s.H = l.d.heads; s.G = l.d.kv_heads; s.D = l.d.dim; s.Dv = l.d.vdim; s.Dp = l.Dp; s.Vp = l.Vp;
     s.window = l.d.window; s.keep = l.d.window > 0 ? l.d.keep_first : 0;
     s.bias = l.d.distance_bias; s.scale = l.d.scale; s.eps = m.d.norm_eps;
-    s.qk_norm = l.d.qk_norm != EFM_QK_NORM_NONE; s.out_scale = l.linear() ? l.d.mix_scale : 1.0f;
+    s.qk_norm = l.d.qk_norm == EFM_QK_NORM_ROW ? 2 : l.d.qk_norm != EFM_QK_NORM_NONE; s.out_scale = l.parallel() ? l.d.mix_scale : 1.0f;
+    s.shift = l.shift;
     s.q_norm = l.q_norm; s.k_norm = l.k_norm; s.temp = l.temp;
     s.rot = rot_shape(l);
     return s;
@@ -146,16 +148,29 @@ LatentShape latent_shape(const DecoderModel& m, const DecoderLayer& l) {
     s.gate = l.d.out_gate;
     return s;
 }
+// column of the gates of an attention layer in its projections
+int gate_column(const DecoderLayer& l) { return (l.d.heads + l.d.kv_heads) * l.d.dim + l.d.kv_heads * l.d.vdim; }
 LinearShape linear_shape(const DecoderModel& m, const DecoderLayer& l) {
     LinearShape s{};
     s.heads = l.d.linear_heads; s.D = l.d.linear_dim; s.Dv = l.d.linear_vdim; s.Vp = l.lin_vp;
-    const int qk = round_up(s.heads * s.D, 8), v = round_up(s.heads * s.Dv, 8);
+    const int qk = l.linear_qk(), v = l.linear_v();
     s.off_q = l.lin_in; s.off_k = l.lin_in + qk; s.off_v = l.lin_in + 2 * qk; s.off_g = l.lin_in + 2 * qk + v;
     s.ld = l.in.Np; s.powers = l.lin_powers; s.norm = l.mix_norm; s.eps = m.d.norm_eps; s.scale = l.d.linear_scale;
+    if (l.alone()) {
+        s.scale = 1.0f / std::sqrt((float)s.D);
+        s.rot = rot_shape(l);
+        if (l.channel_decay()) {
+            s.rank = l.d.decay_rank; s.off_a = s.off_g + v; s.inv_tau = 1.0f / l.d.linear_tau;
+            s.a2 = l.w2.w; s.a2_bias = l.w2.bias; s.ld_a2 = l.w2.Kp;
+        }
+    }
     return s;
 }
+int glu_kind(const DecoderLayer& l) { return !l.gated_experts() ? kGluRelu2 : l.d.expert_glu == EFM_GLU_CLAMPED ? kGluClamped : kGluSilu; }
 RouteShape route_shape(const DecoderLayer& l) {
-    return RouteShape{l.d.experts, l.d.expert_top, l.d.expert_groups, l.d.expert_groups_kept, l.d.expert_score == EFM_SCORE_SIGMOID, l.d.shared_ff > 0};
+    const int shared = l.d.shared_ff <= 0 ? kSharedNone : l.d.shared_gate == EFM_SHARED_PLAIN ? kSharedPlain : kSharedGated;
+    return RouteShape{l.d.experts, l.d.expert_top, l.d.expert_groups, l.d.expert_groups_kept, l.d.expert_score == EFM_SCORE_SIGMOID, shared,
+                      l.d.expert_scale != 0.f ? l.d.expert_scale : 1.0f};
 }
 DeltaShape delta_shape(const DecoderModel& m, const DecoderLayer& l) {
     DeltaShape s{};
@@ -187,7 +202,8 @@ void launch_attn_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, con
     p.state = c.state;
     p.out = m.d_mix;
     p.early = early ? 1 : 0;
-    if (l.linear()) {
+    if (l.d.out_gate) p.gate = m.d_in + gate_column(l);
+    if (l.parallel()) {
         p.lin.s = linear_shape(m, l);
         p.lin.pool = m.state_pool + (size_t)slot.state_slot * m.state_stride + run.state_off;
         p.lin.out = m.d_mix + l.lin_mix;
@@ -269,6 +285,17 @@ void launch_latent_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, con
     }
 }
 
+void launch_linear_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const KvSlot& slot, bool early) {
+    DecoderModel& m = *c.decoder;
+    LinearDecodeParams p{};
+    p.s = linear_shape(m, l);
+    p.pool = m.state_pool + (size_t)slot.state_slot * m.state_stride + run.state_off;
+    p.out = m.d_mix;
+    const int slices = (p.s.Dv + ln::kCols - 1) / ln::kCols;
+    L.cluster_x = slices;
+    L.launch(linear_decode_kernel, dim3(slices, p.s.heads), dim3(256), 0, p, (const float*)m.d_in, c.state, slot.n_pages * kPageTokens, early ? 1 : 0);
+}
+
 void launch_delta_decode(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const KvSlot& slot, bool early) {
     DecoderModel& m = *c.decoder;
     DeltaDecodeParams p{};
@@ -298,6 +325,13 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
         if (L.err == cudaSuccess)
             L.err = cudaMemcpyAsync(m.tap + ((size_t)layer * m.tap_rows + m.tap_row0) * m.Wp, src, (size_t)m.Wp * 4, cudaMemcpyDeviceToDevice, L.stream);
     };
+    // the product that starts layer i closes layer i - 1
+    auto end_of_layer = [&](GemvParams& p, size_t i) {
+        p.hist_out = m.d_hist + i * m.Wp;
+        if (i == 0) return;
+        p.avg = m.d_avg;
+        p.avg_w = m.layers[m.runs[i - 1].layer].dwa + i;
+    };
     for (size_t i = 0; i < m.runs.size(); ++i) {
         const DecoderRun& run = m.runs[i];
         const DecoderLayer& l = m.layers[run.layer];
@@ -305,9 +339,19 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
         // dependency wait: the mixer one layer up releases its dependents only after its own wait, so nothing of an
         // earlier step is still running.
         const bool early = i > 0;
+        float* state = m.state_pool != nullptr ? m.state_pool + (size_t)slot.state_slot * m.state_stride : nullptr;
+        auto convolve = [&](GemvParams& p, const __nv_bfloat16* w, size_t off, bool ready) {
+            if (w == nullptr) return;
+            p.conv_w = w;
+            p.conv_ring = state + off;
+            p.conv_taps = m.d.conv_taps;
+            p.conv_early = ready ? 1 : 0;
+        };
         {
             GemvParams p{};
             stream_input(c, p, pend, i == 0, l.pre1);
+            if (m.d.depth_average) end_of_layer(p, i);
+            convolve(p, l.canon1, run.conv1_off, early);
             p.out_f = m.d_in;
             if (l.in.bias != nullptr) gemv_ext<Epi::Store32Bias>(c, L, l.in, p);
             else gemv_ext<Epi::Store32>(c, L, l.in, p);
@@ -326,6 +370,8 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
             gemv_ext<Epi::Store32>(c, L, l.uq, p);
             if (m.f32) launch_latent_decode<float>(c, L, l, run, slot, early);
             else launch_latent_decode<__nv_bfloat16>(c, L, l, run, slot, early);
+        } else if (l.alone()) {
+            launch_linear_decode(c, L, l, run, slot, early);
         } else {
             launch_delta_decode(c, L, l, run, slot, early);
         }
@@ -333,7 +379,14 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
             GemvParams p{};
             p.prologue = kProPlain;
             p.xf = m.d_mix;
-            if (l.linear()) {
+            if (m.d.depth_average) {                                   // what is known of the average behind this layer
+                p.sum_in = m.d_hist;
+                p.sum_w = l.dwa;
+                p.sum_out = m.d_avg;
+                p.sum_n = (int)i + 1;
+                p.sum_k = m.Wp;
+            }
+            if (l.parallel()) {
                 p.prologue = kProMerge;
                 p.merge0 = l.lin_mix;
                 p.merge_gate = m.d_in + linear_shape(m, l).off_g;
@@ -342,13 +395,15 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
                 p.k_true = l.d.linear_heads * l.d.linear_vdim;
             }
             p.out_f = m.d_y;
-            gemv_ext<Epi::Store32>(c, L, l.out, p);
+            if (l.out.bias != nullptr) gemv_ext<Epi::Store32Bias>(c, L, l.out, p);
+            else gemv_ext<Epi::Store32>(c, L, l.out, p);
             pend.y = m.d_y;
             pend.norm = l.post1;
         }
         if (l.moe()) {
             GemvParams r{};
             stream_input(c, r, pend, false, l.pre2);
+            convolve(r, l.canon2, run.conv2_off, true);
             r.x_out = m.d_h;
             r.out_f = m.d_route;
             r.route = route_shape(l);
@@ -361,12 +416,14 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
             p.W = l.expert_in.w;
             p.xf = m.d_h;
             p.K = l.expert_in.Kp;
-            p.n_items = l.d.expert_top * l.d.expert_ff + l.d.shared_ff;
-            p.glu = l.d.expert_glu == EFM_GLU_CLAMPED ? kGluClamped : kGluSilu;
+            const int pair = l.gated_experts() ? 1 : 2;                // channels of an item
+            p.ff = (l.d.expert_ff + pair - 1) / pair;
+            p.shared_ff = (l.d.shared_ff + pair - 1) / pair;
+            p.n_items = l.d.expert_top * p.ff + p.shared_ff;
+            p.glu = glu_kind(l);
             p.weight_input = l.d.expert_weight_input;
             p.limit = l.d.expert_limit;
             p.shared_limit = l.d.shared_limit;
-            p.shared_ff = l.d.shared_ff;
             p.shared_ffp = l.sfp;
             p.W2 = l.shared_in.w;
             p.N = 2 * p.n_items;
@@ -374,9 +431,8 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
             p.route = route_shape(l);
             p.route_id = m.d_route_id;
             p.route_w = m.d_route_w;
-            p.ff = l.d.expert_ff;
             p.ffp = l.ffp;
-            p.expert_rows = 2 * l.ffp;
+            p.expert_rows = l.up_rows(l.ffp);
             p.out_f = m.d_act;
             launch_gemv_ext<Epi::ExpertUp>(c, L, p);
             GemvParams q = p;
@@ -394,6 +450,7 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
         } else if (l.d.ff > 0) {
             GemvParams p{};
             stream_input(c, p, pend, false, l.pre2);
+            convolve(p, l.canon2, run.conv2_off, true);
             p.out_f = m.d_ff;
             const bool poly = l.d.ff_act == EFM_ACT_POLYNORM;
             if (poly) gemv_ext<Epi::Store32>(c, L, l.up, p);
@@ -447,6 +504,7 @@ void decoder_decode_step(efm_b200_ctx& c, KvSlot& slot, Launcher& L, bool sample
     {
         GemvParams p{};
         stream_input(c, p, pend, false, m.final_norm);
+        if (m.d.depth_average) end_of_layer(p, m.runs.size());
         p.logits = c.logits;
         p.logit_scale = m.d.logit_scale;
         p.logit_softcap = m.d.logit_softcap;
@@ -514,20 +572,20 @@ void launch_delta_scan(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, cons
 }
 
 // The maps of attention and latent attention differ; what is launched is the same.
-template <int DP, int VP, int RP, bool KEEP>
+template <int DP, int VP, int RP, bool KEEP, bool SIG>
 void launch_attention_tc_v(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const WindowAttnShape& s, const WindowTcMaps& maps, const RowPlan& plan,
                            const RowTile* list, int n) {
     const int blocks = n * s.H * ((s.Vp + VP - 1) / VP), first_wave = blocks <= 2 * c.num_sms ? std::min(blocks, c.num_sms) : blocks;
-    L.launch(window_attention_tc_kernel<DP, VP, RP, KEEP>, dim3(blocks), dim3(wt::kThreads), wt::Cfg<DP, VP, RP>::SMEM, maps, static_cast<__nv_bfloat16*>(c.decoder->mix),
+    L.launch(window_attention_tc_kernel<DP, VP, RP, KEEP, SIG>, dim3(blocks), dim3(wt::kThreads), wt::Cfg<DP, VP, RP>::SMEM, maps, static_cast<__nv_bfloat16*>(c.decoder->mix),
              l.mix_wp, s, plan, list, n, first_wave, RP > 0 ? 1 : 0, &c.state->error);
 }
-template <int RP, bool KEEP = false>
+template <int RP, bool KEEP = false, bool SIG = false>
 void launch_attention_tc_r(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const WindowAttnShape& s, const WindowTcMaps& maps, const RowPlan& plan,
                            const RowTile* list, int n) {
-    if (l.Dp <= 64 && l.Vp <= 64) launch_attention_tc_v<64, 64, RP, KEEP>(c, L, l, s, maps, plan, list, n);
-    else if (l.Dp <= 64) launch_attention_tc_v<64, 128, RP, KEEP>(c, L, l, s, maps, plan, list, n);
-    else if (l.Vp <= 64) launch_attention_tc_v<128, 64, RP, KEEP>(c, L, l, s, maps, plan, list, n);
-    else launch_attention_tc_v<128, 128, RP, KEEP>(c, L, l, s, maps, plan, list, n);
+    if (l.Dp <= 64 && l.Vp <= 64) launch_attention_tc_v<64, 64, RP, KEEP, SIG>(c, L, l, s, maps, plan, list, n);
+    else if (l.Dp <= 64) launch_attention_tc_v<64, 128, RP, KEEP, SIG>(c, L, l, s, maps, plan, list, n);
+    else if (l.Vp <= 64) launch_attention_tc_v<128, 64, RP, KEEP, SIG>(c, L, l, s, maps, plan, list, n);
+    else launch_attention_tc_v<128, 128, RP, KEEP, SIG>(c, L, l, s, maps, plan, list, n);
 }
 // [rows][heads][channels] with strides in elements
 bool head_map(CUtensorMap* map, const void* base, int channels, int heads, int rows, int head_stride, int row_stride, int box_rows) {
@@ -548,7 +606,8 @@ void launch_attention_tc(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, co
     }
     maps.qr = maps.q;
     maps.kr = maps.k;
-    if (s.keep > 0) launch_attention_tc_r<0, true>(c, L, l, s, maps, plan, list, n);
+    if (s.shift != nullptr) launch_attention_tc_r<0, false, true>(c, L, l, s, maps, plan, list, n);
+    else if (s.keep > 0) launch_attention_tc_r<0, true>(c, L, l, s, maps, plan, list, n);
     else launch_attention_tc_r<0>(c, L, l, s, maps, plan, list, n);
 }
 // Long entries of a latent layer: visible cache rows into the workspace, keys and values of all heads by one product,
@@ -602,29 +661,73 @@ void linear_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const Deco
     bool tensor_cores = false;
     if constexpr (std::is_same<TA, __nv_bfloat16>::value) tensor_cores = s.D <= 128 && plan.rows >= kLinearChunk;      // short passes: CUDA cores
     const int chunks = max_chunks(plan, tensor_cores ? kLinearChunkTc : kLinearChunk);
+    const int ld_sums = l.w2.Np;
     auto chain = [&](auto kernel) {
         L.launch(kernel, dim3((unsigned)((s.heads * s.head_floats() + 1023) / 1024), plan.n_entries), dim3(256), 0, m.lin_ws, m.state_pool, m.state_stride, run.state_off,
-                 s, plan);
+                 s, plan, (const float*)m.decay, ld_sums);
     };
     auto output = [&] {
+        if (l.alone()) {
+            L.launch(linear_head_output_rows_kernel<TA>, dim3((plan.rows * s.heads + 7) / 8), dim3(256), 0, (const float*)m.o, ld_o, proj, static_cast<TA*>(m.mix), l.mix_wp,
+                     plan.rows, s);
+            return;
+        }
         L.launch(linear_output_rows_kernel<TA>, dim3(plan.rows), dim3(256), 0, (const float*)m.o, ld_o, proj, static_cast<TA*>(m.mix) + l.lin_mix, l.mix_wp,
                  l.mix_wp - l.lin_mix, s);
     };
+    if (s.rank > 0) {                                                  // W_a2 W_a1 x + b, then the decays it stands for
+        if (m.f32) {
+            L.launch(gemm_f32_kernel, dim3((l.w2.Np + 63) / 64, (plan.rows + 63) / 64), dim3(256), 0, reinterpret_cast<const float*>(proj) + s.off_a, s.ld,
+                     (const __nv_bfloat16*)l.w2.w, l.w2.Kp, m.decay, l.w2.Np, plan.rows, l.w2.Np, l.w2.Kp, (const __nv_bfloat16*)l.w2.bias, RowGroups{});
+        } else {
+            GemmParams g{reinterpret_cast<const __nv_bfloat16*>(proj) + s.off_a, l.w2.w, l.w2.bias, nullptr, m.decay, plan.rows, l.w2.Np, l.w2.Kp};
+            g.lda = s.ld;
+            launch_gemm_epi(L, GemmEpi::F32, g, &c.state->error);
+        }
+        if (tensor_cores)
+            L.launch(linear_decay_sums_kernel<kLinearChunkTc>, dim3((ld_sums + 127) / 128, chunks), dim3(128), 0, m.decay, ld_sums, s.inv_tau, plan);
+        else
+            L.launch(linear_decay_rows_kernel, dim3((ld_sums + 255) / 256, plan.rows), dim3(256), 0, m.decay, ld_sums, s.inv_tau);
+    }
     if constexpr (std::is_same<TA, __nv_bfloat16>::value) {
         if (tensor_cores) {
             auto products = [&](auto vp) {
                 constexpr int VP = decltype(vp)::value;
-                const dim3 grid(chunks, s.heads, (s.Dv + VP - 1) / VP);
-                L.launch(linear_chunk_tc_kernel<VP>, grid, dim3(lt::kThreads), lt::Cfg<VP>::CHUNK_SMEM, proj, m.lin_ws, s, plan, &c.state->error);
-                chain(linear_chain_rows_kernel<kLinearChunkTc>);
-                L.launch(linear_attend_tc_kernel<VP>, grid, dim3(lt::kThreads), lt::Cfg<VP>::ATTEND_SMEM, proj, (const float*)m.lin_ws, m.o, ld_o, s, plan,
-                         &c.state->error);
+                using Cf = lt::Cfg<VP>;
+                const dim3 grid(chunks, s.heads, (s.Dv + VP - 1) / VP), block(lt::kThreads);
+                const float *sums = m.decay, *ws = m.lin_ws;
+                const bool whole = l.alone() && s.Dv <= VP;             // a block has all of a head's channels: norm and gate included
+                __nv_bfloat16* out = static_cast<__nv_bfloat16*>(m.mix);
+                if (s.rank > 0) {
+                    L.launch(linear_chunk_tc_kernel<VP, true>, grid, block, Cf::CHUNK_SMEM, proj, m.lin_ws, s, plan, &c.state->error, sums, ld_sums);
+                    chain(linear_chain_rows_kernel<kLinearChunkTc, true>);
+                    L.launch(whole ? linear_attend_ch_tc_kernel<VP, true> : linear_attend_ch_tc_kernel<VP, false>, grid, block, Cf::ATTEND_CH_SMEM, proj, ws, sums, ld_sums,
+                             m.o, ld_o, out, l.mix_wp, s, plan, &c.state->error);
+                } else {
+                    L.launch(linear_chunk_tc_kernel<VP>, grid, block, Cf::CHUNK_SMEM, proj, m.lin_ws, s, plan, &c.state->error, sums, 0);
+                    chain(linear_chain_rows_kernel<kLinearChunkTc>);
+                    L.launch(whole ? linear_attend_tc_kernel<VP, true> : linear_attend_tc_kernel<VP>, grid, block, Cf::ATTEND_SMEM, proj, ws, m.o, ld_o, s, plan,
+                             &c.state->error, out, l.mix_wp);
+                }
+                if (!whole) output();
             };
             if (s.Dv <= 64) products(std::integral_constant<int, 64>{});
             else products(std::integral_constant<int, 128>{});
-            output();
             return;
         }
+    }
+    if (s.rank > 0) {                                                  // token by token
+        auto scan = [&](auto nc) {
+            constexpr int NC = decltype(nc)::value;
+            L.launch(linear_scan_rows_kernel<TA, NC>, dim3(s.heads * ((s.Dv + lc::kCols - 1) / lc::kCols), plan.n_entries), dim3(lc::kThreads), lc::smem_bytes(NC * 32), proj,
+                     (const float*)m.decay, ld_sums, m.o, ld_o, m.state_pool, m.state_stride, run.state_off, s, plan);
+        };
+        if (s.D <= 32) scan(std::integral_constant<int, 1>{});
+        else if (s.D <= 64) scan(std::integral_constant<int, 2>{});
+        else if (s.D <= 128) scan(std::integral_constant<int, 4>{});
+        else scan(std::integral_constant<int, 8>{});
+        output();
+        return;
     }
     auto chunk = [&](auto rm, auto rn) {
         constexpr int RM = decltype(rm)::value, RN = decltype(rn)::value;
@@ -641,17 +744,33 @@ void linear_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const Deco
     if (s.D <= 64) { if (s.Dv <= 64) chunk(k4, k4); else chunk(k4, k8); }
     else if (s.Dv <= 64) chunk(k8, k4);
     else chunk(k8, k8);
-    chain(linear_chain_rows_kernel<kLinearChunk>);
+    chain(linear_chain_rows_kernel<kLinearChunk, false>);
     if (s.Dv <= 64) attend(k4); else attend(k8);
     output();
+}
+
+// A layer of linear attention alone.
+template <typename TA>
+void linear_mixer_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const void* x, const RowPlan& plan) {
+    DecoderModel& m = *c.decoder;
+    const LinearShape s = linear_shape(m, l);
+    if (s.rot.kind == kRotNone) {
+        linear_act(c, L, l.in, x, m.proj_a, plan.rows);
+    } else {                                                           // turned in fp32, rounded once
+        float* proj = std::is_same<TA, float>::value ? static_cast<float*>(m.proj_a) : m.proj_f;
+        linear_f32(c, L, l.in, x, proj, plan.rows);
+        L.launch(linear_rotate_rows_kernel<TA>, dim3(plan.rows), dim3(256), 0, (const float*)proj, static_cast<TA*>(m.proj_a), s, plan);
+    }
+    linear_rows<TA>(c, L, l, run, plan);
 }
 
 // TA: activation and cache type of the pass
 template <typename TA>
 void attention_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const DecoderRun& run, const void* x, const RowPlan& plan, const RowTiles& tiles) {
     DecoderModel& m = *c.decoder;
-    const WindowAttnShape s = attn_shape(m, l);
-    if (l.linear()) {
+    WindowAttnShape s = attn_shape(m, l);
+    if (l.d.out_gate) { s.gate = static_cast<const TA*>(m.proj_a) + gate_column(l); s.gate_ld = l.in.Np; s.gate_heads = 1; }
+    if (l.parallel()) {
         const LinearShape z = linear_shape(m, l);
         if constexpr (std::is_same<TA, float>::value) {
             linear_f32(c, L, l.in, x, static_cast<float*>(m.proj_a), plan.rows);
@@ -740,8 +859,8 @@ SumOf<TA> expert_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const
             L.launch(gemm_f32_kernel, dim3((n + 63) / 64, (max_rows + 63) / 64), dim3(256), 0, a, w.Kp, (const __nv_bfloat16*)w.w, w.Kp, out, n, max_rows, n, w.Kp,
                      (const __nv_bfloat16*)nullptr, RowGroups{m.ex.tile, m.ex.n_tiles, n});
         };
-        product(l.expert_in, 2 * l.ffp, static_cast<const float*>(m.ex_in), m.ex_gu);
-        const int glu = l.d.expert_glu == EFM_GLU_CLAMPED ? kGluClamped : kGluSilu;
+        product(l.expert_in, l.up_rows(l.ffp), static_cast<const float*>(m.ex_in), m.ex_gu);
+        const int glu = glu_kind(l);
         L.launch(glu_rows_kernel, dim3(max_rows / kExpertTile), dim3(256), 0, (const float*)m.ex_gu, static_cast<float*>(m.ex_act), max_rows, l.ffp,
                  (const int32_t*)m.ex.n_tiles, glu, l.d.expert_limit);
         product(l.expert_out, m.Wp, static_cast<const float*>(m.ex_act), static_cast<float*>(m.ex_y));
@@ -761,8 +880,8 @@ SumOf<TA> expert_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const
             g.limit = l.d.expert_limit;
             launch_gemm_epi(L, epi, g, &c.state->error);
         };
-        const GemmEpi glu = l.d.expert_glu == EFM_GLU_CLAMPED ? GemmEpi::ClampGlu : GemmEpi::SwiGlu;
-        product(l.expert_in, 2 * l.ffp, glu, m.ex_in, m.ex_act);
+        const GemmEpi glu = !l.gated_experts() ? GemmEpi::Bf16Relu2 : l.d.expert_glu == EFM_GLU_CLAMPED ? GemmEpi::ClampGlu : GemmEpi::SwiGlu;
+        product(l.expert_in, l.up_rows(l.ffp), glu, m.ex_in, m.ex_act);
         product(l.expert_out, m.Wp, GemmEpi::Bf16Bias, m.ex_act, m.ex_y);
         if (l.d.shared_ff > 0) {
             GemmParams g{static_cast<const __nv_bfloat16*>(h), l.shared_in.w, nullptr, static_cast<__nv_bfloat16*>(m.sh_act), nullptr, T, l.shared_in.Np, l.shared_in.Kp};
@@ -817,7 +936,10 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
     TA* xa = static_cast<TA*>(m.xa);                            // null: 32-bit mode without input norms reads the stream itself
     const void* xin = xa != nullptr ? (const void*)xa : c.resid;
     // the stream takes a sublayer's normed output; xa becomes the next sublayer's input
-    auto add_norm = [&](const float* y, const __nv_bfloat16* w, const DecNorm& norm, const SumOf<TA>& sum = SumOf<TA>{}) {
+    // with an average over depth the embedding stays in its row of the history, behind a layer's last sublayer (avg) its result goes there
+    const float* stream = c.resid;
+    const size_t hist_rows = (size_t)m.d.max_step_tokens * m.Wp;
+    auto add_norm = [&](const float* y, const __nv_bfloat16* w, const DecNorm& norm, const SumOf<TA>& sum = SumOf<TA>{}, const DepthAverage* avg = nullptr) {
         const bool experts = sum.place != nullptr;
         const __nv_bfloat16* pre = norm.w;
         if (m.tanh_norms()) {
@@ -825,12 +947,31 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
                      m.d.residual_mult, xa, norm.w, norm.b, norm.alpha, m.Wp, sum);
             return;
         }
+        if (avg != nullptr) {
+            L.launch(experts ? add_norm_rows_kernel<TA, false, true, true> : add_norm_rows_kernel<TA, false, false, true>, dim3(T), dim3(256), 0, c.resid, stream, y, w,
+                     (TA*)nullptr, (const __nv_bfloat16*)nullptr, m.W, m.Wp, m.d.norm_eps, sum, *avg);
+            stream = c.resid;
+            return;
+        }
         L.launch(pre != nullptr ? (experts ? add_norm_rows_kernel<TA, true, true> : add_norm_rows_kernel<TA, true, false>)
                                 : (experts ? add_norm_rows_kernel<TA, false, true> : add_norm_rows_kernel<TA, false, false>),
-                 dim3(T), dim3(256), 0, c.resid, y, w, xa, pre, m.W, m.Wp, m.d.norm_eps, sum);
+                 dim3(T), dim3(256), 0, c.resid, stream, y, w, m.d.conv_taps > 0 ? (TA*)nullptr : xa, pre, m.W, m.Wp, m.d.norm_eps, sum, DepthAverage{});
+        stream = c.resid;
+    };
+    auto convolve = [&](const __nv_bfloat16* w, size_t off) {
+        if (w == nullptr) return;
+        auto run = [&](auto kernel) {
+            L.launch(kernel, dim3((m.Wp / 4 + 127) / 128, max_chunks(plan, kConvRows)), dim3(128), 0, stream, w, xa, m.Wp, m.state_pool, m.state_stride, off, m.d.conv_taps, plan);
+        };
+        switch (m.d.conv_taps) {
+            case 2: run(input_conv_rows_kernel<TA, 2>); break;
+            case 3: run(input_conv_rows_kernel<TA, 3>); break;
+            case 4: run(input_conv_rows_kernel<TA, 4>); break;
+            default: run(input_conv_rows_kernel<TA, 0>); break;
+        }
     };
     // a sublayer's last product and what follows it; elementwise norms are part of the product
-    auto sublayer_out = [&](const DecLinear& w, const void* a, const __nv_bfloat16* post, const DecNorm& norm) {
+    auto sublayer_out = [&](const DecLinear& w, const void* a, const __nv_bfloat16* post, const DecNorm& norm, const DepthAverage* avg = nullptr) {
         if (m.tanh_norms() && !m.f32) {
             GemmParams g{static_cast<const __nv_bfloat16*>(a), w.w, nullptr, norm.w != nullptr ? static_cast<__nv_bfloat16*>(m.xa) : nullptr, c.resid, T, w.Np, w.Kp};
             g.mult = m.d.residual_mult;
@@ -839,20 +980,26 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
             return;
         }
         linear_f32(c, L, w, a, m.y, T);
-        add_norm(m.y, post, norm);
+        add_norm(m.y, post, norm, SumOf<TA>{}, avg);
     };
-    launch_embed_rows(L, ids, c.embed, nullptr, c.resid, T, c.d.vocab, m.Wp, -1, 0, m.d.embed_scale);
-    if (xa != nullptr) add_norm(nullptr, nullptr, m.layers[m.runs[0].layer].pre1);
+    float* first = m.d.depth_average ? m.hist : c.resid;
+    launch_embed_rows(L, ids, c.embed, nullptr, first, T, c.d.vocab, m.Wp, -1, 0, m.d.embed_scale);
+    stream = first;
+    if (xa != nullptr && m.d.conv_taps == 0) add_norm(nullptr, nullptr, m.layers[m.runs[0].layer].pre1);
     for (size_t i = 0; i < m.runs.size(); ++i) {
         const DecoderRun& run = m.runs[i];
         const DecoderLayer& l = m.layers[run.layer];
         const DecNorm next = i + 1 < m.runs.size() ? m.layers[m.runs[i + 1].layer].pre1 : DecNorm{};
+        const DepthAverage depth{m.hist, hist_rows, l.dwa, (int)i + 1}, *avg = m.d.depth_average ? &depth : nullptr;
+        convolve(l.canon1, run.conv1_off);
         if (l.attention()) attention_rows<TA>(c, L, l, run, xin, plan, tiles);
         else if (l.d.mixer == EFM_MIXER_LATENT_ATTENTION) latent_rows<TA>(c, L, l, run, xin, plan, tiles);
+        else if (l.alone()) linear_mixer_rows<TA>(c, L, l, run, xin, plan);
         else delta_rows<TA>(c, L, l, run, xin, plan);
-        sublayer_out(l.out, m.mix, l.post1, l.mlp() ? l.pre2 : next);
+        sublayer_out(l.out, m.mix, l.post1, l.mlp() ? l.pre2 : next, l.mlp() ? nullptr : avg);
+        if (l.mlp()) convolve(l.canon2, run.conv2_off);
         if (l.moe()) {
-            add_norm(nullptr, l.post2, next, expert_rows<TA>(c, L, l, xin, T));
+            add_norm(nullptr, l.post2, next, expert_rows<TA>(c, L, l, xin, T), avg);
         } else if (l.d.ff > 0) {
             const bool poly = l.d.ff_act == EFM_ACT_POLYNORM;
             if (poly) {
@@ -867,7 +1014,7 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
                 GemmParams g{static_cast<const __nv_bfloat16*>(xin), l.up.w, nullptr, static_cast<__nv_bfloat16*>(m.ff), nullptr, T, l.up.Np, l.up.Kp};
                 launch_gemm_epi(L, GemmEpi::Bf16Relu2, g, &c.state->error);
             }
-            sublayer_out(l.down, poly ? m.ff2 : m.ff, l.post2, next);
+            sublayer_out(l.down, poly ? m.ff2 : m.ff, l.post2, next, avg);
         }
         if (m.d.side_dim > 0) {
             linear_f32(c, L, l.gate, xin, m.side_f, T);
@@ -877,7 +1024,7 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
             add_norm(m.y, l.side_norm, DecNorm{});
         }
         if (m.tap != nullptr && m.tap_row0 + T <= m.tap_rows && L.err == cudaSuccess)
-            L.err = cudaMemcpyAsync(m.tap + ((size_t)i * m.tap_rows + m.tap_row0) * m.Wp, c.resid, (size_t)T * m.Wp * 4, cudaMemcpyDeviceToDevice, L.stream);
+            L.err = cudaMemcpyAsync(m.tap + ((size_t)i * m.tap_rows + m.tap_row0) * m.Wp, stream, (size_t)T * m.Wp * 4, cudaMemcpyDeviceToDevice, L.stream);
     }
 }
 
@@ -1046,6 +1193,8 @@ cudaError_t configure_decoder(DecoderModel& m) {
               gemv_kernel<Epi::Store32Bias, 2>, gemv_kernel<Epi::Router, 2>, gemv_kernel<Epi::ExpertUp, 2>, gemv_kernel<Epi::ExpertDown, 2>);
     gemv_attr(gemv_kernel<Epi::Store32, 3>, gemv_kernel<Epi::Logits, 3>, gemv_kernel<Epi::Relu2, 3>, gemv_kernel<Epi::Router, 3>, gemv_kernel<Epi::ExpertUp, 3>,
               gemv_kernel<Epi::ExpertDown, 3>);
+    gemv_attr(gemv_kernel<Epi::Store32, 4>, gemv_kernel<Epi::Store32Bias, 4>, gemv_kernel<Epi::Logits, 4>, gemv_kernel<Epi::Router, 4>, gemv_kernel<Epi::ExpertUp, 4>,
+              gemv_kernel<Epi::ExpertDown, 4>);
     auto linear_attr = [&](auto type) {
         using T = decltype(type);
         auto chunk = [&](auto kernel, int rm, int rn) { if (e == cudaSuccess) e = smem_attr(kernel, ln::chunk_smem_bytes(rm, rn)); };
@@ -1056,10 +1205,18 @@ cudaError_t configure_decoder(DecoderModel& m) {
     };
     linear_attr(float());
     linear_attr(__nv_bfloat16());
-    if (e == cudaSuccess) e = smem_attr(linear_chunk_tc_kernel<64>, lt::Cfg<64>::CHUNK_SMEM);
-    if (e == cudaSuccess) e = smem_attr(linear_chunk_tc_kernel<128>, lt::Cfg<128>::CHUNK_SMEM);
-    if (e == cudaSuccess) e = smem_attr(linear_attend_tc_kernel<64>, lt::Cfg<64>::ATTEND_SMEM);
-    if (e == cudaSuccess) e = smem_attr(linear_attend_tc_kernel<128>, lt::Cfg<128>::ATTEND_SMEM);
+    auto linear_tc_attr = [&](auto vp) {
+        constexpr int VP = decltype(vp)::value;
+        auto set = [&](auto kernel, size_t bytes) { if (e == cudaSuccess) e = smem_attr(kernel, bytes); };
+        set(linear_chunk_tc_kernel<VP>, lt::Cfg<VP>::CHUNK_SMEM);
+        set(linear_chunk_tc_kernel<VP, true>, lt::Cfg<VP>::CHUNK_SMEM);
+        set(linear_attend_tc_kernel<VP>, lt::Cfg<VP>::ATTEND_SMEM);
+        set(linear_attend_tc_kernel<VP, true>, lt::Cfg<VP>::ATTEND_SMEM);
+        set(linear_attend_ch_tc_kernel<VP, false>, lt::Cfg<VP>::ATTEND_CH_SMEM);
+        set(linear_attend_ch_tc_kernel<VP, true>, lt::Cfg<VP>::ATTEND_CH_SMEM);
+    };
+    linear_tc_attr(std::integral_constant<int, 64>{});
+    linear_tc_attr(std::integral_constant<int, 128>{});
     const size_t rows = wa::rows_smem_bytes(256, 256);
     if (e == cudaSuccess) e = smem_attr(window_attention_rows_kernel<float, float, float>, rows);
     if (e == cudaSuccess) e = smem_attr(window_attention_rows_kernel<__nv_bfloat16, __nv_bfloat16, __nv_bfloat16>, rows);
@@ -1071,6 +1228,7 @@ cudaError_t configure_decoder(DecoderModel& m) {
         constexpr int DP = decltype(dp)::value, VP = decltype(vp)::value;
         if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<DP, VP, 0, false>, wt::Cfg<DP, VP, 0>::SMEM);
         if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<DP, VP, 0, true>, wt::Cfg<DP, VP, 0>::SMEM);
+        if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<DP, VP, 0, false, true>, wt::Cfg<DP, VP, 0>::SMEM);
         if (e == cudaSuccess) e = smem_attr(window_attention_tc_kernel<DP, VP, 64, false>, wt::Cfg<DP, VP, 64>::SMEM);
     };
     const std::integral_constant<int, 64> k64{};

@@ -1,7 +1,8 @@
-// Layered decoder: a list of layers, each with its own mixer (attention | latent attention | generalised delta rule | attention and
-// linear attention side by side) and an optional feed-forward (dense | routed experts), sublayer outputs (and, sandwich layout,
-// inputs; or the inputs alone, elementwise) normalised, optional per-layer token input; a span of layers may run several times.  Weights, buffers and launch sequences (definitions in
-// decoder.cu); the C ABI side is backends/b200/decoder_b200.cu.
+// Layered decoder: a list of layers, each with its own mixer (attention | latent attention | generalised delta rule | linear attention |
+// attention and linear attention side by side) and an optional feed-forward (dense | routed experts), sublayer outputs (and, sandwich
+// layout, inputs; or the inputs alone, elementwise) normalised, optional per-layer token input, short convolutions of the sublayers'
+// inputs, average over depth; a span of layers may run several times.  Weights, buffers and launch sequences (definitions in decoder.cu);
+// the C ABI side is backends/b200/decoder_b200.cu.
 #pragma once
 #include <algorithm>
 #include <set>
@@ -32,9 +33,10 @@ struct DecoderLayer {
     int Dp = 0, Vp = 0;                   // attention: padded channels of a cache row; latent: padded head channels
     int mix_w = 0, mix_wp = 0;            // mixer output width (heads * value channels; parallel: both halves), padded
     DecLinear in;                         // attention: q | k | v; latent: dq | c | r | g, each padded to 8; delta: r | k | v | g | a | w1;
-                                          // parallel: attention's, then q | k | v | g of linear attention, each padded to 8
+                                          // parallel: attention's, then q | k | v | g of linear attention, each padded to 8;
+                                          // linear: q | k | v | g (| a1), each padded to 8; attention with a gate: q | k | v | g
     DecLinear out;                        // W_o (parallel: the two side by side)
-    DecLinear w2;                         // delta: decay projection
+    DecLinear w2;                         // delta, linear with projected decays: second factor of the decay projection
     DecLinear up, down, gate, proj;       // dense feed-forward; token side
     DecNorm pre1, pre2;
     __nv_bfloat16 *post1 = nullptr, *post2 = nullptr, *side_norm = nullptr, *act = nullptr;
@@ -44,18 +46,27 @@ struct DecoderLayer {
     // latent attention
     int Qp = 0, Lc = 0, Rc = 0;           // query latent, cached latent, rotated part: padded to 8
     DecLinear uq, ukv;                    // [heads][Dp + Rc] rows; [heads][Dp] key rows, then [heads][Vp] value rows
-    __nv_bfloat16* sink = nullptr;
+    __nv_bfloat16 *sink = nullptr, *shift = nullptr;      // shift: attention with sigmoid weights
     int la_heads = 1, la_cluster = 1, la_tile = 64;       // absorbed form: heads per block, widest cluster, keys per tile
-    // linear attention beside attention
+    __nv_bfloat16 *canon1 = nullptr, *canon2 = nullptr;   // input convolutions of mixer and feed-forward, [taps][Wp]
+    __nv_bfloat16* dwa = nullptr;         // average over depth, [layer + 2]
+    // linear attention, alone or beside attention
     int lin_in = 0, lin_mix = 0;          // its first column in the projections and in the mixer output
     int lin_vp = 0;                       // value channels padded to 4 (state rows)
     float* lin_powers = nullptr;          // [linear_heads][kLinearPowers + 1]
-    bool linear() const { return d.mixer == EFM_MIXER_PARALLEL; }
+    bool parallel() const { return d.mixer == EFM_MIXER_PARALLEL; }
+    bool alone() const { return d.mixer == EFM_MIXER_LINEAR; }
+    bool linear() const { return parallel() || alone(); }
+    bool channel_decay() const { return alone() && d.linear_tau > 0.f; }
+    int linear_qk() const { return round_up(d.linear_heads * d.linear_dim, 8); }      // columns of q (and k), of v (and g)
+    int linear_v() const { return round_up(d.linear_heads * d.linear_vdim, 8); }
     bool attention() const { return d.mixer == EFM_MIXER_ATTENTION || d.mixer == EFM_MIXER_PARALLEL; }
     // routed experts
-    DecLinear router, expert_in, expert_out;   // [experts], a shared expert's gate behind; [experts][2 * ffp]; [experts][width][ffp]
-    DecLinear shared_in, shared_out;      // [2 * sfp]; [width][sfp]
+    DecLinear router, expert_in, expert_out;   // [experts], a shared expert's gate behind; [experts][up_rows()]; [experts][width][ffp]
+    DecLinear shared_in, shared_out;      // the same of a shared expert
     int ffp = 0, sfp = 0;
+    bool gated_experts() const { return d.expert_glu != EFM_GLU_NONE_RELU2; }
+    int up_rows(int ffp_) const { return gated_experts() ? 2 * ffp_ : ffp_; }
     bool moe() const { return d.experts > 0; }
     bool mlp() const { return d.experts > 0 || d.ff > 0; }
 };
@@ -65,6 +76,7 @@ struct DecoderRun {
     int layer = 0;
     void *k_pool = nullptr, *v_pool = nullptr;       // attention: [pages * 64][kv_heads][Dp / Vp]; latent: [pages * 64][Lc + Rc] (k_pool); bf16 or fp32
     size_t state_off = 0;                 // recurrent mixers: first float of this run inside a state slot
+    size_t conv1_off = 0, conv2_off = 0;  // input convolutions: the last inputs, [taps][Wp] by position modulo taps
 };
 
 struct DecoderModel {
@@ -73,8 +85,9 @@ struct DecoderModel {
     int W = 0, Wp = 0;                    // width, padded to 8
     int side_p = 0;                       // token-side width padded to 8
     bool tanh_norms() const { return d.norm_layout == EFM_NORM_INPUT; }
-    // level of the decode GEMV (gemv.cuh)
-    int gemv_level() const { return tanh_norms() ? 3 : d.norm_layout == EFM_NORM_SANDWICH || d.embed_scale != 1.0f ? 2 : 1; }
+    // something that only level 4 of the decode GEMV (gemv.cuh) has
+    bool extended = false;
+    int gemv_level() const { return extended ? 4 : tanh_norms() ? 3 : d.norm_layout == EFM_NORM_SANDWICH || d.embed_scale != 1.0f ? 2 : 1; }
     std::vector<DecoderLayer> layers;
     std::vector<DecoderRun> runs;         // in order
     __nv_bfloat16* side_embed = nullptr;
@@ -94,6 +107,8 @@ struct DecoderModel {
     __nv_bfloat16 *ws_c = nullptr, *ws_kv = nullptr;
     int ws_pages = 0, ws_window = 0;      // capacity (0: no layer uses it); largest window of the layers that use it (0: no window)
     float* lin_ws = nullptr;              // linear attention: states of a pass's chunks
+    float* hist = nullptr;                // average over depth: the embedding and every layer's result, [layers + 1][rows][Wp]
+    float *d_hist = nullptr, *d_avg = nullptr;            // the same of one row; the sum behind the current layer without its own result
     // routed experts: rows sorted by expert
     void *ex_in = nullptr, *ex_act = nullptr, *ex_y = nullptr;
     void *sh_act = nullptr, *sh_y = nullptr;              // shared expert

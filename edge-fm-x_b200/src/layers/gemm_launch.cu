@@ -77,7 +77,7 @@ static void launch_gemm(Launcher& L, const GemmParams& p, int* error_word = null
     const dim3 block(tc::kThreads);
     const bool pdl = L.pdl;
     L.pdl = false;     // prefill kernels do not use the dependent-launch protocol
-    if constexpr (EPI == GemmEpi::Bf16Bias || gemm_is_glu(EPI)) {
+    if constexpr (EPI == GemmEpi::Bf16Bias || EPI == GemmEpi::Bf16Relu2 || gemm_is_glu(EPI)) {
         if (p.group_tile != nullptr) {
             static bool attr_group = false;
             if (!attr_group) {

@@ -2,6 +2,7 @@
 // gathered final norms, the cap of the logits, and the all-32-bit matrix product.  T = bf16 (tensor-core operands) or fp32.
 #pragma once
 #include "common.cuh"
+#include "conv_limits.h"
 #include "gemv.cuh"
 #include "window_attention.cuh"
 
@@ -41,12 +42,21 @@ struct SumOf {
     const float* shared_weight;       // ... and its weight, [rows]
 };
 
-// x += y / sqrt(mean(y^2) + eps) * w (w null: x unchanged); out (null: none) = x as T, or (PRE) x / sqrt(mean(x^2) + eps) * pre,
-// the next sublayer's input.  One block per row; the first 1024 * KEEP channels stay in registers.
-template <typename T, bool PRE, bool SUM>
-__global__ void __launch_bounds__(256) add_norm_rows_kernel(float* __restrict__ x, const float* __restrict__ y, const __nv_bfloat16* __restrict__ w,
+// Average over depth behind a layer: its result x goes to hist[n], the stream becomes sum_{j < n} w[j] hist[j] + w[n] x.
+struct DepthAverage {
+    float* hist;                      // [n + 1][stride], this pass's rows
+    size_t stride;
+    const __nv_bfloat16* w;
+    int n;
+};
+
+// x = x_in + y / sqrt(mean(y^2) + eps) * w (w null: x unchanged); out (null: none) = x as T, or (PRE) x / sqrt(mean(x^2) + eps) * pre,
+// the next sublayer's input.  AVG: the average over depth behind it (out: none).  One block per row; the first 1024 * KEEP channels
+// stay in registers.
+template <typename T, bool PRE, bool SUM, bool AVG = false>
+__global__ void __launch_bounds__(256) add_norm_rows_kernel(float* x, const float* x_in, const float* __restrict__ y, const __nv_bfloat16* __restrict__ w,
                                                             T* __restrict__ out, const __nv_bfloat16* __restrict__ pre, int n, int ld, float eps,
-                                                            const SumOf<T> sum) {
+                                                            const SumOf<T> sum, const DepthAverage avg) {
     constexpr int KEEP = 4;
     __shared__ float part[2][8];
     const size_t base = (size_t)blockIdx.x * ld;
@@ -62,6 +72,11 @@ __global__ void __launch_bounds__(256) add_norm_rows_kernel(float* __restrict__ 
             const float4 v = load4(sum.ye + (size_t)sum.place[i] * ld + 4 * c);
             a.x = fmaf(g, v.x, a.x); a.y = fmaf(g, v.y, a.y); a.z = fmaf(g, v.z, a.z); a.w = fmaf(g, v.w, a.w);
         }
+        if (sum.shared != nullptr) {
+            const float g = sum.shared_weight[blockIdx.x];
+            const float4 v = load4(sum.shared + base + 4 * c);
+            a.x = fmaf(g, v.x, a.x); a.y = fmaf(g, v.y, a.y); a.z = fmaf(g, v.z, a.z); a.w = fmaf(g, v.w, a.w);
+        }
         return a;
     };
     auto square = [](float s, const float4& v) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s)))); };
@@ -71,7 +86,7 @@ __global__ void __launch_bounds__(256) add_norm_rows_kernel(float* __restrict__ 
         float ss = 0.f;
 #pragma unroll
         for (int i = 0; i < KEEP; ++i)
-            if (tid + 256 * i < nv) { old[i] = load4(x + base + 4 * (tid + 256 * i)); keep[i] = load_y(tid + 256 * i); }
+            if (tid + 256 * i < nv) { old[i] = load4(x_in + base + 4 * (tid + 256 * i)); keep[i] = load_y(tid + 256 * i); }
 #pragma unroll
         for (int i = 0; i < KEEP; ++i)
             if (tid + 256 * i < nv) ss = square(ss, keep[i]);
@@ -80,6 +95,17 @@ __global__ void __launch_bounds__(256) add_norm_rows_kernel(float* __restrict__ 
         auto add = [&](int c, const float4& v, float4 r) {
             const float4 g = load4(w + 4 * c);
             r.x += v.x * inv * g.x; r.y += v.y * inv * g.y; r.z += v.z * inv * g.z; r.w += v.w * inv * g.w;
+            if constexpr (AVG) {
+                store4(avg.hist + avg.n * avg.stride + base + 4 * c, r);
+                const float own = __bfloat162float(avg.w[avg.n]);
+                r.x *= own; r.y *= own; r.z *= own; r.w *= own;
+#pragma unroll 4
+                for (int j = 0; j < avg.n; ++j) {
+                    const float k = __bfloat162float(avg.w[j]);
+                    const float4 h = load4(avg.hist + j * avg.stride + base + 4 * c);
+                    r.x = fmaf(k, h.x, r.x); r.y = fmaf(k, h.y, r.y); r.z = fmaf(k, h.z, r.z); r.w = fmaf(k, h.w, r.w);
+                }
+            }
             store4(x + base + 4 * c, r);
             if constexpr (PRE) s2 = square(s2, r);
             if (!PRE && out != nullptr) store4(out + base + 4 * c, r);
@@ -88,7 +114,7 @@ __global__ void __launch_bounds__(256) add_norm_rows_kernel(float* __restrict__ 
 #pragma unroll
         for (int i = 0; i < KEEP; ++i)
             if (tid + 256 * i < nv) keep[i] = add(tid + 256 * i, keep[i], old[i]);
-        for (int c = tid + 256 * KEEP; c < nv; c += 256) (void)add(c, load_y(c), load4(x + base + 4 * c));
+        for (int c = tid + 256 * KEEP; c < nv; c += 256) (void)add(c, load_y(c), load4(x_in + base + 4 * c));
     } else {
 #pragma unroll
         for (int i = 0; i < KEEP; ++i)
@@ -107,6 +133,49 @@ __global__ void __launch_bounds__(256) add_norm_rows_kernel(float* __restrict__ 
     for (int i = 0; i < KEEP; ++i)
         if (tid + 256 * i < nv) emit(tid + 256 * i, keep[i]);
     for (int c = tid + 256 * KEEP; c < nv; c += 256) emit(c, load4(x + base + 4 * c));
+}
+
+// Input convolution: out = x + sum_back w[taps - 1 - back] x_{t - back}, w [taps][ld]; rows before the pass come from the sequence's
+// ring [taps][ld] (position modulo taps), which the thread with an entry's first rows brings up to date.  Grid (parts of a row, chunks of
+// kConvRows rows); a thread has four channels.  taps - 1 <= kConvRows.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128) input_conv_rows_kernel(const float* __restrict__ x, const __nv_bfloat16* __restrict__ w, T* __restrict__ out, int ld,
+                                                              float* __restrict__ pool, size_t slot_stride, size_t offset, int taps_any, const RowPlan plan) {
+    constexpr int MAXT = TAPS > 0 ? TAPS : kMaxConvTaps;
+    const int taps = TAPS > 0 ? TAPS : taps_any, c = 4 * (blockIdx.x * 128 + threadIdx.x);
+    RowEntry e;
+    int t0;
+    if (!locate_chunk<kConvRows>(plan, blockIdx.y, e, t0) || c >= ld) return;
+    const int n = min(kConvRows, e.n - t0);
+    float* ring = pool + (size_t)e.state * slot_stride + offset + c;
+    const float* src = x + (size_t)(e.row0 + t0) * ld + c;
+    T* dst = out + (size_t)(e.row0 + t0) * ld + c;
+    float4 past[MAXT], k[MAXT];                                        // past[b]: the value b + 1 tokens back
+#pragma unroll
+    for (int b = 0; b < MAXT; ++b) {
+        past[b] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (b < taps) k[b] = load4(w + (size_t)(taps - 1 - b) * ld + c);
+        const int t = t0 - 1 - b;
+        if (b + 1 < taps && e.pos0 + t >= 0) past[b] = t >= 0 ? load4(src - (size_t)(b + 1) * ld) : load4(ring + (size_t)((e.pos0 + t) % taps) * ld);
+    }
+#pragma unroll
+    for (int r = 0; r < kConvRows; ++r) {
+        if (r >= n) break;
+        const float4 v = load4(src + (size_t)r * ld);
+        float4 a = make_float4(fmaf(k[0].x, v.x, v.x), fmaf(k[0].y, v.y, v.y), fmaf(k[0].z, v.z, v.z), fmaf(k[0].w, v.w, v.w));
+#pragma unroll
+        for (int b = 0; b + 1 < MAXT; ++b)
+            if (b + 1 < taps) {
+                a.x = fmaf(k[b + 1].x, past[b].x, a.x); a.y = fmaf(k[b + 1].y, past[b].y, a.y);
+                a.z = fmaf(k[b + 1].z, past[b].z, a.z); a.w = fmaf(k[b + 1].w, past[b].w, a.w);
+            }
+        store4(dst + (size_t)r * ld, a);
+#pragma unroll
+        for (int b = MAXT - 1; b > 0; --b) past[b] = past[b - 1];
+        past[0] = v;
+    }
+    if (t0 == 0)
+        for (int t = max(0, e.n - taps + 1); t < e.n; ++t) store4(ring + (size_t)((e.pos0 + t) % taps) * ld, load4(src + (size_t)t * ld));
 }
 
 __device__ __forceinline__ void load8(const float* p, float (&f)[8]) {

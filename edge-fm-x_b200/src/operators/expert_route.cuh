@@ -6,7 +6,7 @@
 namespace efm {
 
 // z: router logits of all experts.  Scores softmax(z) or sigmoid(z); the groups whose best scores are the largest stay open; the best `top`
-// experts of those are handed to store(k, expert, score) in lane 0.  Ties go to the lower number.
+// experts of those are handed to store(k, expert, score * scale) in lane 0.  Ties go to the lower number.
 template <int N, typename Store>
 __device__ __forceinline__ void route_token_n(const float* z, const RouteShape& r, Store store) {      // at most 32 N experts
     const int lane = threadIdx.x & 31, per = r.experts / r.groups;
@@ -67,7 +67,7 @@ __device__ __forceinline__ void route_token_n(const float* z, const RouteShape& 
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) e = min(e, __shfl_xor_sync(0xffffffffu, e, o));
         e = min(e, r.experts - 1);                                      // logits that are no numbers choose something
-        if (lane == 0) store(k, e, best);
+        if (lane == 0) store(k, e, best * r.scale);
 #pragma unroll
         for (int i = 0; i < N; ++i)
             if (e == lane + 32 * i) v[i] = -2.f;

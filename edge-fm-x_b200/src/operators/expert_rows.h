@@ -8,10 +8,12 @@ namespace efm {
 constexpr int kMaxExperts = 512, kMaxExpertTop = 32, kMaxExpertGroups = 64;
 constexpr int kExpertTile = 128;      // rows of an expert start at multiples of this
 
+enum : int { kSharedNone = 0, kSharedGated = 1, kSharedPlain = 2 };
 struct RouteShape {
     int experts, top, groups, keep;
     int sigmoid;                      // scores: 0 softmax of the logits, 1 sigmoid of each
-    int shared;                       // 1: logit `experts` gates a shared expert
+    int shared;                       // a shared expert: gated by logit `experts`, or as it is
+    float scale;                      // of the choices' weights
 };
 
 struct ExpertRows {

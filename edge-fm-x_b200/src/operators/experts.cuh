@@ -2,8 +2,9 @@
 //   y = sum_k s_k W_down[e_k] (silu(W_gate[e_k] h) * W_up[e_k] h),   s = softmax(W_router h) or sigmoid(W_router h),
 // where e_k are the best experts of the best groups (a group's score is its largest expert score) and s_k their scores as they
 // are; they may scale the experts' inputs instead of their outputs.  A shared expert runs for every token beside them.
-// Weights: [experts][2 * ffp rows][K] with blocks of 64 gate rows followed by the 64 matching up rows, and
-// [experts][n_out][ffp]; ffp is the expert width padded to 64 with zero rows / columns.
+// Experts without a gate are W_down[e_k] relu(W_up[e_k] h)^2.
+// Weights: [experts][2 * ffp rows][K] with blocks of 64 gate rows followed by the 64 matching up rows ([experts][ffp rows][K] without
+// a gate), and [experts][n_out][ffp]; ffp is the expert width padded to 64 with zero rows / columns.
 //
 //   route_token          one token's choice, by one warp (expert_route.cuh; the decode GEMV of gemv.cuh chooses the same way)
 //   expert_route_rows    many rows: choices, weights, and each choice's place among its expert's rows
@@ -27,7 +28,8 @@ __global__ void __launch_bounds__(256) expert_route_rows_kernel(const float* __r
         o.weight[(size_t)row * r.top + k] = w;
         o.place[(size_t)row * r.top + k] = atomicAdd(o.count + e, 1);
     });
-    if (r.shared && (threadIdx.x & 31) == 0) o.shared[row] = 1.0f / (1.0f + expf(-logits[(size_t)row * ld + r.experts]));
+    if (r.shared != kSharedNone && (threadIdx.x & 31) == 0)
+        o.shared[row] = r.shared == kSharedGated ? 1.0f / (1.0f + expf(-logits[(size_t)row * ld + r.experts])) : 1.0f;
 }
 
 // First row of every expert in the sorted order, by the first warp; block 0 describes the tiles.
@@ -89,7 +91,7 @@ __global__ void __launch_bounds__(128) expert_gather_rows_kernel(const T* __rest
     }
 }
 
-// gu: rows of 64 gate values followed by the 64 matching up values -> gated unit, ffp columns.  Grid: tiles of kExpertTile rows, of
+// gu: rows of 64 gate values followed by the 64 matching up values -> gated unit, ffp columns (Relu2: ffp values -> their unit).  Grid: tiles of kExpertTile rows, of
 // which *n_tiles (null: all) are in use.
 __global__ void __launch_bounds__(256) glu_rows_kernel(const float* __restrict__ gu, float* __restrict__ out, int rows, int ffp, const int32_t* __restrict__ n_tiles,
                                                        int kind, float limit) {
@@ -98,6 +100,10 @@ __global__ void __launch_bounds__(256) glu_rows_kernel(const float* __restrict__
     for (int i = threadIdx.x; i < kExpertTile * ffp; i += 256) {
         const int r = i / ffp, c = i - r * ffp;
         if (tile * kExpertTile + r >= rows) return;
+        if (kind == kGluRelu2) {
+            out[(size_t)(tile * kExpertTile + r) * ffp + c] = relu2(gu[(size_t)(tile * kExpertTile + r) * ffp + c]);
+            continue;
+        }
         const float* src = gu + (size_t)(tile * kExpertTile + r) * 2 * ffp + (c >> 6) * 128 + (c & 63);
         out[(size_t)(tile * kExpertTile + r) * ffp + c] = glu(kind, src[0], src[64], limit);
     }

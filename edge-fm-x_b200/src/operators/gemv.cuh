@@ -35,13 +35,15 @@ enum class Epi : int { Plain = 0, Residual = 1, QkvRope = 2, SwiGlu = 3, Logits 
 constexpr int kMaxPeers = 8;
 // Embed and what follows it (and the epilogues from Store32 on) exist in the EXT instantiations only (layered decoders; level 2 adds
 // input norms: Norm, and the second norm and the scale of Embed; level 3 elementwise input norms, AddTanh and Merge, the clamped
-// and the shared expert and the cap of the logits):
+// and the shared expert and the cap of the logits; level 4 input convolutions, the average over depth and experts without a gate):
 //   Embed    x = embed_table[token] * embed_scale; with norm2_w the product reads rmsnorm(x) * norm2_w
 //   Norm     x = rmsnorm(xf) * norm_w
 //   AddNorm  x = xr + rmsnorm(addend) * norm_w: a sublayer whose OUTPUT is normalised, folded into the next product;
 //            with norm2_w the product reads rmsnorm(x) * norm2_w instead of x
 //   PolyNorm x = c0 rms(z) + c1 rms(z^2) + c2 rms(z^3) + c3 with z = xf and the four numbers of `poly`
 //   AddTanh  x = xr + add_mult * addend; the product reads tanh(alpha x) * norm_w + norm_b (Embed does the same when norm_b is given)
+//            level 4, Embed and AddNorm: with avg the stream is avg + avg_w x instead of x, with conv_w the product reads the stream plus
+//            its convolution over the last conv_taps tokens
 //   Merge    channels [0, merge0) of xf as they are, the others rmsnorm(xf) * norm_w * sigmoid(merge_gate) * merge_scale
 enum : int { kProPlain = 0, kProRmsNorm = 1, kProEmbedRmsNorm = 2, kProEmbed = 3, kProAddNorm = 4, kProPolyNorm = 5, kProNorm = 6, kProAddTanh = 7, kProMerge = 8 };
 
@@ -123,10 +125,28 @@ struct GemvParams {
     float limit, shared_limit;
     const __nv_bfloat16* W2;
     int shared_ff, shared_ffp;
+    // level 4.  Relu2 experts: item = (choice, pair of channels), ff and shared_ff count pairs.
+    // conv_ring: [conv_taps][K], the stream's earlier values by position modulo conv_taps; block 0 adds this token's.  conv_early: what
+    // earlier steps left (and the device state) may be read before the dependency wait
+    const __nv_bfloat16* conv_w;          // [conv_taps][K], null: none
+    float* conv_ring;
+    int conv_taps, conv_early;
+    const float* avg;                     // [K], null: none
+    const __nv_bfloat16* avg_w;           // one number
+    float* hist_out;                      // not null: block 0 stores the layer's result (Embed: the embedding) here
+    // a product that runs meanwhile prepares avg for the next one: sum_out = sum_{j < sum_n} sum_w[j] sum_in[j], rows of sum_k numbers
+    const float* sum_in;
+    const __nv_bfloat16* sum_w;
+    float* sum_out;
+    int sum_n, sum_k;
 };
 
 // gated units: silu(g) u, or (clamped) g sigmoid(1.702 g) (u + 1) with g at most and u within +- limit
-enum : int { kGluSilu = 0, kGluClamped = 1 };
+enum : int { kGluSilu = 0, kGluClamped = 1, kGluRelu2 = 2 };       // Relu2: no gate, the square of relu
+__device__ __forceinline__ float relu2(float z) {
+    z = fmaxf(z, 0.f);
+    return z * z;
+}
 __device__ __forceinline__ float glu(int kind, float g, float u, float limit) {
     if (kind == kGluSilu) return g / (1.0f + expf(-g)) * u;
     g = fminf(g, limit);
@@ -173,6 +193,13 @@ __device__ __forceinline__ void item_rows(const GemvParams& p, int item, int& r0
         r1 = r0 + 64;
     } else if constexpr (EPI == Epi::ExpertUp) {
         const int k = item / p.ff, j = item - (EXT > 2 && k >= p.route.top ? p.route.top : k) * p.ff;
+        if constexpr (EXT > 3) {
+            if (p.glu == kGluRelu2) {
+                r0 = (k >= p.route.top ? 0 : chosen[k] * p.expert_rows) + 2 * j;
+                r1 = r0 + 1;
+                return;
+            }
+        }
         r0 = (EXT > 2 && k >= p.route.top ? 0 : chosen[k] * p.expert_rows) + ((j >> 6) << 7) + (j & 63);
         r1 = r0 + 64;
     } else {
@@ -214,6 +241,13 @@ __device__ __forceinline__ void item_epilogue(const GemvParams& p, int item, flo
         if (a1 > best_v) { best_v = a1; best_i = item * 2 + 1; }      // the lowest id on ties
     } else if constexpr (EPI == Epi::ExpertUp) {
         const int k = item / p.ff;
+        if constexpr (EXT > 3) {
+            if (p.glu == kGluRelu2) {
+                const int k2 = min(k, p.route.top);
+                *reinterpret_cast<float2*>(p.out_f + k2 * p.ffp + 2 * (item - k2 * p.ff)) = make_float2(relu2(a0), relu2(a1));
+                return;
+            }
+        }
         if constexpr (EXT > 2) {
             const bool shared = k >= p.route.top;
             const float w = !shared && p.weight_input ? __int_as_float(chosen[kMaxExpertTop + k]) : 1.0f;      // a product is linear in its input
@@ -229,9 +263,7 @@ __device__ __forceinline__ void item_epilogue(const GemvParams& p, int item, flo
     } else if constexpr (EPI == Epi::Store32Bias) {
         *reinterpret_cast<float2*>(p.out_f + item * 2) = make_float2(a0 + __bfloat162float(p.bias[item * 2]), a1 + __bfloat162float(p.bias[item * 2 + 1]));
     } else if constexpr (EPI == Epi::Relu2) {
-        a0 = fmaxf(a0, 0.f);
-        a1 = fmaxf(a1, 0.f);
-        *reinterpret_cast<float2*>(p.out_f + item * 2) = make_float2(a0 * a0, a1 * a1);
+        *reinterpret_cast<float2*>(p.out_f + item * 2) = make_float2(relu2(a0), relu2(a1));
     } else if constexpr (EPI == Epi::Store32) {
         *reinterpret_cast<float2*>(p.out_f + item * 2) = make_float2(a0, a1);
     } else if constexpr (EPI == Epi::TokenGate) {
@@ -370,6 +402,30 @@ __host__ __device__ inline unsigned int gemv_wbytes(int K) { return ((unsigned i
 // Offset of the second staged vector of the EXT prologues (behind red + misc).
 __host__ __device__ inline unsigned int gemv_ext_off(int K) { return gemv_xbytes(K) + gemv_wbytes(K) + (2 * 16 * 2 + 16) * 4u; }
 
+// Behind that, with an input convolution: what the earlier tokens contribute (fp32 K), the weight of the token itself (bf16 K).
+__host__ __device__ inline unsigned int gemv_conv_off(int K) { return gemv_ext_off(K) + gemv_xbytes(K); }
+
+template <int EXT>
+__device__ __forceinline__ void gemv_stage_conv(const GemvParams& p, const int nch, unsigned char* smem) {
+    float* past = reinterpret_cast<float*>(smem + gemv_conv_off(p.K));
+    uint4* own = reinterpret_cast<uint4*>(smem + gemv_conv_off(p.K) + gemv_xbytes(p.K));
+    const int taps = p.conv_taps, pos = (int)p.state->kv_len - 1;
+    for (int c = threadIdx.x; c < nch; c += kGemvThreads) {
+        float a[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+        own[c] = ld_cached(p.conv_w + (size_t)(taps - 1) * p.K + 8 * c);
+        for (int back = 1; back < taps && back <= pos; ++back) {
+            float w[8];
+            unpack8(ld_cached(p.conv_w + (size_t)(taps - 1 - back) * p.K + 8 * c), w);
+            const float4* h = reinterpret_cast<const float4*>(p.conv_ring + (size_t)((pos - back) % taps) * p.K + 8 * c);
+            const float4 x = __ldcg(h), y = __ldcg(h + 1);
+            a[0] = fmaf(w[0], x.x, a[0]); a[1] = fmaf(w[1], x.y, a[1]); a[2] = fmaf(w[2], x.z, a[2]); a[3] = fmaf(w[3], x.w, a[3]);
+            a[4] = fmaf(w[4], y.x, a[4]); a[5] = fmaf(w[5], y.y, a[5]); a[6] = fmaf(w[6], y.z, a[6]); a[7] = fmaf(w[7], y.w, a[7]);
+        }
+        *reinterpret_cast<float4*>(past + 8 * c) = make_float4(a[0], a[1], a[2], a[3]);
+        *reinterpret_cast<float4*>(past + 8 * c + 4) = make_float4(a[4], a[5], a[6], a[7]);
+    }
+}
+
 // Weights only: the first two units into registers, the norm weight into shared memory.
 template <Epi EPI, int EXT>
 __device__ __forceinline__ void gemv_prefetch(const GemvParams& p, const GemvSched& sc, GemvRegs& r, unsigned char* smem,
@@ -388,6 +444,25 @@ __device__ __forceinline__ void gemv_prefetch(const GemvParams& p, const GemvSch
         if (p.prologue == kProMerge) {
             uint4* gs = reinterpret_cast<uint4*>(smem + xbytes);
             for (int c = threadIdx.x; c < sc.nch - p.merge0 / 8; c += kGemvThreads) gs[c] = ld_cached(p.norm_w + (size_t)c * 8);
+        }
+    }
+    if constexpr (EXT > 3) {
+        if (p.conv_w != nullptr && p.conv_early) gemv_stage_conv<EXT>(p, sc.nch, smem);
+        // the rows of the sum are complete: their writers ran before the product this launch may overlap with
+        if (p.sum_n > 0) {
+            const int n4 = p.sum_k / 4, per = (n4 + (int)gridDim.x - 1) / (int)gridDim.x;
+            for (int i = threadIdx.x; i < per; i += kGemvThreads) {
+                const int c = (int)blockIdx.x * per + i;
+                if (c >= n4) break;
+                float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+                for (int j = 0; j < p.sum_n; ++j) {
+                    const float4 v = __ldcg(reinterpret_cast<const float4*>(p.sum_in + (size_t)j * p.sum_k) + c);
+                    const float w = __bfloat162float(p.sum_w[j]);
+                    a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y); a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
+                }
+                reinterpret_cast<float4*>(p.sum_out)[c] = a;
+            }
         }
     }
 }
@@ -449,6 +524,24 @@ __device__ __forceinline__ bool gemv_stage_ext(const GemvParams& p, const int nc
         if (p.x_out != nullptr && blockIdx.x == 0) st8f(p.x_out + 8 * c, f);
     };
     (void)tanh8;
+    // level 4: x, the stream of chunk c, becomes what the product reads (same thread and chunk as in gemv_stage_conv)
+    auto conv8 = [&](int c, float (&x)[8]) {
+        const float* past = reinterpret_cast<const float*>(smem + gemv_conv_off(p.K)) + 8 * c;
+        const uint4 wv = reinterpret_cast<const uint4*>(smem + gemv_conv_off(p.K) + gemv_xbytes(p.K))[c];
+        float w[8];
+        unpack8(wv, w);
+        const int pos = (int)p.state->kv_len - 1;
+        if (blockIdx.x == 0 && pos >= 0) st8f(p.conv_ring + (size_t)(pos % p.conv_taps) * p.K + 8 * c, x);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[j] = x[j] + fmaf(w[j], x[j], past[j]);
+        if (p.x_out != nullptr && blockIdx.x == 0) st8f(p.x_out + 8 * c, x);
+    };
+    (void)conv8;
+    if constexpr (EXT > 3) {
+        if (p.conv_w != nullptr && !p.conv_early) gemv_stage_conv<EXT>(p, nch, smem);
+    }
+    const float avg_w = EXT > 3 && p.avg != nullptr ? __bfloat162float(*p.avg_w) : 0.f;
+    (void)avg_w;
     if (p.prologue == kProEmbed) {
         const int tok = p.state->token;
         const bool zero = tok < 0 || tok >= p.vocab;
@@ -464,6 +557,10 @@ __device__ __forceinline__ bool gemv_stage_ext(const GemvParams& p, const int nc
                 }
             }
             if (blockIdx.x == 0) st8f(p.resid_out + 8 * c, f);
+            if constexpr (EXT > 3) {
+                if (p.hist_out != nullptr && blockIdx.x == 0) st8f(p.hist_out + 8 * c, f);
+                if (p.conv_w != nullptr) conv8(c, f);
+            }
             if constexpr (EXT > 2) {
                 if (p.norm_b != nullptr) tanh8(c, f, ld_cached(p.norm_w + (size_t)c * 8), ld_cached(p.norm_b + (size_t)c * 8));
             }
@@ -552,12 +649,23 @@ __device__ __forceinline__ bool gemv_stage_ext(const GemvParams& p, const int nc
             float w[8], x[8];
             unpack8(gs[c], w);
 #pragma unroll
-            for (int j = 0; j < 8; ++j) {
-                x[j] = xs2[8 * c + j] + xs[8 * c + j] * inv * w[j];
-                s2[0] = fmaf(x[j], x[j], s2[0]);
+            for (int j = 0; j < 8; ++j) x[j] = xs2[8 * c + j] + xs[8 * c + j] * inv * w[j];
+            if constexpr (EXT > 3) {
+                if (p.hist_out != nullptr && blockIdx.x == 0) st8f(p.hist_out + 8 * c, x);
+                if (p.avg != nullptr) {
+                    float a[8];
+                    ld8f(p.avg + 8 * c, a);
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) x[j] = fmaf(avg_w, x[j], a[j]);
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < 8; ++j) s2[0] = fmaf(x[j], x[j], s2[0]);
+            if (blockIdx.x == 0) st8f(p.resid_out + 8 * c, x);
+            if constexpr (EXT > 3) {
+                if (p.conv_w != nullptr) conv8(c, x);
             }
             st8f(xs + 8 * c, x);
-            if (blockIdx.x == 0) st8f(p.resid_out + 8 * c, x);
         }
         if (p.norm2_w != nullptr) norm2(s2);
     } else if (p.prologue == kProPolyNorm) {
@@ -851,7 +959,8 @@ __global__ void __launch_bounds__(kGemvThreads, 1) gemv_kernel(const GemvParams 
         if (last != 0u && threadIdx.x < 32) {
             route_token(p.out_f, p.route, [&](int k, int e, float w) { p.route_id[k] = e; p.route_w[k] = w; });
             if (threadIdx.x == 0) {
-                if (p.route.shared) p.route_w[p.route.top] = 1.0f / (1.0f + expf(-__ldcg(p.out_f + p.route.experts)));
+                if (p.route.shared == kSharedGated) p.route_w[p.route.top] = 1.0f / (1.0f + expf(-__ldcg(p.out_f + p.route.experts)));
+                else if (p.route.shared == kSharedPlain) p.route_w[p.route.top] = 1.0f;
                 *p.route_ticket = 0u;
             }
         }
@@ -873,6 +982,8 @@ __global__ void __launch_bounds__(kGemvThreads, 1) gemv_kernel(const GemvParams 
 __host__ __device__ inline size_t gemv_smem_bytes(int K) {      // xs (fp32) | norm weight | red + misc
     return (size_t)gemv_xbytes(K) + gemv_wbytes(K) + (size_t)(2 * kGemvWarps * 2 + 16) * sizeof(float);
 }
+
+__host__ __device__ inline size_t gemv_conv_smem_bytes(int K) { return (size_t)gemv_conv_off(K) + gemv_xbytes(K) + gemv_wbytes(K); }
 
 // EXT instantiations: room for the second vector of a prologue.
 __host__ __device__ inline size_t gemv_ext_smem_bytes(int K) { return (size_t)gemv_ext_off(K) + (size_t)K * 4; }

@@ -1,7 +1,8 @@
 // Causal softmax attention over a paged cache with a sliding window, kept first tokens and per-head score modification:
 //   score(i, j) = (q_i . k_j) * scale * temp[h] - slope_h * (i - j),   0 <= i - j < window (window 0: no lower bound) or j < keep
-// with slope_h = 2^(-8 (h + 1) / H), q and k RMS-normalised per head (with or without a weight, or not at all) and then rotated
-// before they are used / cached, value width free.  A weightless norm commutes with the rotation, which keeps a head's length.
+// with slope_h = 2^(-8 (h + 1) / H), q and k RMS-normalised per head (with or without a weight, or not at all) or over all heads
+// at once (with a weight), and then rotated before they are used / cached, value width free.  Instead of the softmax a key's weight may be
+// sigmoid(score + shift[h]), not normalised; a head's output may be multiplied by sigmoid(gate_h).  A weightless norm commutes with the rotation, which keeps a head's length.
 // Cache: per layer a K pool [pages * 64][kv_heads][Dp] and a V pool [pages * 64][kv_heads][Vp], channels zero-padded to
 // Dp / Vp (multiples of 64); a sequence's pages are listed in a page table.  TC = bf16 or fp32 (the all-32-bit mode).
 //
@@ -27,18 +28,21 @@ struct WindowAttnShape {
     int window;                       // 0: full causal
     int keep;                         // first tokens that stay visible (with a window)
     int bias;                         // 1: distance bias
-    int qk_norm;                      // 0: q and k as they are
+    int qk_norm;                      // 0: q and k as they are; 1: per head; 2: over all heads, weights [H * D] and [G * D]
+    const __nv_bfloat16* shift;       // not null: sigmoid weights, [H]
     float scale, eps;
     float out_scale;                  // of the result
     const __nv_bfloat16* q_norm;      // [D], null: norm without a weight
     const __nv_bfloat16* k_norm;      // [D]
     const __nv_bfloat16* temp;        // [H], null: 1
     RotShape rot;
-    // tensor-core form with a shared key part only: extra term exp(sink[h]) of the softmax denominator, and heads multiplied by sigmoid(gate)
+    // tensor-core form with a shared key part only: extra term exp(sink[h]) of the softmax denominator, and channels multiplied by
+    // sigmoid(gate)
     const __nv_bfloat16* sink;        // [H], null: none
-    const __nv_bfloat16* gate;        // [T][H * Dv], or (gate_heads) [T][H], with row stride gate_ld, null: none
+    const void* gate;                 // [T][H * Dv], or (gate_heads) [T][H], of the pass's activation type with row stride gate_ld, null: none
     int gate_ld, gate_heads;
 };
+__device__ __forceinline__ float sigmoid_weight(float score) { return 1.0f / (1.0f + expf(-score)); }
 
 __device__ __forceinline__ float head_multiplier(const WindowAttnShape& s, int h) {
     return s.temp != nullptr ? s.scale * __bfloat162float(s.temp[h]) : s.scale;
@@ -96,6 +100,7 @@ __global__ void __launch_bounds__(256, 4) qk_scatter_rows_kernel(const TI* __res
     __shared__ __align__(16) float cs[kRotMaxPairs];
     __shared__ __align__(16) float sn[kRotMaxPairs];
     __shared__ float stage[ROT ? 256 * 8 : 1];
+    __shared__ float row_ss[2][8];
     const int row = blockIdx.x, l = threadIdx.x & (lanes - 1), per = 256 / lanes;
     const RowEntry e = plan.of_row(row);
     const int half = s.rot.dims / 2;
@@ -108,6 +113,21 @@ __global__ void __launch_bounds__(256, 4) qk_scatter_rows_kernel(const TI* __res
     const TI* src = qkv + (size_t)row * ld;                            // ld % 8 == 0
     const bool vec = (s.D & 7) == 0, vecv = vec && (s.Dv & 7) == 0;
     const int units = s.H + 2 * s.G, d = 8 * l;
+    float inv_q = 1.f, inv_k = 1.f;
+    if (s.qk_norm == 2) {
+        float sq = 0.f, sk = 0.f;
+        for (int c = threadIdx.x; c < s.H * s.D; c += 256) { const float v = to_f32(src[c]); sq = fmaf(v, v, sq); }
+        for (int c = threadIdx.x; c < s.G * s.D; c += 256) { const float v = to_f32(src[s.H * s.D + c]); sk = fmaf(v, v, sk); }
+        sq = warp_sum(sq);
+        sk = warp_sum(sk);
+        if ((threadIdx.x & 31) == 0) { row_ss[0][threadIdx.x >> 5] = sq; row_ss[1][threadIdx.x >> 5] = sk; }
+        __syncthreads();
+        sq = sk = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) { sq += row_ss[0][i]; sk += row_ss[1][i]; }
+        inv_q = 1.0f / sqrtf(sq / (float)(s.H * s.D) + s.eps);
+        inv_k = 1.0f / sqrtf(sk / (float)(s.G * s.D) + s.eps);
+    }
     for (int u0 = 0; u0 < units; u0 += per) {                          // every thread takes part in the shuffles
         const int u = u0 + threadIdx.x / lanes;
         const bool qk = u < s.H + s.G;
@@ -115,13 +135,14 @@ __global__ void __launch_bounds__(256, 4) qk_scatter_rows_kernel(const TI* __res
         if (qk) load_head8(src + (size_t)u * s.D, d, s.D, vec, f);     // q heads, then k heads
         else if (u < units) load_head8(src + (size_t)(s.H + s.G) * s.D + (size_t)(u - s.H - s.G) * s.Dv, d, s.Dv, vecv, f);
         const __nv_bfloat16* w = u < s.H ? s.q_norm : s.k_norm;
+        if (s.qk_norm == 2 && qk) w += (size_t)(u < s.H ? u : u - s.H) * s.D;
         float ss = 0.f, g[8];
         if (qk && w != nullptr) load_head8(w, d, s.D, vec, g);
 #pragma unroll
         for (int j = 0; j < 8; ++j) ss = fmaf(f[j], f[j], ss);
         for (int x = lanes / 2; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
         if (qk) {
-            const float inv = s.qk_norm ? 1.0f / sqrtf(ss / (float)s.D + s.eps) : 1.0f;
+            const float inv = s.qk_norm == 2 ? (u < s.H ? inv_q : inv_k) : s.qk_norm ? 1.0f / sqrtf(ss / (float)s.D + s.eps) : 1.0f;
 #pragma unroll
             for (int j = 0; j < 8; ++j) f[j] *= inv;                   // channels past D are zero
             if (w != nullptr) {
@@ -207,6 +228,8 @@ __global__ void __launch_bounds__(256) window_attention_rows_kernel(const TQ* __
     for (int n = 0; n < 4; ++n)
 #pragma unroll
         for (int j = 0; j < 4; ++j) acc[n][j] = 0.f;
+    const bool sig = s.shift != nullptr;
+    const float shift = sig ? __bfloat162float(s.shift[h]) : 0.f;
     float m = -INFINITY, l = 0.f;
     for (int k0 = kept > 0 ? 0 : first_tile; k0 < end; k0 = k0 + KT >= kept ? max(k0 + KT, first_tile) : k0 + KT) {
         __syncthreads();
@@ -232,6 +255,10 @@ __global__ void __launch_bounds__(256) window_attention_rows_kernel(const TQ* __
             }
             sc[u] = ((j >= lo || j < s.keep) && j <= i_pos) ? (d0 + d1) * mul - slope * (float)(i_pos - j) : -INFINITY;
         }
+        if (sig) {
+#pragma unroll
+            for (int u = 0; u < 2; ++u) ps[r * (KT + 1) + c + 16 * u] = sc[u] == -INFINITY ? 0.f : sigmoid_weight(sc[u] + shift);
+        } else {
         float mx = fmaxf(sc[0], sc[1]);
 #pragma unroll
         for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
@@ -252,6 +279,7 @@ __global__ void __launch_bounds__(256) window_attention_rows_kernel(const TQ* __
         for (int n = 0; n < 4; ++n)
 #pragma unroll
             for (int j = 0; j < 4; ++j) acc[n][j] *= alpha;
+        }
         __syncwarp();                                                  // the 16 lanes of a row share a warp
         for (int kr = 0; kr < KT; ++kr) {
             const float p = ps[r * (KT + 1) + kr];
@@ -265,7 +293,8 @@ __global__ void __launch_bounds__(256) window_attention_rows_kernel(const TQ* __
         }
     }
     if (r >= nq) return;
-    const float inv = l > 0.f ? s.out_scale / l : 0.f;
+    float inv = sig ? s.out_scale : l > 0.f ? s.out_scale / l : 0.f;
+    if (s.gate != nullptr) inv *= sigmoid_weight(to_f32(static_cast<const TQ*>(s.gate)[(size_t)(e.row0 + r0 + r) * s.gate_ld + h]));
     TO* dst = out + (size_t)(e.row0 + r0 + r) * ld_out + (size_t)h * s.Dv;
 #pragma unroll
     for (int n = 0; n < 4; ++n)
@@ -304,6 +333,7 @@ struct WindowDecodeParams {
     int max_pages;
     DecodeState* state;
     float* out;                       // [H * Dv]
+    const float* gate;                // [H], null: none
     int early;                        // 1: state and the older cache rows may be read before the dependency wait
     LinearDecodeParams lin;           // linear attention beside this one: its blocks follow in grid.y
 };
@@ -401,10 +431,26 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
     if (p.early) { pdl_wait(); pdl_launch_dependents(); }
 
     // ---- norms and rotation of this token's q heads and k, v ------------------------------------------------------------------
+    float inv_q = 1.f, inv_k = 1.f;
+    if (s.qk_norm == 2) {                                              // over all heads: every block sums for itself
+        float sq = 0.f, sk = 0.f;
+        for (int c = tid; c < s.H * s.D; c += kThreads) { const float v = __ldcg(p.qkv + c); sq = fmaf(v, v, sq); }
+        for (int c = tid; c < s.G * s.D; c += kThreads) { const float v = __ldcg(p.qkv + s.H * s.D + c); sk = fmaf(v, v, sk); }
+        sq = warp_sum(sq);
+        sk = warp_sum(sk);
+        if (lane == 0) { sm.red[warp] = sq; sm.red[8 + warp] = sk; }
+        __syncthreads();
+        sq = sk = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) { sq += sm.red[i]; sk += sm.red[8 + i]; }
+        inv_q = 1.0f / sqrtf(sq / (float)(s.H * s.D) + s.eps);
+        inv_k = 1.0f / sqrtf(sk / (float)(s.G * s.D) + s.eps);
+    }
     for (int u = warp; u < nh + 1; u += 8) {
         const bool is_q = u < nh;
         const float* x = is_q ? p.qkv + (size_t)(h0 + u) * s.D : p.qkv + (size_t)(s.H + g) * s.D;
         const __nv_bfloat16* w = is_q ? s.q_norm : s.k_norm;
+        if (s.qk_norm == 2) w += is_q ? (size_t)(h0 + u) * s.D : (size_t)g * s.D;
         float f[VM / 32], ss = 0.f;
 #pragma unroll
         for (int i = 0; i < VM / 32; ++i) {
@@ -413,7 +459,7 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
         }
 #pragma unroll
         for (int i = 0; i < VM / 32; ++i) ss = fmaf(f[i], f[i], ss);
-        const float inv = s.qk_norm ? 1.0f / sqrtf(warp_sum(ss) / (float)s.D + s.eps) : 1.0f;
+        const float inv = s.qk_norm == 2 ? (is_q ? inv_q : inv_k) : s.qk_norm ? 1.0f / sqrtf(warp_sum(ss) / (float)s.D + s.eps) : 1.0f;
 #pragma unroll
         for (int i = 0; i < VM / 32; ++i) {
             const int d = lane + 32 * i;
@@ -492,7 +538,12 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
         }
         __syncthreads();
         // ---- online softmax: one warp per head --------------------------------------------------------------------
-        if (warp < nh) {
+        if (warp < nh && s.shift != nullptr) {                         // weights that need no other key's
+            const float b = __bfloat162float(s.shift[h0 + warp]), s0 = sm.p[warp][lane], s1 = sm.p[warp][lane + 32];
+            sm.p[warp][lane] = s0 == -INFINITY ? 0.f : sigmoid_weight(s0 + b);
+            sm.p[warp][lane + 32] = s1 == -INFINITY ? 0.f : sigmoid_weight(s1 + b);
+            if (lane == 0) sm.alpha[warp] = 1.0f;
+        } else if (warp < nh) {
             const float s0 = sm.p[warp][lane], s1 = sm.p[warp][lane + 32];
             const float m_old = sm.m[warp], mn = fmaxf(m_old, warp_max(fmaxf(s0, s1)));       // the tile holds a visible key
             const float p0 = expf(s0 - mn), p1 = expf(s1 - mn);
@@ -564,6 +615,13 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
     cl.sync();
     for (int i = tid; i < share && split * share + i < n_out; i += kThreads) {
         const int o = split * share + i, h = o / s.Dv, d = o - h * s.Dv;
+        const float gate = p.gate != nullptr ? sigmoid_weight(__ldcg(p.gate + h0 + h)) : 1.0f;
+        if (s.shift != nullptr) {
+            float sum = 0.f;
+            for (int r = 0; r < n_splits; ++r) sum += sm.rout[r * share + i];
+            p.out[(size_t)(h0 + h) * s.Dv + d] = s.out_scale * gate * sum;
+            continue;
+        }
         float m = -INFINITY;
         for (int r = 0; r < n_splits; ++r) m = fmaxf(m, sm.rm[r][h]);
         float num = 0.f, den = 0.f;
@@ -572,7 +630,7 @@ __global__ void __launch_bounds__(wd::kThreads) window_attention_decode_kernel(c
             num = fmaf(w, sm.rout[r * share + i], num);
             den = fmaf(w, sm.rl[r][h], den);
         }
-        p.out[(size_t)(h0 + h) * s.Dv + d] = den > 0.f ? s.out_scale * (num / den) : 0.f;
+        p.out[(size_t)(h0 + h) * s.Dv + d] = den > 0.f ? s.out_scale * gate * (num / den) : 0.f;
     }
 }
 

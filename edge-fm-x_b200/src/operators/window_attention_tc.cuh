@@ -58,7 +58,8 @@ struct WindowTcMaps {
     CUtensorMap qr, kr;               // RP > 0: rotated parts, [rows][heads][channels] and [rows][1][channels]
 };
 
-template <int DP, int VP, int RP, bool KEEP>
+// SIG: weights sigmoid(score + shift[h]); no maximum, no denominator, and P V of all tiles accumulates in tensor memory.
+template <int DP, int VP, int RP, bool KEEP, bool SIG = false>
 __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(const __grid_constant__ WindowTcMaps maps, __nv_bfloat16* __restrict__ out,
                                                                            int ld_out, const WindowAttnShape s, const RowPlan plan,
                                                                            const RowTile* __restrict__ tiles, int n_tiles_all, int first_wave, int workspace,
@@ -129,7 +130,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     const uint64_t vdesc[2] = {at::umma_desc_mn(sV, (uint32_t)(BN * 128), 1024u), at::umma_desc_mn(sV + C::V_BYTES, (uint32_t)(BN * 128), 1024u)};
     constexpr float kLog2e = 1.4426950408889634f;
     const float f2 = head_multiplier(s, h) * kLog2e;
-    const float b2 = (s.bias ? distance_slope(h, s.H) : 0.f) * kLog2e;
+    const float b2 = (s.bias ? distance_slope(h, s.H) : 0.f) * kLog2e, shift2 = SIG ? __bfloat162float(s.shift[h]) * kLog2e : 0.f;
     float o[C::HALF];
 #pragma unroll
     for (int i = 0; i < C::HALF; ++i) o[i] = 0.f;
@@ -195,11 +196,17 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
         uint32_t sr[32];
         tc::tmem_ld32(tmem + ((uint32_t)((warp & 3) * 32) << 16) + (uint32_t)(hf * 32), sr);
         const int kb = tile_page(j) * BN, key0 = kb + hf * 32;
-        float sc[32];                                            // scores in units of log2
+        float sc[32];                                            // scores in units of log2 (SIG: weights)
         float mx = -INFINITY;
         const float bias0 = b2 * (float)(key0 - i_pos);
         const bool interior = (kb >= lo_max || (KEEP && kb + BN <= keep)) && kb + BN <= hi_min;
-        if (interior && b2 == 0.f) {                             // most tiles: every key visible
+        if constexpr (SIG) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+                const float w = __fdividef(1.0f, 1.0f + at::ex2(-fmaf(__uint_as_float(sr[i]), f2, shift2)));
+                sc[i] = interior || ((key0 + i >= lo || (KEEP && key0 + i < keep)) && key0 + i < hi) ? w : 0.f;
+            }
+        } else if (interior && b2 == 0.f) {                             // most tiles: every key visible
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
                 sc[i] = __uint_as_float(sr[i]) * f2;
@@ -213,7 +220,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
                 mx = fmaxf(mx, sc[i]);
             }
         }
-        xch[hf * BM + row] = mx;
+        if constexpr (!SIG) xch[hf * BM + row] = mx;
         asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
         if (__syncthreads_or(*abort_s != 0)) break;             // every thread takes the same decision
         if (C::KBUF > 1 && tid == 0 && j + 1 < ntiles) {         // every thread holds its scores: S of the next tile
@@ -222,7 +229,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
             else *abort_s = 1;
         }
         __syncwarp();
-        const float m_new = fmaxf(m, fmaxf(xch[row], xch[BM + row]));
+        const float m_new = SIG ? 0.f : fmaxf(m, fmaxf(xch[row], xch[BM + row]));
         const float mb = m_new == -INFINITY ? 0.f : m_new;
         const float alpha = m == -INFINITY ? 0.f : at::ex2(m - mb);
         m = m_new;
@@ -230,7 +237,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
         uint32_t pk[16], pl[16];
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
-            const float a = at::ex2(sc[i] - mb), b = at::ex2(sc[i + 1] - mb);      // exp2(-inf) = 0 for masked keys
+            const float a = SIG ? sc[i] : at::ex2(sc[i] - mb), b = SIG ? sc[i + 1] : at::ex2(sc[i + 1] - mb);      // exp2(-inf) = 0 for masked keys
             rs += a + b;
             pk[i >> 1] = pack_bf16(a, b);                            // the weights as a bf16 pair high + low: 16 bits of mantissa
             pl[i >> 1] = pack_bf16(a - bf16lo(pk[i >> 1]), b - bf16hi(pk[i >> 1]));
@@ -247,7 +254,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
         const uint32_t prow = tmem + ((uint32_t)((warp & 3) * 32) << 16) + (uint32_t)(C::P_COL + hf * 16);
         wt::tmem_st16(prow, pk);
         wt::tmem_st16(prow + 32u, pl);
-        if (j > 0) fold();
+        if (!SIG && j > 0) fold();
         alpha_prev = alpha;
         asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
         asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -258,7 +265,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
             if (ok) {
 #pragma unroll
                 for (int k = 0; k < 2 * (BN / 16); ++k)              // high halves, then low halves
-                    wt::umma_ts(tmem + C::O_COL, tmem + (uint32_t)(C::P_COL + 8 * k), vdesc[j & 1] + (uint64_t)((k % (BN / 16)) * (2048 >> 4)), kDescO, k != 0 ? 1u : 0u);
+                    wt::umma_ts(tmem + C::O_COL, tmem + (uint32_t)(C::P_COL + 8 * k), vdesc[j & 1] + (uint64_t)((k % (BN / 16)) * (2048 >> 4)), kDescO, k != 0 || (SIG && j > 0) ? 1u : 0u);
                 umma_commit(obar);
                 if (C::KBUF == 1 && j + 1 < ntiles) {
                     ok = mbar_wait(kfull0 + 8 * ((j + 1) % C::KBUF), (uint32_t)((j + 1) / C::KBUF) & 1u, abort_s);
@@ -288,7 +295,7 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     __syncthreads();
     xch[hf * BM + row] = l;
     __syncthreads();
-    float L = xch[row] + xch[BM + row], up = 1.0f;
+    float L = SIG ? 1.0f : xch[row] + xch[BM + row], up = 1.0f;
     if (RP > 0 && s.sink != nullptr) {                           // one more term of the denominator
         const float sk = __bfloat162float(s.sink[h]) * kLog2e, mx = fmaxf(m, sk);
         up = at::ex2(m - mx);
@@ -298,10 +305,11 @@ __global__ void __launch_bounds__(wt::kThreads, 2) window_attention_tc_kernel(co
     if (valid && *abort_s == 0) {
         __nv_bfloat16* dst = out + (size_t)(e.row0 + r0 + row) * ld_out + (size_t)h * s.Dv;
         const bool vec = (s.Dv & 7) == 0;                        // ld_out is a multiple of 8
-        if (RP > 0 && s.gate != nullptr && s.gate_heads) {
-            inv *= 1.0f / (1.0f + expf(-__bfloat162float(s.gate[(size_t)(e.row0 + r0 + row) * s.gate_ld + h])));
-        } else if (RP > 0 && s.gate != nullptr) {
-            const __nv_bfloat16* gt = s.gate + (size_t)(e.row0 + r0 + row) * s.gate_ld + (size_t)h * s.Dv;
+        const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(s.gate);
+        if ((RP > 0 || SIG) && gate != nullptr && s.gate_heads) {
+            inv *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)(e.row0 + r0 + row) * s.gate_ld + h])));
+        } else if (RP > 0 && gate != nullptr) {
+            const __nv_bfloat16* gt = gate + (size_t)(e.row0 + r0 + row) * s.gate_ld + (size_t)h * s.Dv;
 #pragma unroll
             for (int i = 0; i < C::HALF; i += 8) {
                 const int d = v0 + hf * C::HALF + i;

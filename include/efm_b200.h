@@ -374,17 +374,23 @@ EFM_API efm_status efm_b200_vit_encode(efm_b200_vit* vit, const void* pixels, in
  * sublayers, l<i>.norm1b / norm2b behind them; input norms: each with .alpha and .b, final.norm too), l<i>.mix.{q,k,v,o} with, as the layer asks, {q.b,k.b,v.b}, {q.norm,k.norm}, temp
  * (attention), l<i>.mix.{dq,dq.norm,uq,dkv,dkv.norm,uk,uv,o} with sink, g (latent attention) or
  * l<i>.mix.{r,k,v,g,a,a.b,w1,w2,w0,norm,o} (delta rule) or l<i>.mix.left.* (as attention) and
- * l<i>.mix.right.{q,k,v,g,norm,o} (parallel), l<i>.mlp.{up,down} with act (dense) or l<i>.mlp.router,
- * l<i>.mlp.e<j>.{gate,up,down} and, with a shared expert, l<i>.mlp.shared.{gate,up,down,sg} (experts),
- * l<i>.side.{gate,proj,norm}; bf16. */
-enum { EFM_MIXER_ATTENTION = 0, EFM_MIXER_GENERAL_DELTA = 1, EFM_MIXER_LATENT_ATTENTION = 2, EFM_MIXER_PARALLEL = 3 };
+ * l<i>.mix.right.{q,k,v,g,norm,o} (parallel) or l<i>.mix.{q,k,v,g,o} with, as the layer asks, norm and {a1,a2,a2.b} (linear
+ * attention), l<i>.mlp.{up,down} with act (dense) or l<i>.mlp.router, l<i>.mlp.e<j>.{gate,up,down} and, with a shared expert,
+ * l<i>.mlp.shared.{gate,up,down,sg} (experts; no gate where the unit has none), l<i>.side.{gate,proj,norm}, l<i>.canon1 / canon2
+ * (input convolutions, [width, taps]), l<i>.dwa (depth average, [i + 2]); attention with sigmoid weights has mix.pb, with an output
+ * bias mix.o.b, with a gate mix.g; bf16. */
+enum { EFM_MIXER_ATTENTION = 0, EFM_MIXER_GENERAL_DELTA = 1, EFM_MIXER_LATENT_ATTENTION = 2, EFM_MIXER_PARALLEL = 3, EFM_MIXER_LINEAR = 4 };
 enum { EFM_PAGE_TOKENS = 64 };
-enum { EFM_QK_NORM_WEIGHTED = 0, EFM_QK_NORM_PLAIN = 1, EFM_QK_NORM_NONE = 2 };   /* RMS norm of q and k per head, with / without a weight */
+/* RMS norm of q and k per head, with / without a weight; none; over all heads at once with a weight */
+enum { EFM_QK_NORM_WEIGHTED = 0, EFM_QK_NORM_PLAIN = 1, EFM_QK_NORM_NONE = 2, EFM_QK_NORM_ROW = 3 };
+enum { EFM_WEIGHTS_SOFTMAX = 0, EFM_WEIGHTS_SIGMOID = 1 };           /* attention: sigmoid(score + pb[h]), not normalised over the keys */
 enum { EFM_ROT_NONE = 0, EFM_ROT_HALF = 1, EFM_ROT_PAIRS = 2 };      /* channel i turns with i + dims / 2; 2 i with 2 i + 1 */
 enum { EFM_NORM_OUTPUT = 0, EFM_NORM_SANDWICH = 1, EFM_NORM_INPUT = 2 };
 enum { EFM_GATE_NONE = 0, EFM_GATE_CHANNELS = 1, EFM_GATE_HEADS = 2 };   /* sigmoid gate per output channel / per head */
 enum { EFM_ACT_POLYNORM = 0, EFM_ACT_RELU2 = 1 };                    /* dense feed-forward */
-enum { EFM_GLU_SILU = 0, EFM_GLU_CLAMPED = 1 };   /* experts: silu(g) u; g' sigmoid(1.702 g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit) */
+/* experts: silu(g) u; g' sigmoid(1.702 g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit); relu(u)^2, no gate */
+enum { EFM_GLU_SILU = 0, EFM_GLU_CLAMPED = 1, EFM_GLU_NONE_RELU2 = 2 };
+enum { EFM_SHARED_GATED = 0, EFM_SHARED_PLAIN = 1 };                 /* shared expert: output times sigmoid(W_sg h), or as it is */
 enum { EFM_SCORE_SOFTMAX = 0, EFM_SCORE_SIGMOID = 1 };               /* router scores */
 
 typedef struct efm_decoder_layer {
@@ -407,7 +413,7 @@ typedef struct efm_decoder_layer {
     float rot_base;               /* pair i of position p turns by p * rot_base^(-2 i / rot_dims) */
     int32_t q_rank, kv_rank;      /* latent: widths of the query latent and of the cached key / value latent (<= 1024) */
     int32_t sink;                 /* latent: 1 = a learned extra term exp(sink[h]) in the softmax denominator */
-    int32_t out_gate;             /* latent: EFM_GATE_* */
+    int32_t out_gate;             /* latent: EFM_GATE_*; attention: none or per head */
     int32_t experts;              /* routed feed-forward: number of experts (<= 512), 0: none */
     int32_t expert_ff;            /* width of an expert */
     int32_t expert_top;           /* experts a token uses (<= 32) */
@@ -428,6 +434,15 @@ typedef struct efm_decoder_layer {
     int32_t linear_heads, linear_dim, linear_vdim;    /* dims <= 256 */
     float mix_scale, linear_scale;                    /* multipliers of the two halves */
     const double* linear_decay;                       /* [linear_heads], read by efm_b200_decoder_create */
+    /* linear: the same sum alone, of q, k and v as projected (rot_kind turns q and k first), with one of the products q . k scaled by
+     * linear_dim^(-1/2); RMS norm per head, with a weight shared by the heads when linear_norm = 1; silu gate.  linear_tau > 0 replaces
+     * linear_decay: a decay per token and key channel, sigmoid(W_a2 W_a1 h + b)^(1 / linear_tau), W_a1 of decay_rank rows */
+    int32_t linear_norm;
+    float linear_tau;
+    int32_t score_weights;        /* attention: EFM_WEIGHTS_* */
+    int32_t out_bias;             /* attention: 1 = the output projection has a bias */
+    float expert_scale;           /* multiplier of the choices' weights; 0: 1 */
+    int32_t shared_gate;          /* EFM_SHARED_* */
 } efm_decoder_layer;
 
 typedef struct efm_decoder_desc {
@@ -448,6 +463,9 @@ typedef struct efm_decoder_desc {
     int32_t tied_head;            /* 1: the head is the embedding table */
     float logit_scale;            /* logits = logit_scale * head . x ... */
     float logit_softcap;          /* ... then softcap * tanh(logits / softcap); 0: off */
+    /* > 0: a sublayer reads h + sum_j w[:, j] h_(t - taps + 1 + j) instead of h, the stream (EFM_NORM_OUTPUT); <= 16 */
+    int32_t conv_taps;
+    int32_t depth_average;        /* 1: behind layer i the stream is the weighted sum of the embedding and the results of layers 0 .. i */
 } efm_decoder_desc;
 
 EFM_API efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decoder_layer* layers, int32_t device_id,

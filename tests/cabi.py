@@ -50,7 +50,8 @@ class DecoderLayer(C.Structure):
         [(n, C.c_float) for n in ("rot_factor", "rot_original", "rot_fast", "rot_slow")] + [("ff_act", C.c_int32), ("expert_glu", C.c_int32),
          ("expert_limit", C.c_float), ("expert_score", C.c_int32), ("expert_weight_input", C.c_int32), ("shared_ff", C.c_int32), ("shared_limit", C.c_float)] + \
         [(n, C.c_int32) for n in ("linear_heads", "linear_dim", "linear_vdim")] + [("mix_scale", C.c_float), ("linear_scale", C.c_float),
-         ("linear_decay", C.POINTER(C.c_double))]
+         ("linear_decay", C.POINTER(C.c_double)), ("linear_norm", C.c_int32), ("linear_tau", C.c_float), ("score_weights", C.c_int32), ("out_bias", C.c_int32),
+         ("expert_scale", C.c_float), ("shared_gate", C.c_int32)]
 
 
 class DecoderDesc(C.Structure):
@@ -58,7 +59,8 @@ class DecoderDesc(C.Structure):
         [("norm_eps", C.c_float)] + [(n, C.c_int32) for n in (
             "compute_dtype", "max_step_tokens", "max_response_tokens", "cache_pages", "state_slots", "max_slots",
             "norm_layout")] + [("embed_scale", C.c_float)] + [(n, C.c_int32) for n in ("loop_start", "loop_stop", "loop_times")] + \
-        [("residual_mult", C.c_float), ("tied_head", C.c_int32), ("logit_scale", C.c_float), ("logit_softcap", C.c_float)]
+        [("residual_mult", C.c_float), ("tied_head", C.c_int32), ("logit_scale", C.c_float), ("logit_softcap", C.c_float), ("conv_taps", C.c_int32),
+         ("depth_average", C.c_int32)]
 
 
 class StepEntry(C.Structure):
@@ -477,17 +479,20 @@ class VlaPolicy:
 
 
 class Decoder(Backend):
-    """A layered-decoder context described by a Folizen, Temuvik or Vekolix configuration dict; one mapped slot per call of map_slot."""
+    """A layered-decoder context described by a Folizen, Temuvik, Vekolix or Viladra configuration dict; one mapped slot per call of map_slot."""
 
     def __init__(self, config, *, decay_rank=64, cache_pages=64, state_slots=4, max_slots=4, max_step_tokens=2048,
                  max_response_tokens=512, dtype=EFM_BF16, device_id=0):
         self.L = lib()
         layers = (DecoderLayer * len(config["layers"]))()
-        temuvik, vekolix = (config["architecture"] == n for n in ("Temuvik", "Vekolix"))
+        temuvik, vekolix, viladra = (config["architecture"] == n for n in ("Temuvik", "Vekolix", "Viladra"))
         decays = []                                                   # read by decoder_create
         for e, l in zip(layers, config["layers"]):
             if vekolix:
                 self._vekolix_layer(e, l, decays)
+                continue
+            if viladra:
+                self._viladra_layer(e, l, decays, decay_rank)
                 continue
             m, mask = l["mixer"], l["mixer"].get("mask") or {}
             e.heads, e.dim, e.window = m["heads"], m["dim"], mask.get("size", 0)
@@ -512,8 +517,9 @@ class Decoder(Backend):
         d = DecoderDesc(C.sizeof(DecoderDesc), len(layers), config["vocab"], config["width"],
                         (config.get("token_side") or {}).get("dim", 0), config["norm"]["eps"], dtype, max_step_tokens,
                         max_response_tokens, cache_pages, state_slots, max_slots, 2 if vekolix else int(temuvik),
-                        config["embedding"]["scale"] if temuvik else 1.0, loop["start"], loop["stop"], loop["times"], config.get("residual_mult", 0.0),
-                        int(vekolix), config.get("logit_scale", 1.0), config.get("logit_softcap", 0.0))
+                        config["embedding"]["scale"] if temuvik or viladra else 1.0, loop["start"], loop["stop"], loop["times"], config.get("residual_mult", 0.0),
+                        int(vekolix or viladra), config.get("logit_scale", 1.0), config.get("logit_softcap", 0.0),
+                        config["canon"]["taps"] if viladra else 0, int(viladra))
         self.cfg = type("Cfg", (), {"vocab": config["vocab"], "mrope_section": None})()
         self.ctx = P()
         st = self.L.efm_b200_decoder_create(C.byref(d), layers, device_id, C.byref(self.ctx))
@@ -544,6 +550,27 @@ class Decoder(Backend):
             e.expert_groups = e.expert_groups_kept = e.expert_glu = e.expert_score = e.expert_weight_input = 1
             if mlp.get("shared"):
                 e.shared_ff, e.shared_limit = mlp["shared"]["ff"], mlp["shared"]["limit"]
+
+    @staticmethod
+    def _viladra_layer(e, l, decays, decay_rank):
+        m, mlp = l["mixer"], l["mlp"]
+        e.heads, e.dim, e.vdim = m["heads"], m["dim"], m["vdim"]
+        if l["type"] == "attention":
+            e.mixer, e.kv_heads, e.scale, e.window = 0, m["kv_heads"], m["scale"], (m.get("mask") or {}).get("size", 0)
+            e.qk_norm, e.qkv_bias, e.out_bias, e.score_weights, e.out_gate = 3, 1, 1, 1, 2
+        else:
+            e.mixer, e.linear_heads, e.linear_dim, e.linear_vdim = 4, m["heads"], m["dim"], m["vdim"]
+            if l["type"] == "retention":
+                e.rot_kind, e.rot_dims, e.rot_base = 1, m["rot"]["dims"], m["rot"]["base"]
+                decays.append((C.c_double * m["heads"])(*m["decay"]))
+                e.linear_decay = decays[-1]
+            else:
+                e.linear_norm, e.linear_tau, e.decay_rank = 1, m["tau"], decay_rank
+        if mlp:
+            r = mlp["router"]
+            e.experts, e.expert_ff, e.expert_top, e.expert_scale = r["experts"], mlp["expert"]["ff"], r["top"], r["scale"]
+            e.expert_groups = e.expert_groups_kept = e.shared_gate = 1
+            e.expert_glu, e.shared_ff = 2, (mlp.get("shared") or {"ff": 0})["ff"]
 
     def map_slot(self, slot, pages, state_slot):
         self.check(self.L.efm_b200_decoder_map_slot(self.ctx, slot, _i32_array(pages), len(pages), state_slot), "decoder_map_slot")

@@ -928,6 +928,7 @@ DESIGN_SIZES = {        # width, heads, kv heads (head dim 128), attention feed-
 DESIGN_LAYERS, DESIGN_WINDOW, DESIGN_PROMPT, DESIGN_DECODE, DESIGN_RANK = 8, 1024, 2048, 64, 64
 
 
+DESIGN_DECAY_RANK = 16
 DESIGN_EXPERTS = {"count": 32, "top": 4, "groups": 4, "keep": 2}
 
 
@@ -1025,6 +1026,39 @@ def vekolix_flops(cfg, n):
     return out
 
 
+def viladra_config(size):
+    """Retention, attention with sigmoid weights in a window and gated linear attention in turn, experts and a shared one everywhere."""
+    W, H, G, ff, V = DESIGN_SIZES[size]
+    e = DESIGN_EXPERTS
+    moe = {"kind": "moe", "expert": {"ff": ff // 8}, "router": {"experts": e["count"], "top": e["top"], "scale": 2.0}, "shared": {"ff": ff // 8}}
+    n = W // 128
+    ret = {"type": "retention", "mlp": moe, "mixer": {"heads": n, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-3.0 - 8.0 * h / n) for h in range(n)],
+                                                      "rot": {"base": 1e5, "dims": 128}}}
+    att = {"type": "attention", "mlp": moe, "mixer": {"heads": H, "kv_heads": G, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": DESIGN_WINDOW}}}
+    gla = {"type": "gla", "mlp": moe, "mixer": {"heads": n, "dim": 128, "vdim": 128, "tau": 16.0}}
+    return {"architecture": "Viladra", "width": W, "vocab": V, "norm": {"eps": 1e-5}, "canon": {"taps": 4}, "embedding": {"scale": 1.0}, "logit_softcap": 30.0,
+            "layers": [(ret, att, gla)[i % 3] for i in range(DESIGN_LAYERS)]}
+
+
+def viladra_flops(cfg, n):
+    """Matrix products (of the experts a token uses) plus visible attention pairs plus the recurrences (2 D Dv multiply-adds per token
+    and head), 2 per multiply-add."""
+    W, out = cfg["width"], 0
+    for l in cfg["layers"]:
+        m, mlp = l["mixer"], l["mlp"]
+        H, D, Dv = m["heads"], m["dim"], m["vdim"]
+        if l["type"] == "attention":
+            seen = sum(min(i + 1, m["mask"]["size"]) for i in range(n))
+            out += 2 * n * W * (H * (D + Dv) + m["kv_heads"] * (D + Dv) + H) + 2 * H * (D + Dv) * seen
+        else:
+            out += 2 * n * W * H * (2 * D + 3 * Dv) + 4 * n * H * D * Dv
+            if l["type"] == "gla":
+                out += 2 * n * DESIGN_DECAY_RANK * (W + H * D)
+        r = mlp["router"]
+        out += 2 * n * W * (r["experts"] + 2 * r["top"] * mlp["expert"]["ff"] + 2 * mlp["shared"]["ff"])
+    return out
+
+
 def time_model(be, slot, prompt, steps, warmup):
     """Median device times: prefill of the whole prompt (no sample), decode per token at that context (captured graph)."""
     pre, dec = [], []
@@ -1057,6 +1091,7 @@ def run_design(args):
     import folizen_util as fu
     import temuvik_util as tu
     import vekolix_util as vu
+    import viladra_util as vl
     from oracle import qwen_text, synth
     hbm, _ = peaks()
     tf, _ = tensor_peak()
@@ -1064,7 +1099,8 @@ def run_design(args):
     name_ = args.design.capitalize()
     design_config, design_flops, design_shapes = {"folizen": (folizen_config, folizen_flops, lambda cfg: fu.shapes(cfg, DESIGN_RANK)),
                                                   "temuvik": (temuvik_config, temuvik_flops, tu.shapes),
-                                                  "vekolix": (vekolix_config, vekolix_flops, vu.shapes)}[args.design]
+                                                  "vekolix": (vekolix_config, vekolix_flops, vu.shapes),
+                                                  "viladra": (viladra_config, viladra_flops, lambda cfg: vl.shapes(cfg, DESIGN_DECAY_RANK))}[args.design]
     out = {"metric": name_ + " prefill / decode throughput beside the text tower at equal size", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic",
            "config": {"layers": DESIGN_LAYERS, "prompt": DESIGN_PROMPT, "decode_steps": DESIGN_DECODE, "window": 0 if args.design == "vekolix" else DESIGN_WINDOW}, "sizes": {}}
     clocks.start()
@@ -1072,7 +1108,7 @@ def run_design(args):
         cfg = design_config(size)
         pages = (DESIGN_PROMPT + DESIGN_DECODE + 64) // 64
         g = torch.Generator(device="cuda").manual_seed(0)
-        be = cabi.Decoder(cfg, decay_rank=DESIGN_RANK, cache_pages=pages, state_slots=1, max_slots=1)
+        be = cabi.Decoder(cfg, decay_rank=DESIGN_DECAY_RANK if args.design == "viladra" else DESIGN_RANK, cache_pages=pages, state_slots=1, max_slots=1)
         shapes = design_shapes(cfg)
         n_weights = 0 if "head" in shapes else cfg["vocab"] * cfg["width"]        # a tied head counts like any other
         for name, shape in shapes.items():
@@ -1119,7 +1155,7 @@ def main():
     ap.add_argument("--config", type=int, default=None, choices=[0, 1, 2, 3, 4],
                     help="run one configuration alone; default: configuration 3 (tensor parallel over the ranks) plus, on one GPU, "
                          "a short pass over the other four")
-    ap.add_argument("--design", choices=["folizen", "temuvik", "vekolix"], default=None, help="layered decoder beside the text tower at equal size (one GPU)")
+    ap.add_argument("--design", choices=["folizen", "temuvik", "vekolix", "viladra"], default=None, help="layered decoder beside the text tower at equal size (one GPU)")
     ap.add_argument("--design-sizes", default="1024,2048,4096", help="comma-separated widths for --design")
     ap.add_argument("--tokens", type=int, default=0, help="override the number of generated tokens")
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")

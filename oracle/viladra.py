@@ -76,19 +76,15 @@ def silu(z: torch.Tensor) -> torch.Tensor:
     return z * torch.sigmoid(z)
 
 
-def sees(i: int, j: int, window: int) -> bool:
-    return 0 <= i - j and (window == 0 or i - j < window)
-
-
 def sigmoid_attention(q, k, v, scale: float, shift: torch.Tensor, window: int) -> torch.Tensor:
-    """Weights sigmoid(scale q . k + shift_h), not normalised.  q [T, H, D], k [T, G, D], v [T, G, Dv] -> [T, H, Dv]."""
+    """Weights sigmoid(scale q . k + shift_h), not normalised; i sees j with 0 <= i - j < window (0: every j <= i).  q [T, H, D], k [T, G, D], v [T, G, Dv] -> [T, H, Dv]."""
     T, H, G = q.shape[0], q.shape[1], k.shape[1]
     out = torch.zeros(T, H, v.shape[-1], dtype=q.dtype)
     for h in range(H):
         g = h // (H // G)
         for i in range(T):
-            js = [j for j in range(max(0, i - window + 1) if window else 0, i + 1) if sees(i, j, window)]
-            out[i, h] = torch.sigmoid((k[js, g] @ q[i, h]) * scale + shift[h]) @ v[js, g]
+            first = max(0, i - window + 1) if window else 0
+            out[i, h] = torch.sigmoid((k[first:i + 1, g] @ q[i, h]) * scale + shift[h]) @ v[first:i + 1, g]
     return out
 
 

@@ -2,9 +2,18 @@
 margin stands out.  Engine, steps and error measure are those of folizen_util."""
 from __future__ import annotations
 
+import numpy as np
 import torch
 
 from folizen_util import LIMIT, engine, error, run_portions, step, taps, tokens  # noqa: F401
+
+
+def row_errors(got, ref):
+    """folizen_util.error, row by row."""
+    d = np.asarray(got, dtype=np.float64) - ref
+    d -= d.mean(-1, keepdims=True)
+    scale = np.sqrt(((ref - ref.mean(-1, keepdims=True)) ** 2).mean())
+    return np.sqrt((d ** 2).mean(-1)) / scale
 
 
 def experts(n=8, top=2, ff=48, scale=1.5, shared=40):

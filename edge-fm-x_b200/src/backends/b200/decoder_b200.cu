@@ -318,7 +318,26 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
             n_lin = std::max(n_lin, decoder_linear_ws_floats(l, S, std::min(desc->max_slots, S)));
             w_lin = std::max(w_lin, (size_t)l.linear_v());
             w_in = std::max(w_in, (size_t)l.in.Np);
-            if (d.rot_kind != EFM_ROT_NONE && !m->f32) w_proj_f = std::max(w_proj_f, (size_t)l.in.Np);
+            if (d.rot_kind != EFM_ROT_NONE && !m->f32) {
+                if (d.linear_dim % 32 == 0 && d.rot_dims % 32 == 0) {
+                    for (size_t k = 0; k < m->rot_tables.size() && l.rot_table < 0; ++k) {
+                        const efm_decoder_layer& o = layers[m->rot_tables[k].layer];
+                        if (o.rot_dims == d.rot_dims && o.rot_base == d.rot_base && o.rot_factor == d.rot_factor && o.rot_original == d.rot_original &&
+                            o.rot_fast == d.rot_fast && o.rot_slow == d.rot_slow)
+                            l.rot_table = (int)k;
+                    }
+                    if (l.rot_table < 0) {
+                        DecoderModel::RotTable t;
+                        t.dims = d.rot_dims;
+                        t.layer = i;
+                        EFM_TRY(dev_alloc(c, &t.cs, (size_t)S * (d.rot_dims / 2)));
+                        l.rot_table = (int)m->rot_tables.size();
+                        m->rot_tables.push_back(t);
+                    }
+                } else {
+                    w_proj_f = std::max(w_proj_f, (size_t)l.in.Np);
+                }
+            }
         } else {
             any_delta = true;
             const int HD = d.heads * d.dim;
@@ -806,7 +825,8 @@ namespace {
 // ---- weights -------------------------------------------------------------------------------------------------------
 // Rows [src, src + n) of a tensor become rows [dst, dst + n) of a (fused, padded) linear, from column `col` on.  Several tensors may
 // be parts of one linear.
-struct Piece { int dst, src, n, col = 0; };
+// step: destination rows from one to the next.
+struct Piece { int dst, src, n, col = 0, step = 1; };
 
 efm_status put_rows(efm_b200_ctx* c, const DecLinear& w, const std::vector<Piece>& pieces, const void* data, const std::string& name, const int64_t* shape,
                     int ndim, int mem_kind, int cols) {
@@ -815,7 +835,7 @@ efm_status put_rows(efm_b200_ctx* c, const DecLinear& w, const std::vector<Piece
     for (const Piece& p : pieces) rows += p.n;
     if (!shape_is(shape, ndim, rows, K)) return fail(c, EFM_ERR_INVALID_ARGUMENT, "unexpected shape for " + name);
     for (const Piece& p : pieces)
-        EFM_CK(c, cudaMemcpy2DAsync(w.w + (size_t)p.dst * w.Kp + p.col, (size_t)w.Kp * 2, static_cast<const char*>(data) + (size_t)p.src * K * 2, (size_t)K * 2,
+        EFM_CK(c, cudaMemcpy2DAsync(w.w + (size_t)p.dst * w.Kp + p.col, (size_t)w.Kp * 2 * p.step, static_cast<const char*>(data) + (size_t)p.src * K * 2, (size_t)K * 2,
                                     (size_t)K * 2, (size_t)p.n, mem_kind == EFM_MEM_DEVICE ? cudaMemcpyDeviceToDevice : cudaMemcpyHostToDevice, c->stream));
     return EFM_OK;
 }
@@ -878,8 +898,21 @@ bool layer_target(DecoderModel& m, DecoderLayer& l, int index, const std::string
     if (rest == "mix.o.b") return vec(l.out.bias, m.W);
     if (l.alone()) {
         const int qk = d.linear_heads * d.linear_dim, v = d.linear_heads * d.linear_vdim, g = 2 * l.linear_qk() + l.linear_v();
-        if (rest == "mix.q") return lin(l.in, 0, qk);
-        if (rest == "mix.k") return lin(l.in, l.linear_qk(), qk);
+        // channels that turn with each other become neighbours: q and k alike, so that their products stay what they are
+        auto turned = [&](int row0) {
+            const int half = d.rot_kind == EFM_ROT_HALF ? d.rot_dims / 2 : 0, D = d.linear_dim;
+            t->lin = &l.in;
+            for (int h = 0; h < d.linear_heads; ++h) {
+                if (half > 0) {
+                    t->pieces.push_back(Piece{row0 + h * D, h * D, half, 0, 2});
+                    t->pieces.push_back(Piece{row0 + h * D + 1, h * D + half, half, 0, 2});
+                }
+                if (D > 2 * half) t->pieces.push_back(Piece{row0 + h * D + 2 * half, h * D + 2 * half, D - 2 * half});
+            }
+            return true;
+        };
+        if (rest == "mix.q") return turned(0);
+        if (rest == "mix.k") return turned(l.linear_qk());
         if (rest == "mix.v") return lin(l.in, 2 * l.linear_qk(), v);
         if (rest == "mix.g") return lin(l.in, g, v);
         if (rest == "mix.norm") return vec(l.mix_norm, d.linear_vdim);

@@ -69,8 +69,9 @@ void launch_gemv_ext(efm_b200_ctx& c, Launcher& L, const GemvParams& p) {
     const int level = c.decoder->gemv_level();
     auto run = [&](auto kernel) { L.launch(kernel, dim3(grid), dim3(kGemvThreads), smem, p, ks); };
     if constexpr (EPI == Epi::Router) {
+        if (level == 4) { run(gemv_kernel<EPI, 4>); return; }          // holds its dependents back itself
         InOrder serial(L);
-        run(level == 4 ? gemv_kernel<EPI, 4> : level == 3 ? gemv_kernel<EPI, 3> : gemv_kernel<EPI, 2>);
+        run(level == 3 ? gemv_kernel<EPI, 3> : gemv_kernel<EPI, 2>);
     } else if constexpr (kExperts) run(level == 4 ? gemv_kernel<EPI, 4> : level == 3 ? gemv_kernel<EPI, 3> : gemv_kernel<EPI, 2>);
     else if constexpr (EPI == Epi::Store32Bias) run(level == 4 ? gemv_kernel<EPI, 4> : gemv_kernel<EPI, 2>);
     else if constexpr (EPI == Epi::TokenGate) run(gemv_kernel<EPI, 1>);
@@ -159,6 +160,7 @@ LinearShape linear_shape(const DecoderModel& m, const DecoderLayer& l) {
     if (l.alone()) {
         s.scale = 1.0f / std::sqrt((float)s.D);
         s.rot = rot_shape(l);
+        if (s.rot.kind == kRotHalf) s.rot.kind = kRotPairs;            // the weights' rows are laid out so
         if (l.channel_decay()) {
             s.rank = l.d.decay_rank; s.off_a = s.off_g + v; s.inv_tau = 1.0f / l.d.linear_tau;
             s.a2 = l.w2.w; s.a2_bias = l.w2.bias; s.ld_a2 = l.w2.Kp;
@@ -675,7 +677,15 @@ void linear_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const Deco
         L.launch(linear_output_rows_kernel<TA>, dim3(plan.rows), dim3(256), 0, (const float*)m.o, ld_o, proj, static_cast<TA*>(m.mix) + l.lin_mix, l.mix_wp,
                  l.mix_wp - l.lin_mix, s);
     };
-    if (s.rank > 0) {                                                  // W_a2 W_a1 x + b, then the decays it stands for
+    auto decay_product = [&](auto rank) {
+        constexpr int RANK = decltype(rank)::value;
+        L.launch(linear_decay_product_sums_kernel<kLinearChunkTc, RANK>, dim3((ld_sums + 63) / 64, chunks), dim3(256), 0, reinterpret_cast<const __nv_bfloat16*>(proj),
+                 m.decay, ld_sums, s, plan);
+    };
+    if (s.rank > 0 && s.rank <= 32 && tensor_cores) {
+        if (s.rank <= 16) decay_product(std::integral_constant<int, 16>{});
+        else decay_product(std::integral_constant<int, 32>{});
+    } else if (s.rank > 0) {                                           // W_a2 W_a1 x + b, then the decays it stands for
         if (m.f32) {
             L.launch(gemm_f32_kernel, dim3((l.w2.Np + 63) / 64, (plan.rows + 63) / 64), dim3(256), 0, reinterpret_cast<const float*>(proj) + s.off_a, s.ld,
                      (const __nv_bfloat16*)l.w2.w, l.w2.Kp, m.decay, l.w2.Np, plan.rows, l.w2.Np, l.w2.Kp, (const __nv_bfloat16*)l.w2.bias, RowGroups{});
@@ -701,7 +711,7 @@ void linear_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const Deco
                 if (s.rank > 0) {
                     L.launch(linear_chunk_tc_kernel<VP, true>, grid, block, Cf::CHUNK_SMEM, proj, m.lin_ws, s, plan, &c.state->error, sums, ld_sums);
                     chain(linear_chain_rows_kernel<kLinearChunkTc, true>);
-                    L.launch(whole ? linear_attend_ch_tc_kernel<VP, true> : linear_attend_ch_tc_kernel<VP, false>, grid, block, Cf::ATTEND_CH_SMEM, proj, ws, sums, ld_sums,
+                    L.launch(whole ? linear_attend_ch_tc_kernel<VP, true> : linear_attend_ch_tc_kernel<VP, false>, grid, dim3(lt::kChThreads), Cf::ATTEND_CH_SMEM, proj, ws, sums, ld_sums,
                              m.o, ld_o, out, l.mix_wp, s, plan, &c.state->error);
                 } else {
                     L.launch(linear_chunk_tc_kernel<VP>, grid, block, Cf::CHUNK_SMEM, proj, m.lin_ws, s, plan, &c.state->error, sums, 0);
@@ -756,6 +766,13 @@ void linear_mixer_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, cons
     const LinearShape s = linear_shape(m, l);
     if (s.rot.kind == kRotNone) {
         linear_act(c, L, l.in, x, m.proj_a, plan.rows);
+    } else if (l.rot_table >= 0) {                                     // turned in the product's epilogue
+        GemmParams g{static_cast<const __nv_bfloat16*>(x), l.in.w, l.in.bias, static_cast<__nv_bfloat16*>(m.proj_a), nullptr, plan.rows, l.in.Np, l.in.Kp};
+        g.rot = m.rot_tables[l.rot_table].cs;
+        g.rot_cols = s.off_v;
+        g.rot_head = s.D;
+        g.rot_dims = s.rot.dims;
+        launch_gemm_epi(L, GemmEpi::Bf16Rotate, g, &c.state->error);
     } else {                                                           // turned in fp32, rounded once
         float* proj = std::is_same<TA, float>::value ? static_cast<float*>(m.proj_a) : m.proj_f;
         linear_f32(c, L, l.in, x, proj, plan.rows);
@@ -961,13 +978,14 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
     auto convolve = [&](const __nv_bfloat16* w, size_t off) {
         if (w == nullptr) return;
         auto run = [&](auto kernel) {
-            L.launch(kernel, dim3((m.Wp / 4 + 127) / 128, max_chunks(plan, kConvRows)), dim3(128), 0, stream, w, xa, m.Wp, m.state_pool, m.state_stride, off, m.d.conv_taps, plan);
+            const int rows = m.d.conv_taps >= 2 && m.d.conv_taps <= 4 ? kConvShortRows : kConvRows;
+            L.launch(kernel, dim3((m.Wp / 4 + 127) / 128, max_chunks(plan, rows)), dim3(128), 0, stream, w, xa, m.Wp, m.state_pool, m.state_stride, off, m.d.conv_taps, plan);
         };
         switch (m.d.conv_taps) {
-            case 2: run(input_conv_rows_kernel<TA, 2>); break;
-            case 3: run(input_conv_rows_kernel<TA, 3>); break;
-            case 4: run(input_conv_rows_kernel<TA, 4>); break;
-            default: run(input_conv_rows_kernel<TA, 0>); break;
+            case 2: run(input_conv_rows_kernel<TA, 2, kConvShortRows>); break;
+            case 3: run(input_conv_rows_kernel<TA, 3, kConvShortRows>); break;
+            case 4: run(input_conv_rows_kernel<TA, 4, kConvShortRows>); break;
+            default: run(input_conv_rows_kernel<TA, 0, kConvRows>); break;
         }
     };
     // a sublayer's last product and what follows it; elementwise norms are part of the product
@@ -982,6 +1000,8 @@ void rows_pass(efm_b200_ctx& c, const RowPlan& plan, const int32_t* ids, const R
         linear_f32(c, L, w, a, m.y, T);
         add_norm(m.y, post, norm, SumOf<TA>{}, avg);
     };
+    for (const DecoderModel::RotTable& t : m.rot_tables)
+        L.launch(rot_rows_kernel, dim3((t.dims / 2 + 127) / 128, T), dim3(128), 0, t.cs, rot_shape(m.layers[t.layer]), plan);
     float* first = m.d.depth_average ? m.hist : c.resid;
     launch_embed_rows(L, ids, c.embed, nullptr, first, T, c.d.vocab, m.Wp, -1, 0, m.d.embed_scale);
     stream = first;

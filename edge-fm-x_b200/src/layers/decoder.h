@@ -52,6 +52,7 @@ struct DecoderLayer {
     __nv_bfloat16* dwa = nullptr;         // average over depth, [layer + 2]
     // linear attention, alone or beside attention
     int lin_in = 0, lin_mix = 0;          // its first column in the projections and in the mixer output
+    int rot_table = -1;                   // alone: its table among those of a pass (bf16), or none
     int lin_vp = 0;                       // value channels padded to 4 (state rows)
     float* lin_powers = nullptr;          // [linear_heads][kLinearPowers + 1]
     bool parallel() const { return d.mixer == EFM_MIXER_PARALLEL; }
@@ -106,6 +107,9 @@ struct DecoderModel {
     // latent attention, long entries: visible cache rows and what they expand to
     __nv_bfloat16 *ws_c = nullptr, *ws_kv = nullptr;
     int ws_pages = 0, ws_window = 0;      // capacity (0: no layer uses it); largest window of the layers that use it (0: no window)
+    // (cos, sin) of a pass's rows, one table for all layers that turn alike
+    struct RotTable { int dims = 0, layer = 0; float2* cs = nullptr; };
+    std::vector<RotTable> rot_tables;
     float* lin_ws = nullptr;              // linear attention: states of a pass's chunks
     float* hist = nullptr;                // average over depth: the embedding and every layer's result, [layers + 1][rows][Wp]
     float *d_hist = nullptr, *d_avg = nullptr;            // the same of one row; the sum behind the current layer without its own result

@@ -92,7 +92,7 @@ static void launch_gemm(Launcher& L, const GemmParams& p, int* error_word = null
     // Few output tiles and a long K: split K so that the whole GPU works, fp32 partials to the workspace, then
     // a fixed-order sum with the epilogue.
     if constexpr (EPI == GemmEpi::Bf16Bias || EPI == GemmEpi::Residual || EPI == GemmEpi::F32 || EPI == GemmEpi::Bf16Relu2 || EPI == GemmEpi::Bf16Silu ||
-                  EPI == GemmEpi::ResidualTanh || gemm_is_glu(EPI)) {
+                  EPI == GemmEpi::Bf16Rotate || EPI == GemmEpi::ResidualTanh || gemm_is_glu(EPI)) {
         const int KB = (p.K + tc::BK - 1) / tc::BK;
         int splits = std::min(L.num_sms / std::max(1, tiles), KB / min_kb_per_split());
         if (L.gemm_ws != nullptr && splits >= 2 && (p.N & 3) == 0 && (!gemm_is_glu(EPI) || (p.N & 127) == 0) &&
@@ -121,7 +121,8 @@ static void launch_gemm(Launcher& L, const GemmParams& p, int* error_word = null
     // they are; the remaining tiles are cut along K into as many slices as fill the GPU once (compact fp32 slots in
     // the workspace) and a small kernel sums the slices in order with the epilogue.  Worth it only when a tile's K
     // loop is long against the two extra launches (about 12 us).
-    if constexpr (EPI == GemmEpi::Bf16Bias || EPI == GemmEpi::Residual || EPI == GemmEpi::F32 || EPI == GemmEpi::Bf16Silu || EPI == GemmEpi::ResidualTanh) {
+    if constexpr (EPI == GemmEpi::Bf16Bias || EPI == GemmEpi::Residual || EPI == GemmEpi::F32 || EPI == GemmEpi::Bf16Silu || EPI == GemmEpi::Bf16Rotate ||
+                  EPI == GemmEpi::ResidualTanh) {
         const int P = L.num_sms, rounds = tiles / P, rem = tiles % P;
         const int KB = (p.K + tc::BK - 1) / tc::BK;
         if (tail_split_enabled() && L.gemm_ws != nullptr && rounds >= 1 && rem > 0 && rem * 2 <= P && (p.N & 3) == 0 && p.kb_per_split == 0 &&
@@ -186,6 +187,7 @@ void launch_gemm_epi(Launcher& L, GemmEpi epi, const GemmParams& p, int* error_w
         case GemmEpi::SwiGlu: launch_gemm<GemmEpi::SwiGlu>(L, p, error_word); break;
         case GemmEpi::Bf16Relu2: launch_gemm<GemmEpi::Bf16Relu2>(L, p, error_word); break;
         case GemmEpi::Bf16Silu: launch_gemm<GemmEpi::Bf16Silu>(L, p, error_word); break;
+        case GemmEpi::Bf16Rotate: launch_gemm<GemmEpi::Bf16Rotate>(L, p, error_word); break;
         case GemmEpi::ResidualTanh: launch_gemm<GemmEpi::ResidualTanh>(L, p, error_word); break;
         case GemmEpi::ClampGlu: launch_gemm<GemmEpi::ClampGlu>(L, p, error_word); break;
     }

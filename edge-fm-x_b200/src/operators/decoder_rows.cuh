@@ -137,20 +137,25 @@ __global__ void __launch_bounds__(256) add_norm_rows_kernel(float* x, const floa
 
 // Input convolution: out = x + sum_back w[taps - 1 - back] x_{t - back}, w [taps][ld]; rows before the pass come from the sequence's
 // ring [taps][ld] (position modulo taps), which the thread with an entry's first rows brings up to date.  Grid (parts of a row, chunks of
-// kConvRows rows); a thread has four channels.  taps - 1 <= kConvRows.
-template <typename T, int TAPS>
+// ROWS rows); a thread has four channels.  taps - 1 <= ROWS.
+template <typename T, int TAPS, int ROWS>
 __global__ void __launch_bounds__(128) input_conv_rows_kernel(const float* __restrict__ x, const __nv_bfloat16* __restrict__ w, T* __restrict__ out, int ld,
                                                               float* __restrict__ pool, size_t slot_stride, size_t offset, int taps_any, const RowPlan plan) {
     constexpr int MAXT = TAPS > 0 ? TAPS : kMaxConvTaps;
     const int taps = TAPS > 0 ? TAPS : taps_any, c = 4 * (blockIdx.x * 128 + threadIdx.x);
     RowEntry e;
     int t0;
-    if (!locate_chunk<kConvRows>(plan, blockIdx.y, e, t0) || c >= ld) return;
-    const int n = min(kConvRows, e.n - t0);
+    if (!locate_chunk<ROWS>(plan, blockIdx.y, e, t0) || c >= ld) return;
+    const int n = min(ROWS, e.n - t0);
     float* ring = pool + (size_t)e.state * slot_stride + offset + c;
     const float* src = x + (size_t)(e.row0 + t0) * ld + c;
     T* dst = out + (size_t)(e.row0 + t0) * ld + c;
-    float4 past[MAXT], k[MAXT];                                        // past[b]: the value b + 1 tokens back
+    float4 past[MAXT], k[MAXT], now[TAPS > 0 ? ROWS : 1];              // past[b]: the value b + 1 tokens back
+    if constexpr (TAPS > 0) {
+#pragma unroll
+        for (int r = 0; r < ROWS; ++r)
+            if (r < n) now[r] = load4(src + (size_t)r * ld);
+    }
 #pragma unroll
     for (int b = 0; b < MAXT; ++b) {
         past[b] = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -159,9 +164,9 @@ __global__ void __launch_bounds__(128) input_conv_rows_kernel(const float* __res
         if (b + 1 < taps && e.pos0 + t >= 0) past[b] = t >= 0 ? load4(src - (size_t)(b + 1) * ld) : load4(ring + (size_t)((e.pos0 + t) % taps) * ld);
     }
 #pragma unroll
-    for (int r = 0; r < kConvRows; ++r) {
+    for (int r = 0; r < ROWS; ++r) {
         if (r >= n) break;
-        const float4 v = load4(src + (size_t)r * ld);
+        const float4 v = TAPS > 0 ? now[TAPS > 0 ? r : 0] : load4(src + (size_t)r * ld);
         float4 a = make_float4(fmaf(k[0].x, v.x, v.x), fmaf(k[0].y, v.y, v.y), fmaf(k[0].z, v.z, v.z), fmaf(k[0].w, v.w, v.w));
 #pragma unroll
         for (int b = 0; b + 1 < MAXT; ++b)

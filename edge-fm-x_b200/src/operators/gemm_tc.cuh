@@ -14,7 +14,7 @@
 //               longer than its MMAs whenever K was short):
 //               tcgen05.ld (row = TMEM lane, 32 columns at a time), bias / activation, staging through
 //               shared memory (XOR-swizzled 16-byte columns) so that global rows are written as contiguous segments:
-//               bf16 (+bias, optionally erf-GELU, tanh-GELU, squared ReLU or silu of a column range) | fp32 residual add | fp32 | a gated unit in bf16 |
+//               bf16 (+bias, optionally erf-GELU, tanh-GELU, squared ReLU, silu or rotary positions of a column range) | fp32 residual add | fp32 | a gated unit in bf16 |
 //               fp32 residual add of a multiple and, in bf16, the elementwise norm tanh(alpha x) w + b of the new residual.
 // Rows past M and columns past N are zero-filled by TMA on load and masked on store.
 // Every mbarrier wait is bounded; a wait that gives up raises *error, all roles leave their loops, the
@@ -26,7 +26,7 @@
 
 namespace efm {
 
-enum class GemmEpi : int { Bf16Bias = 0, Residual = 1, F32 = 2, Bf16Gelu = 3, SwiGlu = 4, Bf16GeluTanh = 5, Bf16Relu2 = 6, ClampGlu = 7, Bf16Silu = 8, ResidualTanh = 9 };
+enum class GemmEpi : int { Bf16Bias = 0, Residual = 1, F32 = 2, Bf16Gelu = 3, SwiGlu = 4, Bf16GeluTanh = 5, Bf16Relu2 = 6, ClampGlu = 7, Bf16Silu = 8, ResidualTanh = 9, Bf16Rotate = 10 };
 
 struct GroupTile { int32_t group, first, count, pad; };      // row tile: its group, the group's first row tile and number of them
 
@@ -55,6 +55,10 @@ struct GemmParams {
     float mult = 1.f;
     const __nv_bfloat16 *norm_w = nullptr, *norm_b = nullptr, *norm_alpha = nullptr;
     int silu0 = 0, silu1 = 0; // Bf16Silu: columns [silu0, silu1) become silu of themselves
+    // Bf16Rotate: columns [0, rot_cols) are heads of rot_head channels, of which the first rot_dims turn in neighbouring pairs by the row's
+    // (cos, sin) of the pair, rot [M][rot_dims / 2]; rot_head and rot_dims are multiples of 32
+    const float2* rot = nullptr;
+    int rot_cols = 0, rot_head = 32, rot_dims = 0;
 };
 
 // Gated units over a fused gate|up weight: half as many output columns.
@@ -70,6 +74,13 @@ __device__ __forceinline__ float gemm_glu(float g, float u, float limit) {
     return __fdividef(g, 1.0f + __expf(-g)) * u;
 }
 
+// four columns from n on of row m
+__device__ __forceinline__ float4 gemm_rotate(float4 a, int m, int n, const GemmParams& p) {
+    const int d = n % p.rot_head;
+    if (n >= p.rot_cols || d >= p.rot_dims) return a;
+    const float4 r = *reinterpret_cast<const float4*>(p.rot + (size_t)m * (p.rot_dims / 2) + d / 2);
+    return make_float4(a.x * r.x - a.y * r.y, a.y * r.x + a.x * r.y, a.z * r.z - a.w * r.w, a.w * r.z + a.z * r.w);
+}
 __device__ __forceinline__ float4 gemm_silu_range(float4 a, int n, const GemmParams& p) {
     float f[4] = {a.x, a.y, a.z, a.w};
 #pragma unroll
@@ -381,6 +392,16 @@ __global__ void __launch_bounds__(tc::kThreads) gemm_tc_kernel(const __grid_cons
                         }
                     }
                 }
+                if constexpr (EPI == GemmEpi::Bf16Rotate) {                    // the chunk lies in one head, in its turned part or behind
+                    const int n = n0 + c0, m = m0 + q * 32 + lane;
+                    if (n < p.rot_cols && n % p.rot_head < p.rot_dims && m < p.M) {
+#pragma unroll
+                        for (int e = 0; e < 32; e += 4) {
+                            const float4 v = gemm_rotate(make_float4(o[e], o[e + 1], o[e + 2], o[e + 3]), m, n + e, p);
+                            o[e] = v.x; o[e + 1] = v.y; o[e + 2] = v.z; o[e + 3] = v.w;
+                        }
+                    }
+                }
                 __syncwarp();                                                  // previous chunk fully written out
 #pragma unroll
                 for (int e = 0; e < 32; e += 4)
@@ -493,6 +514,7 @@ __global__ void __launch_bounds__(256) gemm_splitk_finish_kernel(const float* __
             gemm_residual_tanh(p, gemm_norm(p, n), *reinterpret_cast<const float4*>(p.Cf + i * 4), a, i * 4);
         } else {
             if constexpr (EPI == GemmEpi::Bf16Silu) a = gemm_silu_range(a, n, p);
+            if constexpr (EPI == GemmEpi::Bf16Rotate) a = gemm_rotate(a, (int)((i * 4) / (size_t)p.N), n, p);
             if constexpr (EPI == GemmEpi::Bf16Relu2) {
                 a.x = fmaxf(a.x, 0.f); a.y = fmaxf(a.y, 0.f); a.z = fmaxf(a.z, 0.f); a.w = fmaxf(a.w, 0.f);
                 a.x *= a.x; a.y *= a.y; a.z *= a.z; a.w *= a.w;
@@ -536,6 +558,7 @@ __global__ void __launch_bounds__(256) gemm_tail_finish_kernel(const float* __re
             gemm_residual_tanh(p, gemm_norm(p, n), *reinterpret_cast<const float4*>(p.Cf + off), a, off);
         } else {
             if constexpr (EPI == GemmEpi::Bf16Silu) a = gemm_silu_range(a, n, p);
+            if constexpr (EPI == GemmEpi::Bf16Rotate) a = gemm_rotate(a, m, n, p);
             *reinterpret_cast<uint2*>(p.C + off) = make_uint2(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w));
         }
     }

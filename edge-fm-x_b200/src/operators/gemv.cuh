@@ -929,8 +929,9 @@ __global__ void __launch_bounds__(kGemvThreads, 1) gemv_kernel(const GemvParams 
     // Let the next kernel of the step start its own weight prefetch as soon as every block of this
     // one is resident, then prefetch (independent of every earlier kernel), then wait.
     // ExpertUp holds its dependents back until its own wait is over: the choice it waits for is then there for ExpertDown,
-    // which fetches its first weights before its wait.
-    if constexpr (EPI != Epi::ExpertUp) pdl_launch_dependents();
+    // which fetches its first weights before its wait.  So does the router of level 4, whose dependents would only fill the SMs.
+    constexpr bool kHold = EPI == Epi::ExpertUp || (EPI == Epi::Router && EXT > 3);
+    if constexpr (!kHold) pdl_launch_dependents();
     const GemvSched sc = gemv_sched(p, ks, blockIdx.x, gridDim.x);
     __shared__ int early_s[EPI == Epi::ExpertDown ? 2 * kMaxExpertTop + 1 : 1];  // ids | weights (and that of the shared expert)
     if constexpr (EPI == Epi::ExpertDown) {
@@ -944,7 +945,7 @@ __global__ void __launch_bounds__(kGemvThreads, 1) gemv_kernel(const GemvParams 
     }
     gemv_prefetch<EPI, EXT>(p, sc, regs, gemv_smem, xbytes);
     pdl_wait();
-    if constexpr (EPI == Epi::ExpertUp) pdl_launch_dependents();
+    if constexpr (kHold) pdl_launch_dependents();
     if constexpr (EPI == Epi::Peers) best_i = (int)(__ldcg(p.epoch) + 1u);      // this launch's exchange count rides in best_i
     gemv_run<EPI, EXT>(p, sc, regs, gemv_smem, xbytes, best_v, best_i, EPI == Epi::ExpertDown ? early_s : nullptr);
     if constexpr (EPI == Epi::Router) {

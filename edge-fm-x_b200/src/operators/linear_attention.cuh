@@ -16,7 +16,8 @@
 // (with a weight shared by the heads, or none) and multiplied by silu of the gate.  Its decay is the constant of the head or, from the
 // projections, one number per token and key channel (`rank` > 0):
 //   S_t = diag(alpha_t) S_{t-1} + k_t v_t^T,   alpha_t = sigmoid(W_a2 W_a1 x + b)^(1 / tau)
-//   linear_rotate_rows       q and k of every row turned, everything rounded once
+//   linear_rotate_rows       q and k of every row turned, everything rounded once (32-bit mode, and head sizes that the epilogue of the
+//                            projections' product, gemm_tc.cuh, does not take); the pairs are neighbours, the weights' rows are laid out so
 //   linear_decay_rows        alpha of every row, or (chunks on the tensor cores) sums of log alpha from the chunk's first token on
 //   linear_scan_rows         channel decays token by token: 32-bit mode, short passes and heads the tensor-core form does not take
 //   linear_head_output_rows  scale, norm per head, weight, gate
@@ -362,11 +363,21 @@ __global__ void __launch_bounds__(256, 5) linear_output_rows_kernel(const float*
 // log of alpha; the product z / tau is what matters when z is far below zero
 __device__ __forceinline__ float log_decay(float z, float inv_tau) { return (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau; }
 
+// (cos, sin) of every pair of every row of a pass.  Grid (parts of a row, rows)
+__global__ void __launch_bounds__(128) rot_rows_kernel(float2* __restrict__ out, const RotShape r, const RowPlan plan) {
+    const int i = blockIdx.x * 128 + threadIdx.x, row = blockIdx.y;
+    if (i >= r.dims / 2) return;
+    const RowEntry e = plan.of_row(row);
+    float2 v;
+    rot_sincos(r, e.pos0 + row - e.row0, i, &v.y, &v.x);
+    out[(size_t)row * (r.dims / 2) + i] = v;
+}
+
 // proj -> out with q and k turned; in 32-bit mode both may be the same rows.  One block per row; ld % 8 == 0, dims % 2 == 0.
 template <typename T>
 __global__ void __launch_bounds__(256) linear_rotate_rows_kernel(const float* proj, T* out, const LinearShape s, const RowPlan plan) {
     __shared__ float cs[kRotMaxPairs], sn[kRotMaxPairs];
-    const int row = blockIdx.x, half = s.rot.dims / 2, step = s.rot.kind == kRotHalf ? half : 1;
+    const int row = blockIdx.x, half = s.rot.dims / 2;
     const RowEntry e = plan.of_row(row);
     rot_table(s.rot, e.pos0 + row - e.row0, cs, sn);
     __syncthreads();
@@ -375,10 +386,10 @@ __global__ void __launch_bounds__(256) linear_rotate_rows_kernel(const float* pr
     auto put = [](T* p, float v) { if constexpr (sizeof(T) == 2) *p = __float2bfloat16_rn(v); else *p = v; };
     for (int i = threadIdx.x; i < 2 * s.heads * half; i += 256) {
         const int u = i / half, pair = i - u * half;                    // a head of q, then of k
-        const int c = (u < s.heads ? s.off_q + u * s.D : s.off_k + (u - s.heads) * s.D) + (s.rot.kind == kRotHalf ? pair : 2 * pair);
-        const float a = src[c], b = src[c + step];
+        const int c = (u < s.heads ? s.off_q + u * s.D : s.off_k + (u - s.heads) * s.D) + 2 * pair;
+        const float a = src[c], b = src[c + 1];
         put(dst + c, a * cs[pair] - b * sn[pair]);
-        put(dst + c + step, b * cs[pair] + a * sn[pair]);
+        put(dst + c + 1, b * cs[pair] + a * sn[pair]);
     }
     if constexpr (sizeof(T) == 2) {                                     // everything else
         const int rest = s.D - s.rot.dims;
@@ -421,6 +432,66 @@ __global__ void __launch_bounds__(128) linear_decay_sums_kernel(float* __restric
                 p[(size_t)(r0 + i) * ld] = sum;
             }
     }
+}
+
+// the same without branches; the logarithm of 1 + e as a series in e / (2 + e), at most 1/3
+__device__ __forceinline__ float log_decay_fast(float z, float inv_tau) {
+    const float e = __expf(-fabsf(z)), q = __fdividef(e, 2.0f + e), q2 = q * q;
+    const float l = 2.0f * q * fmaf(q2, fmaf(q2, fmaf(q2, fmaf(q2, fmaf(q2, 1.0f / 11.0f, 1.0f / 9.0f), 1.0f / 7.0f), 0.2f), 1.0f / 3.0f), 1.0f);
+    return (fminf(z, 0.f) - l) * inv_tau;
+}
+// linear_decay_sums with the product W_a2 (W_a1 x) + b in front of it, W_a1 x of at most RANK bf16 numbers a row.  Grid (64 channels, chunks
+// of C tokens): four threads a channel, a quarter of the chunk each.
+template <int C, int RANK>
+__global__ void __launch_bounds__(256) linear_decay_product_sums_kernel(const __nv_bfloat16* __restrict__ proj, float* __restrict__ sums, int ld_sums, const LinearShape s,
+                                                                        const RowPlan plan) {
+    constexpr int PART = C / 4;
+    __shared__ __align__(16) float a1[C][RANK];
+    __shared__ float part[4][64];
+    RowEntry e;
+    int t0;
+    if (!locate_chunk<C>(plan, blockIdx.y, e, t0)) return;
+    const int n = min(C, e.n - t0), tid = threadIdx.x, c = blockIdx.x * 64 + (tid & 63), quarter = tid >> 6, all = s.heads * s.D;
+    const __nv_bfloat16* src = proj + (size_t)(e.row0 + t0) * s.ld + s.off_a;
+    auto row8 = [](const __nv_bfloat16* p, bool in, float (&f)[8]) { unpack8(in ? ld_cached(p) : make_uint4(0u, 0u, 0u, 0u), f); };
+    for (int i = tid; i < C * RANK / 8; i += 256) {                     // columns past the rank are zero in W_a1, so here
+        const int r = i / (RANK / 8), k = 8 * (i - r * (RANK / 8));
+        float f[8];
+        row8(src + (size_t)r * s.ld + k, r < n && k < s.ld_a2, f);
+        *reinterpret_cast<float4*>(&a1[r][k]) = make_float4(f[0], f[1], f[2], f[3]);
+        *reinterpret_cast<float4*>(&a1[r][k + 4]) = make_float4(f[4], f[5], f[6], f[7]);
+    }
+    float w[RANK], b = 0.f;
+#pragma unroll
+    for (int k = 0; k < RANK; k += 8) {
+        float f[8];
+        row8(s.a2 + (size_t)c * s.ld_a2 + k, c < all && k < s.ld_a2, f);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) w[k + j] = f[j];
+    }
+    if (c < all) b = __bfloat162float(s.a2_bias[c]);
+    __syncthreads();
+    float v[PART], sum = 0.f;
+#pragma unroll
+    for (int r = 0; r < PART; ++r) {
+        const float4* x = reinterpret_cast<const float4*>(a1[quarter * PART + r]);
+        float z = b;
+#pragma unroll
+        for (int k = 0; k < RANK / 4; ++k) {
+            const float4 y = x[k];
+            z = fmaf(w[4 * k], y.x, z); z = fmaf(w[4 * k + 1], y.y, z); z = fmaf(w[4 * k + 2], y.z, z); z = fmaf(w[4 * k + 3], y.w, z);
+        }
+        sum += log_decay_fast(z, s.inv_tau);
+        v[r] = sum;
+    }
+    part[quarter][tid & 63] = sum;
+    __syncthreads();
+    float before = 0.f;
+    for (int k = 0; k < quarter; ++k) before += part[k][tid & 63];
+    float* out = sums + (size_t)(e.row0 + t0 + quarter * PART) * ld_sums + c;
+#pragma unroll
+    for (int r = 0; r < PART; ++r)
+        if (quarter * PART + r < n && c < ld_sums) out[(size_t)r * ld_sums] = before + v[r];
 }
 
 namespace lc {

@@ -19,7 +19,7 @@
 namespace efm {
 
 namespace lt {
-constexpr int C = kLinearChunkTc, kThreads = 256;
+constexpr int C = kLinearChunkTc, kThreads = 256, kChThreads = 512;
 constexpr int BOX = C * 128;                                  // bytes of a box of 64 channels
 template <int VP>
 struct Cfg {
@@ -69,10 +69,11 @@ __device__ __forceinline__ void load_sums(const float* row, int c, int width, fl
 }
 // rows [0, n) of a head into an image of `rows` rows and 8 cols8 channels, the rest zero: asynchronous copies where the head's
 // channels come in whole 16-byte pieces
+template <int THREADS = kThreads>
 __device__ __forceinline__ void stage_head(unsigned char* dst, const __nv_bfloat16* head, int ld, int c0, int width, int n, int rows, int cols8) {
     const bool vec = ((reinterpret_cast<uintptr_t>(head) & 15) | (uintptr_t)(width & 7)) == 0;
     const uint32_t to = tc::smem_u32(dst);
-    for (int i = threadIdx.x; i < rows * cols8; i += kThreads) {
+    for (int i = threadIdx.x; i < rows * cols8; i += THREADS) {
         const int r = i / cols8, c8 = i - r * cols8, c = c0 + 8 * c8;
         const bool in = r < n && c < width;
         if (vec)
@@ -84,12 +85,19 @@ __device__ __forceinline__ void stage_head(unsigned char* dst, const __nv_bfloat
 }
 template <int N>
 __device__ __forceinline__ void staged() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-// One row's value channels [hf HALF, (hf + 1) HALF) of a head: scale, norm over the head (both halves), weight, gate, output.  All threads
-// call it.
-template <int HALF>
+__device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&r)[16]) {
+    asm volatile("tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]),
+                   "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+                 : "r"(taddr) : "memory");
+    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+}
+// One row's value channels [hf HALF, (hf + 1) HALF) of a head: scale, norm over the head (all PARTS of it), weight, gate, output.  All
+// threads call it.
+template <int HALF, int PARTS = 2>
 __device__ __forceinline__ void head_output(const float (&f)[HALF], bool valid, int t, int hf, int h, size_t row, const __nv_bfloat16* __restrict__ proj,
                                             __nv_bfloat16* __restrict__ out, int ld_out, const LinearShape& s) {
-    __shared__ float part[2][C];
+    __shared__ float part[PARTS][C];
     const __nv_bfloat16* gate = proj + row * s.ld + s.off_g + h * s.Dv;
     const bool vec = (s.Dv & 7) == 0;                                  // rows, off_g and ld_out are multiples of 8
     float ss = 0.f;
@@ -101,7 +109,10 @@ __device__ __forceinline__ void head_output(const float (&f)[HALF], bool valid, 
     part[hf][t] = ss;
     __syncthreads();
     if (!valid) return;
-    const float inv = s.scale / sqrtf((part[0][t] + part[1][t]) * s.scale * s.scale / (float)s.Dv + s.eps);
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < PARTS; ++i) ss += part[i][t];
+    const float inv = s.scale / sqrtf(ss * s.scale * s.scale / (float)s.Dv + s.eps);
     __nv_bfloat16* dst = out + row * ld_out + h * s.Dv;
 #pragma unroll
     for (int i = 0; i < HALF; i += 8) {
@@ -404,13 +415,13 @@ __global__ void __launch_bounds__(lt::kThreads, 1) linear_attend_tc_kernel(const
 // The same with decays per key channel.  Images: Q high | Q low | K high | K low | V; the state's pair takes the place of K's once P is
 // there.  P V and Q S add up in one accumulator.  HEAD: normed and gated bf16 rows instead of o.
 template <int VP, bool HEAD>
-__global__ void __launch_bounds__(lt::kThreads, 1) linear_attend_ch_tc_kernel(const __nv_bfloat16* __restrict__ proj, const float* __restrict__ ws,
+__global__ void __launch_bounds__(lt::kChThreads, 1) linear_attend_ch_tc_kernel(const __nv_bfloat16* __restrict__ proj, const float* __restrict__ ws,
                                                                             const float* __restrict__ sums, int ld_sums, float* __restrict__ o, int ld_o,
                                                                             __nv_bfloat16* __restrict__ out, int ld_out, const LinearShape s, const RowPlan plan,
                                                                             int* error) {
     using namespace lt;
     using Cf = Cfg<VP>;
-    constexpr int TMEM = 512, QH_OFF = 0, QL_OFF = Cf::K_BYTES, KH_OFF = 2 * Cf::K_BYTES, KL_OFF = 3 * Cf::K_BYTES, V_OFF = 4 * Cf::K_BYTES,
+    constexpr int TMEM = 512, THREADS = kChThreads, COLS = VP / 4, QH_OFF = 0, QL_OFF = Cf::K_BYTES, KH_OFF = 2 * Cf::K_BYTES, KL_OFF = 3 * Cf::K_BYTES, V_OFF = 4 * Cf::K_BYTES,
                   BAR_OFF = V_OFF + Cf::V_BYTES;
     extern __shared__ unsigned char lt_smem[];
     RowEntry e;
@@ -437,7 +448,7 @@ __global__ void __launch_bounds__(lt::kThreads, 1) linear_attend_ch_tc_kernel(co
     const __nv_bfloat16* row = proj + (size_t)(e.row0 + t0) * s.ld;
     const __nv_bfloat16 *q0 = row + s.off_q + h * s.D, *k0 = row + s.off_k + h * s.D, *w0 = row + s.off_v + h * s.Dv;
     const float *b0 = sums + (size_t)(e.row0 + t0) * ld_sums + h * s.D, *b_end = b0 + (size_t)(n - 1) * ld_sums;
-    stage_head(p0 + V_OFF, w0, s.ld, v0, s.Dv, n, steps * 16, VP / 8);
+    stage_head<THREADS>(p0 + V_OFF, w0, s.ld, v0, s.Dv, n, steps * 16, VP / 8);
     const bool strong = __syncthreads_or(tid < s.D && b_end[tid < s.D ? tid : 0] < -kMaxLoss) != 0;
     const int c8 = tid & 15, c = 8 * c8;                              // a thread stays with its eight channels
     float mid[8];
@@ -447,7 +458,7 @@ __global__ void __launch_bounds__(lt::kThreads, 1) linear_attend_ch_tc_kernel(co
     const bool vq = ((reinterpret_cast<uintptr_t>(q0) | reinterpret_cast<uintptr_t>(k0)) & 15) == 0;
     if (c8 < 2 * dsteps) {                                            // rows past n: zero, every row of the product is computed
 #pragma unroll 4
-        for (int r = tid >> 4; r < C; r += kThreads / 16) {
+        for (int r = tid >> 4; r < C; r += THREADS / 16) {
             const bool in = r < n && c < s.D;
             float f[8], k[8], b[8];
             load_sums(b0 + (size_t)min(r, n - 1) * ld_sums, c, s.D, b);
@@ -477,14 +488,14 @@ __global__ void __launch_bounds__(lt::kThreads, 1) linear_attend_ch_tc_kernel(co
         tc::umma_commit(pbar);
     }
     // the state, requested while P is computed
-    constexpr int ITEMS = 128 * (VP / 8) / kThreads;
+    constexpr int ITEMS = 128 * (VP / 8) / THREADS;
     float4 sa[ITEMS], sb[ITEMS];
     float se[ITEMS];
     if (state) {
         const float* S = ws + ((size_t)blockIdx.x * s.heads + h) * s.head_floats();
 #pragma unroll
         for (int u = 0; u < ITEMS; ++u) {
-            const int i = tid + u * kThreads, d = i / (VP / 8), v = v0 + 8 * (i % (VP / 8));
+            const int i = tid + u * THREADS, d = i / (VP / 8), v = v0 + 8 * (i % (VP / 8));
             const bool in = d < s.D;
             sa[u] = in && v < s.Vp ? *reinterpret_cast<const float4*>(S + (size_t)d * s.Vp + v) : make_float4(0.f, 0.f, 0.f, 0.f);
             sb[u] = in && v + 4 < s.Vp ? *reinterpret_cast<const float4*>(S + (size_t)d * s.Vp + v + 4) : make_float4(0.f, 0.f, 0.f, 0.f);
@@ -495,18 +506,18 @@ __global__ void __launch_bounds__(lt::kThreads, 1) linear_attend_ch_tc_kernel(co
     if (!ok) *abort_s = 1;
     __syncwarp();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-    const int t = (warp & 3) * 32 + lane, hf = warp >> 2;             // TMEM lane = token; which half of the columns
+    const int t = (warp & 3) * 32 + lane, part = warp >> 2;           // TMEM lane = token; which quarter of the columns
     const uint32_t lanes = tmem + ((uint32_t)((warp & 3) * 32) << 16);
-#pragma unroll 1
-    for (int c0 = 0; c0 < 64; c0 += 32) {
+    {
         uint32_t r[32], hi[16], lo[16];
+        const int u0 = part * 32;
         if (!strong) {
-            tc::tmem_ld32(lanes + (uint32_t)(hf * 64 + c0), r);
+            tc::tmem_ld32(lanes + (uint32_t)u0, r);
         } else {
             float acc[32];
 #pragma unroll
             for (int j = 0; j < 32; ++j) acc[j] = 0.f;
-            const int tt = min(t, n - 1), u0 = hf * 64 + c0;
+            const int tt = min(t, n - 1);
             for (int d = 0; d < s.D; ++d) {
                 const float q = __bfloat162float(q0[(size_t)tt * s.ld + d]), b = b0[(size_t)tt * ld_sums + d];
 #pragma unroll
@@ -520,19 +531,19 @@ __global__ void __launch_bounds__(lt::kThreads, 1) linear_attend_ch_tc_kernel(co
         }
 #pragma unroll
         for (int j = 0; j < 32; j += 2) {
-            const int u = hf * 64 + c0 + j;
+            const int u = u0 + j;
             const float a = u <= t ? __uint_as_float(r[j]) : 0.f, b = u + 1 <= t ? __uint_as_float(r[j + 1]) : 0.f;
             hi[j >> 1] = pack_bf16(a, b);
             lo[j >> 1] = pack_bf16(a - bf16lo(hi[j >> 1]), b - bf16hi(hi[j >> 1]));
         }
-        wt::tmem_st16(lanes + (uint32_t)(PH_COL + hf * 32 + c0 / 2), hi);
-        wt::tmem_st16(lanes + (uint32_t)(PL_COL + hf * 32 + c0 / 2), lo);
+        wt::tmem_st16(lanes + (uint32_t)(PH_COL + u0 / 2), hi);
+        wt::tmem_st16(lanes + (uint32_t)(PL_COL + u0 / 2), lo);
     }
     asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
     if (state && ok) {                                                // P is complete: K's images are free
 #pragma unroll
         for (int u = 0; u < ITEMS; ++u) {
-            const int i = tid + u * kThreads;
+            const int i = tid + u * THREADS;
             const float x = se[u], f[8] = {x * sa[u].x, x * sa[u].y, x * sa[u].z, x * sa[u].w, x * sb[u].x, x * sb[u].y, x * sb[u].z, x * sb[u].w};
             if (i < dsteps * 16 * (VP / 8)) put_pair(p0 + KH_OFF, p0 + KL_OFF, i / (VP / 8), i % (VP / 8), f);
         }
@@ -557,25 +568,23 @@ __global__ void __launch_bounds__(lt::kThreads, 1) linear_attend_ch_tc_kernel(co
     }
     ok = __all_sync(0xffffffffu, ok && tc::mbar_wait(obar, 0, abort_s));
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-    float f[Cf::HALF];
+    float f[COLS];
     if (ok) {
+        uint32_t y[COLS];
+        if constexpr (COLS == 32) tc::tmem_ld32(lanes + (uint32_t)(O2_COL + part * COLS), y);
+        else tmem_ld16(lanes + (uint32_t)(O2_COL + part * COLS), y);
 #pragma unroll
-        for (int c0 = 0; c0 < Cf::HALF; c0 += 32) {
-            uint32_t y[32];
-            tc::tmem_ld32(lanes + (uint32_t)(O2_COL + hf * Cf::HALF + c0), y);
-#pragma unroll
-            for (int j = 0; j < 32; ++j) f[c0 + j] = __uint_as_float(y[j]);
-        }
+        for (int j = 0; j < COLS; ++j) f[j] = __uint_as_float(y[j]);
     } else if (tid == 0 && error != nullptr) {
         atomicExch(error, 1);
     }
     if constexpr (HEAD) {
-        head_output<Cf::HALF>(f, ok && t < n, t, hf, h, (size_t)(e.row0 + t0 + t), proj, out, ld_out, s);
+        head_output<COLS, 4>(f, ok && t < n, t, part, h, (size_t)(e.row0 + t0 + t), proj, out, ld_out, s);
     } else if (ok && t < n) {
         float* dst = o + (size_t)(e.row0 + t0 + t) * ld_o + h * s.Dv;
 #pragma unroll
-        for (int j = 0; j < Cf::HALF; ++j)
-            if (v0 + hf * Cf::HALF + j < s.Dv) dst[v0 + hf * Cf::HALF + j] = f[j];
+        for (int j = 0; j < COLS; ++j)
+            if (v0 + part * COLS + j < s.Dv) dst[v0 + part * COLS + j] = f[j];
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();

@@ -116,8 +116,18 @@ __global__ void __launch_bounds__(256, 4) qk_scatter_rows_kernel(const TI* __res
     float inv_q = 1.f, inv_k = 1.f;
     if (s.qk_norm == 2) {
         float sq = 0.f, sk = 0.f;
-        for (int c = threadIdx.x; c < s.H * s.D; c += 256) { const float v = to_f32(src[c]); sq = fmaf(v, v, sq); }
-        for (int c = threadIdx.x; c < s.G * s.D; c += 256) { const float v = to_f32(src[s.H * s.D + c]); sk = fmaf(v, v, sk); }
+        auto squares = [&](int c0, int n) {
+            const bool v8 = (c0 & 7) == 0;
+            float t = 0.f, f[8];
+            for (int c = 8 * threadIdx.x; c < n; c += 2048) {
+                load_head8(src + c0, c, n, v8, f);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) t = fmaf(f[j], f[j], t);
+            }
+            return t;
+        };
+        sq = squares(0, s.H * s.D);
+        sk = squares(s.H * s.D, s.G * s.D);
         sq = warp_sum(sq);
         sk = warp_sum(sk);
         if ((threadIdx.x & 31) == 0) { row_ss[0][threadIdx.x >> 5] = sq; row_ss[1][threadIdx.x >> 5] = sk; }

@@ -679,7 +679,7 @@ void linear_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const Deco
     };
     auto decay_product = [&](auto rank) {
         constexpr int RANK = decltype(rank)::value;
-        L.launch(linear_decay_product_sums_kernel<kLinearChunkTc, RANK>, dim3((ld_sums + 63) / 64, chunks), dim3(256), 0, reinterpret_cast<const __nv_bfloat16*>(proj),
+        L.launch(linear_decay_product_sums_kernel<kLinearChunkTc, RANK>, dim3((ld_sums + 63) / 64, chunks), dim3(512), 0, reinterpret_cast<const __nv_bfloat16*>(proj),
                  m.decay, ld_sums, s, plan);
     };
     if (s.rank > 0 && s.rank <= 32 && tensor_cores) {
@@ -711,12 +711,12 @@ void linear_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const Deco
                 if (s.rank > 0) {
                     L.launch(linear_chunk_tc_kernel<VP, true>, grid, block, Cf::CHUNK_SMEM, proj, m.lin_ws, s, plan, &c.state->error, sums, ld_sums);
                     chain(linear_chain_rows_kernel<kLinearChunkTc, true>);
-                    L.launch(whole ? linear_attend_ch_tc_kernel<VP, true> : linear_attend_ch_tc_kernel<VP, false>, grid, dim3(lt::kChThreads), Cf::ATTEND_CH_SMEM, proj, ws, sums, ld_sums,
+                    L.launch(whole ? linear_attend_ch_tc_kernel<VP, true> : linear_attend_ch_tc_kernel<VP, false>, grid, dim3(lt::kAttendThreads), Cf::ATTEND_CH_SMEM, proj, ws, sums, ld_sums,
                              m.o, ld_o, out, l.mix_wp, s, plan, &c.state->error);
                 } else {
                     L.launch(linear_chunk_tc_kernel<VP>, grid, block, Cf::CHUNK_SMEM, proj, m.lin_ws, s, plan, &c.state->error, sums, 0);
                     chain(linear_chain_rows_kernel<kLinearChunkTc>);
-                    L.launch(whole ? linear_attend_tc_kernel<VP, true> : linear_attend_tc_kernel<VP>, grid, block, Cf::ATTEND_SMEM, proj, ws, m.o, ld_o, s, plan,
+                    L.launch(whole ? linear_attend_tc_kernel<VP, true> : linear_attend_tc_kernel<VP>, grid, dim3(lt::kAttendThreads), Cf::ATTEND_SMEM, proj, ws, m.o, ld_o, s, plan,
                              &c.state->error, out, l.mix_wp);
                 }
                 if (!whole) output();

@@ -441,20 +441,20 @@ __device__ __forceinline__ float log_decay_fast(float z, float inv_tau) {
     return (fminf(z, 0.f) - l) * inv_tau;
 }
 // linear_decay_sums with the product W_a2 (W_a1 x) + b in front of it, W_a1 x of at most RANK bf16 numbers a row.  Grid (64 channels, chunks
-// of C tokens): four threads a channel, a quarter of the chunk each.
+// of C tokens): eight threads a channel, an eighth of the chunk each.
 template <int C, int RANK>
-__global__ void __launch_bounds__(256) linear_decay_product_sums_kernel(const __nv_bfloat16* __restrict__ proj, float* __restrict__ sums, int ld_sums, const LinearShape s,
+__global__ void __launch_bounds__(512, 2) linear_decay_product_sums_kernel(const __nv_bfloat16* __restrict__ proj, float* __restrict__ sums, int ld_sums, const LinearShape s,
                                                                         const RowPlan plan) {
-    constexpr int PART = C / 4;
+    constexpr int PART = C / 8;
     __shared__ __align__(16) float a1[C][RANK];
-    __shared__ float part[4][64];
+    __shared__ float part[8][64];
     RowEntry e;
     int t0;
     if (!locate_chunk<C>(plan, blockIdx.y, e, t0)) return;
-    const int n = min(C, e.n - t0), tid = threadIdx.x, c = blockIdx.x * 64 + (tid & 63), quarter = tid >> 6, all = s.heads * s.D;
+    const int n = min(C, e.n - t0), tid = threadIdx.x, c = blockIdx.x * 64 + (tid & 63), eighth = tid >> 6, all = s.heads * s.D;
     const __nv_bfloat16* src = proj + (size_t)(e.row0 + t0) * s.ld + s.off_a;
     auto row8 = [](const __nv_bfloat16* p, bool in, float (&f)[8]) { unpack8(in ? ld_cached(p) : make_uint4(0u, 0u, 0u, 0u), f); };
-    for (int i = tid; i < C * RANK / 8; i += 256) {                     // columns past the rank are zero in W_a1, so here
+    for (int i = tid; i < C * RANK / 8; i += 512) {                     // columns past the rank are zero in W_a1, so here
         const int r = i / (RANK / 8), k = 8 * (i - r * (RANK / 8));
         float f[8];
         row8(src + (size_t)r * s.ld + k, r < n && k < s.ld_a2, f);
@@ -474,7 +474,7 @@ __global__ void __launch_bounds__(256) linear_decay_product_sums_kernel(const __
     float v[PART], sum = 0.f;
 #pragma unroll
     for (int r = 0; r < PART; ++r) {
-        const float4* x = reinterpret_cast<const float4*>(a1[quarter * PART + r]);
+        const float4* x = reinterpret_cast<const float4*>(a1[eighth * PART + r]);
         float z = b;
 #pragma unroll
         for (int k = 0; k < RANK / 4; ++k) {
@@ -484,14 +484,14 @@ __global__ void __launch_bounds__(256) linear_decay_product_sums_kernel(const __
         sum += log_decay_fast(z, s.inv_tau);
         v[r] = sum;
     }
-    part[quarter][tid & 63] = sum;
+    part[eighth][tid & 63] = sum;
     __syncthreads();
     float before = 0.f;
-    for (int k = 0; k < quarter; ++k) before += part[k][tid & 63];
-    float* out = sums + (size_t)(e.row0 + t0 + quarter * PART) * ld_sums + c;
+    for (int k = 0; k < eighth; ++k) before += part[k][tid & 63];
+    float* out = sums + (size_t)(e.row0 + t0 + eighth * PART) * ld_sums + c;
 #pragma unroll
     for (int r = 0; r < PART; ++r)
-        if (quarter * PART + r < n && c < ld_sums) out[(size_t)r * ld_sums] = before + v[r];
+        if (eighth * PART + r < n && c < ld_sums) out[(size_t)r * ld_sums] = before + v[r];
 }
 
 namespace lc {

@@ -19,7 +19,7 @@
 namespace efm {
 
 namespace lt {
-constexpr int C = kLinearChunkTc, kThreads = 256, kChThreads = 512;
+constexpr int C = kLinearChunkTc, kThreads = 256, kAttendThreads = 512;
 constexpr int BOX = C * 128;                                  // bytes of a box of 64 channels
 template <int VP>
 struct Cfg {
@@ -85,6 +85,19 @@ __device__ __forceinline__ void stage_head(unsigned char* dst, const __nv_bfloat
 }
 template <int N>
 __device__ __forceinline__ void staged() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+// o[v ..] = f, channels past Dv left out
+template <int N>
+__device__ __forceinline__ void raw_output(const float (&f)[N], int v, float* __restrict__ o, int Dv) {
+    if ((Dv & 3) == 0) {
+#pragma unroll
+        for (int j = 0; j < N; j += 4)
+            if (v + j < Dv) *reinterpret_cast<float4*>(o + v + j) = make_float4(f[j], f[j + 1], f[j + 2], f[j + 3]);
+    } else {
+#pragma unroll
+        for (int j = 0; j < N; ++j)
+            if (v + j < Dv) o[v + j] = f[j];
+    }
+}
 __device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&r)[16]) {
     asm volatile("tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]),
@@ -92,10 +105,12 @@ __device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&r)[16]) {
                  : "r"(taddr) : "memory");
     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 }
-// One row's value channels [hf HALF, (hf + 1) HALF) of a head: scale, norm over the head (all PARTS of it), weight, gate, output.  All
+__device__ __forceinline__ void tmem_ld_cols(uint32_t taddr, uint32_t (&r)[16]) { tmem_ld16(taddr, r); }
+__device__ __forceinline__ void tmem_ld_cols(uint32_t taddr, uint32_t (&r)[32]) { tc::tmem_ld32(taddr, r); }
+// One row's value channels [k N, (k + 1) N) of a head: scale, norm over the head (all PARTS of it), weight, gate, output.  All
 // threads call it.
-template <int HALF, int PARTS = 2>
-__device__ __forceinline__ void head_output(const float (&f)[HALF], bool valid, int t, int hf, int h, size_t row, const __nv_bfloat16* __restrict__ proj,
+template <int N, int PARTS>
+__device__ __forceinline__ void head_output(const float (&f)[N], bool valid, int t, int k, int h, size_t row, const __nv_bfloat16* __restrict__ proj,
                                             __nv_bfloat16* __restrict__ out, int ld_out, const LinearShape& s) {
     __shared__ float part[PARTS][C];
     const __nv_bfloat16* gate = proj + row * s.ld + s.off_g + h * s.Dv;
@@ -103,10 +118,10 @@ __device__ __forceinline__ void head_output(const float (&f)[HALF], bool valid, 
     float ss = 0.f;
     if (valid) {
 #pragma unroll
-        for (int i = 0; i < HALF; ++i)
-            if (hf * HALF + i < s.Dv) ss = fmaf(f[i], f[i], ss);
+        for (int i = 0; i < N; ++i)
+            if (k * N + i < s.Dv) ss = fmaf(f[i], f[i], ss);
     }
-    part[hf][t] = ss;
+    part[k][t] = ss;
     __syncthreads();
     if (!valid) return;
     ss = 0.f;
@@ -115,8 +130,8 @@ __device__ __forceinline__ void head_output(const float (&f)[HALF], bool valid, 
     const float inv = s.scale / sqrtf(ss * s.scale * s.scale / (float)s.Dv + s.eps);
     __nv_bfloat16* dst = out + row * ld_out + h * s.Dv;
 #pragma unroll
-    for (int i = 0; i < HALF; i += 8) {
-        const int v = hf * HALF + i;
+    for (int i = 0; i < N; i += 8) {
+        const int v = k * N + i;
         if (v >= s.Dv) break;
         float g[8];
         if (vec) unpack8(ld_cached(gate + v), g);
@@ -248,12 +263,12 @@ __global__ void __launch_bounds__(lt::kThreads, 2) linear_chunk_tc_kernel(const 
 
 // grid (chunks, heads, slices of VP value channels)
 template <int VP, bool HEAD = false>
-__global__ void __launch_bounds__(lt::kThreads, 1) linear_attend_tc_kernel(const __nv_bfloat16* __restrict__ proj, const float* __restrict__ ws, float* __restrict__ o,
+__global__ void __launch_bounds__(lt::kAttendThreads, 1) linear_attend_tc_kernel(const __nv_bfloat16* __restrict__ proj, const float* __restrict__ ws, float* __restrict__ o,
                                                                          int ld_o, const LinearShape s, const RowPlan plan, int* error,
                                                                          __nv_bfloat16* __restrict__ out, int ld_out) {
     using namespace lt;
     using Cf = Cfg<VP>;
-    constexpr int TMEM = 512;
+    constexpr int TMEM = 512, THREADS = kAttendThreads, COLS = VP / 4;
     extern __shared__ unsigned char lt_smem[];
     __shared__ float pw[C + 1];
     RowEntry e;
@@ -278,28 +293,28 @@ __global__ void __launch_bounds__(lt::kThreads, 1) linear_attend_tc_kernel(const
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(tc::smem_u32(tmem_slot)), "r"(TMEM) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
-    for (int i = tid; i <= C; i += kThreads) pw[i] = s.powers[(size_t)h * (kLinearPowers + 1) + i];
+    for (int i = tid; i <= C; i += THREADS) pw[i] = s.powers[(size_t)h * (kLinearPowers + 1) + i];
     const __nv_bfloat16* row = proj + (size_t)(e.row0 + t0) * s.ld;
     const __nv_bfloat16 *q0 = row + s.off_q + h * s.D, *k0 = row + s.off_k + h * s.D, *w0 = row + s.off_v + h * s.Dv;
-    stage_head(p0, q0, s.ld, 0, s.D, n, C, 2 * dsteps);               // rows past n: zero, every row of the product is computed
-    stage_head(p0 + K_OFF, k0, s.ld, 0, s.D, n, C, 2 * dsteps);
-    stage_head(p0 + V_OFF, w0, s.ld, v0, s.Dv, n, steps * 16, VP / 8);
+    stage_head<THREADS>(p0, q0, s.ld, 0, s.D, n, C, 2 * dsteps);               // rows past n: zero, every row of the product is computed
+    stage_head<THREADS>(p0 + K_OFF, k0, s.ld, 0, s.D, n, C, 2 * dsteps);
+    stage_head<THREADS>(p0 + V_OFF, w0, s.ld, v0, s.Dv, n, steps * 16, VP / 8);
     if (state) {
         const float* S = ws + ((size_t)blockIdx.x * s.heads + h) * s.head_floats();
         constexpr int U = 4;
         const int all = dsteps * 16 * (VP / 8);
-        for (int i0 = tid; i0 < all; i0 += U * kThreads) {
+        for (int i0 = tid; i0 < all; i0 += U * THREADS) {
             float4 a[U], b[U];
 #pragma unroll
             for (int u = 0; u < U; ++u) {
-                const int i = i0 + u * kThreads, d = i / (VP / 8), v = v0 + 8 * (i % (VP / 8));
+                const int i = i0 + u * THREADS, d = i / (VP / 8), v = v0 + 8 * (i % (VP / 8));
                 const bool in = i < all && d < s.D;
                 a[u] = in && v < s.Vp ? *reinterpret_cast<const float4*>(S + (size_t)d * s.Vp + v) : make_float4(0.f, 0.f, 0.f, 0.f);
                 b[u] = in && v + 4 < s.Vp ? *reinterpret_cast<const float4*>(S + (size_t)d * s.Vp + v + 4) : make_float4(0.f, 0.f, 0.f, 0.f);
             }
 #pragma unroll
             for (int u = 0; u < U; ++u) {
-                const int i = i0 + u * kThreads;
+                const int i = i0 + u * THREADS;
                 const float f[8] = {a[u].x, a[u].y, a[u].z, a[u].w, b[u].x, b[u].y, b[u].z, b[u].w};
                 if (i < all) put_pair(p0 + SH_OFF, p0 + SL_OFF, i / (VP / 8), i % (VP / 8), f);
             }
@@ -324,21 +339,20 @@ __global__ void __launch_bounds__(lt::kThreads, 1) linear_attend_tc_kernel(const
     if (!ok) *abort_s = 1;
     __syncwarp();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-    const int t = (warp & 3) * 32 + lane, hf = warp >> 2;             // TMEM lane = token; which half of the columns
+    const int t = (warp & 3) * 32 + lane, part = warp >> 2;           // TMEM lane = token; which quarter of the columns
     const uint32_t lanes = tmem + ((uint32_t)((warp & 3) * 32) << 16);
-#pragma unroll
-    for (int c0 = 0; c0 < 64; c0 += 32) {
+    {
         uint32_t r[32], hi[16], lo[16];
-        tc::tmem_ld32(lanes + (uint32_t)(hf * 64 + c0), r);
+        tc::tmem_ld32(lanes + (uint32_t)(part * 32), r);
 #pragma unroll
         for (int j = 0; j < 32; j += 2) {
-            const int u = hf * 64 + c0 + j;
+            const int u = part * 32 + j;
             const float a = u <= t ? __uint_as_float(r[j]) * pw[t - u] : 0.f, b = u + 1 <= t ? __uint_as_float(r[j + 1]) * pw[t - u - 1] : 0.f;
             hi[j >> 1] = pack_bf16(a, b);
             lo[j >> 1] = pack_bf16(a - bf16lo(hi[j >> 1]), b - bf16hi(hi[j >> 1]));
         }
-        wt::tmem_st16(lanes + (uint32_t)(PH_COL + hf * 32 + c0 / 2), hi);
-        wt::tmem_st16(lanes + (uint32_t)(PL_COL + hf * 32 + c0 / 2), lo);
+        wt::tmem_st16(lanes + (uint32_t)(PH_COL + part * 16), hi);
+        wt::tmem_st16(lanes + (uint32_t)(PL_COL + part * 16), lo);
     }
     asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -360,50 +374,19 @@ __global__ void __launch_bounds__(lt::kThreads, 1) linear_attend_tc_kernel(const
     }
     ok = __all_sync(0xffffffffu, ok && tc::mbar_wait(obar, 0, abort_s));
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-    if constexpr (HEAD) {
-        float f[Cf::HALF];
-        if (ok) {
-            const float a = pw[t + 1];
-#pragma unroll
-            for (int c0 = 0; c0 < Cf::HALF; c0 += 32) {
-                uint32_t x[32], y[32];
-                tc::tmem_ld32(lanes + (uint32_t)(O2_COL + hf * Cf::HALF + c0), y);
-                if (state) tc::tmem_ld32(lanes + (uint32_t)(O1_COL + hf * Cf::HALF + c0), x);
-#pragma unroll
-                for (int j = 0; j < 32; ++j) f[c0 + j] = state ? fmaf(a, __uint_as_float(x[j]), __uint_as_float(y[j])) : __uint_as_float(y[j]);
-            }
-        }
-        head_output<Cf::HALF>(f, ok && t < n, t, hf, h, (size_t)(e.row0 + t0 + t), proj, out, ld_out, s);
-        if (!ok && tid == 0 && error != nullptr) atomicExch(error, 1);
-    } else if (ok) {
-        float* dst = o + (size_t)(e.row0 + t0 + t) * ld_o + h * s.Dv;
+    float f[COLS];
+    if (ok) {
+        uint32_t x[COLS], y[COLS];
         const float a = pw[t + 1];
-        const bool vec = (s.Dv & 3) == 0;
+        tmem_ld_cols(lanes + (uint32_t)(O2_COL + part * COLS), y);
+        if (state) tmem_ld_cols(lanes + (uint32_t)(O1_COL + part * COLS), x);
 #pragma unroll
-        for (int c0 = 0; c0 < Cf::HALF; c0 += 32) {
-            uint32_t x[32], y[32];
-            tc::tmem_ld32(lanes + (uint32_t)(O2_COL + hf * Cf::HALF + c0), y);
-            if (state) tc::tmem_ld32(lanes + (uint32_t)(O1_COL + hf * Cf::HALF + c0), x);
-            const bool in = t < n;
-#pragma unroll
-            for (int j = 0; j < 32; j += 4) {
-                const int v = v0 + hf * Cf::HALF + c0 + j;
-                float f[4];
-#pragma unroll
-                for (int k = 0; k < 4; ++k) f[k] = state ? fmaf(a, __uint_as_float(x[j + k]), __uint_as_float(y[j + k])) : __uint_as_float(y[j + k]);
-                if (vec) {
-                    if (in && v < s.Dv) *reinterpret_cast<float4*>(dst + v) = make_float4(f[0], f[1], f[2], f[3]);
-                } else {
-#pragma unroll
-                    for (int k = 0; k < 4; ++k)
-                        if (in && v + k < s.Dv) dst[v + k] = f[k];
-                }
-            }
-            __syncwarp();
-        }
+        for (int j = 0; j < COLS; ++j) f[j] = state ? fmaf(a, __uint_as_float(x[j]), __uint_as_float(y[j])) : __uint_as_float(y[j]);
     } else if (tid == 0 && error != nullptr) {
         atomicExch(error, 1);
     }
+    if constexpr (HEAD) head_output<COLS, 4>(f, ok && t < n, t, part, h, (size_t)(e.row0 + t0 + t), proj, out, ld_out, s);
+    else if (ok && t < n) raw_output(f, v0 + part * COLS, o + (size_t)(e.row0 + t0 + t) * ld_o + h * s.Dv, s.Dv);
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();
     if (warp == 0) {
@@ -415,13 +398,13 @@ __global__ void __launch_bounds__(lt::kThreads, 1) linear_attend_tc_kernel(const
 // The same with decays per key channel.  Images: Q high | Q low | K high | K low | V; the state's pair takes the place of K's once P is
 // there.  P V and Q S add up in one accumulator.  HEAD: normed and gated bf16 rows instead of o.
 template <int VP, bool HEAD>
-__global__ void __launch_bounds__(lt::kChThreads, 1) linear_attend_ch_tc_kernel(const __nv_bfloat16* __restrict__ proj, const float* __restrict__ ws,
+__global__ void __launch_bounds__(lt::kAttendThreads, 1) linear_attend_ch_tc_kernel(const __nv_bfloat16* __restrict__ proj, const float* __restrict__ ws,
                                                                             const float* __restrict__ sums, int ld_sums, float* __restrict__ o, int ld_o,
                                                                             __nv_bfloat16* __restrict__ out, int ld_out, const LinearShape s, const RowPlan plan,
                                                                             int* error) {
     using namespace lt;
     using Cf = Cfg<VP>;
-    constexpr int TMEM = 512, THREADS = kChThreads, COLS = VP / 4, QH_OFF = 0, QL_OFF = Cf::K_BYTES, KH_OFF = 2 * Cf::K_BYTES, KL_OFF = 3 * Cf::K_BYTES, V_OFF = 4 * Cf::K_BYTES,
+    constexpr int TMEM = 512, THREADS = kAttendThreads, COLS = VP / 4, QH_OFF = 0, QL_OFF = Cf::K_BYTES, KH_OFF = 2 * Cf::K_BYTES, KL_OFF = 3 * Cf::K_BYTES, V_OFF = 4 * Cf::K_BYTES,
                   BAR_OFF = V_OFF + Cf::V_BYTES;
     extern __shared__ unsigned char lt_smem[];
     RowEntry e;
@@ -571,21 +554,14 @@ __global__ void __launch_bounds__(lt::kChThreads, 1) linear_attend_ch_tc_kernel(
     float f[COLS];
     if (ok) {
         uint32_t y[COLS];
-        if constexpr (COLS == 32) tc::tmem_ld32(lanes + (uint32_t)(O2_COL + part * COLS), y);
-        else tmem_ld16(lanes + (uint32_t)(O2_COL + part * COLS), y);
+        tmem_ld_cols(lanes + (uint32_t)(O2_COL + part * COLS), y);
 #pragma unroll
         for (int j = 0; j < COLS; ++j) f[j] = __uint_as_float(y[j]);
     } else if (tid == 0 && error != nullptr) {
         atomicExch(error, 1);
     }
-    if constexpr (HEAD) {
-        head_output<COLS, 4>(f, ok && t < n, t, part, h, (size_t)(e.row0 + t0 + t), proj, out, ld_out, s);
-    } else if (ok && t < n) {
-        float* dst = o + (size_t)(e.row0 + t0 + t) * ld_o + h * s.Dv;
-#pragma unroll
-        for (int j = 0; j < COLS; ++j)
-            if (v0 + part * COLS + j < s.Dv) dst[v0 + part * COLS + j] = f[j];
-    }
+    if constexpr (HEAD) head_output<COLS, 4>(f, ok && t < n, t, part, h, (size_t)(e.row0 + t0 + t), proj, out, ld_out, s);
+    else if (ok && t < n) raw_output(f, v0 + part * COLS, o + (size_t)(e.row0 + t0 + t) * ld_o + h * s.Dv, s.Dv);
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();
     if (warp == 0) {

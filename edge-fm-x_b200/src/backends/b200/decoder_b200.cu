@@ -480,6 +480,9 @@ efm_status efm_b200_decoder_create(const efm_decoder_desc* desc, const efm_decod
         EFM_TRY(dev_alloc(c, &m->ex.n_tiles, 1));
         EFM_TRY(dev_alloc(c, &m->ex.shared, S));
         if (sh_ff > 0) {
+            EFM_TRY(cudaStreamCreateWithFlags(&m->side, cudaStreamNonBlocking));
+            EFM_TRY(cudaEventCreateWithFlags(&m->side_start, cudaEventDisableTiming));
+            EFM_TRY(cudaEventCreateWithFlags(&m->side_end, cudaEventDisableTiming));
             EFM_TRY(act(&m->sh_act, S * sh_ff));
             EFM_TRY(act(&m->sh_y, (size_t)S * Wp));
             if (m->f32) EFM_TRY(dev_alloc(c, &m->sh_gu, S * 2 * sh_ff));
@@ -1160,6 +1163,10 @@ int64_t decoder_step_bytes(const efm_b200_ctx& c, int32_t kv_len) {
 }
 
 void decoder_destroy(efm_b200_ctx* c) {
+    DecoderModel& m = *c->decoder;
+    if (m.side_start != nullptr) cudaEventDestroy(m.side_start);
+    if (m.side_end != nullptr) cudaEventDestroy(m.side_end);
+    if (m.side != nullptr) cudaStreamDestroy(m.side);
     delete c->decoder;
     c->decoder = nullptr;
 }

@@ -859,13 +859,38 @@ void latent_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const Deco
     launch_latent_rows<TA>(c, L, l, run, plan, nullptr, T);
 }
 
+GemmEpi expert_epi(const DecoderLayer& l) {
+    return !l.gated_experts() ? GemmEpi::Bf16Relu2 : l.d.expert_glu == EFM_GLU_CLAMPED ? GemmEpi::ClampGlu : GemmEpi::SwiGlu;
+}
 // Routed experts of all rows: choice, rows sorted by expert, two grouped products.  The outputs stay sorted (m.ex_y); the norm
 // that follows sums them (SumOf).
 template <typename TA>
 SumOf<TA> expert_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const void* h, int T) {
     DecoderModel& m = *c.decoder;
     const RouteShape r = route_shape(l);
+    // the shared expert on a stream of its own, products unsplit: the split-K workspace belongs to the other stream
+    Launcher S = L;
+    S.stream = m.side;
+    S.gemm_ws = nullptr;
+    auto order = [&](cudaError_t e) { if (L.err == cudaSuccess) L.err = e; };
+    if (l.d.shared_ff > 0) order(cudaEventRecord(m.side_start, L.stream));
     linear_f32(c, L, l.router, h, m.route_logits, T);
+    if (l.d.shared_ff > 0) {
+        order(cudaStreamWaitEvent(m.side, m.side_start, 0));
+        if constexpr (std::is_same<TA, float>::value) {
+            linear_f32(c, S, l.shared_in, h, m.sh_gu, T);
+            S.launch(glu_rows_kernel, dim3((T + kExpertTile - 1) / kExpertTile), dim3(256), 0, (const float*)m.sh_gu, static_cast<float*>(m.sh_act), T, l.sfp,
+                     (const int32_t*)nullptr, glu_kind(l), l.d.shared_limit);
+            linear_f32(c, S, l.shared_out, m.sh_act, static_cast<float*>(m.sh_y), T);
+        } else {
+            GemmParams g{static_cast<const __nv_bfloat16*>(h), l.shared_in.w, nullptr, static_cast<__nv_bfloat16*>(m.sh_act), nullptr, T, l.shared_in.Np, l.shared_in.Kp};
+            g.limit = l.d.shared_limit;
+            launch_gemm_epi(S, expert_epi(l), g, &c.state->error);
+            linear_act(c, S, l.shared_out, m.sh_act, m.sh_y, T);
+        }
+        order(S.err);
+        order(cudaEventRecord(m.side_end, m.side));
+    }
     L.launch(expert_route_rows_kernel, dim3((T + 7) / 8), dim3(256), 0, (const float*)m.route_logits, l.router.Np, T, r, m.ex);
     L.launch(l.d.expert_weight_input ? expert_gather_rows_kernel<TA, true> : expert_gather_rows_kernel<TA, false>, dim3(T), dim3(128), 0, static_cast<const TA*>(h), static_cast<TA*>(m.ex_in), m.Wp, r, m.ex);
     // tiles in use at most: every row tile but the last of an expert is full
@@ -877,16 +902,9 @@ SumOf<TA> expert_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const
                      (const __nv_bfloat16*)nullptr, RowGroups{m.ex.tile, m.ex.n_tiles, n});
         };
         product(l.expert_in, l.up_rows(l.ffp), static_cast<const float*>(m.ex_in), m.ex_gu);
-        const int glu = glu_kind(l);
         L.launch(glu_rows_kernel, dim3(max_rows / kExpertTile), dim3(256), 0, (const float*)m.ex_gu, static_cast<float*>(m.ex_act), max_rows, l.ffp,
-                 (const int32_t*)m.ex.n_tiles, glu, l.d.expert_limit);
+                 (const int32_t*)m.ex.n_tiles, glu_kind(l), l.d.expert_limit);
         product(l.expert_out, m.Wp, static_cast<const float*>(m.ex_act), static_cast<float*>(m.ex_y));
-        if (l.d.shared_ff > 0) {
-            linear_f32(c, L, l.shared_in, h, m.sh_gu, T);
-            L.launch(glu_rows_kernel, dim3((T + kExpertTile - 1) / kExpertTile), dim3(256), 0, (const float*)m.sh_gu, static_cast<float*>(m.sh_act), T, l.sfp,
-                     (const int32_t*)nullptr, glu, l.d.shared_limit);
-            linear_f32(c, L, l.shared_out, m.sh_act, static_cast<float*>(m.sh_y), T);
-        }
     } else {
         auto product = [&](const DecLinear& w, int n, GemmEpi epi, const void* a, void* out) {
             GemmParams g{static_cast<const __nv_bfloat16*>(a), w.w, nullptr, static_cast<__nv_bfloat16*>(out), nullptr, max_rows, n, w.Kp};
@@ -897,16 +915,10 @@ SumOf<TA> expert_rows(efm_b200_ctx& c, Launcher& L, const DecoderLayer& l, const
             g.limit = l.d.expert_limit;
             launch_gemm_epi(L, epi, g, &c.state->error);
         };
-        const GemmEpi glu = !l.gated_experts() ? GemmEpi::Bf16Relu2 : l.d.expert_glu == EFM_GLU_CLAMPED ? GemmEpi::ClampGlu : GemmEpi::SwiGlu;
-        product(l.expert_in, l.up_rows(l.ffp), glu, m.ex_in, m.ex_act);
+        product(l.expert_in, l.up_rows(l.ffp), expert_epi(l), m.ex_in, m.ex_act);
         product(l.expert_out, m.Wp, GemmEpi::Bf16Bias, m.ex_act, m.ex_y);
-        if (l.d.shared_ff > 0) {
-            GemmParams g{static_cast<const __nv_bfloat16*>(h), l.shared_in.w, nullptr, static_cast<__nv_bfloat16*>(m.sh_act), nullptr, T, l.shared_in.Np, l.shared_in.Kp};
-            g.limit = l.d.shared_limit;
-            launch_gemm_epi(L, glu, g, &c.state->error);
-            linear_act(c, L, l.shared_out, m.sh_act, m.sh_y, T);
-        }
     }
+    if (l.d.shared_ff > 0) order(cudaStreamWaitEvent(L.stream, m.side_end, 0));
     return SumOf<TA>{static_cast<const TA*>(m.ex_y), m.ex.place, m.ex.weight, r.top, m.ex.count, r.experts, l.d.expert_weight_input,
                      l.d.shared_ff > 0 ? static_cast<const TA*>(m.sh_y) : nullptr, m.ex.shared};
 }

@@ -119,6 +119,9 @@ struct DecoderModel {
     float *ex_gu = nullptr, *sh_gu = nullptr, *route_logits = nullptr;
     ExpertRows ex{};
     int ex_rows = 0;
+    // a pass's shared expert runs beside the choice and the sorting of the rows
+    cudaStream_t side = nullptr;
+    cudaEvent_t side_start = nullptr, side_end = nullptr;
     int32_t* step_buf = nullptr;          // packed per-step indices
     size_t step_words = 0;
     int max_want = 0;

@@ -432,25 +432,34 @@ __global__ void __launch_bounds__(lt::kAttendThreads, 1) linear_attend_ch_tc_ker
     const __nv_bfloat16 *q0 = row + s.off_q + h * s.D, *k0 = row + s.off_k + h * s.D, *w0 = row + s.off_v + h * s.Dv;
     const float *b0 = sums + (size_t)(e.row0 + t0) * ld_sums + h * s.D, *b_end = b0 + (size_t)(n - 1) * ld_sums;
     stage_head<THREADS>(p0 + V_OFF, w0, s.ld, v0, s.Dv, n, steps * 16, VP / 8);
-    const bool strong = __syncthreads_or(tid < s.D && b_end[tid < s.D ? tid : 0] < -kMaxLoss) != 0;
     const int c8 = tid & 15, c = 8 * c8;                              // a thread stays with its eight channels
-    float mid[8];
+    const bool vq = ((reinterpret_cast<uintptr_t>(q0) | reinterpret_cast<uintptr_t>(k0)) & 15) == 0;
+    constexpr int ROWS = C * 16 / THREADS;
+    uint4 qv[ROWS], kv[ROWS];
+    float bv[ROWS][8], mid[8];
     load_sums(b_end, c, s.D, mid);
 #pragma unroll
+    for (int u = 0; u < ROWS; ++u) {                                  // rows past n: zero, every row of the product is computed
+        const int r = (tid >> 4) + u * (THREADS / 16);
+        const bool in = r < n && c < s.D;
+        load_sums(b0 + (size_t)min(r, n - 1) * ld_sums, c, s.D, bv[u]);
+        qv[u] = in ? load_head(q0 + (size_t)r * s.ld, c, s.D, vq) : make_uint4(0u, 0u, 0u, 0u);
+        kv[u] = in ? load_head(k0 + (size_t)r * s.ld, c, s.D, vq) : make_uint4(0u, 0u, 0u, 0u);
+    }
+    const bool strong = __syncthreads_or(tid < s.D && b_end[tid < s.D ? tid : 0] < -kMaxLoss) != 0;
+#pragma unroll
     for (int j = 0; j < 8; ++j) mid[j] = strong ? 0.f : 0.5f * mid[j];
-    const bool vq = ((reinterpret_cast<uintptr_t>(q0) | reinterpret_cast<uintptr_t>(k0)) & 15) == 0;
-    if (c8 < 2 * dsteps) {                                            // rows past n: zero, every row of the product is computed
-#pragma unroll 4
-        for (int r = tid >> 4; r < C; r += THREADS / 16) {
-            const bool in = r < n && c < s.D;
-            float f[8], k[8], b[8];
-            load_sums(b0 + (size_t)min(r, n - 1) * ld_sums, c, s.D, b);
-            unpack8(in ? load_head(q0 + (size_t)r * s.ld, c, s.D, vq) : make_uint4(0u, 0u, 0u, 0u), f);
-            unpack8(in ? load_head(k0 + (size_t)r * s.ld, c, s.D, vq) : make_uint4(0u, 0u, 0u, 0u), k);
+    if (c8 < 2 * dsteps) {
+#pragma unroll
+        for (int u = 0; u < ROWS; ++u) {
+            const int r = (tid >> 4) + u * (THREADS / 16);
+            float f[8], k[8];
+            unpack8(qv[u], f);
+            unpack8(kv[u], k);
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
-                f[j] *= __expf(b[j] - mid[j]);
-                k[j] = strong ? 0.f : k[j] * __expf(mid[j] - b[j]);
+                f[j] *= __expf(bv[u][j] - mid[j]);
+                k[j] = strong ? 0.f : k[j] * __expf(mid[j] - bv[u][j]);
             }
             put_pair(p0 + QH_OFF, p0 + QL_OFF, r, c8, f);
             put_pair(p0 + KH_OFF, p0 + KL_OFF, r, c8, k);

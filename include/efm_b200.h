@@ -402,7 +402,7 @@ typedef struct efm_decoder_layer {
     int32_t window;               /* both attentions: position i sees j with 0 <= i - j < window; 0: all j <= i */
     int32_t distance_bias;        /* attention: 1 = subtract 2^(-8 (h+1) / heads) * (i - j) from the score of head h */
     float scale;                  /* both attentions: score multiplier */
-    int32_t decay_rank;           /* delta rule: rows of w1, <= 512 */
+    int32_t decay_rank;           /* delta rule: rows of w1; linear with linear_tau: of a1; <= 512 */
     int32_t ff;                   /* dense feed-forward width, 0: none */
     int32_t keep_first;           /* attention with a window: the first keep_first tokens stay visible */
     int32_t qk_norm;              /* attention: EFM_QK_NORM_* */

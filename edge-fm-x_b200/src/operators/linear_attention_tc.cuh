@@ -197,27 +197,27 @@ __global__ void __launch_bounds__(lt::kThreads, 2) linear_chunk_tc_kernel(const 
             put_pair(khi, klo, r, tid & 15, f);
         }
     } else {
-    constexpr int U = 8;
-    for (int i0 = tid; i0 < steps * 16 * 16; i0 += U * kThreads) {   // all 128 key channels: the product has 128 rows
-        uint4 x[U];
-        float a[U];
+        constexpr int U = 8;
+        for (int i0 = tid; i0 < steps * 16 * 16; i0 += U * kThreads) {   // all 128 key channels: the product has 128 rows
+            uint4 x[U];
+            float a[U];
 #pragma unroll
-        for (int u = 0; u < U; ++u) {
-            const int i = i0 + u * kThreads, r = i >> 4, c = 8 * (i & 15);
-            const bool in = r < n && c < s.D;
-            x[u] = in ? load_head(k0 + (size_t)r * s.ld, c, s.D, vk) : make_uint4(0u, 0u, 0u, 0u);
-            a[u] = in ? pw[n - 1 - r] : 0.f;
+            for (int u = 0; u < U; ++u) {
+                const int i = i0 + u * kThreads, r = i >> 4, c = 8 * (i & 15);
+                const bool in = r < n && c < s.D;
+                x[u] = in ? load_head(k0 + (size_t)r * s.ld, c, s.D, vk) : make_uint4(0u, 0u, 0u, 0u);
+                a[u] = in ? pw[n - 1 - r] : 0.f;
+            }
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                const int i = i0 + u * kThreads;
+                float f[8];
+                unpack8(x[u], f);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) f[j] *= a[u];
+                if (i < steps * 16 * 16) put_pair(khi, klo, i >> 4, i & 15, f);
+            }
         }
-#pragma unroll
-        for (int u = 0; u < U; ++u) {
-            const int i = i0 + u * kThreads;
-            float f[8];
-            unpack8(x[u], f);
-#pragma unroll
-            for (int j = 0; j < 8; ++j) f[j] *= a[u];
-            if (i < steps * 16 * 16) put_pair(khi, klo, i >> 4, i & 15, f);
-        }
-    }
     }
     staged<0>();
     fence_async_smem();

@@ -269,26 +269,26 @@ __global__ void __launch_bounds__(256) window_attention_rows_kernel(const TQ* __
 #pragma unroll
             for (int u = 0; u < 2; ++u) ps[r * (KT + 1) + c + 16 * u] = sc[u] == -INFINITY ? 0.f : sigmoid_weight(sc[u] + shift);
         } else {
-        float mx = fmaxf(sc[0], sc[1]);
+            float mx = fmaxf(sc[0], sc[1]);
 #pragma unroll
-        for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-        const float mn = fmaxf(m, mx), mb = mn == -INFINITY ? 0.f : mn;
-        const float alpha = m == -INFINITY ? 0.f : expf(m - mb);
-        m = mn;
-        float rs = 0.f;
+            for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+            const float mn = fmaxf(m, mx), mb = mn == -INFINITY ? 0.f : mn;
+            const float alpha = m == -INFINITY ? 0.f : expf(m - mb);
+            m = mn;
+            float rs = 0.f;
 #pragma unroll
-        for (int u = 0; u < 2; ++u) {
-            const float p = sc[u] == -INFINITY ? 0.f : expf(sc[u] - mb);
-            rs += p;
-            ps[r * (KT + 1) + c + 16 * u] = p;
-        }
+            for (int u = 0; u < 2; ++u) {
+                const float p = sc[u] == -INFINITY ? 0.f : expf(sc[u] - mb);
+                rs += p;
+                ps[r * (KT + 1) + c + 16 * u] = p;
+            }
 #pragma unroll
-        for (int o = 8; o > 0; o >>= 1) rs += __shfl_xor_sync(0xffffffffu, rs, o);
-        l = l * alpha + rs;
+            for (int o = 8; o > 0; o >>= 1) rs += __shfl_xor_sync(0xffffffffu, rs, o);
+            l = l * alpha + rs;
 #pragma unroll
-        for (int n = 0; n < 4; ++n)
+            for (int n = 0; n < 4; ++n)
 #pragma unroll
-            for (int j = 0; j < 4; ++j) acc[n][j] *= alpha;
+                for (int j = 0; j < 4; ++j) acc[n][j] *= alpha;
         }
         __syncwarp();                                                  // the 16 lanes of a row share a warp
         for (int kr = 0; kr < KT; ++kr) {
